@@ -1,0 +1,216 @@
+"""Plain, slow statements of the sequence mixers and of the decoder built from them, one function per mechanism, for the
+tests to compare the framework with.  Everything is float64 NumPy-style torch on the CPU, one token or one head at a time
+where that is clearest; nothing here is shared with the package."""
+import math
+
+import torch
+
+DT = torch.float64
+
+
+def silu(z):
+    return z / (1 + torch.exp(-z))
+
+
+def rms(x, eps):
+    """x divided by the root of its mean square over the last dimension."""
+    return x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps)
+
+
+def centred_norm(x, w, eps):
+    """RMS norm whose stored weight is the deviation from one."""
+    return rms(x, eps) * (1 + w)
+
+
+def swiglu(h, gate, up, down):
+    return (silu(h @ gate.T) * (h @ up.T)) @ down.T
+
+
+# ---------------------------------------------------------------------------------------------------- rotation
+def rope_angles(dims, base, scaling=None):
+    """Frequencies [dims / 2] and the factor on cos and sin."""
+    freqs = []
+    for i in range(dims // 2):
+        f = float(base) ** (-2.0 * i / dims)
+        if scaling:
+            def where(turns):
+                return dims * math.log(scaling["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
+            lo = max(math.floor(where(scaling["fast"])), 0)
+            hi = min(math.ceil(where(scaling["slow"])), dims - 1)
+            r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+            f = f / scaling["factor"] * r + f * (1 - r)
+        freqs.append(f)
+    return freqs, (0.1 * math.log(scaling["factor"]) + 1.0) if scaling else 1.0
+
+
+def rotate(x, pos, dims, base, scaling=None):
+    """x [dim] at one position; the first ``dims`` entries are rotated, entry i with entry i + dims / 2."""
+    freqs, m = rope_angles(dims, base, scaling)
+    y = x.clone()
+    for i, f in enumerate(freqs):
+        c, s = math.cos(pos * f) * m, math.sin(pos * f) * m
+        u, v = x[i], x[i + dims // 2]
+        y[i] = u * c - v * s
+        y[i + dims // 2] = v * c + u * s
+    return y
+
+
+def rotate_rows(x, pos0, dims, base, scaling=None):
+    """The same for x [T, n, dim] at positions pos0, pos0 + 1, ..."""
+    freqs, m = rope_angles(dims, base, scaling)
+    a = torch.arange(pos0, pos0 + x.shape[0], dtype=DT)[:, None] * torch.tensor(freqs, dtype=DT)[None]
+    c, s = (a.cos() * m)[:, None], (a.sin() * m)[:, None]
+    u, v = x[..., :dims // 2], x[..., dims // 2:dims]
+    return torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], -1)
+
+
+# ---------------------------------------------------------------------------------------------------- attention
+def visible(i, j, window=None):
+    return j <= i and (window is None or i - j < window)
+
+
+def attend_one(q, ks, vs, scale):
+    """Softmax attention of one query over the given keys / values."""
+    s = torch.stack([(q * k).sum() for k in ks]) * scale
+    w = torch.exp(s - s.max())
+    return (w[:, None] * torch.stack(list(vs))).sum(0) / w.sum()
+
+
+def attend(q, k, v, scale, window=None):
+    """q [T, dim] (the last T positions) over k [N, dim], v [N, vdim] with causality and an optional window."""
+    T, N = q.shape[0], k.shape[0]
+    i = torch.arange(N - T, N)[:, None]
+    j = torch.arange(N)[None]
+    ok = j <= i
+    if window is not None:
+        ok = ok & (i - j < window)
+    s = (q @ k.T) * scale
+    return torch.softmax(s.masked_fill(~ok, -math.inf), -1) @ v
+
+
+def diff_lambda(lq1, lk1, lq2, lk2, diff):
+    return float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum()) + diff)
+
+
+def diff_attend(q, k, v, heads, kv_heads, scale, lam, diff, eps, window=None):
+    """Differential attention.  q [T, heads, 2, dim] and k [N, kv_heads, 2, dim] are rotated already, v [N, kv_heads, vdim];
+    returns [T, heads, vdim]."""
+    out = []
+    for h in range(heads):
+        g = h // (heads // kv_heads)
+        a1 = attend(q[:, h, 0], k[:, g, 0], v[:, g], scale, window)
+        a2 = attend(q[:, h, 1], k[:, g, 1], v[:, g], scale, window)
+        out.append(rms(a1 - lam * a2, eps) * (1 - diff))
+    return torch.stack(out, 1)
+
+
+# ---------------------------------------------------------------------------------------------------- gated delta rule
+def short_conv(x, w, past=None):
+    """Causal convolution per channel: x [T, C], w [C, taps] (last column: the current token), ``past`` [taps - 1, C]
+    inputs before x (zeros at the start).  Returns (silu of the result, the last taps - 1 inputs)."""
+    taps = w.shape[1]
+    past = torch.zeros(taps - 1, x.shape[1], dtype=x.dtype) if past is None else past
+    full = torch.cat([past, x], 0)
+    y = torch.zeros_like(x)
+    for t in range(x.shape[0]):
+        for j in range(taps):
+            y[t] += w[:, j] * full[t + j]
+    return silu(y), full[full.shape[0] - (taps - 1):]
+
+
+def unit(x):
+    return x / torch.sqrt((x * x).sum(-1, keepdim=True) + 1e-6)
+
+
+def delta_scan(q, k, v, beta, g, state=None):
+    """Gated delta rule of one head: q, k [T, dim] (unit length, q scaled), v [T, vdim], beta, g [T].  State [dim, vdim]."""
+    S = torch.zeros(k.shape[1], v.shape[1], dtype=k.dtype) if state is None else state.clone()
+    out = []
+    for t in range(k.shape[0]):
+        S = g[t] * S
+        u = beta[t] * (v[t] - S.T @ k[t])
+        S = S + torch.outer(k[t], u)
+        out.append(S.T @ q[t])
+    return torch.stack(out), S
+
+
+# ---------------------------------------------------------------------------------------------------- the decoder
+class PlainLanedra:
+    """The whole decoder over a config dictionary and a dictionary of tensors; ``run`` takes the tokens of one sequence and
+    returns logits, and can be called again with more tokens (``state`` carries keys, values and recurrent state)."""
+
+    def __init__(self, cfg, tensors):
+        self.cfg = cfg
+        self.w = {n: t.to(DT) for n, t in tensors.items()}
+
+    def start(self):
+        return {"pos": 0, "layers": [{} for _ in self.cfg["layers"]]}
+
+    def attention(self, i, h, st, pos):
+        c, w, p = self.cfg["layers"][i]["mixer"], self.w, f"l{i}.mix."
+        H, G, D, V = c["heads"], c["kv_heads"], c["dim"], c["vdim"]
+        T = h.shape[0]
+        rot = (c["rot"]["dims"], c["rot"]["base"], c["rot"].get("scaling"))
+        q = rotate_rows((h @ w[p + "q"].T).view(T, 2 * H, D), pos, *rot).view(T, H, 2, D)
+        src = c.get("kv_from")
+        if src is None:
+            k = rotate_rows((h @ w[p + "k"].T).view(T, 2 * G, D), pos, *rot).view(T, G, 2, D)
+            v = (h @ w[p + "v"].T).view(T, G, V)
+            mine = st["layers"][i]
+            mine["k"] = torch.cat([mine["k"], k]) if "k" in mine else k
+            mine["v"] = torch.cat([mine["v"], v]) if "v" in mine else v
+        else:
+            mine = st["layers"][src]
+        lam = diff_lambda(w[p + "lq1"], w[p + "lk1"], w[p + "lq2"], w[p + "lk2"], c["diff"])
+        o = diff_attend(q, mine["k"], mine["v"], H, G, c["scale"], lam, c["diff"], self.cfg["norm"]["eps"],
+                        c["mask"]["size"] if c.get("mask") else None)
+        return o.reshape(T, H * V) @ w[p + "o"].T
+
+    def delta(self, i, h, st):
+        c, w, p = self.cfg["layers"][i]["mixer"], self.w, f"l{i}.mix."
+        H, G, D, V = c["heads"], c["kv_heads"], c["dim"], c["vdim"]
+        T, mine = h.shape[0], st["layers"][i]
+        x = {}
+        for n in "qkv":
+            x[n], mine["conv_" + n] = short_conv(h @ w[p + n].T, w[p + n + ".conv"], mine.get("conv_" + n))
+        q = unit(x["q"].view(T, G, D)) * D ** -0.5
+        k = unit(x["k"].view(T, G, D))
+        v = x["v"].view(T, H, V)
+        beta = 1 / (1 + torch.exp(-(h @ w[p + "b"].T)))
+        z = h @ w[p + "a"].T + w[p + "dt_bias"]
+        g = torch.exp(-torch.exp(w[p + "A_log"]) * torch.log1p(torch.exp(z)))
+        outs, states = [], []
+        for hd in range(H):
+            gr = hd // (H // G)
+            o, S = delta_scan(q[:, gr], k[:, gr], v[:, hd], beta[:, hd], g[:, hd], mine["S"][hd] if "S" in mine else None)
+            outs.append(o)
+            states.append(S)
+        mine["S"] = states
+        o = rms(torch.stack(outs, 1), self.cfg["norm"]["eps"]) * w[p + "norm"] * silu(h @ w[p + "g"].T).view(T, H, V)
+        return o.reshape(T, H * V) @ w[p + "o"].T
+
+    def run(self, tokens, st=None, residuals=None):
+        cfg, w, eps = self.cfg, self.w, self.cfg["norm"]["eps"]
+        st = st if st is not None else self.start()
+        x = w["embed"][torch.tensor(tokens)] * cfg["embedding"]["scale"]
+        for i, layer in enumerate(cfg["layers"]):
+            p = f"l{i}."
+            h = centred_norm(x, w[p + "norm1"], eps)
+            y = self.attention(i, h, st, st["pos"]) if layer["type"] == "attention" else self.delta(i, h, st)
+            x = x + centred_norm(y, w[p + "norm1b"], eps)
+            if layer["mlp"] is not None:
+                h = centred_norm(x, w[p + "norm2"], eps)
+                y = swiglu(h, w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"])
+                x = x + centred_norm(y, w[p + "norm2b"], eps)
+            if residuals is not None:
+                residuals.append(x.clone())
+        st["pos"] += len(tokens)
+        return centred_norm(x, w["final.norm"], eps) @ w["head"].T
+
+    def greedy(self, tokens, n):
+        st, out = self.start(), []
+        lg = self.run(tokens, st)
+        for _ in range(n):
+            out.append(int(lg[-1].argmax()))
+            lg = self.run([out[-1]], st)
+        return out

@@ -28,6 +28,9 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
     "--expt-relaxed-constexpr",
 ]
+# Translation units whose fp32 arithmetic has to be fp32 to the last bits (they serve the 32-bit mode of a model as well):
+# compiled without --use_fast_math.
+PRECISE = {"stack_ops", "delta_rule", "diff_attention"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-Wall", "-Wno-unused-function"]
 
 
@@ -59,13 +62,23 @@ def _compile_many(jobs, workers):
                 print(out)
 
 
-def build_kernels(force=False, verbose=False, bounds_check=False) -> Path:
+def _flags(stem: str):
+    return [f for f in NVCC_FLAGS if f != "--use_fast_math"] if stem in PRECISE else NVCC_FLAGS
+
+
+def build_kernels(force=False, verbose=False, bounds_check=False, units=None, name="tfb_kernels") -> Path:
     """All .cu files under csrc/kernels and csrc/comm -> lib/libtfb_kernels.so.  ``bounds_check`` builds the variant
-    with -DTFB_BOUNDS_CHECK into lib/libtfb_kernels_check.so (loaded when the environment has TFB_BOUNDS_CHECK=1)."""
+    with -DTFB_BOUNDS_CHECK into lib/libtfb_kernels_check.so (loaded when the environment has TFB_BOUNDS_CHECK=1).
+    ``units`` (file stems) restricts the library, then called lib<name>.so, to those translation units."""
     nvcc = _nvcc()
     OBJ.mkdir(parents=True, exist_ok=True)
     suffix, extra = ("_check", ["-DTFB_BOUNDS_CHECK"]) if bounds_check else ("", [])
     srcs = sorted((CSRC / "kernels").glob("*.cu")) + sorted((CSRC / "comm").glob("*.cu"))
+    if units is not None:
+        srcs = [s for s in srcs if s.stem in set(units)]
+        missing = set(units) - {s.stem for s in srcs}
+        if missing:
+            raise RuntimeError(f"no such kernel sources: {sorted(missing)}")
     hdrs = list((CSRC / "kernels").glob("*.cuh")) + list((CSRC / "kernels").glob("*.h")) + \
         list((CSRC / "comm").glob("*.cuh")) + list((CSRC / "comm").glob("*.h"))
     jobs, objs = [], []
@@ -73,13 +86,13 @@ def build_kernels(force=False, verbose=False, bounds_check=False) -> Path:
         o = OBJ / (s.stem + suffix + ".o")
         objs.append(o)
         if force or _newer([s] + hdrs, o):
-            cmd = [nvcc] + NVCC_FLAGS + extra + ["-I", str(CSRC / "kernels"), "-I", str(CSRC / "comm"), "-c", str(s), "-o", str(o)]
+            cmd = [nvcc] + _flags(s.stem) + extra + ["-I", str(CSRC / "kernels"), "-I", str(CSRC / "comm"), "-c", str(s), "-o", str(o)]
             if verbose:
                 cmd += ["-Xptxas", "-v"]
             jobs.append(cmd)
     _compile_many(jobs, workers=min(8, os.cpu_count() or 4))
-    so = LIB / f"libtfb_kernels{suffix}.so"
-    if force or jobs or not so.exists():
+    so = LIB / f"lib{name}{suffix}.so"
+    if force or jobs or _newer(objs, so):
         _run([nvcc, "-shared", "-o", str(so)] + [str(o) for o in objs] + ["-cudart", "static"])
     return so
 

@@ -11,11 +11,11 @@ class Handle:
 
         from .cli.common import load_tokenizer, model_dtype, pick_device
         from .inference.engine import EngineConfig, InferenceEngine
-        from .quant import codec
+        from .models import registry
         if not os.path.exists(path):
             raise FileNotFoundError(path)
         dev = pick_device(os.environ.get("TFB_DEVICE", "auto"))
-        self.model = codec.load_model(path, device=dev, dtype=model_dtype(dev))
+        self.model = registry.load_any(path, device=dev, dtype=model_dtype(dev))
         self.tok = load_tokenizer(path)
         self.engine = InferenceEngine(self.model, self.tok, EngineConfig(num_pages=max(64, 4 * self.model.cfg.max_seq_len // 16)))
 

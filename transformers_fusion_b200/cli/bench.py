@@ -361,10 +361,10 @@ def main(argv=None):
     if a.inference:
         from ..inference.engine import EngineConfig, InferenceEngine
         from ..inference.sampler import SamplerConfig
-        from ..quant import codec
+        from ..models import registry
         from .common import load_tokenizer, model_dtype, pick_device
         dev = pick_device()
-        model = codec.load_model(a.model, device=dev, dtype=model_dtype(dev))
+        model = registry.load_any(a.model, device=dev, dtype=model_dtype(dev))
         eng = InferenceEngine(model, load_tokenizer(a.model), EngineConfig(num_pages=1024))
         t0 = time.perf_counter()
         text, st = eng.generate_with_stats(a.prompt, min(64, model.cfg.max_seq_len - 8), SamplerConfig(0.0))

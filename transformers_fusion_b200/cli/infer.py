@@ -1,4 +1,4 @@
-"""quant_infer: ``<model.quant> [prompt] [--model-dir DIR] [--seed N]``; temperature .7, top_k 40, top_p .9,
+"""quant_infer: ``<model.quant | model folder> [prompt] [--model-dir DIR] [--seed N]``; temperature .7, top_k 40, top_p .9,
 max 512 tokens; prints the completion and tok/s (tools/infer.cpp:15-108)."""
 from __future__ import annotations
 
@@ -23,11 +23,11 @@ def main(argv=None):
     a = ap.parse_args(argv)
     from ..inference.engine import EngineConfig, InferenceEngine
     from ..inference.sampler import SamplerConfig
-    from ..quant import codec
+    from ..models import registry
     dev = pick_device(a.device)
     try:
-        model = codec.load_model(a.model, device=dev, dtype=model_dtype(dev))
-    except (ValueError, OSError) as e:
+        model = registry.load_any(a.model, device=dev, dtype=model_dtype(dev))
+    except (ValueError, KeyError, OSError) as e:
         print(f"Error: {e}", file=sys.stderr)
         return 1
     tok = load_tokenizer(a.model, a.model_dir)

@@ -1,14 +1,48 @@
-"""quant_info <model.quant>: header, tensor list with formats, parameter total (tools/info.cpp:10-70)."""
+"""quant_info <model.quant | model folder>: header, tensor list with formats, parameter total (tools/info.cpp:10-70)."""
 from __future__ import annotations
 
 import sys
 
 
+def _folder_info(path):
+    """Model folder: architecture, sizes, layer list, tensors."""
+    from ..models import registry
+    from ..quant.importers import _sources
+    try:
+        _, c = registry.read_config(path)
+        srcs = list(_sources(path))
+    except (ValueError, KeyError, OSError) as e:
+        print(f"Error: {e}", file=sys.stderr)
+        return 1
+    print(f"Model folder: {path}")
+    print(f"Architecture: {c.architecture}")
+    print(f"Config: vocab={c.vocab_size} hidden={c.hidden_size} layers={c.num_layers}")
+    for i, l in enumerate(c.layers):
+        m = l.mixer
+        extra = "" if m.kind != "attention" else (f" window={m.window}" if m.window else "") + (f" kv_from={m.kv_from}" if m.kv_from is not None else "")
+        print(f"  layer {i}: {m.kind} heads={m.heads} kv_heads={m.kv_heads} dim={m.dim} vdim={m.vdim}{extra} ffn={l.ffn_hidden_size or 'none'}")
+    total = 0
+    for s in srcs:
+        for n in s.names:
+            shape = s.shape(n)
+            numel = 1
+            for d in shape:
+                numel *= d
+            total += numel
+            print(f"  {n} {list(shape)} {s.dtype(n)}")
+        s.close()
+    print(f"Total parameters: {total}")
+    return 0
+
+
 def main(argv=None):
     argv = sys.argv[1:] if argv is None else argv
     if len(argv) != 1 or argv[0] in ("-h", "--help"):
-        print("Usage: quant_info <model.quant>")
+        print("Usage: quant_info <model.quant | model folder>")
         return 0 if argv else 1
+    from ..models import registry
+    if registry.is_folder(argv[0]):
+        return _folder_info(argv[0])
     from ..quant import codec
     try:
         r = codec.QuantReader(argv[0])

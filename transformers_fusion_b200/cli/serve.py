@@ -1,5 +1,5 @@
 """quant_serve / quant_server: OpenAI-compatible HTTP server over the native front end and the
-continuous-batching engine.  ``--model --port(8080) --batch-size --workers(4) --max-tokens`` (tools/serve.cpp:18-148)
+continuous-batching engine.  ``--model`` takes a ``.quant`` container or a model folder.  ``--model --port(8080) --batch-size --workers(4) --max-tokens`` (tools/serve.cpp:18-148)
 plus ``--model-dir --temperature --top-k --top-p`` (tools/quant_server.cpp:50-80) and ``--kv --auth-token``."""
 from __future__ import annotations
 
@@ -103,11 +103,11 @@ def main(argv=None):
     ap.add_argument("--device", default="auto")
     a = ap.parse_args(argv)
     from ..inference.engine import EngineConfig, InferenceEngine
-    from ..quant import codec
+    from ..models import registry
     from ..server import HTTPServer
     dev = pick_device(a.device)
     def build_engine(path):
-        model = codec.load_model(path, device=dev, dtype=model_dtype(dev))
+        model = registry.load_any(path, device=dev, dtype=model_dtype(dev))
         tok = load_tokenizer(path, a.model_dir)
         return InferenceEngine(model, tok, EngineConfig(max_batch=a.batch_size, kv_mode=a.kv, num_pages=4096, weight_format=a.weights))
     eng = build_engine(a.model)

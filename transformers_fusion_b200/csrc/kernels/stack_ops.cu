@@ -1,0 +1,358 @@
+// Row operators of decoders with a 32-bit residual stream and a norm before and after every sublayer: scaled embedding,
+// post-norm + residual + next pre-norm in one pass, gated activation, partial rotary embedding fused with the append to
+// the paged cache, gather of cached rows, and a true fp32 matrix product.  Every kernel exists for bf16 and for fp32
+// activations; the statistics, the residual and the rotation are fp32 in both.
+#include "tfb_elem.cuh"
+#include "tfb_host.h"
+
+namespace tfb {
+TFB_BOUNDS_DEFINE(stack_ops)
+
+// ------------------------------------------------------------------------------------------------
+// x <- x + norm(y) * (1 + w_post);  a = norm(x) * (1 + w_pre)      (norm: division by the root of the mean square)
+// ids != null: x starts as scale * table[id] instead of being read.  rows != null: output row i is computed from row
+// rows[i] of x and y, and x is left alone (the last norm of a step, for the positions whose logits are wanted).
+// One block per row; the row lives in registers between the two statistics.
+// ------------------------------------------------------------------------------------------------
+struct ResNormArgs {
+  const long long* ids;
+  const void* table;
+  long long ld_table;
+  float scale;
+  int vocab;
+  float* x;
+  long long ldx;
+  const void* y;
+  long long ldy;
+  const void *w_post, *w_pre;
+  void* a;
+  long long lda;
+  const int* rows;
+  int H;
+  float eps;
+};
+
+template <class T, int VEC, int NV>
+__global__ void res_norm_kernel(const ResNormArgs p) {
+  tfb::pdl_sync();
+  __shared__ float red[32];
+  const int i = blockIdx.x, nt = blockDim.x;
+  const long long r = p.rows ? p.rows[i] : i;
+  float v[NV][VEC];
+  const T* trow = nullptr;
+  if (p.ids) {
+    long long id = p.ids[r];
+    TFB_BOUNDS(id >= 0 && id < p.vocab, 1, id, p.vocab);
+    id = id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id);
+    trow = static_cast<const T*>(p.table) + id * p.ld_table;
+  }
+#pragma unroll
+  for (int c = 0; c < NV; ++c) {
+    const int col = (c * nt + threadIdx.x) * VEC;
+    if (col >= p.H) continue;
+    if (trow) {
+      load_n<VEC>(trow + col, v[c]);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[c][e] *= p.scale;
+    } else {
+      load_n<VEC>(p.x + r * p.ldx + col, v[c]);
+    }
+  }
+  if (p.y) {
+    float yv[NV][VEC];
+    float ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+      const int col = (c * nt + threadIdx.x) * VEC;
+      if (col >= p.H) continue;
+      load_n<VEC>(static_cast<const T*>(p.y) + r * p.ldy + col, yv[c]);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss = fmaf(yv[c][e], yv[c][e], ss);
+    }
+    const float rs = 1.f / sqrtf(block_add(ss, red) / p.H + p.eps);
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+      const int col = (c * nt + threadIdx.x) * VEC;
+      if (col >= p.H) continue;
+      float w[VEC];
+      load_n<VEC>(static_cast<const T*>(p.w_post) + col, w);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[c][e] += yv[c][e] * rs * (1.f + w[e]);
+    }
+  }
+  if (!p.rows && (p.y || p.ids)) {
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+      const int col = (c * nt + threadIdx.x) * VEC;
+      if (col < p.H) store_n<VEC>(p.x + r * p.ldx + col, v[c]);
+    }
+  }
+  if (!p.a) return;
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < NV; ++c) {
+    const int col = (c * nt + threadIdx.x) * VEC;
+    if (col >= p.H) continue;
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(v[c][e], v[c][e], ss);
+  }
+  const float rs = 1.f / sqrtf(block_add(ss, red) / p.H + p.eps);
+#pragma unroll
+  for (int c = 0; c < NV; ++c) {
+    const int col = (c * nt + threadIdx.x) * VEC;
+    if (col >= p.H) continue;
+    float w[VEC], o[VEC];
+    load_n<VEC>(static_cast<const T*>(p.w_pre) + col, w);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) o[e] = v[c][e] * rs * (1.f + w[e]);
+    store_n<VEC>(static_cast<T*>(p.a) + (long long)i * p.lda + col, o);
+  }
+}
+
+template <class T, int VEC>
+static int launch_res_norm(const ResNormArgs& p, int n, cudaStream_t st) {
+  const int items = (p.H + VEC - 1) / VEC;
+  int nt = (items + 31) / 32 * 32;
+  const int cap = VEC == 1 ? 512 : 256;
+  if (nt > cap) nt = cap;
+  const int nv = (items + nt - 1) / nt;
+  if (nv <= 1) launch_k(res_norm_kernel<T, VEC, 1>, n, nt, 0, st, p);
+  else if (nv <= 2) launch_k(res_norm_kernel<T, VEC, 2>, n, nt, 0, st, p);
+  else if (nv <= 4) launch_k(res_norm_kernel<T, VEC, 4>, n, nt, 0, st, p);
+  else if (nv <= 8) launch_k(res_norm_kernel<T, VEC, 8>, n, nt, 0, st, p);
+  else return TFB_ERR_LIMIT;
+  return int(cudaGetLastError());
+}
+
+// ------------------------------------------------------------------------------------------------
+// [gate | up] -> silu(gate) * up
+// ------------------------------------------------------------------------------------------------
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) glu_silu_kernel(const T* __restrict__ in, long long ldi, T* __restrict__ out, long long ldo, int M, int F) {
+  tfb::pdl_sync();
+  const int per = F / VEC;
+  const long long n = (long long)M * per;
+  for (long long t = blockIdx.x * (long long)blockDim.x + threadIdx.x; t < n; t += (long long)gridDim.x * blockDim.x) {
+    const long long m = t / per;
+    const int c = int(t % per) * VEC;
+    float g[VEC], u[VEC];
+    load_n<VEC>(in + m * ldi + c, g);
+    load_n<VEC>(in + m * ldi + F + c, u);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) g[e] = silu_exact(g[e]) * u[e];
+    store_n<VEC>(out + m * ldo + c, g);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// Rotary embedding of the first `dims` entries of every q and k head, in place, and append of k and v to the paged pools.
+// Rows: [nq heads of D | nk heads of D | v_cols].  Pools are [slots][nk * D] and [slots][v_cols]; a negative slot (padding,
+// or a position no later query can see) is not cached.  nk = 0: the layer has queries only.
+// ------------------------------------------------------------------------------------------------
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) rope_append_kernel(T* __restrict__ qkv, long long ld, const float* __restrict__ cos_t,
+                                                          const float* __restrict__ sin_t, int max_pos, const int* __restrict__ positions,
+                                                          const long long* __restrict__ slots, T* __restrict__ kpool,
+                                                          T* __restrict__ vpool, long long nslots, int rows, int nq, int nk, int D,
+                                                          int dims, int v_cols) {
+  tfb::pdl_sync();
+  const int half = dims >> 1, hv = half / VEC, pv = (D - dims) / VEC, vv = v_cols / VEC;
+  const int per_rot = (nq + nk) * hv, per_pass = nk * pv;
+  const int per = per_rot + per_pass + vv;          // work items of one row: rotated pairs, k entries that pass, v entries
+  const long long n = (long long)rows * per;
+  for (long long t = blockIdx.x * (long long)blockDim.x + threadIdx.x; t < n; t += (long long)gridDim.x * blockDim.x) {
+    const long long r = t / per;
+    int w = int(t % per);
+    T* row = qkv + r * ld;
+    long long slot = (slots && nk) ? slots[r] : -1;
+    TFB_BOUNDS(slot < nslots, 51, slot, nslots);
+    if (slot >= nslots) slot = -1;
+    if (w < per_rot) {
+      int pos = positions[r];
+      TFB_BOUNDS(pos >= 0 && pos < max_pos, 61, pos, max_pos);
+      pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
+      const int head = w / hv, i = (w % hv) * VEC;
+      float u[VEC], v[VEC], c[VEC], s[VEC], a[VEC], b[VEC];
+      load_n<VEC>(row + head * D + i, u);
+      load_n<VEC>(row + head * D + half + i, v);
+      load_n<VEC>(cos_t + (long long)pos * half + i, c);
+      load_n<VEC>(sin_t + (long long)pos * half + i, s);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        a[e] = u[e] * c[e] - v[e] * s[e];
+        b[e] = v[e] * c[e] + u[e] * s[e];
+      }
+      store_n<VEC>(row + head * D + i, a);
+      store_n<VEC>(row + head * D + half + i, b);
+      if (head >= nq && slot >= 0) {
+        T* kp = kpool + (slot * nk + (head - nq)) * D;
+        store_n<VEC>(kp + i, a);
+        store_n<VEC>(kp + half + i, b);
+      }
+    } else if (slot >= 0) {
+      w -= per_rot;
+      float u[VEC];
+      if (w < per_pass) {
+        const int head = w / pv, i = dims + (w % pv) * VEC;
+        load_n<VEC>(row + (nq + head) * D + i, u);
+        store_n<VEC>(kpool + (slot * nk + head) * D + i, u);
+      } else {
+        const int i = (w - per_pass) * VEC;
+        load_n<VEC>(row + (long long)(nq + nk) * D + i, u);
+        store_n<VEC>(vpool + slot * v_cols + i, u);
+      }
+    }
+  }
+}
+
+// rows lo .. lo + n - 1 of one sequence (its page list) out of a pool [slots][width], contiguous
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) gather_rows_kernel(const T* __restrict__ pool, long long nslots, const int* __restrict__ pages,
+                                                          int page, int lo, int n, T* __restrict__ out, int width) {
+  tfb::pdl_sync();
+  const int per = width / VEC;
+  const long long total = (long long)n * per;
+  for (long long t = blockIdx.x * (long long)blockDim.x + threadIdx.x; t < total; t += (long long)gridDim.x * blockDim.x) {
+    const int r = int(t / per), c = int(t % per) * VEC, pos = lo + r;
+    const long long slot = (long long)pages[pos / page] * page + pos % page;
+    TFB_BOUNDS(slot >= 0 && slot < nslots, 53, slot, nslots);
+    float u[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) u[e] = 0.f;
+    if (slot >= 0 && slot < nslots) load_n<VEC>(pool + slot * width + c, u);
+    store_n<VEC>(out + (long long)r * width + c, u);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// C[M, N] = A[M, K] . B[N, K]^T in true fp32 (FFMA), 64 x 64 tiles, any sizes and pitches
+// ------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, long long lda, const float* __restrict__ B, long long ldb,
+                                                       float* __restrict__ C, long long ldc, int M, int N, int K) {
+  tfb::pdl_sync();
+  __shared__ float sA[16][68], sB[16][68];
+  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, tid = threadIdx.x;
+  const int ty = tid >> 4, tx = tid & 15;
+  float acc[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  for (int k0 = 0; k0 < K; k0 += 16) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int e = tid + 256 * i, r = e >> 4, k = e & 15;
+      sA[k][r] = (m0 + r < M && k0 + k < K) ? A[(long long)(m0 + r) * lda + k0 + k] : 0.f;
+      sB[k][r] = (n0 + r < N && k0 + k < K) ? B[(long long)(n0 + r) * ldb + k0 + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k) {
+      const float4 a = *reinterpret_cast<const float4*>(&sA[k][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&sB[k][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+      if (m < M && n < N) C[(long long)m * ldc + n] = acc[i][j];
+    }
+}
+
+static bool aligned(const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
+static int grid_for(long long items) {
+  const long long b = (items + 255) / 256, cap = 148ll * 16;
+  return int(b < 1 ? 1 : (b < cap ? b : cap));
+}
+
+}  // namespace tfb
+
+using bf16 = __nv_bfloat16;
+
+// f32 = 1: activations, table and norm weights are fp32, otherwise bf16.  See ResNormArgs.
+TFB_API int tfb_res_norm(const long long* ids, const void* table, long long ld_table, float scale, int vocab, float* x, long long ldx,
+                         const void* y, long long ldy, const void* w_post, const void* w_pre, void* a, long long lda, const int* rows,
+                         int n, int H, float eps, int f32, void* stream) {
+  using namespace tfb;
+  if (n <= 0 || H <= 0 || (y && !w_post) || (a && !w_pre) || (ids && !table)) return TFB_ERR_ARG;
+  ResNormArgs p{ids, table, ld_table, scale, vocab, x, ldx, y, ldy, w_post, w_pre, a, lda, rows, H, eps};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int es = f32 ? 4 : 2;
+  auto ok = [&](int vec) {
+    return H % vec == 0 && ldx % vec == 0 && aligned(x, 16) && (!y || (ldy % vec == 0 && aligned(y, vec * es))) &&
+           (!a || (lda % vec == 0 && aligned(a, vec * es))) && (!ids || (ld_table % vec == 0 && aligned(table, vec * es))) &&
+           (!w_post || aligned(w_post, vec * es)) && (!w_pre || aligned(w_pre, vec * es));
+  };
+  if (f32) return ok(4) ? launch_res_norm<float, 4>(p, n, st) : launch_res_norm<float, 1>(p, n, st);
+  if (ok(8)) return launch_res_norm<bf16, 8>(p, n, st);
+  return ok(4) ? launch_res_norm<bf16, 4>(p, n, st) : launch_res_norm<bf16, 1>(p, n, st);
+}
+
+TFB_API int tfb_glu_silu(const void* in, long long ldi, void* out, long long ldo, int M, int F, int f32, void* stream) {
+  using namespace tfb;
+  if (M <= 0 || F <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int vec = f32 ? 4 : 8;
+  const bool v = F % vec == 0 && ldi % vec == 0 && ldo % vec == 0 && aligned(in, 16) && aligned(out, 16);
+  const int grid = grid_for((long long)M * (v ? F / vec : F));
+  if (f32) {
+    if (v) launch_k(glu_silu_kernel<float, 4>, grid, 256, 0, st, static_cast<const float*>(in), ldi, static_cast<float*>(out), ldo, M, F);
+    else launch_k(glu_silu_kernel<float, 1>, grid, 256, 0, st, static_cast<const float*>(in), ldi, static_cast<float*>(out), ldo, M, F);
+  } else {
+    if (v) launch_k(glu_silu_kernel<bf16, 8>, grid, 256, 0, st, static_cast<const bf16*>(in), ldi, static_cast<bf16*>(out), ldo, M, F);
+    else launch_k(glu_silu_kernel<bf16, 1>, grid, 256, 0, st, static_cast<const bf16*>(in), ldi, static_cast<bf16*>(out), ldo, M, F);
+  }
+  return int(cudaGetLastError());
+}
+
+TFB_API int tfb_rope_append(void* qkv, long long ld, const float* cos_t, const float* sin_t, int max_pos, const int* positions,
+                            const long long* slots, void* kpool, void* vpool, long long nslots, int rows, int nq, int nk, int D, int dims,
+                            int v_cols, int f32, void* stream) {
+  using namespace tfb;
+  if (rows <= 0 || nq <= 0 || nk < 0 || dims <= 0 || (dims & 1) || dims > D) return TFB_ERR_ARG;
+  if (nk == 0) v_cols = 0;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int vec = f32 ? 4 : 8;
+  const bool v = (dims / 2) % vec == 0 && D % vec == 0 && v_cols % vec == 0 && ld % vec == 0 && aligned(qkv, 16) &&
+                 (!kpool || (aligned(kpool, 16) && aligned(vpool, 16)));
+  const int q = v ? vec : 1;
+  const int grid = grid_for((long long)rows * ((nq + nk) * (dims / 2 / q) + nk * ((D - dims) / q) + v_cols / q));
+#define TFB_RA(T, VEC) launch_k(rope_append_kernel<T, VEC>, grid, 256, 0, st, static_cast<T*>(qkv), ld, cos_t, sin_t, max_pos, positions, \
+                                slots, static_cast<T*>(kpool), static_cast<T*>(vpool), nslots, rows, nq, nk, D, dims, v_cols)
+  if (f32) { if (v) TFB_RA(float, 4); else TFB_RA(float, 1); }
+  else { if (v) TFB_RA(bf16, 8); else TFB_RA(bf16, 1); }
+#undef TFB_RA
+  return int(cudaGetLastError());
+}
+
+TFB_API int tfb_gather_rows(const void* pool, long long nslots, const int* pages, int page, int lo, int n, void* out, int width, int f32,
+                            void* stream) {
+  using namespace tfb;
+  if (n <= 0 || width <= 0 || lo < 0 || page <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int vec = f32 ? 4 : 8;
+  const bool v = width % vec == 0 && aligned(pool, 16) && aligned(out, 16);
+  const int grid = grid_for((long long)n * (v ? width / vec : width));
+#define TFB_GR(T, VEC) launch_k(gather_rows_kernel<T, VEC>, grid, 256, 0, st, static_cast<const T*>(pool), nslots, pages, page, lo, n, \
+                                static_cast<T*>(out), width)
+  if (f32) { if (v) TFB_GR(float, 4); else TFB_GR(float, 1); }
+  else { if (v) TFB_GR(bf16, 8); else TFB_GR(bf16, 1); }
+#undef TFB_GR
+  return int(cudaGetLastError());
+}
+
+TFB_API int tfb_gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N, int K,
+                         void* stream) {
+  using namespace tfb;
+  if (M <= 0 || N <= 0 || K <= 0 || (M + 63) / 64 > 65535) return TFB_ERR_ARG;
+  launch_k(gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64), 256, 0, static_cast<cudaStream_t>(stream), A, lda, B, ldb, C, ldc, M, N, K);
+  return int(cudaGetLastError());
+}

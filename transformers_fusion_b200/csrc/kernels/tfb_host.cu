@@ -60,6 +60,22 @@ int make_tmap_3d(CUtensorMap* out, const void* base, int elem_bytes, uint64_t d0
   return r == CUDA_SUCCESS ? TFB_OK : TFB_ERR_DRIVER;
 }
 
+int make_tmap_4d(CUtensorMap* out, const void* base, int elem_bytes, const uint64_t (&dims)[4], const uint64_t (&strides_bytes)[3],
+                 const uint32_t (&box)[4], int swizzle128) {
+  std::call_once(g_encode_once, load_encode);
+  if (!g_encode) return TFB_ERR_DRIVER;
+  if ((reinterpret_cast<uintptr_t>(base) & 15) || (strides_bytes[0] & 15) || (strides_bytes[1] & 15) || (strides_bytes[2] & 15))
+    return TFB_ERR_ARG;
+  cuuint64_t d[4], s[3];
+  cuuint32_t b[4], estr[4] = {1, 1, 1, 1};
+  for (int i = 0; i < 4; ++i) { d[i] = dims[i]; b[i] = box[i]; }
+  for (int i = 0; i < 3; ++i) s[i] = strides_bytes[i];
+  CUresult r = g_encode(out, dtype_of(elem_bytes), 4, const_cast<void*>(base), d, s, b, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                        swizzle128 ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_NONE,
+                        CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? TFB_OK : TFB_ERR_DRIVER;
+}
+
 int pdl_enabled() {
   static const int on = [] {
     const char* e = getenv("TFB_PDL");

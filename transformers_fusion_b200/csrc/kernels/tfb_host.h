@@ -28,6 +28,11 @@ int make_tmap_2d(CUtensorMap* out, const void* base, int elem_bytes, uint64_t in
 int make_tmap_3d(CUtensorMap* out, const void* base, int elem_bytes, uint64_t d0, uint64_t d1, uint64_t d2,
                  uint64_t s1_bytes, uint64_t s2_bytes, uint32_t b0, uint32_t b1, uint32_t b2, int swizzle128 = 1);
 
+// 4-D variant with byte strides for the three outer dimensions.  A box may be larger than the tensor in any dimension (zero
+// fill), which is how heads of fewer than 64 entries become 64-column tiles.
+int make_tmap_4d(CUtensorMap* out, const void* base, int elem_bytes, const uint64_t (&dims)[4], const uint64_t (&strides_bytes)[3],
+                 const uint32_t (&box)[4], int swizzle128 = 1);
+
 int sm_count();
 
 // 1 when the environment has TFB_PDL=1 (read once): whether launches allow programmatic stream serialization.  Off by

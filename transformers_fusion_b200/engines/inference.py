@@ -59,17 +59,17 @@ class InferenceEngine:
 
     # ---------------------------------------------------------------- set-up
     def load(self, quant_path: str, device: Optional[str] = None) -> Tuple[bool, str]:
-        """Loads ``model.quant`` and the vocabulary beside it (``model.vocab`` or ``model.quant.vocab``)."""
+        """Loads ``model.quant`` (or a model folder) and the vocabulary beside it (``model.vocab`` or ``model.quant.vocab``)."""
         import torch
         from ..cli.common import load_tokenizer
-        from ..quant.codec import load_model
+        from ..models.registry import load_any
         if not os.path.exists(quant_path):
             return False, f"no such file: {quant_path}"
         try:
             dev = device or ("cuda" if torch.cuda.is_available() else "cpu")
-            model = load_model(quant_path, device=dev)
+            model = load_any(quant_path, device=dev)
             tok = load_tokenizer(quant_path, os.path.dirname(quant_path) or ".")
-        except (OSError, ValueError, RuntimeError) as e:
+        except (OSError, ValueError, KeyError, RuntimeError) as e:
             return False, str(e)
         self.init(model, tok, self._cfg)
         return True, ""

@@ -10,6 +10,10 @@ Finished sequences release their pages; a prefix cache lets requests that share 
 pages) reuse the pages instead of recomputing them, and the rest of such a prompt attends over the
 cached pages through a gather + the tensor-core attention kernel.
 
+Models that bring their own pass over the layers (``run``, models/stack.py) are driven by the same scheduler: the engine
+builds the batch description of a prompt, of a portion of one, or of a decode step, and the model's cache
+(``mixer_cache``) holds paged keys and values for the attention layers and a slot of recurrent state per sequence.
+
 Reference counterparts: ContinuousBatching / RequestScheduler (priority desc, deadline asc) /
 PrefixCache / PagedAttention (src/inference/inference_paging.cpp:24-285, inference_kv.cpp:20-205),
 Generator / StreamingGenerator events START / TOKEN / COMPLETE / STOP (src/inference/generator.cpp),
@@ -63,7 +67,9 @@ class Request:
     on_token: Optional[Callable[[int], None]] = None
     # runtime state
     out: List[int] = field(default_factory=list)
-    pages: List[int] = field(default_factory=list)
+    pages: List[int] = field(default_factory=list)   # -1: a page that has left every layer's window
+    first_page: int = 0            # pages below this one have been given back
+    state_slot: int = -1           # recurrent state (models that have some)
     pos: int = 0
     t_submit: float = 0.0
     t_first: float = 0.0
@@ -176,7 +182,8 @@ class _DecodeGraph:
         self.positions = torch.zeros(bucket, dtype=torch.int32, device=dev)
         self.bt = torch.zeros((bucket, eng.max_pages), dtype=torch.int32, device=dev)
         self.slots = torch.full((bucket,), -1, dtype=torch.int64, device=dev)
-        run = lambda: eng._logits(eng._layers_decode(self.tokens, self.positions, self.bt, self.slots))
+        self.state_slots = torch.full((bucket,), -1, dtype=torch.int32, device=dev)
+        run = lambda: eng._logits(eng._layers_decode(self.tokens, self.positions, self.bt, self.slots, self.state_slots))
         side = torch.cuda.Stream(device=dev)
         side.wait_stream(torch.cuda.current_stream(dev))
         with torch.cuda.stream(side):                  # warm-up outside capture: workspaces, status words, lazy tables
@@ -195,15 +202,17 @@ class _DecodeGraph:
             self.logits = run()
             eng._graph_capture_end(self.token)
 
-    def replay(self, tokens, positions, bt, slots):
+    def replay(self, tokens, positions, bt, slots, state_slots):
         n = tokens.shape[0]
         self.tokens[:n].copy_(tokens, non_blocking=True)
         self.positions[:n].copy_(positions, non_blocking=True)
         self.bt[:n].copy_(bt, non_blocking=True)
         self.slots[:n].copy_(slots, non_blocking=True)
+        self.state_slots[:n].copy_(state_slots, non_blocking=True)
         if n < self.bucket and n != self._last_n:      # rows past the live batch: reset once per batch size
             self.positions[n:].zero_()
             self.slots[n:].fill_(-1)
+            self.state_slots[n:].fill_(-1)
         self._last_n = n
         self.eng._graph_before_replay(self.token)
         self.graph.replay()
@@ -216,8 +225,14 @@ class InferenceEngine:
         mc = model.cfg
         self.device = model.tok_embeddings.device
         self.max_len = cfg.max_seq_len or mc.max_seq_len
-        self.cache = PagedKVCache(mc.num_layers, cfg.num_pages, mc.num_kv_heads, mc.head_dim, cfg.kv_mode, self.device)
-        self.prefix = PrefixCache(self.cache.allocator) if cfg.enable_prefix_cache else None
+        self.stack = hasattr(model, "run")     # the model brings its own pass over the layers and its own kind of cache
+        if self.stack:
+            if cfg.kv_mode != "bf16":
+                raise ValueError(f"{type(model).__name__} keeps keys and values in its own dtype; kv_mode '{cfg.kv_mode}' is not available")
+            self.cache = model.make_cache(cfg.num_pages, cfg.max_batch)
+        else:
+            self.cache = PagedKVCache(mc.num_layers, cfg.num_pages, mc.num_kv_heads, mc.head_dim, cfg.kv_mode, self.device)
+        self.prefix = PrefixCache(self.cache.allocator) if cfg.enable_prefix_cache and self.cache.shareable else None
         self.waiting: list = []
         self.running: List[Request] = []
         self._ids = itertools.count(1)
@@ -281,14 +296,40 @@ class InferenceEngine:
 
     def _release(self, r: Request):
         for p in r.pages:
-            self.cache.allocator.release(p)
+            if p >= 0:
+                self.cache.allocator.release(p)
         r.pages = []
+        self.cache.give_slot(r.state_slot)
+        r.state_slot = -1
+
+    def _reserve(self, r: Request, n: int, shared=()):
+        """Pages for tokens 0 .. n - 1 of a sequence that starts (``shared``: pages of a cached prefix; pages that no later
+        query will look at are left out) and its slot of recurrent state."""
+        lo = self.cache.first_live_page(n)
+        r.pages = list(shared) + [self.cache.allocator.alloc() if i >= lo else -1 for i in range(len(shared), (n + PAGE - 1) // PAGE)]
+        r.first_page = min(lo, len(r.pages))
+        r.state_slot = self.cache.take_slot()
+
+    def _drop_old_pages(self, r: Request):
+        """Give back the pages that have left the window of every query from r.pos on."""
+        lo = min(self.cache.first_live_page(r.pos), len(r.pages))
+        for i in range(r.first_page, lo):
+            self.cache.allocator.release(r.pages[i])
+            r.pages[i] = -1
+        r.first_page = max(r.first_page, lo)
+
+    @staticmethod
+    def _slot(r: Request, p: int) -> int:
+        pg = r.pages[p // PAGE]
+        return pg * PAGE + p % PAGE if pg >= 0 else -1
 
     # ------------------------------------------------------------------ model passes
     def _layers_prefill(self, ids, pos0, r: Request, all_positions: bool = False):
         """Prompt tokens ids[pos0:] of one sequence; K/V of all of them go to the pages.  Returns the
         hidden state of the last token (of every new token with ``all_positions``).  (Prefix pages already hold
         positions < pos0.)"""
+        if self.stack:
+            return self._stack_prefill([r], [ids[pos0:]], pos0, [list(range(len(ids) - pos0))] if all_positions else None)
         m, mc = self.model, self.model.cfg
         dev = self.device
         Hq, Hkv, D = mc.num_heads, mc.num_kv_heads, mc.head_dim
@@ -330,10 +371,40 @@ class InferenceEngine:
                 h = h + attn
         return h if all_positions else h[-1:]
 
+    def _stack_prefill(self, reqs: List[Request], ids, pos0: int = 0, want=None):
+        """Prompts (or, for one sequence, the portion ids[0] that starts at ``pos0``) through a stack model, padded on the right.
+        Returns the final-normed rows at the places ``want`` (one list per sequence; default: its last token)."""
+        from ..models.stack import StepBatch
+        dev, B, S = self.device, len(reqs), max(len(t) for t in ids)
+        if B > 1 and pos0:
+            raise ValueError("portions of prompts run one sequence at a time")
+        tok = torch.zeros((B, S), dtype=torch.int64)
+        slots = torch.full((B, S), -1, dtype=torch.int64)
+        for b, (r, t) in enumerate(zip(reqs, ids)):
+            tok[b, :len(t)] = torch.tensor(t, dtype=torch.int64)
+            pos = torch.arange(pos0, pos0 + len(t))
+            pg = torch.tensor(r.pages, dtype=torch.int64)[pos // PAGE]
+            slots[b, :len(t)] = torch.where(pg >= 0, pg * PAGE + pos % PAGE, -1)
+        want = [[len(t) - 1] for t in ids] if want is None else want
+        rows = torch.tensor([b * S + w for b, ws in enumerate(want) for w in ws], dtype=torch.int32, device=dev)
+        batch = StepBatch(tok.to(dev).reshape(-1), torch.arange(pos0, pos0 + S, dtype=torch.int32, device=dev).repeat(B), B, S,
+                          slots.to(dev).reshape(-1), torch.tensor([r.state_slot for r in reqs], dtype=torch.int32, device=dev),
+                          torch.tensor([len(t) for t in ids], dtype=torch.int32, device=dev), pos0,
+                          torch.tensor([max(p, 0) for p in reqs[0].pages], dtype=torch.int32, device=dev) if pos0 else None)
+        return self.model.run(batch, self.cache, self.max_len, rows, self._stack_lin)
+
+    def _stack_lin(self, x, li, name, w):
+        pw = self.packed.get(f"layers.{li}.{name}")
+        if pw is None:
+            return self.model.linear(x, w.data)
+        return self._wq.gemm_wq(x.contiguous(), pw, None)
+
     def _layers_prefill_batch(self, reqs: List[Request]):
         """Whole prompts of several sequences in one pass: rows are [B, S_max] with the shorter prompts padded on the right
         (causal attention keeps padding from reaching real tokens; padded rows carry slot -1 and are not cached).
         Returns the hidden state of every sequence's last prompt token, [B, H]."""
+        if self.stack:
+            return self._stack_prefill(reqs, [r.tokens for r in reqs])
         m, mc = self.model, self.model.cfg
         dev = self.device
         Hq, Hkv, D = mc.num_heads, mc.num_kv_heads, mc.head_dim
@@ -402,7 +473,12 @@ class InferenceEngine:
                 if not r.finished:
                     self.running.append(r)
 
-    def _layers_decode(self, tokens, positions, block_table, slots):
+    def _layers_decode(self, tokens, positions, block_table, slots, state_slots=None):
+        if self.stack:
+            from ..models.stack import StepBatch
+            B = tokens.shape[0]
+            batch = StepBatch(tokens, positions, B, 1, slots, state_slots, block_table=block_table, decode=True)
+            return self.model.run(batch, self.cache, self.max_len, None, self._stack_lin)
         m, mc = self.model, self.model.cfg
         Hq, Hkv, D = mc.num_heads, mc.num_kv_heads, mc.head_dim
         B = tokens.shape[0]
@@ -432,6 +508,8 @@ class InferenceEngine:
 
     def _logits(self, h):
         m = self.model
+        if self.stack:
+            return m.head(h)
         f, _ = _norm_fwd(m.cfg, h, m.norm, m.norm_bias)
         return F.gemm(f, m.lm_head.data)
 
@@ -476,7 +554,7 @@ class InferenceEngine:
             n = min(len(r.tokens), self.max_len - 1)
             r.tokens = r.tokens[:n]
             shared = self.prefix.lookup(r.tokens) if self.prefix else []
-            need = (n + r.max_tokens + PAGE - 1) // PAGE - len(shared)
+            need = self.cache.pages_needed(n + r.max_tokens) - len(shared)
             if need > alloc.num_free:
                 if self.prefix and self.prefix.table and not self.running:
                     for p in shared:
@@ -487,7 +565,7 @@ class InferenceEngine:
                     alloc.release(p)
                 break
             heapq.heappop(self.waiting)
-            r.pages = shared + [alloc.alloc() for _ in range((n + PAGE - 1) // PAGE - len(shared))]
+            self._reserve(r, n, shared)
             pos0 = len(shared) * PAGE
             if pos0 == 0 and self.cfg.batch_prefill:
                 fresh.append(r)
@@ -535,29 +613,9 @@ class InferenceEngine:
             pend, reqs = launch_set()
         if reqs:
             t0 = time.perf_counter()
-            for r in reqs:
-                if r.pos // PAGE >= len(r.pages):
-                    r.pages.append(alloc.alloc())
-            # host tokens (0 where the token is still on the device), positions, slots and the row of the previous step that
-            # holds a pending token (-1: none) travel in one small upload; the block table only re-sends what changed
-            packed = torch.tensor([[0 if id(r) in pend else r.out[-1] for r in reqs], [r.pos for r in reqs],
-                                   [r.pages[r.pos // PAGE] * PAGE + r.pos % PAGE for r in reqs],
-                                   [pend.get(id(r), -1) for r in reqs]], dtype=torch.int64).to(dev)
-            tokens, positions, slots = packed[0], packed[1].to(torch.int32), packed[2]
-            if pend:
-                src = packed[3]
-                tokens = torch.where(src >= 0, prev[1][src.clamp(min=0)], tokens)
-            bt = self._block_table(reqs)
-            if self.cfg.cuda_graph and dev.type == "cuda":
-                bucket = self._bucket(len(reqs))
-                g = self._graphs.get(bucket)
-                if g is None:
-                    g = self._graphs[bucket] = _DecodeGraph(self, bucket)
-                logits = g.replay(tokens, positions, bt, slots)
-            else:
-                logits = self._logits(self._layers_decode(tokens, positions, bt, slots))
-            for r in reqs:
-                r.pos += 1
+            # 0 where the token is still on the device (pend: the row of the previous step that holds it)
+            logits = self._decode_logits(reqs, [0 if id(r) in pend else r.out[-1] for r in reqs],
+                                         [pend.get(id(r), -1) for r in reqs] if pend else None, prev[1] if pend else None)
             toks_dev = self._sample_dev(logits, reqs)
             if pipelined:
                 host = ev = None
@@ -578,6 +636,104 @@ class InferenceEngine:
         elif prev is not None:
             self._collect(prev, finished)
         return finished
+
+    def _decode_logits(self, reqs: List[Request], host_tokens, pending=None, prev_tokens=None):
+        """Append one token to every sequence and return the logits [len(reqs), V] at it.  ``pending[i]`` >= 0: the token of row
+        i is row pending[i] of ``prev_tokens`` (on the device) instead of host_tokens[i]."""
+        dev, alloc = self.device, self.cache.allocator
+        for r in reqs:
+            if r.pos // PAGE >= len(r.pages):
+                r.pages.append(alloc.alloc())
+        # host tokens, positions, slots, state slots and pending rows travel in one small upload; the block table only
+        # re-sends what changed
+        packed = torch.tensor([host_tokens, [r.pos for r in reqs], [self._slot(r, r.pos) for r in reqs],
+                               [r.state_slot for r in reqs], pending or [-1] * len(reqs)], dtype=torch.int64).to(dev)
+        tokens, positions, slots, state_slots = packed[0], packed[1].to(torch.int32), packed[2], packed[3].to(torch.int32)
+        if pending is not None:
+            src = packed[4]
+            tokens = torch.where(src >= 0, prev_tokens[src.clamp(min=0)], tokens)
+        bt = self._block_table(reqs)
+        if self.cfg.cuda_graph and dev.type == "cuda":
+            bucket = self._bucket(len(reqs))
+            g = self._graphs.get(bucket)
+            if g is None:
+                g = self._graphs[bucket] = _DecodeGraph(self, bucket)
+            logits = g.replay(tokens, positions, bt, slots, state_slots)
+        else:
+            logits = self._logits(self._layers_decode(tokens, positions, bt, slots, state_slots))
+        for r in reqs:
+            r.pos += 1
+            self._drop_old_pages(r)
+        return logits
+
+    @torch.no_grad()
+    def feed(self, entries):
+        """Forward passes without sampling: ``entries`` is a list of (request, tokens, want).  A request that has not started
+        (``Request([])``) starts with these tokens; one that has goes on with them.  Returns, per entry, the logits at the
+        places ``want`` among its tokens ([len(want), V]).  All starting entries are one batch, all single tokens of
+        running requests another, portions of several tokens run one by one.  ``end`` gives back what a request holds."""
+        if any(not t for _, t, _ in entries):
+            raise ValueError("an entry brings no tokens")
+        out = [None] * len(entries)
+        for r, t, _ in entries:
+            if r.pos + len(t) > self.max_len:
+                raise ValueError(f"a sequence of {r.pos + len(t)} tokens does not fit into {self.max_len}")
+        fresh = [i for i, (r, _, _) in enumerate(entries) if r.pos == 0]
+        for i in fresh:
+            r, t, _ = entries[i]
+            r.id, r.tokens = next(self._ids), list(t)
+            self._reserve(r, len(t))
+        if fresh and self.stack:
+            lg = self._logits_at([entries[i] for i in fresh], 0)
+            for i, x in zip(fresh, lg):
+                out[i] = x
+        elif fresh:
+            for i in fresh:
+                r, t, w = entries[i]
+                h = self._layers_prefill(r.tokens, 0, r, all_positions=True)
+                out[i] = self._logits(h[torch.tensor(w, dtype=torch.int64, device=self.device)]) if w else None
+        for i in fresh:
+            entries[i][0].pos = len(entries[i][1])
+        going = [i for i in range(len(entries)) if i not in set(fresh)]
+        single = [i for i in going if len(entries[i][1]) == 1]
+        if single:
+            lg = self._decode_logits([entries[i][0] for i in single], [entries[i][1][0] for i in single])
+            for k, i in enumerate(single):
+                entries[i][0].tokens.append(entries[i][1][0])
+                if entries[i][2]:
+                    out[i] = lg[k:k + 1].clone()
+        for i in going:
+            r, t, w = entries[i]
+            if len(t) == 1:
+                continue
+            p0 = r.pos
+            r.tokens = r.tokens + list(t)
+            while len(r.pages) * PAGE < p0 + len(t):
+                r.pages.append(self.cache.allocator.alloc())
+            if self.stack:
+                out[i] = self._logits_at([entries[i]], p0)[0]
+            else:
+                h = self._layers_prefill(r.tokens, p0, r, all_positions=True)
+                out[i] = self._logits(h[torch.tensor(w, dtype=torch.int64, device=self.device)]) if w else None
+            r.pos = p0 + len(t)
+            self._drop_old_pages(r)
+        return out
+
+    def _logits_at(self, entries, pos0: int):
+        """Logits of a stack prefill at the wanted places, one tensor (or None) per entry."""
+        want = [w for _, _, w in entries]
+        some = any(want)
+        h = self._stack_prefill([r for r, _, _ in entries], [t for _, t, _ in entries], pos0,
+                                want if some else None)
+        if not some:
+            return [None] * len(entries)
+        lg = self._logits(h).split([len(w) for w in want])
+        return [x if w else None for x, w in zip(lg, want)]
+
+    def end(self, r: Request):
+        """Give back the pages and the state of a request that ``feed`` has run."""
+        self._release(r)
+        r.finished = True
 
     @staticmethod
     def _bucket(n: int) -> int:
@@ -620,7 +776,7 @@ class InferenceEngine:
             else:
                 continue
             idx.extend(range(i * mp + lo, i * mp + n))
-            val.extend(r.pages[lo:])
+            val.extend(max(p, 0) for p in r.pages[lo:])    # pages behind the window: never looked at
             if i < len(rows):
                 rows[i] = (r.id, n)
             else:

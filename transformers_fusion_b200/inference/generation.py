@@ -171,6 +171,8 @@ class _Seq:
     """One sequence on one engine: pages + position counter."""
 
     def __init__(self, eng: InferenceEngine, max_total: int):
+        if not eng.cache.shareable:        # recurrent state and pages behind a window do not come back
+            raise ValueError(f"{type(eng.model).__name__} keeps state that cannot be rewound; speculative decoding needs a full key / value cache")
         self.eng = eng
         self.r = Request([], max_total)
         self.r.pages = [eng.cache.allocator.alloc() for _ in range((max_total + PAGE - 1) // PAGE)]

@@ -117,6 +117,21 @@ class PagedKVCache:
         self.allocator = PageAllocator(num_pages)
         self._ws = {}
 
+    # what the scheduler asks of every kind of cache (see mixer_cache): no window, no recurrent state, prefixes may be shared
+    shareable = True
+
+    def first_live_page(self, pos: int) -> int:
+        return 0
+
+    def pages_needed(self, tokens: int) -> int:
+        return (tokens + PAGE - 1) // PAGE
+
+    def take_slot(self) -> int:
+        return -1
+
+    def give_slot(self, slot: int):
+        pass
+
     @classmethod
     def init(cls, num_layers: int, max_seq_len: int, num_heads: int, head_dim: int, mode="bf16", device="cuda", sequences: int = 1):
         """A cache with room for ``sequences`` sequences of ``max_seq_len`` tokens (rounded up to whole pages)."""

@@ -150,6 +150,158 @@ class MoEConfig(TransformerConfig):
             self.expert_hidden_size = self.ffn_hidden_size
 
 
+# ---------------------------------------------------------------------------------------------------------------------
+# decoders described layer by layer: every layer names its sequence mixer and its feed-forward
+# ---------------------------------------------------------------------------------------------------------------------
+@dataclass(frozen=True)
+class RotarySpec:
+    """Rotary embedding of the first ``dims`` entries of a head; ``yarn_*`` (factor None: unscaled) as in YaRN."""
+    dims: int
+    base: float
+    yarn_factor: float = None
+    yarn_original: int = 0
+    yarn_fast: float = 32.0
+    yarn_slow: float = 1.0
+
+
+@dataclass(frozen=True)
+class DiffAttentionSpec:
+    """Differential attention: per head two query / key maps of ``dim`` entries over one set of values of ``vdim`` entries.
+    ``window`` 0: plain causal.  ``kv_from``: index of the layer whose keys and values this layer uses instead of its own."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    diff: float
+    rot: RotarySpec
+    window: int = 0
+    kv_from: int = None
+
+    kind = "attention"
+
+
+@dataclass(frozen=True)
+class GatedDeltaSpec:
+    """Gated delta rule: ``kv_heads`` query / key heads of ``dim`` entries, ``heads`` value heads of ``vdim`` entries with a
+    [dim, vdim] state each, after a causal convolution of ``conv`` taps on q, k and v."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    conv: int
+
+    kind = "delta"
+
+    @property
+    def conv_channels(self) -> int:
+        return 2 * self.kv_heads * self.dim + self.heads * self.vdim
+
+
+@dataclass(frozen=True)
+class StackLayer:
+    mixer: object
+    ffn_hidden_size: int = 0     # 0: the layer has no feed-forward
+
+
+@dataclass
+class LanedraConfig:
+    """Lanedra: differential sliding-window attention (optionally on another layer's keys and values) and gated-delta-rule
+    layers in any order, norms before and after every sublayer, a 32-bit residual stream, a scaled embedding and a separate
+    output head.  ``from_dict`` reads the model folder's config.json; the folder sets no context limit, so ``max_seq_len``
+    is what the serving tables are sized for unless the engine's configuration says otherwise."""
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    norm_eps: float
+    embedding_scale: float = 1.0
+    max_seq_len: int = 32768
+
+    architecture = "Lanedra"
+
+    def __post_init__(self):
+        for i, l in enumerate(self.layers):
+            m = l.mixer
+            if m.heads % m.kv_heads:
+                raise ValueError(f"layer {i}: {m.heads} heads do not divide over {m.kv_heads} kv heads")
+            if m.kind == "attention":
+                if m.rot.dims % 2 or not 0 < m.rot.dims <= m.dim:
+                    raise ValueError(f"layer {i}: cannot rotate {m.rot.dims} of {m.dim} entries")
+                if m.kv_from is not None:
+                    src = self.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
+                    if src is None or src.kind != "attention" or src.kv_from is not None:
+                        raise ValueError(f"layer {i}: layer {m.kv_from} has no keys and values to share")
+                    if (src.kv_heads, src.dim, src.vdim) != (m.kv_heads, m.dim, m.vdim):
+                        raise ValueError(f"layer {i}: layer {m.kv_from}'s keys and values have other sizes")
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def window(self) -> int:
+        """Keys that any attention layer may still look at, the current one included; 0: all of them."""
+        w = [l.mixer.window for l in self.layers if l.mixer.kind == "attention"]
+        return 0 if not w or 0 in w else max(w)
+
+    @classmethod
+    def from_dict(cls, d: dict, **extra) -> "LanedraConfig":
+        layers = []
+        for i, e in enumerate(d["layers"]):
+            m = e["mixer"]
+            if e["type"] == "attention":
+                r = m["rot"]
+                y = r.get("scaling")
+                rot = RotarySpec(int(r["dims"]), float(r["base"])) if not y else \
+                    RotarySpec(int(r["dims"]), float(r["base"]), float(y["factor"]), y["original"], float(y["fast"]), float(y["slow"]))
+                mix = DiffAttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), float(m["diff"]), rot,
+                                        (m.get("mask") or {}).get("size") or 0, m.get("kv_from"))
+            elif e["type"] == "delta":
+                mix = GatedDeltaSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"])
+            else:
+                raise ValueError(f"layer {i}: unknown mixer '{e['type']}'")
+            mlp = e.get("mlp")
+            if mlp and mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward '{mlp['kind']}'")
+            layers.append(StackLayer(mix, mlp["ff"] if mlp else 0))
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], layers=layers, norm_eps=float(d["norm"]["eps"]),
+                   embedding_scale=float(d["embedding"]["scale"]), **extra)
+
+    def to_dict(self) -> dict:
+        """The config.json form."""
+        out = []
+        for l in self.layers:
+            m = l.mixer
+            x = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim}
+            if m.kind == "delta":
+                x["conv"] = m.conv
+            else:
+                r = {"dims": m.rot.dims, "base": m.rot.base}
+                if m.rot.yarn_factor is not None:
+                    r["scaling"] = {"factor": m.rot.yarn_factor, "original": m.rot.yarn_original, "fast": m.rot.yarn_fast,
+                                    "slow": m.rot.yarn_slow}
+                x.update(scale=m.scale, diff=m.diff, rot=r)
+                if m.window:
+                    x["mask"] = {"size": m.window}
+                if m.kv_from is not None:
+                    x["kv_from"] = m.kv_from
+            out.append({"type": m.kind, "mixer": x, "mlp": {"kind": "dense", "ff": l.ffn_hidden_size} if l.ffn_hidden_size else None})
+        return {"architecture": self.architecture, "embedding": {"scale": self.embedding_scale}, "layers": out,
+                "norm": {"eps": self.norm_eps}, "vocab": self.vocab_size, "width": self.hidden_size}
+
+    def num_params(self) -> int:
+        H, n = self.hidden_size, 2 * self.vocab_size * self.hidden_size + self.hidden_size
+        for l in self.layers:
+            m = l.mixer
+            if m.kind == "attention":
+                own = 0 if m.kv_from is not None else m.kv_heads * (2 * m.dim + m.vdim)
+                n += H * (2 * m.heads * m.dim + own + m.heads * m.vdim) + 4 * m.dim
+            else:
+                n += H * (m.conv_channels + 2 * m.heads * m.vdim + 2 * m.heads) + m.conv_channels * m.conv + 2 * m.heads + m.vdim
+            n += 2 * H + (3 * H * l.ffn_hidden_size + 2 * H if l.ffn_hidden_size else 0)
+        return n
+
+
 # Named shapes used by the benchmarks and tests (BASELINE configs).
 def preset(name: str) -> TransformerConfig:
     name = name.lower()

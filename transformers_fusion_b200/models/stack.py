@@ -1,0 +1,328 @@
+"""Decoders built from a list of layers with different sequence mixers: the mixers and the feed-forward as parameter modules
+with one forward pass each over a batch description (``StepBatch``), and the model that runs them over a 32-bit residual
+stream with a norm before and after every sublayer.
+
+The engine drives the same passes for prompts, for portions of prompts and for decoding; what is remembered between steps
+lives in ``inference.mixer_cache``.  A pass of one layer is, for a prompt or a decode step alike:
+
+  attention   GEMM [q | k | v], rotation + cache append, attention with its epilogue (difference of the maps, norm, scale), GEMM
+  delta       GEMM [q | k | v | gate | b | a], convolution + unit lengths + gates, recurrence (+ gated norm), GEMM
+  MLP         GEMM [gate | up], silu(gate) * up, GEMM
+  between     post-norm of the sublayer, residual add and pre-norm of the next sublayer, one kernel
+
+bf16 parameters: bf16 activations and tensor-core products; fp32 parameters: everything in true fp32."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+import torch.nn as nn
+
+from ..ops import functional as F
+from ..ops import stack as K
+
+
+@dataclass
+class StepBatch:
+    """B sequences with S rows each (rows past a sequence's length are padding).  ``decode``: one token per sequence over the
+    cache.  Otherwise a prompt (``pos0`` = 0) or, for one sequence, the portion that starts at ``pos0``."""
+    tokens: torch.Tensor                       # [B*S] int64
+    positions: torch.Tensor                    # [B*S] int32
+    B: int
+    S: int
+    slots: Optional[torch.Tensor] = None       # [B*S] int64 flat cache slots, -1: not cached
+    state_slots: Optional[torch.Tensor] = None # [B] int32
+    lens: Optional[torch.Tensor] = None        # [B] int32, None: S
+    pos0: int = 0
+    pages: Optional[torch.Tensor] = None       # int32, the page list of the sequence (pos0 > 0)
+    block_table: Optional[torch.Tensor] = None # [B, max_pages] int32 (decode)
+    decode: bool = False
+
+
+def _param(*shape, device, dtype, pitched=True):
+    w = K.padded_weight(*shape, dtype, device) if pitched and len(shape) == 2 else torch.zeros(shape, dtype=dtype, device=device)
+    return nn.Parameter(w, requires_grad=False)
+
+
+class DiffAttention(nn.Module):
+    """Differential attention with an optional window and optional keys / values of an earlier layer."""
+    linear_names = ("qkv", "o")
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+        super().__init__()
+        self.spec, self.eps, self.index = spec, eps, index
+        self.nq = 2 * spec.heads
+        self.nk = 0 if spec.kv_from is not None else 2 * spec.kv_heads
+        self.v_cols = spec.kv_heads * spec.vdim if self.nk else 0
+        kw = dict(device=device, dtype=dtype)
+        self.qkv = _param((self.nq + self.nk) * spec.dim + self.v_cols, hidden, **kw)
+        self.o = _param(hidden, spec.heads * spec.vdim, **kw)
+        for n in ("lq1", "lk1", "lq2", "lk2"):
+            setattr(self, n, _param(spec.dim, **kw))
+        self._lambda = None
+
+    def tensors(self):
+        s, a = self.spec, self.nq * self.spec.dim
+        b = a + self.nk * s.dim
+        yield "q", self.qkv.data[:a]
+        if self.nk:
+            yield "k", self.qkv.data[a:b]
+            yield "v", self.qkv.data[b:]
+        for n in ("lq1", "lk1", "lq2", "lk2", "o"):
+            yield n, getattr(self, n).data
+
+    def finalize(self):
+        d = lambda n: getattr(self, n).data.double()
+        self._lambda = float(torch.exp((d("lq1") * d("lk1")).sum()) - torch.exp((d("lq2") * d("lk2")).sum()) + self.spec.diff)
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        s = self.spec
+        if self._lambda is None:
+            self.finalize()
+        qkv = lin(h, self.index, "qkv", self.qkv)
+        pool = self.index if self.nk else s.kv_from
+        K.rope_append(qkv, rope, b.positions, self.nq, self.nk, s.dim, s.rot.dims, self.v_cols, b.slots if self.nk else None,
+                      cache.k[pool] if self.nk else None, cache.v[pool] if self.nk else None)
+        q = qkv[:, :self.nq * s.dim]
+        args = (s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.scale, self._lambda, 1.0 - s.diff, self.eps)
+        if b.decode:
+            o = K.diff_decode(q, cache.k[pool], cache.v[pool], b.block_table, b.positions, *args)
+        else:
+            if self.nk:                        # keys and values of this step, for this layer and for those that share them
+                if b.pos0 == 0:
+                    c = self.nq * s.dim
+                    kv[self.index] = (qkv[:, c:c + self.nk * s.dim], qkv[:, c + self.nk * s.dim:], b.S)
+                else:
+                    lo = max(0, b.pos0 - cache.window + 1) if cache.window else 0
+                    n = b.pos0 + b.S - lo
+                    kv[self.index] = (K.gather_rows(cache.k[pool], b.pages, lo, n), K.gather_rows(cache.v[pool], b.pages, lo, n), n)
+            k, v, n = kv[pool]
+            o = K.diff_attn(q, k, v, b.B, b.S, n, *args)
+        return lin(o, self.index, "o", self.o)
+
+
+class GatedDelta(nn.Module):
+    """Gated delta rule with a short convolution in front and a gated norm behind."""
+    linear_names = ("proj", "o")
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+        super().__init__()
+        self.spec, self.eps, self.index = spec, eps, index
+        kw = dict(device=device, dtype=dtype)
+        self.hv = spec.heads * spec.vdim
+        self.proj = _param(spec.conv_channels + self.hv + 2 * spec.heads, hidden, **kw)
+        self.conv = _param(spec.conv_channels, spec.conv, pitched=False, **kw)
+        self.A_log, self.dt_bias, self.norm = _param(spec.heads, **kw), _param(spec.heads, **kw), _param(spec.vdim, **kw)
+        self.o = _param(hidden, self.hv, **kw)
+
+    def tensors(self):
+        s = self.spec
+        gd, c = s.kv_heads * s.dim, s.conv_channels
+        cuts = {"q": (0, gd), "k": (gd, 2 * gd), "v": (2 * gd, c), "g": (c, c + self.hv),
+                "b": (c + self.hv, c + self.hv + s.heads), "a": (c + self.hv + s.heads, c + self.hv + 2 * s.heads)}
+        for n, (lo, hi) in cuts.items():
+            yield n, self.proj.data[lo:hi]
+            if n in ("q", "k", "v"):
+                yield n + ".conv", self.conv.data[lo:hi]
+        for n in ("A_log", "dt_bias", "norm", "o"):
+            yield n, getattr(self, n).data
+
+    def finalize(self):
+        pass
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        s, i = self.spec, self.index
+        G, H, D, V = s.kv_heads, s.heads, s.dim, s.vdim
+        p = lin(h, i, "proj", self.proj)
+        past = b.decode or b.pos0 > 0
+        prep = K.delta_prep(p, self.conv.data, cache.conv[i], b.state_slots, self.A_log.data, self.dt_bias.data, b.lens, b.B, b.S, G, H, D, V, past)
+        gate = p[:, s.conv_channels:s.conv_channels + self.hv]
+        if b.decode:
+            o = K.delta_step(prep, cache.state[i], b.state_slots, gate, self.norm.data, self.eps, b.B, G, H, D, V)
+        else:
+            o = K.gated_norm(K.delta_scan(prep, cache.state[i], b.state_slots, b.lens, b.B, b.S, G, H, D, V, past), gate, self.norm.data, self.eps)
+        return lin(o, i, "o", self.o)
+
+
+class GatedMLP(nn.Module):
+    linear_names = ("gate_up", "down")
+
+    def __init__(self, hidden: int, ff: int, index: int, device, dtype):
+        super().__init__()
+        self.ff, self.index = ff, index
+        self.gate_up = _param(2 * ff, hidden, device=device, dtype=dtype)
+        self.down = _param(hidden, ff, device=device, dtype=dtype)
+
+    def tensors(self):
+        yield "gate", self.gate_up.data[:self.ff]
+        yield "up", self.gate_up.data[self.ff:]
+        yield "down", self.down.data
+
+    def forward(self, h, lin):
+        return lin(K.glu_silu(lin(h, self.index, "gate_up", self.gate_up)), self.index, "down", self.down)
+
+
+MIXERS = {"attention": DiffAttention, "delta": GatedDelta}
+
+
+class SandwichLayer(nn.Module):
+    """norm1, mixer, norm1b and - unless the layer is a mixer alone - norm2, feed-forward, norm2b."""
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+        super().__init__()
+        kw = dict(device=device, dtype=dtype)
+        self.mixer = MIXERS[spec.mixer.kind](spec.mixer, hidden, eps, index, device, dtype)
+        self.norm1, self.norm1b = _param(hidden, **kw), _param(hidden, **kw)
+        self.mlp = GatedMLP(hidden, spec.ffn_hidden_size, index, device, dtype) if spec.ffn_hidden_size else None
+        if self.mlp is not None:
+            self.norm2, self.norm2b = _param(hidden, **kw), _param(hidden, **kw)
+
+    @property
+    def linears(self):
+        """{name: matrix} of the layer's products (what a low-bit weight format may replace)."""
+        return {n: getattr(m, n) for m in (self.mixer, self.mlp) if m is not None for n in m.linear_names}
+
+    def tensors(self):
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if self.mlp is not None else ()):
+            yield n, getattr(self, n).data
+        for n, t in self.mixer.tensors():
+            yield "mix." + n, t
+        if self.mlp is not None:
+            for n, t in self.mlp.tensors():
+                yield "mlp." + n, t
+
+
+def _plain_linear(x, index, name, w):
+    return K.linear(x, w.data)
+
+
+class StackModel(nn.Module):
+    """Embedding, layers, final norm, head.  ``run`` is the pass the engine drives; ``forward`` / ``hidden_states`` are whole
+    sequences without a cache."""
+    kernel_units = K.UNITS
+    linear = staticmethod(K.linear)
+    runs_fp32 = True             # every kernel of the pass has a true fp32 form
+
+    def __init__(self, cfg, device=None, dtype=torch.bfloat16, seed: Optional[int] = 0):
+        super().__init__()
+        self.cfg = cfg
+        device = torch.device(device if device is not None else "cpu")
+        kw = dict(device=device, dtype=dtype)
+        self.tok_embeddings = _param(cfg.vocab_size, cfg.hidden_size, **kw)
+        self.layers = nn.ModuleList([SandwichLayer(l, cfg.hidden_size, cfg.norm_eps, i, device, dtype) for i, l in enumerate(cfg.layers)])
+        self.norm = _param(cfg.hidden_size, **kw)
+        self.lm_head = _param(cfg.vocab_size, cfg.hidden_size, **kw)
+        self._rope = {}
+        if seed is not None:
+            self.init_weights(seed)
+
+    def init_weights(self, seed: int = 0):
+        """Random weights that keep activations of order one: N(0, 1 / fan-in) matrices, small deviations for the norms, decays
+        between about 0.5 and 1."""
+        g = torch.Generator(device="cpu").manual_seed(seed)
+        with torch.no_grad():
+            for name, t in self.named_tensors():
+                leaf = name.rsplit(".", 1)[-1]
+                r = torch.randn(t.shape, generator=g)
+                if leaf == "A_log":
+                    r = r * 0.5 - 1.5
+                elif leaf == "conv":
+                    r = r * t.shape[1] ** -0.5
+                elif t.dim() == 2:
+                    r = r * (1.0 if name == self.embed_name else t.shape[1] ** -0.5)
+                elif name.endswith("mix.norm"):
+                    r = 1 + 0.1 * r
+                else:
+                    r = 0.1 * r
+                t.copy_(r.to(t.dtype))
+        self.finalize()
+
+    def finalize(self):
+        """Derived constants, after the parameters have changed."""
+        for l in self.layers:
+            l.mixer.finalize()
+
+    embed_name, head_name, norm_name = "embed", "head", "final.norm"
+
+    def named_tensors(self):
+        """(name in the model folder, view into the parameters) pairs."""
+        out = [(self.embed_name, self.tok_embeddings.data)]
+        for i, l in enumerate(self.layers):
+            out += [(f"l{i}.{n}", t) for n, t in l.tensors()]
+        return out + [(self.norm_name, self.norm.data), (self.head_name, self.lm_head.data)]
+
+    def get_parameters(self):
+        return list(self.parameters())
+
+    def param_count(self) -> int:
+        return sum(t.numel() for _, t in self.named_tensors())
+
+    def vocab_size(self) -> int:
+        return self.cfg.vocab_size
+
+    @property
+    def dtype(self):
+        return self.tok_embeddings.dtype
+
+    @property
+    def device(self):
+        return self.tok_embeddings.device
+
+    # ------------------------------------------------------------------ passes
+    def rope(self, spec, max_pos: int):
+        """cos / sin tables of one rotation for at least ``max_pos`` positions."""
+        t = self._rope.get(spec)
+        if t is None or t[0].shape[0] < max_pos or t[0].device != self.device:
+            mode = "none" if spec.yarn_factor is None else "yarn"
+            t = F.rope_tables(spec.dims, max_pos, spec.base, mode, spec.yarn_factor or 1.0, spec.yarn_original, 1.0, spec.yarn_fast, spec.yarn_slow,
+                              device=self.device, yarn_ramp_max=spec.dims - 1)
+            self._rope[spec] = t
+        return t
+
+    def make_cache(self, num_pages: int, num_slots: int):
+        from ..inference.mixer_cache import MixerCache
+        return MixerCache(self.cfg, num_pages, num_slots, self.dtype, self.device)
+
+    def run(self, b: StepBatch, cache, max_pos: int, row_index=None, lin=_plain_linear, residuals=None):
+        """One step over all layers.  Returns the final-normed rows (of ``row_index``, int32; all rows without it).
+        ``residuals``: a list that receives a copy of the residual stream after every layer."""
+        cfg = self.cfg
+        eps, n = cfg.norm_eps, b.tokens.shape[0]
+        x = torch.empty((n, cfg.hidden_size), dtype=torch.float32, device=self.device)
+        h = K.res_norm(x, eps, ids=b.tokens, table=self.tok_embeddings.data, scale=cfg.embedding_scale, w_pre=self.layers[0].norm1.data)
+        kv = {}
+        for i, l in enumerate(self.layers):
+            last = i + 1 == len(self.layers)
+            nxt, rows = (self.norm.data, row_index) if last else (self.layers[i + 1].norm1.data, None)
+            rope = self.rope(l.mixer.spec.rot, max_pos) if l.mixer.spec.kind == "attention" else None
+            y = l.mixer(h, b, cache, rope, lin, kv)
+            if l.mlp is not None:
+                h = K.res_norm(x, eps, y=y, w_post=l.norm1b.data, w_pre=l.norm2.data)
+                y = l.mlp(h, lin)
+                post = l.norm2b.data
+            else:
+                post = l.norm1b.data
+            if residuals is not None:
+                z = x.clone()
+                K.res_norm(z, eps, y=y, w_post=post)
+                residuals.append(z)
+            h = K.res_norm(x, eps, y=y, w_post=post, w_pre=nxt, row_index=rows)
+        return h
+
+    def head(self, h):
+        """fp32 logits of final-normed rows."""
+        return K.linear(h, self.lm_head.data, out_dtype=torch.float32)
+
+    @torch.no_grad()
+    def hidden_states(self, ids, residuals=None):
+        """Final-normed rows [B*S, H] of whole sequences ids [B, S]."""
+        B, S = ids.shape
+        dev = self.device
+        b = StepBatch(ids.reshape(-1).to(dev), torch.arange(S, dtype=torch.int32, device=dev).repeat(B), B, S,
+                      state_slots=torch.arange(B, dtype=torch.int32, device=dev))
+        return self.run(b, self.make_cache(0, B), S, residuals=residuals)
+
+    @torch.no_grad()
+    def forward(self, ids):
+        return self.head(self.hidden_states(ids)).view(*ids.shape, -1)

@@ -66,12 +66,12 @@ def bounds_report(reset: bool = True) -> dict:
     (sites: 1 embedding id, 2 embedding-gradient id, 3 cross-entropy label, 5 routed expert id, 11 gather block of a
     fused GEMM, 12 expert of a grouped-GEMM row tile, 21 row owner of the sharded embedding, 31 vocabulary-parallel label,
     41 destination row of an expert-parallel dispatch, 51 KV-cache slot of an append, 52 page of a paged-decode block
-    table, 53 page of a KV gather)."""
+    table, 53 page of a KV gather, 61 position of a rotation, 71 / 72 / 73 recurrent-state slot)."""
     out = {}
     if not bounds_check_build():
         return out
     for unit in ("elementwise", "loss_optim", "moe_routing", "gemm_bf16", "fsdp_fused", "loss_vocab_parallel", "ep_fused",
-                 "paged_attention"):
+                 "paged_attention", "stack_ops", "delta_rule", "diff_attention"):
         fn = getattr(lib(), f"tfb_bounds_report_{unit}", None)
         if fn is None:
             continue
@@ -87,13 +87,26 @@ def available() -> bool:
     return lib_path().exists()
 
 
+_UNITS = None           # set by need_units
+
+
+def need_units(name: str, units):
+    """Called before the library is loaded by a process that runs one kind of model: if the full library has not been built,
+    ``lib()`` then builds and loads lib<name>.so with those translation units only."""
+    global _UNITS
+    _UNITS = (name, tuple(units))
+
+
 def lib():
     """Load (once) and return the kernel library; build it first if the shared object is absent."""
     global _lib
     if _lib is not None:
         return _lib
     p = lib_path()
-    if not p.exists():
+    if not p.exists() and _UNITS is not None and not bounds_check_build() and not os.environ.get("TFB_NO_AUTOBUILD"):
+        from .. import build as _build
+        p = _build.build_kernels(units=_UNITS[1], name=_UNITS[0])
+    elif not p.exists():
         if os.environ.get("TFB_NO_AUTOBUILD"):
             raise KernelError(f"{p} is missing; run `python -m transformers_fusion_b200.build`")
         from .. import build as _build
@@ -112,7 +125,7 @@ def lib():
 def register(name: str, sig):
     """Declare the signature of an entry point defined by another module (attention, comm, quant)."""
     _SIGS[name] = sig
-    if _lib is not None:
+    if _lib is not None and (_UNITS is None or hasattr(_lib, name)):
         fn = getattr(_lib, name)
         fn.argtypes = sig
         fn.restype = c_i

@@ -176,10 +176,12 @@ def layernorm_bwd(dy, h, w, rstd, mean, dw, db, dres=None):
 # rotary embedding
 # ---------------------------------------------------------------------------------------------
 def rope_tables(head_dim, max_pos, theta=10000.0, scaling_mode="none", scaling_factor=1.0, original_max=0,
-                yarn_attn_factor=1.0, yarn_beta_fast=32.0, yarn_beta_slow=1.0, device="cpu"):
+                yarn_attn_factor=1.0, yarn_beta_fast=32.0, yarn_beta_slow=1.0, device="cpu", yarn_ramp_max=None):
     """cos/sin tables [max_pos, head_dim/2] fp32 for rotate-half RoPE with the reference's scaling modes
     (src/model/transformer.cpp:124-211): none, linear (positions / factor), ntk (theta scaled by
-    factor^(d/(d-2))), yarn (per-frequency blend of interpolated and extrapolated frequencies)."""
+    factor^(d/(d-2))), yarn (per-frequency blend of interpolated and extrapolated frequencies).  ``yarn_ramp_max``: the
+    largest index the upper end of the blend may have (default: the last frequency, head_dim/2 - 1); when given, the blend
+    and its factor on cos and sin apply for every scaling factor, 1 and below included."""
     half = head_dim // 2
     j = torch.arange(half, dtype=torch.float64)
     mode = (scaling_mode or "none").lower()
@@ -188,13 +190,13 @@ def rope_tables(head_dim, max_pos, theta=10000.0, scaling_mode="none", scaling_f
         base = base * scaling_factor ** (head_dim / max(head_dim - 2, 1))
     inv = base ** (-2.0 * j / head_dim)
     mscale = 1.0
-    if mode == "yarn" and scaling_factor > 1.0:
+    if mode == "yarn" and (scaling_factor > 1.0 or yarn_ramp_max is not None):
         orig = float(original_max or max_pos)
 
         def corr(n_rot):
             return head_dim * math.log(orig / (n_rot * 2 * math.pi)) / (2 * math.log(theta))
         lo = max(math.floor(corr(yarn_beta_fast)), 0)
-        hi = min(math.ceil(corr(yarn_beta_slow)), half - 1)
+        hi = min(math.ceil(corr(yarn_beta_slow)), half - 1 if yarn_ramp_max is None else yarn_ramp_max)
         ramp = ((j - lo) / max(hi - lo, 1e-3)).clamp(0, 1)
         inv = inv / scaling_factor * ramp + inv * (1 - ramp)
         mscale = yarn_attn_factor * (0.1 * math.log(scaling_factor) + 1.0)

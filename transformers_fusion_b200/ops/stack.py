@@ -1,0 +1,295 @@
+"""Raw operators of decoders that are a stack of different sequence mixers over a 32-bit residual stream: norms around
+every sublayer, partial rotary embedding, differential attention, gated delta rule, true fp32 products.
+
+As in ``functional``: CUDA tensors go to the sm_100a kernels (``csrc/kernels/stack_ops.cu``, ``diff_attention.cu``,
+``delta_rule.cu``), CPU tensors run the plain PyTorch statement of the same math.  Activations are bf16 or fp32 (the dtype of
+the tensors decides); the residual, norms, rotation, attention scores and weights, and the recurrence are fp32 in both."""
+from __future__ import annotations
+
+import math
+from typing import Optional
+
+import torch
+
+from . import _lib
+from . import functional as F
+from ._lib import c_f, c_i, c_ll, c_p, check, ptr, stream
+
+UNITS = ("tfb_host", "gemm_bf16", "stack_ops", "diff_attention", "delta_rule")    # translation units these operators need
+PAGE = 16
+
+_lib.register("tfb_res_norm", [c_p, c_p, c_ll, c_f, c_i, c_p, c_ll, c_p, c_ll, c_p, c_p, c_p, c_ll, c_p, c_i, c_i, c_f, c_i, c_p])
+_lib.register("tfb_glu_silu", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
+_lib.register("tfb_rope_append", [c_p, c_ll, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_gather_rows", [c_p, c_ll, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p])
+_lib.register("tfb_gemm_f32", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
+_lib.register("tfb_diff_attn_fwd", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_f, c_f, c_i,
+                                    c_p, c_p])
+_lib.register("tfb_diff_decode_tc", [c_i, c_i, c_i])
+_lib.register("tfb_diff_decode", [c_p, c_ll, c_p, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f,
+                                  c_f, c_f, c_i, c_p, c_p])
+_lib.register("tfb_delta_prep", [c_p, c_ll, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
+                                 c_i, c_p])
+_lib.register("tfb_delta_scan", [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_gated_norm", [c_p, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_f, c_i, c_p])
+_lib.register("tfb_delta_step", [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
+
+
+def _f32(t) -> int:
+    assert t.dtype in (torch.float32, torch.bfloat16), t.dtype
+    return int(t.dtype == torch.float32)
+
+
+def rows(n: int, width: int, dtype, device) -> torch.Tensor:
+    """Uninitialised [n, width] activations whose row pitch is a multiple of 8 elements (TMA wants 16-byte pitches)."""
+    return torch.empty((n, (width + 7) // 8 * 8), dtype=dtype, device=device)[:, :width]
+
+
+def padded_weight(n: int, width: int, dtype, device) -> torch.Tensor:
+    """Zero [n, width] matrix with the same pitch rule."""
+    return torch.zeros((n, (width + 7) // 8 * 8), dtype=dtype, device=device)[:, :width]
+
+
+# ---------------------------------------------------------------------------------------------------- products
+def linear(x, w, out_dtype=None):
+    """x [M, K] @ w [N, K]^T.  bf16 operands: tensor-core GEMM with fp32 accumulation (``out_dtype`` fp32 keeps the
+    accumulator's precision); fp32 operands: FFMA in true fp32."""
+    out_dtype = out_dtype or x.dtype
+    if not x.is_cuda:
+        return (x.float() @ w.float().t()).to(out_dtype)
+    M, K = x.shape
+    N = w.shape[0]
+    out = rows(M, N, out_dtype, x.device)
+    if x.dtype == torch.float32:
+        assert w.dtype == torch.float32 and w.shape[1] == K and x.stride(1) == 1 and w.stride(1) == 1
+        check(_lib.lib().tfb_gemm_f32(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, stream()),
+              "gemm_f32")
+        return out
+    return F.gemm(x, w, out=out)
+
+
+# ---------------------------------------------------------------------------------------------------- norms
+def centred_rms(x, w, eps):
+    xf = x.float()
+    return xf / torch.sqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * (1 + w.float())
+
+
+def res_norm(x, eps, *, y=None, w_post=None, w_pre=None, ids=None, table=None, scale=1.0, row_index=None, dtype=None):
+    """x += norm(y) * (1 + w_post) on the fp32 residual ``x`` [n, H] in place; returns norm(x) * (1 + w_pre) in the
+    activation dtype (None without ``w_pre``).  ``ids``: x starts as scale * table[ids].  ``row_index`` (int32): only those
+    rows are computed and returned, and x keeps its values."""
+    if not x.is_cuda:
+        v = table[ids.long()].float() * scale if ids is not None else x
+        if y is not None:
+            v = v + centred_rms(y, w_post, eps)
+        if row_index is None:
+            x.copy_(v)
+        else:
+            v = v[row_index.long()]
+        return None if w_pre is None else centred_rms(v, w_pre, eps).to(dtype or w_pre.dtype)
+    H = x.shape[1]
+    n = x.shape[0] if row_index is None else row_index.shape[0]
+    w = w_pre if w_pre is not None else w_post
+    a = rows(n, H, w.dtype, x.device) if w_pre is not None else None
+    check(_lib.lib().tfb_res_norm(ptr(ids), ptr(table), table.stride(0) if table is not None else 0, float(scale),
+                                  table.shape[0] if table is not None else 0, x.data_ptr(), x.stride(0), ptr(y),
+                                  y.stride(0) if y is not None else 0, ptr(w_post), ptr(w_pre), ptr(a), a.stride(0) if a is not None else 0,
+                                  ptr(row_index), n, H, float(eps), _f32(w), stream()), "res_norm")
+    return a
+
+
+def glu_silu(gu):
+    """[gate | up] -> silu(gate) * up."""
+    M, F2 = gu.shape
+    Fh = F2 // 2
+    if not gu.is_cuda:
+        g = gu[:, :Fh].float()
+        return (g * torch.sigmoid(g) * gu[:, Fh:].float()).to(gu.dtype)
+    out = rows(M, Fh, gu.dtype, gu.device)
+    check(_lib.lib().tfb_glu_silu(gu.data_ptr(), gu.stride(0), out.data_ptr(), out.stride(0), M, Fh, _f32(gu), stream()), "glu_silu")
+    return out
+
+
+# ---------------------------------------------------------------------------------------------------- rotation + cache
+def rope_append(qkv, tables, positions, nq, nk, D, dims, v_cols, slots=None, kpool=None, vpool=None):
+    """Rotate the first ``dims`` entries of the nq query and nk key heads of every row of ``qkv`` ([q | k | v]) in place and
+    write k and v to flat slots of the pools ([slots, nk * D], [slots, v_cols]; negative slots are not cached)."""
+    cos, sin = tables
+    T = qkv.shape[0]
+    if not qkv.is_cuda:
+        half = dims // 2
+        c, s = cos[positions.long()][:, None], sin[positions.long()][:, None]
+        x = qkv[:, :(nq + nk) * D].reshape(T, nq + nk, D).float()
+        u, v = x[..., :half], x[..., half:dims]
+        x = torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], -1)
+        qkv[:, :(nq + nk) * D] = x.reshape(T, -1).to(qkv.dtype)
+        if nk and slots is not None:
+            keep = slots >= 0
+            kpool[slots[keep]] = qkv[keep, nq * D:(nq + nk) * D]
+            vpool[slots[keep]] = qkv[keep, (nq + nk) * D:(nq + nk) * D + v_cols]
+        return qkv
+    check(_lib.lib().tfb_rope_append(qkv.data_ptr(), qkv.stride(0), cos.data_ptr(), sin.data_ptr(), cos.shape[0], positions.data_ptr(),
+                                     ptr(slots), ptr(kpool), ptr(vpool), kpool.shape[0] if kpool is not None else 0, T, nq, nk, D, dims,
+                                     v_cols, _f32(qkv), stream()), "rope_append")
+    return qkv
+
+
+def gather_rows(pool, pages, lo, n):
+    """Cached rows of positions lo .. lo + n - 1 of one sequence (``pages``: its page list, int32), contiguous."""
+    width = pool.shape[1]
+    if not pool.is_cuda:
+        p = torch.arange(lo, lo + n)
+        return pool[pages[p // PAGE].long() * PAGE + p % PAGE].clone()
+    out = torch.empty((n, width), dtype=pool.dtype, device=pool.device)
+    check(_lib.lib().tfb_gather_rows(pool.data_ptr(), pool.shape[0], pages.data_ptr(), PAGE, lo, n, out.data_ptr(), width, _f32(pool), stream()),
+          "gather_rows")
+    return out
+
+
+# ---------------------------------------------------------------------------------------------------- differential attention
+def _diff_ref(q, k, v, B, S, Skv, H, G, D, V, window, scale, lam, out_scale, eps):
+    R = H // G
+    Q = q.reshape(B, S, H, 2, D).permute(0, 2, 3, 1, 4).float()                     # [B, H, 2, S, D]
+    K = k.reshape(B, Skv, G, 2, D).permute(0, 2, 3, 1, 4).float().repeat_interleave(R, 1)
+    W = v.reshape(B, Skv, G, V).permute(0, 2, 1, 3).float().repeat_interleave(R, 1)
+    i = torch.arange(S)[:, None] + (Skv - S)
+    j = torch.arange(Skv)[None]
+    hide = (j > i) | ((i - j >= window) if window else torch.zeros(1, dtype=torch.bool))
+    s = (Q @ K.transpose(-1, -2) * scale).masked_fill(hide, -math.inf)
+    a = torch.softmax(s, -1) @ W[:, :, None]                                        # [B, H, 2, S, V]
+    o = a[:, :, 0] - lam * a[:, :, 1]
+    o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * out_scale
+    return o.permute(0, 2, 1, 3).reshape(B * S, H * V).to(q.dtype)
+
+
+def diff_attn(q, k, v, B, S, Skv, H, G, D, V, window, scale, lam, out_scale, eps):
+    """Differential attention of B prompts.  q [B*S, 2 H D], k [B*Skv, 2 G D] (rotated), v [B*Skv, G V]; the queries are the
+    last S of the Skv positions; ``window`` 0: plain causal.  Returns [B*S, H V]."""
+    if not q.is_cuda:
+        return _diff_ref(q, k, v, B, S, Skv, H, G, D, V, window, scale, lam, out_scale, eps)
+    o = rows(B * S, H * V, q.dtype, q.device)
+    check(_lib.lib().tfb_diff_attn_fwd(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), o.data_ptr(), o.stride(0),
+                                       B, S, Skv, H, G, D, V, window, float(scale), float(lam), float(out_scale), float(eps), _f32(q),
+                                       _lib.status_word(q.device).data_ptr(), stream()), "diff_attn_fwd")
+    return o
+
+
+def diff_decode(q, kpool, vpool, block_table, positions, H, G, D, V, window, scale, lam, out_scale, eps, max_keys: int = 0,
+                splits: Optional[int] = None):
+    """One query per sequence (q [B, 2 H D], rotated, at ``positions``) over its cached rows.  ``max_keys``: a bound on the
+    keys any query can see (for the choice of the split count only)."""
+    B = q.shape[0]
+    if not q.is_cuda:
+        out = torch.zeros((B, H * V), dtype=q.dtype)
+        for b in range(B):
+            n = int(positions[b]) + 1
+            lo = max(0, n - window) if window else 0
+            p = torch.arange(lo, n)
+            s = block_table[b, (p // PAGE).long()].long() * PAGE + p % PAGE
+            out[b] = _diff_ref(q[b:b + 1], kpool[s], vpool[s], 1, 1, n - lo, H, G, D, V, window, scale, lam, out_scale, eps)[0]
+        return out
+    o = rows(B, H * V, q.dtype, q.device)
+    L, f32 = _lib.lib(), _f32(q)
+    acc = ml = None
+    if L.tfb_diff_decode_tc(D, V, f32) and q.stride(0) % 8 == 0:
+        chunks = (H // G + 7) // 8
+        if splits is None:
+            keys = max_keys or block_table.shape[1] * PAGE
+            keys = min(keys, window + PAGE) if window else keys
+            splits = max(1, min(32, (4 * 148) // max(1, B * G * chunks), keys // 128))
+        acc = torch.empty(B * G * chunks * splits * 16 * V, dtype=torch.float32, device=q.device)
+        ml = torch.empty(B * G * chunks * splits * 32, dtype=torch.float32, device=q.device)
+    check(L.tfb_diff_decode(q.data_ptr(), q.stride(0), kpool.data_ptr(), vpool.data_ptr(), kpool.shape[0], block_table.data_ptr(),
+                            block_table.shape[1], PAGE, positions.data_ptr(), o.data_ptr(), o.stride(0), ptr(acc), ptr(ml), splits or 1, B, H, G,
+                            D, V, window, float(scale), float(lam), float(out_scale), float(eps), f32, _lib.status_word(q.device).data_ptr(),
+                            stream()), "diff_decode", 2 if acc is not None else 1)
+    return o
+
+
+# ---------------------------------------------------------------------------------------------------- gated delta rule
+def delta_prep(proj, conv_w, conv_state, state_slots, A_log, dt_bias, lens, B, S, G, H, D, V, has_past):
+    """proj [B*S, 2 G D + 2 H V + 2 H] = q | k | v | gate | b | a  ->  (q, k, v, k.q, decay, beta), all fp32.  ``conv_state``
+    [slots, taps - 1, channels] is read for sequences that go on (``has_past``) and left holding their last inputs."""
+    T, C, taps = B * S, 2 * G * D + H * V, conv_w.shape[1]
+    if not proj.is_cuda:
+        x = proj[:, :C].reshape(B, S, C)
+        n = lens if lens is not None else torch.full((B,), S)
+        full = torch.zeros((B, taps - 1 + S, C), dtype=x.dtype)
+        full[:, taps - 1:] = x
+        if taps > 1 and has_past:
+            ok = state_slots >= 0
+            full[ok, :taps - 1] = conv_state[state_slots[ok].long()]
+        w = conv_w.float()
+        y = sum(full[:, j:j + S].float() * w[:, j] for j in range(taps))
+        y = (y * torch.sigmoid(y)).reshape(T, C)
+        if taps > 1:
+            for b in range(B):
+                if int(state_slots[b]) >= 0:
+                    conv_state[int(state_slots[b])] = full[b, int(n[b]): int(n[b]) + taps - 1]
+        q, k = y[:, :G * D].reshape(T, G, D), y[:, G * D:2 * G * D].reshape(T, G, D)
+        q = q / torch.sqrt(q.pow(2).sum(-1, keepdim=True) + 1e-6) * D ** -0.5
+        k = k / torch.sqrt(k.pow(2).sum(-1, keepdim=True) + 1e-6)
+        tail = proj[:, C + H * V:].float()
+        beta = torch.sigmoid(tail[:, :H])
+        decay = torch.exp(-torch.exp(A_log.float()) * torch.nn.functional.softplus(tail[:, H:2 * H] + dt_bias.float()))
+        return q, k, y[:, 2 * G * D:].reshape(T, H, V), (q * k).sum(-1), decay, beta
+    e = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
+    q, k, v, kq, decay, beta = e(T, G, D), e(T, G, D), e(T, H, V), e(T, G), e(T, H), e(T, H)
+    check(_lib.lib().tfb_delta_prep(proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), ptr(conv_state), ptr(state_slots),
+                                    conv_state.shape[0] if conv_state is not None else 0, A_log.data_ptr(), dt_bias.data_ptr(), ptr(lens),
+                                    q.data_ptr(), k.data_ptr(), v.data_ptr(), kq.data_ptr(), decay.data_ptr(), beta.data_ptr(), B, S, G, H, D, V,
+                                    taps, int(has_past), _f32(proj), stream()), "delta_prep", 1 if S == 1 or taps == 1 else 2)
+    return q, k, v, kq, decay, beta
+
+
+def delta_scan(prep, state, state_slots, lens, B, S, G, H, D, V, has_past):
+    """The recurrence over prepared rows; ``state`` [slots, H, D, V] fp32 is read (``has_past``) and updated.  Returns fp32
+    [B*S, H, V] (rows past a sequence's length are unspecified)."""
+    q, k, v, kq, decay, beta = prep
+    if not q.is_cuda:
+        out = torch.zeros(B * S, H, V)
+        n = lens if lens is not None else torch.full((B,), S)
+        rep = H // G
+        for b in range(B):
+            sl = int(state_slots[b])
+            st = state[sl].clone() if has_past and sl >= 0 else torch.zeros(H, D, V)
+            for t in range(int(n[b])):
+                r = b * S + t
+                kk, qq = k[r].repeat_interleave(rep, 0), q[r].repeat_interleave(rep, 0)
+                st = st * decay[r][:, None, None]
+                u = beta[r][:, None] * (v[r] - torch.einsum("hdv,hd->hv", st, kk))
+                st = st + kk[:, :, None] * u[:, None, :]
+                out[r] = torch.einsum("hdv,hd->hv", st, qq)
+            if sl >= 0:
+                state[sl] = st
+        return out
+    o = torch.empty((B * S, H, V), dtype=torch.float32, device=q.device)
+    check(_lib.lib().tfb_delta_scan(q.data_ptr(), k.data_ptr(), v.data_ptr(), kq.data_ptr(), decay.data_ptr(), beta.data_ptr(), o.data_ptr(),
+                                    state.data_ptr(), state_slots.data_ptr(), state.shape[0], ptr(lens), B, S, G, H, D, V, int(has_past),
+                                    stream()), "delta_scan")
+    return o
+
+
+def gated_norm(o, gate, w, eps):
+    """o [T, H, V] fp32 -> o / rms(o) * w * silu(gate), [T, H V] in the dtype of ``gate`` [T, H V]."""
+    T, H, V = o.shape
+    if not o.is_cuda:
+        g = gate.reshape(T, H, V).float()
+        y = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w.float() * (g * torch.sigmoid(g))
+        return y.reshape(T, H * V).to(gate.dtype)
+    out = rows(T, H * V, gate.dtype, o.device)
+    check(_lib.lib().tfb_gated_norm(o.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0), T, H, V, float(eps),
+                                    _f32(gate), stream()), "gated_norm")
+    return out
+
+
+def delta_step(prep, state, state_slots, gate, w, eps, B, G, H, D, V, has_past=True):
+    """One token per sequence with the gated norm of its output; [B, H V]."""
+    q, k, v, kq, decay, beta = prep
+    if not q.is_cuda or V % 4 or V > 256 or D > 256 or (V > 128 and D > 128):
+        return gated_norm(delta_scan(prep, state, state_slots, None, B, 1, G, H, D, V, has_past), gate, w, eps)
+    out = rows(B, H * V, gate.dtype, q.device)
+    check(_lib.lib().tfb_delta_step(q.data_ptr(), k.data_ptr(), v.data_ptr(), kq.data_ptr(), decay.data_ptr(), beta.data_ptr(), state.data_ptr(),
+                                    state_slots.data_ptr(), state.shape[0], gate.data_ptr(), gate.stride(0), w.data_ptr(), out.data_ptr(),
+                                    out.stride(0), B, G, H, D, V, int(has_past), float(eps), _f32(gate), stream()), "delta_step")
+    return out

@@ -269,8 +269,8 @@ def quantize_model_linears(model, fmt="int8", group=64, min_numel=1 << 14):
     """{parameter name: PackedWeight} for every matrix of the model's blocks (norms, embeddings and the head stay bf16)."""
     out = {}
     for i, l in enumerate(model.layers):
-        for name in ("qkv", "o", "gate_up", "down"):
-            w = getattr(l, name).data
+        for name, w in (l.linears if hasattr(l, "linears") else {n: getattr(l, n) for n in ("qkv", "o", "gate_up", "down")}).items():
+            w = w.data
             if w.numel() >= min_numel:
                 out[f"layers.{i}.{name}"] = pack_weight(w, fmt, group)
     return out

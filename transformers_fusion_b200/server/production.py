@@ -143,11 +143,11 @@ class ModelServer:
         """Build an engine for the checkpoint at ``path`` and serve from it (the previous engine is drained first)."""
         try:
             from ..inference.engine import EngineConfig, InferenceEngine
-            from ..quant import codec
+            from ..models import registry
             import torch
             old = self.engine
             dev = old.device if old is not None else ("cuda" if torch.cuda.is_available() else "cpu")
-            model = codec.load_model(path, device=dev, dtype=torch.bfloat16 if str(dev).startswith("cuda") else torch.float32)
+            model = registry.load_any(path, device=dev, dtype=torch.bfloat16 if str(dev).startswith("cuda") else torch.float32)
             eng = InferenceEngine(model, tokenizer or (old.tok if old is not None else None), engine_cfg or (old.cfg if old is not None else EngineConfig()))
         except Exception as e:
             self.last_error = str(e)
@@ -545,8 +545,8 @@ class ModelZoo:
     def get(self, name):
         if name not in self.loaded:
             import torch
-            from ..quant import codec
-            self.loaded[name] = codec.load_model(self.paths[name], device=self.device, dtype=self.dtype or torch.float32)
+            from ..models import registry
+            self.loaded[name] = registry.load_any(self.paths[name], device=self.device, dtype=self.dtype or torch.float32)
         return self.loaded[name]
 
     def unload(self, name):
