@@ -2,18 +2,28 @@
 //
 //   S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q            per head, S is [D, V] in fp32
 //
-// Three kernels:
-//   delta_prep   one block per token row: causal convolution of q, k and v over time (per channel, with the last inputs of
-//                the previous step as history), silu, unit length of q and k per head, the decay g and the step size beta.
-//                Everything it hands on is fp32.
-//   delta_scan   prompts.  The columns of S are independent recurrences that share k and q, so a group of TPC threads
-//                owns one column (D / TPC entries each, in registers as packed fp32 pairs) and walks over the tokens; k,
-//                q, v and the gates of the next tokens travel to shared memory (cp.async) while the current ones are used.
-//                S^T k and S^T q are taken from the same old state (o = g S^T q + (k.q) u), so a token has one reduction
-//                on its critical path instead of two.  The state never leaves the registers between tokens, and the
-//                arithmetic is fp32 FMA throughout: how a prompt is cut into portions changes nothing.
+// Kernels:
+//   delta_prep   one block per (strip of 8 tokens, head): causal convolution of q, k and v over time (per channel, with the last
+//                inputs of the previous step as history), silu, unit length of q and k per head, the decay g and the step
+//                size beta, and the dot products k_i.k_j, q_i.k_j of every four tokens.  Everything it hands on is fp32.
+//   delta_coef   per head and four tokens: those dot products times the decays between the tokens.
+//   delta_scan   prompts.  The columns of S are independent recurrences that share k and q, so a group of TPC threads owns CPT
+//                columns (D / TPC entries of each, in registers as packed fp32 pairs) and walks over the tokens four at a
+//                time.  With S the state before the four tokens and G_i, R_ij the products of the decays up to token i and
+//                between tokens j and i,
+//                    u_i = beta_i (v_i - G_i S^T k_i - sum_{j<i} R_ij (k_i.k_j) u_j)
+//                    o_i = G_i S^T q_i + sum_{j<=i} R_ij (q_i.k_j) u_j
+//                    S  <- G_4 S + sum_j R_4j k_j u_j^T
+//                which is the recurrence itself with its four reductions over D made one: all eight products with S are taken
+//                from the same old state, so four tokens have one shuffle reduction on their critical path.  k, q, v and the
+//                coefficients of the next tokens travel to shared memory (bulk copies) while the current ones are used; the
+//                state never leaves the registers between tokens, and the arithmetic is fp32 FMA throughout.
 //   delta_step   one token per sequence: one block per (sequence, head) streams the state through registers once (read,
 //                two products, rank-one update, write) and applies the gated norm of the head's output.
+//
+// Layouts of the prepared arrays (Sp: rows per sequence, S rounded up to 4, or 1 when decoding; Dp: D rounded up to the
+// register tile, tails zero; Vp: V rounded up to 4): q, k [B, G, Sp, Dp], v [B, H, Sp, Vp], decay, beta [B, H, Sp],
+// pair [B, G, Sp / 4, 16] (decoding: [B, G], k.q), coef [B, H, Sp / 4, 32].
 #include "tfb_elem.cuh"
 #include "tfb_host.h"
 
@@ -31,77 +41,146 @@ struct DeltaPrepArgs {
   const int* state_slots; // [B]; negative: no history is read or kept
   const void *A_log, *dt_bias;  // [H]
   const int* lens;        // [B] tokens of each sequence in this call (null: S)
-  float *q, *k, *v;       // [B*S, G, D], [B*S, G, D], [B*S, H, V]
-  float *kq;              // [B*S, G]: k . q
-  float *decay, *beta;    // [B*S, H]
-  int S, G, H, D, V, taps, has_past, nslots;
+  float *q, *k, *v, *decay, *beta, *pair;
+  int S, Sp, G, H, D, Dp, V, Vp, taps, has_past, nslots;
 };
 
-template <class T>
-__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaPrepArgs p) {
+constexpr int PREP_STRIP = 8;    // tokens per block (a multiple of 4)
+
+// One channel over the strip's tokens s0 .. s0 + n - 1: convolution, silu, emit(token in strip, value).  TAPS > 0: the window
+// moves through registers; TAPS = 0: any number of taps, inputs re-read.
+template <class T, int TAPS, class Emit>
+__device__ __forceinline__ void conv_channel(const DeltaPrepArgs& p, const T* __restrict__ x0, T* hist, bool past, int C, int c, int s0, int n,
+                                             Emit emit) {
+  const T* cw = static_cast<const T*>(p.conv_w) + (long long)c * p.taps;
+  auto input = [&](int s) -> float {     // token s of this call; negative: history
+    if (s >= 0) return to_f(x0[(long long)s * p.ld + c]);
+    return past ? to_f(hist[(long long)(p.taps - 1 + s) * C + c]) : 0.f;
+  };
+  if constexpr (TAPS > 0) {
+    float w[TAPS], win[TAPS];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = to_f(cw[j]);
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) win[j + 1] = input(s0 - (TAPS - 1) + j);
+    float cur[PREP_STRIP];
+#pragma unroll
+    for (int i = 0; i < PREP_STRIP; ++i) cur[i] = i < n ? to_f(x0[(long long)(s0 + i) * p.ld + c]) : 0.f;
+#pragma unroll
+    for (int i = 0; i < PREP_STRIP; ++i) {
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j) win[j] = win[j + 1];
+      win[TAPS - 1] = cur[i];
+      float y = 0.f;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) y = fmaf(w[j], win[j], y);
+      if (i < n) emit(i, silu_exact(y));
+    }
+  } else {
+    for (int i = 0; i < n; ++i) {
+      float y = 0.f;
+      for (int j = 0; j < p.taps; ++j) y = fmaf(to_f(cw[j]), input(s0 + i - (p.taps - 1) + j), y);
+      emit(i, silu_exact(y));
+    }
+  }
+  if (p.S == 1 && hist) {                // decoding: this thread alone uses channel c, so the window moves in place
+    const int m = p.taps - 1;
+    for (int j = 0; j < m - 1; ++j) hist[(long long)j * C + c] = past ? hist[(long long)(j + 1) * C + c] : from_f<T>(0.f);
+    hist[(long long)(m - 1) * C + c] = x0[c];
+  }
+}
+
+// blockIdx.y < G: the q and k heads of group blockIdx.y; otherwise v and the gates of head blockIdx.y - G
+template <class T, int TAPS>
+__global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaPrepArgs p) {
   tfb::pdl_sync();
-  extern __shared__ float sqk[];                      // 2 G D activated q and k channels
-  const int s = blockIdx.x, b = blockIdx.y, tid = threadIdx.x;
+  extern __shared__ float sqk[];         // [PREP_STRIP][2 Dp]
+  const int s0 = blockIdx.x * PREP_STRIP, b = blockIdx.z, tid = threadIdx.x, unit = blockIdx.y;
   const int len = p.lens ? p.lens[b] : p.S;
-  if (s >= len) return;
-  const long long r = (long long)b * p.S + s;
-  const int nqk = 2 * p.G * p.D, C = nqk + p.H * p.V, taps = p.taps;
-  const T* x = static_cast<const T*>(p.proj) + r * p.ld;
-  const T* cw = static_cast<const T*>(p.conv_w);
+  const int len4 = p.Sp == 1 ? len : (len + 3) / 4 * 4;       // rows len .. len4 - 1 become tokens that change nothing
+  if (s0 >= len4) return;
+  const int n = max(0, min(PREP_STRIP, len - s0)), n4 = min(PREP_STRIP, len4 - s0);
+  const T* x0 = static_cast<const T*>(p.proj) + (long long)b * p.S * p.ld;
+  const int C = 2 * p.G * p.D + p.H * p.V;
   int slot = p.state_slots ? p.state_slots[b] : -1;
   TFB_BOUNDS(slot < p.nslots, 71, slot, p.nslots);
   if (slot >= p.nslots) slot = -1;
-  T* hist = (slot >= 0 && taps > 1) ? static_cast<T*>(p.conv_state) + (long long)slot * (taps - 1) * C : nullptr;
+  T* hist = (slot >= 0 && p.taps > 1) ? static_cast<T*>(p.conv_state) + (long long)slot * (p.taps - 1) * C : nullptr;
   const bool past = hist && p.has_past;
-  for (int c = tid; c < C; c += blockDim.x) {
-    const float cur = to_f(x[c]);
-    float y = 0.f;
-    for (int j = 0; j < taps - 1; ++j) {
-      const int t = s - (taps - 1) + j;               // token index within this call; negative: history
-      float in = 0.f;
-      if (t >= 0) in = to_f(x[(long long)(t - s) * p.ld + c]);
-      else if (past) in = to_f(hist[(long long)(taps - 1 + t) * C + c]);
-      y = fmaf(to_f(cw[(long long)c * taps + j]), in, y);
+  if (unit >= p.G) {
+    const int h = unit - p.G;
+    float* vo = p.v + (((long long)b * p.H + h) * p.Sp + s0) * p.Vp;
+    for (int j = tid; j < p.V; j += 128)
+      conv_channel<T, TAPS>(p, x0, hist, past, C, 2 * p.G * p.D + h * p.V + j, s0, n, [&](int i, float y) { vo[(long long)i * p.Vp + j] = y; });
+    for (int i = tid; i < (n4 - n) * p.Vp; i += 128) vo[(long long)n * p.Vp + i] = 0.f;
+    if (tid < n4) {
+      const long long o = ((long long)b * p.H + h) * p.Sp + s0 + tid;
+      if (tid < n) {
+        const T* gb = x0 + (long long)(s0 + tid) * p.ld + C + p.H * p.V;
+        const float z = to_f(gb[p.H + h]) + to_f(static_cast<const T*>(p.dt_bias)[h]);
+        const float sp = z > 20.f ? z : log1pf(expf(z));
+        p.beta[o] = 1.f / (1.f + expf(-to_f(gb[h])));
+        p.decay[o] = expf(-expf(to_f(static_cast<const T*>(p.A_log)[h])) * sp);
+      } else {
+        p.beta[o] = 0.f;
+        p.decay[o] = 1.f;
+      }
     }
-    y = fmaf(to_f(cw[(long long)c * taps + taps - 1]), cur, y);
-    y = silu_exact(y);
-    if (c < nqk) sqk[c] = y;
-    else p.v[r * p.H * p.V + (c - nqk)] = y;
-    if (p.S == 1 && hist) {                           // decoding: this thread alone uses channel c, so the window moves in place
-      for (int j = 0; j < taps - 2; ++j) hist[(long long)j * C + c] = past ? hist[(long long)(j + 1) * C + c] : from_f<T>(0.f);
-      hist[(long long)(taps - 2) * C + c] = x[c];
-    }
+    return;
   }
-  const T* gb = x + C + p.H * p.V;
-  for (int h = tid; h < p.H; h += blockDim.x) {
-    const float bz = to_f(gb[h]);
-    const float z = to_f(gb[p.H + h]) + to_f(static_cast<const T*>(p.dt_bias)[h]);
-    const float sp = z > 20.f ? z : log1pf(expf(z));
-    p.beta[r * p.H + h] = 1.f / (1.f + expf(-bz));
-    p.decay[r * p.H + h] = expf(-expf(to_f(static_cast<const T*>(p.A_log)[h])) * sp);
+  const int g = unit, Dp = p.Dp;
+  for (int i = tid; i < n4 * 2 * Dp; i += 128) {            // rows without a token, and the tails of the others
+    const int r = i / (2 * Dp), d = i % Dp;
+    if (r >= n || d >= p.D) sqk[i] = 0.f;
+  }
+  for (int d = tid; d < p.D; d += 128) {
+    conv_channel<T, TAPS>(p, x0, hist, past, C, g * p.D + d, s0, n, [&](int i, float y) { sqk[i * 2 * Dp + d] = y; });
+    conv_channel<T, TAPS>(p, x0, hist, past, C, (p.G + g) * p.D + d, s0, n, [&](int i, float y) { sqk[i * 2 * Dp + Dp + d] = y; });
   }
   __syncthreads();
   const int warp = tid >> 5, lane = tid & 31;
-  for (int g = warp; g < p.G; g += blockDim.x >> 5) {
-    const float* sq = sqk + g * p.D;
-    const float* sk = sqk + (p.G + g) * p.D;
-    float qq = 0.f, kk = 0.f, qk = 0.f;
-    for (int d = lane; d < p.D; d += 32) {
+  for (int i = warp; i < n4; i += 4) {
+    float* sq = sqk + i * 2 * Dp;
+    float* sk = sq + Dp;
+    float qq = 0.f, kk = 0.f;
+    for (int d = lane; d < Dp; d += 32) {
       qq = fmaf(sq[d], sq[d], qq);
       kk = fmaf(sk[d], sk[d], kk);
-      qk = fmaf(sq[d], sk[d], qk);
     }
     qq = warp_add(qq);
     kk = warp_add(kk);
-    qk = warp_add(qk);
     const float rq = 1.f / sqrtf(qq + 1e-6f) / sqrtf(float(p.D)), rk = 1.f / sqrtf(kk + 1e-6f);
-    float* oq = p.q + (r * p.G + g) * p.D;
-    float* ok = p.k + (r * p.G + g) * p.D;
-    for (int d = lane; d < p.D; d += 32) {
-      oq[d] = sq[d] * rq;
-      ok[d] = sk[d] * rk;
+    const long long o = (((long long)b * p.G + g) * p.Sp + s0 + i) * Dp;
+    for (int d = lane; d < Dp; d += 32) {
+      const float a = sq[d] * rq, c = sk[d] * rk;
+      sq[d] = a;
+      sk[d] = c;
+      p.q[o + d] = a;
+      p.k[o + d] = c;
     }
-    if (lane == 0) p.kq[r * p.G + g] = qk * rq * rk;
+  }
+  __syncthreads();
+  auto dot = [&](const float* a, const float* c) {
+    float v = 0.f;
+    for (int d = lane; d < Dp; d += 32) v = fmaf(a[d], c[d], v);
+    return warp_add(v);
+  };
+  if (p.Sp == 1) {
+    if (warp == 0) {
+      const float v = dot(sqk, sqk + Dp);
+      if (lane == 0) p.pair[(long long)b * p.G + g] = v;
+    }
+    return;
+  }
+  // entries 0-5: k_i.k_j for (i, j) = 10 20 21 30 31 32; 6-15: q_i.k_j for 00 10 11 20 21 22 30 31 32 33
+  for (int e = warp; e < n4 / 4 * 16; e += 4) {
+    const int blk = e >> 4, x = e & 15;
+    const int y = x < 6 ? x : x - 6;
+    int i, j;
+    if (x < 6) { i = y < 1 ? 1 : y < 3 ? 2 : 3; j = y - (i * (i - 1)) / 2; }
+    else { i = y < 1 ? 0 : y < 3 ? 1 : y < 6 ? 2 : 3; j = y - (i * (i + 1)) / 2; }
+    const float v = dot(sqk + (blk * 4 + i) * 2 * Dp + (x < 6 ? Dp : 0), sqk + (blk * 4 + j) * 2 * Dp + Dp);
+    if (lane == 0) p.pair[(((long long)b * p.G + g) * (p.Sp / 4) + s0 / 4 + blk) * 16 + x] = v;
   }
 }
 
@@ -126,15 +205,58 @@ __global__ void __launch_bounds__(256) conv_history_kernel(const DeltaPrepArgs p
 }
 
 // ------------------------------------------------------------------------------------------------
+// coefficients of four tokens of one head: [0,6) beta_i R_ij (k_i.k_j), [6,16) R_ij (q_i.k_j), [16,20) beta_i,
+// [20,24) beta_i G_i, [24,28) G_i, [28,32) R_4j
+// ------------------------------------------------------------------------------------------------
+__global__ void __launch_bounds__(128) delta_coef_kernel(const float* __restrict__ pair, const float* __restrict__ decay,
+                                                         const float* __restrict__ beta, float* __restrict__ coef, const int* __restrict__ lens,
+                                                         int B, int S, int Sp, int G, int H) {
+  tfb::pdl_sync();
+  const int nb = Sp / 4;
+  const long long id = blockIdx.x * 128ll + threadIdx.x;
+  if (id >= (long long)B * H * nb) return;
+  const int blk = int(id % nb), h = int(id / nb % H), b = int(id / nb / H), g = h / (H / G);
+  if (blk * 4 >= (lens ? lens[b] : S)) return;
+  const float4 d4 = *reinterpret_cast<const float4*>(decay + ((long long)b * H + h) * Sp + blk * 4);
+  const float4 b4 = *reinterpret_cast<const float4*>(beta + ((long long)b * H + h) * Sp + blk * 4);
+  const float* pr = pair + (((long long)b * G + g) * nb + blk) * 16;
+  const float d[4] = {d4.x, d4.y, d4.z, d4.w}, be[4] = {b4.x, b4.y, b4.z, b4.w};
+  float R[4][4], c[32];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    R[j][j] = 1.f;
+#pragma unroll
+    for (int i = j + 1; i < 4; ++i) R[i][j] = R[i - 1][j] * d[i];
+  }
+  float Gi = 1.f;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    Gi *= d[i];
+#pragma unroll
+    for (int j = 0; j < i; ++j) c[i * (i - 1) / 2 + j] = be[i] * R[i][j] * pr[i * (i - 1) / 2 + j];
+#pragma unroll
+    for (int j = 0; j <= i; ++j) c[6 + i * (i + 1) / 2 + j] = R[i][j] * pr[6 + i * (i + 1) / 2 + j];
+    c[16 + i] = be[i];
+    c[20 + i] = be[i] * Gi;
+    c[24 + i] = Gi;
+    c[28 + i] = R[3][i];
+  }
+  float4* out = reinterpret_cast<float4*>(coef + id * 32);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) out[i] = make_float4(c[4 * i], c[4 * i + 1], c[4 * i + 2], c[4 * i + 3]);
+}
+
+// ------------------------------------------------------------------------------------------------
 // scan over a prompt
 // ------------------------------------------------------------------------------------------------
 struct DeltaScanArgs {
-  const float *q, *k, *v, *kq, *decay, *beta;
+  const float *q, *k, *v, *coef;
   float* o;               // [B*S, H, V]
   float* state;           // [slots, H, D, V]
   const int* state_slots; // [B]
   const int* lens;        // [B] or null
-  int S, G, H, D, V, has_past, nslots;
+  int S, Sp, G, H, D, V, Vp, has_past, nslots;
+  int* status;
 };
 
 typedef unsigned long long u64;
@@ -148,6 +270,11 @@ __device__ __forceinline__ u64 mul2(u64 a, u64 b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
 }
+__device__ __forceinline__ u64 add2(u64 a, u64 b) {
+  u64 d;
+  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
 __device__ __forceinline__ u64 pack2(float lo, float hi) {
   u64 d;
   asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
@@ -158,164 +285,226 @@ __device__ __forceinline__ float2 unpack2(u64 v) {
   asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
   return f;
 }
-__device__ __forceinline__ void cp_async_bytes16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_bytes4(uint32_t dst, const void* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory");
-}
 
 constexpr int SCAN_CHUNK = 16;   // tokens per shared-memory stage
 
-// EPT: entries of one column per thread (a multiple of 4); TPC: threads per column; D <= EPT * TPC.
-// Shared memory per stage: k, q [CHUNK][Dp] (Dp = EPT * TPC, the tail is zero), v [CHUNK][cols], and 3 scalars per token.
-template <int EPT, int TPC>
-__global__ void delta_scan_kernel(const DeltaScanArgs p) {
+// EPT: entries of one column per thread (a multiple of 4); TPC: threads per column group; CPT: columns per group (a power of
+// two, 2 CPT <= TPC); Dp = EPT TPC.  Of a group's 2 CPT sets of products (S^T k and S^T q of each column, four tokens each) a
+// shuffle reduction leaves one set with each thread (or with each TPC / (2 CPT) threads): bits of the thread index, from the
+// top: column, then k or q.
+template <int EPT, int TPC, int CPT>
+__global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaScanArgs p) {
   tfb::pdl_sync();
-  extern __shared__ __align__(16) float sm[];
-  constexpr int Dp = EPT * TPC, CPW = 32 / TPC;
-  const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31;
-  const int cols = (nt >> 5) * CPW;
+  extern __shared__ __align__(128) float sm[];
+  constexpr int Dp = EPT * TPC, CPW = 32 / TPC * CPT, SETS = 2 * CPT, W = TPC / SETS;
+  static_assert(SETS <= TPC && EPT % 4 == 0, "tile shape");
+  const int tid = threadIdx.x, lane = tid & 31, cols = (blockDim.x >> 5) * CPW;
   const int h = blockIdx.y, b = blockIdx.z, g = h / (p.H / p.G), col0 = blockIdx.x * cols;
-  const int cl = (tid >> 5) * CPW + lane / TPC, t = lane % TPC, col = col0 + cl;
-  const bool live = col < p.V;
+  const int t = lane % TPC, cl = (tid >> 5) * CPW + lane / TPC * CPT;      // first column of the group, within the block
+  const int set = t / W, my_col = col0 + cl + (set >> 1);                   // the products this thread ends up with
+  const bool is_q = set & 1;
   const int len = p.lens ? p.lens[b] : p.S;
-  const long long r0 = (long long)b * p.S;
-  const int stage_f = 2 * SCAN_CHUNK * Dp + SCAN_CHUNK * cols + 4 * SCAN_CHUNK;
-  const bool vec_d = (p.D & 3) == 0, vec_v = (p.V & 3) == 0 && (cols & 3) == 0;
-  const int cshift = 31 - __clz(cols);      // cols is a power of two
+  const int stage_f = 2 * SCAN_CHUNK * Dp + SCAN_CHUNK * cols + SCAN_CHUNK * 8;
+  const uint32_t bar = smem_u32(sm + 2 * stage_f);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + 2 * stage_f + 4);
+  if (tid == 0) {
+    mbar_init(bar, 1);
+    mbar_init(bar + 8, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  for (int i = tid; i < 2 * stage_f; i += blockDim.x) sm[i] = 0.f;        // columns past V stay zero
+  fence_proxy_async_smem();
+  __syncthreads();
+  const float* kb = p.k + ((long long)b * p.G + g) * p.Sp * Dp;
+  const float* qb = p.q + ((long long)b * p.G + g) * p.Sp * Dp;
+  const float* vb = p.v + ((long long)b * p.H + h) * p.Sp * p.Vp + col0;
+  const float* cb = p.coef + ((long long)b * p.H + h) * (p.Sp / 4) * 32;
+  const int nrow = (len + 3) / 4 * 4, nc = min(cols, p.Vp - col0);
+  auto issue = [&](int c) {              // warp 0: the rows of chunk c (whole groups of four)
+    const int s0 = c * SCAN_CHUNK, n = min(SCAN_CHUNK, nrow - s0);
+    if (n <= 0 || tid >= 32) return;
+    float* base = sm + (c & 1) * stage_f;
+    const uint32_t br = bar + (c & 1) * 8;
+    if (lane == 0) mbar_expect_tx(br, uint32_t(n) * (2 * Dp + nc + 8) * 4);
+    __syncwarp();
+    if (lane == 0) bulk_load(smem_u32(base), kb + (long long)s0 * Dp, n * Dp * 4, br);
+    if (lane == 1) bulk_load(smem_u32(base + SCAN_CHUNK * Dp), qb + (long long)s0 * Dp, n * Dp * 4, br);
+    if (lane == 2) bulk_load(smem_u32(base + 2 * SCAN_CHUNK * Dp + SCAN_CHUNK * cols), cb + (long long)s0 * 8, n * 32, br);
+    if (lane >= 16 && lane - 16 < n)
+      bulk_load(smem_u32(base + 2 * SCAN_CHUNK * Dp + (lane - 16) * cols), vb + (long long)(s0 + lane - 16) * p.Vp, nc * 4, br);
+  };
+  issue(0);
+  issue(1);
 
-  for (int i = tid; i < 2 * stage_f; i += nt) sm[i] = 0.f;      // tails of k and q stay zero
   int slot = p.state_slots ? p.state_slots[b] : -1;
   TFB_BOUNDS(slot < p.nslots, 72, slot, p.nslots);
   if (slot >= p.nslots) slot = -1;
   float* S0 = slot >= 0 ? p.state + ((long long)slot * p.H + h) * p.D * p.V : nullptr;
-  // entry d of the column sits with thread (d / 4) % TPC, register (d / 4) / TPC * 4 + d % 4
-  u64 st[EPT / 2];
+  // entry d of a column sits with thread (d / 4) % TPC, register (d / 4) / TPC * 4 + d % 4
+  u64 st[CPT][EPT / 2];
 #pragma unroll
-  for (int i = 0; i < EPT / 4; ++i) {
-    float f[4];
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int d = (i * TPC + t) * 4 + e;
-      f[e] = (S0 && p.has_past && live && d < p.D) ? S0[(long long)d * p.V + col] : 0.f;
-    }
-    st[2 * i] = pack2(f[0], f[1]);
-    st[2 * i + 1] = pack2(f[2], f[3]);
-  }
-  __syncthreads();
-
-  auto issue = [&](int c) {
-    const int s0 = c * SCAN_CHUNK, n = min(SCAN_CHUNK, len - s0);
-    float* base = sm + (c & 1) * stage_f;
-    if (n > 0) {
-      constexpr int QV = Dp / 4;                                 // index arithmetic in powers of two
-      for (int i = tid; i < 2 * SCAN_CHUNK * QV; i += nt) {
-        const int w = i / (SCAN_CHUNK * QV), tk = (i / QV) % SCAN_CHUNK, d = (i % QV) * 4;
-        if (tk >= n || d >= p.D) continue;
-        const float* src = (w ? p.q : p.k) + ((r0 + s0 + tk) * p.G + g) * p.D + d;
-        const uint32_t dst = smem_u32(base + (w * SCAN_CHUNK + tk) * Dp + d);
-        if (vec_d) cp_async_bytes16(dst, src);
-        else
-          for (int e = 0; e < min(4, p.D - d); ++e) cp_async_bytes4(dst + 4 * e, src + e);
-      }
-      float* sv = base + 2 * SCAN_CHUNK * Dp;
-      const int vs = vec_v ? cshift - 2 : cshift;
-      for (int i = tid; i < (SCAN_CHUNK << vs); i += nt) {
-        const int tk = i >> vs, j = (i & ((1 << vs) - 1)) << (cshift - vs);
-        if (tk >= n || col0 + j >= p.V) continue;
-        const float* src = p.v + ((r0 + s0 + tk) * p.H + h) * p.V + col0 + j;
-        if (vec_v) cp_async_bytes16(smem_u32(sv + tk * cols + j), src);
-        else cp_async_bytes4(smem_u32(sv + tk * cols + j), src);
-      }
-      float* sg = sv + SCAN_CHUNK * cols;
-      for (int i = tid; i < 4 * SCAN_CHUNK; i += nt) {
-        const int tk = i >> 2, w = i & 3;
-        if (tk >= n || w == 3) continue;
-        const float* src = w == 0 ? p.decay + (r0 + s0 + tk) * p.H + h : w == 1 ? p.beta + (r0 + s0 + tk) * p.H + h : p.kq + (r0 + s0 + tk) * p.G + g;
-        cp_async_bytes4(smem_u32(sg + tk * 4 + w), src);
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-
-  const int nchunk = (len + SCAN_CHUNK - 1) / SCAN_CHUNK;
-  issue(0);
-  for (int c = 0; c < nchunk; ++c) {
-    issue(c + 1);
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
-    __syncthreads();
-    const float* base = sm + (c & 1) * stage_f;
-    const float* sv = base + 2 * SCAN_CHUNK * Dp;
-    const float* sg = sv + SCAN_CHUNK * cols;
-    const int n = min(SCAN_CHUNK, len - c * SCAN_CHUNK);
-    float* orow = p.o + ((r0 + c * SCAN_CHUNK) * p.H + h) * p.V + col;
-#pragma unroll 2
-    for (int tk = 0; tk < n; ++tk) {
-      const ulonglong2* sk = reinterpret_cast<const ulonglong2*>(base + tk * Dp) + t;
-      const ulonglong2* sq = reinterpret_cast<const ulonglong2*>(base + (SCAN_CHUNK + tk) * Dp) + t;
-      const float4 gs = *reinterpret_cast<const float4*>(sg + tk * 4);     // decay, beta, k.q
-      const float v = sv[tk * cols + cl];
-      u64 kk[EPT / 2];
-      u64 dk0 = 0, dk1 = 0, dq0 = 0, dq1 = 0;
-#pragma unroll
-      for (int i = 0; i < EPT / 4; ++i) {
-        const ulonglong2 a = sk[i * TPC], q = sq[i * TPC];
-        kk[2 * i] = a.x;
-        kk[2 * i + 1] = a.y;
-        dk0 = fma2(st[2 * i], a.x, dk0);
-        dk1 = fma2(st[2 * i + 1], a.y, dk1);
-        dq0 = fma2(st[2 * i], q.x, dq0);
-        dq1 = fma2(st[2 * i + 1], q.y, dq1);
-      }
-      const float2 ka = unpack2(dk0), kb = unpack2(dk1), qa = unpack2(dq0), qb = unpack2(dq1);
-      float dk = (ka.x + ka.y) + (kb.x + kb.y), dq = (qa.x + qa.y) + (qb.x + qb.y);
-#pragma unroll
-      for (int o = TPC >> 1; o > 0; o >>= 1) {
-        dk += __shfl_xor_sync(0xffffffffu, dk, o);
-        dq += __shfl_xor_sync(0xffffffffu, dq, o);
-      }
-      const float u = gs.y * (v - gs.x * dk);
-      const u64 uu = pack2(u, u), gg = pack2(gs.x, gs.x);
-#pragma unroll
-      for (int i = 0; i < EPT / 2; ++i) st[i] = fma2(kk[i], uu, mul2(st[i], gg));
-      if (t == 0 && live) orow[(long long)tk * p.H * p.V] = fmaf(gs.x, dq, gs.z * u);
-    }
-    __syncthreads();
-  }
-  if (S0 && live) {
+  for (int x = 0; x < CPT; ++x)
 #pragma unroll
     for (int i = 0; i < EPT / 4; ++i) {
-      const float2 a = unpack2(st[2 * i]), c = unpack2(st[2 * i + 1]);
-      const float f[4] = {a.x, a.y, c.x, c.y};
+      float f[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int d = (i * TPC + t) * 4 + e;
-        if (d < p.D) S0[(long long)d * p.V + col] = f[e];
+        const int d = (i * TPC + t) * 4 + e, col = col0 + cl + x;
+        f[e] = (S0 && p.has_past && col < p.V && d < p.D) ? S0[(long long)d * p.V + col] : 0.f;
+      }
+      st[x][2 * i] = pack2(f[0], f[1]);
+      st[x][2 * i + 1] = pack2(f[2], f[3]);
+    }
+
+  const int nchunk = (len + SCAN_CHUNK - 1) / SCAN_CHUNK;
+  const long long ostep = (long long)p.H * p.V;
+  float* orow = p.o + ((long long)b * p.S * p.H + h) * p.V + my_col;
+  const bool writer = is_q && t % W == 0 && my_col < p.V;
+  for (int c = 0; c < nchunk; ++c) {
+    if (!mbar_wait_warp(bar + (c & 1) * 8, (c >> 1) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) break;
+    const float* base = sm + (c & 1) * stage_f;
+    const float* sv = base + 2 * SCAN_CHUNK * Dp;
+    const float* sc = sv + SCAN_CHUNK * cols;
+    const int n = min(SCAN_CHUNK, len - c * SCAN_CHUNK);
+#pragma unroll 1
+    for (int r = 0; r < n; r += 4) {
+      u64 kk[4][EPT / 2];
+      float val[SETS][4];                // [2 column + (k: 0, q: 1)][token]
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const ulonglong2* sk = reinterpret_cast<const ulonglong2*>(base + (r + i) * Dp) + t;
+        const ulonglong2* sq = reinterpret_cast<const ulonglong2*>(base + (SCAN_CHUNK + r + i) * Dp) + t;
+        u64 qq[EPT / 2];
+#pragma unroll
+        for (int e = 0; e < EPT / 4; ++e) {
+          const ulonglong2 a = sk[e * TPC], q = sq[e * TPC];
+          kk[i][2 * e] = a.x;
+          kk[i][2 * e + 1] = a.y;
+          qq[2 * e] = q.x;
+          qq[2 * e + 1] = q.y;
+        }
+#pragma unroll
+        for (int x = 0; x < CPT; ++x) {
+          u64 dk0 = mul2(st[x][0], kk[i][0]), dk1 = mul2(st[x][1], kk[i][1]);
+          u64 dq0 = mul2(st[x][0], qq[0]), dq1 = mul2(st[x][1], qq[1]);
+#pragma unroll
+          for (int e = 2; e < EPT / 2; e += 2) {
+            dk0 = fma2(st[x][e], kk[i][e], dk0);
+            dk1 = fma2(st[x][e + 1], kk[i][e + 1], dk1);
+            dq0 = fma2(st[x][e], qq[e], dq0);
+            dq1 = fma2(st[x][e + 1], qq[e + 1], dq1);
+          }
+          const float2 a = unpack2(add2(dk0, dk1)), q = unpack2(add2(dq0, dq1));
+          val[2 * x][i] = a.x + a.y;
+          val[2 * x + 1][i] = q.x + q.y;
+        }
+      }
+#pragma unroll
+      for (int o = TPC >> 1, m = SETS; o > 0; o >>= 1) {
+        if (m > 1) {                     // halve the sets: keep those of this thread's half, send the others
+          const bool up = t & o;
+#pragma unroll
+          for (int y = 0; y < m / 2; ++y)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float send = up ? val[y][i] : val[y + m / 2][i], keep = up ? val[y + m / 2][i] : val[y][i];
+              val[y][i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+          m >>= 1;
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) val[0][i] += __shfl_xor_sync(0xffffffffu, val[0][i], o);
+        }
+      }
+      const float4* cf = reinterpret_cast<const float4*>(sc + r * 8);
+      const float4 c0 = cf[0], c1 = cf[1], c2 = cf[2], c3 = cf[3], be = cf[4], bg = cf[5], gi = cf[6], r4 = cf[7];
+      float u[4];                        // right in the threads that hold a k set
+      {
+        const float* vr = sv + r * cols + cl + (set >> 1);
+        u[0] = fmaf(be.x, vr[0], -bg.x * val[0][0]);
+        u[1] = fmaf(-c0.x, u[0], fmaf(be.y, vr[cols], -bg.y * val[0][1]));
+        u[2] = fmaf(-c0.z, u[1], fmaf(-c0.y, u[0], fmaf(be.z, vr[2 * cols], -bg.z * val[0][2])));
+        u[3] = fmaf(-c1.y, u[2], fmaf(-c1.x, u[1], fmaf(-c0.w, u[0], fmaf(be.w, vr[3 * cols], -bg.w * val[0][3]))));
+      }
+      const u64 g4 = pack2(gi.w, gi.w);
+      float mine[4] = {0.f, 0.f, 0.f, 0.f};      // u of this thread's column
+#pragma unroll
+      for (int x = 0; x < CPT; ++x) {
+        float w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          w[i] = __shfl_sync(0xffffffffu, u[i], (lane & ~(TPC - 1)) + 2 * x * W);
+          if (CPT == 1 || (set >> 1) == x) mine[i] = w[i];
+        }
+        const u64 w0 = pack2(w[0] * r4.x, w[0] * r4.x), w1 = pack2(w[1] * r4.y, w[1] * r4.y);
+        const u64 w2 = pack2(w[2] * r4.z, w[2] * r4.z), w3 = pack2(w[3] * r4.w, w[3] * r4.w);
+#pragma unroll
+        for (int e = 0; e < EPT / 2; ++e)
+          st[x][e] = fma2(kk[3][e], w3, fma2(kk[2][e], w2, fma2(kk[1][e], w1, fma2(kk[0][e], w0, mul2(st[x][e], g4)))));
+      }
+      if (writer) {
+        float* op = orow + (long long)(c * SCAN_CHUNK + r) * ostep;
+        op[0] = fmaf(c1.z, mine[0], gi.x * val[0][0]);
+        if (r + 1 < n) op[ostep] = fmaf(c2.x, mine[1], fmaf(c1.w, mine[0], gi.y * val[0][1]));
+        if (r + 2 < n) op[2 * ostep] = fmaf(c2.w, mine[2], fmaf(c2.z, mine[1], fmaf(c2.y, mine[0], gi.z * val[0][2])));
+        if (r + 3 < n)
+          op[3 * ostep] = fmaf(c3.w, mine[3], fmaf(c3.z, mine[2], fmaf(c3.y, mine[1], fmaf(c3.x, mine[0], gi.w * val[0][3]))));
       }
     }
+    __syncthreads();
+    issue(c + 2);
   }
+  if (*abort_flag) {                     // a copy never landed: the status word says so, the state is left alone
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) {}      // bounded wait for copies already issued
+    return;
+  }
+  if (S0) {
+#pragma unroll
+    for (int x = 0; x < CPT; ++x)
+#pragma unroll
+      for (int i = 0; i < EPT / 4; ++i) {
+        const float2 a = unpack2(st[x][2 * i]), c = unpack2(st[x][2 * i + 1]);
+        const float f[4] = {a.x, a.y, c.x, c.y};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int d = (i * TPC + t) * 4 + e, col = col0 + cl + x;
+          if (d < p.D && col < p.V) S0[(long long)d * p.V + col] = f[e];
+        }
+      }
+  }
+}
+
+template <int EPT, int TPC, int CPT>
+static int launch_scan_tile(const DeltaScanArgs& p, int B, int nw, cudaStream_t st) {
+  constexpr int CPW = 32 / TPC * CPT;
+  auto bytes = [](int w) { return (2 * (2 * SCAN_CHUNK * EPT * TPC + SCAN_CHUNK * w * CPW + SCAN_CHUNK * 8) + 8) * int(sizeof(float)); };
+  static DeviceOnce once;
+  auto kern = delta_scan_kernel<EPT, TPC, CPT>;
+  if (int e = ensure_dyn_smem(once, kern, bytes(4))) return e;
+  const int cols = nw * CPW;
+  launch_k(kern, dim3((p.V + cols - 1) / cols, p.H, B), nw * 32, bytes(nw), st, p);
+  return int(cudaGetLastError());
 }
 
 template <int EPT, int TPC>
 static int launch_scan(const DeltaScanArgs& p, int B, cudaStream_t st) {
-  // warps per block: few blocks leave SMs idle when there is one sequence, many small blocks fetch k and q more often
+  // Wide groups (four columns) read k and q from shared memory a quarter as often; narrow ones spread few sequences over more
+  // warps.  A scheduler wants at least one warp either way.
+  constexpr int CPW4 = 32 / TPC * 4, CPW1 = 32 / TPC;
+  const long long warps4 = (long long)((p.V + CPW4 - 1) / CPW4) * p.H * B;
+  if (warps4 >= 3ll * sm_count()) return launch_scan_tile<EPT, TPC, 4>(p, B, 4, st);
   int nw = 4;
-  const int cpw = 32 / TPC;
-  while (nw > 1 && (long long)((p.V + nw * cpw - 1) / (nw * cpw)) * p.H * B < sm_count()) nw >>= 1;
-  const int cols = nw * cpw;
-  const int smem = 2 * (2 * SCAN_CHUNK * EPT * TPC + SCAN_CHUNK * cols + 4 * SCAN_CHUNK) * int(sizeof(float));
-  static DeviceOnce once;
-  auto kern = delta_scan_kernel<EPT, TPC>;
-  if (int e = ensure_dyn_smem(once, kern, 2 * (2 * SCAN_CHUNK * EPT * TPC + SCAN_CHUNK * 4 * cpw + 4 * SCAN_CHUNK) * int(sizeof(float)))) return e;
-  launch_k(kern, dim3((p.V + cols - 1) / cols, p.H, B), nw * 32, smem, st, p);
-  return int(cudaGetLastError());
+  while (nw * CPW1 > 4 && (nw * CPW1 > 4 * ((p.V + 3) / 4) ||      // at least four columns: rows of v are copied in 16-byte pieces
+                           (long long)((p.V + nw * CPW1 - 1) / (nw * CPW1)) * p.H * B < sm_count())) nw >>= 1;
+  return launch_scan_tile<EPT, TPC, 1>(p, B, nw, st);
 }
 
 // ------------------------------------------------------------------------------------------------
 // gated norm of the head outputs:  o / rms(o) * w * silu(gate)
 // ------------------------------------------------------------------------------------------------
-template <class T>
+template <class T, int VEC>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ldg,
                                                          const T* __restrict__ w, T* __restrict__ out, long long ldo, int rows, int H, int V,
                                                          float eps) {
@@ -326,21 +515,51 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
     const long long r = i / H;
     const int h = int(i % H);
     const float* src = o + i * V;
+    const T* gt = gate + r * ldg + h * V;
+    T* dst = out + r * ldo + h * V;
+    float x0[VEC], g0[VEC], x[VEC], g[VEC], wv[VEC];
     float ss = 0.f;
-    for (int j = lane; j < V; j += 32) ss = fmaf(src[j], src[j], ss);
+    for (int j = lane * VEC; j < V; j += 32 * VEC) {
+      load_n<VEC>(src + j, x);
+      if (j == lane * VEC) {
+        load_n<VEC>(gt + j, g0);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x0[e] = x[e];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss = fmaf(x[e], x[e], ss);
+    }
     const float rs = 1.f / sqrtf(warp_add(ss) / V + eps);
-    for (int j = lane; j < V; j += 32)
-      out[r * ldo + h * V + j] = from_f<T>(src[j] * rs * to_f(w[j]) * silu_exact(to_f(gate[r * ldg + h * V + j])));
+    for (int j = lane * VEC; j < V; j += 32 * VEC) {
+      load_n<VEC>(w + j, wv);
+      if (j == lane * VEC) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { x[e] = x0[e]; g[e] = g0[e]; }
+      } else {
+        load_n<VEC>(src + j, x);
+        load_n<VEC>(gt + j, g);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] = x[e] * rs * wv[e] * silu_exact(g[e]);
+      store_n<VEC>(dst + j, x);
+    }
   }
 }
 
 // ------------------------------------------------------------------------------------------------
 // one token per sequence
 // ------------------------------------------------------------------------------------------------
+struct DeltaStepArgs {
+  const float *q, *k, *v, *kq, *decay, *beta;   // Sp = 1 layouts: [B, G, Dp], [B, G, Dp], [B, H, Vp], [B, G], [B, H], [B, H]
+  float* state;
+  const int* state_slots;
+  int G, H, D, Dp, V, Vp, has_past, nslots;
+};
+
 // 256 threads = 8 warps; warp w holds rows w, w + 8, ... (NR of them) of the state, lane l the columns 4 l .. 4 l + 3 of
 // each 128-column part.  D <= 8 NR, V <= 128 CV, V % 4 == 0.
 template <class T, int NR, int CV>
-__global__ void __launch_bounds__(256) delta_step_kernel(const DeltaScanArgs p, const T* __restrict__ gate, long long ldg,
+__global__ void __launch_bounds__(256) delta_step_kernel(const DeltaStepArgs p, const T* __restrict__ gate, long long ldg,
                                                          const T* __restrict__ w, T* __restrict__ out, long long ldo, float eps) {
   tfb::pdl_sync();
   constexpr int VM = 128 * CV;
@@ -359,8 +578,8 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaScanArgs p, 
       s[i][c] = (S0 && p.has_past && d < p.D && j < p.V) ? *reinterpret_cast<const float4*>(S0 + (long long)d * p.V + j) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   for (int d = tid; d < 8 * NR; d += 256) {
-    sk[d] = d < p.D ? p.k[((long long)b * p.G + g) * p.D + d] : 0.f;
-    sq[d] = d < p.D ? p.q[((long long)b * p.G + g) * p.D + d] : 0.f;
+    sk[d] = d < p.D ? p.k[((long long)b * p.G + g) * p.Dp + d] : 0.f;
+    sq[d] = d < p.D ? p.q[((long long)b * p.G + g) * p.Dp + d] : 0.f;
   }
   const float dec = p.decay[(long long)b * p.H + h], bet = p.beta[(long long)b * p.H + h], kq = p.kq[(long long)b * p.G + g];
   __syncthreads();
@@ -386,7 +605,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaScanArgs p, 
       dk += red_k[i][tid];
       dq += red_q[i][tid];
     }
-    const float u = bet * (p.v[((long long)b * p.H + h) * p.V + tid] - dec * dk);
+    const float u = bet * (p.v[((long long)b * p.H + h) * p.Vp + tid] - dec * dk);
     su[tid] = u;
     ov = fmaf(dec, dq, kq * u);
   } else if (tid < VM) {
@@ -416,7 +635,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const DeltaScanArgs p, 
 }
 
 template <class T>
-static int launch_step(const DeltaScanArgs& p, int B, const void* gate, long long ldg, const void* w, void* out, long long ldo, float eps,
+static int launch_step(const DeltaStepArgs& p, int B, const void* gate, long long ldg, const void* w, void* out, long long ldo, float eps,
                        cudaStream_t st) {
   const T* gt = static_cast<const T*>(gate);
   const T* wt = static_cast<const T*>(w);
@@ -440,47 +659,64 @@ static int launch_step(const DeltaScanArgs& p, int B, const void* gate, long lon
 
 using bf16 = __nv_bfloat16;
 
-// Convolution, activation, unit lengths and gates of B sequences with S rows each (lens[b] of them real).  has_past: the
-// history in conv_state belongs to these sequences (otherwise they start here and see zeros).
+// entries per key head in the prepared arrays (0: the head size is not supported)
+TFB_API int tfb_delta_padded_dim(int D) {
+  for (int d = 32; d <= 512; d *= 2)
+    if (D <= d) return d;
+  return 0;
+}
+
+// Convolution, activation, unit lengths, gates and (Sp > 1) the coefficients of B sequences with S rows each, lens[b] of them
+// real.  has_past: the history in conv_state belongs to these sequences (otherwise they start here and see zeros).
 TFB_API int tfb_delta_prep(const void* proj, long long ld, const void* conv_w, void* conv_state, const int* state_slots, int nslots,
-                           const void* A_log, const void* dt_bias, const int* lens, float* q, float* k, float* v, float* kq, float* decay,
-                           float* beta, int B, int S, int G, int H, int D, int V, int taps, int has_past, int f32, void* stream) {
+                           const void* A_log, const void* dt_bias, const int* lens, float* q, float* k, float* v, float* decay, float* beta,
+                           float* pair, float* coef, int B, int S, int Sp, int G, int H, int D, int V, int taps, int has_past, int f32,
+                           void* stream) {
   using namespace tfb;
-  if (B <= 0 || B > 65535 || S <= 0 || G <= 0 || H % G || D <= 0 || V <= 0 || taps < 1) return TFB_ERR_ARG;
-  const int smem = 2 * G * D * int(sizeof(float));
-  if (smem > 200 * 1024) return TFB_ERR_LIMIT;
-  DeltaPrepArgs p{proj, ld, conv_w, conv_state, state_slots, A_log, dt_bias, lens, q, k, v, kq, decay, beta, S, G, H, D, V, taps, has_past, nslots};
+  const int Dp = tfb_delta_padded_dim(D);
+  if (B <= 0 || B > 65535 || S <= 0 || G <= 0 || H % G || G + H > 65535 || D <= 0 || V <= 0 || taps < 1) return TFB_ERR_ARG;
+  if (Sp != 1 && (Sp != (S + 3) / 4 * 4 || !coef)) return TFB_ERR_ARG;
+  if (Sp == 1 && S != 1) return TFB_ERR_ARG;
+  if (!Dp) return TFB_ERR_LIMIT;
+  DeltaPrepArgs p{proj, ld, conv_w, conv_state, state_slots, A_log, dt_bias, lens, q, k, v, decay, beta, pair,
+                  S, Sp, G, H, D, Dp, V, (V + 3) / 4 * 4, taps, has_past, nslots};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  static DeviceOnce once16, once32;
-  if (f32) {
-    if (int e = ensure_dyn_smem(once32, delta_prep_kernel<float>, 200 * 1024)) return e;
-    launch_k(delta_prep_kernel<float>, dim3(S, B), 256, smem, st, p);
-  } else {
-    if (int e = ensure_dyn_smem(once16, delta_prep_kernel<bf16>, 200 * 1024)) return e;
-    launch_k(delta_prep_kernel<bf16>, dim3(S, B), 256, smem, st, p);
+  const dim3 grid((Sp + PREP_STRIP - 1) / PREP_STRIP, G + H, B);
+  const int smem = (Sp == 1 ? 1 : PREP_STRIP) * 2 * Dp * int(sizeof(float));     // at most 32 KB
+#define TFB_PREP(T)                                                                       \
+  switch (taps) {                                                                         \
+    case 2: launch_k(delta_prep_kernel<T, 2>, grid, 128, smem, st, p); break;             \
+    case 3: launch_k(delta_prep_kernel<T, 3>, grid, 128, smem, st, p); break;             \
+    case 4: launch_k(delta_prep_kernel<T, 4>, grid, 128, smem, st, p); break;             \
+    default: launch_k(delta_prep_kernel<T, 0>, grid, 128, smem, st, p); break;            \
   }
+  if (f32) { TFB_PREP(float) } else { TFB_PREP(bf16) }
+#undef TFB_PREP
   if (S > 1 && taps > 1 && state_slots) {
-    const dim3 grid((2 * G * D + H * V + 255) / 256, B);
-    if (f32) launch_k(conv_history_kernel<float>, grid, 256, 0, st, p);
-    else launch_k(conv_history_kernel<bf16>, grid, 256, 0, st, p);
+    const dim3 hg((2 * G * D + H * V + 255) / 256, B);
+    if (f32) launch_k(conv_history_kernel<float>, hg, 256, 0, st, p);
+    else launch_k(conv_history_kernel<bf16>, hg, 256, 0, st, p);
   }
+  if (Sp > 1)
+    launch_k(delta_coef_kernel, int(((long long)B * H * (Sp / 4) + 127) / 128), 128, 0, st, pair, decay, beta, coef, lens, B, S, Sp, G, H);
   return int(cudaGetLastError());
 }
 
-// The recurrence over the prepared rows; o [B*S, H, V] fp32.
-TFB_API int tfb_delta_scan(const float* q, const float* k, const float* v, const float* kq, const float* decay, const float* beta, float* o,
-                           float* state, const int* state_slots, int nslots, const int* lens, int B, int S, int G, int H, int D, int V,
-                           int has_past, void* stream) {
+// The recurrence over the prepared rows (Sp > 1); o [B*S, H, V] fp32.
+TFB_API int tfb_delta_scan(const float* q, const float* k, const float* v, const float* coef, float* o, float* state, const int* state_slots,
+                           int nslots, const int* lens, int B, int S, int G, int H, int D, int V, int has_past, int* status, void* stream) {
   using namespace tfb;
   if (B <= 0 || B > 65535 || S <= 0 || G <= 0 || H % G || H > 65535 || D <= 0 || V <= 0) return TFB_ERR_ARG;
-  DeltaScanArgs p{q, k, v, kq, decay, beta, o, state, state_slots, lens, S, G, H, D, V, has_past, nslots};
+  DeltaScanArgs p{q, k, v, coef, o, state, state_slots, lens, S, (S + 3) / 4 * 4, G, H, D, V, (V + 3) / 4 * 4, has_past, nslots, status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (D <= 32) return launch_scan<8, 4>(p, B, st);
-  if (D <= 64) return launch_scan<16, 4>(p, B, st);
-  if (D <= 128) return launch_scan<32, 4>(p, B, st);
-  if (D <= 256) return launch_scan<32, 8>(p, B, st);
-  if (D <= 512) return launch_scan<32, 16>(p, B, st);
-  return TFB_ERR_LIMIT;
+  switch (tfb_delta_padded_dim(D)) {
+    case 32: return launch_scan<4, 8>(p, B, st);
+    case 64: return launch_scan<8, 8>(p, B, st);
+    case 128: return launch_scan<16, 8>(p, B, st);
+    case 256: return launch_scan<16, 16>(p, B, st);
+    case 512: return launch_scan<16, 32>(p, B, st);
+    default: return TFB_ERR_LIMIT;
+  }
 }
 
 TFB_API int tfb_gated_norm(const float* o, const void* gate, long long ldg, const void* w, void* out, long long ldo, int rows, int H, int V,
@@ -489,23 +725,27 @@ TFB_API int tfb_gated_norm(const float* o, const void* gate, long long ldg, cons
   if (rows <= 0 || H <= 0 || V <= 0) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const long long blocks = ((long long)rows * H + 7) / 8;
-  const int grid = int(blocks < 148ll * 16 ? blocks : 148ll * 16);
-  if (f32) launch_k(gated_norm_kernel<float>, grid, 256, 0, st, o, static_cast<const float*>(gate), ldg, static_cast<const float*>(w),
-                    static_cast<float*>(out), ldo, rows, H, V, eps);
-  else launch_k(gated_norm_kernel<bf16>, grid, 256, 0, st, o, static_cast<const bf16*>(gate), ldg, static_cast<const bf16*>(w),
-                static_cast<bf16*>(out), ldo, rows, H, V, eps);
+  const int grid = int(blocks < 148ll * 32 ? blocks : 148ll * 32);
+  auto al = [](const void* x, int n) { return (reinterpret_cast<uintptr_t>(x) & (n - 1)) == 0; };
+  const int es = f32 ? 4 : 2;
+  const bool v4 = V % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && al(o, 16) && al(gate, 4 * es) && al(w, 4 * es) && al(out, 4 * es);
+#define TFB_GN(T, VEC) launch_k(gated_norm_kernel<T, VEC>, grid, 256, 0, st, o, static_cast<const T*>(gate), ldg, static_cast<const T*>(w), \
+                                static_cast<T*>(out), ldo, rows, H, V, eps)
+  if (f32) { if (v4) TFB_GN(float, 4); else TFB_GN(float, 1); }
+  else { if (v4) TFB_GN(bf16, 4); else TFB_GN(bf16, 1); }
+#undef TFB_GN
   return int(cudaGetLastError());
 }
 
-// One token for each of B sequences, gated norm included.  Returns TFB_ERR_LIMIT for head sizes it does not hold in
-// registers (the caller then takes the scan with S = 1 and the norm kernel).
+// One token for each of B sequences (prepared with Sp = 1), gated norm included.  Returns TFB_ERR_LIMIT for head sizes it
+// does not hold in registers (the caller then takes the scan and the norm kernel).
 TFB_API int tfb_delta_step(const float* q, const float* k, const float* v, const float* kq, const float* decay, const float* beta, float* state,
                            const int* state_slots, int nslots, const void* gate, long long ldg, const void* w, void* out, long long ldo, int B,
                            int G, int H, int D, int V, int has_past, float eps, int f32, void* stream) {
   using namespace tfb;
   if (B <= 0 || B > 65535 || G <= 0 || H % G || D <= 0 || V <= 0 || !state_slots) return TFB_ERR_ARG;
   if ((V & 3) || V > 256 || D > 256 || (V > 128 && D > 128)) return TFB_ERR_LIMIT;
-  DeltaScanArgs p{q, k, v, kq, decay, beta, nullptr, state, state_slots, nullptr, 1, G, H, D, V, has_past, nslots};
+  DeltaStepArgs p{q, k, v, kq, decay, beta, state, state_slots, G, H, D, tfb_delta_padded_dim(D), V, V, has_past, nslots};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   return f32 ? launch_step<float>(p, B, gate, ldg, w, out, ldo, eps, st) : launch_step<bf16>(p, B, gate, ldg, w, out, ldo, eps, st);
 }

@@ -136,7 +136,7 @@ class GatedDelta(nn.Module):
         G, H, D, V = s.kv_heads, s.heads, s.dim, s.vdim
         p = lin(h, i, "proj", self.proj)
         past = b.decode or b.pos0 > 0
-        prep = K.delta_prep(p, self.conv.data, cache.conv[i], b.state_slots, self.A_log.data, self.dt_bias.data, b.lens, b.B, b.S, G, H, D, V, past)
+        prep = K.delta_prep(p, self.conv.data, cache.conv[i], b.state_slots, self.A_log.data, self.dt_bias.data, b.lens, b.B, b.S, G, H, D, V, past, b.decode)
         gate = p[:, s.conv_channels:s.conv_channels + self.hv]
         if b.decode:
             o = K.delta_step(prep, cache.state[i], b.state_slots, gate, self.norm.data, self.eps, b.B, G, H, D, V)

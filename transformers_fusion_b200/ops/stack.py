@@ -7,6 +7,7 @@ the tensors decides); the residual, norms, rotation, attention scores and weight
 from __future__ import annotations
 
 import math
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -28,9 +29,9 @@ _lib.register("tfb_diff_attn_fwd", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, 
 _lib.register("tfb_diff_decode_tc", [c_i, c_i, c_i])
 _lib.register("tfb_diff_decode", [c_p, c_ll, c_p, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f,
                                   c_f, c_f, c_i, c_p, c_p])
-_lib.register("tfb_delta_prep", [c_p, c_ll, c_p, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i,
-                                 c_i, c_p])
-_lib.register("tfb_delta_scan", [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_delta_padded_dim", [c_i])
+_lib.register("tfb_delta_prep", [c_p, c_ll, c_p, c_p, c_p, c_i] + [c_p] * 10 + [c_i] * 10 + [c_p])
+_lib.register("tfb_delta_scan", [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_p])
 _lib.register("tfb_gated_norm", [c_p, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_delta_step", [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
 
@@ -207,9 +208,27 @@ def diff_decode(q, kpool, vpool, block_table, positions, H, G, D, V, window, sca
 
 
 # ---------------------------------------------------------------------------------------------------- gated delta rule
-def delta_prep(proj, conv_w, conv_state, state_slots, A_log, dt_bias, lens, B, S, G, H, D, V, has_past):
-    """proj [B*S, 2 G D + 2 H V + 2 H] = q | k | v | gate | b | a  ->  (q, k, v, k.q, decay, beta), all fp32.  ``conv_state``
-    [slots, taps - 1, channels] is read for sequences that go on (``has_past``) and left holding their last inputs."""
+@dataclass
+class DeltaRows:
+    """Prepared rows of B sequences: on CUDA the kernels' own layouts (see csrc/kernels/delta_rule.cu), ``pair`` holding k.q
+    when every sequence has one row; on the CPU q, k [T, G, D], v [T, H, V], decay, beta [T, H]."""
+    q: torch.Tensor
+    k: torch.Tensor
+    v: torch.Tensor
+    decay: torch.Tensor
+    beta: torch.Tensor
+    pair: Optional[torch.Tensor] = None
+    coef: Optional[torch.Tensor] = None
+
+
+def _step_fits(D, V) -> bool:
+    return V % 4 == 0 and V <= 256 and D <= 256 and (V <= 128 or D <= 128)
+
+
+def delta_prep(proj, conv_w, conv_state, state_slots, A_log, dt_bias, lens, B, S, G, H, D, V, has_past, step=False) -> DeltaRows:
+    """proj [B*S, 2 G D + 2 H V + 2 H] = q | k | v | gate | b | a  ->  convolved, activated, unit-length rows and gates, all
+    fp32.  ``conv_state`` [slots, taps - 1, channels] is read for sequences that go on (``has_past``) and left holding their last
+    inputs.  ``step``: the rows are for ``delta_step`` (one token per sequence)."""
     T, C, taps = B * S, 2 * G * D + H * V, conv_w.shape[1]
     if not proj.is_cuda:
         x = proj[:, :C].reshape(B, S, C)
@@ -232,41 +251,45 @@ def delta_prep(proj, conv_w, conv_state, state_slots, A_log, dt_bias, lens, B, S
         tail = proj[:, C + H * V:].float()
         beta = torch.sigmoid(tail[:, :H])
         decay = torch.exp(-torch.exp(A_log.float()) * torch.nn.functional.softplus(tail[:, H:2 * H] + dt_bias.float()))
-        return q, k, y[:, 2 * G * D:].reshape(T, H, V), (q * k).sum(-1), decay, beta
+        return DeltaRows(q, k, y[:, 2 * G * D:].reshape(T, H, V), decay, beta)
+    L = _lib.lib()
+    Dp, Vp = L.tfb_delta_padded_dim(D), (V + 3) // 4 * 4
+    Sp = 1 if step and _step_fits(D, V) else (S + 3) // 4 * 4
     e = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
-    q, k, v, kq, decay, beta = e(T, G, D), e(T, G, D), e(T, H, V), e(T, G), e(T, H), e(T, H)
-    check(_lib.lib().tfb_delta_prep(proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), ptr(conv_state), ptr(state_slots),
-                                    conv_state.shape[0] if conv_state is not None else 0, A_log.data_ptr(), dt_bias.data_ptr(), ptr(lens),
-                                    q.data_ptr(), k.data_ptr(), v.data_ptr(), kq.data_ptr(), decay.data_ptr(), beta.data_ptr(), B, S, G, H, D, V,
-                                    taps, int(has_past), _f32(proj), stream()), "delta_prep", 1 if S == 1 or taps == 1 else 2)
-    return q, k, v, kq, decay, beta
+    r = DeltaRows(e(B, G, Sp, Dp), e(B, G, Sp, Dp), e(B, H, Sp, Vp), e(B, H, Sp), e(B, H, Sp))
+    r.pair = e(B, G) if Sp == 1 else e(B, G, Sp // 4, 16)
+    r.coef = None if Sp == 1 else e(B, H, Sp // 4, 32)
+    check(L.tfb_delta_prep(proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), ptr(conv_state), ptr(state_slots),
+                           conv_state.shape[0] if conv_state is not None else 0, A_log.data_ptr(), dt_bias.data_ptr(), ptr(lens), r.q.data_ptr(),
+                           r.k.data_ptr(), r.v.data_ptr(), r.decay.data_ptr(), r.beta.data_ptr(), r.pair.data_ptr(), ptr(r.coef), B, S, Sp, G, H,
+                           D, V, taps, int(has_past), _f32(proj), stream()), "delta_prep", 1 + int(S > 1 and taps > 1) + int(Sp > 1))
+    return r
 
 
-def delta_scan(prep, state, state_slots, lens, B, S, G, H, D, V, has_past):
+def delta_scan(rows_: DeltaRows, state, state_slots, lens, B, S, G, H, D, V, has_past):
     """The recurrence over prepared rows; ``state`` [slots, H, D, V] fp32 is read (``has_past``) and updated.  Returns fp32
     [B*S, H, V] (rows past a sequence's length are unspecified)."""
-    q, k, v, kq, decay, beta = prep
-    if not q.is_cuda:
+    r = rows_
+    if not r.q.is_cuda:
         out = torch.zeros(B * S, H, V)
         n = lens if lens is not None else torch.full((B,), S)
         rep = H // G
         for b in range(B):
             sl = int(state_slots[b])
             st = state[sl].clone() if has_past and sl >= 0 else torch.zeros(H, D, V)
-            for t in range(int(n[b])):
-                r = b * S + t
-                kk, qq = k[r].repeat_interleave(rep, 0), q[r].repeat_interleave(rep, 0)
-                st = st * decay[r][:, None, None]
-                u = beta[r][:, None] * (v[r] - torch.einsum("hdv,hd->hv", st, kk))
+            for t in range(b * S, b * S + int(n[b])):
+                kk, qq = r.k[t].repeat_interleave(rep, 0), r.q[t].repeat_interleave(rep, 0)
+                st = st * r.decay[t][:, None, None]
+                u = r.beta[t][:, None] * (r.v[t] - torch.einsum("hdv,hd->hv", st, kk))
                 st = st + kk[:, :, None] * u[:, None, :]
-                out[r] = torch.einsum("hdv,hd->hv", st, qq)
+                out[t] = torch.einsum("hdv,hd->hv", st, qq)
             if sl >= 0:
                 state[sl] = st
         return out
-    o = torch.empty((B * S, H, V), dtype=torch.float32, device=q.device)
-    check(_lib.lib().tfb_delta_scan(q.data_ptr(), k.data_ptr(), v.data_ptr(), kq.data_ptr(), decay.data_ptr(), beta.data_ptr(), o.data_ptr(),
-                                    state.data_ptr(), state_slots.data_ptr(), state.shape[0], ptr(lens), B, S, G, H, D, V, int(has_past),
-                                    stream()), "delta_scan")
+    o = torch.empty((B * S, H, V), dtype=torch.float32, device=r.q.device)
+    check(_lib.lib().tfb_delta_scan(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.coef.data_ptr(), o.data_ptr(), state.data_ptr(),
+                                    state_slots.data_ptr(), state.shape[0], ptr(lens), B, S, G, H, D, V, int(has_past),
+                                    _lib.status_word(o.device).data_ptr(), stream()), "delta_scan")
     return o
 
 
@@ -283,13 +306,13 @@ def gated_norm(o, gate, w, eps):
     return out
 
 
-def delta_step(prep, state, state_slots, gate, w, eps, B, G, H, D, V, has_past=True):
-    """One token per sequence with the gated norm of its output; [B, H V]."""
-    q, k, v, kq, decay, beta = prep
-    if not q.is_cuda or V % 4 or V > 256 or D > 256 or (V > 128 and D > 128):
-        return gated_norm(delta_scan(prep, state, state_slots, None, B, 1, G, H, D, V, has_past), gate, w, eps)
-    out = rows(B, H * V, gate.dtype, q.device)
-    check(_lib.lib().tfb_delta_step(q.data_ptr(), k.data_ptr(), v.data_ptr(), kq.data_ptr(), decay.data_ptr(), beta.data_ptr(), state.data_ptr(),
-                                    state_slots.data_ptr(), state.shape[0], gate.data_ptr(), gate.stride(0), w.data_ptr(), out.data_ptr(),
-                                    out.stride(0), B, G, H, D, V, int(has_past), float(eps), _f32(gate), stream()), "delta_step")
+def delta_step(rows_: DeltaRows, state, state_slots, gate, w, eps, B, G, H, D, V, has_past=True):
+    """One token per sequence (rows prepared with ``step``) with the gated norm of its output; [B, H V]."""
+    r = rows_
+    if not r.q.is_cuda or not _step_fits(D, V):
+        return gated_norm(delta_scan(r, state, state_slots, None, B, 1, G, H, D, V, has_past), gate, w, eps)
+    out = rows(B, H * V, gate.dtype, r.q.device)
+    check(_lib.lib().tfb_delta_step(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.pair.data_ptr(), r.decay.data_ptr(), r.beta.data_ptr(),
+                                    state.data_ptr(), state_slots.data_ptr(), state.shape[0], gate.data_ptr(), gate.stride(0), w.data_ptr(),
+                                    out.data_ptr(), out.stride(0), B, G, H, D, V, int(has_past), float(eps), _f32(gate), stream()), "delta_step")
     return out
