@@ -51,8 +51,9 @@ CONFIGS = {
     "mixed": cfg(96, 211, [delta(4, 2, 24, 40, 4, ff=160), att(6, 3, 16, 48, 20, 0.3, 12, yarn=YA),
                            att(6, 3, 16, 48, 37, 0.6, 12, yarn=YA, scale=0.5, kv_from=1, ff=112), delta(3, 3, 32, 16, 2),
                            att(6, 3, 16, 48, 5, 0.2, 12, yarn=YA, kv_from=1)], eps=1e-4, scale=1.7),
-    # sizes that fit no vector width, one tap, a window of one page exactly
-    "odd": cfg(50, 101, [att(2, 1, 10, 14, 16, 0.8, 6, base=500.0, ff=30), delta(2, 1, 9, 7, 1, ff=22), delta(2, 2, 12, 6, 3)], scale=0.3),
+    # sizes that fit no vector width, one tap, a window of one page exactly (a large eps: heads this small can read out nearly
+    # nothing, and a norm with a small one would turn the bf16 rounding of that into anything)
+    "odd": cfg(50, 101, [att(2, 1, 10, 14, 16, 0.4, 6, base=500.0, ff=30), delta(2, 1, 9, 7, 1, ff=22), delta(2, 2, 12, 6, 3)], eps=0.02, scale=0.3),
     # attention alone; every head has its own keys; windows below and above a page
     "attention": cfg(64, 128, [att(4, 4, 32, 24, 9, 0.5, 32, ff=96), att(4, 4, 32, 24, 33, 0.1, 16, yarn=(0.5, 40, 4.0, 1.0))]),
     "delta": cfg(48, 90, [delta(4, 1, 16, 20, 5, ff=64), delta(2, 2, 40, 12, 3)], eps=1e-6),

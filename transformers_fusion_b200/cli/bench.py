@@ -4,7 +4,9 @@ L2-sized write between timed launches, best and median of ``--iters`` launches; 
 fraction of the copy / GEMM peaks when ``--peaks <json>`` (keys hbm_gbs, bf16_tflops) is given.
 
 Kernels: gemm, gemm_nt_wgrad, gemm_fp8, attention_fwd, attention_bwd, rmsnorm, rmsnorm_bwd, swiglu, rope,
-cross_entropy, adamw, paged_decode, sampling, moe_ffn.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
+cross_entropy, adamw, paged_decode, sampling, moe_ffn; those of stack models (``STACK_KERNELS``): diff_attention,
+diff_attention_window, attention_fwd_gqa128 (the plain form of the same layer), diff_decode, delta_prep, delta_scan,
+delta_scan_one, gated_norm, delta_prep_step, delta_step, res_norm, glu_silu, rope_append.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
 against their NCCL forms (cli/bench_comm.py)."""
 from __future__ import annotations
 
@@ -18,11 +20,84 @@ from .common import add_int
 
 KERNELS = ("gemm", "gemm_wgrad", "gemm_fp8", "attention_fwd", "attention_bwd", "rmsnorm", "rmsnorm_bwd", "swiglu", "rope",
            "cross_entropy", "adamw", "paged_decode", "sampling", "moe_ffn")
+STACK_KERNELS = ("diff_attention", "diff_attention_window", "attention_fwd_gqa128", "diff_decode", "delta_prep", "delta_scan", "delta_scan_one",
+                 "gated_norm", "delta_prep_step", "delta_step", "res_norm", "glu_silu", "rope_append")
+FP32_FMA_PER_SM = 128          # fp32 FMA lanes of an SM (delta_scan is reported against them as well)
+
+
+def _build_stack(kernel, n, dev):
+    """One launch (or one prepared operator call) of a stack model's kernel; layer sizes of a 2048-wide model: 16 heads, 4 kv heads,
+    two maps of 64 and values of 128; delta rule with 16 heads of 128 x 128.  ``n``: tokens per sequence (prompts; about 16 k
+    tokens in all) or cached tokens (decoding, 64 sequences)."""
+    import torch
+
+    from ..ops import functional as F
+    from ..ops import stack as K
+    bf = torch.bfloat16
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s, dtype=bf: torch.randn(*s, device=dev, generator=g).to(dtype)
+    H, G, D, V = 16, 4, 64, 128
+    B = 1 if kernel == "delta_scan_one" else max(1, (1 << 14) // n)
+    T = B * n
+    if kernel in ("diff_attention", "diff_attention_window", "attention_fwd_gqa128"):
+        qkv = rnd(T, (2 * H + 2 * G) * D + G * V)
+        if kernel == "attention_fwd_gqa128":
+            return (lambda: F.attn_fwd(qkv, qkv, qkv, B, n, H, G, 128, k_col0=H * 128, v_col0=(H + G) * 128)), 4.0 * B * H * n * n / 2 * 128, 2 * T * 2 * H * 128
+        W = 1024 if kernel == "diff_attention_window" else 0
+        keys = sum(min(i + 1, W or n) for i in range(n))
+        c = 2 * H * D
+        q, k, v = qkv[:, :c], qkv[:, c:c + 2 * G * D], qkv[:, c + 2 * G * D:]
+        return (lambda: K.diff_attn(q, k, v, B, n, n, H, G, D, V, W, 0.125, 0.4, 0.5, 1e-5)), 4.0 * B * H * keys * (D + V), T * (qkv.shape[1] + H * V) * 2
+    if kernel == "diff_decode":
+        B, pages = 64, 64 * (n // 16)
+        kp, vp = rnd(pages * 16, G * 2 * D), rnd(pages * 16, G * V)
+        bt = torch.randperm(pages, device=dev, generator=g).int().view(B, -1).contiguous()
+        pos, q = torch.full((B,), n - 1, dtype=torch.int32, device=dev), rnd(B, 2 * H * D)
+        return (lambda: K.diff_decode(q, kp, vp, bt, pos, H, G, D, V, 0, 0.125, 0.4, 0.5, 1e-5)), 4.0 * B * H * n * (D + V), B * n * G * (2 * D + V) * 2
+    if kernel in ("res_norm", "glu_silu", "rope_append"):
+        T, Hd = 1 << 14, 2048
+        if kernel == "res_norm":
+            x, y, w = rnd(T, Hd, dtype=torch.float32), rnd(T, Hd), rnd(Hd)
+            return (lambda: K.res_norm(x, 1e-5, y=y, w_post=w, w_pre=w)), 0.0, T * Hd * 12
+        if kernel == "glu_silu":
+            gu = rnd(T, 2 * 5632)
+            return (lambda: K.glu_silu(gu)), 0.0, T * 5632 * 6
+        qkv, tab = rnd(T, (2 * H + 2 * G) * D + G * V), F.rope_tables(D, T, device=dev)
+        pos, slots = torch.arange(T, device=dev, dtype=torch.int32), torch.arange(T, device=dev)
+        kp, vp = rnd(T, 2 * G * D), rnd(T, G * V)
+        return (lambda: K.rope_append(qkv, tab, pos, 2 * H, 2 * G, D, D, G * V, slots, kp, vp)), 0.0, T * ((2 * H + 2 * G) * D * 4 + 2 * G * D * 2 + G * V * 4)
+    step = kernel in ("delta_prep_step", "delta_step")
+    if step:
+        B, n, T = 64, 1, 64
+    G = H
+    D = V = 128
+    C = 2 * G * D + H * V
+    p = K.rows(T, C + H * V + 2 * H, bf, dev)
+    p.copy_(rnd(T, p.shape[1]))
+    conv, A, dtb, w = rnd(C, 4), torch.full((H,), -1.5, device=dev).to(bf), torch.zeros(H, device=dev).to(bf), torch.ones(V, device=dev).to(bf)
+    cs, st = torch.zeros(B, 3, C, dtype=bf, device=dev), torch.zeros(B, H, D, V, device=dev)
+    sl = torch.arange(B, dtype=torch.int32, device=dev)
+    prep = lambda: K.delta_prep(p, conv, cs, sl, A, dtb, None, B, n, G, H, D, V, step, step=step)
+    if kernel in ("delta_prep", "delta_prep_step"):
+        return prep, 0.0, T * C * (2 + 4) + (T * C * 2 * 6 if step else 0)
+    r = prep()
+    gate = p[:, C:C + H * V]
+    if kernel == "delta_step":
+        return (lambda: K.delta_step(r, st, sl, gate, w, 1e-5, B, G, H, D, V)), 0.0, B * H * D * V * 8
+    if kernel == "gated_norm":
+        o = K.delta_scan(r, st, sl, None, B, n, G, H, D, V, False)
+        return (lambda: K.gated_norm(o, gate, w, 1e-5)), 0.0, T * H * V * 8
+    if kernel in ("delta_scan", "delta_scan_one"):
+        return (lambda: K.delta_scan(r, st, sl, None, B, n, G, H, D, V, False)), 6.0 * T * H * D * V, T * (2 * G * D + 2 * H * V) * 4
+    raise SystemExit(f"Error: unknown kernel '{kernel}'")
 
 
 def _build(kernel, n, dev, heads=0, shape=None):
     """Returns (callable, flops, bytes) for one launch of ``kernel`` at problem size ``n``."""
     import torch
+
+    if kernel in STACK_KERNELS:
+        return _build_stack(kernel, n, dev)
 
     from ..ops import functional as F
     bf = torch.bfloat16
@@ -339,7 +414,7 @@ def main(argv=None):
         if not torch.cuda.is_available():
             print("Error: kernel benchmarks need a CUDA device", file=sys.stderr)
             return 1
-        names = KERNELS if a.kernel == "all" else [a.kernel]
+        names = KERNELS if a.kernel == "all" else STACK_KERNELS if a.kernel == "stack" else [a.kernel]
         peaks = json.load(open(a.peaks)) if a.peaks else {}
         for name in names:
             shape = None
@@ -353,7 +428,10 @@ def main(argv=None):
                    "gbs": round(nbytes / best / 1e6, 1), "tflops": round(flops / best / 1e9, 2)}
             if peaks:
                 rec["frac_hbm_of_measured"] = round(rec["gbs"] / peaks["hbm_gbs"], 3)
-                if flops:
+                if name.startswith("delta_scan"):      # fp32 arithmetic: against the FMA lanes at the largest clock
+                    sms = torch.cuda.get_device_properties(0).multi_processor_count
+                    rec["frac_fp32_fma"] = round(rec["tflops"] / (2 * FP32_FMA_PER_SM * sms * peaks.get("sm_max_mhz", 1965.0) * 1e-6), 3)
+                elif flops:
                     rec["frac_bf16_of_measured"] = round(rec["tflops"] / peaks["bf16_tflops"], 3)
             print(json.dumps(rec) if a.json else "  ".join(f"{k}={v}" for k, v in rec.items()), flush=True)
     if a.serve:
