@@ -3,7 +3,7 @@
 //   S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q            per head, S is [D, V] in fp32
 //
 // Kernels:
-//   delta_prep   one block per (strip of 8 tokens, head): causal convolution of q, k and v over time (per channel, with the last
+//   delta_prep   one block per (strip of 16 tokens, head): causal convolution of q, k and v over time (per channel, with the last
 //                inputs of the previous step as history), silu, unit length of q and k per head, the decay g and the step
 //                size beta, and the dot products k_i.k_j, q_i.k_j of every four tokens.  Everything it hands on is fp32.
 //   delta_coef   per head and four tokens: those dot products times the decays between the tokens.
@@ -45,7 +45,11 @@ struct DeltaPrepArgs {
   int S, Sp, G, H, D, Dp, V, Vp, taps, has_past, nslots;
 };
 
-constexpr int PREP_STRIP = 8;    // tokens per block (a multiple of 4)
+constexpr int PREP_STRIP = 16;   // tokens per block: four groups of four, one per warp
+
+// the convolution's activation may be bf16-accurate when its inputs are bf16; the fp32 form is exact
+template <class T> __device__ __forceinline__ float conv_silu(float x) { return silu_exact(x); }
+template <> __device__ __forceinline__ float conv_silu<__nv_bfloat16>(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 
 // One channel over the strip's tokens s0 .. s0 + n - 1: convolution, silu, emit(token in strip, value).  TAPS > 0: the window
 // moves through registers; TAPS = 0: any number of taps, inputs re-read.
@@ -53,40 +57,51 @@ template <class T, int TAPS, class Emit>
 __device__ __forceinline__ void conv_channel(const DeltaPrepArgs& p, const T* __restrict__ x0, T* hist, bool past, int C, int c, int s0, int n,
                                              Emit emit) {
   const T* cw = static_cast<const T*>(p.conv_w) + (long long)c * p.taps;
-  auto input = [&](int s) -> float {     // token s of this call; negative: history
-    if (s >= 0) return to_f(x0[(long long)s * p.ld + c]);
-    return past ? to_f(hist[(long long)(p.taps - 1 + s) * C + c]) : 0.f;
+  const T* xc = x0 + (long long)s0 * p.ld + c;          // token s0, channel c
+  auto before = [&](int j) -> float {    // the input j tokens before s0; before the call's first token: history
+    if (s0 >= j) return to_f(xc[-(long long)j * p.ld]);
+    return past ? to_f(hist[(long long)(p.taps - 1 + s0 - j) * C + c]) : 0.f;
   };
+  const T newest = xc[0];
   if constexpr (TAPS > 0) {
     float w[TAPS], win[TAPS];
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) w[j] = to_f(cw[j]);
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) win[j + 1] = input(s0 - (TAPS - 1) + j);
-    float cur[PREP_STRIP];
+    for (int j = 0; j < TAPS - 1; ++j) win[j + 1] = before(TAPS - 1 - j);
+    const T* xp = xc;
+    for (int i0 = 0; i0 < n; i0 += 8) {
+      T cur[8];
 #pragma unroll
-    for (int i = 0; i < PREP_STRIP; ++i) cur[i] = i < n ? to_f(x0[(long long)(s0 + i) * p.ld + c]) : 0.f;
+      for (int i = 0; i < 8; ++i) {
+        cur[i] = i0 + i < n ? *xp : from_f<T>(0.f);
+        xp += p.ld;
+      }
 #pragma unroll
-    for (int i = 0; i < PREP_STRIP; ++i) {
+      for (int i = 0; i < 8; ++i) {
 #pragma unroll
-      for (int j = 0; j < TAPS - 1; ++j) win[j] = win[j + 1];
-      win[TAPS - 1] = cur[i];
-      float y = 0.f;
+        for (int j = 0; j < TAPS - 1; ++j) win[j] = win[j + 1];
+        win[TAPS - 1] = to_f(cur[i]);
+        float y = 0.f;
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) y = fmaf(w[j], win[j], y);
-      if (i < n) emit(i, silu_exact(y));
+        for (int j = 0; j < TAPS; ++j) y = fmaf(w[j], win[j], y);
+        if (i0 + i < n) emit(i0 + i, conv_silu<T>(y));
+      }
     }
   } else {
     for (int i = 0; i < n; ++i) {
       float y = 0.f;
-      for (int j = 0; j < p.taps; ++j) y = fmaf(to_f(cw[j]), input(s0 + i - (p.taps - 1) + j), y);
-      emit(i, silu_exact(y));
+      for (int j = 0; j < p.taps; ++j) {
+        const int back = p.taps - 1 - j - i;          // tokens before s0; <= 0: in the strip
+        y = fmaf(to_f(cw[j]), back > 0 ? before(back) : to_f(xc[-(long long)back * p.ld]), y);
+      }
+      emit(i, conv_silu<T>(y));
     }
   }
   if (p.S == 1 && hist) {                // decoding: this thread alone uses channel c, so the window moves in place
     const int m = p.taps - 1;
     for (int j = 0; j < m - 1; ++j) hist[(long long)j * C + c] = past ? hist[(long long)(j + 1) * C + c] : from_f<T>(0.f);
-    hist[(long long)(m - 1) * C + c] = x0[c];
+    hist[(long long)(m - 1) * C + c] = newest;
   }
 }
 
@@ -94,7 +109,7 @@ __device__ __forceinline__ void conv_channel(const DeltaPrepArgs& p, const T* __
 template <class T, int TAPS>
 __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaPrepArgs p) {
   tfb::pdl_sync();
-  extern __shared__ float sqk[];         // [PREP_STRIP][2 Dp]
+  extern __shared__ float sqk[];         // [rows][2 Dp]; rows: the strip's, or 4 when decoding
   const int s0 = blockIdx.x * PREP_STRIP, b = blockIdx.z, tid = threadIdx.x, unit = blockIdx.y;
   const int len = p.lens ? p.lens[b] : p.S;
   const int len4 = p.Sp == 1 ? len : (len + 3) / 4 * 4;       // rows len .. len4 - 1 become tokens that change nothing
@@ -111,8 +126,8 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaPrepArgs p) 
     const int h = unit - p.G;
     float* vo = p.v + (((long long)b * p.H + h) * p.Sp + s0) * p.Vp;
     for (int j = tid; j < p.V; j += 128)
-      conv_channel<T, TAPS>(p, x0, hist, past, C, 2 * p.G * p.D + h * p.V + j, s0, n, [&](int i, float y) { vo[(long long)i * p.Vp + j] = y; });
-    for (int i = tid; i < (n4 - n) * p.Vp; i += 128) vo[(long long)n * p.Vp + i] = 0.f;
+      conv_channel<T, TAPS>(p, x0, hist, past, C, 2 * p.G * p.D + h * p.V + j, s0, n, [&](int i, float y) { vo[i * p.Vp + j] = y; });
+    for (int i = tid; i < (n4 - n) * p.Vp; i += 128) vo[n * p.Vp + i] = 0.f;
     if (tid < n4) {
       const long long o = ((long long)b * p.H + h) * p.Sp + s0 + tid;
       if (tid < n) {
@@ -128,59 +143,85 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaPrepArgs p) 
     }
     return;
   }
-  const int g = unit, Dp = p.Dp;
-  for (int i = tid; i < n4 * 2 * Dp; i += 128) {            // rows without a token, and the tails of the others
-    const int r = i / (2 * Dp), d = i % Dp;
-    if (r >= n || d >= p.D) sqk[i] = 0.f;
-  }
+  const int g = unit, Dp = p.Dp, W = 2 * Dp;
+  const int rows = (n4 + 3) / 4 * 4;
+  if (p.D < Dp || n < rows)              // the tails of the rows, and rows without a token
+    for (int i = tid; i < rows * W; i += 128)
+      if (i / W >= n || i % Dp >= p.D) sqk[i] = 0.f;
   for (int d = tid; d < p.D; d += 128) {
-    conv_channel<T, TAPS>(p, x0, hist, past, C, g * p.D + d, s0, n, [&](int i, float y) { sqk[i * 2 * Dp + d] = y; });
-    conv_channel<T, TAPS>(p, x0, hist, past, C, (p.G + g) * p.D + d, s0, n, [&](int i, float y) { sqk[i * 2 * Dp + Dp + d] = y; });
+    conv_channel<T, TAPS>(p, x0, hist, past, C, g * p.D + d, s0, n, [&](int i, float y) { sqk[i * W + d] = y; });
+    conv_channel<T, TAPS>(p, x0, hist, past, C, (p.G + g) * p.D + d, s0, n, [&](int i, float y) { sqk[i * W + Dp + d] = y; });
   }
   __syncthreads();
-  const int warp = tid >> 5, lane = tid & 31;
-  for (int i = warp; i < n4; i += 4) {
-    float* sq = sqk + i * 2 * Dp;
-    float* sk = sq + Dp;
-    float qq = 0.f, kk = 0.f;
-    for (int d = lane; d < Dp; d += 32) {
-      qq = fmaf(sq[d], sq[d], qq);
-      kk = fmaf(sk[d], sk[d], kk);
+  // one warp per four tokens: the 24 products of their q and k vectors (as they are), reduced so that lane x holds product x;
+  // the unit lengths come from the diagonal and scale the others
+  const int blk = tid >> 5, lane = tid & 31;
+  if (blk * 4 >= n4) return;
+  const float* base = sqk + blk * 4 * W;
+  float pr[32];
+#pragma unroll
+  for (int i = 0; i < 32; ++i) pr[i] = 0.f;
+  for (int d = lane; d < Dp; d += 32) {
+    float q[4], k[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      q[i] = base[i * W + d];
+      k[i] = base[i * W + Dp + d];
     }
-    qq = warp_add(qq);
-    kk = warp_add(kk);
-    const float rq = 1.f / sqrtf(qq + 1e-6f) / sqrtf(float(p.D)), rk = 1.f / sqrtf(kk + 1e-6f);
-    const long long o = (((long long)b * p.G + g) * p.Sp + s0 + i) * Dp;
-    for (int d = lane; d < Dp; d += 32) {
-      const float a = sq[d] * rq, c = sk[d] * rk;
-      sq[d] = a;
-      sk[d] = c;
-      p.q[o + d] = a;
-      p.k[o + d] = c;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {        // order of the products: see coef; then the squares of k (16-19) and of q (20-23)
+#pragma unroll
+      for (int j = 0; j < i; ++j) pr[i * (i - 1) / 2 + j] = fmaf(k[i], k[j], pr[i * (i - 1) / 2 + j]);
+#pragma unroll
+      for (int j = 0; j <= i; ++j) pr[6 + i * (i + 1) / 2 + j] = fmaf(q[i], k[j], pr[6 + i * (i + 1) / 2 + j]);
+      pr[16 + i] = fmaf(k[i], k[i], pr[16 + i]);
+      pr[20 + i] = fmaf(q[i], q[i], pr[20 + i]);
     }
   }
-  __syncthreads();
-  auto dot = [&](const float* a, const float* c) {
-    float v = 0.f;
-    for (int d = lane; d < Dp; d += 32) v = fmaf(a[d], c[d], v);
-    return warp_add(v);
-  };
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {     // o values stay with each half
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float send = up ? pr[i] : pr[i + o], keep = up ? pr[i + o] : pr[i];
+      pr[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+    }
+  }
+  const float mine = pr[0];
+  // lanes 16-19: 1 / |k_i|, lanes 20-23: 1 / (|q_i| sqrt(D))
+  float r = 1.f / sqrtf(mine + 1e-6f);
+  if (lane >= 20) r = r / sqrtf(float(p.D));
+  float rk[4], rq[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    rk[i] = __shfl_sync(0xffffffffu, r, 16 + i);
+    rq[i] = __shfl_sync(0xffffffffu, r, 20 + i);
+  }
+  const long long row0 = ((long long)b * p.G + g) * p.Sp + s0 + blk * 4;
+  const int nr = min(4, n4 - blk * 4);
+  for (int d = lane; d < Dp; d += 32)
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (i < nr) {
+        p.q[(row0 + i) * Dp + d] = base[i * W + d] * rq[i];
+        p.k[(row0 + i) * Dp + d] = base[i * W + Dp + d] * rk[i];
+      }
   if (p.Sp == 1) {
-    if (warp == 0) {
-      const float v = dot(sqk, sqk + Dp);
-      if (lane == 0) p.pair[(long long)b * p.G + g] = v;
-    }
+    if (lane == 6) p.pair[(long long)b * p.G + g] = mine * rq[0] * rk[0];
     return;
   }
-  // entries 0-5: k_i.k_j for (i, j) = 10 20 21 30 31 32; 6-15: q_i.k_j for 00 10 11 20 21 22 30 31 32 33
-  for (int e = warp; e < n4 / 4 * 16; e += 4) {
-    const int blk = e >> 4, x = e & 15;
-    const int y = x < 6 ? x : x - 6;
+  if (lane < 16) {
+    const int y = lane < 6 ? lane : lane - 6;
     int i, j;
-    if (x < 6) { i = y < 1 ? 1 : y < 3 ? 2 : 3; j = y - (i * (i - 1)) / 2; }
+    if (lane < 6) { i = y < 1 ? 1 : y < 3 ? 2 : 3; j = y - (i * (i - 1)) / 2; }
     else { i = y < 1 ? 0 : y < 3 ? 1 : y < 6 ? 2 : 3; j = y - (i * (i + 1)) / 2; }
-    const float v = dot(sqk + (blk * 4 + i) * 2 * Dp + (x < 6 ? Dp : 0), sqk + (blk * 4 + j) * 2 * Dp + Dp);
-    if (lane == 0) p.pair[(((long long)b * p.G + g) * (p.Sp / 4) + s0 / 4 + blk) * 16 + x] = v;
+    float f = 0.f, e = 0.f;
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      if (x == i) f = lane < 6 ? rk[x] : rq[x];
+      if (x == j) e = rk[x];
+    }
+    p.pair[(((long long)b * p.G + g) * (p.Sp / 4) + s0 / 4 + blk) * 16 + lane] = mine * f * e;
   }
 }
 
@@ -268,11 +309,6 @@ __device__ __forceinline__ u64 fma2(u64 a, u64 b, u64 c) {
 __device__ __forceinline__ u64 mul2(u64 a, u64 b) {
   u64 d;
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ u64 add2(u64 a, u64 b) {
-  u64 d;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
   return d;
 }
 __device__ __forceinline__ u64 pack2(float lo, float hi) {
@@ -386,16 +422,13 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaScanArgs p) 
         }
 #pragma unroll
         for (int x = 0; x < CPT; ++x) {
-          u64 dk0 = mul2(st[x][0], kk[i][0]), dk1 = mul2(st[x][1], kk[i][1]);
-          u64 dq0 = mul2(st[x][0], qq[0]), dq1 = mul2(st[x][1], qq[1]);
+          u64 dk = mul2(st[x][0], kk[i][0]), dq = mul2(st[x][0], qq[0]);     // 8 CPT independent chains over the four tokens
 #pragma unroll
-          for (int e = 2; e < EPT / 2; e += 2) {
-            dk0 = fma2(st[x][e], kk[i][e], dk0);
-            dk1 = fma2(st[x][e + 1], kk[i][e + 1], dk1);
-            dq0 = fma2(st[x][e], qq[e], dq0);
-            dq1 = fma2(st[x][e + 1], qq[e + 1], dq1);
+          for (int e = 1; e < EPT / 2; ++e) {
+            dk = fma2(st[x][e], kk[i][e], dk);
+            dq = fma2(st[x][e], qq[e], dq);
           }
-          const float2 a = unpack2(add2(dk0, dk1)), q = unpack2(add2(dq0, dq1));
+          const float2 a = unpack2(dk), q = unpack2(dq);
           val[2 * x][i] = a.x + a.y;
           val[2 * x + 1][i] = q.x + q.y;
         }
@@ -682,16 +715,23 @@ TFB_API int tfb_delta_prep(const void* proj, long long ld, const void* conv_w, v
                   S, Sp, G, H, D, Dp, V, (V + 3) / 4 * 4, taps, has_past, nslots};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const dim3 grid((Sp + PREP_STRIP - 1) / PREP_STRIP, G + H, B);
-  const int smem = (Sp == 1 ? 1 : PREP_STRIP) * 2 * Dp * int(sizeof(float));     // at most 32 KB
+  const int smem = (Sp == 1 ? 4 : PREP_STRIP) * 2 * Dp * int(sizeof(float));     // at most 64 KB
+#define TFB_PREP1(T, TAPS)                                                                 \
+  {                                                                                       \
+    static DeviceOnce once;                                                               \
+    if (int e = ensure_dyn_smem(once, delta_prep_kernel<T, TAPS>, 64 * 1024)) return e;   \
+    launch_k(delta_prep_kernel<T, TAPS>, grid, 128, smem, st, p);                         \
+  }
 #define TFB_PREP(T)                                                                       \
   switch (taps) {                                                                         \
-    case 2: launch_k(delta_prep_kernel<T, 2>, grid, 128, smem, st, p); break;             \
-    case 3: launch_k(delta_prep_kernel<T, 3>, grid, 128, smem, st, p); break;             \
-    case 4: launch_k(delta_prep_kernel<T, 4>, grid, 128, smem, st, p); break;             \
-    default: launch_k(delta_prep_kernel<T, 0>, grid, 128, smem, st, p); break;            \
+    case 2: TFB_PREP1(T, 2) break;                                                    \
+    case 3: TFB_PREP1(T, 3) break;                                                    \
+    case 4: TFB_PREP1(T, 4) break;                                                    \
+    default: TFB_PREP1(T, 0) break;                                                   \
   }
   if (f32) { TFB_PREP(float) } else { TFB_PREP(bf16) }
 #undef TFB_PREP
+#undef TFB_PREP1
   if (S > 1 && taps > 1 && state_slots) {
     const dim3 hg((2 * G * D + H * V + 255) / 256, B);
     if (f32) launch_k(conv_history_kernel<float>, hg, 256, 0, st, p);
