@@ -248,7 +248,10 @@ def serve_bench(a):
         symm = SymmetricHeap(rank, world, dev)
     cfg = preset(a.preset)
     if a.layers > 0:
-        cfg.num_layers = a.layers
+        if hasattr(cfg, "layers"):
+            cfg.layers = cfg.layers[:a.layers]
+        else:
+            cfg.num_layers = a.layers
     if a.tp_shape > 1:
         # one rank's share of a tensor-parallel deployment, alone on this GPU: its heads, kv heads and FFN slice, the
         # replicated embedding / head, and no all-reduce - the compute side of a rank without the peers
@@ -259,6 +262,9 @@ def serve_bench(a):
     if hasattr(cfg, "num_experts"):
         from ..models.moe import MoEModel
         model = MoEModel(cfg, device=dev, dtype=torch.bfloat16, seed=0)
+    elif hasattr(cfg, "architecture"):
+        from ..models.registry import model_class
+        model = model_class(cfg.architecture)(cfg, device=dev, dtype=torch.bfloat16, seed=0)
     else:
         model = DenseModel(cfg, device=dev, dtype=torch.bfloat16, seed=0)
     g = torch.Generator().manual_seed(0)

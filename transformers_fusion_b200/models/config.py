@@ -319,6 +319,23 @@ def preset(name: str) -> TransformerConfig:
         return TransformerConfig(vocab_size=50257, hidden_size=768, num_layers=12, num_heads=12, ffn_hidden_size=3072,
                                  max_seq_len=1024, activation="gelu", norm_type="layernorm", position_type="learned",
                                  attention_bias=True, tie_embeddings=True)
+    if name in ("lanedra-1.5b", "lanedra-8b"):
+        # layer sizes of the dense models they stand beside (dense-1.5b, llama-3-8b): the same width, feed-forward, key / value
+        # bytes per token of an attention layer and query rows; half of the layers are the delta rule, and every second
+        # attention layer looks at the keys of the one before it
+        H, heads, kv, ff, n, V, win = (2048, 16, 4, 5632, 24, 32000, 2048) if name == "lanedra-1.5b" else (4096, 32, 8, 14336, 32, 128256, 4096)
+        rot = RotarySpec(64, 500000.0, 4.0, 8192)
+        layers = []
+        for i in range(n):
+            if i % 2 == 0:
+                mix = GatedDeltaSpec(heads, heads, 128, 128, 4)
+            else:
+                mix = DiffAttentionSpec(heads, kv, 64, 128, 64 ** -0.5, 0.5, rot, win, i - 2 if i % 4 == 3 else None)
+            layers.append(StackLayer(mix, ff))
+        return LanedraConfig(V, H, layers, 1e-5, 1.0, max_seq_len=32768)
+    if name == "dense-1.5b":
+        return TransformerConfig(vocab_size=32000, hidden_size=2048, num_layers=24, num_heads=16, num_kv_heads=4, ffn_hidden_size=5632,
+                                 rope_theta=500000.0, max_seq_len=32768, activation="swiglu")
     if name == "tiny":
         return TransformerConfig(vocab_size=256, hidden_size=128, num_layers=2, num_heads=2, ffn_hidden_size=256,
                                  max_seq_len=128)
