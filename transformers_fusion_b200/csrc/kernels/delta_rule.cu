@@ -3,27 +3,27 @@
 //   S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q            per head, S is [D, V] in fp32
 //
 // Kernels:
-//   delta_prep   one block per (16 tokens, head): causal convolution of q, k and v over time (per channel, with the last inputs
-//                of the previous step as history), silu, unit length of q and k per head, the decay g and the step size beta.
-//                Everything it hands on is fp32.
-//   delta_wy     prompts: one block per (16 tokens, head).  With S the state before the 16 tokens, G_i and R_ij the products of
-//                the decays up to token i and between tokens j and i, the recurrence reads
+//   delta_prep   one block per (strip of 16 tokens, head): causal convolution of q, k and v over time (per channel, with the last
+//                inputs of the previous step as history), silu, unit length of q and k per head, the decay g and the step
+//                size beta, and the dot products k_i.k_j, q_i.k_j of every four tokens.  Everything it hands on is fp32.
+//   delta_coef   per head and four tokens: those dot products times the decays between the tokens.
+//   delta_scan   prompts.  The columns of S are independent recurrences that share k and q, so a group of TPC threads owns CPT
+//                columns (D / TPC entries of each, in registers as packed fp32 pairs) and walks over the tokens four at a
+//                time.  With S the state before the four tokens and G_i, R_ij the products of the decays up to token i and
+//                between tokens j and i,
 //                    u_i = beta_i (v_i - G_i S^T k_i - sum_{j<i} R_ij (k_i.k_j) u_j)
 //                    o_i = G_i S^T q_i + sum_{j<=i} R_ij (q_i.k_j) u_j
-//                    S  <- G_last S + sum_j R_last,j k_j u_j^T
-//                The triangular system for u does not need S: forward substitution turns beta v and beta G k into rows y and w
-//                with u_i = y_i - S^T w_i.
-//   delta_scan   prompts: what is left of the recurrence, 16 tokens at a time.  The columns of S are independent, so a group
-//                of TPC threads owns CPT columns (D / TPC entries of each, in registers as packed fp32 pairs): 32 products with
-//                the old state, one shuffle reduction, u, o, and the update.  The rows of the next 16 tokens travel to shared
-//                memory (bulk copies) meanwhile; the state never leaves the registers between tokens.
-//   delta_step   decoding: one block per (sequence, head) streams the state through registers once (read, two products,
-//                rank-one update, write) and applies the gated norm of the head's output.
-// All of it is fp32 FMA arithmetic.
+//                    S  <- G_4 S + sum_j R_4j k_j u_j^T
+//                which is the recurrence itself with its four reductions over D made one: all eight products with S are taken
+//                from the same old state, so four tokens have one shuffle reduction on their critical path.  k, q, v and the
+//                coefficients of the next tokens travel to shared memory (bulk copies) while the current ones are used; the
+//                state never leaves the registers between tokens, and the arithmetic is fp32 FMA throughout.
+//   delta_step   one token per sequence: one block per (sequence, head) streams the state through registers once (read,
+//                two products, rank-one update, write) and applies the gated norm of the head's output.
 //
-// Layouts of the prepared arrays (Sp: rows per sequence, S rounded up to 16, or 1 when decoding; Dp: D rounded up to the
-// register tile, tails zero; Vp: V rounded up to 4): q, k [B, G, Sp, Dp], v (later y) [B, H, Sp, Vp], w [B, H, Sp, Dp],
-// decay, beta [B, H, Sp], kq [B, G] (decoding), coef [B, H, Sp / 16, COEF].
+// Layouts of the prepared arrays (Sp: rows per sequence, S rounded up to 4, or 1 when decoding; Dp: D rounded up to the
+// register tile, tails zero; Vp: V rounded up to 4): q, k [B, G, Sp, Dp], v [B, H, Sp, Vp], decay, beta [B, H, Sp],
+// pair [B, G, Sp / 4, 16] (decoding: [B, G], k.q), coef [B, H, Sp / 4, 32].
 #include "tfb_elem.cuh"
 #include "tfb_host.h"
 
@@ -41,13 +41,11 @@ struct DeltaPrepArgs {
   const int* state_slots; // [B]; negative: no history is read or kept
   const void *A_log, *dt_bias;  // [H]
   const int* lens;        // [B] tokens of each sequence in this call (null: S)
-  float *q, *k, *v, *decay, *beta, *kq;
+  float *q, *k, *v, *decay, *beta, *pair;
   int S, Sp, G, H, D, Dp, V, Vp, taps, has_past, nslots;
 };
 
-constexpr int CHUNK = 16;              // tokens per block of the preparation and per step of the scan
-constexpr int P_PITCH = CHUNK + 4;     // row pitch of the o-from-u coefficients (conflict-free 16-byte reads of eight rows)
-constexpr int COEF = CHUNK * P_PITCH + 2 * CHUNK;    // R_ij (q_i.k_j) for j <= i, then G_i, then R_last,i
+constexpr int PREP_STRIP = 16;   // tokens per block: four groups of four, one per warp
 
 // the convolution's activation may be bf16-accurate when its inputs are bf16; the fp32 form is exact
 template <class T> __device__ __forceinline__ float conv_silu(float x) { return silu_exact(x); }
@@ -111,11 +109,12 @@ __device__ __forceinline__ void conv_channel(const DeltaPrepArgs& p, const T* __
 template <class T, int TAPS>
 __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaPrepArgs p) {
   tfb::pdl_sync();
-  extern __shared__ float sqk[];         // [rows][2 Dp]; rows: CHUNK, or 4 when decoding
-  const int s0 = blockIdx.x * CHUNK, b = blockIdx.z, tid = threadIdx.x, unit = blockIdx.y;
+  extern __shared__ float sqk[];         // [rows][2 Dp]; rows: the strip's, or 4 when decoding
+  const int s0 = blockIdx.x * PREP_STRIP, b = blockIdx.z, tid = threadIdx.x, unit = blockIdx.y;
   const int len = p.lens ? p.lens[b] : p.S;
-  if (s0 >= len) return;
-  const int n = min(CHUNK, len - s0), nr = p.Sp == 1 ? 1 : CHUNK;      // rows n .. nr - 1 become tokens that change nothing
+  const int len4 = p.Sp == 1 ? len : (len + 3) / 4 * 4;       // rows len .. len4 - 1 become tokens that change nothing
+  if (s0 >= len4) return;
+  const int n = max(0, min(PREP_STRIP, len - s0)), n4 = min(PREP_STRIP, len4 - s0);
   const T* x0 = static_cast<const T*>(p.proj) + (long long)b * p.S * p.ld;
   const int C = 2 * p.G * p.D + p.H * p.V;
   int slot = p.state_slots ? p.state_slots[b] : -1;
@@ -128,8 +127,8 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaPrepArgs p) 
     float* vo = p.v + (((long long)b * p.H + h) * p.Sp + s0) * p.Vp;
     for (int j = tid; j < p.V; j += 128)
       conv_channel<T, TAPS>(p, x0, hist, past, C, 2 * p.G * p.D + h * p.V + j, s0, n, [&](int i, float y) { vo[i * p.Vp + j] = y; });
-    for (int i = tid; i < (nr - n) * p.Vp; i += 128) vo[n * p.Vp + i] = 0.f;
-    if (tid < nr) {
+    for (int i = tid; i < (n4 - n) * p.Vp; i += 128) vo[n * p.Vp + i] = 0.f;
+    if (tid < n4) {
       const long long o = ((long long)b * p.H + h) * p.Sp + s0 + tid;
       if (tid < n) {
         const T* gb = x0 + (long long)(s0 + tid) * p.ld + C + p.H * p.V;
@@ -145,7 +144,7 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaPrepArgs p) 
     return;
   }
   const int g = unit, Dp = p.Dp, W = 2 * Dp;
-  const int rows = (nr + 3) / 4 * 4;
+  const int rows = (n4 + 3) / 4 * 4;
   if (p.D < Dp || n < rows)              // the tails of the rows, and rows without a token
     for (int i = tid; i < rows * W; i += 128)
       if (i / W >= n || i % Dp >= p.D) sqk[i] = 0.f;
@@ -154,50 +153,76 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const DeltaPrepArgs p) 
     conv_channel<T, TAPS>(p, x0, hist, past, C, (p.G + g) * p.D + d, s0, n, [&](int i, float y) { sqk[i * W + Dp + d] = y; });
   }
   __syncthreads();
-  // one warp per four tokens: squares of their k (0-3) and q (4-7) and, for decoding, q_0.k_0 (8); reduced so that lanes 2 x and
-  // 2 x + 1 hold sum x
+  // one warp per four tokens: the 24 products of their q and k vectors (as they are), reduced so that lane x holds product x;
+  // the unit lengths come from the diagonal and scale the others
   const int blk = tid >> 5, lane = tid & 31;
-  if (blk * 4 >= nr) return;
+  if (blk * 4 >= n4) return;
   const float* base = sqk + blk * 4 * W;
-  float pr[16];
+  float pr[32];
 #pragma unroll
-  for (int i = 0; i < 16; ++i) pr[i] = 0.f;
+  for (int i = 0; i < 32; ++i) pr[i] = 0.f;
   for (int d = lane; d < Dp; d += 32) {
+    float q[4], k[4];
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      const float q = base[i * W + d], k = base[i * W + Dp + d];
-      pr[i] = fmaf(k, k, pr[i]);
-      pr[4 + i] = fmaf(q, q, pr[4 + i]);
-      if (i == 0) pr[8] = fmaf(q, k, pr[8]);
+      q[i] = base[i * W + d];
+      k[i] = base[i * W + Dp + d];
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {        // order of the products: see coef; then the squares of k (16-19) and of q (20-23)
+#pragma unroll
+      for (int j = 0; j < i; ++j) pr[i * (i - 1) / 2 + j] = fmaf(k[i], k[j], pr[i * (i - 1) / 2 + j]);
+#pragma unroll
+      for (int j = 0; j <= i; ++j) pr[6 + i * (i + 1) / 2 + j] = fmaf(q[i], k[j], pr[6 + i * (i + 1) / 2 + j]);
+      pr[16 + i] = fmaf(k[i], k[i], pr[16 + i]);
+      pr[20 + i] = fmaf(q[i], q[i], pr[20 + i]);
     }
   }
 #pragma unroll
-  for (int m = 8; m > 0; m >>= 1) {      // m sums stay with each half of the lanes that share 2 m
-    const bool up = lane & (2 * m);
+  for (int o = 16; o > 0; o >>= 1) {     // o values stay with each half
+    const bool up = lane & o;
 #pragma unroll
-    for (int i = 0; i < m; ++i) {
-      const float send = up ? pr[i] : pr[i + m], keep = up ? pr[i + m] : pr[i];
-      pr[i] = keep + __shfl_xor_sync(0xffffffffu, send, 2 * m);
+    for (int i = 0; i < o; ++i) {
+      const float send = up ? pr[i] : pr[i + o], keep = up ? pr[i + o] : pr[i];
+      pr[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
     }
   }
-  const float sum = pr[0] + __shfl_xor_sync(0xffffffffu, pr[0], 1);
-  float r = 1.f / sqrtf(sum + 1e-6f);    // 1 / |k_i|, or 1 / (|q_i| sqrt(D))
-  if (lane >= 8) r = r / sqrtf(float(p.D));
+  const float mine = pr[0];
+  // lanes 16-19: 1 / |k_i|, lanes 20-23: 1 / (|q_i| sqrt(D))
+  float r = 1.f / sqrtf(mine + 1e-6f);
+  if (lane >= 20) r = r / sqrtf(float(p.D));
   float rk[4], rq[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    rk[i] = __shfl_sync(0xffffffffu, r, 2 * i);
-    rq[i] = __shfl_sync(0xffffffffu, r, 8 + 2 * i);
+    rk[i] = __shfl_sync(0xffffffffu, r, 16 + i);
+    rq[i] = __shfl_sync(0xffffffffu, r, 20 + i);
   }
   const long long row0 = ((long long)b * p.G + g) * p.Sp + s0 + blk * 4;
+  const int nr = min(4, n4 - blk * 4);
   for (int d = lane; d < Dp; d += 32)
 #pragma unroll
     for (int i = 0; i < 4; ++i)
-      if (blk * 4 + i < nr) {
+      if (i < nr) {
         p.q[(row0 + i) * Dp + d] = base[i * W + d] * rq[i];
         p.k[(row0 + i) * Dp + d] = base[i * W + Dp + d] * rk[i];
       }
-  if (p.Sp == 1 && lane == 16) p.kq[(long long)b * p.G + g] = sum * rq[0] * rk[0];
+  if (p.Sp == 1) {
+    if (lane == 6) p.pair[(long long)b * p.G + g] = mine * rq[0] * rk[0];
+    return;
+  }
+  if (lane < 16) {
+    const int y = lane < 6 ? lane : lane - 6;
+    int i, j;
+    if (lane < 6) { i = y < 1 ? 1 : y < 3 ? 2 : 3; j = y - (i * (i - 1)) / 2; }
+    else { i = y < 1 ? 0 : y < 3 ? 1 : y < 6 ? 2 : 3; j = y - (i * (i + 1)) / 2; }
+    float f = 0.f, e = 0.f;
+#pragma unroll
+    for (int x = 0; x < 4; ++x) {
+      if (x == i) f = lane < 6 ? rk[x] : rq[x];
+      if (x == j) e = rk[x];
+    }
+    p.pair[(((long long)b * p.G + g) * (p.Sp / 4) + s0 / 4 + blk) * 16 + lane] = mine * f * e;
+  }
 }
 
 // after a prompt portion: the inputs of its last taps - 1 tokens become the history (shorter portions keep part of the old one)
@@ -221,98 +246,52 @@ __global__ void __launch_bounds__(256) conv_history_kernel(const DeltaPrepArgs p
 }
 
 // ------------------------------------------------------------------------------------------------
-// the part of 16 tokens' recurrence that does not need the state: w, y (over v) and the coefficients of o
+// coefficients of four tokens of one head: [0,6) beta_i R_ij (k_i.k_j), [6,16) R_ij (q_i.k_j), [16,20) beta_i,
+// [20,24) beta_i G_i, [24,28) G_i, [28,32) R_4j
 // ------------------------------------------------------------------------------------------------
-struct DeltaWyArgs {
-  const float *q, *k, *decay, *beta;
-  float *v, *w, *coef;
-  const int* lens;
-  int S, Sp, G, H, Dp, Vp;
-};
-
-__global__ void __launch_bounds__(128) delta_wy_kernel(const DeltaWyArgs p) {
+__global__ void __launch_bounds__(128) delta_coef_kernel(const float* __restrict__ pair, const float* __restrict__ decay,
+                                                         const float* __restrict__ beta, float* __restrict__ coef, const int* __restrict__ lens,
+                                                         int B, int S, int Sp, int G, int H) {
   tfb::pdl_sync();
-  extern __shared__ __align__(16) float ws[];
-  __shared__ __align__(16) float sA[CHUNK][CHUNK];       // beta_i R_ij (k_i.k_j), j < i
-  __shared__ float sd[CHUNK], sb[CHUNK], sg[CHUNK];      // decay, beta, G
-  const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, g = h / (p.H / p.G);
-  const int Dp = p.Dp, KP = Dp + 4;
-  if (c * CHUNK >= (p.lens ? p.lens[b] : p.S)) return;
-  float* sK = ws;
-  float* sQ = ws + CHUNK * KP;
-  const float4* kb = reinterpret_cast<const float4*>(p.k + (((long long)b * p.G + g) * p.Sp + c * CHUNK) * Dp);
-  const float4* qb = reinterpret_cast<const float4*>(p.q + (((long long)b * p.G + g) * p.Sp + c * CHUNK) * Dp);
-  for (int i = tid; i < CHUNK * Dp / 4; i += 128) {
-    const int r = i / (Dp / 4), d = i % (Dp / 4) * 4;
-    *reinterpret_cast<float4*>(sK + r * KP + d) = kb[i];
-    *reinterpret_cast<float4*>(sQ + r * KP + d) = qb[i];
-  }
-  const long long hrow = ((long long)b * p.H + h) * p.Sp + c * CHUNK;
-  if (tid < CHUNK) {
-    sd[tid] = p.decay[hrow + tid];
-    sb[tid] = p.beta[hrow + tid];
-  }
-  __syncthreads();
-  if (tid < CHUNK) {
-    float x = 1.f;
-    for (int i = 0; i <= tid; ++i) x *= sd[i];
-    sg[tid] = x;
-  }
-  float* coef = p.coef + (((long long)b * p.H + h) * (p.Sp / CHUNK) + c) * COEF;
-  const int i = tid >> 3, j0 = tid & 7;
-  float kk[2] = {0.f, 0.f}, qk[2] = {0.f, 0.f};
-  for (int d = 0; d < Dp; d += 4) {
-    const float4 ki = *reinterpret_cast<const float4*>(sK + i * KP + d), qi = *reinterpret_cast<const float4*>(sQ + i * KP + d);
+  const int nb = Sp / 4;
+  const long long id = blockIdx.x * 128ll + threadIdx.x;
+  if (id >= (long long)B * H * nb) return;
+  const int blk = int(id % nb), h = int(id / nb % H), b = int(id / nb / H), g = h / (H / G);
+  if (blk * 4 >= (lens ? lens[b] : S)) return;
+  const float4 d4 = *reinterpret_cast<const float4*>(decay + ((long long)b * H + h) * Sp + blk * 4);
+  const float4 b4 = *reinterpret_cast<const float4*>(beta + ((long long)b * H + h) * Sp + blk * 4);
+  const float* pr = pair + (((long long)b * G + g) * nb + blk) * 16;
+  const float d[4] = {d4.x, d4.y, d4.z, d4.w}, be[4] = {b4.x, b4.y, b4.z, b4.w};
+  float R[4][4], c[32];
 #pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const float4 kj = *reinterpret_cast<const float4*>(sK + (j0 + 8 * e) * KP + d);
-      kk[e] = fmaf(ki.x, kj.x, fmaf(ki.y, kj.y, fmaf(ki.z, kj.z, fmaf(ki.w, kj.w, kk[e]))));
-      qk[e] = fmaf(qi.x, kj.x, fmaf(qi.y, kj.y, fmaf(qi.z, kj.z, fmaf(qi.w, kj.w, qk[e]))));
-    }
+  for (int j = 0; j < 4; ++j) {
+    R[j][j] = 1.f;
+#pragma unroll
+    for (int i = j + 1; i < 4; ++i) R[i][j] = R[i - 1][j] * d[i];
   }
+  float Gi = 1.f;
 #pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const int j = j0 + 8 * e;
-    float R = 1.f;
-    for (int l = j + 1; l <= i; ++l) R *= sd[l];
-    sA[i][j] = j < i ? sb[i] * R * kk[e] : 0.f;
-    coef[i * P_PITCH + j] = j <= i ? R * qk[e] : 0.f;
-    if (i == CHUNK - 1) coef[CHUNK * P_PITCH + CHUNK + j] = R;
+  for (int i = 0; i < 4; ++i) {
+    Gi *= d[i];
+#pragma unroll
+    for (int j = 0; j < i; ++j) c[i * (i - 1) / 2 + j] = be[i] * R[i][j] * pr[i * (i - 1) / 2 + j];
+#pragma unroll
+    for (int j = 0; j <= i; ++j) c[6 + i * (i + 1) / 2 + j] = R[i][j] * pr[6 + i * (i + 1) / 2 + j];
+    c[16 + i] = be[i];
+    c[20 + i] = be[i] * Gi;
+    c[24 + i] = Gi;
+    c[28 + i] = R[3][i];
   }
-  __syncthreads();
-  if (tid < CHUNK) coef[CHUNK * P_PITCH + tid] = sg[tid];
-  else if (tid < 2 * CHUNK)
-    for (int e = CHUNK; e < P_PITCH; ++e) coef[(tid - CHUNK) * P_PITCH + e] = 0.f;
-  // forward substitution, one column per thread
-  for (int col = tid; col < Dp + p.Vp; col += 128) {
-    const bool is_k = col < Dp;
-    float* vp = p.v + hrow * p.Vp + (col - Dp);
-    float x[CHUNK];
+  float4* out = reinterpret_cast<float4*>(coef + id * 32);
 #pragma unroll
-    for (int r = 0; r < CHUNK; ++r) x[r] = is_k ? sb[r] * sg[r] * sK[r * KP + col] : sb[r] * vp[(long long)r * p.Vp];
-#pragma unroll
-    for (int r = 1; r < CHUNK; ++r) {
-#pragma unroll
-      for (int q = 0; q < (r + 3) / 4; ++q) {
-        const float4 a = *reinterpret_cast<const float4*>(&sA[r][4 * q]);      // zeros from the diagonal on
-        x[r] = fmaf(-a.x, x[4 * q], x[r]);
-        if (4 * q + 1 < r) x[r] = fmaf(-a.y, x[4 * q + 1], x[r]);
-        if (4 * q + 2 < r) x[r] = fmaf(-a.z, x[4 * q + 2], x[r]);
-        if (4 * q + 3 < r) x[r] = fmaf(-a.w, x[4 * q + 3], x[r]);
-      }
-    }
-    float* out = is_k ? p.w + hrow * Dp + col : vp;
-    const int pitch = is_k ? Dp : p.Vp;
-#pragma unroll
-    for (int r = 0; r < CHUNK; ++r) out[(long long)r * pitch] = x[r];
-  }
+  for (int i = 0; i < 8; ++i) out[i] = make_float4(c[4 * i], c[4 * i + 1], c[4 * i + 2], c[4 * i + 3]);
 }
 
 // ------------------------------------------------------------------------------------------------
 // scan over a prompt
 // ------------------------------------------------------------------------------------------------
 struct DeltaScanArgs {
-  const float *q, *k, *w, *y, *coef;
+  const float *q, *k, *v, *coef;
   float* o;               // [B*S, H, V]
   float* state;           // [slots, H, D, V]
   const int* state_slots; // [B]
@@ -343,20 +322,25 @@ __device__ __forceinline__ float2 unpack2(u64 v) {
   return f;
 }
 
-// EPT: entries of one column per thread (a multiple of 4); TPC >= 8: threads per column group; CPT: columns per group;
-// Dp = EPT TPC.  The products of token s ^ (t & 7) of a half chunk sit in register slot s of thread t, so that each round of the
-// reduction adds a partner's upper slots to this thread's lower ones and thread t ends up with token t & 7.
+constexpr int SCAN_CHUNK = 16;   // tokens per shared-memory stage
+
+// EPT: entries of one column per thread (a multiple of 4); TPC: threads per column group; CPT: columns per group (a power of
+// two, 2 CPT <= TPC); Dp = EPT TPC.  Of a group's 2 CPT sets of products (S^T k and S^T q of each column, four tokens each) a
+// shuffle reduction leaves one set with each thread (or with each TPC / (2 CPT) threads): bits of the thread index, from the
+// top: column, then k or q.
 template <int EPT, int TPC, int CPT>
 __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaScanArgs p) {
   tfb::pdl_sync();
   extern __shared__ __align__(128) float sm[];
-  constexpr int Dp = EPT * TPC, CPW = 32 / TPC * CPT;
-  static_assert(TPC >= 8 && EPT % 4 == 0 && CHUNK == 16, "tile shape");
+  constexpr int Dp = EPT * TPC, CPW = 32 / TPC * CPT, SETS = 2 * CPT, W = TPC / SETS;
+  static_assert(SETS <= TPC && EPT % 4 == 0, "tile shape");
   const int tid = threadIdx.x, lane = tid & 31, cols = (blockDim.x >> 5) * CPW;
   const int h = blockIdx.y, b = blockIdx.z, g = h / (p.H / p.G), col0 = blockIdx.x * cols;
-  const int t = lane % TPC, t8 = t & 7, cl = (tid >> 5) * CPW + lane / TPC * CPT;   // first column of the group, within the block
+  const int t = lane % TPC, cl = (tid >> 5) * CPW + lane / TPC * CPT;      // first column of the group, within the block
+  const int set = t / W, my_col = col0 + cl + (set >> 1);                   // the products this thread ends up with
+  const bool is_q = set & 1;
   const int len = p.lens ? p.lens[b] : p.S;
-  const int stage_f = 3 * CHUNK * Dp + CHUNK * cols + COEF;
+  const int stage_f = 2 * SCAN_CHUNK * Dp + SCAN_CHUNK * cols + SCAN_CHUNK * 8;
   const uint32_t bar = smem_u32(sm + 2 * stage_f);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + 2 * stage_f + 4);
   if (tid == 0) {
@@ -370,22 +354,21 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaScanArgs p) 
   __syncthreads();
   const float* kb = p.k + ((long long)b * p.G + g) * p.Sp * Dp;
   const float* qb = p.q + ((long long)b * p.G + g) * p.Sp * Dp;
-  const float* wb = p.w + ((long long)b * p.H + h) * p.Sp * Dp;
-  const float* yb = p.y + ((long long)b * p.H + h) * p.Sp * p.Vp + col0;
-  const float* cb = p.coef + ((long long)b * p.H + h) * (p.Sp / CHUNK) * COEF;
-  const int nchunk = (len + CHUNK - 1) / CHUNK, nc = min(cols, p.Vp - col0);
-  auto issue = [&](int c) {              // warp 0: the rows of chunk c
-    if (c >= nchunk || tid >= 32) return;
+  const float* vb = p.v + ((long long)b * p.H + h) * p.Sp * p.Vp + col0;
+  const float* cb = p.coef + ((long long)b * p.H + h) * (p.Sp / 4) * 32;
+  const int nrow = (len + 3) / 4 * 4, nc = min(cols, p.Vp - col0);
+  auto issue = [&](int c) {              // warp 0: the rows of chunk c (whole groups of four)
+    const int s0 = c * SCAN_CHUNK, n = min(SCAN_CHUNK, nrow - s0);
+    if (n <= 0 || tid >= 32) return;
     float* base = sm + (c & 1) * stage_f;
     const uint32_t br = bar + (c & 1) * 8;
-    if (lane == 0) mbar_expect_tx(br, uint32_t(CHUNK * (3 * Dp + nc) + COEF) * 4);
+    if (lane == 0) mbar_expect_tx(br, uint32_t(n) * (2 * Dp + nc + 8) * 4);
     __syncwarp();
-    if (lane == 0) bulk_load(smem_u32(base), wb + (long long)c * CHUNK * Dp, CHUNK * Dp * 4, br);
-    if (lane == 1) bulk_load(smem_u32(base + CHUNK * Dp), qb + (long long)c * CHUNK * Dp, CHUNK * Dp * 4, br);
-    if (lane == 2) bulk_load(smem_u32(base + 2 * CHUNK * Dp), kb + (long long)c * CHUNK * Dp, CHUNK * Dp * 4, br);
-    if (lane == 3) bulk_load(smem_u32(base + 3 * CHUNK * Dp + CHUNK * cols), cb + (long long)c * COEF, COEF * 4, br);
-    if (lane >= 16)
-      bulk_load(smem_u32(base + 3 * CHUNK * Dp + (lane - 16) * cols), yb + (long long)(c * CHUNK + lane - 16) * p.Vp, nc * 4, br);
+    if (lane == 0) bulk_load(smem_u32(base), kb + (long long)s0 * Dp, n * Dp * 4, br);
+    if (lane == 1) bulk_load(smem_u32(base + SCAN_CHUNK * Dp), qb + (long long)s0 * Dp, n * Dp * 4, br);
+    if (lane == 2) bulk_load(smem_u32(base + 2 * SCAN_CHUNK * Dp + SCAN_CHUNK * cols), cb + (long long)s0 * 8, n * 32, br);
+    if (lane >= 16 && lane - 16 < n)
+      bulk_load(smem_u32(base + 2 * SCAN_CHUNK * Dp + (lane - 16) * cols), vb + (long long)(s0 + lane - 16) * p.Vp, nc * 4, br);
   };
   issue(0);
   issue(1);
@@ -410,110 +393,96 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaScanArgs p) 
       st[x][2 * i + 1] = pack2(f[2], f[3]);
     }
 
+  const int nchunk = (len + SCAN_CHUNK - 1) / SCAN_CHUNK;
   const long long ostep = (long long)p.H * p.V;
-  float* orow = p.o + ((long long)b * p.S * p.H + h) * p.V + col0 + cl;
+  float* orow = p.o + ((long long)b * p.S * p.H + h) * p.V + my_col;
+  const bool writer = is_q && t % W == 0 && my_col < p.V;
   for (int c = 0; c < nchunk; ++c) {
     if (!mbar_wait_warp(bar + (c & 1) * 8, (c >> 1) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) break;
     const float* base = sm + (c & 1) * stage_f;
-    const float* sy = base + 3 * CHUNK * Dp;
-    const float* sc = sy + CHUNK * cols;
-    float um[2][CPT], oq[2][CPT];        // u, and S^T q, of tokens t8 and t8 + 8
+    const float* sv = base + 2 * SCAN_CHUNK * Dp;
+    const float* sc = sv + SCAN_CHUNK * cols;
+    const int n = min(SCAN_CHUNK, len - c * SCAN_CHUNK);
+#pragma unroll 1
+    for (int r = 0; r < n; r += 4) {
+      u64 kk[4][EPT / 2];
+      float val[SETS][4];                // [2 column + (k: 0, q: 1)][token]
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      float val[8][2 * CPT];             // [slot][2 column + (w: 0, q: 1)]
+      for (int i = 0; i < 4; ++i) {
+        const ulonglong2* sk = reinterpret_cast<const ulonglong2*>(base + (r + i) * Dp) + t;
+        const ulonglong2* sq = reinterpret_cast<const ulonglong2*>(base + (SCAN_CHUNK + r + i) * Dp) + t;
+        u64 qq[EPT / 2];
 #pragma unroll
-      for (int s = 0; s < 8; ++s) {
-        const ulonglong2* sw = reinterpret_cast<const ulonglong2*>(base + (half * 8 + (s ^ t8)) * Dp) + t;
-        const ulonglong2* sq = sw + CHUNK * Dp / 4;
-        u64 a[EPT / 2];
+        for (int e = 0; e < EPT / 4; ++e) {
+          const ulonglong2 a = sk[e * TPC], q = sq[e * TPC];
+          kk[i][2 * e] = a.x;
+          kk[i][2 * e + 1] = a.y;
+          qq[2 * e] = q.x;
+          qq[2 * e + 1] = q.y;
+        }
 #pragma unroll
-        for (int y = 0; y < 2; ++y) {
+        for (int x = 0; x < CPT; ++x) {
+          u64 dk = mul2(st[x][0], kk[i][0]), dq = mul2(st[x][0], qq[0]);     // 8 CPT independent chains over the four tokens
 #pragma unroll
-          for (int e = 0; e < EPT / 4; ++e) {
-            const ulonglong2 r = y ? sq[e * TPC] : sw[e * TPC];
-            a[2 * e] = r.x;
-            a[2 * e + 1] = r.y;
+          for (int e = 1; e < EPT / 2; ++e) {
+            dk = fma2(st[x][e], kk[i][e], dk);
+            dq = fma2(st[x][e], qq[e], dq);
           }
-#pragma unroll
-          for (int x = 0; x < CPT; ++x) {
-            u64 d = mul2(st[x][0], a[0]);
-#pragma unroll
-            for (int e = 1; e < EPT / 2; ++e) d = fma2(st[x][e], a[e], d);
-            const float2 f = unpack2(d);
-            val[s][2 * x + y] = f.x + f.y;
-          }
+          const float2 a = unpack2(dk), q = unpack2(dq);
+          val[2 * x][i] = a.x + a.y;
+          val[2 * x + 1][i] = q.x + q.y;
         }
       }
 #pragma unroll
-      for (int o = TPC >> 1; o >= 8; o >>= 1)
+      for (int o = TPC >> 1, m = SETS; o > 0; o >>= 1) {
+        if (m > 1) {                     // halve the sets: keep those of this thread's half, send the others
+          const bool up = t & o;
 #pragma unroll
-        for (int s = 0; s < 8; ++s)
+          for (int y = 0; y < m / 2; ++y)
 #pragma unroll
-          for (int y = 0; y < 2 * CPT; ++y) val[s][y] += __shfl_xor_sync(0xffffffffu, val[s][y], o);
+            for (int i = 0; i < 4; ++i) {
+              const float send = up ? val[y][i] : val[y + m / 2][i], keep = up ? val[y + m / 2][i] : val[y][i];
+              val[y][i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+          m >>= 1;
+        } else {
 #pragma unroll
-      for (int o = 4; o > 0; o >>= 1)
-#pragma unroll
-        for (int s = 0; s < o; ++s)
-#pragma unroll
-          for (int y = 0; y < 2 * CPT; ++y) val[s][y] += __shfl_xor_sync(0xffffffffu, val[s + o][y], o);
+          for (int i = 0; i < 4; ++i) val[0][i] += __shfl_xor_sync(0xffffffffu, val[0][i], o);
+        }
+      }
+      const float4* cf = reinterpret_cast<const float4*>(sc + r * 8);
+      const float4 c0 = cf[0], c1 = cf[1], c2 = cf[2], c3 = cf[3], be = cf[4], bg = cf[5], gi = cf[6], r4 = cf[7];
+      float u[4];                        // right in the threads that hold a k set
+      {
+        const float* vr = sv + r * cols + cl + (set >> 1);
+        u[0] = fmaf(be.x, vr[0], -bg.x * val[0][0]);
+        u[1] = fmaf(-c0.x, u[0], fmaf(be.y, vr[cols], -bg.y * val[0][1]));
+        u[2] = fmaf(-c0.z, u[1], fmaf(-c0.y, u[0], fmaf(be.z, vr[2 * cols], -bg.z * val[0][2])));
+        u[3] = fmaf(-c1.y, u[2], fmaf(-c1.x, u[1], fmaf(-c0.w, u[0], fmaf(be.w, vr[3 * cols], -bg.w * val[0][3]))));
+      }
+      const u64 g4 = pack2(gi.w, gi.w);
+      float mine[4] = {0.f, 0.f, 0.f, 0.f};      // u of this thread's column
 #pragma unroll
       for (int x = 0; x < CPT; ++x) {
-        um[half][x] = sy[(half * 8 + t8) * cols + cl + x] - val[0][2 * x];
-        oq[half][x] = val[0][2 * x + 1];
+        float w[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          w[i] = __shfl_sync(0xffffffffu, u[i], (lane & ~(TPC - 1)) + 2 * x * W);
+          if (CPT == 1 || (set >> 1) == x) mine[i] = w[i];
+        }
+        const u64 w0 = pack2(w[0] * r4.x, w[0] * r4.x), w1 = pack2(w[1] * r4.y, w[1] * r4.y);
+        const u64 w2 = pack2(w[2] * r4.z, w[2] * r4.z), w3 = pack2(w[3] * r4.w, w[3] * r4.w);
+#pragma unroll
+        for (int e = 0; e < EPT / 2; ++e)
+          st[x][e] = fma2(kk[3][e], w3, fma2(kk[2][e], w2, fma2(kk[1][e], w1, fma2(kk[0][e], w0, mul2(st[x][e], g4)))));
       }
-    }
-    // every thread gets the 16 u of its columns
-    float u[CPT][CHUNK];
-#pragma unroll
-    for (int x = 0; x < CPT; ++x)
-#pragma unroll
-      for (int j = 0; j < CHUNK; ++j) u[x][j] = __shfl_sync(0xffffffffu, um[j >> 3][x], (lane & ~(TPC - 1)) + (j & 7));
-    const float* sG = sc + CHUNK * P_PITCH;
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      const int row = half * 8 + t8, tok = c * CHUNK + row;
-      const float4* pr = reinterpret_cast<const float4*>(sc + row * P_PITCH);
-      const float gi = sG[row];
-      float ov[CPT];
-#pragma unroll
-      for (int x = 0; x < CPT; ++x) ov[x] = gi * oq[half][x];
-#pragma unroll
-      for (int j = 0; j < 2 * (half + 1); ++j) {          // tokens 0-7 have no coefficients past the first eight
-        const float4 f = pr[j];
-#pragma unroll
-        for (int x = 0; x < CPT; ++x)
-          ov[x] = fmaf(f.w, u[x][4 * j + 3], fmaf(f.z, u[x][4 * j + 2], fmaf(f.y, u[x][4 * j + 1], fmaf(f.x, u[x][4 * j], ov[x]))));
-      }
-      if (t < 8 && tok < len) {
-#pragma unroll
-        for (int x = 0; x < CPT; ++x)
-          if (col0 + cl + x < p.V) orow[(long long)tok * ostep + x] = ov[x];
-      }
-    }
-    const u64 gl = pack2(sG[CHUNK - 1], sG[CHUNK - 1]);
-#pragma unroll
-    for (int x = 0; x < CPT; ++x)
-#pragma unroll
-      for (int e = 0; e < EPT / 2; ++e) st[x][e] = mul2(st[x][e], gl);
-    const float4* sR = reinterpret_cast<const float4*>(sG + CHUNK);
-#pragma unroll
-    for (int j = 0; j < CHUNK; ++j) {
-      const float4 R4 = sR[j >> 2];
-      const float R = (j & 3) == 0 ? R4.x : (j & 3) == 1 ? R4.y : (j & 3) == 2 ? R4.z : R4.w;
-      const ulonglong2* sk = reinterpret_cast<const ulonglong2*>(base + (2 * CHUNK + j) * Dp) + t;
-      u64 a[EPT / 2];
-#pragma unroll
-      for (int e = 0; e < EPT / 4; ++e) {
-        const ulonglong2 r = sk[e * TPC];
-        a[2 * e] = r.x;
-        a[2 * e + 1] = r.y;
-      }
-#pragma unroll
-      for (int x = 0; x < CPT; ++x) {
-        const float f = u[x][j] * R;
-        const u64 ff = pack2(f, f);
-#pragma unroll
-        for (int e = 0; e < EPT / 2; ++e) st[x][e] = fma2(a[e], ff, st[x][e]);
+      if (writer) {
+        float* op = orow + (long long)(c * SCAN_CHUNK + r) * ostep;
+        op[0] = fmaf(c1.z, mine[0], gi.x * val[0][0]);
+        if (r + 1 < n) op[ostep] = fmaf(c2.x, mine[1], fmaf(c1.w, mine[0], gi.y * val[0][1]));
+        if (r + 2 < n) op[2 * ostep] = fmaf(c2.w, mine[2], fmaf(c2.z, mine[1], fmaf(c2.y, mine[0], gi.z * val[0][2])));
+        if (r + 3 < n)
+          op[3 * ostep] = fmaf(c3.w, mine[3], fmaf(c3.z, mine[2], fmaf(c3.y, mine[1], fmaf(c3.x, mine[0], gi.w * val[0][3]))));
       }
     }
     __syncthreads();
@@ -543,8 +512,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const DeltaScanArgs p) 
 template <int EPT, int TPC, int CPT>
 static int launch_scan_tile(const DeltaScanArgs& p, int B, int nw, cudaStream_t st) {
   constexpr int CPW = 32 / TPC * CPT;
-  auto bytes = [](int w) { return (2 * (3 * CHUNK * EPT * TPC + CHUNK * w * CPW + COEF) + 8) * int(sizeof(float)); };
-  if (nw < 1 || nw > 4 || (nw * CPW) % 4) return TFB_ERR_ARG;      // rows of y are copied in 16-byte pieces
+  auto bytes = [](int w) { return (2 * (2 * SCAN_CHUNK * EPT * TPC + SCAN_CHUNK * w * CPW + SCAN_CHUNK * 8) + 8) * int(sizeof(float)); };
+  if (nw < 1 || nw > 4 || (nw * CPW) % 4) return TFB_ERR_ARG;      // rows of v are copied in 16-byte pieces
   static DeviceOnce once;
   auto kern = delta_scan_kernel<EPT, TPC, CPT>;
   if (int e = ensure_dyn_smem(once, kern, bytes(4))) return e;
@@ -555,11 +524,11 @@ static int launch_scan_tile(const DeltaScanArgs& p, int B, int nw, cudaStream_t 
 
 template <int EPT, int TPC>
 static int launch_scan(const DeltaScanArgs& p, int B, int tile, cudaStream_t st) {
-  // Wide groups (four columns) read w, q and k from shared memory a quarter as often; narrow ones spread few sequences over more
+  // Wide groups (four columns) read q and k from shared memory a quarter as often; narrow ones spread few sequences over more
   // warps.
   constexpr int GPW = 32 / TPC;
   auto warps = [&](int cpt) { return (long long)((p.V + GPW * cpt - 1) / (GPW * cpt)) * p.H * B; };
-  int cpt = warps(4) >= 3ll * sm_count() ? 4 : warps(2) >= sm_count() ? 2 : 1, nw = 4;
+  int cpt = warps(4) >= 3ll * sm_count() ? 4 : warps(2) >= 2ll * sm_count() ? 2 : 1, nw = 4;
   while (nw > 1 && nw / 2 * GPW * cpt >= 4 && (nw * GPW * cpt > (p.V + 3) / 4 * 4 || (warps(cpt) + nw - 1) / nw < 4 * sm_count() / 5)) nw >>= 1;
   if (tile > 0) {
     cpt = tile >> 4;
@@ -738,23 +707,23 @@ TFB_API int tfb_delta_padded_dim(int D) {
   return 0;
 }
 
-// Convolution, activation, unit lengths, gates and (Sp > 1) w, y and the coefficients of B sequences with S rows each, lens[b] of them
+// Convolution, activation, unit lengths, gates and (Sp > 1) the coefficients of B sequences with S rows each, lens[b] of them
 // real.  has_past: the history in conv_state belongs to these sequences (otherwise they start here and see zeros).
 TFB_API int tfb_delta_prep(const void* proj, long long ld, const void* conv_w, void* conv_state, const int* state_slots, int nslots,
                            const void* A_log, const void* dt_bias, const int* lens, float* q, float* k, float* v, float* decay, float* beta,
-                           float* kq, float* w, float* coef, int B, int S, int Sp, int G, int H, int D, int V, int taps, int has_past, int f32,
+                           float* pair, float* coef, int B, int S, int Sp, int G, int H, int D, int V, int taps, int has_past, int f32,
                            void* stream) {
   using namespace tfb;
   const int Dp = tfb_delta_padded_dim(D);
   if (B <= 0 || B > 65535 || S <= 0 || G <= 0 || H % G || G + H > 65535 || D <= 0 || V <= 0 || taps < 1) return TFB_ERR_ARG;
-  if (Sp != 1 && (Sp != (S + CHUNK - 1) / CHUNK * CHUNK || !coef || !w)) return TFB_ERR_ARG;
+  if (Sp != 1 && (Sp != (S + 3) / 4 * 4 || !coef)) return TFB_ERR_ARG;
   if (Sp == 1 && S != 1) return TFB_ERR_ARG;
   if (!Dp) return TFB_ERR_LIMIT;
-  DeltaPrepArgs p{proj, ld, conv_w, conv_state, state_slots, A_log, dt_bias, lens, q, k, v, decay, beta, kq,
+  DeltaPrepArgs p{proj, ld, conv_w, conv_state, state_slots, A_log, dt_bias, lens, q, k, v, decay, beta, pair,
                   S, Sp, G, H, D, Dp, V, (V + 3) / 4 * 4, taps, has_past, nslots};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const dim3 grid((Sp + CHUNK - 1) / CHUNK, G + H, B);
-  const int smem = (Sp == 1 ? 4 : CHUNK) * 2 * Dp * int(sizeof(float));     // at most 64 KB
+  const dim3 grid((Sp + PREP_STRIP - 1) / PREP_STRIP, G + H, B);
+  const int smem = (Sp == 1 ? 4 : PREP_STRIP) * 2 * Dp * int(sizeof(float));     // at most 64 KB
 #define TFB_PREP1(T, TAPS)                                                                 \
   {                                                                                       \
     static DeviceOnce once;                                                               \
@@ -776,22 +745,18 @@ TFB_API int tfb_delta_prep(const void* proj, long long ld, const void* conv_w, v
     if (f32) launch_k(conv_history_kernel<float>, hg, 256, 0, st, p);
     else launch_k(conv_history_kernel<bf16>, hg, 256, 0, st, p);
   }
-  if (Sp > 1) {
-    static DeviceOnce once;
-    if (int e = ensure_dyn_smem(once, delta_wy_kernel, 2 * CHUNK * (512 + 4) * int(sizeof(float)))) return e;
-    DeltaWyArgs a{q, k, decay, beta, v, w, coef, lens, S, Sp, G, H, Dp, (V + 3) / 4 * 4};
-    launch_k(delta_wy_kernel, dim3(Sp / CHUNK, H, B), 128, 2 * CHUNK * (Dp + 4) * int(sizeof(float)), st, a);
-  }
+  if (Sp > 1)
+    launch_k(delta_coef_kernel, int(((long long)B * H * (Sp / 4) + 127) / 128), 128, 0, st, pair, decay, beta, coef, lens, B, S, Sp, G, H);
   return int(cudaGetLastError());
 }
 
-// The recurrence over the prepared rows (Sp > 1); o [B*S, H, V] fp32.
-// tile 0: the launch shape is chosen from the sizes; 16 CPT + warps per block: that shape (CPT 1, 2 or 4; up to 4 warps).
-TFB_API int tfb_delta_scan(const float* q, const float* k, const float* w, const float* y, const float* coef, float* o, float* state, const int* state_slots,
+// The recurrence over the prepared rows (Sp > 1); o [B*S, H, V] fp32.  tile 0: the launch shape is chosen from the sizes;
+// 16 CPT + warps per block: that shape (CPT 1, 2 or 4; up to 4 warps).
+TFB_API int tfb_delta_scan(const float* q, const float* k, const float* v, const float* coef, float* o, float* state, const int* state_slots,
                            int nslots, const int* lens, int B, int S, int G, int H, int D, int V, int has_past, int tile, int* status, void* stream) {
   using namespace tfb;
   if (B <= 0 || B > 65535 || S <= 0 || G <= 0 || H % G || H > 65535 || D <= 0 || V <= 0) return TFB_ERR_ARG;
-  DeltaScanArgs p{q, k, w, y, coef, o, state, state_slots, lens, S, (S + CHUNK - 1) / CHUNK * CHUNK, G, H, D, V, (V + 3) / 4 * 4, has_past, nslots, status};
+  DeltaScanArgs p{q, k, v, coef, o, state, state_slots, lens, S, (S + 3) / 4 * 4, G, H, D, V, (V + 3) / 4 * 4, has_past, nslots, status};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   switch (tfb_delta_padded_dim(D)) {
     case 32: return launch_scan<4, 8>(p, B, tile, st);

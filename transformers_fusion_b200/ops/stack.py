@@ -18,7 +18,6 @@ from ._lib import c_f, c_i, c_ll, c_p, check, ptr, stream
 
 UNITS = ("tfb_host", "gemm_bf16", "stack_ops", "diff_attention", "delta_rule")    # translation units these operators need
 PAGE = 16
-CHUNK = 16           # tokens per step of the delta rule's scan
 
 _lib.register("tfb_res_norm", [c_p, c_p, c_ll, c_f, c_i, c_p, c_ll, c_p, c_ll, c_p, c_p, c_p, c_ll, c_p, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_glu_silu", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
@@ -31,8 +30,8 @@ _lib.register("tfb_diff_decode_tc", [c_i, c_i, c_i])
 _lib.register("tfb_diff_decode", [c_p, c_ll, c_p, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f,
                                   c_f, c_f, c_i, c_p, c_p])
 _lib.register("tfb_delta_padded_dim", [c_i])
-_lib.register("tfb_delta_prep", [c_p, c_ll, c_p, c_p, c_p, c_i] + [c_p] * 11 + [c_i] * 10 + [c_p])
-_lib.register("tfb_delta_scan", [c_p] * 8 + [c_i, c_p] + [c_i] * 8 + [c_p, c_p])
+_lib.register("tfb_delta_prep", [c_p, c_ll, c_p, c_p, c_p, c_i] + [c_p] * 10 + [c_i] * 10 + [c_p])
+_lib.register("tfb_delta_scan", [c_p] * 7 + [c_i, c_p] + [c_i] * 8 + [c_p, c_p])
 _lib.register("tfb_gated_norm", [c_p, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_delta_step", [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
 
@@ -211,15 +210,14 @@ def diff_decode(q, kpool, vpool, block_table, positions, H, G, D, V, window, sca
 # ---------------------------------------------------------------------------------------------------- gated delta rule
 @dataclass
 class DeltaRows:
-    """Prepared rows of B sequences: on CUDA the kernels' own layouts (see csrc/kernels/delta_rule.cu), ``v`` already
-    being y for a prompt; on the CPU q, k [T, G, D], v [T, H, V], decay, beta [T, H]."""
+    """Prepared rows of B sequences: on CUDA the kernels' own layouts (see csrc/kernels/delta_rule.cu), ``pair`` holding k.q
+    when every sequence has one row; on the CPU q, k [T, G, D], v [T, H, V], decay, beta [T, H]."""
     q: torch.Tensor
     k: torch.Tensor
     v: torch.Tensor
     decay: torch.Tensor
     beta: torch.Tensor
-    kq: Optional[torch.Tensor] = None
-    w: Optional[torch.Tensor] = None
+    pair: Optional[torch.Tensor] = None
     coef: Optional[torch.Tensor] = None
 
 
@@ -256,16 +254,14 @@ def delta_prep(proj, conv_w, conv_state, state_slots, A_log, dt_bias, lens, B, S
         return DeltaRows(q, k, y[:, 2 * G * D:].reshape(T, H, V), decay, beta)
     L = _lib.lib()
     Dp, Vp = L.tfb_delta_padded_dim(D), (V + 3) // 4 * 4
-    Sp = 1 if step and _step_fits(D, V) else (S + CHUNK - 1) // CHUNK * CHUNK
+    Sp = 1 if step and _step_fits(D, V) else (S + 3) // 4 * 4
     e = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
     r = DeltaRows(e(B, G, Sp, Dp), e(B, G, Sp, Dp), e(B, H, Sp, Vp), e(B, H, Sp), e(B, H, Sp))
-    if Sp == 1:
-        r.kq = e(B, G)
-    else:
-        r.w, r.coef = e(B, H, Sp, Dp), e(B, H, Sp // CHUNK, CHUNK * (CHUNK + 4) + 2 * CHUNK)
+    r.pair = e(B, G) if Sp == 1 else e(B, G, Sp // 4, 16)
+    r.coef = None if Sp == 1 else e(B, H, Sp // 4, 32)
     check(L.tfb_delta_prep(proj.data_ptr(), proj.stride(0), conv_w.data_ptr(), ptr(conv_state), ptr(state_slots),
                            conv_state.shape[0] if conv_state is not None else 0, A_log.data_ptr(), dt_bias.data_ptr(), ptr(lens), r.q.data_ptr(),
-                           r.k.data_ptr(), r.v.data_ptr(), r.decay.data_ptr(), r.beta.data_ptr(), ptr(r.kq), ptr(r.w), ptr(r.coef), B, S, Sp, G, H,
+                           r.k.data_ptr(), r.v.data_ptr(), r.decay.data_ptr(), r.beta.data_ptr(), r.pair.data_ptr(), ptr(r.coef), B, S, Sp, G, H,
                            D, V, taps, int(has_past), _f32(proj), stream()), "delta_prep", 1 + int(S > 1 and taps > 1) + int(Sp > 1))
     return r
 
@@ -291,7 +287,7 @@ def delta_scan(rows_: DeltaRows, state, state_slots, lens, B, S, G, H, D, V, has
                 state[sl] = st
         return out
     o = torch.empty((B * S, H, V), dtype=torch.float32, device=r.q.device)
-    check(_lib.lib().tfb_delta_scan(r.q.data_ptr(), r.k.data_ptr(), r.w.data_ptr(), r.v.data_ptr(), r.coef.data_ptr(), o.data_ptr(), state.data_ptr(),
+    check(_lib.lib().tfb_delta_scan(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.coef.data_ptr(), o.data_ptr(), state.data_ptr(),
                                     state_slots.data_ptr(), state.shape[0], ptr(lens), B, S, G, H, D, V, int(has_past), tile,
                                     _lib.status_word(o.device).data_ptr(), stream()), "delta_scan")
     return o
@@ -316,7 +312,7 @@ def delta_step(rows_: DeltaRows, state, state_slots, gate, w, eps, B, G, H, D, V
     if not r.q.is_cuda or not _step_fits(D, V):
         return gated_norm(delta_scan(r, state, state_slots, None, B, 1, G, H, D, V, has_past), gate, w, eps)
     out = rows(B, H * V, gate.dtype, r.q.device)
-    check(_lib.lib().tfb_delta_step(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.kq.data_ptr(), r.decay.data_ptr(), r.beta.data_ptr(),
+    check(_lib.lib().tfb_delta_step(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.pair.data_ptr(), r.decay.data_ptr(), r.beta.data_ptr(),
                                     state.data_ptr(), state_slots.data_ptr(), state.shape[0], gate.data_ptr(), gate.stride(0), w.data_ptr(),
                                     out.data_ptr(), out.stride(0), B, G, H, D, V, int(has_past), float(eps), _f32(gate), stream()), "delta_step")
     return out
