@@ -110,7 +110,7 @@ def feed_all(eng, seq, cuts):
 
 
 # ------------------------------------------------------------------------------------------------ mechanisms
-@pytest.mark.parametrize("dims,dim,base,yarn", [(16, 16, 1e4, None), (12, 20, 500.0, YA), (48, 64, 1e6, (2.0, 2048, 32.0, 1.0)),
+@pytest.mark.parametrize("dims,dim,base,yarn", [(16, 16, 1e4, None), (12, 20, 500.0, YA), (40, 64, 1e5, (3.0, 1024, 24.0, 2.0)),
                                                 (8, 8, 1e4, (0.5, 40, 4.0, 1.0)), (6, 10, 100.0, (1.0, 16, 2.0, 1.0))])
 def test_rotation(dims, dim, base, yarn):
     sc = dict(zip(("factor", "original", "fast", "slow"), yarn)) if yarn else None
@@ -300,7 +300,7 @@ def test_products_gpu(M, N, KK):
 
 
 @pytest.mark.gpu
-@pytest.mark.parametrize("D,dims,G,V", [(48, 48, 1, 96), (40, 12, 3, 72), (10, 6, 1, 14)])
+@pytest.mark.parametrize("D,dims,G,V", [(56, 56, 2, 88), (40, 12, 3, 72), (10, 6, 1, 14)])
 def test_rope_append_and_gather_gpu(D, dims, G, V):
     T, nq, nk = 90, 4, 2 * G
     tab = F.rope_tables(dims, 128, 1e4, "yarn", 2.0, 64, yarn_ramp_max=dims - 1)
