@@ -31,7 +31,7 @@ _lib.register("tfb_diff_decode", [c_p, c_ll, c_p, c_p, c_ll, c_p, c_i, c_i, c_p,
                                   c_f, c_f, c_i, c_p, c_p])
 _lib.register("tfb_delta_padded_dim", [c_i])
 _lib.register("tfb_delta_prep", [c_p, c_ll, c_p, c_p, c_p, c_i] + [c_p] * 10 + [c_i] * 10 + [c_p])
-_lib.register("tfb_delta_scan", [c_p] * 7 + [c_i, c_p] + [c_i] * 8 + [c_p, c_p])
+_lib.register("tfb_delta_scan", [c_p] * 7 + [c_i, c_p] + [c_i] * 7 + [c_p, c_p])
 _lib.register("tfb_gated_norm", [c_p, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_delta_step", [c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
 
@@ -266,9 +266,9 @@ def delta_prep(proj, conv_w, conv_state, state_slots, A_log, dt_bias, lens, B, S
     return r
 
 
-def delta_scan(rows_: DeltaRows, state, state_slots, lens, B, S, G, H, D, V, has_past, tile: int = 0):
+def delta_scan(rows_: DeltaRows, state, state_slots, lens, B, S, G, H, D, V, has_past):
     """The recurrence over prepared rows; ``state`` [slots, H, D, V] fp32 is read (``has_past``) and updated.  Returns fp32
-    [B*S, H, V] (rows past a sequence's length are unspecified).  ``tile``: launch shape of the kernel (0: chosen from the sizes)."""
+    [B*S, H, V] (rows past a sequence's length are unspecified)."""
     r = rows_
     if not r.q.is_cuda:
         out = torch.zeros(B * S, H, V)
@@ -288,7 +288,7 @@ def delta_scan(rows_: DeltaRows, state, state_slots, lens, B, S, G, H, D, V, has
         return out
     o = torch.empty((B * S, H, V), dtype=torch.float32, device=r.q.device)
     check(_lib.lib().tfb_delta_scan(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.coef.data_ptr(), o.data_ptr(), state.data_ptr(),
-                                    state_slots.data_ptr(), state.shape[0], ptr(lens), B, S, G, H, D, V, int(has_past), tile,
+                                    state_slots.data_ptr(), state.shape[0], ptr(lens), B, S, G, H, D, V, int(has_past),
                                     _lib.status_word(o.device).data_ptr(), stream()), "delta_scan")
     return o
 
