@@ -214,3 +214,102 @@ class PlainLanedra:
             out.append(int(lg[-1].argmax()))
             lg = self.run([out[-1]], st)
         return out
+
+
+# ---------------------------------------------------------------------------------------------------- latent attention
+def layer_norm(x, w, b, eps):
+    m = x.mean(-1, keepdim=True)
+    d = x - m
+    return d / torch.sqrt((d * d).mean(-1, keepdim=True) + eps) * w + b
+
+
+def latent_rows(h, dkv, norm, eps):
+    """What latent attention remembers of a token: a projection of its input, divided by its root mean square and weighted."""
+    return rms(h @ dkv.T, eps) * norm
+
+
+def latent_attend(q, c, uk, uv, heads, dim, vdim, scale):
+    """Softmax attention of q [T, heads * dim] (the last T positions) whose keys and values are read out of the latents c [N, rank],
+    head by head; returns [T, heads, vdim]."""
+    out = []
+    for h in range(heads):
+        k = c @ uk[h * dim:(h + 1) * dim].T
+        v = c @ uv[h * vdim:(h + 1) * vdim].T
+        out.append(attend(q[:, h * dim:(h + 1) * dim], k, v, scale))
+    return torch.stack(out, 1)
+
+
+def head_gate(o, z):
+    """o [T, heads, vdim], one gate logit per head z [T, heads]."""
+    return o / (1 + torch.exp(-z))[..., None]
+
+
+# ---------------------------------------------------------------------------------------------------- feed-forwards
+def relu2(z):
+    return torch.where(z > 0, z * z, torch.zeros_like(z))
+
+
+def squared_mlp(h, up, down):
+    return relu2(h @ up.T) @ down.T
+
+
+def route(z, top):
+    """One token's router logits -> [(expert, weight)]: the ``top`` largest logits, softmax over those alone."""
+    order = sorted(range(len(z)), key=lambda e: (-float(z[e]), e))[:top]
+    e = [math.exp(float(z[i]) - float(z[order[0]])) for i in order]
+    return [(i, x / sum(e)) for i, x in zip(order, e)]
+
+
+def mixture(h, router, bias, top, experts, shared=None):
+    """Gated feed-forward experts ((gate, up, down) each) chosen per token, plus one that every token runs."""
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for i, w in route(router @ h[t] + bias, top):
+            out[t] += w * swiglu(h[t], *experts[i])
+    return out if shared is None else out + swiglu(h, *shared)
+
+
+class PlainTekenex:
+    """As PlainLanedra, for layers of latent attention with dense or mixture feed-forwards, a layer norm and a scale on every
+    sublayer's output and the embedding as the head."""
+
+    def __init__(self, cfg, tensors):
+        self.cfg = cfg
+        self.w = {n: t.to(DT) for n, t in tensors.items()}
+
+    def start(self):
+        return {"pos": 0, "c": [torch.zeros(0, l["mixer"]["kv_rank"], dtype=DT) for l in self.cfg["layers"]]}
+
+    def mixer(self, i, x, st):
+        m, w, p = self.cfg["layers"][i]["mixer"], self.w, f"l{i}.mix."
+        st["c"][i] = torch.cat([st["c"][i], latent_rows(x, w[p + "dkv"], w[p + "dkv.norm"], self.cfg["norm"]["eps"])])
+        o = latent_attend(x @ w[p + "q"].T, st["c"][i], w[p + "uk"], w[p + "uv"], m["heads"], m["dim"], m["vdim"], m["scale"])
+        return head_gate(o, x @ w[p + "g"].T).reshape(x.shape[0], -1) @ w[p + "o"].T
+
+    def ff(self, i, x):
+        m, w, p = self.cfg["layers"][i]["mlp"], self.w, f"l{i}.mlp."
+        if m["kind"] == "dense":
+            return squared_mlp(x, w[p + "up"], w[p + "down"])
+        three = lambda q: tuple(w[p + q + n] for n in (".gate", ".up", ".down"))
+        r = m["router"]
+        return mixture(x, w[p + "router"], w[p + "router.b"], r["top"], [three(f"e{e}") for e in range(r["experts"])],
+                       three("shared") if m.get("shared") else None)
+
+    def norm(self, name, x):
+        return layer_norm(x, self.w[name], self.w[name + ".b"], self.cfg["norm"]["eps"])
+
+    def run(self, tokens, st=None, residuals=None):
+        w = self.w
+        st = st if st is not None else self.start()
+        x = w["embed"][torch.tensor(tokens)]
+        for i, layer in enumerate(self.cfg["layers"]):
+            p = f"l{i}."
+            x = x + self.norm(p + "norm1", self.mixer(i, x, st)) * w[p + "ls1"]
+            if layer["mlp"] is not None:
+                x = x + self.norm(p + "norm2", self.ff(i, x)) * w[p + "ls2"]
+            if residuals is not None:
+                residuals.append(x.clone())
+        st["pos"] += len(tokens)
+        return self.norm("final.norm", x) @ w["embed"].T
+
+    greedy = PlainLanedra.greedy

@@ -18,9 +18,11 @@ def _folder_info(path):
     print(f"Architecture: {c.architecture}")
     print(f"Config: vocab={c.vocab_size} hidden={c.hidden_size} layers={c.num_layers}")
     for i, l in enumerate(c.layers):
-        m = l.mixer
+        m, x = l.mixer, l.mixture
+        sizes = "".join(f" {n}={getattr(m, n)}" for n in ("heads", "kv_heads", "dim", "vdim", "kv_rank") if hasattr(m, n))
         extra = "" if m.kind != "attention" else (f" window={m.window}" if m.window else "") + (f" kv_from={m.kv_from}" if m.kv_from is not None else "")
-        print(f"  layer {i}: {m.kind} heads={m.heads} kv_heads={m.kv_heads} dim={m.dim} vdim={m.vdim}{extra} ffn={l.ffn_hidden_size or 'none'}")
+        ffn = f"ffn={l.ffn_hidden_size or 'none'}" if x is None else f"experts={x.experts} top={x.top} ffn={x.ff}" + (f" shared={x.shared_ff}" if x.shared_ff else "")
+        print(f"  layer {i}: {m.kind}{sizes}{extra} {ffn}")
     total = 0
     for s in srcs:
         for n in s.names:

@@ -61,7 +61,7 @@ struct GemmParams {
   const __nv_bfloat16* residual;  // [M, ldr] or null (bf16 output mode only)
   long long ldr;
   float alpha;
-  int act;       // 0 none, 1 relu, 2 gelu(tanh), 3 silu
+  int act;       // 0 none, 1 relu, 2 gelu(tanh), 3 silu, 4 relu squared
   int out_mode;  // 0 bf16 store, 1 fp32 store, 2 fp32 atomic accumulate
   int splits, kb_per_split, tiles_m, tiles_n;
   int raster_gn;   // tile order: groups of raster_gn tile columns; inside a group n runs fastest, then m
@@ -281,6 +281,7 @@ __device__ __forceinline__ float apply_act(float v, int act) {
     case 1: return fmaxf(v, 0.f);
     case 2: return gelu_tanh(v);
     case 3: return silu(v);
+    case 4: v = fmaxf(v, 0.f); return v * v;
     default: return v;
   }
 }

@@ -1,0 +1,1032 @@
+// Latent attention: per token one latent c of R entries is cached, from which every head h reads its key W_uk,h c and its value
+// W_uv,h c; causal softmax without positions, one output gate per head.
+//
+//   latent_append      norm of the latents and their append to the pages
+//   head_attn_fwd      prompts, bf16, tcgen05, over keys and values that a product has read out of the latents: one CTA per (sequence,
+//                      head, 256 queries) as two 128-query tiles that share every key / value tile and take turns on the
+//                      tensor core; keys and values may have different sizes; the gate is applied in the epilogue
+//   head_linear        one small product per head for the rows of a decode step (mma.sync): queries into the latent space
+//                      (q . W_uk c = (W_uk^T q) . c), and values out of the attention's result (sum_j a_j W_uv c_j = W_uv sum_j a_j c_j)
+//   latent_decode      one query per sequence over the paged latents, bf16, mma.sync: the query heads are the rows of one or two 16-row
+//                      tiles, and the latents are keys and values of all of them, so a cached row is read once.  Split over
+//                      the keys; a second kernel merges the splits.
+//   attn_any           any sizes, bf16 or fp32, prompts (keys and values read out) or decoding (over the latents): fp32 FMA
+//                      throughout, online softmax over 32-key tiles.
+#include "tfb_elem.cuh"
+#include "tfb_host.h"
+#include "tfb_mma.cuh"
+
+namespace tfb {
+TFB_BOUNDS_DEFINE(latent_attention)
+
+constexpr float LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
+
+// ------------------------------------------------------------------------------------------------
+// v = c / rms(c) * w, to out and to the pools' slots; one warp per row
+// ------------------------------------------------------------------------------------------------
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) latent_append_kernel(const T* __restrict__ c, long long ldc, const T* __restrict__ w, float eps,
+                                                            const long long* __restrict__ slots, T* __restrict__ out, long long ldo,
+                                                            T* __restrict__ pool, long long nslots, int width, int rows, int R) {
+  tfb::pdl_sync();
+  const int r = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (r >= rows) return;
+  const T* src = c + r * ldc;
+  float ss = 0.f;
+  for (int i = lane * VEC; i < R; i += 32 * VEC) {
+    float v[VEC];
+    load_n<VEC>(src + i, v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss = fmaf(v[e], v[e], ss);
+  }
+  const float f = 1.f / sqrtf(warp_add(ss) / R + eps);
+  long long slot = slots ? slots[r] : -1;
+  TFB_BOUNDS(slot < nslots, 51, slot, nslots);
+  if (slot >= nslots) slot = -1;
+  for (int i = lane * VEC; i < R; i += 32 * VEC) {
+    float v[VEC], g[VEC];
+    load_n<VEC>(src + i, v);
+    load_n<VEC>(w + i, g);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = v[e] * f * g[e];
+    if (out) store_n<VEC>(out + r * ldo + i, v);
+    if (slot >= 0) store_n<VEC>(pool + slot * width + i, v);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// prompts on tcgen05
+// ------------------------------------------------------------------------------------------------
+struct HeadAttnParams {
+  int B, S, H, G;
+  int Skv, q_off;         // keys per sequence; query i sees keys 0 .. i + q_off
+  int V;
+  float scale;
+  const __nv_bfloat16* gate;    // [B*S, ldg] or null
+  long long ldg;
+  __nv_bfloat16* O;
+  long long ldo;
+  int* status;
+};
+
+constexpr int HA_THREADS = 320;
+constexpr int HA_BM = 128, HA_BN = 128;
+constexpr int HA_BOX = 128 * 128;       // bytes of 128 rows of 64 entries
+
+template <int DK, int DV>
+struct HeadSmem {
+  static constexpr int NBK = DK / 64, NBV = DV / 64;
+  static constexpr int QT = NBK * HA_BOX, KT = NBK * HA_BOX, VT = NBV * HA_BOX, STAGE = KT + VT;
+  static constexpr int AVAIL = 227 * 1024 - 1024 - 256 - 2 * QT;
+  static constexpr int STAGES = AVAIL / STAGE > 4 ? 4 : AVAIL / STAGE;
+  static constexpr int KV_OFF = 2 * QT;
+  static constexpr int BAR_OFF = KV_OFF + STAGES * STAGE;
+  static constexpr int TOTAL = BAR_OFF + 256 + 1024;
+  static_assert(STAGES >= 2, "two stages at least");
+};
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// running maximum over the 128 scores of this thread's row; keys after `hi` (index within the tile) do not count
+template <bool MASK>
+__device__ __forceinline__ float tile_max(uint32_t tS, float m, int hi) {
+  float mx0 = m, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
+#pragma unroll 1
+  for (int c = 0; c < HA_BN / 32; ++c) {
+    uint32_t v[32];
+    tmem_ld_32x32(tS + c * 32, v);
+    tmem_ld_wait();
+    if (MASK) {
+#pragma unroll
+      for (int i = 0; i < 32; ++i)
+        if (c * 32 + i > hi) v[i] = 0xff800000u;
+    }
+#pragma unroll
+    for (int i = 0; i < 32; i += 8) {
+      mx0 = fmax3(mx0, __uint_as_float(v[i]), __uint_as_float(v[i + 1]));
+      mx1 = fmax3(mx1, __uint_as_float(v[i + 2]), __uint_as_float(v[i + 3]));
+      mx2 = fmax3(mx2, __uint_as_float(v[i + 4]), __uint_as_float(v[i + 5]));
+      mx3 = fmax3(mx3, __uint_as_float(v[i + 6]), __uint_as_float(v[i + 7]));
+    }
+  }
+  return fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3));
+}
+
+// p = 2^(s * sl2 - mb) over the row, written back over the scores as bf16 pairs; returns the row sum
+template <bool MASK>
+__device__ __forceinline__ float tile_probs(uint32_t tS, float sl2, float mb, int hi) {
+  float rs[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 1
+  for (int c = 0; c < HA_BN / 32; ++c) {
+    uint32_t v[32], pk[16];
+    tmem_ld_32x32(tS + c * 32, v);
+    tmem_ld_wait();
+#pragma unroll
+    for (int i = 0; i < 16; i += 2) {
+      float q[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        q[e] = ex2(fmaf(__uint_as_float(v[2 * i + e]), sl2, -mb));
+        if (MASK && c * 32 + 2 * i + e > hi) q[e] = 0.f;
+        rs[e] += q[e];
+      }
+      pk[i] = pack_bf16(q[0], q[1]);
+      pk[i + 1] = pack_bf16(q[2], q[3]);
+    }
+    tmem_st_32x16(tS + c * 16, pk);
+  }
+  return (rs[0] + rs[1]) + (rs[2] + rs[3]);
+}
+
+template <int DK, int DV>
+__global__ void __launch_bounds__(HA_THREADS, 1)
+head_attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk, const __grid_constant__ CUtensorMap tv,
+                     const HeadAttnParams p) {
+  using L = HeadSmem<DK, DV>;
+  constexpr int ST = L::STAGES;
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const uint32_t sQ = smem_u32(smem);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::BAR_OFF);
+  const uint32_t bar_q = smem_u32(bars);
+  const uint32_t bar_kv_full = bar_q + 8;
+  const uint32_t bar_kv_empty = bar_kv_full + ST * 8;
+  const uint32_t bar_s_full = bar_kv_empty + ST * 8;
+  const uint32_t bar_p_ready = bar_s_full + 16;
+  const uint32_t bar_o_full = bar_p_ready + 16;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 1 + 2 * ST + 6);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int npair = (p.S + 2 * HA_BM - 1) / (2 * HA_BM);
+  const int bh = p.B * p.H;
+  const int pair = npair - 1 - int(blockIdx.x) / bh;   // the longest (latest) query blocks first
+  const int rem = int(blockIdx.x) % bh;
+  const int b = rem / p.H, h = rem % p.H, hk = h / (p.H / p.G);
+  int n_t[2];                                          // key blocks each tile visits (0: the tile lies past the end)
+#pragma unroll
+  for (int t = 0; t < 2; ++t) {
+    const int q0 = (pair * 2 + t) * HA_BM;
+    n_t[t] = q0 >= p.S ? 0 : (min(q0 + HA_BM, p.S) - 1 + p.q_off) / HA_BN + 1;
+  }
+  const int n_kv = max(n_t[0], n_t[1]);
+
+  if (threadIdx.x == 0) {
+    mbar_init(bar_q, 1);
+    for (int s = 0; s < ST; ++s) {
+      mbar_init(bar_kv_full + s * 8, 1);
+      mbar_init(bar_kv_empty + s * 8, 1);
+    }
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(bar_s_full + i * 8, 1);
+      mbar_init(bar_p_ready + i * 8, 128);
+      mbar_init(bar_o_full + i * 8, 1);
+    }
+    *abort_flag = 0;
+    mbar_fence_init();
+    tma_prefetch_desc(&tq);
+    tma_prefetch_desc(&tk);
+    tma_prefetch_desc(&tv);
+  }
+  if (warp == 1) {
+    tmem_alloc(smem_u32(tmem_slot), 512);
+    tmem_relinquish();
+  }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = *tmem_slot;
+  tfb::pdl_sync();
+  const uint32_t tS0 = tmem_base, tO0 = tmem_base + 256;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      mbar_expect_tx(bar_q, 2 * L::QT);
+#pragma unroll
+      for (int t = 0; t < 2; ++t)
+#pragma unroll
+        for (int i = 0; i < L::NBK; ++i) tma_load_4d(sQ + t * L::QT + i * HA_BOX, &tq, bar_q, i * 64, h, (pair * 2 + t) * HA_BM, b);
+      for (int j = 0; j < n_kv; ++j) {
+        const int st = j % ST;
+        if (!mbar_wait(bar_kv_empty + st * 8, ((j / ST) & 1) ^ 1, abort_flag, p.status, ST_TIMEOUT_EMPTY)) break;
+        const uint32_t fb = bar_kv_full + st * 8, base = sQ + L::KV_OFF + st * L::STAGE;
+        mbar_expect_tx(fb, L::STAGE);
+#pragma unroll
+        for (int i = 0; i < L::NBK; ++i) tma_load_4d(base + i * HA_BOX, &tk, fb, i * 64, hk, j * HA_BN, b);
+#pragma unroll
+        for (int i = 0; i < L::NBV; ++i) tma_load_4d(base + L::KT + i * HA_BOX, &tv, fb, i * 64, hk, j * HA_BN, b);
+      }
+      if (*abort_flag) {  // unwinding: bounded wait for copies already issued
+        const uint64_t t0 = globaltimer_ns();
+        while (globaltimer_ns() - t0 < 200000ull) {}
+      }
+    }
+  } else if (warp == 1) {
+    if (lane == 0) {
+      constexpr uint32_t idesc_s = umma_idesc(FMT_BF16, FMT_BF16, false, false, HA_BM, HA_BN);
+      constexpr uint32_t idesc_o = umma_idesc(FMT_BF16, FMT_BF16, false, true, HA_BM, DV);
+      auto issue_s = [&](int t, int j) {
+        const uint32_t sK = sQ + L::KV_OFF + (j % ST) * L::STAGE, sQt = sQ + t * L::QT, tS = tS0 + t * 128;
+#pragma unroll
+        for (int k = 0; k < DK / 16; ++k) {
+          const uint32_t off = (k >> 2) * HA_BOX + (k & 3) * 32;
+          umma_f16_ss(tS, umma_smem_desc(sQt + off, 16, 1024), umma_smem_desc(sK + off, 16, 1024), idesc_s, k > 0);
+        }
+        umma_commit(bar_s_full + t * 8);
+      };
+      bool ok = mbar_wait(bar_q, 0, abort_flag, p.status, ST_TIMEOUT_FULL) &&
+                mbar_wait(bar_kv_full, 0, abort_flag, p.status, ST_TIMEOUT_FULL);
+      if (ok) {
+        tc_fence_after();
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+          if (n_t[t] > 0) issue_s(t, 0);
+      }
+      for (int j = 0; j < n_kv && ok; ++j) {
+        if (j + 1 < n_kv) {
+          const int st1 = (j + 1) % ST;
+          if (!mbar_wait(bar_kv_full + st1 * 8, ((j + 1) / ST) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) break;
+          tc_fence_after();
+        }
+        const int st = j % ST;
+        const uint32_t sV = sQ + L::KV_OFF + st * L::STAGE + L::KT;
+#pragma unroll
+        for (int t = 0; t < 2; ++t) {
+          if (!ok || j >= n_t[t]) continue;
+          if (!mbar_wait(bar_p_ready + t * 8, j & 1, abort_flag, p.status, ST_TIMEOUT_TMEM_EMPTY)) {
+            ok = false;
+            continue;
+          }
+          tc_fence_after();
+          const uint32_t tP = tS0 + t * 128, tO = tO0 + t * 128;
+#pragma unroll
+          for (int k = 0; k < HA_BN / 16; ++k)     // V tile: [key rows][64-column boxes], MN-major B
+            umma_f16_ts(tO, tP + k * 8, umma_smem_desc(sV + k * 2048, HA_BOX, 1024), idesc_o, k > 0);
+          if (j + 1 < n_t[t]) issue_s(t, j + 1);   // its commit also covers the P V product above
+          else umma_commit(bar_o_full + t * 8);
+        }
+        if (ok) umma_commit(bar_kv_empty + st * 8);
+      }
+    }
+  } else {
+    const int t = (warp - 2) >> 2, quad = warp & 3, r = quad * 32 + lane;
+    const int q0 = (pair * 2 + t) * HA_BM, q_idx = q0 + r;
+    const int n_mine = t ? n_t[1] : n_t[0];
+    const uint32_t lane_off = uint32_t(quad * 32) << 16;
+    const uint32_t tS = tS0 + t * 128 + lane_off, tO = tO0 + t * 128 + lane_off;
+    const float sl2 = p.scale * LOG2E;
+    const int hi_g = min(q_idx + p.q_off, p.Skv - 1);
+    float m = -INFINITY, l = 0.f, alpha_prev = 1.f;
+    float o[DV];
+#pragma unroll
+    for (int i = 0; i < DV; ++i) o[i] = 0.f;
+    bool ok = true;
+    for (int j = 0; j < n_mine; ++j) {
+      if (!mbar_wait_warp(bar_s_full + t * 8, j & 1, abort_flag, p.status, ST_TIMEOUT_TMEM_FULL)) {
+        ok = false;
+        break;
+      }
+      tc_fence_after();
+      const int k0 = j * HA_BN, hi = hi_g - k0;
+      const bool need_mask = k0 + HA_BN - 1 > q0 + p.q_off || k0 + HA_BN > p.Skv;
+      // a query that sits past the end of its sequence may see no key of its last block; its row is not stored
+      const float mx = need_mask ? tile_max<true>(tS, m, hi) : tile_max<false>(tS, m, hi);
+      if (j > 0) {  // O(j-1) is complete: the commit behind S(j) was issued after it
+#pragma unroll
+        for (int c = 0; c < DV / 32; ++c) {
+          uint32_t v[32];
+          tmem_ld_32x32(tO + c * 32, v);
+          tmem_ld_wait();
+#pragma unroll
+          for (int i = 0; i < 32; ++i) o[c * 32 + i] = fmaf(o[c * 32 + i], alpha_prev, __uint_as_float(v[i]));
+        }
+      }
+      const float mb = (mx == -INFINITY) ? 0.f : mx * sl2;
+      const float alpha = (m == -INFINITY) ? 0.f : ex2(m * sl2 - mb);
+      const float rs = need_mask ? tile_probs<true>(tS, sl2, mb, hi) : tile_probs<false>(tS, sl2, mb, hi);
+      l = fmaf(l, alpha, rs);
+      m = mx;
+      tmem_st_wait();
+      tc_fence_before();
+      mbar_arrive(bar_p_ready + t * 8);
+      alpha_prev = alpha;
+    }
+    if (ok && n_mine > 0 && mbar_wait_warp(bar_o_full + t * 8, 0, abort_flag, p.status, ST_TIMEOUT_TMEM_FULL)) {
+      tc_fence_after();
+#pragma unroll
+      for (int c = 0; c < DV / 32; ++c) {
+        uint32_t v[32];
+        tmem_ld_32x32(tO + c * 32, v);
+        tmem_ld_wait();
+#pragma unroll
+        for (int i = 0; i < 32; ++i) o[c * 32 + i] = fmaf(o[c * 32 + i], alpha_prev, __uint_as_float(v[i]));
+      }
+      if (q_idx < p.S) {
+        const long long row = (long long)b * p.S + q_idx;
+        float f = l > 0.f ? 1.f / l : 0.f;
+        if (p.gate) f *= sigmoid_exact(__bfloat162float(p.gate[row * p.ldg + h]));
+        __nv_bfloat16* op = p.O + row * p.ldo + h * p.V;
+#pragma unroll
+        for (int c = 0; c < DV / 8; ++c) {
+          if (c * 8 < p.V) {
+            uint4 u;
+            u.x = pack_bf16(o[c * 8 + 0] * f, o[c * 8 + 1] * f);
+            u.y = pack_bf16(o[c * 8 + 2] * f, o[c * 8 + 3] * f);
+            u.z = pack_bf16(o[c * 8 + 4] * f, o[c * 8 + 5] * f);
+            u.w = pack_bf16(o[c * 8 + 6] * f, o[c * 8 + 7] * f);
+            *reinterpret_cast<uint4*>(op + c * 8) = u;
+          }
+        }
+      }
+    }
+  }
+
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, 512);
+  }
+}
+
+template <int DK, int DV>
+static int launch_head_attn(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, int D, const HeadAttnParams& p,
+                            cudaStream_t st) {
+  using L = HeadSmem<DK, DV>;
+  static DeviceOnce once;
+  auto kern = head_attn_fwd_kernel<DK, DV>;
+  if (int e = ensure_dyn_smem(once, kern, L::TOTAL)) return e;
+  CUtensorMap tq, tk, tv;
+  int rc;
+  const uint64_t d = D, vv = p.V, S = p.S, Skv = p.Skv, B = p.B;
+  if ((rc = make_tmap_4d(&tq, q, 2, {d, uint64_t(p.H), S, B}, {d * 2, uint64_t(ldq) * 2, uint64_t(ldq) * 2 * S}, {64, 1, HA_BM, 1}))) return rc;
+  if ((rc = make_tmap_4d(&tk, k, 2, {d, uint64_t(p.G), Skv, B}, {d * 2, uint64_t(ldk) * 2, uint64_t(ldk) * 2 * Skv}, {64, 1, HA_BN, 1}))) return rc;
+  if ((rc = make_tmap_4d(&tv, v, 2, {vv, uint64_t(p.G), Skv, B}, {vv * 2, uint64_t(ldv) * 2, uint64_t(ldv) * 2 * Skv}, {64, 1, HA_BN, 1}))) return rc;
+  launch_k(kern, ((p.S + 2 * HA_BM - 1) / (2 * HA_BM)) * p.B * p.H, HA_THREADS, L::TOTAL, st, tq, tk, tv, p);
+  return int(cudaGetLastError());
+}
+
+// ------------------------------------------------------------------------------------------------
+// one product per head for few rows: out[m, h * out_head + n] = sum_k x[m, h * x_head + k] W_h[n, k] (* sigmoid(gate[m, h]))
+// KN: the blocks of W are stored [K, N].  64 rows x 32 columns per block, the next 64-deep chunk in registers while one is used.
+// ------------------------------------------------------------------------------------------------
+struct HeadLinearArgs {
+  const __nv_bfloat16 *x, *w;
+  long long ldx, ldw;
+  __nv_bfloat16* out;
+  long long ldo;
+  const __nv_bfloat16* gate;
+  long long ldg;
+  int M, N, K, x_head, out_head;     // columns N .. out_head of a head are written as zeros
+  int vec_x, vec_w;                  // 16-byte loads are aligned
+};
+
+constexpr int HL_M = 64, HL_N = 32, HL_K = 64;
+
+__device__ __forceinline__ uint4 load8(const __nv_bfloat16* p, int n, int vec) {   // n of 8 entries, the others zero
+  if (n <= 0) return make_uint4(0u, 0u, 0u, 0u);
+  if (vec && n >= 8) return *reinterpret_cast<const uint4*>(p);
+  uint32_t u[4] = {0u, 0u, 0u, 0u};
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+    if (i < n) u[i >> 1] |= uint32_t(__bfloat16_as_ushort(p[i])) << ((i & 1) * 16);
+  return make_uint4(u[0], u[1], u[2], u[3]);
+}
+
+template <bool KN>
+__global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinearArgs p) {
+  tfb::pdl_sync();
+  constexpr int PA = HL_K * 2 + 16, PB = KN ? HL_N * 2 + 16 : HL_K * 2 + 16;        // byte pitches
+  constexpr int RB = KN ? HL_K : HL_N, CB = KN ? HL_N / 8 : HL_K / 8;               // rows and 16-byte pieces of the W chunk
+  __shared__ __align__(16) uint8_t sA[2][HL_M * PA];
+  __shared__ __align__(16) uint8_t sB[2][RB * PB];
+  const int n0 = blockIdx.x * HL_N, h = blockIdx.y, m0 = blockIdx.z * HL_M;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const __nv_bfloat16* x = p.x + (long long)h * p.x_head;
+  const __nv_bfloat16* w = p.w + (long long)h * (KN ? p.K : p.N) * p.ldw;
+  uint4 ra[4], rb[2];
+  auto fetch = [&](int k0) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int e = tid + i * 128, r = e >> 3, c = (e & 7) * 8;
+      ra[i] = m0 + r < p.M ? load8(x + (m0 + r) * p.ldx + k0 + c, p.K - k0 - c, p.vec_x) : make_uint4(0u, 0u, 0u, 0u);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int e = tid + i * 128, r = e / CB, c = (e % CB) * 8;
+      if (KN) rb[i] = k0 + r < p.K ? load8(w + (k0 + r) * p.ldw + n0 + c, p.N - n0 - c, p.vec_w) : make_uint4(0u, 0u, 0u, 0u);
+      else rb[i] = n0 + r < p.N ? load8(w + (n0 + r) * p.ldw + k0 + c, p.K - k0 - c, p.vec_w) : make_uint4(0u, 0u, 0u, 0u);
+    }
+  };
+  auto put = [&](int s) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int e = tid + i * 128;
+      *reinterpret_cast<uint4*>(sA[s] + (e >> 3) * PA + (e & 7) * 16) = ra[i];
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int e = tid + i * 128;
+      *reinterpret_cast<uint4*>(sB[s] + (e / CB) * PB + (e % CB) * 16) = rb[i];
+    }
+  };
+  float acc[4][4];
+#pragma unroll
+  for (int n = 0; n < 4; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+  fetch(0);
+  put(0);
+  __syncthreads();
+  int s = 0;
+  for (int k0 = 0; k0 < p.K; k0 += HL_K, s ^= 1) {
+    if (k0 + HL_K < p.K) fetch(k0 + HL_K);
+    if (m0 + warp * 16 < p.M) {
+      const uint32_t a0 = smem_u32(sA[s]) + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PA + (lane >> 4) * 16;
+      const uint32_t b0 = KN ? smem_u32(sB[s]) + ((lane & 7) + ((lane >> 3) & 1) * 8) * PB + (lane >> 4) * 16
+                             : smem_u32(sB[s]) + ((lane & 7) + (lane >> 4) * 8) * PB + ((lane >> 3) & 1) * 16;
+#pragma unroll
+      for (int ks = 0; ks < HL_K / 16; ++ks) {
+        uint32_t a[4];
+        ldsm(a0 + ks * 32, a);
+#pragma unroll
+        for (int nb = 0; nb < 2; ++nb) {
+          uint32_t b[4];
+          if (KN) ldsm_t(b0 + ks * 16 * PB + nb * 32, b);
+          else ldsm(b0 + nb * 16 * PB + ks * 32, b);
+          mma_bf16(acc[2 * nb], a, b[0], b[1]);
+          mma_bf16(acc[2 * nb + 1], a, b[2], b[3]);
+        }
+      }
+    }
+    if (k0 + HL_K < p.K) put(s ^ 1);
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int m = m0 + warp * 16 + (lane >> 2) + 8 * i;
+    if (m >= p.M) continue;
+    const float f = p.gate ? sigmoid_exact(__bfloat162float(p.gate[m * p.ldg + h])) : 1.f;
+    __nv_bfloat16* o = p.out + m * p.ldo + (long long)h * p.out_head;
+#pragma unroll
+    for (int n = 0; n < 4; ++n)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int col = n0 + n * 8 + (lane & 3) * 2 + e;
+        if (col < p.out_head) o[col] = __float2bfloat16(acc[n][2 * i + e] * f);
+      }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// decoding over the paged latents on mma.sync
+// ------------------------------------------------------------------------------------------------
+struct LatentDecodeArgs {
+  const __nv_bfloat16* q;     // [B, ldq]: H heads of W entries
+  long long ldq;
+  const __nv_bfloat16* pool;  // [slots][W]
+  long long nslots;
+  const int* block_table;
+  int max_pages, page;
+  const int* positions;       // [B] position of the query (it sees itself: its row is in the cache)
+  int H, W, splits;
+  float scale;
+  __nv_bfloat16* o;           // [B, ldo] (one split)
+  long long ldo;
+  float *acc, *ml;            // [B, H, splits, W], [B, H, splits, 2] (several)
+  int* status;
+};
+
+constexpr int LD_THREADS = 256;
+constexpr int LD_KEYS = 64;
+
+// RC: columns of a latent in shared memory (zeros past W); MT: 16-row tiles of query heads.  Of the eight warps, two share the keys
+// and four the columns in the scores (the partial scores meet in shared memory); each takes an eighth of the columns in the
+// product with the weights.
+template <int RC, int MT>
+struct LatentSmem {
+  static constexpr int RP = RC * 2 + 16;                 // byte pitch of a row: ldmatrix reads eight rows without bank conflicts
+  static constexpr int TILE = LD_KEYS * RP;
+  static constexpr int SP = LD_KEYS + 4;                 // floats of a score row
+  static constexpr int PP = LD_KEYS * 2 + 16;            // bytes of a weight row
+  static constexpr int S_BYTES = 4 * MT * 16 * SP * 4, P_BYTES = MT * 16 * PP, A_BYTES = MT * 16 * 8;
+  static constexpr int REST = S_BYTES + P_BYTES + A_BYTES + 64;
+  static constexpr int FIT = (226 * 1024 - REST) / TILE;
+  static constexpr int ST = FIT > 4 ? 4 : FIT;
+  static constexpr int S_OFF = ST * TILE, P_OFF = S_OFF + S_BYTES, A_OFF = P_OFF + P_BYTES, BAR_OFF = A_OFF + A_BYTES;
+  static constexpr int TOTAL = BAR_OFF + 64;
+  static_assert(ST >= 2, "two stages at least");
+};
+
+template <int RC, int MT>
+__global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const LatentDecodeArgs p) {
+  using L = LatentSmem<RC, MT>;
+  constexpr int ST = L::ST, RP = L::RP, KS = RC / 64, NT = RC / 64;   // k steps of a warp's column quarter; 8-column blocks of its eighth
+  extern __shared__ __align__(128) uint8_t sm[];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int b = blockIdx.x, h0 = blockIdx.y * MT * 16, sp = blockIdx.z;
+  const int kg = warp & 1, rg = warp >> 1;
+  const uint32_t s0 = smem_u32(sm), bars = s0 + L::BAR_OFF;
+  float* sS = reinterpret_cast<float*>(sm + L::S_OFF);
+  float* sAl = reinterpret_cast<float*>(sm + L::A_OFF);                // rescale of a row; at the end: its maximum, then its sum
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + L::BAR_OFF + 48);
+  if (tid == 0) {
+    for (int s = 0; s < ST; ++s) mbar_init(bars + s * 8, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  tfb::pdl_sync();
+  const int n_keys = p.positions[b] + 1;
+  const int per = ((n_keys + p.splits - 1) / p.splits + LD_KEYS - 1) / LD_KEYS * LD_KEYS;
+  const int t_begin = sp * per, t_end = min(n_keys, t_begin + per);
+  const int nt = t_end > t_begin ? (t_end - t_begin + LD_KEYS - 1) / LD_KEYS : 0;
+  const int* bt = p.block_table + (long long)b * p.max_pages;
+  // what no copy writes but the products read: columns past W, and the missing rows of a last tile that is a stage's first
+  if (p.W < RC) {
+    const int pieces = (RC - p.W) / 8;
+    for (int i = tid; i < ST * LD_KEYS * pieces; i += LD_THREADS)
+      *reinterpret_cast<uint4*>(sm + (i / pieces) * RP + p.W * 2 + (i % pieces) * 16) = make_uint4(0u, 0u, 0u, 0u);
+  }
+  if (nt > 0 && nt <= ST) {
+    const int first = t_end - t_begin - (nt - 1) * LD_KEYS;           // rows of the last tile
+    uint8_t* base = sm + (nt - 1) * L::TILE + first * RP;
+    for (int i = tid; i < (LD_KEYS - first) * (RP / 16); i += LD_THREADS) reinterpret_cast<uint4*>(base)[i] = make_uint4(0u, 0u, 0u, 0u);
+  }
+  fence_proxy_async_smem();
+  __syncthreads();
+
+  // lanes 0-7 of warp w bring rows 8 w .. 8 w + 7 of a tile
+  const int my_row = warp * 8 + lane;
+  auto page_of = [&](int j) -> long long {
+    const int t = t_begin + j * LD_KEYS + my_row;
+    long long page = (lane < 8 && j < nt && t < t_end) ? bt[t / p.page] : 0;
+    TFB_BOUNDS(page >= 0 && (page + 1) * p.page <= p.nslots, 52, page, p.nslots / p.page);
+    if (page < 0 || (page + 1) * p.page > p.nslots) page = 0;
+    return page;
+  };
+  auto issue = [&](int j, long long page) {
+    const int t0 = t_begin + j * LD_KEYS, rows = min(LD_KEYS, t_end - t0), st = j % ST;
+    if (tid == 0) mbar_expect_tx(bars + st * 8, uint32_t(rows) * p.W * 2);
+    if (lane < 8 && my_row < rows)
+      bulk_load(s0 + st * L::TILE + my_row * RP, p.pool + (page * p.page + (t0 + my_row) % p.page) * p.W, p.W * 2, bars + st * 8);
+  };
+  for (int j = 0; j < ST - 1 && j < nt; ++j) issue(j, page_of(j));
+  long long page_next = page_of(ST - 1);
+
+  uint32_t qa[MT][KS][4];                                              // this warp's columns of the queries
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int k = 0; k < KS; ++k)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int h = h0 + m * 16 + (lane >> 2) + (e & 1) * 8, c = rg * (RC / 4) + k * 16 + (lane & 3) * 2 + (e >> 1) * 8;
+        qa[m][k][e] = (h < p.H && c < p.W) ? *reinterpret_cast<const uint32_t*>(p.q + b * p.ldq + (long long)h * p.W + c) : 0u;
+      }
+  float o[MT][NT][4];
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < NT; ++n) o[m][n][0] = o[m][n][1] = o[m][n][2] = o[m][n][3] = 0.f;
+  float m_run[2 * MT], l_run[2 * MT];                                  // rows 2 MT warp + i; the sum: this lane's part
+#pragma unroll
+  for (int i = 0; i < 2 * MT; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+  const float sl2 = p.scale * LOG2E;
+  bool ok = true;
+
+  for (int j = 0; j < nt; ++j) {
+    const uint32_t tile = s0 + (j % ST) * L::TILE;
+    if (ok && !mbar_wait_warp(bars + (j % ST) * 8, (j / ST) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) ok = false;
+    // scores of 32 keys over a quarter of the columns
+    float sc[MT][4][4];
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < 4; ++n) sc[m][n][0] = sc[m][n][1] = sc[m][n][2] = sc[m][n][3] = 0.f;
+    const uint32_t krow = tile + (kg * 32 + (lane & 7) + (lane >> 4) * 8) * RP + rg * (RC / 2) + ((lane >> 3) & 1) * 16;
+#pragma unroll
+    for (int k = 0; k < KS; ++k) {
+      uint32_t f0[4], f1[4];
+      ldsm(krow + k * 32, f0);
+      ldsm(krow + 16 * RP + k * 32, f1);
+#pragma unroll
+      for (int m = 0; m < MT; ++m) {
+        mma_bf16(sc[m][0], qa[m][k], f0[0], f0[1]);
+        mma_bf16(sc[m][1], qa[m][k], f0[2], f0[3]);
+        mma_bf16(sc[m][2], qa[m][k], f1[0], f1[1]);
+        mma_bf16(sc[m][3], qa[m][k], f1[2], f1[3]);
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < 4; ++n)
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+          *reinterpret_cast<float2*>(sS + (rg * MT * 16 + m * 16 + (lane >> 2) + 8 * i) * L::SP + kg * 32 + n * 8 + (lane & 3) * 2) =
+              make_float2(sc[m][n][2 * i], sc[m][n][2 * i + 1]);
+    __syncthreads();
+    // every warp is past tile j - 1: its stage takes tile j - 1 + ST
+    if (ok && j - 1 + ST < nt) {
+      fence_proxy_async_smem();
+      issue(j - 1 + ST, page_next);
+    }
+    page_next = page_of(j + ST);
+    const int n_valid = t_end - (t_begin + j * LD_KEYS);
+#pragma unroll
+    for (int i = 0; i < 2 * MT; ++i) {
+      const int row = warp * 2 * MT + i;
+      float2 s = *reinterpret_cast<const float2*>(sS + row * L::SP + 2 * lane);
+#pragma unroll
+      for (int g = 1; g < 4; ++g) {
+        const float2 u = *reinterpret_cast<const float2*>(sS + (g * MT * 16 + row) * L::SP + 2 * lane);
+        s.x += u.x;
+        s.y += u.y;
+      }
+      s.x = 2 * lane < n_valid ? s.x * sl2 : -INFINITY;
+      s.y = 2 * lane + 1 < n_valid ? s.y * sl2 : -INFINITY;
+      const float mx = fmaxf(m_run[i], warp_max(fmaxf(s.x, s.y)));
+      const float mb = mx == -INFINITY ? 0.f : mx;
+      const float alpha = m_run[i] == -INFINITY ? 0.f : exp2f(m_run[i] - mb);
+      const float p0 = exp2f(s.x - mb), p1 = exp2f(s.y - mb);
+      m_run[i] = mx;
+      l_run[i] = fmaf(l_run[i], alpha, p0 + p1);
+      *reinterpret_cast<uint32_t*>(sm + L::P_OFF + row * L::PP + lane * 4) = pack_bf16(p0, p1);
+      if (lane == 0) sAl[row] = alpha;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const float a0 = sAl[m * 16 + (lane >> 2)], a1 = sAl[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        o[m][n][0] *= a0;
+        o[m][n][1] *= a0;
+        o[m][n][2] *= a1;
+        o[m][n][3] *= a1;
+      }
+    }
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      uint32_t pa[MT][2][4];
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+          ldsm(s0 + L::P_OFF + (m * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * L::PP + half * 64 + k * 32 + (lane >> 4) * 16, pa[m][k]);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        uint32_t f[4];
+        ldsm_t(tile + (half * 32 + lane) * RP + (warp * (RC / 8) + n * 8) * 2, f);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_bf16(o[m][n], pa[m][0], f[0], f[1]);
+          mma_bf16(o[m][n], pa[m][1], f[2], f[3]);
+        }
+      }
+    }
+  }
+  if (!ok) {   // give copies already issued a bounded time to land before shared memory goes away
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) {}
+  }
+#pragma unroll
+  for (int i = 0; i < 2 * MT; ++i) l_run[i] = warp_add(l_run[i]);
+  __syncthreads();
+  if (lane == 0) {
+#pragma unroll
+    for (int i = 0; i < 2 * MT; ++i) {
+      sAl[warp * 2 * MT + i] = m_run[i];
+      sAl[MT * 16 + warp * 2 * MT + i] = l_run[i];
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int row = m * 16 + (lane >> 2) + 8 * i, h = h0 + row;
+      if (h >= p.H) continue;
+      if (p.splits == 1) {
+        const float inv = 1.f / sAl[MT * 16 + row];
+        __nv_bfloat16* dst = p.o + b * p.ldo + (long long)h * p.W;
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          const int c = warp * (RC / 8) + n * 8 + (lane & 3) * 2;
+          if (c < p.W) *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16(o[m][n][2 * i] * inv, o[m][n][2 * i + 1] * inv);
+        }
+      } else {
+        const long long at = ((long long)b * p.H + h) * p.splits + sp;
+        if (nt > 0) {
+#pragma unroll
+          for (int n = 0; n < NT; ++n) {
+            const int c = warp * (RC / 8) + n * 8 + (lane & 3) * 2;
+            if (c < p.W) *reinterpret_cast<float2*>(p.acc + at * p.W + c) = make_float2(o[m][n][2 * i], o[m][n][2 * i + 1]);
+          }
+        }
+        if (warp == 0 && (lane & 3) == 0) {
+          p.ml[at * 2] = sAl[row];
+          p.ml[at * 2 + 1] = sAl[MT * 16 + row];
+        }
+      }
+    }
+}
+
+// one block per (sequence, head): merge the splits
+__global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ acc, const float* __restrict__ ml, __nv_bfloat16* __restrict__ o,
+                                                             long long ldo, int H, int W, int splits) {
+  tfb::pdl_sync();
+  __shared__ float f[128];
+  const int b = blockIdx.x / H, h = blockIdx.x % H;
+  const long long base = (long long)blockIdx.x * splits;
+  if (threadIdx.x < 32) {                   // splits <= 128
+    float m = -INFINITY;
+    for (int s = threadIdx.x; s < splits; s += 32) m = fmaxf(m, ml[(base + s) * 2]);
+    m = warp_max(m);
+    float l = 0.f;
+    for (int s = threadIdx.x; s < splits; s += 32) {
+      const float ms = ml[(base + s) * 2], e = ms == -INFINITY ? 0.f : exp2f(ms - m);
+      f[s] = e;
+      l = fmaf(ml[(base + s) * 2 + 1], e, l);
+    }
+    l = warp_add(l);
+    for (int s = threadIdx.x; s < splits; s += 32) f[s] /= l;
+  }
+  __syncthreads();
+  for (int c = threadIdx.x * 4; c < W; c += 512) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int s = 0; s < splits; ++s) {
+      if (f[s] == 0.f) continue;
+      const float4 u = *reinterpret_cast<const float4*>(acc + (base + s) * W + c);
+      v.x = fmaf(u.x, f[s], v.x);
+      v.y = fmaf(u.y, f[s], v.y);
+      v.z = fmaf(u.z, f[s], v.z);
+      v.w = fmaf(u.w, f[s], v.w);
+    }
+    uint2 r;
+    r.x = pack_bf16(v.x, v.y);
+    r.y = pack_bf16(v.z, v.w);
+    *reinterpret_cast<uint2*>(o + b * ldo + (long long)h * W + c) = r;
+  }
+}
+
+template <int RC, int MT>
+static int launch_latent_decode(const LatentDecodeArgs& p, int B, cudaStream_t st) {
+  using L = LatentSmem<RC, MT>;
+  static DeviceOnce once;
+  auto kern = latent_decode_kernel<RC, MT>;
+  if (int e = ensure_dyn_smem(once, kern, L::TOTAL)) return e;
+  launch_k(kern, dim3(B, (p.H + MT * 16 - 1) / (MT * 16), p.splits), LD_THREADS, L::TOTAL, st, p);
+  return int(cudaGetLastError());
+}
+
+// ------------------------------------------------------------------------------------------------
+// any sizes, fp32 arithmetic
+// ------------------------------------------------------------------------------------------------
+template <class T>
+struct AttnAnyArgs {
+  const T* q;               // [B*S, ldq], H heads of D entries
+  long long ldq;
+  const T *k, *v;           // prompts: [B*Skv, ldk], [B*Skv, ldv], G heads; decoding: k = the pool [slots][ldk], keys and values of every head
+  long long ldk, ldv, nslots;
+  const int* block_table;   // decoding only
+  int max_pages, page;
+  const int* positions;     // decoding: position of the one query of each sequence
+  const T* gate;            // [B*S, ldg] or null
+  long long ldg;
+  T* o;
+  long long ldo;
+  int B, S, Skv, q_off, H, G, D, V, QR;
+  float scale;
+};
+
+constexpr int AN_K = 32;    // keys per tile
+
+// QR (4, 8 or 16) query rows per block: positions of one head (prompts) or heads of one sequence (decoding)
+template <class T, bool PAGED>
+__global__ void __launch_bounds__(128) attn_any_kernel(const AttnAnyArgs<T> p) {
+  tfb::pdl_sync();
+  extern __shared__ float am[];
+  const int D = p.D, V = p.V, QR = p.QR, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, DP = D + 1;
+  float* sQ = am;                       // [QR][D]
+  float* sK = sQ + QR * D;              // [AN_K][D + 1]
+  float* sV = sK + AN_K * DP;           // [AN_K][V]; decoding: the keys
+  float* sP = PAGED ? sV : sV + AN_K * V;   // [QR][AN_K]
+  float* sO = sP + QR * AN_K;           // [QR][V]
+  float* sA = sO + QR * V;              // [QR] rescale of this tile, then row sums
+  const int VP = PAGED ? DP : V;
+  if (PAGED) sV = sK;
+  int b, h0, i0, n, hi_max;
+  if (PAGED) {
+    b = blockIdx.y;
+    h0 = blockIdx.x * QR;
+    n = min(QR, p.H - h0);
+    i0 = 0;
+    hi_max = p.positions[b];
+  } else {
+    b = blockIdx.z;
+    h0 = blockIdx.y;
+    i0 = blockIdx.x * QR;
+    n = min(QR, p.S - i0);
+    hi_max = min(i0 + n - 1 + p.q_off, p.Skv - 1);
+  }
+  const int g = PAGED ? 0 : h0 / (p.H / p.G);
+  const int q_head = PAGED ? int(p.ldk) : D;      // entries between the heads of q and o
+  const int o_head = PAGED ? int(p.ldk) : V;
+  for (int i = tid; i < QR * D; i += 128) {
+    const int r = i / D, d = i % D;
+    const long long row = PAGED ? b : (long long)b * p.S + i0 + r;
+    sQ[i] = r < n ? to_f(p.q[row * p.ldq + (long long)(PAGED ? h0 + r : h0) * q_head + d]) : 0.f;
+  }
+  for (int i = tid; i < QR * V; i += 128) sO[i] = 0.f;
+  float m_run[4], l_run[4];             // this warp's rows: warp, warp + 4, ...
+#pragma unroll
+  for (int i = 0; i < 4; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
+  for (int t0 = 0; t0 <= hi_max; t0 += AN_K) {
+    const int nk = min(AN_K, hi_max + 1 - t0);
+    __syncthreads();
+    for (int j = warp; j < AN_K; j += 4) {
+      long long row = (long long)b * p.Skv + t0 + j;
+      if (PAGED && j < nk) {
+        long long page = p.block_table[(long long)b * p.max_pages + (t0 + j) / p.page];
+        TFB_BOUNDS(page >= 0 && (page + 1) * p.page <= p.nslots, 52, page, p.nslots / p.page);
+        if (page < 0 || (page + 1) * p.page > p.nslots) page = 0;
+        row = page * p.page + (t0 + j) % p.page;
+      }
+      for (int d = lane; d < D; d += 32) sK[j * DP + d] = j < nk ? to_f(p.k[row * p.ldk + (long long)g * D + d]) : 0.f;
+      if (!PAGED)
+        for (int d = lane; d < V; d += 32) sV[j * VP + d] = j < nk ? to_f(p.v[row * p.ldv + (long long)g * V + d]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = warp + 4 * i;
+      if (r >= QR) continue;
+      const float* q = sQ + r * D;
+      const float* k = sK + lane * DP;
+      float s = 0.f;
+      for (int d = 0; d < D; ++d) s = fmaf(q[d], k[d], s);
+      const int hi = PAGED ? hi_max : i0 + r + p.q_off;
+      s = (r < n && lane < nk && t0 + lane <= hi) ? s * p.scale : -INFINITY;
+      const float mx = fmaxf(m_run[i], warp_max(s));
+      const float mb = mx == -INFINITY ? 0.f : mx;
+      const float a = m_run[i] == -INFINITY ? 0.f : expf(m_run[i] - mb);
+      const float e = expf(s - mb);
+      l_run[i] = fmaf(l_run[i], a, warp_add(e));
+      m_run[i] = mx;
+      sP[r * AN_K + lane] = e;
+      if (lane == 0) sA[r] = a;
+    }
+    __syncthreads();
+    for (int i = tid; i < QR * V; i += 128) {
+      const int r = i / V, d = i % V;
+      float acc = sO[i] * sA[r];
+#pragma unroll 8
+      for (int j = 0; j < AN_K; ++j) acc = fmaf(sP[r * AN_K + j], sV[j * VP + d], acc);
+      sO[i] = acc;
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (lane == 0 && warp + 4 * i < QR) sA[warp + 4 * i] = l_run[i];
+  __syncthreads();
+  for (int r = warp; r < n; r += 4) {
+    const long long row = PAGED ? b : (long long)b * p.S + i0 + r;
+    const int h = PAGED ? h0 + r : h0;
+    float f = 1.f / sA[r];
+    if (p.gate) f *= sigmoid_exact(to_f(p.gate[row * p.ldg + h]));
+    for (int d = lane; d < o_head; d += 32) p.o[row * p.ldo + (long long)h * o_head + d] = from_f<T>(d < V ? sO[r * V + d] * f : 0.f);
+  }
+}
+
+template <class T, bool PAGED>
+static int launch_any(AttnAnyArgs<T> p, cudaStream_t st) {
+  long long smem = 0;
+  for (p.QR = 16; p.QR >= 4; p.QR >>= 1) {
+    smem = 4ll * (p.QR * p.D + AN_K * (p.D + 1) + (PAGED ? 0 : AN_K * p.V) + p.QR * AN_K + p.QR * p.V + p.QR);
+    if (smem <= 220 * 1024) break;
+  }
+  if (p.QR < 4) return TFB_ERR_LIMIT;
+  static DeviceOnce once;
+  auto kern = attn_any_kernel<T, PAGED>;
+  if (int e = ensure_dyn_smem(once, kern, 220 * 1024)) return e;
+  const dim3 grid = PAGED ? dim3((p.H + p.QR - 1) / p.QR, p.B) : dim3((p.S + p.QR - 1) / p.QR, p.H, p.B);
+  launch_k(kern, grid, 128, size_t(smem), st, p);
+  return int(cudaGetLastError());
+}
+
+static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+}  // namespace tfb
+
+using bf16 = __nv_bfloat16;
+
+// rows c [rows, ldc] of R entries -> out (may be null) and the pool [nslots][width] at slots (null: none; negative: not this row)
+TFB_API int tfb_latent_append(const void* c, long long ldc, const void* w, float eps, const long long* slots, void* out, long long ldo, void* pool,
+                              long long nslots, int width, int rows, int R, int f32, void* stream) {
+  using namespace tfb;
+  if (rows <= 0 || R <= 0 || width < R) return TFB_ERR_ARG;
+  if (!slots || nslots == 0) slots = nullptr;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int vec = f32 ? 4 : 8, grid = (rows + 7) / 8;
+  const bool v = R % vec == 0 && ldc % vec == 0 && ldo % vec == 0 && width % vec == 0 && al16(c) && al16(w) && al16(out) && al16(pool);
+#define TFB_LA(T, VEC) launch_k(latent_append_kernel<T, VEC>, grid, 256, 0, st, static_cast<const T*>(c), ldc, static_cast<const T*>(w), eps, slots, \
+                                static_cast<T*>(out), ldo, static_cast<T*>(pool), nslots, width, rows, R)
+  if (f32) { if (v) TFB_LA(float, 4); else TFB_LA(float, 1); }
+  else { if (v) TFB_LA(bf16, 8); else TFB_LA(bf16, 1); }
+#undef TFB_LA
+  return int(cudaGetLastError());
+}
+
+// q [B*S, ldq]: H heads of D entries; k, v [B*Skv, ldk / ldv]: G heads of D / V entries; gate [B*S, ldg]: one logit per head, or null.
+// The queries are the last S of the Skv positions.  o [B*S, ldo]: H heads of V entries.
+TFB_API int tfb_head_attn(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, void* o, long long ldo,
+                          const void* gate, long long ldg, int B, int S, int Skv, int H, int G, int D, int V, float scale, int f32, int* status,
+                          void* stream) {
+  using namespace tfb;
+  if (B <= 0 || B > 65535 || S <= 0 || Skv < S || G <= 0 || H % G || H > 65535 || D <= 0 || V <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool tc = !f32 && D % 8 == 0 && V % 8 == 0 && D <= 128 && V <= 128 && ldq % 8 == 0 && ldk % 8 == 0 && ldv % 8 == 0 && ldo % 8 == 0 &&
+                  al16(q) && al16(k) && al16(v) && al16(o);
+  if (tc) {
+    HeadAttnParams p{B, S, H, G, Skv, Skv - S, V, scale, static_cast<const bf16*>(gate), ldg, static_cast<bf16*>(o), ldo, status};
+    if (D <= 64) return V <= 64 ? launch_head_attn<64, 64>(q, ldq, k, ldk, v, ldv, D, p, st) : launch_head_attn<64, 128>(q, ldq, k, ldk, v, ldv, D, p, st);
+    return V <= 64 ? launch_head_attn<128, 64>(q, ldq, k, ldk, v, ldv, D, p, st) : launch_head_attn<128, 128>(q, ldq, k, ldk, v, ldv, D, p, st);
+  }
+#define TFB_ANY(T)                                                                                                                           \
+  launch_any<T, false>(AttnAnyArgs<T>{static_cast<const T*>(q), ldq, static_cast<const T*>(k), static_cast<const T*>(v), ldk, ldv, 0, nullptr, 0, 1, \
+                                      nullptr, static_cast<const T*>(gate), ldg, static_cast<T*>(o), ldo, B, S, Skv, Skv - S, H, G, D, V, 16, scale}, st)
+  return f32 ? TFB_ANY(float) : TFB_ANY(bf16);
+#undef TFB_ANY
+}
+
+TFB_API int tfb_gemm_f32_heads(const float* A, long long lda, int a_head, const float* B, long long ldb, int b_kn, float* C, long long ldc, int c_head,
+                               const float* gate, long long ldg, int M, int heads, int N, int K, void* stream);
+
+// One product per head: x [M, ldx] (x_head entries between heads, K of them used), w: heads blocks [N, K] ([K, N] with kn) stacked on the
+// rows, out [M, ldo] (out_head >= N entries between heads; those past N become zero), gate [M, ldg] or null.
+TFB_API int tfb_head_linear(const void* x, long long ldx, const void* w, long long ldw, int kn, void* out, long long ldo, int out_head, const void* gate,
+                            long long ldg, int M, int heads, int K, int N, int x_head, int f32, void* stream) {
+  using namespace tfb;
+  if (M <= 0 || heads <= 0 || heads > 65535 || K <= 0 || N <= 0 || x_head < K || out_head < N) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) {
+    if (out_head > N)
+      if (cudaError_t e = cudaMemset2DAsync(out, size_t(ldo) * 4, 0, size_t(heads) * out_head * 4, M, st)) return int(e);
+    return tfb_gemm_f32_heads(static_cast<const float*>(x), ldx, x_head, static_cast<const float*>(w), ldw, kn, static_cast<float*>(out), ldo, out_head,
+                              static_cast<const float*>(gate), ldg, M, heads, N, K, stream);
+  }
+  HeadLinearArgs p{static_cast<const bf16*>(x), static_cast<const bf16*>(w), ldx, ldw, static_cast<bf16*>(out), ldo, static_cast<const bf16*>(gate), ldg,
+                   M, N, K, x_head, out_head, x_head % 8 == 0 && ldx % 8 == 0 && al16(x), ldw % 8 == 0 && al16(w)};
+  const dim3 grid((out_head + HL_N - 1) / HL_N, heads, (M + HL_M - 1) / HL_M);
+  if (kn) launch_k(head_linear_kernel<true>, grid, 128, 0, st, p);
+  else launch_k(head_linear_kernel<false>, grid, 128, 0, st, p);
+  return int(cudaGetLastError());
+}
+
+// Key splits of the tensor-core form of tfb_latent_decode for these sizes (it then needs acc / ml for more than one); 0: the other form.
+// A wide latent's CTA fills an SM, and all of a step's CTAs should run at once: a second wave of a few would double the time.
+TFB_API int tfb_latent_decode_plan(int B, int H, int W, int max_keys, int f32) {
+  if (f32 || W > 512 || W % 8) return 0;
+  const long long items = (long long)B * ((H + 31) / 32), slots = 148ll * (W > 256 ? 1 : 2);
+  long long s = slots / (items > 0 ? items : 1);
+  const long long most = (max_keys + 2 * tfb::LD_KEYS - 1) / (2 * tfb::LD_KEYS);     // two tiles each at least
+  if (s > most) s = most;
+  return int(s < 1 ? 1 : (s > 64 ? 64 : s));
+}
+
+// One query per sequence at positions[b] over the cached rows of the pool [slots][W] (latents of R entries, zeros behind them); q and o
+// [B, ldq / ldo]: H heads of W entries.
+TFB_API int tfb_latent_decode(const void* q, long long ldq, const void* pool, long long nslots, const int* block_table, int max_pages, int page,
+                              const int* positions, void* o, long long ldo, float* acc, float* ml, int splits, int B, int H, int R, int W,
+                              float scale, int f32, int* status, void* stream) {
+  using namespace tfb;
+  if (B <= 0 || B > 65535 || H <= 0 || R <= 0 || W < R || page <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (splits > 0 && tfb_latent_decode_plan(B, H, W, 1, f32) > 0) {
+    if (splits > 128 || (splits > 1 && (!acc || !ml)) || ldq % 8 || ldo % 8 || !al16(q) || !al16(pool) || !al16(o)) return TFB_ERR_ARG;
+    LatentDecodeArgs p{static_cast<const bf16*>(q), ldq, static_cast<const bf16*>(pool), nslots, block_table, max_pages, page, positions, H, W,
+                       splits, scale, static_cast<bf16*>(o), ldo, acc, ml, status};
+    int rc;
+#define TFB_LD(RC) (H <= 16 ? launch_latent_decode<RC, 1>(p, B, st) : launch_latent_decode<RC, 2>(p, B, st))
+    if (W <= 64) rc = TFB_LD(64);
+    else if (W <= 128) rc = TFB_LD(128);
+    else if (W <= 256) rc = TFB_LD(256);
+    else rc = TFB_LD(512);
+#undef TFB_LD
+    if (rc) return rc;
+    if (splits > 1) launch_k(latent_combine_kernel, B * H, 128, 0, st, acc, ml, static_cast<bf16*>(o), ldo, H, W, splits);
+    return int(cudaGetLastError());
+  }
+#define TFB_ANY(T)                                                                                                                             \
+  launch_any<T, true>(AttnAnyArgs<T>{static_cast<const T*>(q), ldq, static_cast<const T*>(pool), nullptr, W, 0, nslots, block_table, max_pages, page, \
+                                     positions, nullptr, 0, static_cast<T*>(o), ldo, B, 1, 0, 0, H, 1, R, R, 16, scale}, st)
+  return f32 ? TFB_ANY(float) : TFB_ANY(bf16);
+#undef TFB_ANY
+}

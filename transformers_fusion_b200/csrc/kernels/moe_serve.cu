@@ -1,0 +1,286 @@
+// Mixture-of-experts feed-forward for serving: any sizes and pitches, bf16 or fp32 rows, no statistics and nothing kept for a
+// backward pass (the training form is moe_routing.cu).
+//
+//   moe_route          per token: the k largest of logits + bias (fp32, the lower index first among equals) and the softmax over them;
+//                      then the rows of the expert buffers: every expert's assignments are consecutive rows from a multiple
+//                      of 128 on, so that a 128-row tile of the grouped product belongs to one expert.  Few tokens (decode
+//                      steps): one block does all of it; many: selection with per-block counts, a scan, row numbers.
+//   moe_gather         token rows to their assignments' rows
+//   moe_glu            silu(gate) * up of the assigned rows (a decode step's buffers are mostly padding)
+//   moe_weighted_sum   y[t] = base[t] + sum_k w[t, k] * rows[row_of[t, k]], summed in fp32
+#include <limits.h>
+
+#include "tfb_elem.cuh"
+#include "tfb_host.h"
+
+namespace tfb {
+TFB_BOUNDS_DEFINE(moe_serve)
+
+struct RouteArgs {
+  const float* logits;        // [T, ld]
+  long long ld;
+  const void* bias;           // [E], bf16 or fp32
+  int bias_f32, T, E, K;
+  int* idx;                   // [T, K]
+  float* w;                   // [T, K]
+  int *rank, *row_of;         // [T, K]
+  int* expert_of_tile;        // [tiles]
+  int *counts, *start;        // [E]
+  int tiles;
+};
+
+// Chooses the experts of token t (one warp): `K` rounds, each the largest entry that comes after the last one in the order
+// (value descending, index ascending).  Lane 0 writes; `count` (shared memory) numbers the assignments of each expert.
+__device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int lane, int* count) {
+  const float* z = p.logits + t * p.ld;
+  float last = INFINITY, first = 0.f, sum = 0.f;
+  int last_e = -1;
+  for (int k = 0; k < p.K; ++k) {
+    float best = -INFINITY;
+    int e_best = INT_MAX;
+    for (int e = lane; e < p.E; e += 32) {
+      const float v = z[e] + (p.bias_f32 ? static_cast<const float*>(p.bias)[e] : to_f(static_cast<const __nv_bfloat16*>(p.bias)[e]));
+      const bool after = v < last || (v == last && e > last_e);
+      if (after && (v > best || e_best == INT_MAX)) { best = v; e_best = e; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float v = __shfl_xor_sync(0xffffffffu, best, o);
+      const int e = __shfl_xor_sync(0xffffffffu, e_best, o);
+      if (e != INT_MAX && (e_best == INT_MAX || v > best || (v == best && e < e_best))) { best = v; e_best = e; }
+    }
+    if (e_best == INT_MAX) e_best = k;       // logits that compare with nothing
+    last = best;
+    last_e = e_best;
+    if (k == 0) first = best;
+    const float x = expf(best - first);
+    sum += x;
+    if (lane == 0) {
+      const long long i = (long long)t * p.K + k;
+      p.idx[i] = e_best;
+      p.w[i] = x;
+      p.rank[i] = atomicAdd(count + e_best, 1);
+    }
+  }
+  __syncwarp();
+  for (int k = lane; k < p.K; k += 32) p.w[(long long)t * p.K + k] /= sum;
+}
+
+// start[e] = first row of expert e, expert_of_tile; one block of 1024 threads; `count` may be shared or global memory
+__device__ __forceinline__ void plan_segments(const RouteArgs& p, const int* count) {
+  __shared__ int part[32], carry;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  if (threadIdx.x == 0) carry = 0;
+  __syncthreads();
+  for (int e0 = 0; e0 < p.E; e0 += 1024) {
+    const int e = e0 + threadIdx.x;
+    const int n = e < p.E ? (count[e] + 127) / 128 : 0;
+    int s = n;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int v = __shfl_up_sync(0xffffffffu, s, o);
+      if (lane >= o) s += v;
+    }
+    if (lane == 31) part[warp] = s;
+    __syncthreads();
+    if (warp == 0) {
+      int q = part[lane];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, q, o);
+        if (lane >= o) q += v;
+      }
+      part[lane] = q;
+    }
+    __syncthreads();
+    const int base = carry + (warp ? part[warp - 1] : 0) + s - n;
+    if (e < p.E) {
+      p.start[e] = base * 128;
+      for (int i = 0; i < n && base + i < p.tiles; ++i) p.expert_of_tile[base + i] = e;
+    }
+    __syncthreads();
+    if (threadIdx.x == 0) carry += part[31];
+    __syncthreads();
+  }
+  for (int i = carry + threadIdx.x; i < p.tiles; i += 1024) p.expert_of_tile[i] = -1;
+}
+
+__global__ void __launch_bounds__(1024) moe_route_small_kernel(const RouteArgs p) {
+  tfb::pdl_sync();
+  extern __shared__ int count[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  for (int e = threadIdx.x; e < p.E; e += 1024) count[e] = 0;
+  __syncthreads();
+  for (int t = warp; t < p.T; t += 32) choose_experts(p, t, lane, count);
+  __syncthreads();
+  plan_segments(p, count);
+  for (int e = threadIdx.x; e < p.E; e += 1024) p.counts[e] = count[e];
+  __syncthreads();
+  for (int i = threadIdx.x; i < p.T * p.K; i += 1024) p.row_of[i] = p.start[p.idx[i]] + p.rank[i];
+}
+
+constexpr int ROUTE_TOKENS = 64;      // tokens of a block
+__global__ void __launch_bounds__(256) moe_route_choose_kernel(const RouteArgs p) {
+  tfb::pdl_sync();
+  extern __shared__ int count[];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int t0 = blockIdx.x * ROUTE_TOKENS, t1 = min(p.T, t0 + ROUTE_TOKENS);
+  for (int e = threadIdx.x; e < p.E; e += 256) count[e] = 0;
+  __syncthreads();
+  for (int t = t0 + warp; t < t1; t += 8) choose_experts(p, t, lane, count);
+  __syncthreads();
+  for (int e = threadIdx.x; e < p.E; e += 256) count[e] = count[e] ? atomicAdd(p.counts + e, count[e]) : 0;
+  __syncthreads();
+  for (long long i = (long long)t0 * p.K + threadIdx.x; i < (long long)t1 * p.K; i += 256) p.rank[i] += count[p.idx[i]];
+}
+__global__ void __launch_bounds__(1024) moe_route_plan_kernel(const RouteArgs p) {
+  tfb::pdl_sync();
+  plan_segments(p, p.counts);
+}
+__global__ void __launch_bounds__(256) moe_route_rows_kernel(const RouteArgs p) {
+  tfb::pdl_sync();
+  const long long i = blockIdx.x * 256ll + threadIdx.x;
+  if (i < (long long)p.T * p.K) p.row_of[i] = p.start[p.idx[i]] + p.rank[i];
+}
+
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ x, long long ldx, const int* __restrict__ row_of, T* __restrict__ xp,
+                                                         long long ldp, long long assignments, int K, int H) {
+  tfb::pdl_sync();
+  const int per = H / VEC;
+  const long long n = assignments * per;
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
+    const long long a = i / per;
+    const int c = int(i - a * per) * VEC;
+    float v[VEC];
+    load_n<VEC>(x + a / K * ldx + c, v);
+    store_n<VEC>(xp + row_of[a] * ldp + c, v);
+  }
+}
+
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) moe_glu_kernel(const T* __restrict__ in, long long ldi, const int* __restrict__ row_of, T* __restrict__ out,
+                                                      long long ldo, long long assignments, int F) {
+  tfb::pdl_sync();
+  const int per = F / VEC;
+  const long long n = assignments * per;
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
+    const long long a = i / per, row = row_of[a];
+    const int c = int(i - a * per) * VEC;
+    float g[VEC], u[VEC];
+    load_n<VEC>(in + row * ldi + c, g);
+    load_n<VEC>(in + row * ldi + F + c, u);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) g[e] = silu_exact(g[e]) * u[e];
+    store_n<VEC>(out + row * ldo + c, g);
+  }
+}
+
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) moe_weighted_sum_kernel(const T* __restrict__ yp, long long ldp, const int* __restrict__ row_of,
+                                                               const float* __restrict__ w, const T* __restrict__ base, long long ldb,
+                                                               T* __restrict__ y, long long ldy, int Tn, int K, int H) {
+  tfb::pdl_sync();
+  const int per = H / VEC;
+  const long long n = (long long)Tn * per;
+  for (long long i = blockIdx.x * 256ll + threadIdx.x; i < n; i += gridDim.x * 256ll) {
+    const long long t = i / per;
+    const int c = int(i - t * per) * VEC;
+    float acc[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) acc[e] = 0.f;
+    for (int k = 0; k < K; ++k) {
+      float v[VEC];
+      load_n<VEC>(yp + row_of[t * K + k] * ldp + c, v);
+      const float f = w[t * K + k];
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[e] = fmaf(f, v[e], acc[e]);
+    }
+    if (base) {
+      float v[VEC];
+      load_n<VEC>(base + t * ldb + c, v);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) acc[e] += v[e];
+    }
+    store_n<VEC>(y + t * ldy + c, acc);
+  }
+}
+
+static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+static int blocks_for(long long items) {
+  const long long b = (items + 255) / 256, cap = 148ll * 16;
+  return int(b < 1 ? 1 : (b < cap ? b : cap));
+}
+
+}  // namespace tfb
+
+using bf16 = __nv_bfloat16;
+
+// logits [T, ld] fp32, bias [E] (bias_f32: fp32, otherwise bf16).  idx, row_of, rank (scratch): int [T, K]; w: fp32 [T, K]; counts, start
+// (scratch): int [E]; expert_of_tile: int [tiles], tiles >= T K / 128 + min(E, T K).
+TFB_API int tfb_moe_route(const float* logits, const void* bias, int T, int E, int K, int* idx, float* w, int* row_of, int* expert_of_tile,
+                          int* counts, int* rank, int* start, int tiles, long long ld, int bias_f32, void* stream) {
+  using namespace tfb;
+  if (T <= 0 || E <= 0 || K <= 0 || K > E || !bias) return TFB_ERR_ARG;
+  const long long a = (long long)T * K;
+  if (tiles < a / 128 + (E < a ? E : a)) return TFB_ERR_ARG;
+  if (E > 8192) return TFB_ERR_LIMIT;
+  RouteArgs p{logits, ld, bias, bias_f32, T, E, K, idx, w, rank, row_of, expert_of_tile, counts, start, tiles};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const size_t smem = size_t(E) * 4;
+  if (T <= 256) {
+    launch_k(moe_route_small_kernel, 1, 1024, smem, st, p);
+    return int(cudaGetLastError());
+  }
+  if (cudaError_t e = cudaMemsetAsync(counts, 0, smem, st)) return int(e);
+  launch_k(moe_route_choose_kernel, (T + ROUTE_TOKENS - 1) / ROUTE_TOKENS, 256, smem, st, p);
+  launch_k(moe_route_plan_kernel, 1, 1024, 0, st, p);
+  launch_k(moe_route_rows_kernel, int((a + 255) / 256), 256, 0, st, p);
+  return int(cudaGetLastError());
+}
+
+#define TFB_BY_TYPE(KERN, GRID, VECOK, ...)                                                                \
+  do {                                                                                                     \
+    if (f32) { if (VECOK) launch_k(KERN<float, 4>, GRID, 256, 0, st, __VA_ARGS__(float)); else launch_k(KERN<float, 1>, GRID, 256, 0, st, __VA_ARGS__(float)); } \
+    else { if (VECOK) launch_k(KERN<bf16, 8>, GRID, 256, 0, st, __VA_ARGS__(bf16)); else launch_k(KERN<bf16, 1>, GRID, 256, 0, st, __VA_ARGS__(bf16)); } \
+  } while (0)
+
+TFB_API int tfb_moe_gather(const void* x, long long ldx, const int* row_of, void* xp, long long ldp, int T, int K, int H, int f32, void* stream) {
+  using namespace tfb;
+  if (T <= 0 || K <= 0 || H <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int vec = f32 ? 4 : 8;
+  const bool v = H % vec == 0 && ldx % vec == 0 && ldp % vec == 0 && al16(x) && al16(xp);
+  const long long a = (long long)T * K;
+#define TFB_ARGS(T) static_cast<const T*>(x), ldx, row_of, static_cast<T*>(xp), ldp, a, K, H
+  TFB_BY_TYPE(moe_gather_kernel, blocks_for(a * (v ? H / vec : H)), v, TFB_ARGS);
+#undef TFB_ARGS
+  return int(cudaGetLastError());
+}
+
+// rows [gate | up] of 2 F entries -> silu(gate) * up, for the `assignments` rows that row_of names
+TFB_API int tfb_moe_glu(const void* in, long long ldi, const int* row_of, void* out, long long ldo, int assignments, int F, int f32, void* stream) {
+  using namespace tfb;
+  if (assignments <= 0 || F <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int vec = f32 ? 4 : 8;
+  const bool v = F % vec == 0 && ldi % vec == 0 && ldo % vec == 0 && al16(in) && al16(out);
+  const long long a = assignments;
+#define TFB_ARGS(T) static_cast<const T*>(in), ldi, row_of, static_cast<T*>(out), ldo, a, F
+  TFB_BY_TYPE(moe_glu_kernel, blocks_for(a * (v ? F / vec : F)), v, TFB_ARGS);
+#undef TFB_ARGS
+  return int(cudaGetLastError());
+}
+
+TFB_API int tfb_moe_weighted_sum(const void* yp, long long ldp, const int* row_of, const float* w, const void* base, long long ldb, void* y,
+                                 long long ldy, int T, int K, int H, int f32, void* stream) {
+  using namespace tfb;
+  if (T <= 0 || K <= 0 || H <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int vec = f32 ? 4 : 8;
+  const bool v = H % vec == 0 && ldp % vec == 0 && ldy % vec == 0 && al16(yp) && al16(y) && (!base || (ldb % vec == 0 && al16(base)));
+#define TFB_ARGS(Ty) static_cast<const Ty*>(yp), ldp, row_of, w, static_cast<const Ty*>(base), ldb, static_cast<Ty*>(y), ldy, T, K, H
+  TFB_BY_TYPE(moe_weighted_sum_kernel, blocks_for((long long)T * (v ? H / vec : H)), v, TFB_ARGS);
+#undef TFB_ARGS
+  return int(cudaGetLastError());
+}

@@ -1,6 +1,6 @@
-// Row operators of decoders with a 32-bit residual stream and a norm before and after every sublayer: scaled embedding,
-// post-norm + residual + next pre-norm in one pass, gated activation, partial rotary embedding fused with the append to
-// the paged cache, gather of cached rows, and a true fp32 matrix product.  Every kernel exists for bf16 and for fp32
+// Row operators of decoders with a 32-bit residual stream: scaled embedding, norm of a sublayer's output + residual + norm of (or
+// rounding for) the next sublayer's input in one pass, activations, partial rotary embedding fused with the append to the paged
+// cache, gather of cached rows, and a true fp32 matrix product (dense, one block per head, or rows grouped by expert).  Every kernel exists for bf16 and for fp32
 // activations; the statistics, the residual and the rotation are fp32 in both.
 #include "tfb_elem.cuh"
 #include "tfb_host.h"
@@ -9,7 +9,8 @@ namespace tfb {
 TFB_BOUNDS_DEFINE(stack_ops)
 
 // ------------------------------------------------------------------------------------------------
-// x <- x + norm(y) * (1 + w_post);  a = norm(x) * (1 + w_pre)      (norm: division by the root of the mean square)
+// x <- x + norm(y) [* scale_post];  a = norm(x), or x itself without w_pre
+// norm: LAYER false: v / rms(v) * (1 + w); LAYER true: (v - mean) / sqrt(mean squared deviation + eps) * w + b.
 // ids != null: x starts as scale * table[id] instead of being read.  rows != null: output row i is computed from row
 // rows[i] of x and y, and x is left alone (the last norm of a step, for the positions whose logits are wanted).
 // One block per row; the row lives in registers between the two statistics.
@@ -24,7 +25,7 @@ struct ResNormArgs {
   long long ldx;
   const void* y;
   long long ldy;
-  const void *w_post, *w_pre;
+  const void *w_post, *b_post, *scale_post, *w_pre, *b_pre;
   void* a;
   long long lda;
   const int* rows;
@@ -32,7 +33,50 @@ struct ResNormArgs {
   float eps;
 };
 
-template <class T, int VEC, int NV>
+// statistics of a row held in the block's registers: the mean to subtract (0 unless LAYER) and the factor
+template <bool LAYER, int VEC, int NV>
+__device__ __forceinline__ float2 row_stats(const float (&v)[NV][VEC], int H, float eps, float* red) {
+  const int nt = blockDim.x;
+  float mean = 0.f;
+  if constexpr (LAYER) {
+    float s = 0.f;
+#pragma unroll
+    for (int c = 0; c < NV; ++c)
+      if (int((c * nt + threadIdx.x) * VEC) < H) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) s += v[c][e];
+      }
+    mean = block_add(s, red) / H;
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < NV; ++c)
+    if (int((c * nt + threadIdx.x) * VEC) < H) {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        const float d = LAYER ? v[c][e] - mean : v[c][e];
+        ss = fmaf(d, d, ss);
+      }
+    }
+  return make_float2(mean, 1.f / sqrtf(block_add(ss, red) / H + eps));
+}
+
+template <class T, bool LAYER, int VEC>
+__device__ __forceinline__ void apply_norm(float (&v)[VEC], float2 st, const void* w, const void* b, int col) {
+  float wv[VEC];
+  load_n<VEC>(static_cast<const T*>(w) + col, wv);
+  if constexpr (LAYER) {
+    float bv[VEC];
+    load_n<VEC>(static_cast<const T*>(b) + col, bv);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = (v[e] - st.x) * st.y * wv[e] + bv[e];
+  } else {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) v[e] = v[e] * st.y * (1.f + wv[e]);
+  }
+}
+
+template <class T, bool LAYER, int VEC, int NV>
 __global__ void res_norm_kernel(const ResNormArgs p) {
   tfb::pdl_sync();
   __shared__ float red[32];
@@ -60,24 +104,25 @@ __global__ void res_norm_kernel(const ResNormArgs p) {
   }
   if (p.y) {
     float yv[NV][VEC];
-    float ss = 0.f;
 #pragma unroll
     for (int c = 0; c < NV; ++c) {
       const int col = (c * nt + threadIdx.x) * VEC;
-      if (col >= p.H) continue;
-      load_n<VEC>(static_cast<const T*>(p.y) + r * p.ldy + col, yv[c]);
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) ss = fmaf(yv[c][e], yv[c][e], ss);
+      if (col < p.H) load_n<VEC>(static_cast<const T*>(p.y) + r * p.ldy + col, yv[c]);
     }
-    const float rs = 1.f / sqrtf(block_add(ss, red) / p.H + p.eps);
+    const float2 st = row_stats<LAYER, VEC, NV>(yv, p.H, p.eps, red);
 #pragma unroll
     for (int c = 0; c < NV; ++c) {
       const int col = (c * nt + threadIdx.x) * VEC;
       if (col >= p.H) continue;
-      float w[VEC];
-      load_n<VEC>(static_cast<const T*>(p.w_post) + col, w);
+      apply_norm<T, LAYER, VEC>(yv[c], st, p.w_post, p.b_post, col);
+      if (p.scale_post) {
+        float s[VEC];
+        load_n<VEC>(static_cast<const T*>(p.scale_post) + col, s);
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) v[c][e] += yv[c][e] * rs * (1.f + w[e]);
+        for (int e = 0; e < VEC; ++e) yv[c][e] *= s[e];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[c][e] += yv[c][e];
     }
   }
   if (!p.rows && (p.y || p.ids)) {
@@ -88,40 +133,49 @@ __global__ void res_norm_kernel(const ResNormArgs p) {
     }
   }
   if (!p.a) return;
-  float ss = 0.f;
+  float2 st = make_float2(0.f, 1.f);
+  if (p.w_pre) st = row_stats<LAYER, VEC, NV>(v, p.H, p.eps, red);
 #pragma unroll
   for (int c = 0; c < NV; ++c) {
     const int col = (c * nt + threadIdx.x) * VEC;
     if (col >= p.H) continue;
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) ss = fmaf(v[c][e], v[c][e], ss);
-  }
-  const float rs = 1.f / sqrtf(block_add(ss, red) / p.H + p.eps);
-#pragma unroll
-  for (int c = 0; c < NV; ++c) {
-    const int col = (c * nt + threadIdx.x) * VEC;
-    if (col >= p.H) continue;
-    float w[VEC], o[VEC];
-    load_n<VEC>(static_cast<const T*>(p.w_pre) + col, w);
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) o[e] = v[c][e] * rs * (1.f + w[e]);
-    store_n<VEC>(static_cast<T*>(p.a) + (long long)i * p.lda + col, o);
+    if (p.w_pre) apply_norm<T, LAYER, VEC>(v[c], st, p.w_pre, p.b_pre, col);
+    store_n<VEC>(static_cast<T*>(p.a) + (long long)i * p.lda + col, v[c]);
   }
 }
 
-template <class T, int VEC>
+template <class T, bool LAYER, int VEC>
 static int launch_res_norm(const ResNormArgs& p, int n, cudaStream_t st) {
   const int items = (p.H + VEC - 1) / VEC;
   int nt = (items + 31) / 32 * 32;
   const int cap = VEC == 1 ? 512 : 256;
   if (nt > cap) nt = cap;
   const int nv = (items + nt - 1) / nt;
-  if (nv <= 1) launch_k(res_norm_kernel<T, VEC, 1>, n, nt, 0, st, p);
-  else if (nv <= 2) launch_k(res_norm_kernel<T, VEC, 2>, n, nt, 0, st, p);
-  else if (nv <= 4) launch_k(res_norm_kernel<T, VEC, 4>, n, nt, 0, st, p);
-  else if (nv <= 8) launch_k(res_norm_kernel<T, VEC, 8>, n, nt, 0, st, p);
+  if (nv <= 1) launch_k(res_norm_kernel<T, LAYER, VEC, 1>, n, nt, 0, st, p);
+  else if (nv <= 2) launch_k(res_norm_kernel<T, LAYER, VEC, 2>, n, nt, 0, st, p);
+  else if (nv <= 4) launch_k(res_norm_kernel<T, LAYER, VEC, 4>, n, nt, 0, st, p);
+  else if (nv <= 8) launch_k(res_norm_kernel<T, LAYER, VEC, 8>, n, nt, 0, st, p);
   else return TFB_ERR_LIMIT;
   return int(cudaGetLastError());
+}
+
+// ------------------------------------------------------------------------------------------------
+// act of every entry (codes of the product epilogue: 4 = squared relu)
+// ------------------------------------------------------------------------------------------------
+__device__ __forceinline__ float act_f32(float v, int act) {
+  if (act == 4) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  return v;
+}
+
+template <class T>
+__global__ void __launch_bounds__(256) act_rows_kernel(const T* __restrict__ in, long long ldi, T* __restrict__ out, long long ldo, int M, int N, int act) {
+  tfb::pdl_sync();
+  const long long n = (long long)M * N;
+  for (long long t = blockIdx.x * (long long)blockDim.x + threadIdx.x; t < n; t += (long long)gridDim.x * blockDim.x)
+    out[t / N * ldo + t % N] = from_f<T>(act_f32(to_f(in[t / N * ldi + t % N]), act));
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -225,25 +279,53 @@ __global__ void __launch_bounds__(256) gather_rows_kernel(const T* __restrict__ 
 }
 
 // ------------------------------------------------------------------------------------------------
-// C[M, N] = A[M, K] . B[N, K]^T in true fp32 (FFMA), 64 x 64 tiles, any sizes and pitches
+// C[M, N] = act(A[M, K] . B^T) in true fp32 (FFMA), 64 x 64 tiles, any sizes and pitches.
+// B is [N, K], or [K, N] with b_kn.  Products of several heads (grid z): A, B, C advance by a_head, b_head, c_head entries per
+// head, and row m of head h may be multiplied by sigmoid(gate[m, h]).  Rows grouped by expert: B of a row tile is that of
+// expert_of_tile[first row / 128] (negative: the tile is left out).
 // ------------------------------------------------------------------------------------------------
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ A, long long lda, const float* __restrict__ B, long long ldb,
-                                                       float* __restrict__ C, long long ldc, int M, int N, int K) {
+struct GemmF32 {
+  const float *A, *B;
+  float* C;
+  long long lda, ldb, ldc;
+  int M, N, K, b_kn, act;
+  long long a_head, b_head, c_head;
+  const float* gate;
+  long long ldg;
+  const int* expert_of_tile;
+  int experts;
+};
+
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32 p) {
   tfb::pdl_sync();
   __shared__ float sA[16][68], sB[16][68];
-  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, tid = threadIdx.x;
+  const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, h = blockIdx.z, tid = threadIdx.x;
   const int ty = tid >> 4, tx = tid & 15;
+  const float *A = p.A + h * p.a_head, *B = p.B + h * p.b_head;
+  float* C = p.C + h * p.c_head;
+  if (p.expert_of_tile) {
+    const int e = p.expert_of_tile[m0 / 128];
+    if (e < 0) return;
+    TFB_BOUNDS(e < p.experts, 12, e, p.experts);
+    if (e >= p.experts) return;
+    B += e * p.b_head;
+  }
   float acc[4][4];
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-  for (int k0 = 0; k0 < K; k0 += 16) {
+  for (int k0 = 0; k0 < p.K; k0 += 16) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int e = tid + 256 * i, r = e >> 4, k = e & 15;
-      sA[k][r] = (m0 + r < M && k0 + k < K) ? A[(long long)(m0 + r) * lda + k0 + k] : 0.f;
-      sB[k][r] = (n0 + r < N && k0 + k < K) ? B[(long long)(n0 + r) * ldb + k0 + k] : 0.f;
+      sA[k][r] = (m0 + r < p.M && k0 + k < p.K) ? A[(long long)(m0 + r) * p.lda + k0 + k] : 0.f;
+      if (p.b_kn) {
+        const int kk = e >> 6, n = e & 63;
+        sB[kk][n] = (n0 + n < p.N && k0 + kk < p.K) ? B[(long long)(k0 + kk) * p.ldb + n0 + n] : 0.f;
+      } else {
+        sB[k][r] = (n0 + r < p.N && k0 + k < p.K) ? B[(long long)(n0 + r) * p.ldb + k0 + k] : 0.f;
+      }
     }
     __syncthreads();
 #pragma unroll
@@ -259,12 +341,22 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     __syncthreads();
   }
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= p.M) continue;
+    const float f = p.gate ? 1.f / (1.f + expf(-p.gate[m * p.ldg + h])) : 1.f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-      if (m < M && n < N) C[(long long)m * ldc + n] = acc[i][j];
+      const int n = n0 + tx * 4 + j;
+      if (n < p.N) C[(long long)m * p.ldc + n] = act_f32(acc[i][j], p.act) * f;
     }
+  }
+}
+
+static int launch_gemm_f32(const GemmF32& p, int heads, void* stream) {
+  if (p.M <= 0 || p.N <= 0 || p.K <= 0 || heads <= 0 || heads > 65535 || (p.M + 63) / 64 > 65535) return TFB_ERR_ARG;
+  launch_k(gemm_f32_kernel, dim3((p.N + 63) / 64, (p.M + 63) / 64, heads), 256, 0, static_cast<cudaStream_t>(stream), p);
+  return int(cudaGetLastError());
 }
 
 static bool aligned(const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) & (bytes - 1)) == 0; }
@@ -277,23 +369,36 @@ static int grid_for(long long items) {
 
 using bf16 = __nv_bfloat16;
 
-// f32 = 1: activations, table and norm weights are fp32, otherwise bf16.  See ResNormArgs.
+// f32 = 1: activations, table and norm weights are fp32, otherwise bf16.  layer: the kind of norm.  See ResNormArgs.
 TFB_API int tfb_res_norm(const long long* ids, const void* table, long long ld_table, float scale, int vocab, float* x, long long ldx,
-                         const void* y, long long ldy, const void* w_post, const void* w_pre, void* a, long long lda, const int* rows,
-                         int n, int H, float eps, int f32, void* stream) {
+                         const void* y, long long ldy, const void* w_post, const void* b_post, const void* scale_post, const void* w_pre,
+                         const void* b_pre, void* a, long long lda, const int* rows, int n, int H, float eps, int layer, int f32, void* stream) {
   using namespace tfb;
-  if (n <= 0 || H <= 0 || (y && !w_post) || (a && !w_pre) || (ids && !table)) return TFB_ERR_ARG;
-  ResNormArgs p{ids, table, ld_table, scale, vocab, x, ldx, y, ldy, w_post, w_pre, a, lda, rows, H, eps};
+  if (n <= 0 || H <= 0 || (y && (!w_post || (layer && !b_post))) || (w_pre && (!a || (layer && !b_pre))) || (ids && !table)) return TFB_ERR_ARG;
+  ResNormArgs p{ids, table, ld_table, scale, vocab, x, ldx, y, ldy, w_post, b_post, scale_post, w_pre, b_pre, a, lda, rows, H, eps};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int es = f32 ? 4 : 2;
   auto ok = [&](int vec) {
+    for (const void* q : {w_post, b_post, scale_post, w_pre, b_pre})
+      if (q && !aligned(q, vec * es)) return false;
     return H % vec == 0 && ldx % vec == 0 && aligned(x, 16) && (!y || (ldy % vec == 0 && aligned(y, vec * es))) &&
-           (!a || (lda % vec == 0 && aligned(a, vec * es))) && (!ids || (ld_table % vec == 0 && aligned(table, vec * es))) &&
-           (!w_post || aligned(w_post, vec * es)) && (!w_pre || aligned(w_pre, vec * es));
+           (!a || (lda % vec == 0 && aligned(a, vec * es))) && (!ids || (ld_table % vec == 0 && aligned(table, vec * es)));
   };
-  if (f32) return ok(4) ? launch_res_norm<float, 4>(p, n, st) : launch_res_norm<float, 1>(p, n, st);
-  if (ok(8)) return launch_res_norm<bf16, 8>(p, n, st);
-  return ok(4) ? launch_res_norm<bf16, 4>(p, n, st) : launch_res_norm<bf16, 1>(p, n, st);
+#define TFB_RN(T, VEC) (layer ? launch_res_norm<T, true, VEC>(p, n, st) : launch_res_norm<T, false, VEC>(p, n, st))
+  if (f32) return ok(4) ? TFB_RN(float, 4) : TFB_RN(float, 1);
+  if (ok(8)) return TFB_RN(bf16, 8);
+  return ok(4) ? TFB_RN(bf16, 4) : TFB_RN(bf16, 1);
+#undef TFB_RN
+}
+
+TFB_API int tfb_act_rows(const void* in, long long ldi, void* out, long long ldo, int M, int N, int act, int f32, void* stream) {
+  using namespace tfb;
+  if (M <= 0 || N <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const int grid = grid_for((long long)M * N);
+  if (f32) launch_k(act_rows_kernel<float>, grid, 256, 0, st, static_cast<const float*>(in), ldi, static_cast<float*>(out), ldo, M, N, act);
+  else launch_k(act_rows_kernel<bf16>, grid, 256, 0, st, static_cast<const bf16*>(in), ldi, static_cast<bf16*>(out), ldo, M, N, act);
+  return int(cudaGetLastError());
 }
 
 TFB_API int tfb_glu_silu(const void* in, long long ldi, void* out, long long ldo, int M, int F, int f32, void* stream) {
@@ -349,10 +454,24 @@ TFB_API int tfb_gather_rows(const void* pool, long long nslots, const int* pages
   return int(cudaGetLastError());
 }
 
-TFB_API int tfb_gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N, int K,
+TFB_API int tfb_gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N, int K, int act,
                          void* stream) {
   using namespace tfb;
-  if (M <= 0 || N <= 0 || K <= 0 || (M + 63) / 64 > 65535) return TFB_ERR_ARG;
-  launch_k(gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64), 256, 0, static_cast<cudaStream_t>(stream), A, lda, B, ldb, C, ldc, M, N, K);
-  return int(cudaGetLastError());
+  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, 0, act, 0, 0, 0, nullptr, 0, nullptr, 0}, 1, stream);
+}
+
+// One product per head: C[:, h * c_head ...] = A[:, h * a_head ...] . B_h^T (B_h: N rows of B, or K rows with b_kn) * sigmoid(gate[:, h]).
+TFB_API int tfb_gemm_f32_heads(const float* A, long long lda, int a_head, const float* B, long long ldb, int b_kn, float* C, long long ldc, int c_head,
+                               const float* gate, long long ldg, int M, int heads, int N, int K, void* stream) {
+  using namespace tfb;
+  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, b_kn, 0, a_head, (long long)(b_kn ? K : N) * ldb, c_head, gate, ldg, nullptr, 0},
+                         heads, stream);
+}
+
+// Rows grouped by expert (M: rows of the expert buffers), B [experts][N][K] with `stride` entries between experts.
+TFB_API int tfb_moe_gemm_f32(const float* A, long long lda, const float* B, long long ldb, long long stride, float* C, long long ldc,
+                             const int* expert_of_tile, int experts, int M, int N, int K, void* stream) {
+  using namespace tfb;
+  if (!expert_of_tile || experts <= 0) return TFB_ERR_ARG;
+  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, 0, 0, 0, stride, 0, nullptr, 0, expert_of_tile, experts}, 1, stream);
 }

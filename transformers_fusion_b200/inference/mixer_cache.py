@@ -4,6 +4,8 @@
   values per token, with the page allocator and block tables of ``kv_cache``; the layers share one page list per
   sequence.  When every attention layer looks back over a window only, pages that have left the longest window go back to
   the allocator (``first_live_page``), and a prompt's earlier tokens are never written.
+* Latent attention layers: one paged pool with a row of ``latent_width`` entries per token (the latent, zeros behind it), under the
+  same page list.
 * Recurrent layers: a slot per sequence with the fp32 state matrices and the last inputs of the short convolution.  A slot's
   contents are only read by a sequence that goes on; a sequence that starts ignores and overwrites them, so slots need no
   clearing when they change hands.
@@ -27,6 +29,7 @@ class MixerCache:
         self.window = cfg.window
         self.k: Dict[int, torch.Tensor] = {}
         self.v: Dict[int, torch.Tensor] = {}
+        self.latent: Dict[int, torch.Tensor] = {}
         self.state: Dict[int, torch.Tensor] = {}
         self.conv: Dict[int, torch.Tensor] = {}
         for i, l in enumerate(cfg.layers):
@@ -34,6 +37,8 @@ class MixerCache:
             if m.kind == "attention" and m.kv_from is None:
                 self.k[i] = torch.zeros((num_pages * PAGE, m.kv_heads * 2 * m.dim), dtype=dtype, device=device)
                 self.v[i] = torch.zeros((num_pages * PAGE, m.kv_heads * m.vdim), dtype=dtype, device=device)
+            elif m.kind == "latent_attention":
+                self.latent[i] = torch.zeros((num_pages * PAGE, m.latent_width), dtype=dtype, device=device)
             elif m.kind == "delta":
                 self.state[i] = torch.zeros((num_slots, m.heads, m.dim, m.vdim), dtype=torch.float32, device=device)
                 self.conv[i] = torch.zeros((num_slots, m.conv - 1, m.conv_channels), dtype=dtype, device=device)
@@ -67,7 +72,7 @@ class MixerCache:
         return min(n, (self.window - 1) // PAGE + 2) if self.window else n
 
     def bytes_per_token(self) -> float:
-        return float(sum(t.shape[1] * t.element_size() for d in (self.k, self.v) for t in d.values()))
+        return float(sum(t.shape[1] * t.element_size() for d in (self.k, self.v, self.latent) for t in d.values()))
 
     def bytes_per_sequence(self) -> float:
         """Recurrent state of one sequence, whatever its length."""

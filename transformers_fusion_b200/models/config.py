@@ -199,9 +199,39 @@ class GatedDeltaSpec:
 
 
 @dataclass(frozen=True)
+class LatentAttentionSpec:
+    """Latent attention without positions: the keys (``dim`` entries) and values (``vdim``) of every head are read out of one
+    latent of ``kv_rank`` entries per token, which is all that is cached; one output gate per head."""
+    heads: int
+    dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+
+    kind = "latent_attention"
+    window = 0
+
+    @property
+    def latent_width(self) -> int:
+        """Entries of a cached row: the latent, padded to 16 bytes in bf16."""
+        return (self.kv_rank + 7) // 8 * 8
+
+
+@dataclass(frozen=True)
+class MixtureSpec:
+    """Mixture of gated feed-forward experts: ``top`` of ``experts`` per token, weighted by the softmax over the chosen router
+    logits; ``shared_ff`` > 0: one more expert of that size that every token runs."""
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0
+
+
+@dataclass(frozen=True)
 class StackLayer:
     mixer: object
-    ffn_hidden_size: int = 0     # 0: the layer has no feed-forward
+    ffn_hidden_size: int = 0     # dense feed-forward; 0: the layer has none
+    mixture: MixtureSpec = None  # mixture of experts instead of a dense feed-forward
 
 
 @dataclass
@@ -218,6 +248,7 @@ class LanedraConfig:
     max_seq_len: int = 32768
 
     architecture = "Lanedra"
+    tie_embeddings = False
 
     def __post_init__(self):
         for i, l in enumerate(self.layers):
@@ -300,6 +331,87 @@ class LanedraConfig:
                 n += H * (m.conv_channels + 2 * m.heads * m.vdim + 2 * m.heads) + m.conv_channels * m.conv + 2 * m.heads + m.vdim
             n += 2 * H + (3 * H * l.ffn_hidden_size + 2 * H if l.ffn_hidden_size else 0)
         return n
+
+
+@dataclass
+class TekenexConfig:
+    """Tekenex: latent attention and dense (squared-relu) or mixture-of-experts feed-forwards in any order, a layer norm and a
+    learnt per-channel scale on every sublayer's output (the sublayers read the 32-bit residual itself), the embedding table as
+    the head.  ``from_dict`` reads the model folder's config.json; ``max_seq_len`` as in ``LanedraConfig``."""
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    norm_eps: float
+    max_seq_len: int = 32768
+
+    architecture = "Tekenex"
+    embedding_scale = 1.0
+    tie_embeddings = True
+    window = 0                   # every attention layer looks at all earlier keys
+
+    def __post_init__(self):
+        for i, l in enumerate(self.layers):
+            m, x = l.mixer, l.mixture
+            if min(m.heads, m.dim, m.vdim, m.kv_rank) < 1:
+                raise ValueError(f"layer {i}: sizes of the mixer have to be positive")
+            if x is not None and not 1 <= x.top <= x.experts:
+                raise ValueError(f"layer {i}: cannot choose {x.top} of {x.experts} experts")
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @classmethod
+    def from_dict(cls, d: dict, **extra) -> "TekenexConfig":
+        layers = []
+        for i, e in enumerate(d["layers"]):
+            if e["type"] != "latent_attention":
+                raise ValueError(f"layer {i}: unknown mixer '{e['type']}'")
+            m, f = e["mixer"], e.get("mlp")
+            mix = LatentAttentionSpec(m["heads"], m["dim"], m["vdim"], m["kv_rank"], float(m["scale"]))
+            kind = f.get("kind", "dense") if f else None
+            if kind == "dense":
+                layers.append(StackLayer(mix, f["ff"]))
+            elif kind == "moe":
+                r, sh = f["router"], f.get("shared")
+                layers.append(StackLayer(mix, 0, MixtureSpec(r["experts"], r["top"], f["expert"]["ff"], sh["ff"] if sh else 0)))
+            elif kind is None:
+                layers.append(StackLayer(mix))
+            else:
+                raise ValueError(f"layer {i}: unknown feed-forward '{kind}'")
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], layers=layers, norm_eps=float(d["norm"]["eps"]), **extra)
+
+    def to_dict(self) -> dict:
+        """The config.json form."""
+        out = []
+        for l in self.layers:
+            m, x = l.mixer, l.mixture
+            f = {"kind": "dense", "ff": l.ffn_hidden_size} if l.ffn_hidden_size else None
+            if x is not None:
+                f = {"kind": "moe", "expert": {"ff": x.ff}, "router": {"experts": x.experts, "top": x.top}}
+                if x.shared_ff:
+                    f["shared"] = {"ff": x.shared_ff}
+            out.append({"type": m.kind, "mlp": f,
+                        "mixer": {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "kv_rank": m.kv_rank, "scale": m.scale}})
+        return {"architecture": self.architecture, "layers": out, "norm": {"eps": self.norm_eps}, "vocab": self.vocab_size,
+                "width": self.hidden_size}
+
+    def _count(self, active: bool) -> int:
+        H, n = self.hidden_size, self.vocab_size * self.hidden_size + 2 * self.hidden_size
+        for l in self.layers:
+            m, x = l.mixer, l.mixture
+            n += H * (m.heads * m.dim + m.kv_rank + m.heads + m.heads * m.vdim) + m.kv_rank * (1 + m.heads * (m.dim + m.vdim)) + 3 * H
+            n += 2 * H * l.ffn_hidden_size + (3 * H if l.ffn_hidden_size else 0)
+            if x is not None:
+                n += 3 * H * (x.ff * (x.top if active else x.experts) + x.shared_ff) + x.experts * (H + 1) + 3 * H
+        return n
+
+    def num_params(self) -> int:
+        return self._count(False)
+
+    def active_params(self) -> int:
+        """Parameters that take part in one token's pass."""
+        return self._count(True)
 
 
 # Named shapes used by the benchmarks and tests (BASELINE configs).

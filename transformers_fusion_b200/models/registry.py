@@ -14,6 +14,7 @@ import torch
 # architecture -> (module, model class); the class names its configuration in ``config_cls``
 ARCHITECTURES: Dict[str, Tuple[str, str]] = {
     "Lanedra": ("lanedra", "LanedraModel"),
+    "Tekenex": ("tekenex", "TekenexModel"),
 }
 
 

@@ -1,14 +1,21 @@
-"""Decoders built from a list of layers with different sequence mixers: the mixers and the feed-forward as parameter modules
+"""Decoders built from a list of layers with different sequence mixers: the mixers and the feed-forwards as parameter modules
 with one forward pass each over a batch description (``StepBatch``), and the model that runs them over a 32-bit residual
-stream with a norm before and after every sublayer.
+stream.  Where the norms stand is the layer class's business: before and after every sublayer (``SandwichLayer``) or on its output
+only (``OutputNormLayer``).
 
 The engine drives the same passes for prompts, for portions of prompts and for decoding; what is remembered between steps
 lives in ``inference.mixer_cache``.  A pass of one layer is, for a prompt or a decode step alike:
 
   attention   GEMM [q | k | v], rotation + cache append, attention with its epilogue (difference of the maps, norm, scale), GEMM
+  latent      GEMM [q | latent | gates], norm of the latent + cache append, then
+                prompts   GEMM latent -> [k | v], attention with the head gates in its epilogue, GEMM
+                decoding  queries taken to the latent space, attention over the cached latents, values read out of the result
+                          head by head with the gates, GEMM
   delta       GEMM [q | k | v | gate | b | a], convolution + unit lengths + gates, recurrence (+ gated norm), GEMM
-  MLP         GEMM [gate | up], silu(gate) * up, GEMM
-  between     post-norm of the sublayer, residual add and pre-norm of the next sublayer, one kernel
+  MLP         GEMM [gate | up], silu(gate) * up, GEMM;  or GEMM with the squared relu in its epilogue, GEMM
+  mixture     router GEMM (fp32 logits), top-k + expert segments, rows by expert, grouped GEMM, silu(gate) * up, grouped GEMM,
+              weighted sum + shared expert
+  between     norm and scale of the sublayer's output, residual add and norm of (or rounding for) the next sublayer, one kernel
 
 bf16 parameters: bf16 activations and tensor-core products; fp32 parameters: everything in true fp32."""
 from __future__ import annotations
@@ -20,6 +27,7 @@ import torch
 import torch.nn as nn
 
 from ..ops import functional as F
+from ..ops import moe as X
 from ..ops import stack as K
 
 
@@ -41,7 +49,7 @@ class StepBatch:
 
 
 def _param(*shape, device, dtype, pitched=True):
-    w = K.padded_weight(*shape, dtype, device) if pitched and len(shape) == 2 else torch.zeros(shape, dtype=dtype, device=device)
+    w = K.padded_weight(*shape[-2:], dtype, device, shape[:-2]) if pitched and len(shape) > 1 else torch.zeros(shape, dtype=dtype, device=device)
     return nn.Parameter(w, requires_grad=False)
 
 
@@ -145,6 +153,53 @@ class GatedDelta(nn.Module):
         return lin(o, i, "o", self.o)
 
 
+class LatentAttention(nn.Module):
+    """Attention without positions over one cached latent per token, with an output gate per head."""
+    linear_names = ("proj", "o")
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+        super().__init__()
+        self.spec, self.eps, self.index = spec, eps, index
+        kw = dict(device=device, dtype=dtype)
+        self.nq, self.nv = spec.heads * spec.dim, spec.heads * spec.vdim
+        self.proj = _param(self.nq + spec.kv_rank + spec.heads, hidden, **kw)
+        self.norm = _param(spec.kv_rank, **kw)
+        self.ukv = _param(self.nq + self.nv, spec.kv_rank, **kw)
+        self.o = _param(hidden, self.nv, **kw)
+
+    def tensors(self):
+        a = self.nq + self.spec.kv_rank
+        yield "q", self.proj.data[:self.nq]
+        yield "dkv", self.proj.data[self.nq:a]
+        yield "dkv.norm", self.norm.data
+        yield "uk", self.ukv.data[:self.nq]
+        yield "uv", self.ukv.data[self.nq:]
+        yield "g", self.proj.data[a:]
+        yield "o", self.o.data
+
+    def finalize(self):
+        pass
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        s, i = self.spec, self.index
+        p = lin(h, i, "proj", self.proj)
+        q, gate = p[:, :self.nq], p[:, self.nq + s.kv_rank:]
+        pool = cache.latent[i]
+        c = K.latent_append(p[:, self.nq:self.nq + s.kv_rank], self.norm.data, self.eps, b.slots, pool, want_rows=not b.decode and b.pos0 == 0)
+        if b.decode:
+            u = K.head_linear(q, self.ukv.data[:self.nq], s.heads, s.dim, s.kv_rank, transposed=True)
+            u = K.latent_decode(u, pool, b.block_table, b.positions, s.heads, s.kv_rank, s.scale)
+            o = K.head_linear(u, self.ukv.data[self.nq:], s.heads, s.kv_rank, s.vdim, gate=gate)
+        else:
+            n = b.S
+            if b.pos0:                         # the latents of the whole sequence so far, this portion's included
+                n = b.pos0 + b.S
+                c = K.gather_rows(pool, b.pages, 0, n)[:, :s.kv_rank]
+            e = lin(c, i, "ukv", self.ukv)
+            o = K.head_attn(q, e[:, :self.nq], e[:, self.nq:], b.B, b.S, n, s.heads, s.heads, s.dim, s.vdim, s.scale, gate)
+        return lin(o, i, "o", self.o)
+
+
 class GatedMLP(nn.Module):
     linear_names = ("gate_up", "down")
 
@@ -163,29 +218,89 @@ class GatedMLP(nn.Module):
         return lin(K.glu_silu(lin(h, self.index, "gate_up", self.gate_up)), self.index, "down", self.down)
 
 
-MIXERS = {"attention": DiffAttention, "delta": GatedDelta}
+class SquaredMLP(nn.Module):
+    """down(relu(up h)^2)."""
+    linear_names = ("up", "down")
+
+    def __init__(self, hidden: int, ff: int, index: int, device, dtype):
+        super().__init__()
+        self.index = index
+        self.up, self.down = _param(ff, hidden, device=device, dtype=dtype), _param(hidden, ff, device=device, dtype=dtype)
+
+    def tensors(self):
+        yield "up", self.up.data
+        yield "down", self.down.data
+
+    def forward(self, h, lin):
+        return lin(lin(h, self.index, "up", self.up, act="relu2"), self.index, "down", self.down)
 
 
-class SandwichLayer(nn.Module):
-    """norm1, mixer, norm1b and - unless the layer is a mixer alone - norm2, feed-forward, norm2b."""
+class MixtureMLP(nn.Module):
+    """Gated experts chosen per token, and a gated expert that every token runs."""
+
+    def __init__(self, hidden: int, spec, index: int, device, dtype):
+        super().__init__()
+        self.spec, self.index = spec, index
+        kw = dict(device=device, dtype=dtype)
+        self.router, self.router_bias = _param(spec.experts, hidden, **kw), _param(spec.experts, **kw)
+        self.gate_up, self.down = _param(spec.experts, 2 * spec.ff, hidden, **kw), _param(spec.experts, hidden, spec.ff, **kw)
+        self.shared = GatedMLP(hidden, spec.shared_ff, index, device, dtype) if spec.shared_ff else None
+
+    def tensors(self):
+        F = self.spec.ff
+        for e in range(self.spec.experts):
+            yield f"e{e}.gate", self.gate_up.data[e, :F]
+            yield f"e{e}.up", self.gate_up.data[e, F:]
+            yield f"e{e}.down", self.down.data[e]
+        yield "router", self.router.data
+        yield "router.b", self.router_bias.data
+        if self.shared is not None:
+            for n, t in self.shared.tensors():
+                yield "shared." + n, t
+
+    def forward(self, h, lin):
+        r = X.route(K.linear(h, self.router.data, out_dtype=torch.float32), self.router_bias.data, self.spec.top)
+        g = X.expert_linear(X.expert_rows(h, r), self.gate_up.data, r)
+        y = X.expert_linear(X.expert_glu(g, r), self.down.data, r)
+        return X.weighted_sum(y, r, self.shared(h, lin) if self.shared is not None else None)
+
+
+MIXERS = {"attention": DiffAttention, "delta": GatedDelta, "latent_attention": LatentAttention}
+
+
+class ResidualLayer(nn.Module):
+    """A mixer and, unless the layer is a mixer alone, a feed-forward.  ``parts`` lists the sublayers with what ``K.res_norm`` does
+    to the input of each (``pre``) and to its output (``post``)."""
+    norm_kind = "rms"
+    dense_mlp = GatedMLP
 
     def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
         super().__init__()
-        kw = dict(device=device, dtype=dtype)
         self.mixer = MIXERS[spec.mixer.kind](spec.mixer, hidden, eps, index, device, dtype)
-        self.norm1, self.norm1b = _param(hidden, **kw), _param(hidden, **kw)
-        self.mlp = GatedMLP(hidden, spec.ffn_hidden_size, index, device, dtype) if spec.ffn_hidden_size else None
-        if self.mlp is not None:
-            self.norm2, self.norm2b = _param(hidden, **kw), _param(hidden, **kw)
+        self.mlp = None
+        if spec.mixture is not None:
+            self.mlp = MixtureMLP(hidden, spec.mixture, index, device, dtype)
+        elif spec.ffn_hidden_size:
+            self.mlp = self.dense_mlp(hidden, spec.ffn_hidden_size, index, device, dtype)
+        for n in self.vector_names():
+            setattr(self, n.replace(".", "_"), _param(hidden, device=device, dtype=dtype))
+
+    def vector(self, name):
+        return getattr(self, name.replace(".", "_")).data
 
     @property
     def linears(self):
         """{name: matrix} of the layer's products (what a low-bit weight format may replace)."""
-        return {n: getattr(m, n) for m in (self.mixer, self.mlp) if m is not None for n in m.linear_names}
+        out = {}
+        for m in (self.mixer, self.mlp):
+            m = m.shared if isinstance(m, MixtureMLP) else m
+            if m is not None:
+                out.update({n: getattr(m, n) for n in m.linear_names})
+        return out
 
     def tensors(self):
-        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if self.mlp is not None else ()):
-            yield n, getattr(self, n).data
+        for n in self.vector_names():
+            yield n, self.vector(n)
         for n, t in self.mixer.tensors():
             yield "mix." + n, t
         if self.mlp is not None:
@@ -193,15 +308,47 @@ class SandwichLayer(nn.Module):
                 yield "mlp." + n, t
 
 
-def _plain_linear(x, index, name, w):
-    return K.linear(x, w.data)
+class SandwichLayer(ResidualLayer):
+    """norm1, mixer, norm1b and norm2, feed-forward, norm2b: RMS norms whose weight is the deviation from one."""
+    final_names = ("final.norm",)
+
+    def vector_names(self):
+        return ("norm1", "norm1b") + (("norm2", "norm2b") if self.mlp is not None else ())
+
+    def parts(self):
+        v = self.vector
+        yield self.mixer, {"w_pre": v("norm1")}, {"w_post": v("norm1b")}
+        if self.mlp is not None:
+            yield self.mlp, {"w_pre": v("norm2")}, {"w_post": v("norm2b")}
+
+
+class OutputNormLayer(ResidualLayer):
+    """The sublayers read the residual itself; a layer norm (norm1, norm2) and a per-channel scale (ls1, ls2) on what they return."""
+    norm_kind = "layer"
+    dense_mlp = SquaredMLP
+    final_names = ("final.norm", "final.norm.b")
+
+    def vector_names(self):
+        return sum(((f"norm{k}", f"norm{k}.b", f"ls{k}") for k in ((1, 2) if self.mlp is not None else (1,))), ())
+
+    def parts(self):
+        v = self.vector
+        for k, m in ((1, self.mixer), (2, self.mlp)):
+            if m is not None:
+                w = v(f"norm{k}")
+                yield m, {"cast": w.dtype}, {"w_post": w, "b_post": v(f"norm{k}.b"), "scale_post": v(f"ls{k}")}
+
+
+def _plain_linear(x, index, name, w, act=None):
+    return K.linear(x, w.data, act=act)
 
 
 class StackModel(nn.Module):
     """Embedding, layers, final norm, head.  ``run`` is the pass the engine drives; ``forward`` / ``hidden_states`` are whole
     sequences without a cache."""
     kernel_units = K.UNITS
-    linear = staticmethod(K.linear)
+    layer_cls = SandwichLayer
+    linear, activation = staticmethod(K.linear), staticmethod(K.activation)
     runs_fp32 = True             # every kernel of the pass has a true fp32 form
 
     def __init__(self, cfg, device=None, dtype=torch.bfloat16, seed: Optional[int] = 0):
@@ -210,9 +357,10 @@ class StackModel(nn.Module):
         device = torch.device(device if device is not None else "cpu")
         kw = dict(device=device, dtype=dtype)
         self.tok_embeddings = _param(cfg.vocab_size, cfg.hidden_size, **kw)
-        self.layers = nn.ModuleList([SandwichLayer(l, cfg.hidden_size, cfg.norm_eps, i, device, dtype) for i, l in enumerate(cfg.layers)])
+        self.layers = nn.ModuleList([self.layer_cls(l, cfg.hidden_size, cfg.norm_eps, i, device, dtype) for i, l in enumerate(cfg.layers)])
         self.norm = _param(cfg.hidden_size, **kw)
-        self.lm_head = _param(cfg.vocab_size, cfg.hidden_size, **kw)
+        self.norm_bias = _param(cfg.hidden_size, **kw) if len(self.layer_cls.final_names) > 1 else None
+        self.lm_head = self.tok_embeddings if cfg.tie_embeddings else _param(cfg.vocab_size, cfg.hidden_size, **kw)
         self._rope = {}
         if seed is not None:
             self.init_weights(seed)
@@ -220,6 +368,8 @@ class StackModel(nn.Module):
     def init_weights(self, seed: int = 0):
         """Random weights that keep activations of order one: N(0, 1 / fan-in) matrices, small deviations for the norms, decays
         between about 0.5 and 1."""
+        about_one = lambda n: n.endswith(("mix.norm", "dkv.norm")) or \
+            (self.layer_cls.norm_kind == "layer" and n.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2", "ls1", "ls2"))
         g = torch.Generator(device="cpu").manual_seed(seed)
         with torch.no_grad():
             for name, t in self.named_tensors():
@@ -231,7 +381,7 @@ class StackModel(nn.Module):
                     r = r * t.shape[1] ** -0.5
                 elif t.dim() == 2:
                     r = r * (1.0 if name == self.embed_name else t.shape[1] ** -0.5)
-                elif name.endswith("mix.norm"):
+                elif about_one(name):
                     r = 1 + 0.1 * r
                 else:
                     r = 0.1 * r
@@ -243,14 +393,15 @@ class StackModel(nn.Module):
         for l in self.layers:
             l.mixer.finalize()
 
-    embed_name, head_name, norm_name = "embed", "head", "final.norm"
+    embed_name, head_name = "embed", "head"
 
     def named_tensors(self):
         """(name in the model folder, view into the parameters) pairs."""
         out = [(self.embed_name, self.tok_embeddings.data)]
         for i, l in enumerate(self.layers):
             out += [(f"l{i}.{n}", t) for n, t in l.tensors()]
-        return out + [(self.norm_name, self.norm.data), (self.head_name, self.lm_head.data)]
+        out += list(zip(self.layer_cls.final_names, (t.data for t in (self.norm, self.norm_bias) if t is not None)))
+        return out if self.cfg.tie_embeddings else out + [(self.head_name, self.lm_head.data)]
 
     def get_parameters(self):
         return list(self.parameters())
@@ -288,26 +439,24 @@ class StackModel(nn.Module):
         """One step over all layers.  Returns the final-normed rows (of ``row_index``, int32; all rows without it).
         ``residuals``: a list that receives a copy of the residual stream after every layer."""
         cfg = self.cfg
-        eps, n = cfg.norm_eps, b.tokens.shape[0]
+        eps, n, kind = cfg.norm_eps, b.tokens.shape[0], self.layer_cls.norm_kind
         x = torch.empty((n, cfg.hidden_size), dtype=torch.float32, device=self.device)
-        h = K.res_norm(x, eps, ids=b.tokens, table=self.tok_embeddings.data, scale=cfg.embedding_scale, w_pre=self.layers[0].norm1.data)
+        parts = [(i, l) + p for i, l in enumerate(self.layers) for p in l.parts()]
+        pre = [p[3] for p in parts] + [{"w_pre": self.norm.data, "b_pre": self.norm_bias.data if self.norm_bias is not None else None}]
+        h = K.res_norm(x, eps, ids=b.tokens, table=self.tok_embeddings.data, scale=cfg.embedding_scale, kind=kind, **pre[0])
         kv = {}
-        for i, l in enumerate(self.layers):
-            last = i + 1 == len(self.layers)
-            nxt, rows = (self.norm.data, row_index) if last else (self.layers[i + 1].norm1.data, None)
-            rope = self.rope(l.mixer.spec.rot, max_pos) if l.mixer.spec.kind == "attention" else None
-            y = l.mixer(h, b, cache, rope, lin, kv)
-            if l.mlp is not None:
-                h = K.res_norm(x, eps, y=y, w_post=l.norm1b.data, w_pre=l.norm2.data)
-                y = l.mlp(h, lin)
-                post = l.norm2b.data
+        for k, (i, l, m, _, post) in enumerate(parts):
+            if m is l.mixer:
+                rope = self.rope(m.spec.rot, max_pos) if m.spec.kind == "attention" else None
+                y = m(h, b, cache, rope, lin, kv)
             else:
-                post = l.norm1b.data
-            if residuals is not None:
+                y = m(h, lin)
+            last = k + 1 == len(parts)
+            if residuals is not None and (last or parts[k + 1][0] != i):
                 z = x.clone()
-                K.res_norm(z, eps, y=y, w_post=post)
+                K.res_norm(z, eps, y=y, kind=kind, **post)
                 residuals.append(z)
-            h = K.res_norm(x, eps, y=y, w_post=post, w_pre=nxt, row_index=rows)
+            h = K.res_norm(x, eps, y=y, kind=kind, row_index=row_index if last else None, **post, **pre[k + 1])
         return h
 
     def head(self, h):

@@ -13,6 +13,8 @@ moe_gather / moe_scatter kernels (src/backend/gpu_compute_cuda.cpp:539-616).
 from __future__ import annotations
 
 import ctypes as C
+from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -28,6 +30,13 @@ _lib.register("tfb_moe_permute", [c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c
 _lib.register("tfb_moe_combine", [c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_p])
 _lib.register("tfb_moe_combine_bwd", [c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_i, c_p])
 _lib.register("tfb_moe_permute_bwd", [c_p, c_p, c_p, c_i, c_i, c_i, c_p])
+
+
+_lib.register("tfb_moe_route", [c_p, c_p, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_ll, c_i, c_p])
+_lib.register("tfb_moe_gather", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_moe_glu", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_p])
+_lib.register("tfb_moe_gemm_f32", [c_p, c_ll, c_p, c_ll, c_ll, c_p, c_ll, c_p, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_moe_weighted_sum", [c_p, c_ll, c_p, c_p, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 
 
 class _Group(C.Structure):
@@ -300,3 +309,114 @@ class MoEFFN(torch.autograd.Function):
 
 def moe_ffn(x, logits, gate_up, down, k=2, renormalize=True, act="silu", lb_weight=0.01, z_weight=0.0):
     return MoEFFN.apply(x, logits, gate_up, down, k, renormalize, act, lb_weight, z_weight)
+
+
+# ---------------------------------------------------------------------------------------------
+# the serving form: no gradients, fp32 or bf16, any sizes (kernels in csrc/kernels/moe_serve.cu)
+# ---------------------------------------------------------------------------------------------
+@dataclass
+class Routing:
+    """Chosen experts and weights of T tokens, and the rows of the expert buffers that serve them: every expert's assignments are
+    consecutive rows from a multiple of 128 on; rows without an assignment hold nothing."""
+    idx: torch.Tensor                          # int32 [T, k]
+    w: torch.Tensor                            # fp32 [T, k]
+    row_of: torch.Tensor                       # int32 [T, k]
+    expert_of_tile: torch.Tensor               # int32 [max_rows / 128], -1: no expert
+    max_rows: int
+    counts: Optional[torch.Tensor] = None      # int32 [E] (CUDA)
+
+
+def route(logits, bias, k) -> Routing:
+    """The k largest of the fp32 logits [T, E] + bias (the lower index first among equals), weighted by the softmax over them."""
+    T, E = logits.shape
+    assert logits.dtype == torch.float32
+    tiles = T * k // 128 + min(E, T * k)       # enough for any distribution of the assignments
+    dev = logits.device
+    if not logits.is_cuda:
+        z = logits + bias.float()
+        idx = torch.argsort(z, dim=-1, descending=True, stable=True)[:, :k]
+        w = torch.softmax(z.gather(1, idx), -1)
+        row_of, of_tile, off = torch.empty(T * k, dtype=torch.int32), [], 0
+        flat = idx.reshape(-1)
+        for e in range(E):
+            mine = (flat == e).nonzero()[:, 0]
+            row_of[mine] = off + torch.arange(len(mine), dtype=torch.int32)
+            n = (len(mine) + 127) // 128
+            of_tile += [e] * n
+            off += n * 128
+        of_tile += [-1] * (tiles - len(of_tile))
+        return Routing(idx.int(), w, row_of.view(T, k), torch.tensor(of_tile, dtype=torch.int32), tiles * 128)
+    i32 = lambda *s: torch.empty(s, dtype=torch.int32, device=dev)
+    r = Routing(i32(T, k), torch.empty((T, k), dtype=torch.float32, device=dev), i32(T, k), i32(tiles), tiles * 128, i32(E))
+    rank, start = i32(T, k), i32(E)
+    check(_lib.lib().tfb_moe_route(logits.data_ptr(), bias.data_ptr(), T, E, k, r.idx.data_ptr(), r.w.data_ptr(), r.row_of.data_ptr(),
+                                   r.expert_of_tile.data_ptr(), r.counts.data_ptr(), rank.data_ptr(), start.data_ptr(), tiles,
+                                   logits.stride(0), int(bias.dtype == torch.float32), stream()), "moe_route", 1 if T <= 256 else 3)
+    return r
+
+
+def _out_rows(n, width, like):
+    return torch.empty((n, (width + 7) // 8 * 8), dtype=like.dtype, device=like.device)[:, :width]
+
+
+def _is32(t):
+    return int(t.dtype == torch.float32)
+
+
+def expert_rows(x, r: Routing):
+    """x [T, H] -> [max_rows, H] with the row of every assignment in its expert's segment."""
+    T, H = x.shape
+    k = r.idx.shape[1]
+    if not x.is_cuda:
+        xp = torch.zeros((r.max_rows, H), dtype=x.dtype)
+        xp[r.row_of.reshape(-1).long()] = x.repeat_interleave(k, 0)
+        return xp
+    xp = _out_rows(r.max_rows, H, x)
+    check(_lib.lib().tfb_moe_gather(x.data_ptr(), x.stride(0), r.row_of.data_ptr(), xp.data_ptr(), xp.stride(0), T, k, H, _is32(x), stream()),
+          "moe_gather")
+    return xp
+
+
+def expert_linear(xp, w, r: Routing):
+    """xp [max_rows, K] @ w[e]^T per expert segment, w [E, N, K]."""
+    n, Kd = xp.shape
+    E, N, _ = w.shape
+    out = _out_rows(n, N, xp) if xp.is_cuda else torch.zeros((n, N), dtype=xp.dtype)
+    if not xp.is_cuda:
+        for i, e in enumerate(r.expert_of_tile.tolist()):
+            if e >= 0:
+                out[i * 128:(i + 1) * 128] = (xp[i * 128:(i + 1) * 128].float() @ w[e].float().t()).to(xp.dtype)
+    elif xp.dtype == torch.float32:
+        check(_lib.lib().tfb_moe_gemm_f32(xp.data_ptr(), xp.stride(0), w.data_ptr(), w.stride(1), w.stride(0), out.data_ptr(), out.stride(0),
+                                          r.expert_of_tile.data_ptr(), E, n, N, Kd, stream()), "moe_gemm_f32")
+    else:
+        g = _Group(1, E, r.expert_of_tile.data_ptr(), None, w.stride(0), 0)
+        check(_grouped_fn()(xp.data_ptr(), xp.stride(0), 0, w.data_ptr(), w.stride(1), 0, out.data_ptr(), out.stride(0), n, N, Kd, 1.0, 0, C.byref(g),
+                            _lib.status_word(xp.device).data_ptr(), stream()), "gemm_grouped")
+    return out
+
+
+def expert_glu(gu, r: Routing):
+    """silu(gate) * up of the assigned rows of [gate | up]."""
+    Fh = gu.shape[1] // 2
+    if not gu.is_cuda:
+        g = gu[:, :Fh].float()
+        return (g * torch.sigmoid(g) * gu[:, Fh:].float()).to(gu.dtype)
+    out = _out_rows(gu.shape[0], Fh, gu)
+    check(_lib.lib().tfb_moe_glu(gu.data_ptr(), gu.stride(0), r.row_of.data_ptr(), out.data_ptr(), out.stride(0), r.row_of.numel(), Fh, _is32(gu),
+                                 stream()), "moe_glu")
+    return out
+
+
+def weighted_sum(yp, r: Routing, base=None):
+    """sum_k w[t, k] * yp[row_of[t, k]] (+ base[t])."""
+    T, k = r.idx.shape
+    H = yp.shape[1]
+    if not yp.is_cuda:
+        y = (yp[r.row_of.reshape(-1).long()].view(T, k, H).float() * r.w[..., None]).sum(1)
+        return (y if base is None else y + base.float()).to(yp.dtype)
+    y = _out_rows(T, H, yp)
+    check(_lib.lib().tfb_moe_weighted_sum(yp.data_ptr(), yp.stride(0), r.row_of.data_ptr(), r.w.data_ptr(), ptr(base),
+                                          base.stride(0) if base is not None else 0, y.data_ptr(), y.stride(0), T, k, H, _is32(yp), stream()),
+          "moe_weighted_sum")
+    return y

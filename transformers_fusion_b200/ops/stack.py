@@ -1,8 +1,8 @@
 """Raw operators of decoders that are a stack of different sequence mixers over a 32-bit residual stream: norms around
-every sublayer, partial rotary embedding, differential attention, gated delta rule, true fp32 products.
+every sublayer, partial rotary embedding, differential attention, latent attention, gated delta rule, true fp32 products.
 
 As in ``functional``: CUDA tensors go to the sm_100a kernels (``csrc/kernels/stack_ops.cu``, ``diff_attention.cu``,
-``delta_rule.cu``), CPU tensors run the plain PyTorch statement of the same math.  Activations are bf16 or fp32 (the dtype of
+``latent_attention.cu``, ``delta_rule.cu``), CPU tensors run the plain PyTorch statement of the same math.  Activations are bf16 or fp32 (the dtype of
 the tensors decides); the residual, norms, rotation, attention scores and weights, and the recurrence are fp32 in both."""
 from __future__ import annotations
 
@@ -17,13 +17,21 @@ from . import functional as F
 from ._lib import c_f, c_i, c_ll, c_p, check, ptr, stream
 
 UNITS = ("tfb_host", "gemm_bf16", "stack_ops", "diff_attention", "delta_rule")    # translation units these operators need
+UNITS_LATENT = ("tfb_host", "gemm_bf16", "stack_ops", "latent_attention", "moe_serve")
 PAGE = 16
+ACT = {None: 0, "relu2": 4}      # codes of the product epilogues (gemm_bf16.cu: apply_act)
 
-_lib.register("tfb_res_norm", [c_p, c_p, c_ll, c_f, c_i, c_p, c_ll, c_p, c_ll, c_p, c_p, c_p, c_ll, c_p, c_i, c_i, c_f, c_i, c_p])
+_lib.register("tfb_res_norm", [c_p, c_p, c_ll, c_f, c_i, c_p, c_ll, c_p, c_ll, c_p, c_p, c_p, c_p, c_p, c_p, c_ll, c_p, c_i, c_i, c_f, c_i, c_i, c_p])
 _lib.register("tfb_glu_silu", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
 _lib.register("tfb_rope_append", [c_p, c_ll, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_gather_rows", [c_p, c_ll, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p])
-_lib.register("tfb_gemm_f32", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
+_lib.register("tfb_gemm_f32", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_act_rows", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_latent_append", [c_p, c_ll, c_p, c_f, c_p, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_head_linear", [c_p, c_ll, c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_head_attn", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p])
+_lib.register("tfb_latent_decode_plan", [c_i, c_i, c_i, c_i, c_i])
+_lib.register("tfb_latent_decode", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p])
 _lib.register("tfb_diff_attn_fwd", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_f, c_f, c_i,
                                     c_p, c_p])
 _lib.register("tfb_diff_decode_tc", [c_i, c_i, c_i])
@@ -46,27 +54,44 @@ def rows(n: int, width: int, dtype, device) -> torch.Tensor:
     return torch.empty((n, (width + 7) // 8 * 8), dtype=dtype, device=device)[:, :width]
 
 
-def padded_weight(n: int, width: int, dtype, device) -> torch.Tensor:
-    """Zero [n, width] matrix with the same pitch rule."""
-    return torch.zeros((n, (width + 7) // 8 * 8), dtype=dtype, device=device)[:, :width]
+def padded_weight(n: int, width: int, dtype, device, lead=()) -> torch.Tensor:
+    """Zero [*lead, n, width] matrices with the same pitch rule."""
+    return torch.zeros((*lead, n, (width + 7) // 8 * 8), dtype=dtype, device=device)[..., :width]
 
 
 # ---------------------------------------------------------------------------------------------------- products
-def linear(x, w, out_dtype=None):
-    """x [M, K] @ w [N, K]^T.  bf16 operands: tensor-core GEMM with fp32 accumulation (``out_dtype`` fp32 keeps the
-    accumulator's precision); fp32 operands: FFMA in true fp32."""
+def linear(x, w, out_dtype=None, act=None):
+    """act(x [M, K] @ w [N, K]^T).  bf16 operands: tensor-core GEMM with fp32 accumulation (``out_dtype`` fp32 keeps the
+    accumulator's precision); fp32 operands: FFMA in true fp32.  ``act``: None or "relu2"."""
     out_dtype = out_dtype or x.dtype
     if not x.is_cuda:
-        return (x.float() @ w.float().t()).to(out_dtype)
+        return activation(x.float() @ w.float().t(), act).to(out_dtype)
     M, K = x.shape
     N = w.shape[0]
     out = rows(M, N, out_dtype, x.device)
     if x.dtype == torch.float32:
         assert w.dtype == torch.float32 and w.shape[1] == K and x.stride(1) == 1 and w.stride(1) == 1
-        check(_lib.lib().tfb_gemm_f32(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, stream()),
-              "gemm_f32")
+        check(_lib.lib().tfb_gemm_f32(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, ACT[act],
+                                      stream()), "gemm_f32")
         return out
-    return F.gemm(x, w, out=out)
+    if act is None:
+        return F.gemm(x, w, out=out)
+    assert x.dtype == w.dtype == torch.bfloat16 and x.stride(1) == w.stride(1) == 1 and out_dtype == torch.bfloat16
+    check(_lib.lib().tfb_gemm_bf16(x.data_ptr(), x.stride(0), 0, w.data_ptr(), w.stride(0), 0, out.data_ptr(), out.stride(0), M, N, K, None, None, 0,
+                                   1.0, ACT[act], 0, 0, _lib.status_word(x.device).data_ptr(), stream()), "gemm_bf16")
+    return out
+
+
+def activation(x, act):
+    """The activation of ``linear`` alone."""
+    if act is None:
+        return x
+    assert act == "relu2", act
+    if not x.is_cuda:
+        return torch.relu(x.float()).square().to(x.dtype)
+    out = rows(*x.shape, x.dtype, x.device)
+    check(_lib.lib().tfb_act_rows(x.data_ptr(), x.stride(0), out.data_ptr(), out.stride(0), *x.shape, ACT[act], _f32(x), stream()), "act_rows")
+    return out
 
 
 # ---------------------------------------------------------------------------------------------------- norms
@@ -75,27 +100,41 @@ def centred_rms(x, w, eps):
     return xf / torch.sqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * (1 + w.float())
 
 
-def res_norm(x, eps, *, y=None, w_post=None, w_pre=None, ids=None, table=None, scale=1.0, row_index=None, dtype=None):
-    """x += norm(y) * (1 + w_post) on the fp32 residual ``x`` [n, H] in place; returns norm(x) * (1 + w_pre) in the
-    activation dtype (None without ``w_pre``).  ``ids``: x starts as scale * table[ids].  ``row_index`` (int32): only those
+def layer_norm(x, w, b, eps):
+    d = x.float()
+    d = d - d.mean(-1, keepdim=True)
+    return d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w.float() + b.float()
+
+
+def res_norm(x, eps, *, y=None, w_post=None, b_post=None, scale_post=None, w_pre=None, b_pre=None, cast=None, ids=None, table=None, scale=1.0,
+             row_index=None, dtype=None, kind="rms"):
+    """x += norm(y; w_post, b_post) * scale_post on the fp32 residual ``x`` [n, H] in place; returns norm(x; w_pre, b_pre) in the
+    activation dtype, x itself in the dtype ``cast`` without ``w_pre``, None without both.  ``kind``: "rms" (weights are
+    deviations from one, no bias) or "layer".  ``ids``: x starts as scale * table[ids].  ``row_index`` (int32): only those
     rows are computed and returned, and x keeps its values."""
     if not x.is_cuda:
+        norm = (lambda t, w, b: centred_rms(t, w, eps)) if kind == "rms" else (lambda t, w, b: layer_norm(t, w, b, eps))
         v = table[ids.long()].float() * scale if ids is not None else x
         if y is not None:
-            v = v + centred_rms(y, w_post, eps)
+            z = norm(y, w_post, b_post)
+            v = v + (z if scale_post is None else z * scale_post.float())
         if row_index is None:
             x.copy_(v)
         else:
             v = v[row_index.long()]
-        return None if w_pre is None else centred_rms(v, w_pre, eps).to(dtype or w_pre.dtype)
+        if w_pre is None:
+            return None if cast is None else v.to(cast, copy=True)
+        return norm(v, w_pre, b_pre).to(dtype or w_pre.dtype)
     H = x.shape[1]
     n = x.shape[0] if row_index is None else row_index.shape[0]
-    w = w_pre if w_pre is not None else w_post
-    a = rows(n, H, w.dtype, x.device) if w_pre is not None else None
+    w = next(t for t in (w_pre, w_post, table) if t is not None)
+    a = rows(n, H, w.dtype if w_pre is not None else cast, x.device) if w_pre is not None or cast is not None else None
+    assert kind in ("rms", "layer") and (a is None or a.dtype == w.dtype)
     check(_lib.lib().tfb_res_norm(ptr(ids), ptr(table), table.stride(0) if table is not None else 0, float(scale),
                                   table.shape[0] if table is not None else 0, x.data_ptr(), x.stride(0), ptr(y),
-                                  y.stride(0) if y is not None else 0, ptr(w_post), ptr(w_pre), ptr(a), a.stride(0) if a is not None else 0,
-                                  ptr(row_index), n, H, float(eps), _f32(w), stream()), "res_norm")
+                                  y.stride(0) if y is not None else 0, ptr(w_post), ptr(b_post), ptr(scale_post), ptr(w_pre), ptr(b_pre), ptr(a),
+                                  a.stride(0) if a is not None else 0, ptr(row_index), n, H, float(eps), int(kind == "layer"), _f32(w), stream()),
+          "res_norm")
     return a
 
 
@@ -204,6 +243,96 @@ def diff_decode(q, kpool, vpool, block_table, positions, H, G, D, V, window, sca
                             block_table.shape[1], PAGE, positions.data_ptr(), o.data_ptr(), o.stride(0), ptr(acc), ptr(ml), splits or 1, B, H, G,
                             D, V, window, float(scale), float(lam), float(out_scale), float(eps), f32, _lib.status_word(q.device).data_ptr(),
                             stream()), "diff_decode", 2 if acc is not None else 1)
+    return o
+
+
+# ---------------------------------------------------------------------------------------------------- latent attention
+def latent_append(c, w, eps, slots, pool, want_rows=True):
+    """Rows c [T, R] divided by their root mean square and weighted with w, written to flat slots of ``pool`` [slots, R padded to 8]
+    (negative slots are not cached; ``slots`` None: nothing is).  Returns the rows, or None without ``want_rows``."""
+    T, R = c.shape
+    if not c.is_cuda:
+        cf = c.float()
+        v = (cf / torch.sqrt(cf.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(c.dtype)
+        if slots is not None:
+            keep = slots >= 0
+            pool[slots[keep], :R] = v[keep]
+        return v
+    out = rows(T, R, c.dtype, c.device) if want_rows else None
+    check(_lib.lib().tfb_latent_append(c.data_ptr(), c.stride(0), w.data_ptr(), float(eps), ptr(slots), ptr(out), out.stride(0) if want_rows else 0,
+                                       pool.data_ptr(), pool.shape[0], pool.shape[1], T, R, _f32(c), stream()), "latent_append")
+    return out
+
+
+def head_linear(x, w, heads, k, n, gate=None, transposed=False):
+    """One small product per head: x [M, heads * k] with w of heads blocks [n, k] ([k, n] when ``transposed``) stacked on the rows
+    -> [M, heads * n8] where n8 is n for plain and n rounded up to 8 (zero filled) for transposed blocks; ``gate`` [M, heads]: head h
+    is multiplied by sigmoid(gate[:, h])."""
+    M = x.shape[0]
+    n8 = (n + 7) // 8 * 8 if transposed else n
+    if not x.is_cuda:
+        W = w.float().reshape(heads, k, n).transpose(1, 2) if transposed else w.float().reshape(heads, n, k)
+        k_in = x.shape[1] // heads                       # rows of an earlier product may be padded
+        o = torch.einsum("mhk,hnk->mhn", x.float().reshape(M, heads, k_in)[..., :k], W)
+        if gate is not None:
+            o = o * torch.sigmoid(gate.float())[..., None]
+        out = torch.zeros((M, heads, n8), dtype=x.dtype)
+        out[..., :n] = o.to(x.dtype)
+        return out.view(M, heads * n8)
+    out = rows(M, heads * n8, x.dtype, x.device)
+    check(_lib.lib().tfb_head_linear(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), int(transposed), out.data_ptr(), out.stride(0), n8,
+                                     ptr(gate), gate.stride(0) if gate is not None else 0, M, heads, k, n, x.shape[1] // heads, _f32(x), stream()),
+          "head_linear")
+    return out
+
+
+def _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None):
+    R = H // G
+    Q = q.reshape(B, S, H, D).transpose(1, 2).float()
+    K = k.reshape(B, Skv, G, D).transpose(1, 2).float().repeat_interleave(R, 1)
+    W = v.reshape(B, Skv, G, V).transpose(1, 2).float().repeat_interleave(R, 1)
+    hide = torch.arange(Skv)[None] > torch.arange(S)[:, None] + (Skv - S)
+    o = (torch.softmax((Q @ K.transpose(-1, -2) * scale).masked_fill(hide, -math.inf), -1) @ W).transpose(1, 2)        # [B, S, H, V]
+    if gate is not None:
+        o = o * torch.sigmoid(gate.float()).reshape(B, S, H, 1)
+    return o.reshape(B * S, H * V).to(q.dtype)
+
+
+def head_attn(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None):
+    """Causal softmax attention of B prompts whose keys and values may have different sizes.  q [B*S, H D], k [B*Skv, G D],
+    v [B*Skv, G V]; the queries are the last S of the Skv positions; ``gate`` [B*S, H]: head h is multiplied by
+    sigmoid(gate[:, h]).  Returns [B*S, H V]."""
+    if not q.is_cuda:
+        return _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate)
+    o = rows(B * S, H * V, q.dtype, q.device)
+    check(_lib.lib().tfb_head_attn(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), o.data_ptr(), o.stride(0),
+                                   ptr(gate), gate.stride(0) if gate is not None else 0, B, S, Skv, H, G, D, V, float(scale), _f32(q),
+                                   _lib.status_word(q.device).data_ptr(), stream()), "head_attn")
+    return o
+
+
+def latent_decode(q, pool, block_table, positions, H, R, scale, splits: Optional[int] = None):
+    """One query per sequence and head over the cached latents, which are keys and values of every head at once: q [B, H * R8] (in the
+    latent space, R8 = R padded to 8 with zeros, at ``positions``), pool [slots, R8].  Returns softmax(scale q c) c, [B, H * R8]."""
+    B, W = q.shape[0], pool.shape[1]
+    if not q.is_cuda:
+        out = torch.zeros((B, H, W), dtype=q.dtype)
+        for b in range(B):
+            p = torch.arange(int(positions[b]) + 1)
+            c = pool[block_table[b, (p // PAGE).long()].long() * PAGE + p % PAGE].float()
+            out[b] = (torch.softmax(q[b].float().view(H, W) @ c.t() * scale, -1) @ c).to(q.dtype)
+        return out.view(B, H * W)
+    L, f32 = _lib.lib(), _f32(q)
+    o = rows(B, H * W, q.dtype, q.device)
+    acc = ml = None
+    s = L.tfb_latent_decode_plan(B, H, W, block_table.shape[1] * PAGE, f32)      # key splits of the tensor-core form, 0: the other form
+    if s:
+        s = splits or s
+        acc = torch.empty(B * H * s * W if s > 1 else 0, dtype=torch.float32, device=q.device)
+        ml = torch.empty(B * H * s * 2 if s > 1 else 0, dtype=torch.float32, device=q.device)
+    check(L.tfb_latent_decode(q.data_ptr(), q.stride(0), pool.data_ptr(), pool.shape[0], block_table.data_ptr(), block_table.shape[1], PAGE,
+                              positions.data_ptr(), o.data_ptr(), o.stride(0), ptr(acc), ptr(ml), s, B, H, R, W, float(scale), f32,
+                              _lib.status_word(q.device).data_ptr(), stream()), "latent_decode", 1 + int(s > 1))
     return o
 
 
