@@ -226,17 +226,25 @@ def torch_library_arm(cfg, world, rank, dev, local_batch, seq, steps, warmup, di
     return local_batch * world * seq * steps / (float(ms) / 1e3)
 
 
-def lanedra_serving_config(args):
-    """Prefill and decode throughput of Lanedra beside the dense decoder of equal layer sizes, on one GPU, random-init bf16 weights
-    and seeded token ids, through the serving engine's own passes (paged cache, state slots, decode CUDA graphs).  Two sizes:
-    2048 wide (24 layers) and 4096 wide (8 layers of the 32-layer shape).  Device-timed (CUDA events around K steps, W untimed ones
-    first); each step reads the weights (larger than L2).  One JSON line; ``rows`` has every measurement."""
+SERVING = {   # --config -> [(preset, layers), ...] (the first one's decode rate is the metric)
+    "lanedra-serving": [("lanedra-1.5b", 24), ("dense-1.5b", 24), ("lanedra-8b", 8), ("llama-3-8b", 8)],
+    "tekenex-serving": [("tekenex-7b", 24), ("mixture-7b", 24), ("tekenex-8x7b", 8), ("mixtral-8x7b", 8)],
+}
+
+
+def serving_config(args):
+    """Prefill and decode throughput of a stack model beside the closest model of the framework at equal layer sizes (Lanedra: the dense
+    decoder; Tekenex: the mixture-of-experts decoder), on one GPU, random-init bf16 weights and seeded token ids, through the
+    serving engine's own passes (paged cache, state slots, decode CUDA graphs).  Two sizes: 2048 wide (24 layers) and 4096 wide
+    (8 layers of the 32-layer shape).  Device-timed (CUDA events around K steps, W untimed ones first); each step reads the weights
+    (larger than L2).  One JSON line; ``rows`` has every measurement."""
     import torch
 
     from transformers_fusion_b200.inference.engine import EngineConfig, InferenceEngine, Request
     from transformers_fusion_b200.models.config import preset
     from transformers_fusion_b200.models.dense import DenseModel
-    from transformers_fusion_b200.models.lanedra import LanedraModel
+    from transformers_fusion_b200.models.moe import MoEModel
+    from transformers_fusion_b200.models.registry import model_class
     from transformers_fusion_b200.ops import _lib
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
@@ -260,63 +268,67 @@ def lanedra_serving_config(args):
         torch.cuda.synchronize()
         return e0.elapsed_time(e1) / steps
 
-    for ours, dense, layers in (("lanedra-1.5b", "dense-1.5b", 24), ("lanedra-8b", "llama-3-8b", 8)):
-        for name in (ours, dense):
-            cfg = preset(name)
-            if hasattr(cfg, "layers"):
-                cfg.layers = cfg.layers[:layers]
-            else:
-                cfg.num_layers = layers
-                cfg.max_seq_len = max(cfg.max_seq_len, 16384)
-            model = (LanedraModel if hasattr(cfg, "layers") else DenseModel)(cfg, device=dev, dtype=torch.bfloat16, seed=None)
-            with torch.no_grad():
-                gen = torch.Generator(device=dev).manual_seed(0)
-                for p in model.parameters():
-                    if p.dim() >= 2:
-                        p.normal_(0, p.shape[1] ** -0.5, generator=gen)
-                if hasattr(model, "finalize"):
-                    model.finalize()
-            row = {"model": name, "layers": layers, "params": sum(p.numel() for p in model.parameters())}
-            for B, S in prompts:
-                eng = InferenceEngine(model, None, EngineConfig(max_batch=B, num_pages=B * ((S + 15) // 16) + 8, max_seq_len=S + 16,
-                                                                enable_prefix_cache=False))
-                reqs = [Request(torch.randint(0, cfg.vocab_size, (S,), generator=g).tolist()) for _ in range(B)]
-                for r in reqs:
-                    eng._reserve(r, S)
+    for name, layers in SERVING[args.config]:
+        cfg = preset(name)
+        if hasattr(cfg, "layers"):
+            cfg.layers = cfg.layers[:layers]
+        else:
+            cfg.num_layers = layers
+            cfg.max_seq_len = max(cfg.max_seq_len, 16384)
+            if hasattr(cfg, "expert_fp8"):
+                cfg.expert_fp8 = False
+        cls = model_class(cfg.architecture) if hasattr(cfg, "architecture") else MoEModel if hasattr(cfg, "num_experts") else DenseModel
+        model = cls(cfg, device=dev, dtype=torch.bfloat16, seed=None)
+        with torch.no_grad():
+            gen = torch.Generator(device=dev).manual_seed(0)
+            for p in model.parameters():
+                if p.dim() >= 2:
+                    p.normal_(0, p.shape[-1] ** -0.5, generator=gen)
+                elif getattr(getattr(cls, "layer_cls", None), "norm_kind", "") == "layer":
+                    p.fill_(1.0)               # norms and scales whose stored weight is the factor itself
+            if hasattr(model, "finalize"):
+                model.finalize()
+        row = {"model": name, "layers": layers, "params": sum(p.numel() for p in model.parameters())}
+        for B, S in prompts:
+            eng = InferenceEngine(model, None, EngineConfig(max_batch=B, num_pages=B * ((S + 15) // 16) + 8, max_seq_len=S + 16,
+                                                            enable_prefix_cache=False))
+            reqs = [Request(torch.randint(0, cfg.vocab_size, (S,), generator=g).tolist()) for _ in range(B)]
+            for r in reqs:
+                eng._reserve(r, S)
 
-                @torch.no_grad()
-                def prefill(i):
-                    eng._logits(eng._layers_prefill_batch(reqs) if B > 1 else eng._layers_prefill(reqs[0].tokens, 0, reqs[0]))
-                ms = timed(prefill, max(3, K // 4))
-                row[f"prefill_{B}x{S}_tok_s"] = round(B * S / ms * 1e3)
-                row[f"prefill_{B}x{S}_ms"] = round(ms, 3)
-                del eng
-            for B, ctx in decodes:
-                n = ctx + W + K + 8
-                eng = InferenceEngine(model, None, EngineConfig(max_batch=B, num_pages=B * ((n + 15) // 16) + 8, max_seq_len=n + 16,
-                                                                enable_prefix_cache=False))
-                reqs = [Request([]) for _ in range(B)]
-                for lo in range(0, B, 8):
-                    eng.feed([(r, torch.randint(0, cfg.vocab_size, (ctx,), generator=g).tolist(), []) for r in reqs[lo:lo + 8]])
-                tok = torch.randint(0, cfg.vocab_size, (W + K, B), generator=g).tolist()
+            @torch.no_grad()
+            def prefill(i):
+                eng._logits(eng._layers_prefill_batch(reqs) if B > 1 else eng._layers_prefill(reqs[0].tokens, 0, reqs[0]))
+            ms = timed(prefill, max(3, K // 4))
+            row[f"prefill_{B}x{S}_tok_s"] = round(B * S / ms * 1e3)
+            row[f"prefill_{B}x{S}_ms"] = round(ms, 3)
+            del eng
+        for B, ctx in decodes:
+            n = ctx + W + K + 8
+            eng = InferenceEngine(model, None, EngineConfig(max_batch=B, num_pages=B * ((n + 15) // 16) + 8, max_seq_len=n + 16,
+                                                            enable_prefix_cache=False))
+            reqs = [Request([]) for _ in range(B)]
+            for lo in range(0, B, 8):
+                eng.feed([(r, torch.randint(0, cfg.vocab_size, (ctx,), generator=g).tolist(), []) for r in reqs[lo:lo + 8]])
+            tok = torch.randint(0, cfg.vocab_size, (W + K, B), generator=g).tolist()
 
-                @torch.no_grad()
-                def decode(i):
-                    eng._decode_logits(reqs, tok[i])
-                ms = timed(decode, K)
-                row[f"decode_{B}x{ctx}_tok_s"] = round(B / ms * 1e3)
-                row[f"decode_{B}x{ctx}_ms"] = round(ms, 3)
-                del eng
-            _lib.check_status(dev)
-            rows.append(row)
-            del model
-            torch.cuda.empty_cache()
+            @torch.no_grad()
+            def decode(i):
+                eng._decode_logits(reqs, tok[i])
+            ms = timed(decode, K)
+            row[f"decode_{B}x{ctx}_tok_s"] = round(B / ms * 1e3)
+            row[f"decode_{B}x{ctx}_ms"] = round(ms, 3)
+            del eng
+        _lib.check_status(dev)
+        rows.append(row)
+        del model
+        torch.cuda.empty_cache()
     clocks = sampler.stop()
     best = rows[0]["decode_64x2048_tok_s"]
     print(json.dumps({"metric": "decode_tokens_per_s", "value": best, "unit": "tokens/s", "n_gpus": 1, "steps": K, "warmup": W,
                       "ms_per_step": rows[0]["decode_64x2048_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16",
                       "data": "synthetic (seeded token ids; random-init weights)",
-                      "config": {"model": "lanedra-1.5b (24L d2048)", "global_batch": 64, "seq_len": 2048, "parallelism": "none",
+                      "config": {"model": f"{rows[0]['model']} (24L d2048)", "global_batch": 64, "seq_len": 2048, "parallelism": "none",
                                  "l2": "weights larger than L2"}, "clocks": clocks, "gpu_launches": _lib.LAUNCHES[0], "rows": rows}))
     return 0
 
@@ -327,12 +339,13 @@ def main(argv=None):
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference", "nccl"])
-    ap.add_argument("--config", default="llama-50m-zero2", choices=["llama-50m-zero2", "llama3-8b-fsdp-tp2", "mixtral-8x7b-ep", "gpt2-small-cpu", "lanedra-serving"],
+    ap.add_argument("--config", default="llama-50m-zero2", choices=["llama-50m-zero2", "llama3-8b-fsdp-tp2", "mixtral-8x7b-ep", "gpt2-small-cpu", *SERVING],
                     help="llama-50m-zero2: ~50M Llama, ZeRO-2 data parallel, seq 1024, global batch 64 (the default; runs on "
                          "1/2/4/8 GPUs).  llama3-8b-fsdp-tp2: Llama-3-8B shape, ZeRO-3 over dp x tensor parallel 2, seq 4096, "
                          "one sequence per GPU (2, 4 or 8 GPUs).  gpt2-small-cpu: GPT-2-small-shaped greedy generation on the CPU "
-                         "(32 prompt + 64 new tokens), the configuration the reference's own build can run as well.  lanedra-serving: prefill and "
-                         "decode throughput of Lanedra beside the dense decoder of equal sizes (1 GPU)")
+                         "(32 prompt + 64 new tokens), the configuration the reference's own build can run as well.  lanedra-serving, "
+                         "tekenex-serving: prefill and decode throughput of the stack model beside the dense / mixture-of-experts decoder of "
+                         "equal sizes (1 GPU)")
     ap.add_argument("--capacity-factor", type=float, default=2.0,
                     help="mixtral-8x7b-ep: expert buffer rows per rank as a multiple of the balanced load")
     ap.add_argument("--no-graph", action="store_true", help="launch kernels eagerly instead of replaying a CUDA graph")
@@ -354,8 +367,8 @@ def main(argv=None):
         return cpu_inference_config(args)
     if args.impl == "reference":
         return reference_arm(args)
-    if args.config == "lanedra-serving":
-        return lanedra_serving_config(args)
+    if args.config in SERVING:
+        return serving_config(args)
     if args.config == "llama3-8b-fsdp-tp2":
         return main_sharded(args)
     if args.config == "mixtral-8x7b-ep":

@@ -6,7 +6,9 @@ fraction of the copy / GEMM peaks when ``--peaks <json>`` (keys hbm_gbs, bf16_tf
 Kernels: gemm, gemm_nt_wgrad, gemm_fp8, attention_fwd, attention_bwd, rmsnorm, rmsnorm_bwd, swiglu, rope,
 cross_entropy, adamw, paged_decode, sampling, moe_ffn; those of stack models (``STACK_KERNELS``): diff_attention,
 diff_attention_window, attention_fwd_gqa128 (the plain form of the same layer), diff_decode, delta_prep, delta_scan,
-delta_scan_one, gated_norm, delta_prep_step, delta_step, res_norm, glu_silu, rope_append.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
+delta_scan_one, gated_norm, delta_prep_step, delta_step, res_norm, glu_silu, rope_append; those of latent attention and the serving
+mixture with the like kernels of the mixture-of-experts decoder (``LATENT_KERNELS``).  ``--kernel all | stack | latent`` or names
+with commas between them.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
 against their NCCL forms (cli/bench_comm.py)."""
 from __future__ import annotations
 
@@ -22,6 +24,10 @@ KERNELS = ("gemm", "gemm_wgrad", "gemm_fp8", "attention_fwd", "attention_bwd", "
            "cross_entropy", "adamw", "paged_decode", "sampling", "moe_ffn")
 STACK_KERNELS = ("diff_attention", "diff_attention_window", "attention_fwd_gqa128", "diff_decode", "delta_prep", "delta_scan", "delta_scan_one",
                  "gated_norm", "delta_prep_step", "delta_step", "res_norm", "glu_silu", "rope_append")
+LATENT_KERNELS = ("head_attn", "attention_fwd_mha128", "latent_decode", "latent_decode_32", "latent_append", "latent_append_step", "head_linear_q",
+                  "head_linear_v", "output_norm", "layernorm", "linear_relu2", "linear_relu2_step", "route", "route_step", "router_topk", "expert_rows",
+                  "moe_permute", "expert_gate_up", "expert_gate_up_step", "expert_down", "expert_down_step", "expert_glu", "expert_glu_step",
+                  "weighted_sum", "moe_combine", "mixture", "mixture_step", "moe_ffn_step", "kv_append")
 FP32_FMA_PER_SM = 128          # fp32 FMA lanes of an SM (delta_scan is reported against them as well)
 
 
@@ -92,12 +98,112 @@ def _build_stack(kernel, n, dev):
     raise SystemExit(f"Error: unknown kernel '{kernel}'")
 
 
+def _build_latent(kernel, n, dev):
+    """The same for the kernels of latent attention and of the serving mixture, beside the like ones of the mixture-of-experts
+    decoder (attention_fwd_mha128, layernorm, router_topk, moe_permute, moe_combine, moe_ffn_step, kv_append): 2048 wide, 16 heads of
+    128 over latents of 512, 64 experts of 704, six per token.  ``n``: tokens per sequence (prompts; 16 k tokens in all) or
+    cached tokens (decoding); *_step: 64 rows."""
+    import torch
+
+    from ..ops import functional as F
+    from ..ops import moe as M
+    from ..ops import stack as K
+    bf = torch.bfloat16
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s, dtype=bf, scale=1.0: (torch.randn(*s, device=dev, generator=g) * scale).to(dtype)
+    Hd, H, D, R, E, k, Fh = 2048, 16, 128, 512, 64, 6, 704
+    T = 64 if kernel.endswith("_step") or kernel.startswith("head_linear") else 1 << 14
+    if kernel in ("head_attn", "attention_fwd_mha128"):
+        B = max(1, T // n)
+        q, kv, fl = rnd(B * n, H * D + H), rnd(B * n, 2 * H * D), 4.0 * B * H * n * n / 2 * D
+        if kernel == "head_attn":
+            return (lambda: K.head_attn(q[:, :H * D], kv[:, :H * D], kv[:, H * D:], B, n, n, H, H, D, D, D ** -0.5, q[:, H * D:])), fl, B * n * 4 * H * D * 2
+        return (lambda: F.attn_fwd(q, kv, kv, B, n, H, H, D, q_col0=0, k_col0=0, v_col0=H * D)), fl, B * n * 4 * H * D * 2
+    if kernel in ("latent_decode", "latent_decode_32"):
+        B, H = 64, 32 if kernel.endswith("32") else 16
+        pages = B * (n // 16)
+        pool, q = rnd(pages * 16, R), rnd(B, H * R)
+        bt = torch.randperm(pages, device=dev, generator=g).int().view(B, -1).contiguous()
+        pos = torch.full((B,), n - 1, dtype=torch.int32, device=dev)
+        return (lambda: K.latent_decode(q, pool, bt, pos, H, R, D ** -0.5)), 4.0 * B * H * n * R, B * n * R * 2
+    if kernel.startswith("latent_append") or kernel == "kv_append":
+        slots = torch.randperm(T, device=dev, generator=g)
+        if kernel == "kv_append":
+            from ..inference.kv_cache import PagedKVCache
+            kv, qkv = PagedKVCache(1, T // 16, 4, 128, "bf16", dev), rnd(T, 24 * 128)
+            return (lambda: kv.append(0, qkv, 16 * 128, 20 * 128, slots)), 0.0, T * 8 * 128 * 4
+        p, w, pool = rnd(T, H * D + R + H), rnd(R), rnd(T, R)
+        step = kernel.endswith("_step")
+        return (lambda: K.latent_append(p[:, H * D:H * D + R], w, 1e-5, slots, pool, want_rows=not step)), 0.0, T * R * (4 if step else 6)
+    if kernel.startswith("head_linear"):
+        x, w, gate = rnd(T, H * (D if kernel.endswith("q") else R)), rnd(H * D, R), rnd(T, H)
+        fn = (lambda: K.head_linear(x, w, H, D, R, transposed=True)) if kernel.endswith("q") else (lambda: K.head_linear(x, w, H, R, D, gate=gate))
+        return fn, 2.0 * T * H * D * R, (w.numel() + T * H * (D + R)) * 2
+    if kernel in ("output_norm", "layernorm"):
+        x, y, w, b = rnd(T, Hd, dtype=torch.float32), rnd(T, Hd), rnd(Hd), rnd(Hd)
+        if kernel == "layernorm":
+            return (lambda: F.layernorm_fwd(y, w, b, 1e-5)), 0.0, T * Hd * 4
+        return (lambda: K.res_norm(x, 1e-5, y=y, w_post=w, b_post=b, scale_post=w, cast=bf, kind="layer")), 0.0, T * Hd * 12
+    if kernel.startswith("linear_relu2"):
+        N = 8448
+        x, w = rnd(T, Hd), rnd(N, Hd, scale=Hd ** -0.5)
+        return (lambda: K.linear(x, w, act="relu2")), 2.0 * T * N * Hd, (w.numel() + T * (N + Hd)) * 2
+    h, z, bias = rnd(T, Hd), rnd(T, E, dtype=torch.float32), rnd(E)
+    if kernel.startswith("route_") or kernel == "route":
+        return (lambda: M.route(z, bias, k)), 0.0, T * (E * 4 + k * 12)
+    if kernel == "router_topk":
+        def old():
+            idx, _, _, counts, _ = M.router_topk(z, k)
+            return M.Plan(idx, counts, E)
+        return old, 0.0, T * (E * 8 + k * 8)
+    r = M.route(z, bias, k)
+    if kernel in ("moe_permute", "moe_combine"):
+        idx, w, _, counts, _ = M.router_topk(z, k)
+
+        def rows():
+            pl = M.Plan(idx, counts, E)
+            return pl, M.permute(h, idx, pl)
+        pl, xp = rows()
+        if kernel == "moe_permute":
+            return rows, 0.0, T * (k + 1) * Hd * 2
+        return (lambda: M.combine(xp, w, pl)), 0.0, T * (k + 1) * Hd * 2
+    if kernel == "expert_rows":
+        return (lambda: M.expert_rows(h, r)), 0.0, T * (k + 1) * Hd * 2
+    gu, dn = rnd(E, 2 * Fh, Hd, scale=Hd ** -0.5), rnd(E, Hd, Fh, scale=Fh ** -0.5)
+    xp, fl = M.expert_rows(h, r), 2.0 * T * k * 2 * Fh * Hd
+    y = M.expert_linear(xp, gu, r)
+    if kernel.startswith("expert_gate_up"):
+        return (lambda: M.expert_linear(xp, gu, r)), fl, (gu.numel() + T * k * (Hd + 2 * Fh)) * 2
+    a = M.expert_glu(y, r)
+    if kernel.startswith("expert_glu"):
+        return (lambda: M.expert_glu(y, r)), 0.0, T * k * Fh * 6
+    if kernel.startswith("expert_down"):
+        return (lambda: M.expert_linear(a, dn, r)), fl / 2, (dn.numel() + T * k * (Hd + Fh)) * 2
+    o = M.expert_linear(a, dn, r)
+    if kernel == "weighted_sum":
+        return (lambda: M.weighted_sum(o, r, h)), 0.0, T * (k + 2) * Hd * 2
+    wr, nbytes = rnd(E, Hd, scale=Hd ** -0.5), (gu.numel() + dn.numel() + 2 * T * Hd) * 2
+    if kernel in ("mixture", "mixture_step"):
+        def ours():
+            s = M.route(K.linear(h, wr, out_dtype=torch.float32), bias, k)
+            return M.weighted_sum(M.expert_linear(M.expert_glu(M.expert_linear(M.expert_rows(h, s), gu, s), s), dn, s), s)
+        return ours, 1.5 * fl, nbytes
+    if kernel == "moe_ffn_step":
+        def theirs():
+            with torch.no_grad():
+                return M.moe_ffn(h, F.gemm(h, wr, out_dtype=torch.float32), gu, dn, k, True, "silu", 0.0, 0.0)
+        return theirs, 1.5 * fl, nbytes
+    raise SystemExit(f"Error: unknown kernel '{kernel}'")
+
+
 def _build(kernel, n, dev, heads=0, shape=None):
     """Returns (callable, flops, bytes) for one launch of ``kernel`` at problem size ``n``."""
     import torch
 
     if kernel in STACK_KERNELS:
         return _build_stack(kernel, n, dev)
+    if kernel in LATENT_KERNELS:
+        return _build_latent(kernel, n, dev)
 
     from ..ops import functional as F
     bf = torch.bfloat16
@@ -420,7 +526,7 @@ def main(argv=None):
         if not torch.cuda.is_available():
             print("Error: kernel benchmarks need a CUDA device", file=sys.stderr)
             return 1
-        names = KERNELS if a.kernel == "all" else STACK_KERNELS if a.kernel == "stack" else [a.kernel]
+        names = {"all": KERNELS, "stack": STACK_KERNELS, "latent": LATENT_KERNELS}.get(a.kernel) or a.kernel.split(",")
         peaks = json.load(open(a.peaks)) if a.peaks else {}
         for name in names:
             shape = None

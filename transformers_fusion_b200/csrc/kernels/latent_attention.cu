@@ -5,8 +5,9 @@
 //   head_attn_fwd      prompts, bf16, tcgen05, over keys and values that a product has read out of the latents: one CTA per (sequence,
 //                      head, 256 queries) as two 128-query tiles that share every key / value tile and take turns on the
 //                      tensor core; keys and values may have different sizes; the gate is applied in the epilogue
-//   head_linear        one small product per head for the rows of a decode step (mma.sync): queries into the latent space
-//                      (q . W_uk c = (W_uk^T q) . c), and values out of the attention's result (sum_j a_j W_uv c_j = W_uv sum_j a_j c_j)
+//   head_linear        one small product per head for the rows of a decode step (mma.sync): queries into the latent space,
+//                      q . W_uk c = (W_uk^T q) . c; the values come out of the attention's result, sum_j a_j W_uv c_j =
+//                      W_uv sum_j a_j c_j, by the per-head form of skinny_linear.cu
 //   latent_decode      one query per sequence over the paged latents, bf16, mma.sync: the query heads are the rows of one or two 16-row
 //                      tiles, and the latents are keys and values of all of them, so a cached row is read once.  Split over
 //                      the keys; a second kernel merges the splits.
@@ -373,21 +374,19 @@ static int launch_head_attn(const void* q, long long ldq, const void* k, long lo
 }
 
 // ------------------------------------------------------------------------------------------------
-// one product per head for few rows: out[m, h * out_head + n] = sum_k x[m, h * x_head + k] W_h[n, k] (* sigmoid(gate[m, h]))
-// KN: the blocks of W are stored [K, N].  64 rows x 32 columns per block, the next 64-deep chunk in registers while one is used.
+// one product per head for few rows, weights stored [K, N]: out[m, h * out_head + n] = sum_k x[m, h * x_head + k] W_h[k, n].
+// 64 rows x 32 columns per block, the next 128-deep chunk in registers while one is used.
 // ------------------------------------------------------------------------------------------------
 struct HeadLinearArgs {
   const __nv_bfloat16 *x, *w;
   long long ldx, ldw;
   __nv_bfloat16* out;
   long long ldo;
-  const __nv_bfloat16* gate;
-  long long ldg;
   int M, N, K, x_head, out_head;     // columns N .. out_head of a head are written as zeros
   int vec_x, vec_w;                  // 16-byte loads are aligned
 };
 
-constexpr int HL_M = 64, HL_N = 32, HL_K = 64;
+constexpr int HL_M = 64, HL_N = 32, HL_K = 128;
 
 __device__ __forceinline__ uint4 load8(const __nv_bfloat16* p, int n, int vec) {   // n of 8 entries, the others zero
   if (n <= 0) return make_uint4(0u, 0u, 0u, 0u);
@@ -399,85 +398,77 @@ __device__ __forceinline__ uint4 load8(const __nv_bfloat16* p, int n, int vec) {
   return make_uint4(u[0], u[1], u[2], u[3]);
 }
 
-template <bool KN>
 __global__ void __launch_bounds__(128) head_linear_kernel(const HeadLinearArgs p) {
   tfb::pdl_sync();
-  constexpr int PA = HL_K * 2 + 16, PB = KN ? HL_N * 2 + 16 : HL_K * 2 + 16;        // byte pitches
-  constexpr int RB = KN ? HL_K : HL_N, CB = KN ? HL_N / 8 : HL_K / 8;               // rows and 16-byte pieces of the W chunk
-  __shared__ __align__(16) uint8_t sA[2][HL_M * PA];
-  __shared__ __align__(16) uint8_t sB[2][RB * PB];
+  constexpr int PA = HL_K * 2 + 16, PB = HL_N * 2 + 16;                              // byte pitches
+  constexpr int CA = HL_K / 8, CB = HL_N / 8;                                        // 16-byte pieces of a row
+  constexpr int NA = HL_M * CA / 128, NB = HL_K * CB / 128;
+  __shared__ __align__(16) uint8_t sA[HL_M * PA];
+  __shared__ __align__(16) uint8_t sB[HL_K * PB];
   const int n0 = blockIdx.x * HL_N, h = blockIdx.y, m0 = blockIdx.z * HL_M;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const __nv_bfloat16* x = p.x + (long long)h * p.x_head;
-  const __nv_bfloat16* w = p.w + (long long)h * (KN ? p.K : p.N) * p.ldw;
-  uint4 ra[4], rb[2];
+  const __nv_bfloat16* w = p.w + (long long)h * p.K * p.ldw;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  uint4 ra[NA], rb[NB];
   auto fetch = [&](int k0) {
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int e = tid + i * 128, r = e >> 3, c = (e & 7) * 8;
-      ra[i] = m0 + r < p.M ? load8(x + (m0 + r) * p.ldx + k0 + c, p.K - k0 - c, p.vec_x) : make_uint4(0u, 0u, 0u, 0u);
-    }
-#pragma unroll
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < NB; ++i) {
       const int e = tid + i * 128, r = e / CB, c = (e % CB) * 8;
-      if (KN) rb[i] = k0 + r < p.K ? load8(w + (k0 + r) * p.ldw + n0 + c, p.N - n0 - c, p.vec_w) : make_uint4(0u, 0u, 0u, 0u);
-      else rb[i] = n0 + r < p.N ? load8(w + (n0 + r) * p.ldw + k0 + c, p.K - k0 - c, p.vec_w) : make_uint4(0u, 0u, 0u, 0u);
-    }
-  };
-  auto put = [&](int s) {
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int e = tid + i * 128;
-      *reinterpret_cast<uint4*>(sA[s] + (e >> 3) * PA + (e & 7) * 16) = ra[i];
+      rb[i] = k0 + r < p.K ? load8(w + (k0 + r) * p.ldw + n0 + c, p.N - n0 - c, p.vec_w) : zero;
     }
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int e = tid + i * 128;
-      *reinterpret_cast<uint4*>(sB[s] + (e / CB) * PB + (e % CB) * 16) = rb[i];
+    for (int i = 0; i < NA; ++i) {
+      const int e = tid + i * 128, r = e / CA, c = (e % CA) * 8;
+      ra[i] = m0 + r < p.M ? load8(x + (m0 + r) * p.ldx + k0 + c, p.K - k0 - c, p.vec_x) : zero;
     }
   };
   float acc[4][4];
 #pragma unroll
   for (int n = 0; n < 4; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
   fetch(0);
-  put(0);
-  __syncthreads();
-  int s = 0;
-  for (int k0 = 0; k0 < p.K; k0 += HL_K, s ^= 1) {
+  for (int k0 = 0; k0 < p.K; k0 += HL_K) {
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < NA; ++i) {
+      const int e = tid + i * 128;
+      *reinterpret_cast<uint4*>(sA + (e / CA) * PA + (e % CA) * 16) = ra[i];
+    }
+#pragma unroll
+    for (int i = 0; i < NB; ++i) {
+      const int e = tid + i * 128;
+      *reinterpret_cast<uint4*>(sB + (e / CB) * PB + (e % CB) * 16) = rb[i];
+    }
+    __syncthreads();
     if (k0 + HL_K < p.K) fetch(k0 + HL_K);
-    if (m0 + warp * 16 < p.M) {
-      const uint32_t a0 = smem_u32(sA[s]) + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PA + (lane >> 4) * 16;
-      const uint32_t b0 = KN ? smem_u32(sB[s]) + ((lane & 7) + ((lane >> 3) & 1) * 8) * PB + (lane >> 4) * 16
-                             : smem_u32(sB[s]) + ((lane & 7) + (lane >> 4) * 8) * PB + ((lane >> 3) & 1) * 16;
+    if (m0 + warp * 16 >= p.M) continue;
+    const uint32_t a0 = smem_u32(sA) + (warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * PA + (lane >> 4) * 16;
+    const uint32_t b0 = smem_u32(sB) + ((lane & 7) + ((lane >> 3) & 1) * 8) * PB + (lane >> 4) * 16;
 #pragma unroll
-      for (int ks = 0; ks < HL_K / 16; ++ks) {
-        uint32_t a[4];
-        ldsm(a0 + ks * 32, a);
+    for (int ks = 0; ks < HL_K / 16; ++ks) {
+      if (k0 + ks * 16 >= p.K) break;
+      uint32_t a[4];
+      ldsm(a0 + ks * 32, a);
 #pragma unroll
-        for (int nb = 0; nb < 2; ++nb) {
-          uint32_t b[4];
-          if (KN) ldsm_t(b0 + ks * 16 * PB + nb * 32, b);
-          else ldsm(b0 + nb * 16 * PB + ks * 32, b);
-          mma_bf16(acc[2 * nb], a, b[0], b[1]);
-          mma_bf16(acc[2 * nb + 1], a, b[2], b[3]);
-        }
+      for (int nb = 0; nb < 2; ++nb) {
+        uint32_t b[4];
+        ldsm_t(b0 + ks * 16 * PB + nb * 32, b);
+        mma_bf16(acc[2 * nb], a, b[0], b[1]);
+        mma_bf16(acc[2 * nb + 1], a, b[2], b[3]);
       }
     }
-    if (k0 + HL_K < p.K) put(s ^ 1);
-    __syncthreads();
   }
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int m = m0 + warp * 16 + (lane >> 2) + 8 * i;
     if (m >= p.M) continue;
-    const float f = p.gate ? sigmoid_exact(__bfloat162float(p.gate[m * p.ldg + h])) : 1.f;
     __nv_bfloat16* o = p.out + m * p.ldo + (long long)h * p.out_head;
 #pragma unroll
     for (int n = 0; n < 4; ++n)
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int col = n0 + n * 8 + (lane & 3) * 2 + e;
-        if (col < p.out_head) o[col] = __float2bfloat16(acc[n][2 * i + e] * f);
+        if (col < p.out_head) o[col] = __float2bfloat16(acc[n][2 * i + e]);
       }
   }
 }
@@ -502,7 +493,7 @@ struct LatentDecodeArgs {
 };
 
 constexpr int LD_THREADS = 256;
-constexpr int LD_KEYS = 64;
+constexpr int LD_KEYS = 64, LD_HALF = 32;      // keys of a step; keys of a ring slot
 
 // RC: columns of a latent in shared memory (zeros past W); MT: 16-row tiles of query heads.  Of the eight warps, two share the keys
 // and four the columns in the scores (the partial scores meet in shared memory); each takes an eighth of the columns in the
@@ -510,22 +501,22 @@ constexpr int LD_KEYS = 64;
 template <int RC, int MT>
 struct LatentSmem {
   static constexpr int RP = RC * 2 + 16;                 // byte pitch of a row: ldmatrix reads eight rows without bank conflicts
-  static constexpr int TILE = LD_KEYS * RP;
-  static constexpr int SP = LD_KEYS + 4;                 // floats of a score row
+  static constexpr int SLOT = LD_HALF * RP;
+  static constexpr int SP = LD_KEYS + 8;                 // floats of a score row
   static constexpr int PP = LD_KEYS * 2 + 16;            // bytes of a weight row
   static constexpr int S_BYTES = 4 * MT * 16 * SP * 4, P_BYTES = MT * 16 * PP, A_BYTES = MT * 16 * 8;
-  static constexpr int REST = S_BYTES + P_BYTES + A_BYTES + 64;
-  static constexpr int FIT = (226 * 1024 - REST) / TILE;
-  static constexpr int ST = FIT > 4 ? 4 : FIT;
-  static constexpr int S_OFF = ST * TILE, P_OFF = S_OFF + S_BYTES, A_OFF = P_OFF + P_BYTES, BAR_OFF = A_OFF + A_BYTES;
-  static constexpr int TOTAL = BAR_OFF + 64;
-  static_assert(ST >= 2, "two stages at least");
+  static constexpr int REST = S_BYTES + P_BYTES + A_BYTES + 128;
+  static constexpr int FIT = (226 * 1024 - REST) / SLOT;
+  static constexpr int NS = FIT > 8 ? 8 : FIT;           // ring slots
+  static constexpr int S_OFF = NS * SLOT, P_OFF = S_OFF + S_BYTES, A_OFF = P_OFF + P_BYTES, BAR_OFF = A_OFF + A_BYTES;
+  static constexpr int TOTAL = BAR_OFF + 128;
+  static_assert(NS >= 4, "two steps at least");
 };
 
 template <int RC, int MT>
 __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const LatentDecodeArgs p) {
   using L = LatentSmem<RC, MT>;
-  constexpr int ST = L::ST, RP = L::RP, KS = RC / 64, NT = RC / 64;   // k steps of a warp's column quarter; 8-column blocks of its eighth
+  constexpr int NS = L::NS, RP = L::RP, KS = RC / 64, NT = RC / 64;   // k steps of a warp's column quarter; 8-column blocks of its eighth
   extern __shared__ __align__(128) uint8_t sm[];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int b = blockIdx.x, h0 = blockIdx.y * MT * 16, sp = blockIdx.z;
@@ -533,50 +524,13 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const Late
   const uint32_t s0 = smem_u32(sm), bars = s0 + L::BAR_OFF;
   float* sS = reinterpret_cast<float*>(sm + L::S_OFF);
   float* sAl = reinterpret_cast<float*>(sm + L::A_OFF);                // rescale of a row; at the end: its maximum, then its sum
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + L::BAR_OFF + 48);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + L::BAR_OFF + 64);
   if (tid == 0) {
-    for (int s = 0; s < ST; ++s) mbar_init(bars + s * 8, 1);
+    for (int s = 0; s < NS; ++s) mbar_init(bars + s * 8, 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
   tfb::pdl_sync();
-  const int n_keys = p.positions[b] + 1;
-  const int per = ((n_keys + p.splits - 1) / p.splits + LD_KEYS - 1) / LD_KEYS * LD_KEYS;
-  const int t_begin = sp * per, t_end = min(n_keys, t_begin + per);
-  const int nt = t_end > t_begin ? (t_end - t_begin + LD_KEYS - 1) / LD_KEYS : 0;
-  const int* bt = p.block_table + (long long)b * p.max_pages;
-  // what no copy writes but the products read: columns past W, and the missing rows of a last tile that is a stage's first
-  if (p.W < RC) {
-    const int pieces = (RC - p.W) / 8;
-    for (int i = tid; i < ST * LD_KEYS * pieces; i += LD_THREADS)
-      *reinterpret_cast<uint4*>(sm + (i / pieces) * RP + p.W * 2 + (i % pieces) * 16) = make_uint4(0u, 0u, 0u, 0u);
-  }
-  if (nt > 0 && nt <= ST) {
-    const int first = t_end - t_begin - (nt - 1) * LD_KEYS;           // rows of the last tile
-    uint8_t* base = sm + (nt - 1) * L::TILE + first * RP;
-    for (int i = tid; i < (LD_KEYS - first) * (RP / 16); i += LD_THREADS) reinterpret_cast<uint4*>(base)[i] = make_uint4(0u, 0u, 0u, 0u);
-  }
-  fence_proxy_async_smem();
-  __syncthreads();
-
-  // lanes 0-7 of warp w bring rows 8 w .. 8 w + 7 of a tile
-  const int my_row = warp * 8 + lane;
-  auto page_of = [&](int j) -> long long {
-    const int t = t_begin + j * LD_KEYS + my_row;
-    long long page = (lane < 8 && j < nt && t < t_end) ? bt[t / p.page] : 0;
-    TFB_BOUNDS(page >= 0 && (page + 1) * p.page <= p.nslots, 52, page, p.nslots / p.page);
-    if (page < 0 || (page + 1) * p.page > p.nslots) page = 0;
-    return page;
-  };
-  auto issue = [&](int j, long long page) {
-    const int t0 = t_begin + j * LD_KEYS, rows = min(LD_KEYS, t_end - t0), st = j % ST;
-    if (tid == 0) mbar_expect_tx(bars + st * 8, uint32_t(rows) * p.W * 2);
-    if (lane < 8 && my_row < rows)
-      bulk_load(s0 + st * L::TILE + my_row * RP, p.pool + (page * p.page + (t0 + my_row) % p.page) * p.W, p.W * 2, bars + st * 8);
-  };
-  for (int j = 0; j < ST - 1 && j < nt; ++j) issue(j, page_of(j));
-  long long page_next = page_of(ST - 1);
-
   uint32_t qa[MT][KS][4];                                              // this warp's columns of the queries
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -587,6 +541,44 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const Late
         const int h = h0 + m * 16 + (lane >> 2) + (e & 1) * 8, c = rg * (RC / 4) + k * 16 + (lane & 3) * 2 + (e >> 1) * 8;
         qa[m][k][e] = (h < p.H && c < p.W) ? *reinterpret_cast<const uint32_t*>(p.q + b * p.ldq + (long long)h * p.W + c) : 0u;
       }
+  const int n_keys = p.positions[b] + 1;
+  const int per = ((n_keys + p.splits - 1) / p.splits + LD_KEYS - 1) / LD_KEYS * LD_KEYS;
+  const int t_begin = sp * per, count = max(0, min(n_keys, t_begin + per) - t_begin);
+  const int nt = (count + LD_KEYS - 1) / LD_KEYS, nh = (count + LD_HALF - 1) / LD_HALF;
+  // what no copy writes but the products read: columns past W, and rows past the end in a slot that no earlier rows have filled
+  if (p.W < RC) {
+    const int pieces = (RC - p.W) / 8;
+    for (int i = tid; i < NS * LD_HALF * pieces; i += LD_THREADS)
+      *reinterpret_cast<uint4*>(sm + (i / pieces) * RP + p.W * 2 + (i % pieces) * 16) = make_uint4(0u, 0u, 0u, 0u);
+  }
+  {
+    const int from = min(count, NS * LD_HALF), to = min(nt * LD_KEYS, NS * LD_HALF);
+    for (int i = tid; i < (to - from) * (RP / 16); i += LD_THREADS) reinterpret_cast<uint4*>(sm + from * RP)[i] = make_uint4(0u, 0u, 0u, 0u);
+  }
+  fence_proxy_async_smem();
+  __syncthreads();
+
+  // lanes 0-7 of warp w bring rows 4 w .. 4 w + 3 of two halves; pages divide a half (checked by the caller), so a row's place in its
+  // page never changes
+  const int my_row = warp * 4 + (lane & 3), my_half = lane >> 2, in_page = my_row % p.page;
+  const int* bt = p.block_table + (long long)b * p.max_pages + (t_begin + my_row) / p.page;
+  const int pages_half = LD_HALF / p.page;
+  auto page_of = [&](int h) { return (lane < 8 && h < nh && h * LD_HALF + my_row < count) ? bt[h * pages_half] : 0; };
+  auto issue = [&](int h, long long page) {                            // h: this lane's half
+    if (lane >= 8 || h >= nh) return;
+    const int rows = min(LD_HALF, count - h * LD_HALF), slot = h % NS;
+    if (warp == 0 && (lane & 3) == 0) mbar_expect_tx(bars + slot * 8, uint32_t(rows) * p.W * 2);
+    if (my_row < rows) {
+      TFB_BOUNDS(page >= 0 && (page + 1) * p.page <= p.nslots, 52, page, p.nslots / p.page);
+      if (page < 0 || (page + 1) * p.page > p.nslots) page = 0;
+      bulk_load(s0 + slot * L::SLOT + my_row * RP, p.pool + (page * p.page + in_page) * p.W, p.W * 2, bars + slot * 8);
+    }
+  };
+#pragma unroll
+  for (int h = 0; h < NS; h += 2)
+    if (h + my_half < NS) issue(h + my_half, page_of(h + my_half));
+  int page_next = page_of(NS + my_half);
+
   float o[MT][NT][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -598,45 +590,88 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const Late
   const float sl2 = p.scale * LOG2E;
   bool ok = true;
 
-  for (int j = 0; j < nt; ++j) {
-    const uint32_t tile = s0 + (j % ST) * L::TILE;
-    if (ok && !mbar_wait_warp(bars + (j % ST) * 8, (j / ST) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) ok = false;
-    // scores of 32 keys over a quarter of the columns
-    float sc[MT][4][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int n = 0; n < 4; ++n) sc[m][n][0] = sc[m][n][1] = sc[m][n][2] = sc[m][n][3] = 0.f;
-    const uint32_t krow = tile + (kg * 32 + (lane & 7) + (lane >> 4) * 8) * RP + rg * (RC / 2) + ((lane >> 3) & 1) * 16;
-#pragma unroll
-    for (int k = 0; k < KS; ++k) {
-      uint32_t f0[4], f1[4];
-      ldsm(krow + k * 32, f0);
-      ldsm(krow + 16 * RP + k * 32, f1);
+  // step j: values of tile j - 1 and scores of tile j back to back (no barrier between them), then the softmax of tile j
+  for (int j = 0; j <= nt && nt > 0; ++j) {
+    if (j > 0) {
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
-        mma_bf16(sc[m][0], qa[m][k], f0[0], f0[1]);
-        mma_bf16(sc[m][1], qa[m][k], f0[2], f0[3]);
-        mma_bf16(sc[m][2], qa[m][k], f1[0], f1[1]);
-        mma_bf16(sc[m][3], qa[m][k], f1[2], f1[3]);
+        const float a0 = sAl[m * 16 + (lane >> 2)], a1 = sAl[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          o[m][n][0] *= a0;
+          o[m][n][1] *= a0;
+          o[m][n][2] *= a1;
+          o[m][n][3] *= a1;
+        }
+      }
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        const uint32_t slot = s0 + ((2 * (j - 1) + half) % NS) * L::SLOT;
+        uint32_t pa[MT][2][4];
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+          for (int k = 0; k < 2; ++k)
+            ldsm(s0 + L::P_OFF + (m * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * L::PP + half * 64 + k * 32 + (lane >> 4) * 16, pa[m][k]);
+#pragma unroll
+        for (int n = 0; n < NT; ++n) {
+          uint32_t f[4];
+          ldsm_t(slot + lane * RP + (warp * (RC / 8) + n * 8) * 2, f);
+#pragma unroll
+          for (int m = 0; m < MT; ++m) {
+            mma_bf16(o[m][n], pa[m][0], f[0], f[1]);
+            mma_bf16(o[m][n], pa[m][1], f[2], f[3]);
+          }
+        }
       }
     }
+    if (j < nt) {
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
+      for (int half = 0; half < 2; ++half) {
+        const int h = 2 * j + half;
+        if (ok && h < nh && !mbar_wait_warp(bars + (h % NS) * 8, (h / NS) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) ok = false;
+      }
+      // scores of 32 keys over a quarter of the columns
+      float sc[MT][4][4];
 #pragma unroll
-      for (int n = 0; n < 4; ++n)
+      for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int i = 0; i < 2; ++i)
-          *reinterpret_cast<float2*>(sS + (rg * MT * 16 + m * 16 + (lane >> 2) + 8 * i) * L::SP + kg * 32 + n * 8 + (lane & 3) * 2) =
-              make_float2(sc[m][n][2 * i], sc[m][n][2 * i + 1]);
-    __syncthreads();
-    // every warp is past tile j - 1: its stage takes tile j - 1 + ST
-    if (ok && j - 1 + ST < nt) {
-      fence_proxy_async_smem();
-      issue(j - 1 + ST, page_next);
+        for (int n = 0; n < 4; ++n) sc[m][n][0] = sc[m][n][1] = sc[m][n][2] = sc[m][n][3] = 0.f;
+      const uint32_t krow = s0 + ((2 * j + kg) % NS) * L::SLOT + ((lane & 7) + (lane >> 4) * 8) * RP + rg * (RC / 2) + ((lane >> 3) & 1) * 16;
+#pragma unroll
+      for (int k = 0; k < KS; ++k) {
+        uint32_t f0[4], f1[4];
+        ldsm(krow + k * 32, f0);
+        ldsm(krow + 16 * RP + k * 32, f1);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+          mma_bf16(sc[m][0], qa[m][k], f0[0], f0[1]);
+          mma_bf16(sc[m][1], qa[m][k], f0[2], f0[3]);
+          mma_bf16(sc[m][2], qa[m][k], f1[0], f1[1]);
+          mma_bf16(sc[m][3], qa[m][k], f1[2], f1[3]);
+        }
+      }
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+#pragma unroll
+          for (int i = 0; i < 2; ++i)
+            *reinterpret_cast<float2*>(sS + (rg * MT * 16 + m * 16 + (lane >> 2) + 8 * i) * L::SP + kg * 32 + n * 8 + (lane & 3) * 2) =
+                make_float2(sc[m][n][2 * i], sc[m][n][2 * i + 1]);
     }
-    page_next = page_of(j + ST);
-    const int n_valid = t_end - (t_begin + j * LD_KEYS);
+    __syncthreads();
+    if (j == nt) break;
+    // every warp is done with tile j - 1: its slots take the next two halves
+    if (j > 0) {
+      const int h = NS + 2 * (j - 1) + my_half;
+      if (ok) {
+        fence_proxy_async_smem();
+        issue(h, page_next);
+      }
+      page_next = page_of(h + 2);
+    }
+    const int n_valid = count - j * LD_KEYS;
 #pragma unroll
     for (int i = 0; i < 2 * MT; ++i) {
       const int row = warp * 2 * MT + i;
@@ -649,46 +684,15 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const Late
       }
       s.x = 2 * lane < n_valid ? s.x * sl2 : -INFINITY;
       s.y = 2 * lane + 1 < n_valid ? s.y * sl2 : -INFINITY;
-      const float mx = fmaxf(m_run[i], warp_max(fmaxf(s.x, s.y)));
-      const float mb = mx == -INFINITY ? 0.f : mx;
-      const float alpha = m_run[i] == -INFINITY ? 0.f : exp2f(m_run[i] - mb);
-      const float p0 = exp2f(s.x - mb), p1 = exp2f(s.y - mb);
+      const float mx = fmaxf(m_run[i], warp_max(fmaxf(s.x, s.y)));     // finite: a tile has a key
+      const float alpha = ex2(m_run[i] - mx);
+      const float p0 = ex2(s.x - mx), p1 = ex2(s.y - mx);
       m_run[i] = mx;
       l_run[i] = fmaf(l_run[i], alpha, p0 + p1);
       *reinterpret_cast<uint32_t*>(sm + L::P_OFF + row * L::PP + lane * 4) = pack_bf16(p0, p1);
       if (lane == 0) sAl[row] = alpha;
     }
     __syncthreads();
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const float a0 = sAl[m * 16 + (lane >> 2)], a1 = sAl[m * 16 + (lane >> 2) + 8];
-#pragma unroll
-      for (int n = 0; n < NT; ++n) {
-        o[m][n][0] *= a0;
-        o[m][n][1] *= a0;
-        o[m][n][2] *= a1;
-        o[m][n][3] *= a1;
-      }
-    }
-#pragma unroll
-    for (int half = 0; half < 2; ++half) {
-      uint32_t pa[MT][2][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m)
-#pragma unroll
-        for (int k = 0; k < 2; ++k)
-          ldsm(s0 + L::P_OFF + (m * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * L::PP + half * 64 + k * 32 + (lane >> 4) * 16, pa[m][k]);
-#pragma unroll
-      for (int n = 0; n < NT; ++n) {
-        uint32_t f[4];
-        ldsm_t(tile + (half * 32 + lane) * RP + (warp * (RC / 8) + n * 8) * 2, f);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          mma_bf16(o[m][n], pa[m][0], f[0], f[1]);
-          mma_bf16(o[m][n], pa[m][1], f[2], f[3]);
-        }
-      }
-    }
   }
   if (!ok) {   // give copies already issued a bounded time to land before shared memory goes away
     const uint64_t t0 = globaltimer_ns();
@@ -966,27 +970,15 @@ TFB_API int tfb_head_attn(const void* q, long long ldq, const void* k, long long
 #undef TFB_ANY
 }
 
-TFB_API int tfb_gemm_f32_heads(const float* A, long long lda, int a_head, const float* B, long long ldb, int b_kn, float* C, long long ldc, int c_head,
-                               const float* gate, long long ldg, int M, int heads, int N, int K, void* stream);
-
-// One product per head: x [M, ldx] (x_head entries between heads, K of them used), w: heads blocks [N, K] ([K, N] with kn) stacked on the
-// rows, out [M, ldo] (out_head >= N entries between heads; those past N become zero), gate [M, ldg] or null.
-TFB_API int tfb_head_linear(const void* x, long long ldx, const void* w, long long ldw, int kn, void* out, long long ldo, int out_head, const void* gate,
-                            long long ldg, int M, int heads, int K, int N, int x_head, int f32, void* stream) {
+// One product per head: x [M, ldx] (x_head entries between heads, K of them used), w: heads blocks [K, N] stacked on the rows, out [M, ldo]
+// (out_head >= N entries between heads; those past N become zero).
+TFB_API int tfb_head_linear(const void* x, long long ldx, int x_head, const void* w, long long ldw, void* out, long long ldo, int out_head, int M,
+                            int heads, int N, int K, void* stream) {
   using namespace tfb;
   if (M <= 0 || heads <= 0 || heads > 65535 || K <= 0 || N <= 0 || x_head < K || out_head < N) return TFB_ERR_ARG;
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) {
-    if (out_head > N)
-      if (cudaError_t e = cudaMemset2DAsync(out, size_t(ldo) * 4, 0, size_t(heads) * out_head * 4, M, st)) return int(e);
-    return tfb_gemm_f32_heads(static_cast<const float*>(x), ldx, x_head, static_cast<const float*>(w), ldw, kn, static_cast<float*>(out), ldo, out_head,
-                              static_cast<const float*>(gate), ldg, M, heads, N, K, stream);
-  }
-  HeadLinearArgs p{static_cast<const bf16*>(x), static_cast<const bf16*>(w), ldx, ldw, static_cast<bf16*>(out), ldo, static_cast<const bf16*>(gate), ldg,
-                   M, N, K, x_head, out_head, x_head % 8 == 0 && ldx % 8 == 0 && al16(x), ldw % 8 == 0 && al16(w)};
-  const dim3 grid((out_head + HL_N - 1) / HL_N, heads, (M + HL_M - 1) / HL_M);
-  if (kn) launch_k(head_linear_kernel<true>, grid, 128, 0, st, p);
-  else launch_k(head_linear_kernel<false>, grid, 128, 0, st, p);
+  HeadLinearArgs p{static_cast<const bf16*>(x), static_cast<const bf16*>(w), ldx, ldw, static_cast<bf16*>(out), ldo, M, N, K, x_head, out_head,
+                   x_head % 8 == 0 && ldx % 8 == 0 && al16(x), ldw % 8 == 0 && al16(w)};
+  launch_k(head_linear_kernel, dim3((out_head + HL_N - 1) / HL_N, heads, (M + HL_M - 1) / HL_M), 128, 0, static_cast<cudaStream_t>(stream), p);
   return int(cudaGetLastError());
 }
 
@@ -1007,7 +999,7 @@ TFB_API int tfb_latent_decode(const void* q, long long ldq, const void* pool, lo
                               const int* positions, void* o, long long ldo, float* acc, float* ml, int splits, int B, int H, int R, int W,
                               float scale, int f32, int* status, void* stream) {
   using namespace tfb;
-  if (B <= 0 || B > 65535 || H <= 0 || R <= 0 || W < R || page <= 0) return TFB_ERR_ARG;
+  if (B <= 0 || B > 65535 || H <= 0 || R <= 0 || W < R || page <= 0 || LD_HALF % page) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (splits > 0 && tfb_latent_decode_plan(B, H, W, 1, f32) > 0) {
     if (splits > 128 || (splits > 1 && (!acc || !ml)) || ldq % 8 || ldo % 8 || !al16(q) || !al16(pool) || !al16(o)) return TFB_ERR_ARG;

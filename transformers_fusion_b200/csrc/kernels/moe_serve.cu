@@ -4,7 +4,7 @@
 //   moe_route          per token: the k largest of logits + bias (fp32, the lower index first among equals) and the softmax over them;
 //                      then the rows of the expert buffers: every expert's assignments are consecutive rows from a multiple
 //                      of 128 on, so that a 128-row tile of the grouped product belongs to one expert.  Few tokens (decode
-//                      steps): one block does all of it; many: selection with per-block counts, a scan, row numbers.
+//                      steps): one block does all of it; many: selection with per-block counts, then the scan and row numbers.
 //   moe_gather         token rows to their assignments' rows
 //   moe_glu            silu(gate) * up of the assigned rows (a decode step's buffers are mostly padding)
 //   moe_weighted_sum   y[t] = base[t] + sum_k w[t, k] * rows[row_of[t, k]], summed in fp32
@@ -25,54 +25,100 @@ struct RouteArgs {
   float* w;                   // [T, K]
   int *rank, *row_of;         // [T, K]
   int* expert_of_tile;        // [tiles]
-  int *counts, *start;        // [E]
+  int* counts;                // [E]
   int tiles;
 };
 
-// Chooses the experts of token t (one warp): `K` rounds, each the largest entry that comes after the last one in the order
-// (value descending, index ascending).  Lane 0 writes; `count` (shared memory) numbers the assignments of each expert.
-__device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int lane, int* count) {
+__device__ __forceinline__ float biased_logit(const RouteArgs& p, const float* z, int e) {
+  return z[e] + (p.bias_f32 ? static_cast<const float*>(p.bias)[e] : to_f(static_cast<const __nv_bfloat16*>(p.bias)[e]));
+}
+// unsigned numbers in the order of the floats; 0 stands for "taken"
+__device__ __forceinline__ uint32_t ordered(float v) {
+  const uint32_t u = __float_as_uint(v);
+  return u ^ (uint32_t(int32_t(u) >> 31) | 0x80000000u);
+}
+__device__ __forceinline__ float unordered(uint32_t k) { return __uint_as_float(k & 0x80000000u ? k ^ 0x80000000u : ~k); }
+
+// Chooses the experts of token t (one warp); `count` (shared memory) numbers the assignments of each expert.  note(i, expert, rank)
+// is called once per assignment i = t K + k.
+// PER > 0: up to 32 PER experts and K <= 32, the logits in registers (lane l: experts l, l + 32, ...).  PER 0: any sizes; K
+// rounds, each the largest entry that comes after the last one in the order (value descending, index ascending).
+template <int PER, class Note>
+__device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int lane, int* count, Note note) {
   const float* z = p.logits + t * p.ld;
-  float last = INFINITY, first = 0.f, sum = 0.f;
-  int last_e = -1;
-  for (int k = 0; k < p.K; ++k) {
-    float best = -INFINITY;
-    int e_best = INT_MAX;
-    for (int e = lane; e < p.E; e += 32) {
-      const float v = z[e] + (p.bias_f32 ? static_cast<const float*>(p.bias)[e] : to_f(static_cast<const __nv_bfloat16*>(p.bias)[e]));
-      const bool after = v < last || (v == last && e > last_e);
-      if (after && (v > best || e_best == INT_MAX)) { best = v; e_best = e; }
-    }
+  if constexpr (PER > 0) {
+    uint32_t key[PER];
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float v = __shfl_xor_sync(0xffffffffu, best, o);
-      const int e = __shfl_xor_sync(0xffffffffu, e_best, o);
-      if (e != INT_MAX && (e_best == INT_MAX || v > best || (v == best && e < e_best))) { best = v; e_best = e; }
+    for (int i = 0; i < PER; ++i) key[i] = lane + i * 32 < p.E ? ordered(biased_logit(p, z, lane + i * 32)) : 0u;
+    float first = 0.f, sum = 0.f, mine = 0.f;
+    int e_mine = 0;
+    for (int k = 0; k < p.K; ++k) {
+      uint32_t best = key[0];
+      int e = lane;
+#pragma unroll
+      for (int i = 1; i < PER; ++i)
+        if (key[i] > best) { best = key[i]; e = lane + i * 32; }
+      const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+      int chosen = int(__reduce_min_sync(0xffffffffu, best == top ? uint32_t(e) : 0x7fffffffu));
+      if (chosen >= p.E) chosen = k;        // logits that compare with nothing
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if (chosen == lane + i * 32) key[i] = 0u;
+      const float v = unordered(top);
+      if (k == 0) first = v;
+      const float x = expf(v - first);
+      sum += x;
+      if (lane == k) { mine = x; e_mine = chosen; }
     }
-    if (e_best == INT_MAX) e_best = k;       // logits that compare with nothing
-    last = best;
-    last_e = e_best;
-    if (k == 0) first = best;
-    const float x = expf(best - first);
-    sum += x;
-    if (lane == 0) {
-      const long long i = (long long)t * p.K + k;
-      p.idx[i] = e_best;
-      p.w[i] = x;
-      p.rank[i] = atomicAdd(count + e_best, 1);
+    if (lane < p.K) {
+      const int i = t * p.K + lane;
+      p.idx[i] = e_mine;
+      p.w[i] = mine / sum;
+      note(i, e_mine, atomicAdd(count + e_mine, 1));
     }
+  } else {
+    float last = INFINITY, first = 0.f, sum = 0.f;
+    int last_e = -1;
+    for (int k = 0; k < p.K; ++k) {
+      float best = -INFINITY;
+      int e_best = INT_MAX;
+      for (int e = lane; e < p.E; e += 32) {
+        const float v = biased_logit(p, z, e);
+        const bool after = v < last || (v == last && e > last_e);
+        if (after && (v > best || e_best == INT_MAX)) { best = v; e_best = e; }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float v = __shfl_xor_sync(0xffffffffu, best, o);
+        const int e = __shfl_xor_sync(0xffffffffu, e_best, o);
+        if (e != INT_MAX && (e_best == INT_MAX || v > best || (v == best && e < e_best))) { best = v; e_best = e; }
+      }
+      if (e_best == INT_MAX) e_best = k;
+      last = best;
+      last_e = e_best;
+      if (k == 0) first = best;
+      const float x = expf(best - first);
+      sum += x;
+      if (lane == 0) {
+        const int i = t * p.K + k;
+        p.idx[i] = e_best;
+        p.w[i] = x;
+        note(i, e_best, atomicAdd(count + e_best, 1));
+      }
+    }
+    __syncwarp();
+    for (int k = lane; k < p.K; k += 32) p.w[(long long)t * p.K + k] /= sum;
   }
-  __syncwarp();
-  for (int k = lane; k < p.K; k += 32) p.w[(long long)t * p.K + k] /= sum;
 }
 
-// start[e] = first row of expert e, expert_of_tile; one block of 1024 threads; `count` may be shared or global memory
-__device__ __forceinline__ void plan_segments(const RouteArgs& p, const int* count) {
+// start[e] (shared memory) = first row of expert e, and expert_of_tile if this block writes it; all NTHR threads of a block
+template <int NTHR>
+__device__ __forceinline__ void plan_segments(const RouteArgs& p, const int* count, int* start, bool write) {
   __shared__ int part[32], carry;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   if (threadIdx.x == 0) carry = 0;
   __syncthreads();
-  for (int e0 = 0; e0 < p.E; e0 += 1024) {
+  for (int e0 = 0; e0 < p.E; e0 += NTHR) {
     const int e = e0 + threadIdx.x;
     const int n = e < p.E ? (count[e] + 127) / 128 : 0;
     int s = n;
@@ -84,7 +130,7 @@ __device__ __forceinline__ void plan_segments(const RouteArgs& p, const int* cou
     if (lane == 31) part[warp] = s;
     __syncthreads();
     if (warp == 0) {
-      int q = part[lane];
+      int q = lane < NTHR / 32 ? part[lane] : 0;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const int v = __shfl_up_sync(0xffffffffu, q, o);
@@ -95,31 +141,37 @@ __device__ __forceinline__ void plan_segments(const RouteArgs& p, const int* cou
     __syncthreads();
     const int base = carry + (warp ? part[warp - 1] : 0) + s - n;
     if (e < p.E) {
-      p.start[e] = base * 128;
-      for (int i = 0; i < n && base + i < p.tiles; ++i) p.expert_of_tile[base + i] = e;
+      start[e] = base * 128;
+      if (write)
+        for (int i = 0; i < n && base + i < p.tiles; ++i) p.expert_of_tile[base + i] = e;
     }
     __syncthreads();
     if (threadIdx.x == 0) carry += part[31];
     __syncthreads();
   }
-  for (int i = carry + threadIdx.x; i < p.tiles; i += 1024) p.expert_of_tile[i] = -1;
+  if (write)
+    for (int i = carry + threadIdx.x; i < p.tiles; i += NTHR) p.expert_of_tile[i] = -1;
 }
 
+constexpr int ROUTE_SMALL = 256, ROUTE_SMALL_ASSIGN = 4096;     // tokens and assignments that one block takes
+template <int PER>
 __global__ void __launch_bounds__(1024) moe_route_small_kernel(const RouteArgs p) {
   tfb::pdl_sync();
-  extern __shared__ int count[];
+  extern __shared__ int sh[];               // count[E], start[E], expert[T K], rank[T K]
+  int *count = sh, *start = sh + p.E, *s_e = start + p.E, *s_r = s_e + p.T * p.K;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   for (int e = threadIdx.x; e < p.E; e += 1024) count[e] = 0;
   __syncthreads();
-  for (int t = warp; t < p.T; t += 32) choose_experts(p, t, lane, count);
+  for (int t = warp; t < p.T; t += 32)
+    choose_experts<PER>(p, t, lane, count, [&](int i, int e, int r) { s_e[i] = e; s_r[i] = r; });
   __syncthreads();
-  plan_segments(p, count);
-  for (int e = threadIdx.x; e < p.E; e += 1024) p.counts[e] = count[e];
+  plan_segments<1024>(p, count, start, true);
   __syncthreads();
-  for (int i = threadIdx.x; i < p.T * p.K; i += 1024) p.row_of[i] = p.start[p.idx[i]] + p.rank[i];
+  for (int i = threadIdx.x; i < p.T * p.K; i += 1024) p.row_of[i] = start[s_e[i]] + s_r[i];
 }
 
-constexpr int ROUTE_TOKENS = 64;      // tokens of a block
+constexpr int ROUTE_TOKENS = 32;      // tokens of a block
+template <int PER>
 __global__ void __launch_bounds__(256) moe_route_choose_kernel(const RouteArgs p) {
   tfb::pdl_sync();
   extern __shared__ int count[];
@@ -127,20 +179,34 @@ __global__ void __launch_bounds__(256) moe_route_choose_kernel(const RouteArgs p
   const int t0 = blockIdx.x * ROUTE_TOKENS, t1 = min(p.T, t0 + ROUTE_TOKENS);
   for (int e = threadIdx.x; e < p.E; e += 256) count[e] = 0;
   __syncthreads();
-  for (int t = t0 + warp; t < t1; t += 8) choose_experts(p, t, lane, count);
+  for (int t = t0 + warp; t < t1; t += 8) choose_experts<PER>(p, t, lane, count, [&](int i, int, int r) { p.rank[i] = r; });
   __syncthreads();
   for (int e = threadIdx.x; e < p.E; e += 256) count[e] = count[e] ? atomicAdd(p.counts + e, count[e]) : 0;
   __syncthreads();
-  for (long long i = (long long)t0 * p.K + threadIdx.x; i < (long long)t1 * p.K; i += 256) p.rank[i] += count[p.idx[i]];
+  for (int i = t0 * p.K + threadIdx.x; i < t1 * p.K; i += 256) p.rank[i] += count[p.idx[i]];
 }
-__global__ void __launch_bounds__(1024) moe_route_plan_kernel(const RouteArgs p) {
-  tfb::pdl_sync();
-  plan_segments(p, p.counts);
-}
+constexpr int ROUTE_ROWS = 2048;      // assignments of a block
 __global__ void __launch_bounds__(256) moe_route_rows_kernel(const RouteArgs p) {
   tfb::pdl_sync();
-  const long long i = blockIdx.x * 256ll + threadIdx.x;
-  if (i < (long long)p.T * p.K) p.row_of[i] = p.start[p.idx[i]] + p.rank[i];
+  extern __shared__ int start[];
+  plan_segments<256>(p, p.counts, start, blockIdx.x == 0);
+  __syncthreads();
+  const long long i0 = blockIdx.x * (long long)ROUTE_ROWS, n = (long long)p.T * p.K;
+  for (int i = threadIdx.x; i < ROUTE_ROWS && i0 + i < n; i += 256) p.row_of[i0 + i] = start[p.idx[i0 + i]] + p.rank[i0 + i];
+}
+
+template <int PER>
+static int launch_route(const RouteArgs& p, cudaStream_t st) {
+  const size_t e4 = size_t(p.E) * 4;
+  const long long a = (long long)p.T * p.K;
+  if (p.T <= ROUTE_SMALL && a <= ROUTE_SMALL_ASSIGN && p.E <= 1024) {
+    launch_k(moe_route_small_kernel<PER>, 1, 1024, 2 * e4 + size_t(a) * 8, st, p);
+    return int(cudaGetLastError());
+  }
+  if (cudaError_t e = cudaMemsetAsync(p.counts, 0, e4, st)) return int(e);
+  launch_k(moe_route_choose_kernel<PER>, (p.T + ROUTE_TOKENS - 1) / ROUTE_TOKENS, 256, e4, st, p);
+  launch_k(moe_route_rows_kernel, int((a + ROUTE_ROWS - 1) / ROUTE_ROWS), 256, e4, st, p);
+  return int(cudaGetLastError());
 }
 
 template <class T, int VEC>
@@ -216,27 +282,19 @@ static int blocks_for(long long items) {
 
 using bf16 = __nv_bfloat16;
 
-// logits [T, ld] fp32, bias [E] (bias_f32: fp32, otherwise bf16).  idx, row_of, rank (scratch): int [T, K]; w: fp32 [T, K]; counts, start
+// logits [T, ld] fp32, bias [E] (bias_f32: fp32, otherwise bf16).  idx, row_of, rank (scratch): int [T, K]; w: fp32 [T, K]; counts
 // (scratch): int [E]; expert_of_tile: int [tiles], tiles >= T K / 128 + min(E, T K).
 TFB_API int tfb_moe_route(const float* logits, const void* bias, int T, int E, int K, int* idx, float* w, int* row_of, int* expert_of_tile,
-                          int* counts, int* rank, int* start, int tiles, long long ld, int bias_f32, void* stream) {
+                          int* counts, int* rank, int tiles, long long ld, int bias_f32, void* stream) {
   using namespace tfb;
   if (T <= 0 || E <= 0 || K <= 0 || K > E || !bias) return TFB_ERR_ARG;
   const long long a = (long long)T * K;
   if (tiles < a / 128 + (E < a ? E : a)) return TFB_ERR_ARG;
-  if (E > 8192) return TFB_ERR_LIMIT;
-  RouteArgs p{logits, ld, bias, bias_f32, T, E, K, idx, w, rank, row_of, expert_of_tile, counts, start, tiles};
+  if (E > 8192 || a > INT_MAX / 2) return TFB_ERR_LIMIT;
+  RouteArgs p{logits, ld, bias, bias_f32, T, E, K, idx, w, rank, row_of, expert_of_tile, counts, tiles};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const size_t smem = size_t(E) * 4;
-  if (T <= 256) {
-    launch_k(moe_route_small_kernel, 1, 1024, smem, st, p);
-    return int(cudaGetLastError());
-  }
-  if (cudaError_t e = cudaMemsetAsync(counts, 0, smem, st)) return int(e);
-  launch_k(moe_route_choose_kernel, (T + ROUTE_TOKENS - 1) / ROUTE_TOKENS, 256, smem, st, p);
-  launch_k(moe_route_plan_kernel, 1, 1024, 0, st, p);
-  launch_k(moe_route_rows_kernel, int((a + 255) / 256), 256, 0, st, p);
-  return int(cudaGetLastError());
+  if (K > 32 || E > 256) return launch_route<0>(p, st);
+  return E <= 32 ? launch_route<1>(p, st) : E <= 64 ? launch_route<2>(p, st) : E <= 128 ? launch_route<4>(p, st) : launch_route<8>(p, st);
 }
 
 #define TFB_BY_TYPE(KERN, GRID, VECOK, ...)                                                                \

@@ -445,6 +445,16 @@ def preset(name: str) -> TransformerConfig:
                 mix = DiffAttentionSpec(heads, kv, 64, 128, 64 ** -0.5, 0.5, rot, win, i - 2 if i % 4 == 3 else None)
             layers.append(StackLayer(mix, ff))
         return LanedraConfig(V, H, layers, 1e-5, 1.0, max_seq_len=32768)
+    if name in ("tekenex-7b", "tekenex-8x7b"):
+        # beside mixture-7b and mixtral-8x7b: the same width, query rows and experts, of which one (two of mixture-7b's) is shared;
+        # the first layer is dense
+        H, heads, n, V, mix, ff = (2048, 16, 24, 32000, MixtureSpec(62, 6, 704, 1408), 8448) if name == "tekenex-7b" else \
+            (4096, 32, 32, 32000, MixtureSpec(7, 1, 14336, 14336), 43008)
+        att = LatentAttentionSpec(heads, 128, 128, 512, 128 ** -0.5)
+        return TekenexConfig(V, H, [StackLayer(att, 0 if i else ff, mix if i else None) for i in range(n)], 1e-5)
+    if name == "mixture-7b":
+        return MoEConfig(vocab_size=32000, hidden_size=2048, num_layers=24, num_heads=16, num_kv_heads=4, ffn_hidden_size=704, rope_theta=500000.0,
+                         max_seq_len=32768, activation="swiglu", num_experts=64, top_k=8)
     if name == "dense-1.5b":
         return TransformerConfig(vocab_size=32000, hidden_size=2048, num_layers=24, num_heads=16, num_kv_heads=4, ffn_hidden_size=5632,
                                  rope_theta=500000.0, max_seq_len=32768, activation="swiglu")

@@ -14,7 +14,6 @@ from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass
-from typing import Optional
 
 import torch
 
@@ -32,7 +31,7 @@ _lib.register("tfb_moe_combine_bwd", [c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_
 _lib.register("tfb_moe_permute_bwd", [c_p, c_p, c_p, c_i, c_i, c_i, c_p])
 
 
-_lib.register("tfb_moe_route", [c_p, c_p, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_ll, c_i, c_p])
+_lib.register("tfb_moe_route", [c_p, c_p, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_ll, c_i, c_p])
 _lib.register("tfb_moe_gather", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_moe_glu", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_p])
 _lib.register("tfb_moe_gemm_f32", [c_p, c_ll, c_p, c_ll, c_ll, c_p, c_ll, c_p, c_i, c_i, c_i, c_i, c_p])
@@ -323,7 +322,6 @@ class Routing:
     row_of: torch.Tensor                       # int32 [T, k]
     expert_of_tile: torch.Tensor               # int32 [max_rows / 128], -1: no expert
     max_rows: int
-    counts: Optional[torch.Tensor] = None      # int32 [E] (CUDA)
 
 
 def route(logits, bias, k) -> Routing:
@@ -347,11 +345,11 @@ def route(logits, bias, k) -> Routing:
         of_tile += [-1] * (tiles - len(of_tile))
         return Routing(idx.int(), w, row_of.view(T, k), torch.tensor(of_tile, dtype=torch.int32), tiles * 128)
     i32 = lambda *s: torch.empty(s, dtype=torch.int32, device=dev)
-    r = Routing(i32(T, k), torch.empty((T, k), dtype=torch.float32, device=dev), i32(T, k), i32(tiles), tiles * 128, i32(E))
-    rank, start = i32(T, k), i32(E)
+    r = Routing(i32(T, k), torch.empty((T, k), dtype=torch.float32, device=dev), i32(T, k), i32(tiles), tiles * 128)
+    rank, counts = i32(T, k), i32(E)
     check(_lib.lib().tfb_moe_route(logits.data_ptr(), bias.data_ptr(), T, E, k, r.idx.data_ptr(), r.w.data_ptr(), r.row_of.data_ptr(),
-                                   r.expert_of_tile.data_ptr(), r.counts.data_ptr(), rank.data_ptr(), start.data_ptr(), tiles,
-                                   logits.stride(0), int(bias.dtype == torch.float32), stream()), "moe_route", 1 if T <= 256 else 3)
+                                   r.expert_of_tile.data_ptr(), counts.data_ptr(), rank.data_ptr(), tiles,
+                                   logits.stride(0), int(bias.dtype == torch.float32), stream()), "moe_route", 1 if T <= 256 else 2)
     return r
 
 

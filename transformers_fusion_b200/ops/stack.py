@@ -16,8 +16,8 @@ from . import _lib
 from . import functional as F
 from ._lib import c_f, c_i, c_ll, c_p, check, ptr, stream
 
-UNITS = ("tfb_host", "gemm_bf16", "stack_ops", "diff_attention", "delta_rule")    # translation units these operators need
-UNITS_LATENT = ("tfb_host", "gemm_bf16", "stack_ops", "latent_attention", "moe_serve")
+UNITS = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "diff_attention", "delta_rule")    # translation units these operators need
+UNITS_LATENT = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "latent_attention", "moe_serve")
 PAGE = 16
 ACT = {None: 0, "relu2": 4}      # codes of the product epilogues (gemm_bf16.cu: apply_act)
 
@@ -26,9 +26,13 @@ _lib.register("tfb_glu_silu", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
 _lib.register("tfb_rope_append", [c_p, c_ll, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_gather_rows", [c_p, c_ll, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p])
 _lib.register("tfb_gemm_f32", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_skinny_fits", [c_i, c_i, c_i])
+_lib.register("tfb_skinny_linear", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_act_rows", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_latent_append", [c_p, c_ll, c_p, c_f, c_p, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
-_lib.register("tfb_head_linear", [c_p, c_ll, c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_head_linear", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_skinny_linear_heads", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_gemm_f32_heads", [c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_head_attn", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p])
 _lib.register("tfb_latent_decode_plan", [c_i, c_i, c_i, c_i, c_i])
 _lib.register("tfb_latent_decode", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p])
@@ -61,8 +65,8 @@ def padded_weight(n: int, width: int, dtype, device, lead=()) -> torch.Tensor:
 
 # ---------------------------------------------------------------------------------------------------- products
 def linear(x, w, out_dtype=None, act=None):
-    """act(x [M, K] @ w [N, K]^T).  bf16 operands: tensor-core GEMM with fp32 accumulation (``out_dtype`` fp32 keeps the
-    accumulator's precision); fp32 operands: FFMA in true fp32.  ``act``: None or "relu2"."""
+    """act(x [M, K] @ w [N, K]^T).  bf16 operands: tensor-core product with fp32 accumulation (``out_dtype`` fp32 keeps the
+    accumulator's precision), in a form of its own for few rows; fp32 operands: FFMA in true fp32.  ``act``: None or "relu2"."""
     out_dtype = out_dtype or x.dtype
     if not x.is_cuda:
         return activation(x.float() @ w.float().t(), act).to(out_dtype)
@@ -73,6 +77,11 @@ def linear(x, w, out_dtype=None, act=None):
         assert w.dtype == torch.float32 and w.shape[1] == K and x.stride(1) == 1 and w.stride(1) == 1
         check(_lib.lib().tfb_gemm_f32(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, ACT[act],
                                       stream()), "gemm_f32")
+        return out
+    if x.dtype == w.dtype == torch.bfloat16 and x.stride(1) == w.stride(1) == 1 and (x.stride(0) | w.stride(0)) % 8 == 0 and \
+            (x.data_ptr() | w.data_ptr()) % 16 == 0 and _lib.lib().tfb_skinny_fits(M, N, K):
+        check(_lib.lib().tfb_skinny_linear(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, ACT[act],
+                                           int(out_dtype == torch.float32), stream()), "skinny_linear")
         return out
     if act is None:
         return F.gemm(x, w, out=out)
@@ -267,7 +276,8 @@ def latent_append(c, w, eps, slots, pool, want_rows=True):
 def head_linear(x, w, heads, k, n, gate=None, transposed=False):
     """One small product per head: x [M, heads * k] with w of heads blocks [n, k] ([k, n] when ``transposed``) stacked on the rows
     -> [M, heads * n8] where n8 is n for plain and n rounded up to 8 (zero filled) for transposed blocks; ``gate`` [M, heads]: head h
-    is multiplied by sigmoid(gate[:, h])."""
+    is multiplied by sigmoid(gate[:, h]) (plain blocks only).  Plain blocks: x comes with every head padded to a multiple of 8 entries
+    with zeros (as ``latent_decode`` returns it)."""
     M = x.shape[0]
     n8 = (n + 7) // 8 * 8 if transposed else n
     if not x.is_cuda:
@@ -279,10 +289,22 @@ def head_linear(x, w, heads, k, n, gate=None, transposed=False):
         out = torch.zeros((M, heads, n8), dtype=x.dtype)
         out[..., :n] = o.to(x.dtype)
         return out.view(M, heads * n8)
+    L, x_head = _lib.lib(), x.shape[1] // heads
+    assert gate is None or not transposed
+    if x.dtype == torch.float32:
+        out = torch.zeros((M, heads * n8), dtype=x.dtype, device=x.device)
+        check(L.tfb_gemm_f32_heads(x.data_ptr(), x.stride(0), x_head, w.data_ptr(), w.stride(0), int(transposed), out.data_ptr(), out.stride(0), n8,
+                                   ptr(gate), gate.stride(0) if gate is not None else 0, M, heads, n, k, stream()), "gemm_f32_heads")
+        return out
     out = rows(M, heads * n8, x.dtype, x.device)
-    check(_lib.lib().tfb_head_linear(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), int(transposed), out.data_ptr(), out.stride(0), n8,
-                                     ptr(gate), gate.stride(0) if gate is not None else 0, M, heads, k, n, x.shape[1] // heads, _f32(x), stream()),
-          "head_linear")
+    if transposed:
+        check(L.tfb_head_linear(x.data_ptr(), x.stride(0), x_head, w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), n8, M, heads, n, k,
+                                stream()), "head_linear")
+    else:                                      # k rounded up to 8: the padding of x is zero and that of w finite
+        k8 = (k + 7) // 8 * 8
+        assert x_head >= k8 and w.stride(0) >= k8
+        check(L.tfb_skinny_linear_heads(x.data_ptr(), x.stride(0), x_head, w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), ptr(gate),
+                                        gate.stride(0) if gate is not None else 0, M, heads, n, k8, stream()), "skinny_linear_heads")
     return out
 
 
