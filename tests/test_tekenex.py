@@ -476,7 +476,7 @@ def test_config_reader():
         c = TekenexConfig.from_dict(d)
         assert c.to_dict() == d
         m = TekenexModel(c, seed=None)
-        assert m.param_count() == c.num_params() == sum(t.numel() for t in m.parameters()) + 0
+        assert m.param_count() == c.num_params() == sum(t.numel() for t in m.parameters())
         assert c.active_params() <= c.num_params()
     assert TekenexConfig.from_dict(CONFIGS["large"]).active_params() < TekenexConfig.from_dict(CONFIGS["large"]).num_params()
     for change, what in ((lambda l: l["mlp"]["router"].update(top=7), "choose 7 of 6"), (lambda l: l.update(type="attention"), "unknown mixer"),

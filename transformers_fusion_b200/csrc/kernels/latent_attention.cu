@@ -94,6 +94,12 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
+__device__ __forceinline__ float redux_max(float x) {      // over the warp, one instruction
+  float y;
+  asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // running maximum over the 128 scores of this thread's row; keys after `hi` (index within the tile) do not count
 template <bool MASK>
 __device__ __forceinline__ float tile_max(uint32_t tS, float m, int hi) {
@@ -596,6 +602,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const Late
 #pragma unroll
       for (int m = 0; m < MT; ++m) {
         const float a0 = sAl[m * 16 + (lane >> 2)], a1 = sAl[m * 16 + (lane >> 2) + 8];
+        if (__all_sync(0xffffffffu, a0 == 1.f && a1 == 1.f)) continue;       // no maximum of these rows has moved
 #pragma unroll
         for (int n = 0; n < NT; ++n) {
           o[m][n][0] *= a0;
@@ -684,7 +691,7 @@ __global__ void __launch_bounds__(LD_THREADS, 1) latent_decode_kernel(const Late
       }
       s.x = 2 * lane < n_valid ? s.x * sl2 : -INFINITY;
       s.y = 2 * lane + 1 < n_valid ? s.y * sl2 : -INFINITY;
-      const float mx = fmaxf(m_run[i], warp_max(fmaxf(s.x, s.y)));     // finite: a tile has a key
+      const float mx = fmaxf(m_run[i], redux_max(fmaxf(s.x, s.y)));     // finite: a tile has a key
       const float alpha = ex2(m_run[i] - mx);
       const float p0 = ex2(s.x - mx), p1 = ex2(s.y - mx);
       m_run[i] = mx;
