@@ -7,8 +7,8 @@ Kernels: gemm, gemm_nt_wgrad, gemm_fp8, attention_fwd, attention_bwd, rmsnorm, r
 cross_entropy, adamw, paged_decode, sampling, moe_ffn; those of stack models (``STACK_KERNELS``): diff_attention,
 diff_attention_window, attention_fwd_gqa128 (the plain form of the same layer), diff_decode, delta_prep, delta_scan,
 delta_scan_one, gated_norm, delta_prep_step, delta_step, res_norm, glu_silu, rope_append; those of latent attention and the serving
-mixture with the like kernels of the mixture-of-experts decoder (``LATENT_KERNELS``).  ``--kernel all | stack | latent`` or names
-with commas between them.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
+mixture with the like kernels of the mixture-of-experts decoder (``LATENT_KERNELS``).  ``--kernel`` takes names and the groups all, stack, latent, with commas
+between them.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
 against their NCCL forms (cli/bench_comm.py)."""
 from __future__ import annotations
 
@@ -309,7 +309,8 @@ def _build(kernel, n, dev, heads=0, shape=None):
 
 
 def time_kernel(fn, iters=20, warmup=5, flush=True):
-    """Per-launch milliseconds (list) measured with CUDA events; a 256 MiB write evicts L2 between launches."""
+    """Per-launch milliseconds (list) measured with CUDA events; writes of 256 MiB evict L2 between launches (several: they
+    also cover the host's time to enqueue an operator of more than one launch, which would be measured otherwise)."""
     import torch
     scrub = torch.empty(256 << 20, dtype=torch.uint8, device="cuda") if flush else None
     for _ in range(warmup):
@@ -318,7 +319,8 @@ def time_kernel(fn, iters=20, warmup=5, flush=True):
     out = []
     for _ in range(iters):
         if scrub is not None:
-            scrub.fill_(1)
+            for v in range(5):
+                scrub.fill_(v)
         e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
         e0.record()
         fn()
@@ -526,7 +528,8 @@ def main(argv=None):
         if not torch.cuda.is_available():
             print("Error: kernel benchmarks need a CUDA device", file=sys.stderr)
             return 1
-        names = {"all": KERNELS, "stack": STACK_KERNELS, "latent": LATENT_KERNELS}.get(a.kernel) or a.kernel.split(",")
+        groups = {"all": KERNELS, "stack": STACK_KERNELS, "latent": LATENT_KERNELS}
+        names = [n for k in a.kernel.split(",") for n in groups.get(k, (k,))]
         peaks = json.load(open(a.peaks)) if a.peaks else {}
         for name in names:
             shape = None

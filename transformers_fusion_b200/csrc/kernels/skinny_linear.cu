@@ -39,7 +39,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) skinny_linear_kernel(const Skin
   tfb::pdl_sync();
   __shared__ float red[SK_WARPS][MT * 16][SK_N + 1];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, q = lane & 3;
-  const int n0 = blockIdx.x * SK_N, h = blockIdx.y, m0 = blockIdx.z * 64, M = min(64, p.M - m0);
+  const int n0 = blockIdx.x * SK_N, h = blockIdx.y, m0 = blockIdx.z * MT * 16, M = min(MT * 16, p.M - m0);
   float acc[MT][2][4];
 #pragma unroll
   for (int m = 0; m < MT; ++m)
@@ -92,36 +92,42 @@ __global__ void __launch_bounds__(SK_WARPS * 32) skinny_linear_kernel(const Skin
 
 using bf16 = __nv_bfloat16;
 
-static int launch_skinny(const tfb::SkinnyArgs& p, int heads, void* stream) {
+// 16-row, 16-column blocks x their depth: every block reads its rows and columns of both operands
+static long long tfb_skinny_work(int M, long long N, int K) { return (N + 15) / 16 * ((M + 15) / 16) * K; }
+
+static int launch_skinny(const tfb::SkinnyArgs& p, int heads, int rows, void* stream) {
   using namespace tfb;
-  if (p.M <= 0 || p.N <= 0 || p.K <= 0 || p.K % 8 || p.ldx % 8 || p.ldw % 8 || p.x_head % 8 || heads <= 0 || heads > 65535 || p.M > 64 * 65535 ||
+  if (p.M <= 0 || p.N <= 0 || p.K <= 0 || p.K % 8 || p.ldx % 8 || p.ldw % 8 || p.x_head % 8 || heads <= 0 || heads > 65535 || p.M > 16 * 65535 ||
       (reinterpret_cast<uintptr_t>(p.x) & 15) || (reinterpret_cast<uintptr_t>(p.w) & 15))
     return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const dim3 grid((p.N + SK_N - 1) / SK_N, heads, (p.M + 63) / 64);
-  if (p.M <= 16) launch_k(skinny_linear_kernel<1>, grid, SK_WARPS * 32, 0, st, p);
-  else if (p.M <= 32) launch_k(skinny_linear_kernel<2>, grid, SK_WARPS * 32, 0, st, p);
-  else launch_k(skinny_linear_kernel<4>, grid, SK_WARPS * 32, 0, st, p);
+  if (rows == 0) rows = p.M <= 16 || tfb_skinny_work(p.M, p.N * heads, p.K) <= 1500000 ? 16 : 32;
+  const dim3 grid((p.N + SK_N - 1) / SK_N, heads, (p.M + rows - 1) / rows);
+  if (rows == 16) launch_k(skinny_linear_kernel<1>, grid, SK_WARPS * 32, 0, st, p);
+  else if (rows == 32) launch_k(skinny_linear_kernel<2>, grid, SK_WARPS * 32, 0, st, p);
+  else if (rows == 64) launch_k(skinny_linear_kernel<4>, grid, SK_WARPS * 32, 0, st, p);
+  else return TFB_ERR_ARG;
   return int(cudaGetLastError());
 }
 
-// 1 where the few-row form is the one to take: every block reads all of x, so that (blocks x rows) bounds what it may cost.
+// 1 where the few-row form is the one to take.  Measured against the tcgen05 form (with its split-K finalize): it wins while a warp's share
+// of K is short and, for more than 16 rows, while reading the operands once per block stays cheap.
 TFB_API int tfb_skinny_fits(int M, int N, int K) {
-  return M <= 64 && K % 8 == 0 && (long long)N * ((M + 15) / 16 * 16) <= 420000;
+  return M <= 64 && K % 8 == 0 && K <= 6144 && (M <= 16 || tfb_skinny_work(M, N, K) <= 2000000);
 }
 
-// act: 0 none, 4 relu squared.  Row pitches are multiples of 8 entries, x and w aligned to 16 bytes.
+// act: 0 none, 4 relu squared.  rows: rows of a block (16, 32 or 64; 0: the kernel's choice).  Row pitches are multiples of 8 entries, x and w aligned to 16 bytes.
 TFB_API int tfb_skinny_linear(const void* x, long long ldx, const void* w, long long ldw, void* out, long long ldo, int M, int N, int K, int act,
-                              int out_f32, void* stream) {
+                              int out_f32, int rows, void* stream) {
   if (M > 64 || (act != 0 && act != 4)) return TFB_ERR_ARG;
   return launch_skinny(tfb::SkinnyArgs{static_cast<const bf16*>(x), static_cast<const bf16*>(w), ldx, ldw, out, ldo, M, N, K, act, out_f32, 0, 0,
-                                       nullptr, 0}, 1, stream);
+                                       nullptr, 0}, 1, rows, stream);
 }
 
 // One product per head: x [M, ldx] (x_head entries between heads), w: heads blocks [N, K] stacked on the rows, out [M, ldo] (N entries per
 // head), gate [M, ldg] or null.
 TFB_API int tfb_skinny_linear_heads(const void* x, long long ldx, int x_head, const void* w, long long ldw, void* out, long long ldo, const void* gate,
-                                    long long ldg, int M, int heads, int N, int K, void* stream) {
+                                    long long ldg, int M, int heads, int N, int K, int rows, void* stream) {
   return launch_skinny(tfb::SkinnyArgs{static_cast<const bf16*>(x), static_cast<const bf16*>(w), ldx, ldw, out, ldo, M, N, K, 0, 0, x_head, N,
-                                       static_cast<const bf16*>(gate), ldg}, heads, stream);
+                                       static_cast<const bf16*>(gate), ldg}, heads, rows, stream);
 }

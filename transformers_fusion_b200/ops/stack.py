@@ -27,11 +27,11 @@ _lib.register("tfb_rope_append", [c_p, c_ll, c_p, c_p, c_i, c_p, c_p, c_p, c_p, 
 _lib.register("tfb_gather_rows", [c_p, c_ll, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p])
 _lib.register("tfb_gemm_f32", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_skinny_fits", [c_i, c_i, c_i])
-_lib.register("tfb_skinny_linear", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_skinny_linear", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_act_rows", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_latent_append", [c_p, c_ll, c_p, c_f, c_p, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_head_linear", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
-_lib.register("tfb_skinny_linear_heads", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_skinny_linear_heads", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_gemm_f32_heads", [c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_head_attn", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p])
 _lib.register("tfb_latent_decode_plan", [c_i, c_i, c_i, c_i, c_i])
@@ -81,7 +81,7 @@ def linear(x, w, out_dtype=None, act=None):
     if x.dtype == w.dtype == torch.bfloat16 and x.stride(1) == w.stride(1) == 1 and (x.stride(0) | w.stride(0)) % 8 == 0 and \
             (x.data_ptr() | w.data_ptr()) % 16 == 0 and _lib.lib().tfb_skinny_fits(M, N, K):
         check(_lib.lib().tfb_skinny_linear(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, ACT[act],
-                                           int(out_dtype == torch.float32), stream()), "skinny_linear")
+                                           int(out_dtype == torch.float32), 0, stream()), "skinny_linear")
         return out
     if act is None:
         return F.gemm(x, w, out=out)
@@ -304,7 +304,7 @@ def head_linear(x, w, heads, k, n, gate=None, transposed=False):
         k8 = (k + 7) // 8 * 8
         assert x_head >= k8 and w.stride(0) >= k8
         check(L.tfb_skinny_linear_heads(x.data_ptr(), x.stride(0), x_head, w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), ptr(gate),
-                                        gate.stride(0) if gate is not None else 0, M, heads, n, k8, stream()), "skinny_linear_heads")
+                                        gate.stride(0) if gate is not None else 0, M, heads, n, k8, 0, stream()), "skinny_linear_heads")
     return out
 
 
