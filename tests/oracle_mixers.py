@@ -313,3 +313,164 @@ class PlainTekenex:
         return self.norm("final.norm", x) @ w["embed"].T
 
     greedy = PlainLanedra.greedy
+
+
+# ---------------------------------------------------------------------------------------------------- attention with options
+def plain_norm(x, w, eps):
+    return rms(x, eps) * w
+
+
+def sigmoid(z):
+    return 1 / (1 + torch.exp(-z))
+
+
+def rotate_linear(x, pos0, dims, base, factor=1.0):
+    """x [T, n, dim] at positions pos0, pos0 + 1, ...: entry i of the first ``dims`` with entry i + dims / 2, all frequencies divided
+    by ``factor``."""
+    y = x.clone()
+    for t in range(x.shape[0]):
+        for i in range(dims // 2):
+            a = (pos0 + t) * float(base) ** (-2.0 * i / dims) / factor
+            u, v = x[t, :, i], x[t, :, i + dims // 2]
+            y[t, :, i] = u * math.cos(a) - v * math.sin(a)
+            y[t, :, i + dims // 2] = v * math.cos(a) + u * math.sin(a)
+    return y
+
+
+def query_temperature(p, coef, every):
+    """Factor of the query at position p."""
+    return 1 + coef * math.log((p + 1) // every + 1)
+
+
+def soft_cap(s, cap):
+    return cap * torch.tanh(s / cap)
+
+
+def seen(i, j, window=None, keep_first=0):
+    """Whether position i looks at position j."""
+    return j <= i and (window is None or i - j < window or j < keep_first)
+
+
+def attend_options(q, k, v, pos0, scale, window=None, keep_first=0, cap=None, sink=False, temp=None):
+    """One head.  q [T, dim] at positions pos0 ..., k [N, dim] and v [N, vdim] at 0 ...; ``cap``: soft cap of the scores; ``sink``: one
+    more key of score 0 that has no value; ``temp``: (coef, every) of the queries' factor."""
+    out = []
+    for t in range(q.shape[0]):
+        i = pos0 + t
+        at = torch.tensor([j for j in range(k.shape[0]) if seen(i, j, window, keep_first)])
+        s = (k[at] @ (q[t] * (query_temperature(i, *temp) if temp else 1.0))) * scale
+        if cap:
+            s = soft_cap(s, cap)
+        m = max(float(s.max()), 0.0)
+        e = torch.exp(s - m)
+        out.append((e @ v[at]) / (e.sum() + (math.exp(-m) if sink else 0.0)))
+    return torch.stack(out)
+
+
+# ---------------------------------------------------------------------------------------------------- gated linear attention
+def channel_decay(z, tau):
+    return sigmoid(z) ** (1 / tau)
+
+
+def gated_linear_scan(q, k, v, alpha, state=None):
+    """One head: q, k, alpha [T, dim], v [T, vdim]; the state [dim, vdim] decays by key channel.  Returns (o [T, vdim], state)."""
+    S = torch.zeros(k.shape[1], v.shape[1], dtype=k.dtype) if state is None else state.clone()
+    out = []
+    for t in range(k.shape[0]):
+        S = alpha[t][:, None] * S + torch.outer(k[t], v[t])
+        out.append(S.T @ q[t])
+    return torch.stack(out), S
+
+
+# ---------------------------------------------------------------------------------------------------- feed-forwards
+def gelu_tanh(z):
+    return 0.5 * z * (1 + torch.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def geglu(h, gate, up, down):
+    return (gelu_tanh(h @ gate.T) * (h @ up.T)) @ down.T
+
+
+def route_groups(z, top, groups, keep, scale):
+    """One token's router logits -> [(expert, weight)].  Scores are sigmoids; the ``keep`` groups of neighbouring experts with the
+    largest sums of two scores stay; of their experts the ``top`` best, weighted by their scores over the scores' sum, times scale."""
+    s = [1 / (1 + math.exp(-float(x))) for x in z]
+    n = len(s) // groups
+    mark = [sum(sorted(s[g * n:(g + 1) * n], reverse=True)[:2]) for g in range(groups)]
+    stay = sorted(range(groups), key=lambda g: (-mark[g], g))[:keep]
+    order = sorted((e for e in range(len(s)) if e // n in stay), key=lambda e: (-s[e], e))[:top]
+    total = sum(s[e] for e in order) + 1e-20
+    return [(e, s[e] / total * scale) for e in order]
+
+
+def grouped_mixture(h, router, top, groups, keep, scale, experts, shared=None, shared_gate=None):
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for i, w in route_groups(router @ h[t], top, groups, keep, scale):
+            out[t] += w * swiglu(h[t], *experts[i])
+    return out if shared is None else out + sigmoid(h @ shared_gate.T) * swiglu(h, *shared)
+
+
+class PlainFigudra:
+    """As PlainLanedra, for parallel layers (one norm, mixer and feed-forward side by side) of attention with options or gated linear
+    attention, whose tensors may be those of another layer, under a normed embedding."""
+
+    def __init__(self, cfg, tensors):
+        self.cfg = cfg
+        self.w = {n: t.to(DT) for n, t in tensors.items()}
+
+    def start(self):
+        return {"pos": 0, "layers": [{} for _ in self.cfg["layers"]]}
+
+    def attention(self, m, p, h, mine, pos, eps):
+        w, H, G, D, V, T = self.w, m["heads"], m["kv_heads"], m["dim"], m["vdim"], h.shape[0]
+        q, k, v = (h @ w[p + "q"].T).view(T, H, D), (h @ w[p + "k"].T).view(T, G, D), (h @ w[p + "v"].T).view(T, G, V)
+        second = "rot" in m
+        if second:
+            rot = (m["rot"]["dims"], m["rot"]["base"], m["rot"].get("scaling", {}).get("factor", 1.0))
+            q = rotate_linear(plain_norm(q, w[p + "q.norm"], eps), pos, *rot)
+            k = rotate_linear(plain_norm(k, w[p + "k.norm"], eps), pos, *rot)
+            opt = dict(window=m["mask"]["size"], keep_first=m["mask"]["keep_first"], sink=True)
+        else:
+            opt = dict(cap=m["softcap"], temp=(m["q_temp"]["coef"], m["q_temp"]["every"]))
+        mine["k"] = torch.cat([mine["k"], k]) if "k" in mine else k
+        mine["v"] = torch.cat([mine["v"], v]) if "v" in mine else v
+        o = torch.stack([attend_options(q[:, x], mine["k"][:, x // (H // G)], mine["v"][:, x // (H // G)], pos, m["scale"], **opt)
+                         for x in range(H)], 1).reshape(T, H * V)
+        if not second:
+            o = o * sigmoid(h @ w[p + "g"].T)
+        return o @ w[p + "o"].T
+
+    def gla(self, m, p, h, mine, pos, eps):
+        w, H, D, V, T = self.w, m["heads"], m["dim"], m["vdim"], h.shape[0]
+        q, k, v = (h @ w[p + "q"].T).view(T, H, D) * D ** -0.5, (h @ w[p + "k"].T).view(T, H, D), (h @ w[p + "v"].T).view(T, H, V)
+        a = channel_decay((h @ w[p + "a1"].T) @ w[p + "a2"].T + w[p + "a2.b"], m["tau"]).view(T, H, D)
+        both = [gated_linear_scan(q[:, x], k[:, x], v[:, x], a[:, x], mine["S"][x] if "S" in mine else None) for x in range(H)]
+        mine["S"] = [s for _, s in both]
+        o = plain_norm(torch.stack([o for o, _ in both], 1), w[p + "norm"], eps) * silu(h @ w[p + "g"].T).view(T, H, V)
+        return o.reshape(T, H * V) @ w[p + "o"].T
+
+    def ff(self, m, p, h):
+        three = lambda q: tuple(self.w[p + q + n] for n in ("gate", "up", "down"))
+        if m["kind"] == "dense":
+            return geglu(h, *three(""))
+        r = m["router"]
+        return grouped_mixture(h, self.w[p + "router"], r["top"], r["groups"]["count"], r["groups"]["keep"], r["scale"],
+                               [three(f"e{e}.") for e in range(r["experts"])], three("shared.") if m.get("shared") else None,
+                               self.w.get(p + "shared.sg"))
+
+    def run(self, tokens, st=None, residuals=None):
+        w, eps = self.w, self.cfg["norm"]["eps"]
+        st = st if st is not None else self.start()
+        x = plain_norm(w["embed"][torch.tensor(tokens)], w["embed.norm"], eps)
+        for i, l in enumerate(self.cfg["layers"]):
+            p = f"l{l.get('weights_of', i)}."
+            h = plain_norm(x, w[p + "norm1"], eps)
+            y = (self.gla if l["type"] == "gla" else self.attention)(l["mixer"], p + "mix.", h, st["layers"][i], st["pos"], eps)
+            x = x + (y + self.ff(l["mlp"], p + "mlp.", h) if l["mlp"] else y)
+            if residuals is not None:
+                residuals.append(x.clone())
+        st["pos"] += len(tokens)
+        return plain_norm(x, w["final.norm"], eps) @ w["head"].T
+
+    greedy = PlainLanedra.greedy
