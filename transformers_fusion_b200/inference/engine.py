@@ -68,7 +68,7 @@ class Request:
     # runtime state
     out: List[int] = field(default_factory=list)
     pages: List[int] = field(default_factory=list)   # -1: a page that has left every layer's window
-    first_page: int = 0            # pages below this one have been given back
+    first_page: int = 0            # pages below this one have been given back, or are kept for good
     state_slot: int = -1           # recurrent state (models that have some)
     pos: int = 0
     t_submit: float = 0.0
@@ -305,15 +305,15 @@ class InferenceEngine:
     def _reserve(self, r: Request, n: int, shared=()):
         """Pages for tokens 0 .. n - 1 of a sequence that starts (``shared``: pages of a cached prefix; pages that no later
         query will look at are left out) and its slot of recurrent state."""
-        lo = self.cache.first_live_page(n)
-        r.pages = list(shared) + [self.cache.allocator.alloc() if i >= lo else -1 for i in range(len(shared), (n + PAGE - 1) // PAGE)]
-        r.first_page = min(lo, len(r.pages))
+        lo, kept = self.cache.first_live_page(n), self.cache.kept_pages
+        r.pages = list(shared) + [self.cache.allocator.alloc() if i >= lo or i < kept else -1 for i in range(len(shared), (n + PAGE - 1) // PAGE)]
+        r.first_page = min(max(lo, kept), len(r.pages))
         r.state_slot = self.cache.take_slot()
 
     def _drop_old_pages(self, r: Request):
         """Give back the pages that have left the window of every query from r.pos on."""
         lo = min(self.cache.first_live_page(r.pos), len(r.pages))
-        for i in range(r.first_page, lo):
+        for i in range(max(r.first_page, self.cache.kept_pages), lo):
             self.cache.allocator.release(r.pages[i])
             r.pages[i] = -1
         r.first_page = max(r.first_page, lo)

@@ -119,6 +119,7 @@ class PagedKVCache:
 
     # what the scheduler asks of every kind of cache (see mixer_cache): no window, no recurrent state, prefixes may be shared
     shareable = True
+    kept_pages = 0
 
     def first_live_page(self, pos: int) -> int:
         return 0

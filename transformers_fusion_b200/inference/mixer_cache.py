@@ -3,10 +3,11 @@
 * Attention layers that have keys and values of their own: paged pools, one row of keys ([kv_heads, maps * dim]) and one of
   values per token, with the page allocator and block tables of ``kv_cache``; the layers share one page list per
   sequence.  When every attention layer looks back over a window only, pages that have left the longest window go back to
-  the allocator (``first_live_page``), and a prompt's earlier tokens are never written.
+  the allocator (``first_live_page``), and a prompt's earlier tokens are never written; the pages of the first tokens stay when
+  some layer keeps them in sight (``kept_pages``).
 * Latent attention layers: one paged pool with a row of ``latent_width`` entries per token (the latent, zeros behind it), under the
   same page list.
-* Recurrent layers: a slot per sequence with the fp32 state matrices and the last inputs of the short convolution.  A slot's
+* Recurrent layers: a slot per sequence with the fp32 state matrices and, where there is one, the last inputs of the short convolution.  A slot's
   contents are only read by a sequence that goes on; a sequence that starts ignores and overwrites them, so slots need no
   clearing when they change hands.
 
@@ -27,6 +28,7 @@ class MixerCache:
         self.allocator = PageAllocator(num_pages)
         self.free_slots: List[int] = list(range(num_slots - 1, -1, -1))
         self.window = cfg.window
+        self.kept_pages = (getattr(cfg, "keep_first", 0) + PAGE - 1) // PAGE if self.window else 0
         self.k: Dict[int, torch.Tensor] = {}
         self.v: Dict[int, torch.Tensor] = {}
         self.latent: Dict[int, torch.Tensor] = {}
@@ -37,6 +39,11 @@ class MixerCache:
             if m.kind == "attention" and m.kv_from is None:
                 self.k[i] = torch.zeros((num_pages * PAGE, m.kv_heads * 2 * m.dim), dtype=dtype, device=device)
                 self.v[i] = torch.zeros((num_pages * PAGE, m.kv_heads * m.vdim), dtype=dtype, device=device)
+            elif m.kind == "head_attention":
+                self.k[i] = torch.zeros((num_pages * PAGE, m.kv_heads * m.dim), dtype=dtype, device=device)
+                self.v[i] = torch.zeros((num_pages * PAGE, m.kv_heads * m.vdim), dtype=dtype, device=device)
+            elif m.kind == "gla":
+                self.state[i] = torch.zeros((num_slots, m.heads, m.dim, m.vdim), dtype=torch.float32, device=device)
             elif m.kind == "latent_attention":
                 self.latent[i] = torch.zeros((num_pages * PAGE, m.latent_width), dtype=dtype, device=device)
             elif m.kind == "delta":
@@ -63,13 +70,13 @@ class MixerCache:
             self.free_slots.append(slot)
 
     def first_live_page(self, pos: int) -> int:
-        """The first page that a query at position ``pos`` or later can still look at."""
+        """The first page, kept ones aside, that a query at position ``pos`` or later can still look at."""
         return max(0, pos - self.window + 1) // PAGE if self.window else 0
 
     def pages_needed(self, tokens: int) -> int:
         """The most pages a sequence of ``tokens`` tokens holds at a time."""
         n = (tokens + PAGE - 1) // PAGE
-        return min(n, (self.window - 1) // PAGE + 2) if self.window else n
+        return min(n, (self.window - 1) // PAGE + 2 + self.kept_pages) if self.window else n
 
     def bytes_per_token(self) -> float:
         return float(sum(t.shape[1] * t.element_size() for d in (self.k, self.v, self.latent) for t in d.values()))

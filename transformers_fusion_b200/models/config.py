@@ -155,13 +155,15 @@ class MoEConfig(TransformerConfig):
 # ---------------------------------------------------------------------------------------------------------------------
 @dataclass(frozen=True)
 class RotarySpec:
-    """Rotary embedding of the first ``dims`` entries of a head; ``yarn_*`` (factor None: unscaled) as in YaRN."""
+    """Rotary embedding of the first ``dims`` entries of a head; ``yarn_*`` (factor None: unscaled) as in YaRN; ``linear``: every
+    frequency is divided by it."""
     dims: int
     base: float
     yarn_factor: float = None
     yarn_original: int = 0
     yarn_fast: float = 32.0
     yarn_slow: float = 1.0
+    linear: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -218,13 +220,58 @@ class LatentAttentionSpec:
 
 
 @dataclass(frozen=True)
+class HeadAttentionSpec:
+    """Softmax attention of ``heads`` query heads over ``kv_heads`` key / value heads.  ``rot``: rotation of queries and keys (None:
+    no positions); ``qk_norm``: RMS norm of every query and key head in front of it; ``gate``: one output gate per entry of the
+    heads; ``window`` > 0: a position sees that many keys up to itself, and the first ``keep_first`` of the sequence; ``softcap``
+    > 0: scores are cap tanh(score / cap); ``sink``: the denominator counts one more key of score 0; queries at position p are
+    multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: RotarySpec = None
+    qk_norm: bool = False
+    gate: bool = False
+    window: int = 0
+    keep_first: int = 0
+    softcap: float = 0.0
+    sink: bool = False
+    temp_coef: float = 0.0
+    temp_every: int = 1
+
+    kind = "head_attention"
+
+
+@dataclass(frozen=True)
+class GatedLinearSpec:
+    """Gated linear attention: per head a [dim, vdim] state whose rows decay by sigmoid(z)^(1/tau), z from a projection of rank
+    ``rank`` per key channel."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int = 16
+
+    kind = "gla"
+
+
+@dataclass(frozen=True)
 class MixtureSpec:
-    """Mixture of gated feed-forward experts: ``top`` of ``experts`` per token, weighted by the softmax over the chosen router
-    logits; ``shared_ff`` > 0: one more expert of that size that every token runs."""
+    """Mixture of gated feed-forward experts: ``top`` of ``experts`` per token; ``shared_ff`` > 0: one more expert of that size that
+    every token runs (``shared_gate``: times the sigmoid of a logit per token).  ``score`` "softmax": the largest logits (plus a
+    bias), weighted by the softmax over the chosen ones.  "sigmoid": the largest sigmoids (no bias) among the experts of the ``keep``
+    best of ``groups`` equal groups (by the sum of a group's two largest), weighted by them over their sum, times ``scale``."""
     experts: int
     top: int
     ff: int
     shared_ff: int = 0
+    shared_gate: bool = False
+    score: str = "softmax"
+    groups: int = 1
+    keep: int = 1
+    scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -232,6 +279,7 @@ class StackLayer:
     mixer: object
     ffn_hidden_size: int = 0     # dense feed-forward; 0: the layer has none
     mixture: MixtureSpec = None  # mixture of experts instead of a dense feed-forward
+    weights_of: int = None       # the layer whose tensors this one uses
 
 
 @dataclass
@@ -411,6 +459,155 @@ class TekenexConfig:
 
     def active_params(self) -> int:
         """Parameters that take part in one token's pass."""
+        return self._count(True)
+
+
+@dataclass
+class FigudraConfig:
+    """Figudra: softmax attention of two kinds (capped scores and an output gate, no positions; or normed, rotated queries and keys in
+    a window with kept first tokens and a sink) and gated linear attention in any order, with a dense (gelu) or grouped
+    mixture-of-experts feed-forward beside the mixer under one norm, a normed embedding and a separate head.  A layer may use
+    another layer's tensors.  ``from_dict`` reads the model folder's config.json; the rank of the decay projection is that of its
+    tensor (``shapes``: tensor name -> shape).  ``max_seq_len`` as in ``LanedraConfig``."""
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    norm_eps: float
+    max_seq_len: int = 32768
+
+    architecture = "Figudra"
+    embedding_scale = 1.0
+    tie_embeddings = False
+
+    def __post_init__(self):
+        for i, l in enumerate(self.layers):
+            m, x = l.mixer, l.mixture
+            if m.kind == "head_attention":
+                if m.heads % m.kv_heads:
+                    raise ValueError(f"layer {i}: {m.heads} heads do not divide over {m.kv_heads} kv heads")
+                if m.rot is not None and (m.rot.dims % 2 or not 0 < m.rot.dims <= m.dim):
+                    raise ValueError(f"layer {i}: cannot rotate {m.rot.dims} of {m.dim} entries")
+            elif not 1 <= m.dim <= 512:
+                raise ValueError(f"layer {i}: key channels per head {m.dim} are not in 1 .. 512")
+            if x is not None:
+                if x.experts % x.groups or not 1 <= x.keep <= x.groups or not 1 <= x.top <= x.experts // x.groups * x.keep:
+                    raise ValueError(f"layer {i}: cannot choose {x.top} of {x.experts} experts in {x.keep} of {x.groups} groups")
+                if x.groups > 1 and (x.groups > 32 or x.experts > 1024 or x.top > 32):
+                    raise ValueError(f"layer {i}: grouped routing takes up to 32 groups, 1024 experts and 32 of them per token")
+            if l.weights_of is not None:
+                j = l.weights_of
+                if not 0 <= j < len(self.layers) or j == i or self.layers[j].weights_of is not None:
+                    raise ValueError(f"layer {i}: layer {j} has no tensors to share")
+                if (self.layers[j].mixer, self.layers[j].ffn_hidden_size, self.layers[j].mixture) != (m, l.ffn_hidden_size, x):
+                    raise ValueError(f"layer {i}: layer {j}'s tensors have other sizes or constants")
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def _attention(self):
+        return [l.mixer for l in self.layers if l.mixer.kind == "head_attention"]
+
+    @property
+    def window(self) -> int:
+        """As ``LanedraConfig.window``, the kept first tokens aside."""
+        w = [m.window for m in self._attention]
+        return 0 if not w or 0 in w else max(w)
+
+    @property
+    def keep_first(self) -> int:
+        return max((m.keep_first for m in self._attention), default=0)
+
+    @classmethod
+    def from_dict(cls, d: dict, shapes=None, **extra) -> "FigudraConfig":
+        layers = []
+        for i, e in enumerate(d["layers"]):
+            m, f, src = e["mixer"], e.get("mlp"), e.get("weights_of")
+            seen = set()
+            while src is not None and d["layers"][src].get("weights_of") is not None and src not in seen:
+                seen.add(src)                  # the layer at the end of the chain has the tensors
+                src = d["layers"][src]["weights_of"]
+            if e["type"] == "attention":
+                t = m["q_temp"]
+                if t["every"] != int(t["every"]):
+                    raise ValueError(f"layer {i}: q_temp.every has to be whole")
+                mix = HeadAttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), gate=True, softcap=float(m["softcap"]),
+                                        temp_coef=float(t["coef"]), temp_every=int(t["every"]))
+            elif e["type"] == "attention_2":
+                r, k = m["rot"], m["mask"]
+                rot = RotarySpec(int(r["dims"]), float(r["base"]), linear=float((r.get("scaling") or {}).get("factor", 1.0)))
+                mix = HeadAttentionSpec(m["heads"], m["kv_heads"], m["dim"], m["vdim"], float(m["scale"]), rot, qk_norm=True, window=k["size"],
+                                        keep_first=k.get("keep_first") or 0, sink=True)
+            elif e["type"] == "gla":
+                a1 = (shapes or {}).get(f"l{i if src is None else src}.mix.a1")
+                mix = GatedLinearSpec(m["heads"], m["dim"], m["vdim"], float(m["tau"]), *(() if a1 is None else (a1[0],)))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer '{e['type']}'")
+            kind = f.get("kind", "dense") if f else None
+            if kind == "dense":
+                layers.append(StackLayer(mix, f["ff"], weights_of=src))
+            elif kind == "moe":
+                r, sh = f["router"], f.get("shared")
+                g = r.get("groups") or {"count": 1, "keep": 1}
+                layers.append(StackLayer(mix, 0, MixtureSpec(r["experts"], r["top"], f["expert"]["ff"], sh["ff"] if sh else 0, bool(sh), "sigmoid",
+                                                             g["count"], g["keep"], float(r["scale"])), src))
+            elif kind is None:
+                layers.append(StackLayer(mix, weights_of=src))
+            else:
+                raise ValueError(f"layer {i}: unknown feed-forward '{kind}'")
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], layers=layers, norm_eps=float(d["norm"]["eps"]), **extra)
+
+    def to_dict(self) -> dict:
+        """The config.json form."""
+        out = []
+        for l in self.layers:
+            m, x = l.mixer, l.mixture
+            a = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+            kind = m.kind
+            if kind == "gla":
+                a["tau"] = m.tau
+            else:
+                a.update(kv_heads=m.kv_heads, scale=m.scale)
+                if m.rot is None:
+                    kind = "attention"
+                    a.update(softcap=m.softcap, q_temp={"coef": m.temp_coef, "every": m.temp_every})
+                else:
+                    kind = "attention_2"
+                    a.update(mask={"size": m.window, "keep_first": m.keep_first},
+                             rot={"dims": m.rot.dims, "base": m.rot.base, "scaling": {"factor": m.rot.linear}})
+            f = {"kind": "dense", "ff": l.ffn_hidden_size} if l.ffn_hidden_size else None
+            if x is not None:
+                f = {"kind": "moe", "expert": {"ff": x.ff},
+                     "router": {"experts": x.experts, "top": x.top, "scale": x.scale, "groups": {"count": x.groups, "keep": x.keep}}}
+                if x.shared_ff:
+                    f["shared"] = {"ff": x.shared_ff}
+            e = {"type": kind, "mixer": a, "mlp": f}
+            if l.weights_of is not None:
+                e["weights_of"] = l.weights_of
+            out.append(e)
+        return {"architecture": self.architecture, "layers": out, "norm": {"eps": self.norm_eps}, "vocab": self.vocab_size, "width": self.hidden_size}
+
+    def _count(self, active: bool) -> int:
+        H, n = self.hidden_size, 2 * self.vocab_size * self.hidden_size + 2 * self.hidden_size
+        for l in self.layers:
+            m, x = l.mixer, l.mixture
+            if l.weights_of is not None and not active:
+                continue
+            if m.kind == "gla":
+                n += H * (m.heads * (2 * m.dim + 3 * m.vdim) + m.rank) + m.heads * m.dim * (m.rank + 1) + m.vdim
+            else:
+                n += H * (m.dim * (m.heads + m.kv_heads) + m.vdim * (m.kv_heads + m.heads * (2 if m.gate else 1))) + (2 * m.dim if m.qk_norm else 0)
+            n += H + 3 * H * l.ffn_hidden_size
+            if x is not None:
+                n += 3 * H * (x.ff * (x.top if active else x.experts) + x.shared_ff) + H * (x.experts + int(x.shared_gate))
+        return n
+
+    def num_params(self) -> int:
+        return self._count(False)
+
+    def active_params(self) -> int:
+        """Parameters that take part in one token's pass (those of a layer that is run twice count twice)."""
         return self._count(True)
 
 

@@ -5,6 +5,7 @@
 from __future__ import annotations
 
 import importlib
+import inspect
 import json
 import os
 from typing import Dict, Tuple
@@ -15,6 +16,7 @@ import torch
 ARCHITECTURES: Dict[str, Tuple[str, str]] = {
     "Lanedra": ("lanedra", "LanedraModel"),
     "Tekenex": ("tekenex", "TekenexModel"),
+    "Figudra": ("figudra", "FigudraModel"),
 }
 
 
@@ -41,7 +43,14 @@ def read_config(path):
     if "architecture" not in d:
         raise ValueError(f"{path}: config.json names no architecture")
     cls = model_class(d["architecture"])
-    return cls, cls.config_cls.from_dict(d)
+    if "shapes" not in inspect.signature(cls.config_cls.from_dict).parameters:
+        return cls, cls.config_cls.from_dict(d)
+    from ..quant.importers import _sources
+    shapes = {}                      # sizes that only the tensors give
+    for src in _sources(path):
+        shapes.update((n, tuple(src.shape(n))) for n in src.names)
+        src.close()
+    return cls, cls.config_cls.from_dict(d, shapes=shapes)
 
 
 def load_folder(path, device="cpu", dtype=torch.float32):
@@ -71,7 +80,8 @@ def limit_build(path):
     """For a process that only runs the forward passes of this folder's model: a kernel library that still has to be built is
     built from the translation units of that model's passes alone."""
     from ..ops import _lib
-    cls, _ = read_config(path)
+    with open(os.path.join(path, "config.json")) as f:
+        cls = model_class(json.load(f)["architecture"])
     _lib.need_units(f"tfb_kernels_{cls.__name__.lower()}", cls.kernel_units)
 
 

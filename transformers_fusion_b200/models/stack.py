@@ -7,19 +7,23 @@ The engine drives the same passes for prompts, for portions of prompts and for d
 lives in ``inference.mixer_cache``.  A pass of one layer is, for a prompt or a decode step alike:
 
   attention   GEMM [q | k | v], rotation + cache append, attention with its epilogue (difference of the maps, norm, scale), GEMM
+  head_attention  GEMM [q | k | v | gates], head norms + rotation + cache append, attention with its epilogue (sink, gates), GEMM
   latent      GEMM [q | latent | gates], norm of the latent + cache append, then
                 prompts   GEMM latent -> [k | v], attention with the head gates in its epilogue, GEMM
                 decoding  queries taken to the latent space, attention over the cached latents, values read out of the result
                           head by head with the gates, GEMM
   delta       GEMM [q | k | v | gate | b | a], convolution + unit lengths + gates, recurrence (+ gated norm), GEMM
-  MLP         GEMM [gate | up], silu(gate) * up, GEMM;  or GEMM with the squared relu in its epilogue, GEMM
+  gla         GEMM [q | k | v | gate | a1], decays + products of four tokens, recurrence, gated norm (decoding: one kernel), GEMM
+  MLP         GEMM [gate | up], act(gate) * up, GEMM;  or GEMM with the squared relu in its epilogue, GEMM
   mixture     router GEMM (fp32 logits), top-k + expert segments, rows by expert, grouped GEMM, silu(gate) * up, grouped GEMM,
-              weighted sum + shared expert
-  between     norm and scale of the sublayer's output, residual add and norm of (or rounding for) the next sublayer, one kernel
+              weighted sum + (gated) shared expert
+  between     norm and scale of the sublayer's output (or the sum of two), residual add and norm of (or rounding for) the next
+              sublayer, one kernel
 
 bf16 parameters: bf16 activations and tensor-core products; fp32 parameters: everything in true fp32."""
 from __future__ import annotations
 
+import copy
 from dataclasses import dataclass
 from typing import Optional
 
@@ -53,13 +57,30 @@ def _param(*shape, device, dtype, pitched=True):
     return nn.Parameter(w, requires_grad=False)
 
 
-class DiffAttention(nn.Module):
+class Sublayer(nn.Module):
+    """A mixer or feed-forward of layer ``index`` (its cache) with the tensors of layer ``source``."""
+
+    def __init__(self, index: int):
+        super().__init__()
+        self.index = self.source = index
+
+    def finalize(self):
+        pass
+
+    def at(self, index: int):
+        """The same tensors as a part of another layer."""
+        m = copy.copy(self)
+        m.index = index
+        return m
+
+
+class DiffAttention(Sublayer):
     """Differential attention with an optional window and optional keys / values of an earlier layer."""
     linear_names = ("qkv", "o")
 
     def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
-        super().__init__()
-        self.spec, self.eps, self.index = spec, eps, index
+        super().__init__(index)
+        self.spec, self.eps = spec, eps
         self.nq = 2 * spec.heads
         self.nk = 0 if spec.kv_from is not None else 2 * spec.kv_heads
         self.v_cols = spec.kv_heads * spec.vdim if self.nk else 0
@@ -88,7 +109,7 @@ class DiffAttention(nn.Module):
         s = self.spec
         if self._lambda is None:
             self.finalize()
-        qkv = lin(h, self.index, "qkv", self.qkv)
+        qkv = lin(h, self.source, "qkv", self.qkv)
         pool = self.index if self.nk else s.kv_from
         K.rope_append(qkv, rope, b.positions, self.nq, self.nk, s.dim, s.rot.dims, self.v_cols, b.slots if self.nk else None,
                       cache.k[pool] if self.nk else None, cache.v[pool] if self.nk else None)
@@ -107,16 +128,71 @@ class DiffAttention(nn.Module):
                     kv[self.index] = (K.gather_rows(cache.k[pool], b.pages, lo, n), K.gather_rows(cache.v[pool], b.pages, lo, n), n)
             k, v, n = kv[pool]
             o = K.diff_attn(q, k, v, b.B, b.S, n, *args)
-        return lin(o, self.index, "o", self.o)
+        return lin(o, self.source, "o", self.o)
 
 
-class GatedDelta(nn.Module):
+class HeadAttention(Sublayer):
+    """Softmax attention with the options of its spec (see ``HeadAttentionSpec``)."""
+    linear_names = ("proj", "o")
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+        super().__init__(index)
+        self.spec, self.eps = spec, eps
+        kw = dict(device=device, dtype=dtype)
+        self.nq, self.nk, self.nv, self.no = spec.heads * spec.dim, spec.kv_heads * spec.dim, spec.kv_heads * spec.vdim, spec.heads * spec.vdim
+        self.proj = _param(self.nq + self.nk + self.nv + (self.no if spec.gate else 0), hidden, **kw)
+        self.o = _param(hidden, self.no, **kw)
+        if spec.qk_norm:
+            self.q_norm, self.k_norm = _param(spec.dim, **kw), _param(spec.dim, **kw)
+        self.options = K.HeadOptions(spec.window, spec.keep_first, spec.softcap, spec.sink, spec.temp_coef, spec.temp_every)
+
+    def tensors(self):
+        a, b, c = self.nq, self.nq + self.nk, self.nq + self.nk + self.nv
+        yield "q", self.proj.data[:a]
+        yield "k", self.proj.data[a:b]
+        yield "v", self.proj.data[b:c]
+        if self.spec.gate:
+            yield "g", self.proj.data[c:]
+        if self.spec.qk_norm:
+            yield "q.norm", self.q_norm.data
+            yield "k.norm", self.k_norm.data
+        yield "o", self.o.data
+
+    def _past(self, cache, b):
+        """Keys and values that the portion from b.pos0 on looks at: the kept first tokens and the window of its first query, or
+        the whole sequence, this portion's included."""
+        s, n = self.spec, b.pos0 + b.S
+        lo = max(0, b.pos0 - s.window + 1) if s.window else 0
+        kept = min(s.keep_first, lo)
+        out = []
+        for pool in (cache.k[self.index], cache.v[self.index]):
+            t = K.gather_rows(pool, b.pages, lo, n - lo)
+            out.append(torch.cat([K.gather_rows(pool, b.pages, 0, kept), t]) if kept else t)
+        return out[0], out[1], kept + n - lo
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        s, i = self.spec, self.index
+        p = lin(h, self.source, "proj", self.proj)
+        K.rope_append(p, rope, b.positions, s.heads, s.kv_heads, s.dim, s.rot.dims if s.rot else 0, self.nv, b.slots, cache.k[i], cache.v[i],
+                      (self.q_norm.data, self.k_norm.data, self.eps) if s.qk_norm else None)
+        c = self.nq + self.nk
+        q, gate = p[:, :self.nq], p[:, c + self.nv:] if s.gate else None
+        sizes = (s.heads, s.kv_heads, s.dim, s.vdim, s.scale, gate, self.options)
+        if b.decode:
+            o = K.head_decode(q, cache.k[i], cache.v[i], b.block_table, b.positions, *sizes)
+        else:
+            k, v, n = self._past(cache, b) if b.pos0 else (p[:, self.nq:c], p[:, c:c + self.nv], b.S)
+            o = K.head_attn(q, k, v, b.B, b.S, n, *sizes, b.pos0)
+        return lin(o, self.source, "o", self.o)
+
+
+class GatedDelta(Sublayer):
     """Gated delta rule with a short convolution in front and a gated norm behind."""
     linear_names = ("proj", "o")
 
     def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
-        super().__init__()
-        self.spec, self.eps, self.index = spec, eps, index
+        super().__init__(index)
+        self.spec, self.eps = spec, eps
         kw = dict(device=device, dtype=dtype)
         self.hv = spec.heads * spec.vdim
         self.proj = _param(spec.conv_channels + self.hv + 2 * spec.heads, hidden, **kw)
@@ -136,13 +212,10 @@ class GatedDelta(nn.Module):
         for n in ("A_log", "dt_bias", "norm", "o"):
             yield n, getattr(self, n).data
 
-    def finalize(self):
-        pass
-
     def forward(self, h, b: StepBatch, cache, rope, lin, kv):
         s, i = self.spec, self.index
         G, H, D, V = s.kv_heads, s.heads, s.dim, s.vdim
-        p = lin(h, i, "proj", self.proj)
+        p = lin(h, self.source, "proj", self.proj)
         past = b.decode or b.pos0 > 0
         prep = K.delta_prep(p, self.conv.data, cache.conv[i], b.state_slots, self.A_log.data, self.dt_bias.data, b.lens, b.B, b.S, G, H, D, V, past, b.decode)
         gate = p[:, s.conv_channels:s.conv_channels + self.hv]
@@ -150,16 +223,52 @@ class GatedDelta(nn.Module):
             o = K.delta_step(prep, cache.state[i], b.state_slots, gate, self.norm.data, self.eps, b.B, G, H, D, V)
         else:
             o = K.gated_norm(K.delta_scan(prep, cache.state[i], b.state_slots, b.lens, b.B, b.S, G, H, D, V, past), gate, self.norm.data, self.eps)
-        return lin(o, i, "o", self.o)
+        return lin(o, self.source, "o", self.o)
 
 
-class LatentAttention(nn.Module):
+class GatedLinear(Sublayer):
+    """Gated linear attention with a decay per key channel and a gated norm behind."""
+    linear_names = ("proj", "o")
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+        super().__init__(index)
+        self.spec, self.eps = spec, eps
+        kw = dict(device=device, dtype=dtype)
+        self.hd, self.hv = spec.heads * spec.dim, spec.heads * spec.vdim
+        self.proj = _param(2 * self.hd + 2 * self.hv + spec.rank, hidden, **kw)
+        self.a2, self.a2_b, self.norm = _param(self.hd, spec.rank, **kw), _param(self.hd, **kw), _param(spec.vdim, **kw)
+        self.o = _param(hidden, self.hv, **kw)
+
+    def tensors(self):
+        at = 0
+        for n, width in (("q", self.hd), ("k", self.hd), ("v", self.hv), ("g", self.hv), ("a1", self.spec.rank)):
+            yield n, self.proj.data[at:at + width]
+            at += width
+        yield "a2", self.a2.data
+        yield "a2.b", self.a2_b.data
+        yield "norm", self.norm.data
+        yield "o", self.o.data
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        s, state = self.spec, cache.state[self.index]
+        p = lin(h, self.source, "proj", self.proj)
+        low, sizes = (p, self.a2.data, self.a2_b.data, s.tau), (s.heads, s.dim, s.vdim)
+        if b.decode:
+            o = K.gla_step(*low, state, b.state_slots, self.norm.data, self.eps, b.B, *sizes)
+        else:
+            r = K.gla_prep(*low, b.lens, b.B, b.S, *sizes)
+            o = K.gla_scan(r, state, b.state_slots, b.lens, b.B, b.S, *sizes, b.pos0 > 0)
+            o = K.gated_norm(o, p[:, 2 * self.hd + self.hv:2 * (self.hd + self.hv)], self.norm.data, self.eps)
+        return lin(o, self.source, "o", self.o)
+
+
+class LatentAttention(Sublayer):
     """Attention without positions over one cached latent per token, with an output gate per head."""
     linear_names = ("proj", "o")
 
     def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
-        super().__init__()
-        self.spec, self.eps, self.index = spec, eps, index
+        super().__init__(index)
+        self.spec, self.eps = spec, eps
         kw = dict(device=device, dtype=dtype)
         self.nq, self.nv = spec.heads * spec.dim, spec.heads * spec.vdim
         self.proj = _param(self.nq + spec.kv_rank + spec.heads, hidden, **kw)
@@ -177,12 +286,9 @@ class LatentAttention(nn.Module):
         yield "g", self.proj.data[a:]
         yield "o", self.o.data
 
-    def finalize(self):
-        pass
-
     def forward(self, h, b: StepBatch, cache, rope, lin, kv):
         s, i = self.spec, self.index
-        p = lin(h, i, "proj", self.proj)
+        p = lin(h, self.source, "proj", self.proj)
         q, gate = p[:, :self.nq], p[:, self.nq + s.kv_rank:]
         pool = cache.latent[i]
         c = K.latent_append(p[:, self.nq:self.nq + s.kv_rank], self.norm.data, self.eps, b.slots, pool, want_rows=not b.decode and b.pos0 == 0)
@@ -195,17 +301,18 @@ class LatentAttention(nn.Module):
             if b.pos0:                         # the latents of the whole sequence so far, this portion's included
                 n = b.pos0 + b.S
                 c = K.gather_rows(pool, b.pages, 0, n)[:, :s.kv_rank]
-            e = lin(c, i, "ukv", self.ukv)
+            e = lin(c, self.source, "ukv", self.ukv)
             o = K.head_attn(q, e[:, :self.nq], e[:, self.nq:], b.B, b.S, n, s.heads, s.heads, s.dim, s.vdim, s.scale, gate)
-        return lin(o, i, "o", self.o)
+        return lin(o, self.source, "o", self.o)
 
 
-class GatedMLP(nn.Module):
+class GatedMLP(Sublayer):
     linear_names = ("gate_up", "down")
+    act = "silu"
 
     def __init__(self, hidden: int, ff: int, index: int, device, dtype):
-        super().__init__()
-        self.ff, self.index = ff, index
+        super().__init__(index)
+        self.ff = ff
         self.gate_up = _param(2 * ff, hidden, device=device, dtype=dtype)
         self.down = _param(hidden, ff, device=device, dtype=dtype)
 
@@ -215,16 +322,19 @@ class GatedMLP(nn.Module):
         yield "down", self.down.data
 
     def forward(self, h, lin):
-        return lin(K.glu_silu(lin(h, self.index, "gate_up", self.gate_up)), self.index, "down", self.down)
+        return lin(K.glu(lin(h, self.source, "gate_up", self.gate_up), self.act), self.source, "down", self.down)
 
 
-class SquaredMLP(nn.Module):
+class GeluMLP(GatedMLP):
+    act = "gelu_tanh"
+
+
+class SquaredMLP(Sublayer):
     """down(relu(up h)^2)."""
     linear_names = ("up", "down")
 
     def __init__(self, hidden: int, ff: int, index: int, device, dtype):
-        super().__init__()
-        self.index = index
+        super().__init__(index)
         self.up, self.down = _param(ff, hidden, device=device, dtype=dtype), _param(hidden, ff, device=device, dtype=dtype)
 
     def tensors(self):
@@ -232,17 +342,19 @@ class SquaredMLP(nn.Module):
         yield "down", self.down.data
 
     def forward(self, h, lin):
-        return lin(lin(h, self.index, "up", self.up, act="relu2"), self.index, "down", self.down)
+        return lin(lin(h, self.source, "up", self.up, act="relu2"), self.source, "down", self.down)
 
 
-class MixtureMLP(nn.Module):
-    """Gated experts chosen per token, and a gated expert that every token runs."""
+class MixtureMLP(Sublayer):
+    """Gated experts chosen per token, and a gated expert that every token runs (with ``shared_gate`` times the sigmoid of one more
+    row of the router's matrix)."""
 
     def __init__(self, hidden: int, spec, index: int, device, dtype):
-        super().__init__()
-        self.spec, self.index = spec, index
+        super().__init__(index)
+        self.spec = spec
         kw = dict(device=device, dtype=dtype)
-        self.router, self.router_bias = _param(spec.experts, hidden, **kw), _param(spec.experts, **kw)
+        self.router = _param(spec.experts + int(spec.shared_gate), hidden, **kw)
+        self.router_bias = _param(spec.experts, **kw) if spec.score == "softmax" else None
         self.gate_up, self.down = _param(spec.experts, 2 * spec.ff, hidden, **kw), _param(spec.experts, hidden, spec.ff, **kw)
         self.shared = GatedMLP(hidden, spec.shared_ff, index, device, dtype) if spec.shared_ff else None
 
@@ -252,25 +364,30 @@ class MixtureMLP(nn.Module):
             yield f"e{e}.gate", self.gate_up.data[e, :F]
             yield f"e{e}.up", self.gate_up.data[e, F:]
             yield f"e{e}.down", self.down.data[e]
-        yield "router", self.router.data
-        yield "router.b", self.router_bias.data
+        yield "router", self.router.data[:self.spec.experts]
+        if self.router_bias is not None:
+            yield "router.b", self.router_bias.data
         if self.shared is not None:
             for n, t in self.shared.tensors():
                 yield "shared." + n, t
+        if self.spec.shared_gate:
+            yield "shared.sg", self.router.data[self.spec.experts:]
 
     def forward(self, h, lin):
-        r = X.route(K.linear(h, self.router.data, out_dtype=torch.float32), self.router_bias.data, self.spec.top)
+        s, E = self.spec, self.spec.experts
+        z = K.linear(h, self.router.data, out_dtype=torch.float32)
+        r = X.route(z[:, :E], self.router_bias.data if self.router_bias is not None else None, s.top, s.score, s.groups, s.keep, s.scale)
         g = X.expert_linear(X.expert_rows(h, r), self.gate_up.data, r)
         y = X.expert_linear(X.expert_glu(g, r), self.down.data, r)
-        return X.weighted_sum(y, r, self.shared(h, lin) if self.shared is not None else None)
+        return X.weighted_sum(y, r, self.shared(h, lin) if self.shared is not None else None, z[:, E:] if s.shared_gate else None)
 
 
-MIXERS = {"attention": DiffAttention, "delta": GatedDelta, "latent_attention": LatentAttention}
+MIXERS = {"attention": DiffAttention, "delta": GatedDelta, "latent_attention": LatentAttention, "head_attention": HeadAttention, "gla": GatedLinear}
 
 
 class ResidualLayer(nn.Module):
-    """A mixer and, unless the layer is a mixer alone, a feed-forward.  ``parts`` lists the sublayers with what ``K.res_norm`` does
-    to the input of each (``pre``) and to its output (``post``)."""
+    """A mixer and, unless the layer is a mixer alone, a feed-forward.  ``parts`` lists the groups of sublayers that read the same
+    input, with what ``K.res_norm`` does to that input (``pre``) and to their outputs (``post``)."""
     norm_kind = "rms"
     dense_mlp = GatedMLP
 
@@ -288,10 +405,18 @@ class ResidualLayer(nn.Module):
     def vector(self, name):
         return getattr(self, name.replace(".", "_")).data
 
+    def at(self, index: int):
+        """The same tensors as another layer, with a cache of its own."""
+        l = copy.copy(self)
+        l._modules = dict(self._modules, mixer=self.mixer.at(index))
+        return l
+
     @property
     def linears(self):
-        """{name: matrix} of the layer's products (what a low-bit weight format may replace)."""
+        """{name: matrix} of the layer's own products (what a low-bit weight format may replace)."""
         out = {}
+        if self.mixer.index != self.mixer.source:
+            return out
         for m in (self.mixer, self.mlp):
             m = m.shared if isinstance(m, MixtureMLP) else m
             if m is not None:
@@ -317,9 +442,9 @@ class SandwichLayer(ResidualLayer):
 
     def parts(self):
         v = self.vector
-        yield self.mixer, {"w_pre": v("norm1")}, {"w_post": v("norm1b")}
+        yield (self.mixer,), {"w_pre": v("norm1")}, {"w_post": v("norm1b")}
         if self.mlp is not None:
-            yield self.mlp, {"w_pre": v("norm2")}, {"w_post": v("norm2b")}
+            yield (self.mlp,), {"w_pre": v("norm2")}, {"w_post": v("norm2b")}
 
 
 class OutputNormLayer(ResidualLayer):
@@ -336,7 +461,20 @@ class OutputNormLayer(ResidualLayer):
         for k, m in ((1, self.mixer), (2, self.mlp)):
             if m is not None:
                 w = v(f"norm{k}")
-                yield m, {"cast": w.dtype}, {"w_post": w, "b_post": v(f"norm{k}.b"), "scale_post": v(f"ls{k}")}
+                yield (m,), {"cast": w.dtype}, {"w_post": w, "b_post": v(f"norm{k}.b"), "scale_post": v(f"ls{k}")}
+
+
+class ParallelLayer(ResidualLayer):
+    """One RMS norm (norm1), whose output the mixer and the feed-forward both read; their sum goes to the residual as it is."""
+    norm_kind = "plain"
+    dense_mlp = GeluMLP
+    final_names = ("final.norm",)
+
+    def vector_names(self):
+        return ("norm1",)
+
+    def parts(self):
+        yield (self.mixer,) if self.mlp is None else (self.mixer, self.mlp), {"w_pre": self.vector("norm1")}, {}
 
 
 def _plain_linear(x, index, name, w, act=None):
@@ -348,6 +486,7 @@ class StackModel(nn.Module):
     sequences without a cache."""
     kernel_units = K.UNITS
     layer_cls = SandwichLayer
+    embed_norm_name = None       # a norm between the embedding and the residual
     linear, activation = staticmethod(K.linear), staticmethod(K.activation)
     runs_fp32 = True             # every kernel of the pass has a true fp32 form
 
@@ -357,7 +496,9 @@ class StackModel(nn.Module):
         device = torch.device(device if device is not None else "cpu")
         kw = dict(device=device, dtype=dtype)
         self.tok_embeddings = _param(cfg.vocab_size, cfg.hidden_size, **kw)
-        self.layers = nn.ModuleList([self.layer_cls(l, cfg.hidden_size, cfg.norm_eps, i, device, dtype) for i, l in enumerate(cfg.layers)])
+        own = {i: self.layer_cls(l, cfg.hidden_size, cfg.norm_eps, i, device, dtype) for i, l in enumerate(cfg.layers) if l.weights_of is None}
+        self.layers = nn.ModuleList([own[i] if i in own else own[l.weights_of].at(i) for i, l in enumerate(cfg.layers)])
+        self.embed_norm = _param(cfg.hidden_size, **kw) if self.embed_norm_name else None
         self.norm = _param(cfg.hidden_size, **kw)
         self.norm_bias = _param(cfg.hidden_size, **kw) if len(self.layer_cls.final_names) > 1 else None
         self.lm_head = self.tok_embeddings if cfg.tie_embeddings else _param(cfg.vocab_size, cfg.hidden_size, **kw)
@@ -369,7 +510,7 @@ class StackModel(nn.Module):
         """Random weights that keep activations of order one: N(0, 1 / fan-in) matrices, small deviations for the norms, decays
         between about 0.5 and 1."""
         about_one = lambda n: n.endswith(("mix.norm", "dkv.norm")) or \
-            (self.layer_cls.norm_kind == "layer" and n.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2", "ls1", "ls2"))
+            (self.layer_cls.norm_kind != "rms" and n.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2", "ls1", "ls2"))
         g = torch.Generator(device="cpu").manual_seed(seed)
         with torch.no_grad():
             for name, t in self.named_tensors():
@@ -398,8 +539,11 @@ class StackModel(nn.Module):
     def named_tensors(self):
         """(name in the model folder, view into the parameters) pairs."""
         out = [(self.embed_name, self.tok_embeddings.data)]
+        if self.embed_norm is not None:
+            out.append((self.embed_norm_name, self.embed_norm.data))
         for i, l in enumerate(self.layers):
-            out += [(f"l{i}.{n}", t) for n, t in l.tensors()]
+            if l.mixer.source == i:
+                out += [(f"l{i}.{n}", t) for n, t in l.tensors()]
         out += list(zip(self.layer_cls.final_names, (t.data for t in (self.norm, self.norm_bias) if t is not None)))
         return out if self.cfg.tie_embeddings else out + [(self.head_name, self.lm_head.data)]
 
@@ -425,8 +569,8 @@ class StackModel(nn.Module):
         """cos / sin tables of one rotation for at least ``max_pos`` positions."""
         t = self._rope.get(spec)
         if t is None or t[0].shape[0] < max_pos or t[0].device != self.device:
-            mode = "none" if spec.yarn_factor is None else "yarn"
-            t = F.rope_tables(spec.dims, max_pos, spec.base, mode, spec.yarn_factor or 1.0, spec.yarn_original, 1.0, spec.yarn_fast, spec.yarn_slow,
+            mode, factor = ("linear", spec.linear) if spec.yarn_factor is None else ("yarn", spec.yarn_factor)
+            t = F.rope_tables(spec.dims, max_pos, spec.base, mode, factor, spec.yarn_original, 1.0, spec.yarn_fast, spec.yarn_slow,
                               device=self.device, yarn_ramp_max=spec.dims - 1)
             self._rope[spec] = t
         return t
@@ -443,20 +587,24 @@ class StackModel(nn.Module):
         x = torch.empty((n, cfg.hidden_size), dtype=torch.float32, device=self.device)
         parts = [(i, l) + p for i, l in enumerate(self.layers) for p in l.parts()]
         pre = [p[3] for p in parts] + [{"w_pre": self.norm.data, "b_pre": self.norm_bias.data if self.norm_bias is not None else None}]
-        h = K.res_norm(x, eps, ids=b.tokens, table=self.tok_embeddings.data, scale=cfg.embedding_scale, kind=kind, **pre[0])
+        h = K.res_norm(x, eps, ids=b.tokens, table=self.tok_embeddings.data, scale=cfg.embedding_scale, kind=kind,
+                       w_post=self.embed_norm.data if self.embed_norm is not None else None, **pre[0])
         kv = {}
-        for k, (i, l, m, _, post) in enumerate(parts):
-            if m is l.mixer:
-                rope = self.rope(m.spec.rot, max_pos) if m.spec.kind == "attention" else None
-                y = m(h, b, cache, rope, lin, kv)
-            else:
-                y = m(h, lin)
+        for k, (i, l, group, _, post) in enumerate(parts):
+            ys = []
+            for m in group:
+                if m is l.mixer:
+                    rot = getattr(m.spec, "rot", None)
+                    ys.append(m(h, b, cache, self.rope(rot, max_pos) if rot is not None else None, lin, kv))
+                else:
+                    ys.append(m(h, lin))
+            post = dict(post, y=ys[0], y2=ys[1] if len(ys) > 1 else None)
             last = k + 1 == len(parts)
             if residuals is not None and (last or parts[k + 1][0] != i):
                 z = x.clone()
-                K.res_norm(z, eps, y=y, kind=kind, **post)
+                K.res_norm(z, eps, kind=kind, **post)
                 residuals.append(z)
-            h = K.res_norm(x, eps, y=y, kind=kind, row_index=row_index if last else None, **post, **pre[k + 1])
+            h = K.res_norm(x, eps, kind=kind, row_index=row_index if last else None, **post, **pre[k + 1])
         return h
 
     def head(self, h):

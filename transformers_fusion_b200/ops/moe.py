@@ -31,11 +31,11 @@ _lib.register("tfb_moe_combine_bwd", [c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_i, c_
 _lib.register("tfb_moe_permute_bwd", [c_p, c_p, c_p, c_i, c_i, c_i, c_p])
 
 
-_lib.register("tfb_moe_route", [c_p, c_p, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_ll, c_i, c_p])
+_lib.register("tfb_moe_route", [c_p, c_p, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_ll, c_i, c_i, c_i, c_i, c_f, c_p])
 _lib.register("tfb_moe_gather", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_moe_glu", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_p])
 _lib.register("tfb_moe_gemm_f32", [c_p, c_ll, c_p, c_ll, c_ll, c_p, c_ll, c_p, c_i, c_i, c_i, c_i, c_p])
-_lib.register("tfb_moe_weighted_sum", [c_p, c_ll, c_p, c_p, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_moe_weighted_sum", [c_p, c_ll, c_p, c_p, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 
 
 class _Group(C.Structure):
@@ -324,16 +324,27 @@ class Routing:
     max_rows: int
 
 
-def route(logits, bias, k) -> Routing:
-    """The k largest of the fp32 logits [T, E] + bias (the lower index first among equals), weighted by the softmax over them."""
+def route(logits, bias, k, score="softmax", groups=1, keep=1, scale=1.0) -> Routing:
+    """The k largest of the fp32 logits [T, E] (+ bias) (the lower index first among equals), weighted by the softmax over them.
+    ``score`` "sigmoid": the k largest sigmoids among the experts of the ``keep`` best of ``groups`` equal groups of neighbours (by the
+    sum of a group's two largest), weighted by them over their sum, times ``scale``."""
     T, E = logits.shape
     assert logits.dtype == torch.float32
     tiles = T * k // 128 + min(E, T * k)       # enough for any distribution of the assignments
     dev = logits.device
     if not logits.is_cuda:
-        z = logits + bias.float()
-        idx = torch.argsort(z, dim=-1, descending=True, stable=True)[:, :k]
-        w = torch.softmax(z.gather(1, idx), -1)
+        z = logits if bias is None else logits + bias.float()
+        if score == "sigmoid":
+            z = torch.sigmoid(z)
+            mark = z.reshape(T, groups, -1).topk(min(2, E // groups), -1).values.sum(-1)
+            best = torch.argsort(mark, dim=-1, descending=True, stable=True)[:, :keep]
+            kept = torch.zeros(T, groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(E // groups, 1)
+            idx = torch.argsort(z.masked_fill(~kept, -1.0), dim=-1, descending=True, stable=True)[:, :k]
+            w = z.gather(1, idx)
+            w = w / (w.sum(-1, keepdim=True) + 1e-20) * scale
+        else:
+            idx = torch.argsort(z, dim=-1, descending=True, stable=True)[:, :k]
+            w = torch.softmax(z.gather(1, idx), -1)
         row_of, of_tile, off = torch.empty(T * k, dtype=torch.int32), [], 0
         flat = idx.reshape(-1)
         for e in range(E):
@@ -347,9 +358,10 @@ def route(logits, bias, k) -> Routing:
     i32 = lambda *s: torch.empty(s, dtype=torch.int32, device=dev)
     r = Routing(i32(T, k), torch.empty((T, k), dtype=torch.float32, device=dev), i32(T, k), i32(tiles), tiles * 128)
     rank, counts = i32(T, k), i32(E)
-    check(_lib.lib().tfb_moe_route(logits.data_ptr(), bias.data_ptr(), T, E, k, r.idx.data_ptr(), r.w.data_ptr(), r.row_of.data_ptr(),
+    check(_lib.lib().tfb_moe_route(logits.data_ptr(), ptr(bias), T, E, k, r.idx.data_ptr(), r.w.data_ptr(), r.row_of.data_ptr(),
                                    r.expert_of_tile.data_ptr(), counts.data_ptr(), rank.data_ptr(), tiles,
-                                   logits.stride(0), int(bias.dtype == torch.float32), stream()), "moe_route", 1 if T <= 256 else 2)
+                                   logits.stride(0), int(bias is not None and bias.dtype == torch.float32), int(score == "sigmoid"), groups, keep,
+                                   float(scale), stream()), "moe_route", 1 if T <= 256 else 2)
     return r
 
 
@@ -406,15 +418,19 @@ def expert_glu(gu, r: Routing):
     return out
 
 
-def weighted_sum(yp, r: Routing, base=None):
-    """sum_k w[t, k] * yp[row_of[t, k]] (+ base[t])."""
+def weighted_sum(yp, r: Routing, base=None, base_gate=None):
+    """sum_k w[t, k] * yp[row_of[t, k]] (+ base[t], times sigmoid(base_gate[t]): fp32 logits [T, 1])."""
     T, k = r.idx.shape
     H = yp.shape[1]
     if not yp.is_cuda:
         y = (yp[r.row_of.reshape(-1).long()].view(T, k, H).float() * r.w[..., None]).sum(1)
-        return (y if base is None else y + base.float()).to(yp.dtype)
+        if base is not None:
+            y = y + (base.float() if base_gate is None else base.float() * torch.sigmoid(base_gate))
+        return y.to(yp.dtype)
     y = _out_rows(T, H, yp)
+    assert base_gate is None or base_gate.dtype == torch.float32
     check(_lib.lib().tfb_moe_weighted_sum(yp.data_ptr(), yp.stride(0), r.row_of.data_ptr(), r.w.data_ptr(), ptr(base),
-                                          base.stride(0) if base is not None else 0, y.data_ptr(), y.stride(0), T, k, H, _is32(yp), stream()),
+                                          base.stride(0) if base is not None else 0, ptr(base_gate),
+                                          base_gate.stride(0) if base_gate is not None else 0, y.data_ptr(), y.stride(0), T, k, H, _is32(yp), stream()),
           "moe_weighted_sum")
     return y

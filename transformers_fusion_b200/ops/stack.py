@@ -1,14 +1,15 @@
 """Raw operators of decoders that are a stack of different sequence mixers over a 32-bit residual stream: norms around
-every sublayer, partial rotary embedding, differential attention, latent attention, gated delta rule, true fp32 products.
+every sublayer, partial rotary embedding, differential attention, softmax attention with options, latent attention, gated delta rule, gated linear
+attention, true fp32 products.
 
-As in ``functional``: CUDA tensors go to the sm_100a kernels (``csrc/kernels/stack_ops.cu``, ``diff_attention.cu``,
-``latent_attention.cu``, ``delta_rule.cu``), CPU tensors run the plain PyTorch statement of the same math.  Activations are bf16 or fp32 (the dtype of
+As in ``functional``: CUDA tensors go to the sm_100a kernels (``csrc/kernels/stack_ops.cu``, ``diff_attention.cu``, ``head_attention.cu``,
+``latent_attention.cu``, ``delta_rule.cu``, ``gated_linear.cu``), CPU tensors run the plain PyTorch statement of the same math.  Activations are bf16 or fp32 (the dtype of
 the tensors decides); the residual, norms, rotation, attention scores and weights, and the recurrence are fp32 in both."""
 from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Optional
+from typing import NamedTuple, Optional
 
 import torch
 
@@ -17,13 +18,17 @@ from . import functional as F
 from ._lib import c_f, c_i, c_ll, c_p, check, ptr, stream
 
 UNITS = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "diff_attention", "delta_rule")    # translation units these operators need
-UNITS_LATENT = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "latent_attention", "moe_serve")
+UNITS_LATENT = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "head_attention", "latent_attention", "moe_serve")
+UNITS_GATED = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "head_attention", "gated_linear", "delta_rule", "moe_serve")
 PAGE = 16
 ACT = {None: 0, "relu2": 4}      # codes of the product epilogues (gemm_bf16.cu: apply_act)
+GLU = {"silu": 0, "gelu_tanh": 1}
+NORM = {"rms": 0, "layer": 1, "plain": 2}
 
-_lib.register("tfb_res_norm", [c_p, c_p, c_ll, c_f, c_i, c_p, c_ll, c_p, c_ll, c_p, c_p, c_p, c_p, c_p, c_p, c_ll, c_p, c_i, c_i, c_f, c_i, c_i, c_p])
-_lib.register("tfb_glu_silu", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_p])
+_lib.register("tfb_res_norm", [c_p, c_p, c_ll, c_f, c_i, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_p, c_p, c_p, c_p, c_p, c_ll, c_p, c_i, c_i, c_f, c_i, c_i, c_p])
+_lib.register("tfb_glu", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_rope_append", [c_p, c_ll, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_norm_rope_append", [c_p, c_ll, c_p, c_p, c_f, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_gather_rows", [c_p, c_ll, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p])
 _lib.register("tfb_gemm_f32", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_skinny_fits", [c_i, c_i, c_i])
@@ -33,7 +38,14 @@ _lib.register("tfb_latent_append", [c_p, c_ll, c_p, c_f, c_p, c_p, c_ll, c_p, c_
 _lib.register("tfb_head_linear", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_skinny_linear_heads", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_gemm_f32_heads", [c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
-_lib.register("tfb_head_attn", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p])
+_lib.register("tfb_head_attn", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_f, c_i,
+                                c_f, c_i, c_i, c_i, c_p, c_p])
+_lib.register("tfb_head_decode_blocks", [c_i, c_i, c_i, c_i, c_i])
+_lib.register("tfb_head_decode", [c_p, c_ll, c_p, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_ll, c_i, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
+                                  c_i, c_i, c_f, c_i, c_f, c_i, c_i, c_p, c_p])
+_lib.register("tfb_gla_prep", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_f, c_p] + [c_p] * 5 + [c_i] * 7 + [c_p])
+_lib.register("tfb_gla_scan", [c_p] * 7 + [c_i, c_p] + [c_i] * 6 + [c_p, c_p, c_p])
+_lib.register("tfb_gla_step", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_f, c_p, c_p, c_i, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_latent_decode_plan", [c_i, c_i, c_i, c_i, c_i])
 _lib.register("tfb_latent_decode", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p])
 _lib.register("tfb_diff_attn_fwd", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_f, c_f, c_i,
@@ -109,24 +121,34 @@ def centred_rms(x, w, eps):
     return xf / torch.sqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * (1 + w.float())
 
 
+def plain_rms(x, w, eps):
+    xf = x.float()
+    return xf / torch.sqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+
 def layer_norm(x, w, b, eps):
     d = x.float()
     d = d - d.mean(-1, keepdim=True)
     return d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w.float() + b.float()
 
 
-def res_norm(x, eps, *, y=None, w_post=None, b_post=None, scale_post=None, w_pre=None, b_pre=None, cast=None, ids=None, table=None, scale=1.0,
-             row_index=None, dtype=None, kind="rms"):
-    """x += norm(y; w_post, b_post) * scale_post on the fp32 residual ``x`` [n, H] in place; returns norm(x; w_pre, b_pre) in the
-    activation dtype, x itself in the dtype ``cast`` without ``w_pre``, None without both.  ``kind``: "rms" (weights are
-    deviations from one, no bias) or "layer".  ``ids``: x starts as scale * table[ids].  ``row_index`` (int32): only those
-    rows are computed and returned, and x keeps its values."""
+def res_norm(x, eps, *, y=None, y2=None, w_post=None, b_post=None, scale_post=None, w_pre=None, b_pre=None, cast=None, ids=None, table=None,
+             scale=1.0, row_index=None, dtype=None, kind="rms"):
+    """x += norm(y; w_post, b_post) * scale_post + y2 on the fp32 residual ``x`` [n, H] in place (y itself without ``w_post``); returns
+    norm(x; w_pre, b_pre) in the activation dtype, x itself in the dtype ``cast`` without ``w_pre``, None without both.  ``kind``:
+    "rms" (weights are deviations from one, no bias), "plain" (weights themselves, no bias) or "layer".  ``ids``: x starts as
+    scale * table[ids], normed with ``w_post`` if there is no y.  ``row_index`` (int32): only those rows are computed and
+    returned, and x keeps its values."""
     if not x.is_cuda:
-        norm = (lambda t, w, b: centred_rms(t, w, eps)) if kind == "rms" else (lambda t, w, b: layer_norm(t, w, b, eps))
+        norm = {"rms": lambda t, w, b: centred_rms(t, w, eps), "plain": lambda t, w, b: plain_rms(t, w, eps),
+                "layer": lambda t, w, b: layer_norm(t, w, b, eps)}[kind]
         v = table[ids.long()].float() * scale if ids is not None else x
+        if y is None and w_post is not None:
+            v = norm(v, w_post, b_post)
         if y is not None:
-            z = norm(y, w_post, b_post)
-            v = v + (z if scale_post is None else z * scale_post.float())
+            z = y.float() if w_post is None else norm(y, w_post, b_post)
+            z = z if scale_post is None else z * scale_post.float()
+            v = v + (z if y2 is None else z + y2.float())
         if row_index is None:
             x.copy_(v)
         else:
@@ -136,48 +158,65 @@ def res_norm(x, eps, *, y=None, w_post=None, b_post=None, scale_post=None, w_pre
         return norm(v, w_pre, b_pre).to(dtype or w_pre.dtype)
     H = x.shape[1]
     n = x.shape[0] if row_index is None else row_index.shape[0]
-    w = next(t for t in (w_pre, w_post, table) if t is not None)
+    w = next(t for t in (w_pre, w_post, table, y) if t is not None)
     a = rows(n, H, w.dtype if w_pre is not None else cast, x.device) if w_pre is not None or cast is not None else None
-    assert kind in ("rms", "layer") and (a is None or a.dtype == w.dtype)
+    assert (a is None or a.dtype == w.dtype) and (y2 is None or (y is not None and y2.dtype == y.dtype))
     check(_lib.lib().tfb_res_norm(ptr(ids), ptr(table), table.stride(0) if table is not None else 0, float(scale),
                                   table.shape[0] if table is not None else 0, x.data_ptr(), x.stride(0), ptr(y),
-                                  y.stride(0) if y is not None else 0, ptr(w_post), ptr(b_post), ptr(scale_post), ptr(w_pre), ptr(b_pre), ptr(a),
-                                  a.stride(0) if a is not None else 0, ptr(row_index), n, H, float(eps), int(kind == "layer"), _f32(w), stream()),
+                                  y.stride(0) if y is not None else 0, ptr(y2), y2.stride(0) if y2 is not None else 0, ptr(w_post), ptr(b_post), ptr(scale_post), ptr(w_pre), ptr(b_pre), ptr(a),
+                                  a.stride(0) if a is not None else 0, ptr(row_index), n, H, float(eps), NORM[kind], _f32(w), stream()),
           "res_norm")
     return a
 
 
 def glu_silu(gu):
-    """[gate | up] -> silu(gate) * up."""
+    return glu(gu, "silu")
+
+
+def glu(gu, act):
+    """[gate | up] -> act(gate) * up; ``act``: "silu" or "gelu_tanh"."""
     M, F2 = gu.shape
     Fh = F2 // 2
     if not gu.is_cuda:
         g = gu[:, :Fh].float()
-        return (g * torch.sigmoid(g) * gu[:, Fh:].float()).to(gu.dtype)
+        g = g * torch.sigmoid(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
+        return (g * gu[:, Fh:].float()).to(gu.dtype)
     out = rows(M, Fh, gu.dtype, gu.device)
-    check(_lib.lib().tfb_glu_silu(gu.data_ptr(), gu.stride(0), out.data_ptr(), out.stride(0), M, Fh, _f32(gu), stream()), "glu_silu")
+    check(_lib.lib().tfb_glu(gu.data_ptr(), gu.stride(0), out.data_ptr(), out.stride(0), M, Fh, GLU[act], _f32(gu), stream()), "glu")
     return out
 
 
 # ---------------------------------------------------------------------------------------------------- rotation + cache
-def rope_append(qkv, tables, positions, nq, nk, D, dims, v_cols, slots=None, kpool=None, vpool=None):
-    """Rotate the first ``dims`` entries of the nq query and nk key heads of every row of ``qkv`` ([q | k | v]) in place and
-    write k and v to flat slots of the pools ([slots, nk * D], [slots, v_cols]; negative slots are not cached)."""
-    cos, sin = tables
+def rope_append(qkv, tables, positions, nq, nk, D, dims, v_cols, slots=None, kpool=None, vpool=None, norms=None):
+    """Rotate the first ``dims`` entries of the nq query and nk key heads of every row of ``qkv`` ([q | k | v | ...]) in place and
+    write k and v to flat slots of the pools ([slots, nk * D], [slots, v_cols]; negative slots are not cached).  ``norms``
+    (weights of the queries, of the keys, eps): every head is divided by its root mean square and weighted first.  ``dims`` 0:
+    no rotation (``tables`` None)."""
+    cos, sin = tables or (None, None)
     T = qkv.shape[0]
     if not qkv.is_cuda:
         half = dims // 2
-        c, s = cos[positions.long()][:, None], sin[positions.long()][:, None]
         x = qkv[:, :(nq + nk) * D].reshape(T, nq + nk, D).float()
-        u, v = x[..., :half], x[..., half:dims]
-        x = torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], -1)
-        qkv[:, :(nq + nk) * D] = x.reshape(T, -1).to(qkv.dtype)
+        if norms:
+            x = torch.cat([plain_rms(x[:, :nq], norms[0], norms[2]), plain_rms(x[:, nq:], norms[1], norms[2])], 1)
+        if dims:
+            c, s = cos[positions.long()][:, None], sin[positions.long()][:, None]
+            u, v = x[..., :half], x[..., half:dims]
+            x = torch.cat([u * c - v * s, v * c + u * s, x[..., dims:]], -1)
+        if norms or dims:
+            qkv[:, :(nq + nk) * D] = x.reshape(T, -1).to(qkv.dtype)
         if nk and slots is not None:
             keep = slots >= 0
             kpool[slots[keep]] = qkv[keep, nq * D:(nq + nk) * D]
             vpool[slots[keep]] = qkv[keep, (nq + nk) * D:(nq + nk) * D + v_cols]
         return qkv
-    check(_lib.lib().tfb_rope_append(qkv.data_ptr(), qkv.stride(0), cos.data_ptr(), sin.data_ptr(), cos.shape[0], positions.data_ptr(),
+    if norms:
+        check(_lib.lib().tfb_norm_rope_append(qkv.data_ptr(), qkv.stride(0), norms[0].data_ptr(), norms[1].data_ptr(), float(norms[2]), ptr(cos),
+                                              ptr(sin), cos.shape[0] if dims else 0, positions.data_ptr(), ptr(slots), ptr(kpool), ptr(vpool),
+                                              kpool.shape[0] if kpool is not None else 0, T, nq, nk, D, dims, v_cols, _f32(qkv), stream()),
+              "norm_rope_append")
+        return qkv
+    check(_lib.lib().tfb_rope_append(qkv.data_ptr(), qkv.stride(0), ptr(cos), ptr(sin), cos.shape[0] if dims else 0, positions.data_ptr(),
                                      ptr(slots), ptr(kpool), ptr(vpool), kpool.shape[0] if kpool is not None else 0, T, nq, nk, D, dims,
                                      v_cols, _f32(qkv), stream()), "rope_append")
     return qkv
@@ -255,6 +294,92 @@ def diff_decode(q, kpool, vpool, block_table, positions, H, G, D, V, window, sca
     return o
 
 
+# ---------------------------------------------------------------------------------------------------- softmax attention with options
+class HeadOptions(NamedTuple):
+    """``window`` > 0: a query sees that many keys up to its own, and the first ``keep_first`` of the sequence; ``softcap`` > 0: scores
+    become cap tanh(score / cap); ``sink``: one more key of score 0 in the denominator; the query at position p is multiplied by
+    1 + temp_coef ln(floor((p + 1) / temp_every) + 1)."""
+    window: int = 0
+    keep_first: int = 0
+    softcap: float = 0.0
+    sink: bool = False
+    temp_coef: float = 0.0
+    temp_every: int = 1
+
+
+PLAIN = HeadOptions()
+
+
+def _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None, opt=PLAIN, pos0=0):
+    R = H // G
+    Q = q.reshape(B, S, H, D).transpose(1, 2).float()
+    K = k.reshape(B, Skv, G, D).transpose(1, 2).float().repeat_interleave(R, 1)
+    W = v.reshape(B, Skv, G, V).transpose(1, 2).float().repeat_interleave(R, 1)
+    i, j = torch.arange(S)[:, None] + (Skv - S), torch.arange(Skv)[None]
+    hide = j > i
+    if opt.window:
+        hide = hide | ((i - j >= opt.window) & (j >= opt.keep_first))
+    temp = 1 + opt.temp_coef * torch.log(((torch.arange(S) + pos0 + 1) // opt.temp_every + 1).float())
+    s = Q * temp[:, None] @ K.transpose(-1, -2) * scale
+    if opt.softcap:
+        s = opt.softcap * torch.tanh(s / opt.softcap)
+    s = s.masked_fill(hide, -math.inf)
+    if opt.sink:
+        s = torch.cat([s, torch.zeros(B, H, S, 1)], -1)
+        W = torch.cat([W, torch.zeros(B, H, 1, V)], 2)
+    o = (torch.softmax(s, -1) @ W).transpose(1, 2)                                 # [B, S, H, V]
+    if gate is not None:
+        o = o * torch.sigmoid(gate.float()).reshape(B, S, H, -1)
+    return o.reshape(B * S, H * V).to(q.dtype)
+
+
+def head_attn(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None, opt=PLAIN, pos0=0):
+    """Causal softmax attention of B prompts whose keys and values may have different sizes.  q [B*S, H D], k [B*Skv, G D],
+    v [B*Skv, G V]; the queries are the last S of the Skv keys and stand at positions pos0 ... (with a window, keys between the
+    kept ones and the window of the first query may be left out); ``gate`` [B*S, H] or [B*S, H V]: heads, or their entries, are
+    multiplied by its sigmoid.  Returns [B*S, H V]."""
+    if not q.is_cuda:
+        return _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate, opt, pos0)
+    o = rows(B * S, H * V, q.dtype, q.device)
+    check(_lib.lib().tfb_head_attn(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), o.data_ptr(), o.stride(0),
+                                   ptr(gate), gate.stride(0) if gate is not None else 0, int(gate is not None and gate.shape[1] != H), B, S, Skv, H,
+                                   G, D, V, float(scale), opt.window, opt.keep_first, opt.softcap, int(opt.sink), opt.temp_coef, opt.temp_every, pos0,
+                                   _f32(q), _lib.status_word(q.device).data_ptr(), stream()), "head_attn")
+    return o
+
+
+def head_decode(q, kpool, vpool, block_table, positions, H, G, D, V, scale, gate=None, opt=PLAIN, splits: Optional[int] = None):
+    """One query per sequence (q [B, H D] at ``positions``) over its cached rows (pools [slots, G D] and [slots, G V]); ``gate`` [B, H]
+    or [B, H V]."""
+    B = q.shape[0]
+    if not q.is_cuda:
+        out = torch.zeros((B, H * V), dtype=q.dtype)
+        for b in range(B):
+            n = int(positions[b]) + 1
+            lo = max(0, n - opt.window) if opt.window else 0
+            p = torch.cat([torch.arange(min(opt.keep_first, lo)), torch.arange(lo, n)])
+            s = block_table[b, (p // PAGE).long()].long() * PAGE + p % PAGE
+            out[b] = _head_attn_ref(q[b:b + 1], kpool[s], vpool[s], 1, 1, len(p), H, G, D, V, scale, gate[b:b + 1] if gate is not None else None, opt,
+                                    n - 1)[0]
+        return out
+    L, f32 = _lib.lib(), _f32(q)
+    o = rows(B, H * V, q.dtype, q.device)
+    acc = ml = None
+    n = L.tfb_head_decode_blocks(H, G, D, V, f32)        # blocks per sequence of the tensor-core form, 0: the other form
+    if n and q.stride(0) % 8 == 0:
+        keys = block_table.shape[1] * PAGE
+        keys = min(keys, opt.window + opt.keep_first) if opt.window else keys
+        splits = splits or max(1, min(32, (4 * 148) // (B * n), keys // 128))
+        acc = torch.empty(B * H * splits * V, dtype=torch.float32, device=q.device)
+        ml = torch.empty(B * H * splits * 2, dtype=torch.float32, device=q.device)
+    check(L.tfb_head_decode(q.data_ptr(), q.stride(0), kpool.data_ptr(), vpool.data_ptr(), kpool.shape[0], block_table.data_ptr(),
+                            block_table.shape[1], PAGE, positions.data_ptr(), o.data_ptr(), o.stride(0), ptr(gate),
+                            gate.stride(0) if gate is not None else 0, int(gate is not None and gate.shape[1] != H), ptr(acc), ptr(ml), splits or 1, B,
+                            H, G, D, V, float(scale), opt.window, opt.keep_first, opt.softcap, int(opt.sink), opt.temp_coef, opt.temp_every, f32,
+                            _lib.status_word(q.device).data_ptr(), stream()), "head_decode", 2 if acc is not None else 1)
+    return o
+
+
 # ---------------------------------------------------------------------------------------------------- latent attention
 def latent_append(c, w, eps, slots, pool, want_rows=True):
     """Rows c [T, R] divided by their root mean square and weighted with w, written to flat slots of ``pool`` [slots, R padded to 8]
@@ -306,31 +431,6 @@ def head_linear(x, w, heads, k, n, gate=None, transposed=False):
         check(L.tfb_skinny_linear_heads(x.data_ptr(), x.stride(0), x_head, w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), ptr(gate),
                                         gate.stride(0) if gate is not None else 0, M, heads, n, k8, 0, stream()), "skinny_linear_heads")
     return out
-
-
-def _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None):
-    R = H // G
-    Q = q.reshape(B, S, H, D).transpose(1, 2).float()
-    K = k.reshape(B, Skv, G, D).transpose(1, 2).float().repeat_interleave(R, 1)
-    W = v.reshape(B, Skv, G, V).transpose(1, 2).float().repeat_interleave(R, 1)
-    hide = torch.arange(Skv)[None] > torch.arange(S)[:, None] + (Skv - S)
-    o = (torch.softmax((Q @ K.transpose(-1, -2) * scale).masked_fill(hide, -math.inf), -1) @ W).transpose(1, 2)        # [B, S, H, V]
-    if gate is not None:
-        o = o * torch.sigmoid(gate.float()).reshape(B, S, H, 1)
-    return o.reshape(B * S, H * V).to(q.dtype)
-
-
-def head_attn(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None):
-    """Causal softmax attention of B prompts whose keys and values may have different sizes.  q [B*S, H D], k [B*Skv, G D],
-    v [B*Skv, G V]; the queries are the last S of the Skv positions; ``gate`` [B*S, H]: head h is multiplied by
-    sigmoid(gate[:, h]).  Returns [B*S, H V]."""
-    if not q.is_cuda:
-        return _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate)
-    o = rows(B * S, H * V, q.dtype, q.device)
-    check(_lib.lib().tfb_head_attn(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), o.data_ptr(), o.stride(0),
-                                   ptr(gate), gate.stride(0) if gate is not None else 0, B, S, Skv, H, G, D, V, float(scale), _f32(q),
-                                   _lib.status_word(q.device).data_ptr(), stream()), "head_attn")
-    return o
 
 
 def latent_decode(q, pool, block_table, positions, H, R, scale, splits: Optional[int] = None):
@@ -466,4 +566,71 @@ def delta_step(rows_: DeltaRows, state, state_slots, gate, w, eps, B, G, H, D, V
     check(_lib.lib().tfb_delta_step(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.pair.data_ptr(), r.decay.data_ptr(), r.beta.data_ptr(),
                                     state.data_ptr(), state_slots.data_ptr(), state.shape[0], gate.data_ptr(), gate.stride(0), w.data_ptr(),
                                     out.data_ptr(), out.stride(0), B, G, H, D, V, int(has_past), float(eps), _f32(gate), stream()), "delta_step")
+    return out
+
+
+# ---------------------------------------------------------------------------------------------------- gated linear attention
+@dataclass
+class GlaRows:
+    """Prepared rows of B sequences.  On CUDA the scan's own layouts (see csrc/kernels/gated_linear.cu): per four tokens queries times
+    the decays up to them, keys times those behind them, the decay over all four, and the products between them; on the CPU q, k,
+    decay [T, H, D], v [T, H, V]."""
+    q: torch.Tensor
+    k: torch.Tensor
+    v: torch.Tensor
+    decay: torch.Tensor
+    pair: Optional[torch.Tensor] = None
+
+
+def gla_prep(proj, a2, bias, tau, lens, B, S, H, D, V) -> GlaRows:
+    """proj [B*S, 2 H D + 2 H V + rank] = q | k | v | gate | a1, a2 [H D, rank], bias [H D]: scaled queries, decays
+    sigmoid(a2 a1 + bias)^(1/tau) and rows for ``gla_scan``, all fp32."""
+    if not proj.is_cuda:
+        T, n = proj.shape[0], H * D
+        x = proj.float()
+        z = x[:, 2 * n + 2 * H * V:] @ a2.float().t() + bias.float()
+        return GlaRows(x[:, :n].reshape(T, H, D) * D ** -0.5, x[:, n:2 * n].reshape(T, H, D), x[:, 2 * n:2 * n + H * V].reshape(T, H, V),
+                       torch.exp(torch.nn.functional.logsigmoid(z) / tau).reshape(T, H, D))
+    L = _lib.lib()
+    Dp, Vp, n4 = L.tfb_delta_padded_dim(D), (V + 3) // 4 * 4, (S + 3) // 4
+    e = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
+    r = GlaRows(e(B, H, 4 * n4, Dp), e(B, H, 4 * n4, Dp), e(B, H, 4 * n4, Vp), e(B, H, n4, Dp), e(B, H, n4, 16))
+    check(L.tfb_gla_prep(proj.data_ptr(), proj.stride(0), a2.data_ptr(), a2.stride(0), bias.data_ptr(), a2.shape[1], float(tau), ptr(lens),
+                         r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.decay.data_ptr(), r.pair.data_ptr(), B, S, H, D, Dp, V, _f32(proj),
+                         stream()), "gla_prep")
+    return r
+
+
+def gla_scan(rows_: GlaRows, state, state_slots, lens, B, S, H, D, V, has_past):
+    """S <- diag(decay) S + k v^T, o = S^T q over prepared rows; ``state`` [slots, H, D, V] fp32 is read (``has_past``) and updated.
+    Returns fp32 [B*S, H, V] (rows past a sequence's length are unspecified)."""
+    r = rows_
+    if not r.q.is_cuda:
+        out = torch.zeros(B * S, H, V)
+        n = lens if lens is not None else torch.full((B,), S)
+        for b in range(B):
+            sl = int(state_slots[b])
+            st = state[sl].clone() if has_past and sl >= 0 else torch.zeros(H, D, V)
+            for t in range(b * S, b * S + int(n[b])):
+                st = st * r.decay[t][..., None] + r.k[t][..., None] * r.v[t][:, None]
+                out[t] = torch.einsum("hdv,hd->hv", st, r.q[t])
+            if sl >= 0:
+                state[sl] = st
+        return out
+    o = torch.empty((B * S, H, V), dtype=torch.float32, device=r.q.device)
+    check(_lib.lib().tfb_gla_scan(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.decay.data_ptr(), r.pair.data_ptr(), o.data_ptr(),
+                                  state.data_ptr(), state.shape[0], state_slots.data_ptr(), B, S, H, D, V, int(has_past), ptr(lens),
+                                  _lib.status_word(o.device).data_ptr(), stream()), "gla_scan")
+    return o
+
+
+def gla_step(proj, a2, bias, tau, state, state_slots, w, eps, B, H, D, V):
+    """One token per sequence: decays, recurrence and the gated norm of its output; [B, H V]."""
+    gate = proj[:, 2 * H * D + H * V:2 * H * D + 2 * H * V]
+    if not proj.is_cuda or not _step_fits(D, V):
+        return gated_norm(gla_scan(gla_prep(proj, a2, bias, tau, None, B, 1, H, D, V), state, state_slots, None, B, 1, H, D, V, True), gate, w, eps)
+    out = rows(B, H * V, proj.dtype, proj.device)
+    check(_lib.lib().tfb_gla_step(proj.data_ptr(), proj.stride(0), a2.data_ptr(), a2.stride(0), bias.data_ptr(), a2.shape[1], float(tau),
+                                  state.data_ptr(), state_slots.data_ptr(), state.shape[0], w.data_ptr(), out.data_ptr(), out.stride(0), B, H, D, V,
+                                  float(eps), _f32(proj), stream()), "gla_step")
     return out
