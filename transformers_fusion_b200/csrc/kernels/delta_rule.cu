@@ -300,28 +300,6 @@ struct DeltaScanArgs {
   int* status;
 };
 
-typedef unsigned long long u64;
-__device__ __forceinline__ u64 fma2(u64 a, u64 b, u64 c) {
-  u64 d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ u64 mul2(u64 a, u64 b) {
-  u64 d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ u64 pack2(float lo, float hi) {
-  u64 d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ float2 unpack2(u64 v) {
-  float2 f;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
-  return f;
-}
-
 constexpr int SCAN_CHUNK = 16;   // tokens per shared-memory stage
 
 // EPT: entries of one column per thread (a multiple of 4); TPC: threads per column group; CPT: columns per group (a power of

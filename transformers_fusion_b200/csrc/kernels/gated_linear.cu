@@ -1,0 +1,535 @@
+// Gated linear attention (a matrix state per head whose rows decay by key channel) for prompts and for decoding.
+//
+//   a = sigmoid(z)^(1/tau);   S <- diag(a) S + k v^T;   o = S^T q            per head, S is [D, V] in fp32
+//
+// Kernels:
+//   gla_prep    one warp per (four tokens, head): the decays out of their low-rank projection, and what the scan needs of four
+//               tokens.  With G_i and R_ij the products of the decays up to token i and between tokens j and i (per channel),
+//                   q'_i = G_i q_i,   k'_j = R_3j k_j,   G_3,   P_ij = sum over the channels of q_i R_ij k_j   (j <= i)
+//               Every factor is a product of decays, at most one: nothing is divided, and a channel that forgets at once is
+//               no special case.
+//   gla_scan    prompts:  o_i = S^T q'_i + sum_{j<=i} P_ij v_j,   S <- diag(G_3) S + sum_j k'_j v_j^T,   which is the recurrence itself over four
+//               tokens.  The columns of S are independent, so a group of TPC threads owns CPT columns (D / TPC entries of each, in
+//               registers as packed fp32 pairs).  The sums over D are needed for the output alone: no reduction is on the
+//               path from one state to the next.  The rows of the next tokens travel to shared memory (bulk copies) while the
+//               current ones are used; fp32 FMA throughout.
+//   gla_step    one token per sequence: one block per (sequence, head) computes the decays, streams the state through registers once
+//               (read, updated, written back), and applies the gated norm to the output.
+#include "tfb_elem.cuh"
+#include "tfb_host.h"
+
+namespace tfb {
+TFB_BOUNDS_DEFINE(gated_linear)
+
+struct GlaProj {
+  const void* proj;       // [B*S, ld]: q (H D) | k (H D) | v (H V) | gate (H V) | a1 (rank)
+  long long ld;
+  const void* a2;         // [H D, ld2]
+  long long ld2;
+  const void* bias;       // [H D]
+  int rank;
+  float tau;
+  int H, D, V;
+};
+
+// sigmoid(z)^(1 / tau)
+__device__ __forceinline__ float channel_decay(float z, float tau) {
+  const float ls = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+  return expf(ls / tau);
+}
+
+// z of channel c (of all heads) for N tokens with rows a1[i]
+template <class T, int N>
+__device__ __forceinline__ void decay_logits(const GlaProj& p, const T* const (&a1)[N], long long c, bool vec, float (&z)[N]) {
+  const T* w = static_cast<const T*>(p.a2) + c * p.ld2;
+  const float b = to_f(static_cast<const T*>(p.bias)[c]);
+#pragma unroll
+  for (int i = 0; i < N; ++i) z[i] = b;
+  if (vec) {
+    for (int r = 0; r < p.rank; r += 8) {
+      float x[8], y[8];
+      load_n<8>(w + r, x);
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        load_n<8>(a1[i] + r, y);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) z[i] = fmaf(x[e], y[e], z[i]);
+      }
+    }
+  } else {
+    for (int r = 0; r < p.rank; ++r) {
+      const float x = to_f(w[r]);
+#pragma unroll
+      for (int i = 0; i < N; ++i) z[i] = fmaf(x, to_f(a1[i][r]), z[i]);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// preparation
+// ------------------------------------------------------------------------------------------------
+struct GlaPrepArgs {
+  GlaProj g;
+  const int* lens;                  // [B] tokens of each sequence in this call (null: S)
+  float *q, *k, *v, *decay, *pair;  // [B, H, Sp, Dp] twice, [B, H, Sp, Vp], [B, H, Sp / 4, Dp], [B, H, Sp / 4, 16]
+  int S, Sp, Dp, Vp;
+  int vec;                          // rows of a1 and a2 can be read eight entries at a time
+};
+
+template <class T>
+__global__ void __launch_bounds__(128) gla_prep_kernel(const GlaPrepArgs p) {
+  tfb::pdl_sync();
+  const GlaProj& g = p.g;
+  const int blk = blockIdx.x * 4 + (threadIdx.x >> 5), h = blockIdx.y, b = blockIdx.z, lane = threadIdx.x & 31;
+  const int len = p.lens ? p.lens[b] : p.S, s0 = blk * 4, n = min(4, len - s0);
+  if (n <= 0) return;
+  const T* row[4];
+  const T* a1[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {         // tokens past the end read the last one's rows and are made to change nothing
+    row[i] = static_cast<const T*>(g.proj) + ((long long)b * p.S + s0 + min(i, n - 1)) * g.ld;
+    a1[i] = row[i] + 2 * g.H * (g.D + g.V);
+  }
+  const long long hb = (long long)b * g.H + h;
+  float* qo = p.q + (hb * p.Sp + s0) * p.Dp;
+  float* ko = p.k + (hb * p.Sp + s0) * p.Dp;
+  const float scale = 1.f / sqrtf(float(g.D));
+  float pr[16];
+#pragma unroll
+  for (int i = 0; i < 16; ++i) pr[i] = 0.f;
+  for (int d = lane; d < p.Dp; d += 32) {
+    float q[4], k[4], a[4];
+    if (d < g.D) {
+      const long long c = (long long)h * g.D + d;
+      decay_logits<T, 4>(g, a1, c, p.vec, a);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        q[i] = i < n ? to_f(row[i][c]) * scale : 0.f;
+        k[i] = i < n ? to_f(row[i][(long long)g.H * g.D + c]) : 0.f;
+        a[i] = i < n ? channel_decay(a[i], g.tau) : 1.f;
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) q[i] = k[i] = 0.f, a[i] = 1.f;
+    }
+    float G = 1.f, t[4];                // t[j] = R_ij k_j for the current i
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      G *= a[i];
+#pragma unroll
+      for (int j = 0; j < i; ++j) t[j] *= a[i];
+      t[i] = k[i];
+#pragma unroll
+      for (int j = 0; j <= i; ++j) pr[i * (i + 1) / 2 + j] = fmaf(q[i], t[j], pr[i * (i + 1) / 2 + j]);
+      qo[i * p.Dp + d] = G * q[i];
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) ko[j * p.Dp + d] = t[j];
+    p.decay[(hb * (p.Sp / 4) + blk) * p.Dp + d] = G;
+  }
+#pragma unroll
+  for (int i = 0; i < 16; ++i) pr[i] += __shfl_xor_sync(0xffffffffu, pr[i], 16);
+#pragma unroll
+  for (int o = 8; o > 0; o >>= 1) {     // o values stay with each half: lane x ends up with product x
+    const bool up = lane & o;
+#pragma unroll
+    for (int i = 0; i < o; ++i) {
+      const float send = up ? pr[i] : pr[i + o], keep = up ? pr[i + o] : pr[i];
+      pr[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+    }
+  }
+  if (lane < 16) p.pair[(hb * (p.Sp / 4) + blk) * 16 + lane] = pr[0];
+  float* vo = p.v + (hb * p.Sp + s0) * p.Vp;
+  const long long v0 = 2ll * g.H * g.D + (long long)h * g.V;
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    for (int j = lane; j < p.Vp; j += 32) vo[i * p.Vp + j] = i < n && j < g.V ? to_f(row[i][v0 + j]) : 0.f;
+}
+
+// ------------------------------------------------------------------------------------------------
+// scan over a prompt
+// ------------------------------------------------------------------------------------------------
+struct GlaScanArgs {
+  const float *q, *k, *v, *decay, *pair;
+  float* o;               // [B*S, H, V]
+  float* state;           // [slots, H, D, V]
+  const int* state_slots; // [B]
+  const int* lens;        // [B] or null
+  int S, Sp, H, D, V, Vp, has_past, nslots;
+  int* status;
+};
+
+constexpr int GS_CHUNK = 16;   // tokens per shared-memory stage
+
+// EPT: entries of one column per thread (a multiple of 4); TPC: threads per column group; CPT: columns per group (powers of two, CPT <=
+// TPC); Dp = EPT TPC.  A shuffle reduction of the CPT columns' four sums each leaves one column with each TPC / CPT threads.
+template <int EPT, int TPC, int CPT>
+__global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
+  tfb::pdl_sync();
+  extern __shared__ __align__(128) float sm[];
+  constexpr int Dp = EPT * TPC, CPW = 32 / TPC * CPT, W = TPC / CPT;
+  static_assert(CPT <= TPC && EPT % 4 == 0, "tile shape");
+  const int tid = threadIdx.x, lane = tid & 31, cols = (blockDim.x >> 5) * CPW;
+  const int h = blockIdx.y, b = blockIdx.z, col0 = blockIdx.x * cols;
+  const int t = lane % TPC, cl = (tid >> 5) * CPW + lane / TPC * CPT;      // first column of the group, within the block
+  const int my_cl = cl + t / W, my_col = col0 + my_cl;                      // the column this thread ends up with
+  const int len = p.lens ? p.lens[b] : p.S;
+  constexpr int KQ = GS_CHUNK * Dp, DEC = GS_CHUNK / 4 * Dp, PR = GS_CHUNK * 4;
+  const int stage_f = 2 * KQ + DEC + PR + GS_CHUNK * cols;
+  const uint32_t bar = smem_u32(sm + 2 * stage_f);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(sm + 2 * stage_f + 4);
+  if (tid == 0) {
+    mbar_init(bar, 1);
+    mbar_init(bar + 8, 1);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  for (int s = 0; s < 2; ++s)                                              // columns of v past V stay zero
+    for (int i = tid; i < GS_CHUNK * cols; i += blockDim.x) sm[s * stage_f + 2 * KQ + DEC + PR + i] = 0.f;
+  fence_proxy_async_smem();
+  __syncthreads();
+  const long long hb = (long long)b * p.H + h;
+  const float* qb = p.q + hb * p.Sp * Dp;
+  const float* kb = p.k + hb * p.Sp * Dp;
+  const float* db = p.decay + hb * (p.Sp / 4) * Dp;
+  const float* pb = p.pair + hb * (p.Sp / 4) * 16;
+  const float* vb = p.v + hb * p.Sp * p.Vp + col0;
+  const int nrow = (len + 3) / 4 * 4, nc = min(cols, p.Vp - col0);
+  auto issue = [&](int c) {              // warp 0: the rows of chunk c (whole groups of four)
+    const int s0 = c * GS_CHUNK, n = min(GS_CHUNK, nrow - s0);
+    if (n <= 0 || tid >= 32) return;
+    float* base = sm + (c & 1) * stage_f;
+    const uint32_t br = bar + (c & 1) * 8;
+    if (lane == 0) mbar_expect_tx(br, uint32_t(n) * (2 * Dp + Dp / 4 + 4 + nc) * 4);
+    __syncwarp();
+    if (lane == 0) bulk_load(smem_u32(base), qb + (long long)s0 * Dp, n * Dp * 4, br);
+    if (lane == 1) bulk_load(smem_u32(base + KQ), kb + (long long)s0 * Dp, n * Dp * 4, br);
+    if (lane == 2) bulk_load(smem_u32(base + 2 * KQ), db + (long long)(s0 / 4) * Dp, n * Dp, br);
+    if (lane == 3) bulk_load(smem_u32(base + 2 * KQ + DEC), pb + (long long)s0 * 4, n * 16, br);
+    if (lane >= 16 && lane - 16 < n)
+      bulk_load(smem_u32(base + 2 * KQ + DEC + PR + (lane - 16) * cols), vb + (long long)(s0 + lane - 16) * p.Vp, nc * 4, br);
+  };
+  issue(0);
+  issue(1);
+
+  int slot = p.state_slots ? p.state_slots[b] : -1;
+  TFB_BOUNDS(slot < p.nslots, 72, slot, p.nslots);
+  if (slot >= p.nslots) slot = -1;
+  float* S0 = slot >= 0 ? p.state + ((long long)slot * p.H + h) * p.D * p.V : nullptr;
+  // entry d of a column sits with thread (d / 4) % TPC, register (d / 4) / TPC * 4 + d % 4
+  u64 st[CPT][EPT / 2];
+#pragma unroll
+  for (int x = 0; x < CPT; ++x)
+#pragma unroll
+    for (int i = 0; i < EPT / 4; ++i) {
+      float f[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = (i * TPC + t) * 4 + e, col = col0 + cl + x;
+        f[e] = (S0 && p.has_past && col < p.V && d < p.D) ? S0[(long long)d * p.V + col] : 0.f;
+      }
+      st[x][2 * i] = pack2(f[0], f[1]);
+      st[x][2 * i + 1] = pack2(f[2], f[3]);
+    }
+
+  const int nchunk = (len + GS_CHUNK - 1) / GS_CHUNK;
+  const long long ostep = (long long)p.H * p.V;
+  float* orow = p.o + ((long long)b * p.S * p.H + h) * p.V + my_col;
+  const bool writer = t % W == 0 && my_col < p.V;
+  for (int c = 0; c < nchunk; ++c) {
+    if (!mbar_wait_warp(bar + (c & 1) * 8, (c >> 1) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) break;
+    const float* base = sm + (c & 1) * stage_f;
+    const float* sp = base + 2 * KQ + DEC;
+    const float* sv = sp + PR;
+    const int n = min(GS_CHUNK, len - c * GS_CHUNK);
+#pragma unroll 1
+    for (int r = 0; r < n; r += 4) {
+      u64 acc[CPT][4], vv[CPT][4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int x = 0; x < CPT; ++x) {
+          const float w = sv[(r + i) * cols + cl + x];
+          vv[x][i] = pack2(w, w);
+          acc[x][i] = pack2(0.f, 0.f);
+        }
+      const ulonglong2* sq = reinterpret_cast<const ulonglong2*>(base + r * Dp) + t;
+      const ulonglong2* sk = reinterpret_cast<const ulonglong2*>(base + KQ + r * Dp) + t;
+      const ulonglong2* sg = reinterpret_cast<const ulonglong2*>(base + 2 * KQ + r / 4 * Dp) + t;
+#pragma unroll
+      for (int e = 0; e < EPT / 4; ++e) {
+        ulonglong2 q[4], k[4];
+        const ulonglong2 g = sg[e * TPC];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          q[i] = sq[i * (Dp / 4) + e * TPC];
+          k[i] = sk[i * (Dp / 4) + e * TPC];
+        }
+#pragma unroll
+        for (int x = 0; x < CPT; ++x) {
+          const u64 s0 = st[x][2 * e], s1 = st[x][2 * e + 1];
+#pragma unroll
+          for (int i = 0; i < 4; ++i) acc[x][i] = fma2(s1, q[i].y, fma2(s0, q[i].x, acc[x][i]));
+          u64 u0 = mul2(s0, g.x), u1 = mul2(s1, g.y);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            u0 = fma2(k[i].x, vv[x][i], u0);
+            u1 = fma2(k[i].y, vv[x][i], u1);
+          }
+          st[x][2 * e] = u0;
+          st[x][2 * e + 1] = u1;
+        }
+      }
+      float val[CPT][4];
+#pragma unroll
+      for (int x = 0; x < CPT; ++x)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float2 f = unpack2(acc[x][i]);
+          val[x][i] = f.x + f.y;
+        }
+#pragma unroll
+      for (int o = TPC >> 1, m = CPT; o > 0; o >>= 1) {
+        if (m > 1) {                     // halve the columns: keep those of this thread's half, send the others
+          const bool up = t & o;
+#pragma unroll
+          for (int y = 0; y < m / 2; ++y)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+              const float send = up ? val[y][i] : val[y + m / 2][i], keep = up ? val[y + m / 2][i] : val[y][i];
+              val[y][i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+          m >>= 1;
+        } else {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) val[0][i] += __shfl_xor_sync(0xffffffffu, val[0][i], o);
+        }
+      }
+      if (writer) {
+        const float4* pp = reinterpret_cast<const float4*>(sp + r * 4);
+        const float4 p0 = pp[0], p1 = pp[1], p2 = pp[2];                   // (0,0) (1,0) (1,1) (2,0) | (2,1) (2,2) (3,0) (3,1) | (3,2) (3,3)
+        const float* vr = sv + r * cols + my_cl;
+        const float v0 = vr[0], v1 = vr[cols], v2 = vr[2 * cols], v3 = vr[3 * cols];
+        float* op = orow + (long long)(c * GS_CHUNK + r) * ostep;
+        op[0] = fmaf(p0.x, v0, val[0][0]);
+        if (r + 1 < n) op[ostep] = fmaf(p0.z, v1, fmaf(p0.y, v0, val[0][1]));
+        if (r + 2 < n) op[2 * ostep] = fmaf(p1.y, v2, fmaf(p1.x, v1, fmaf(p0.w, v0, val[0][2])));
+        if (r + 3 < n) op[3 * ostep] = fmaf(p2.y, v3, fmaf(p2.x, v2, fmaf(p1.w, v1, fmaf(p1.z, v0, val[0][3]))));
+      }
+    }
+    __syncthreads();
+    fence_proxy_async_smem();
+    issue(c + 2);
+  }
+  if (*abort_flag) {                     // a copy never landed: the status word says so, the state is left alone
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) {}      // bounded wait for copies already issued
+    return;
+  }
+  if (S0) {
+#pragma unroll
+    for (int x = 0; x < CPT; ++x)
+#pragma unroll
+      for (int i = 0; i < EPT / 4; ++i) {
+        const float2 a = unpack2(st[x][2 * i]), c = unpack2(st[x][2 * i + 1]);
+        const float f[4] = {a.x, a.y, c.x, c.y};
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int d = (i * TPC + t) * 4 + e, col = col0 + cl + x;
+          if (d < p.D && col < p.V) S0[(long long)d * p.V + col] = f[e];
+        }
+      }
+  }
+}
+
+template <int EPT, int TPC, int CPT>
+static int launch_scan_tile(const GlaScanArgs& p, int B, cudaStream_t st) {
+  constexpr int CPW = 32 / TPC * CPT;
+  auto bytes = [](int w) { return (2 * (2 * GS_CHUNK * EPT * TPC + GS_CHUNK / 4 * EPT * TPC + GS_CHUNK * 4 + GS_CHUNK * w * CPW) + 8) * int(sizeof(float)); };
+  // warps per block: rows of v are copied in 16-byte pieces, so at least four columns; blocks for most of the SMs
+  const long long warps = (long long)((p.V + CPW - 1) / CPW) * p.H * B;
+  int nw = 4;
+  while (nw > 1 && nw / 2 * CPW >= 4 && (nw * CPW > p.Vp || (warps + nw - 1) / nw < 4 * sm_count() / 5)) nw >>= 1;
+  if ((nw * CPW) % 4) return TFB_ERR_ARG;
+  static DeviceOnce once;
+  auto kern = gla_scan_kernel<EPT, TPC, CPT>;
+  if (int e = ensure_dyn_smem(once, kern, bytes(4))) return e;
+  const int cols = nw * CPW;
+  launch_k(kern, dim3((p.V + cols - 1) / cols, p.H, B), nw * 32, bytes(nw), st, p);
+  return int(cudaGetLastError());
+}
+
+template <int EPT, int TPC>
+static int launch_scan(const GlaScanArgs& p, int B, cudaStream_t st) {
+  // Four columns per group read q' and k' from shared memory a quarter as often; for few sequences two columns per group of twice as
+  // many threads give each scheduler something to do.
+  constexpr int CPW = 32 / TPC * 4;
+  if ((long long)((p.V + CPW - 1) / CPW) * p.H * B >= 3ll * sm_count()) return launch_scan_tile<EPT, TPC, 4>(p, B, st);
+  if constexpr (EPT >= 8 && TPC <= 16) return launch_scan_tile<EPT / 2, TPC * 2, 2>(p, B, st);
+  else return launch_scan_tile<EPT, TPC, 2>(p, B, st);
+}
+
+// ------------------------------------------------------------------------------------------------
+// one token per sequence
+// ------------------------------------------------------------------------------------------------
+struct GlaStepArgs {
+  GlaProj g;
+  float* state;
+  const int* state_slots;
+  int nslots, vec;
+  const void* w;          // [V] weight of the norm
+  void* out;
+  long long ldo;
+  float eps;
+};
+
+// 256 threads = 8 warps; warp w holds rows w, w + 8, ... (NR of them) of the state, lane l the columns 4 l .. 4 l + 3 of each 128-column
+// part.  D <= 8 NR, V <= 128 CV, V % 4 == 0.
+template <class T, int NR, int CV>
+__global__ void __launch_bounds__(256) gla_step_kernel(const GlaStepArgs p) {
+  tfb::pdl_sync();
+  constexpr int VM = 128 * CV;
+  __shared__ float sk[8 * NR], sq[8 * NR], sa[8 * NR], sv[VM], so[8][VM], red[32];
+  const GlaProj& g = p.g;
+  const int h = blockIdx.x, b = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, D = g.D, V = g.V;
+  int slot = p.state_slots[b];
+  TFB_BOUNDS(slot < p.nslots, 73, slot, p.nslots);
+  if (slot >= p.nslots) slot = -1;
+  float* S0 = slot >= 0 ? p.state + ((long long)slot * g.H + h) * D * V : nullptr;
+  float4 s[NR][CV];
+#pragma unroll
+  for (int i = 0; i < NR; ++i)
+#pragma unroll
+    for (int c = 0; c < CV; ++c) {
+      const int d = warp + 8 * i, j = c * 128 + lane * 4;
+      s[i][c] = (S0 && d < D && j < V) ? *reinterpret_cast<const float4*>(S0 + (long long)d * V + j) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  const T* row = static_cast<const T*>(g.proj) + (long long)b * g.ld;
+  const T* const a1[1] = {row + 2 * g.H * (D + V)};
+  for (int d = tid; d < 8 * NR; d += 256) {
+    float q = 0.f, k = 0.f, z[1] = {0.f};
+    if (d < D) {
+      const long long c = (long long)h * D + d;
+      decay_logits<T, 1>(g, a1, c, p.vec, z);
+      q = to_f(row[c]) / sqrtf(float(D));
+      k = to_f(row[(long long)g.H * D + c]);
+    }
+    sq[d] = q;
+    sk[d] = k;
+    sa[d] = d < D ? channel_decay(z[0], g.tau) : 1.f;
+  }
+  const T* vrow = row + 2ll * g.H * D + (long long)h * V;
+  for (int j = tid; j < VM; j += 256) sv[j] = j < V ? to_f(vrow[j]) : 0.f;
+  __syncthreads();
+#pragma unroll
+  for (int c = 0; c < CV; ++c) {
+    const float4 v = *reinterpret_cast<const float4*>(&sv[c * 128 + lane * 4]);
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int d = warp + 8 * i, j = c * 128 + lane * 4;
+      const float a = sa[d], k = sk[d], q = sq[d];
+      float4 x = s[i][c];
+      x.x = fmaf(a, x.x, k * v.x);
+      x.y = fmaf(a, x.y, k * v.y);
+      x.z = fmaf(a, x.z, k * v.z);
+      x.w = fmaf(a, x.w, k * v.w);
+      if (S0 && d < D && j < V) *reinterpret_cast<float4*>(S0 + (long long)d * V + j) = x;
+      o.x = fmaf(x.x, q, o.x);
+      o.y = fmaf(x.y, q, o.y);
+      o.z = fmaf(x.z, q, o.z);
+      o.w = fmaf(x.w, q, o.w);
+    }
+    *reinterpret_cast<float4*>(&so[warp][c * 128 + lane * 4]) = o;
+  }
+  __syncthreads();
+  float ov = 0.f;                       // VM <= 256: at most one column per thread
+  if (tid < V) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) ov += so[i][tid];
+  }
+  const float rs = 1.f / sqrtf(block_add(ov * ov, red) / V + p.eps);
+  if (tid < V) {
+    const float gt = to_f(vrow[(long long)g.H * V + tid]);
+    static_cast<T*>(p.out)[(long long)b * p.ldo + h * V + tid] = from_f<T>(ov * rs * to_f(static_cast<const T*>(p.w)[tid]) * silu_exact(gt));
+  }
+}
+
+template <class T>
+static int launch_step(const GlaStepArgs& p, int B, cudaStream_t st) {
+  const dim3 grid(p.g.H, B);
+#define TFB_STEP(NR, CV) launch_k(gla_step_kernel<T, NR, CV>, grid, 256, 0, st, p)
+  if (p.g.V <= 128) {
+    if (p.g.D <= 32) TFB_STEP(4, 1);
+    else if (p.g.D <= 64) TFB_STEP(8, 1);
+    else if (p.g.D <= 128) TFB_STEP(16, 1);
+    else TFB_STEP(32, 1);
+  } else {
+    if (p.g.D <= 64) TFB_STEP(8, 2);
+    else TFB_STEP(16, 2);
+  }
+#undef TFB_STEP
+  return int(cudaGetLastError());
+}
+
+static int padded_dim(int D) {
+  for (int d = 32; d <= 512; d *= 2)
+    if (D <= d) return d;
+  return 0;
+}
+
+static int vector_rows(const GlaProj& g, int f32) {
+  const int es = f32 ? 4 : 2, m = f32 ? 4 : 8;
+  auto al = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
+  const char* a1 = static_cast<const char*>(g.proj) + 2ll * g.H * (g.D + g.V) * es;
+  return g.rank % 8 == 0 && g.ld % m == 0 && g.ld2 % m == 0 && al(a1) && al(g.a2);
+}
+
+}  // namespace tfb
+
+// proj, a2, bias: see GlaProj (fp32 or bf16); outputs: see GlaPrepArgs, Sp = S rounded up to 4, Dp as tfb_delta_padded_dim.
+TFB_API int tfb_gla_prep(const void* proj, long long ld, const void* a2, long long ld2, const void* bias, int rank, float tau, const int* lens,
+                         float* q, float* k, float* v, float* decay, float* pair, int B, int S, int H, int D, int Dp, int V, int f32,
+                         void* stream) {
+  using namespace tfb;
+  if (B <= 0 || B > 65535 || S <= 0 || H <= 0 || H > 65535 || D <= 0 || V <= 0 || rank <= 0 || !(tau > 0.f) || Dp != padded_dim(D)) return TFB_ERR_ARG;
+  if (!Dp) return TFB_ERR_LIMIT;
+  const GlaProj g{proj, ld, a2, ld2, bias, rank, tau, H, D, V};
+  const GlaPrepArgs p{g, lens, q, k, v, decay, pair, S, (S + 3) / 4 * 4, Dp, (V + 3) / 4 * 4, vector_rows(g, f32)};
+  const dim3 grid((p.Sp / 4 + 3) / 4, H, B);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) launch_k(gla_prep_kernel<float>, grid, 128, 0, st, p);
+  else launch_k(gla_prep_kernel<__nv_bfloat16>, grid, 128, 0, st, p);
+  return int(cudaGetLastError());
+}
+
+// The recurrence over prepared rows; o [B*S, H, V] fp32.
+TFB_API int tfb_gla_scan(const float* q, const float* k, const float* v, const float* decay, const float* pair, float* o, float* state, int nslots,
+                         const int* state_slots, int B, int S, int H, int D, int V, int has_past, const int* lens, int* status, void* stream) {
+  using namespace tfb;
+  if (B <= 0 || B > 65535 || S <= 0 || H <= 0 || H > 65535 || D <= 0 || V <= 0) return TFB_ERR_ARG;
+  const GlaScanArgs p{q, k, v, decay, pair, o, state, state_slots, lens, S, (S + 3) / 4 * 4, H, D, V, (V + 3) / 4 * 4, has_past, nslots, status};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  switch (padded_dim(D)) {
+    case 32: return launch_scan<4, 8>(p, B, st);
+    case 64: return launch_scan<8, 8>(p, B, st);
+    case 128: return launch_scan<16, 8>(p, B, st);
+    case 256: return launch_scan<16, 16>(p, B, st);
+    case 512: return launch_scan<16, 32>(p, B, st);
+    default: return TFB_ERR_LIMIT;
+  }
+}
+
+// One token for each of B sequences that go on, gated norm included.  Returns TFB_ERR_LIMIT for head sizes it does not hold in
+// registers (the caller then takes the preparation, the scan and the norm kernel).
+TFB_API int tfb_gla_step(const void* proj, long long ld, const void* a2, long long ld2, const void* bias, int rank, float tau, float* state,
+                         const int* state_slots, int nslots, const void* w, void* out, long long ldo, int B, int H, int D, int V, float eps, int f32,
+                         void* stream) {
+  using namespace tfb;
+  if (B <= 0 || B > 65535 || H <= 0 || D <= 0 || V <= 0 || rank <= 0 || !(tau > 0.f) || !state_slots) return TFB_ERR_ARG;
+  if ((V & 3) || V > 256 || D > 256 || (V > 128 && D > 128)) return TFB_ERR_LIMIT;
+  const GlaProj g{proj, ld, a2, ld2, bias, rank, tau, H, D, V};
+  const GlaStepArgs p{g, state, state_slots, nslots, vector_rows(g, f32), w, out, ldo, eps};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return f32 ? launch_step<float>(p, B, st) : launch_step<__nv_bfloat16>(p, B, st);
+}

@@ -2,17 +2,14 @@
 // W_uv,h c; causal softmax without positions, one output gate per head.
 //
 //   latent_append      norm of the latents and their append to the pages
-//   head_attn_fwd      prompts, bf16, tcgen05, over keys and values that a product has read out of the latents: one CTA per (sequence,
-//                      head, 256 queries) as two 128-query tiles that share every key / value tile and take turns on the
-//                      tensor core; keys and values may have different sizes; the gate is applied in the epilogue
+//   prompts            attend over keys and values that a product has read out of the latents: head_attention.cu
 //   head_linear        one small product per head for the rows of a decode step (mma.sync): queries into the latent space,
 //                      q . W_uk c = (W_uk^T q) . c; the values come out of the attention's result, sum_j a_j W_uv c_j =
 //                      W_uv sum_j a_j c_j, by the per-head form of skinny_linear.cu
 //   latent_decode      one query per sequence over the paged latents, bf16, mma.sync: the query heads are the rows of one or two 16-row
 //                      tiles, and the latents are keys and values of all of them, so a cached row is read once.  Split over
 //                      the keys; a second kernel merges the splits.
-//   attn_any           any sizes, bf16 or fp32, prompts (keys and values read out) or decoding (over the latents): fp32 FMA
-//                      throughout, online softmax over 32-key tiles.
+//   latent_any         decoding, any sizes, bf16 or fp32: fp32 FMA throughout, online softmax over 32-key tiles.
 #include "tfb_elem.cuh"
 #include "tfb_host.h"
 #include "tfb_mma.cuh"
@@ -21,8 +18,6 @@ namespace tfb {
 TFB_BOUNDS_DEFINE(latent_attention)
 
 constexpr float LOG2E = 1.4426950408889634f;
-
-__device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
 
 // ------------------------------------------------------------------------------------------------
 // v = c / rms(c) * w, to out and to the pools' slots; one warp per row
@@ -57,37 +52,6 @@ __global__ void __launch_bounds__(256) latent_append_kernel(const T* __restrict_
   }
 }
 
-// ------------------------------------------------------------------------------------------------
-// prompts on tcgen05
-// ------------------------------------------------------------------------------------------------
-struct HeadAttnParams {
-  int B, S, H, G;
-  int Skv, q_off;         // keys per sequence; query i sees keys 0 .. i + q_off
-  int V;
-  float scale;
-  const __nv_bfloat16* gate;    // [B*S, ldg] or null
-  long long ldg;
-  __nv_bfloat16* O;
-  long long ldo;
-  int* status;
-};
-
-constexpr int HA_THREADS = 320;
-constexpr int HA_BM = 128, HA_BN = 128;
-constexpr int HA_BOX = 128 * 128;       // bytes of 128 rows of 64 entries
-
-template <int DK, int DV>
-struct HeadSmem {
-  static constexpr int NBK = DK / 64, NBV = DV / 64;
-  static constexpr int QT = NBK * HA_BOX, KT = NBK * HA_BOX, VT = NBV * HA_BOX, STAGE = KT + VT;
-  static constexpr int AVAIL = 227 * 1024 - 1024 - 256 - 2 * QT;
-  static constexpr int STAGES = AVAIL / STAGE > 4 ? 4 : AVAIL / STAGE;
-  static constexpr int KV_OFF = 2 * QT;
-  static constexpr int BAR_OFF = KV_OFF + STAGES * STAGE;
-  static constexpr int TOTAL = BAR_OFF + 256 + 1024;
-  static_assert(STAGES >= 2, "two stages at least");
-};
-
 __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -98,285 +62,6 @@ __device__ __forceinline__ float redux_max(float x) {      // over the warp, one
   float y;
   asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(y) : "f"(x));
   return y;
-}
-
-// running maximum over the 128 scores of this thread's row; keys after `hi` (index within the tile) do not count
-template <bool MASK>
-__device__ __forceinline__ float tile_max(uint32_t tS, float m, int hi) {
-  float mx0 = m, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
-#pragma unroll 1
-  for (int c = 0; c < HA_BN / 32; ++c) {
-    uint32_t v[32];
-    tmem_ld_32x32(tS + c * 32, v);
-    tmem_ld_wait();
-    if (MASK) {
-#pragma unroll
-      for (int i = 0; i < 32; ++i)
-        if (c * 32 + i > hi) v[i] = 0xff800000u;
-    }
-#pragma unroll
-    for (int i = 0; i < 32; i += 8) {
-      mx0 = fmax3(mx0, __uint_as_float(v[i]), __uint_as_float(v[i + 1]));
-      mx1 = fmax3(mx1, __uint_as_float(v[i + 2]), __uint_as_float(v[i + 3]));
-      mx2 = fmax3(mx2, __uint_as_float(v[i + 4]), __uint_as_float(v[i + 5]));
-      mx3 = fmax3(mx3, __uint_as_float(v[i + 6]), __uint_as_float(v[i + 7]));
-    }
-  }
-  return fmaxf(fmaxf(mx0, mx1), fmaxf(mx2, mx3));
-}
-
-// p = 2^(s * sl2 - mb) over the row, written back over the scores as bf16 pairs; returns the row sum
-template <bool MASK>
-__device__ __forceinline__ float tile_probs(uint32_t tS, float sl2, float mb, int hi) {
-  float rs[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 1
-  for (int c = 0; c < HA_BN / 32; ++c) {
-    uint32_t v[32], pk[16];
-    tmem_ld_32x32(tS + c * 32, v);
-    tmem_ld_wait();
-#pragma unroll
-    for (int i = 0; i < 16; i += 2) {
-      float q[4];
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        q[e] = ex2(fmaf(__uint_as_float(v[2 * i + e]), sl2, -mb));
-        if (MASK && c * 32 + 2 * i + e > hi) q[e] = 0.f;
-        rs[e] += q[e];
-      }
-      pk[i] = pack_bf16(q[0], q[1]);
-      pk[i + 1] = pack_bf16(q[2], q[3]);
-    }
-    tmem_st_32x16(tS + c * 16, pk);
-  }
-  return (rs[0] + rs[1]) + (rs[2] + rs[3]);
-}
-
-template <int DK, int DV>
-__global__ void __launch_bounds__(HA_THREADS, 1)
-head_attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_constant__ CUtensorMap tk, const __grid_constant__ CUtensorMap tv,
-                     const HeadAttnParams p) {
-  using L = HeadSmem<DK, DV>;
-  constexpr int ST = L::STAGES;
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const uint32_t sQ = smem_u32(smem);
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::BAR_OFF);
-  const uint32_t bar_q = smem_u32(bars);
-  const uint32_t bar_kv_full = bar_q + 8;
-  const uint32_t bar_kv_empty = bar_kv_full + ST * 8;
-  const uint32_t bar_s_full = bar_kv_empty + ST * 8;
-  const uint32_t bar_p_ready = bar_s_full + 16;
-  const uint32_t bar_o_full = bar_p_ready + 16;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 1 + 2 * ST + 6);
-  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int npair = (p.S + 2 * HA_BM - 1) / (2 * HA_BM);
-  const int bh = p.B * p.H;
-  const int pair = npair - 1 - int(blockIdx.x) / bh;   // the longest (latest) query blocks first
-  const int rem = int(blockIdx.x) % bh;
-  const int b = rem / p.H, h = rem % p.H, hk = h / (p.H / p.G);
-  int n_t[2];                                          // key blocks each tile visits (0: the tile lies past the end)
-#pragma unroll
-  for (int t = 0; t < 2; ++t) {
-    const int q0 = (pair * 2 + t) * HA_BM;
-    n_t[t] = q0 >= p.S ? 0 : (min(q0 + HA_BM, p.S) - 1 + p.q_off) / HA_BN + 1;
-  }
-  const int n_kv = max(n_t[0], n_t[1]);
-
-  if (threadIdx.x == 0) {
-    mbar_init(bar_q, 1);
-    for (int s = 0; s < ST; ++s) {
-      mbar_init(bar_kv_full + s * 8, 1);
-      mbar_init(bar_kv_empty + s * 8, 1);
-    }
-    for (int i = 0; i < 2; ++i) {
-      mbar_init(bar_s_full + i * 8, 1);
-      mbar_init(bar_p_ready + i * 8, 128);
-      mbar_init(bar_o_full + i * 8, 1);
-    }
-    *abort_flag = 0;
-    mbar_fence_init();
-    tma_prefetch_desc(&tq);
-    tma_prefetch_desc(&tk);
-    tma_prefetch_desc(&tv);
-  }
-  if (warp == 1) {
-    tmem_alloc(smem_u32(tmem_slot), 512);
-    tmem_relinquish();
-  }
-  tc_fence_before();
-  __syncthreads();
-  tc_fence_after();
-  const uint32_t tmem_base = *tmem_slot;
-  tfb::pdl_sync();
-  const uint32_t tS0 = tmem_base, tO0 = tmem_base + 256;
-
-  if (warp == 0) {
-    if (lane == 0) {
-      mbar_expect_tx(bar_q, 2 * L::QT);
-#pragma unroll
-      for (int t = 0; t < 2; ++t)
-#pragma unroll
-        for (int i = 0; i < L::NBK; ++i) tma_load_4d(sQ + t * L::QT + i * HA_BOX, &tq, bar_q, i * 64, h, (pair * 2 + t) * HA_BM, b);
-      for (int j = 0; j < n_kv; ++j) {
-        const int st = j % ST;
-        if (!mbar_wait(bar_kv_empty + st * 8, ((j / ST) & 1) ^ 1, abort_flag, p.status, ST_TIMEOUT_EMPTY)) break;
-        const uint32_t fb = bar_kv_full + st * 8, base = sQ + L::KV_OFF + st * L::STAGE;
-        mbar_expect_tx(fb, L::STAGE);
-#pragma unroll
-        for (int i = 0; i < L::NBK; ++i) tma_load_4d(base + i * HA_BOX, &tk, fb, i * 64, hk, j * HA_BN, b);
-#pragma unroll
-        for (int i = 0; i < L::NBV; ++i) tma_load_4d(base + L::KT + i * HA_BOX, &tv, fb, i * 64, hk, j * HA_BN, b);
-      }
-      if (*abort_flag) {  // unwinding: bounded wait for copies already issued
-        const uint64_t t0 = globaltimer_ns();
-        while (globaltimer_ns() - t0 < 200000ull) {}
-      }
-    }
-  } else if (warp == 1) {
-    if (lane == 0) {
-      constexpr uint32_t idesc_s = umma_idesc(FMT_BF16, FMT_BF16, false, false, HA_BM, HA_BN);
-      constexpr uint32_t idesc_o = umma_idesc(FMT_BF16, FMT_BF16, false, true, HA_BM, DV);
-      auto issue_s = [&](int t, int j) {
-        const uint32_t sK = sQ + L::KV_OFF + (j % ST) * L::STAGE, sQt = sQ + t * L::QT, tS = tS0 + t * 128;
-#pragma unroll
-        for (int k = 0; k < DK / 16; ++k) {
-          const uint32_t off = (k >> 2) * HA_BOX + (k & 3) * 32;
-          umma_f16_ss(tS, umma_smem_desc(sQt + off, 16, 1024), umma_smem_desc(sK + off, 16, 1024), idesc_s, k > 0);
-        }
-        umma_commit(bar_s_full + t * 8);
-      };
-      bool ok = mbar_wait(bar_q, 0, abort_flag, p.status, ST_TIMEOUT_FULL) &&
-                mbar_wait(bar_kv_full, 0, abort_flag, p.status, ST_TIMEOUT_FULL);
-      if (ok) {
-        tc_fence_after();
-#pragma unroll
-        for (int t = 0; t < 2; ++t)
-          if (n_t[t] > 0) issue_s(t, 0);
-      }
-      for (int j = 0; j < n_kv && ok; ++j) {
-        if (j + 1 < n_kv) {
-          const int st1 = (j + 1) % ST;
-          if (!mbar_wait(bar_kv_full + st1 * 8, ((j + 1) / ST) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) break;
-          tc_fence_after();
-        }
-        const int st = j % ST;
-        const uint32_t sV = sQ + L::KV_OFF + st * L::STAGE + L::KT;
-#pragma unroll
-        for (int t = 0; t < 2; ++t) {
-          if (!ok || j >= n_t[t]) continue;
-          if (!mbar_wait(bar_p_ready + t * 8, j & 1, abort_flag, p.status, ST_TIMEOUT_TMEM_EMPTY)) {
-            ok = false;
-            continue;
-          }
-          tc_fence_after();
-          const uint32_t tP = tS0 + t * 128, tO = tO0 + t * 128;
-#pragma unroll
-          for (int k = 0; k < HA_BN / 16; ++k)     // V tile: [key rows][64-column boxes], MN-major B
-            umma_f16_ts(tO, tP + k * 8, umma_smem_desc(sV + k * 2048, HA_BOX, 1024), idesc_o, k > 0);
-          if (j + 1 < n_t[t]) issue_s(t, j + 1);   // its commit also covers the P V product above
-          else umma_commit(bar_o_full + t * 8);
-        }
-        if (ok) umma_commit(bar_kv_empty + st * 8);
-      }
-    }
-  } else {
-    const int t = (warp - 2) >> 2, quad = warp & 3, r = quad * 32 + lane;
-    const int q0 = (pair * 2 + t) * HA_BM, q_idx = q0 + r;
-    const int n_mine = t ? n_t[1] : n_t[0];
-    const uint32_t lane_off = uint32_t(quad * 32) << 16;
-    const uint32_t tS = tS0 + t * 128 + lane_off, tO = tO0 + t * 128 + lane_off;
-    const float sl2 = p.scale * LOG2E;
-    const int hi_g = min(q_idx + p.q_off, p.Skv - 1);
-    float m = -INFINITY, l = 0.f, alpha_prev = 1.f;
-    float o[DV];
-#pragma unroll
-    for (int i = 0; i < DV; ++i) o[i] = 0.f;
-    bool ok = true;
-    for (int j = 0; j < n_mine; ++j) {
-      if (!mbar_wait_warp(bar_s_full + t * 8, j & 1, abort_flag, p.status, ST_TIMEOUT_TMEM_FULL)) {
-        ok = false;
-        break;
-      }
-      tc_fence_after();
-      const int k0 = j * HA_BN, hi = hi_g - k0;
-      const bool need_mask = k0 + HA_BN - 1 > q0 + p.q_off || k0 + HA_BN > p.Skv;
-      // a query that sits past the end of its sequence may see no key of its last block; its row is not stored
-      const float mx = need_mask ? tile_max<true>(tS, m, hi) : tile_max<false>(tS, m, hi);
-      if (j > 0) {  // O(j-1) is complete: the commit behind S(j) was issued after it
-#pragma unroll
-        for (int c = 0; c < DV / 32; ++c) {
-          uint32_t v[32];
-          tmem_ld_32x32(tO + c * 32, v);
-          tmem_ld_wait();
-#pragma unroll
-          for (int i = 0; i < 32; ++i) o[c * 32 + i] = fmaf(o[c * 32 + i], alpha_prev, __uint_as_float(v[i]));
-        }
-      }
-      const float mb = (mx == -INFINITY) ? 0.f : mx * sl2;
-      const float alpha = (m == -INFINITY) ? 0.f : ex2(m * sl2 - mb);
-      const float rs = need_mask ? tile_probs<true>(tS, sl2, mb, hi) : tile_probs<false>(tS, sl2, mb, hi);
-      l = fmaf(l, alpha, rs);
-      m = mx;
-      tmem_st_wait();
-      tc_fence_before();
-      mbar_arrive(bar_p_ready + t * 8);
-      alpha_prev = alpha;
-    }
-    if (ok && n_mine > 0 && mbar_wait_warp(bar_o_full + t * 8, 0, abort_flag, p.status, ST_TIMEOUT_TMEM_FULL)) {
-      tc_fence_after();
-#pragma unroll
-      for (int c = 0; c < DV / 32; ++c) {
-        uint32_t v[32];
-        tmem_ld_32x32(tO + c * 32, v);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 32; ++i) o[c * 32 + i] = fmaf(o[c * 32 + i], alpha_prev, __uint_as_float(v[i]));
-      }
-      if (q_idx < p.S) {
-        const long long row = (long long)b * p.S + q_idx;
-        float f = l > 0.f ? 1.f / l : 0.f;
-        if (p.gate) f *= sigmoid_exact(__bfloat162float(p.gate[row * p.ldg + h]));
-        __nv_bfloat16* op = p.O + row * p.ldo + h * p.V;
-#pragma unroll
-        for (int c = 0; c < DV / 8; ++c) {
-          if (c * 8 < p.V) {
-            uint4 u;
-            u.x = pack_bf16(o[c * 8 + 0] * f, o[c * 8 + 1] * f);
-            u.y = pack_bf16(o[c * 8 + 2] * f, o[c * 8 + 3] * f);
-            u.z = pack_bf16(o[c * 8 + 4] * f, o[c * 8 + 5] * f);
-            u.w = pack_bf16(o[c * 8 + 6] * f, o[c * 8 + 7] * f);
-            *reinterpret_cast<uint4*>(op + c * 8) = u;
-          }
-        }
-      }
-    }
-  }
-
-  tc_fence_before();
-  __syncthreads();
-  if (warp == 1) {
-    tc_fence_after();
-    tmem_dealloc(tmem_base, 512);
-  }
-}
-
-template <int DK, int DV>
-static int launch_head_attn(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, int D, const HeadAttnParams& p,
-                            cudaStream_t st) {
-  using L = HeadSmem<DK, DV>;
-  static DeviceOnce once;
-  auto kern = head_attn_fwd_kernel<DK, DV>;
-  if (int e = ensure_dyn_smem(once, kern, L::TOTAL)) return e;
-  CUtensorMap tq, tk, tv;
-  int rc;
-  const uint64_t d = D, vv = p.V, S = p.S, Skv = p.Skv, B = p.B;
-  if ((rc = make_tmap_4d(&tq, q, 2, {d, uint64_t(p.H), S, B}, {d * 2, uint64_t(ldq) * 2, uint64_t(ldq) * 2 * S}, {64, 1, HA_BM, 1}))) return rc;
-  if ((rc = make_tmap_4d(&tk, k, 2, {d, uint64_t(p.G), Skv, B}, {d * 2, uint64_t(ldk) * 2, uint64_t(ldk) * 2 * Skv}, {64, 1, HA_BN, 1}))) return rc;
-  if ((rc = make_tmap_4d(&tv, v, 2, {vv, uint64_t(p.G), Skv, B}, {vv * 2, uint64_t(ldv) * 2, uint64_t(ldv) * 2 * Skv}, {64, 1, HA_BN, 1}))) return rc;
-  launch_k(kern, ((p.S + 2 * HA_BM - 1) / (2 * HA_BM)) * p.B * p.H, HA_THREADS, L::TOTAL, st, tq, tk, tv, p);
-  return int(cudaGetLastError());
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -800,78 +485,54 @@ static int launch_latent_decode(const LatentDecodeArgs& p, int B, cudaStream_t s
 // any sizes, fp32 arithmetic
 // ------------------------------------------------------------------------------------------------
 template <class T>
-struct AttnAnyArgs {
-  const T* q;               // [B*S, ldq], H heads of D entries
+struct LatentAnyArgs {
+  const T* q;               // [B, ldq], H heads of W entries, R of them used
   long long ldq;
-  const T *k, *v;           // prompts: [B*Skv, ldk], [B*Skv, ldv], G heads; decoding: k = the pool [slots][ldk], keys and values of every head
-  long long ldk, ldv, nslots;
-  const int* block_table;   // decoding only
+  const T* pool;            // [slots][W]: keys and values of every head
+  long long nslots;
+  const int* block_table;
   int max_pages, page;
-  const int* positions;     // decoding: position of the one query of each sequence
-  const T* gate;            // [B*S, ldg] or null
-  long long ldg;
+  const int* positions;     // [B] position of the one query of each sequence
   T* o;
   long long ldo;
-  int B, S, Skv, q_off, H, G, D, V, QR;
+  int H, R, W, QR;
   float scale;
 };
 
 constexpr int AN_K = 32;    // keys per tile
 
-// QR (4, 8 or 16) query rows per block: positions of one head (prompts) or heads of one sequence (decoding)
-template <class T, bool PAGED>
-__global__ void __launch_bounds__(128) attn_any_kernel(const AttnAnyArgs<T> p) {
+// QR (4, 8 or 16) heads of one sequence per block
+template <class T>
+__global__ void __launch_bounds__(128) latent_any_kernel(const LatentAnyArgs<T> p) {
   tfb::pdl_sync();
   extern __shared__ float am[];
-  const int D = p.D, V = p.V, QR = p.QR, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, DP = D + 1;
+  const int D = p.R, QR = p.QR, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, DP = D + 1;
   float* sQ = am;                       // [QR][D]
   float* sK = sQ + QR * D;              // [AN_K][D + 1]
-  float* sV = sK + AN_K * DP;           // [AN_K][V]; decoding: the keys
-  float* sP = PAGED ? sV : sV + AN_K * V;   // [QR][AN_K]
-  float* sO = sP + QR * AN_K;           // [QR][V]
-  float* sA = sO + QR * V;              // [QR] rescale of this tile, then row sums
-  const int VP = PAGED ? DP : V;
-  if (PAGED) sV = sK;
-  int b, h0, i0, n, hi_max;
-  if (PAGED) {
-    b = blockIdx.y;
-    h0 = blockIdx.x * QR;
-    n = min(QR, p.H - h0);
-    i0 = 0;
-    hi_max = p.positions[b];
-  } else {
-    b = blockIdx.z;
-    h0 = blockIdx.y;
-    i0 = blockIdx.x * QR;
-    n = min(QR, p.S - i0);
-    hi_max = min(i0 + n - 1 + p.q_off, p.Skv - 1);
-  }
-  const int g = PAGED ? 0 : h0 / (p.H / p.G);
-  const int q_head = PAGED ? int(p.ldk) : D;      // entries between the heads of q and o
-  const int o_head = PAGED ? int(p.ldk) : V;
+  float* sP = sK + AN_K * DP;           // [QR][AN_K]
+  float* sO = sP + QR * AN_K;           // [QR][D]
+  float* sA = sO + QR * D;              // [QR] rescale of this tile, then row sums
+  const int b = blockIdx.y, h0 = blockIdx.x * QR, n = min(QR, p.H - h0), hi = p.positions[b];
   for (int i = tid; i < QR * D; i += 128) {
-    const int r = i / D, d = i % D;
-    const long long row = PAGED ? b : (long long)b * p.S + i0 + r;
-    sQ[i] = r < n ? to_f(p.q[row * p.ldq + (long long)(PAGED ? h0 + r : h0) * q_head + d]) : 0.f;
+    const int r = i / D;
+    sQ[i] = r < n ? to_f(p.q[b * p.ldq + (long long)(h0 + r) * p.W + i % D]) : 0.f;
+    sO[i] = 0.f;
   }
-  for (int i = tid; i < QR * V; i += 128) sO[i] = 0.f;
   float m_run[4], l_run[4];             // this warp's rows: warp, warp + 4, ...
 #pragma unroll
   for (int i = 0; i < 4; ++i) { m_run[i] = -INFINITY; l_run[i] = 0.f; }
-  for (int t0 = 0; t0 <= hi_max; t0 += AN_K) {
-    const int nk = min(AN_K, hi_max + 1 - t0);
+  for (int t0 = 0; t0 <= hi; t0 += AN_K) {
+    const int nk = min(AN_K, hi + 1 - t0);
     __syncthreads();
     for (int j = warp; j < AN_K; j += 4) {
-      long long row = (long long)b * p.Skv + t0 + j;
-      if (PAGED && j < nk) {
+      long long row = 0;
+      if (j < nk) {
         long long page = p.block_table[(long long)b * p.max_pages + (t0 + j) / p.page];
         TFB_BOUNDS(page >= 0 && (page + 1) * p.page <= p.nslots, 52, page, p.nslots / p.page);
         if (page < 0 || (page + 1) * p.page > p.nslots) page = 0;
         row = page * p.page + (t0 + j) % p.page;
       }
-      for (int d = lane; d < D; d += 32) sK[j * DP + d] = j < nk ? to_f(p.k[row * p.ldk + (long long)g * D + d]) : 0.f;
-      if (!PAGED)
-        for (int d = lane; d < V; d += 32) sV[j * VP + d] = j < nk ? to_f(p.v[row * p.ldv + (long long)g * V + d]) : 0.f;
+      for (int d = lane; d < D; d += 32) sK[j * DP + d] = j < nk ? to_f(p.pool[row * p.W + d]) : 0.f;
     }
     __syncthreads();
 #pragma unroll
@@ -882,8 +543,7 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const AttnAnyArgs<T> p) {
       const float* k = sK + lane * DP;
       float s = 0.f;
       for (int d = 0; d < D; ++d) s = fmaf(q[d], k[d], s);
-      const int hi = PAGED ? hi_max : i0 + r + p.q_off;
-      s = (r < n && lane < nk && t0 + lane <= hi) ? s * p.scale : -INFINITY;
+      s = (r < n && lane < nk) ? s * p.scale : -INFINITY;
       const float mx = fmaxf(m_run[i], warp_max(s));
       const float mb = mx == -INFINITY ? 0.f : mx;
       const float a = m_run[i] == -INFINITY ? 0.f : expf(m_run[i] - mb);
@@ -894,11 +554,11 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const AttnAnyArgs<T> p) {
       if (lane == 0) sA[r] = a;
     }
     __syncthreads();
-    for (int i = tid; i < QR * V; i += 128) {
-      const int r = i / V, d = i % V;
+    for (int i = tid; i < QR * D; i += 128) {
+      const int r = i / D, d = i % D;
       float acc = sO[i] * sA[r];
 #pragma unroll 8
-      for (int j = 0; j < AN_K; ++j) acc = fmaf(sP[r * AN_K + j], sV[j * VP + d], acc);
+      for (int j = 0; j < AN_K; ++j) acc = fmaf(sP[r * AN_K + j], sK[j * DP + d], acc);
       sO[i] = acc;
     }
   }
@@ -908,27 +568,23 @@ __global__ void __launch_bounds__(128) attn_any_kernel(const AttnAnyArgs<T> p) {
     if (lane == 0 && warp + 4 * i < QR) sA[warp + 4 * i] = l_run[i];
   __syncthreads();
   for (int r = warp; r < n; r += 4) {
-    const long long row = PAGED ? b : (long long)b * p.S + i0 + r;
-    const int h = PAGED ? h0 + r : h0;
-    float f = 1.f / sA[r];
-    if (p.gate) f *= sigmoid_exact(to_f(p.gate[row * p.ldg + h]));
-    for (int d = lane; d < o_head; d += 32) p.o[row * p.ldo + (long long)h * o_head + d] = from_f<T>(d < V ? sO[r * V + d] * f : 0.f);
+    const float f = 1.f / sA[r];
+    for (int d = lane; d < p.W; d += 32) p.o[b * p.ldo + (long long)(h0 + r) * p.W + d] = from_f<T>(d < D ? sO[r * D + d] * f : 0.f);
   }
 }
 
-template <class T, bool PAGED>
-static int launch_any(AttnAnyArgs<T> p, cudaStream_t st) {
+template <class T>
+static int launch_latent_any(LatentAnyArgs<T> p, int B, cudaStream_t st) {
   long long smem = 0;
   for (p.QR = 16; p.QR >= 4; p.QR >>= 1) {
-    smem = 4ll * (p.QR * p.D + AN_K * (p.D + 1) + (PAGED ? 0 : AN_K * p.V) + p.QR * AN_K + p.QR * p.V + p.QR);
+    smem = 4ll * (2 * p.QR * p.R + AN_K * (p.R + 1) + p.QR * AN_K + p.QR);
     if (smem <= 220 * 1024) break;
   }
   if (p.QR < 4) return TFB_ERR_LIMIT;
   static DeviceOnce once;
-  auto kern = attn_any_kernel<T, PAGED>;
+  auto kern = latent_any_kernel<T>;
   if (int e = ensure_dyn_smem(once, kern, 220 * 1024)) return e;
-  const dim3 grid = PAGED ? dim3((p.H + p.QR - 1) / p.QR, p.B) : dim3((p.S + p.QR - 1) / p.QR, p.H, p.B);
-  launch_k(kern, grid, 128, size_t(smem), st, p);
+  launch_k(kern, dim3((p.H + p.QR - 1) / p.QR, B), 128, size_t(smem), st, p);
   return int(cudaGetLastError());
 }
 
@@ -953,28 +609,6 @@ TFB_API int tfb_latent_append(const void* c, long long ldc, const void* w, float
   else { if (v) TFB_LA(bf16, 8); else TFB_LA(bf16, 1); }
 #undef TFB_LA
   return int(cudaGetLastError());
-}
-
-// q [B*S, ldq]: H heads of D entries; k, v [B*Skv, ldk / ldv]: G heads of D / V entries; gate [B*S, ldg]: one logit per head, or null.
-// The queries are the last S of the Skv positions.  o [B*S, ldo]: H heads of V entries.
-TFB_API int tfb_head_attn(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, void* o, long long ldo,
-                          const void* gate, long long ldg, int B, int S, int Skv, int H, int G, int D, int V, float scale, int f32, int* status,
-                          void* stream) {
-  using namespace tfb;
-  if (B <= 0 || B > 65535 || S <= 0 || Skv < S || G <= 0 || H % G || H > 65535 || D <= 0 || V <= 0) return TFB_ERR_ARG;
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool tc = !f32 && D % 8 == 0 && V % 8 == 0 && D <= 128 && V <= 128 && ldq % 8 == 0 && ldk % 8 == 0 && ldv % 8 == 0 && ldo % 8 == 0 &&
-                  al16(q) && al16(k) && al16(v) && al16(o);
-  if (tc) {
-    HeadAttnParams p{B, S, H, G, Skv, Skv - S, V, scale, static_cast<const bf16*>(gate), ldg, static_cast<bf16*>(o), ldo, status};
-    if (D <= 64) return V <= 64 ? launch_head_attn<64, 64>(q, ldq, k, ldk, v, ldv, D, p, st) : launch_head_attn<64, 128>(q, ldq, k, ldk, v, ldv, D, p, st);
-    return V <= 64 ? launch_head_attn<128, 64>(q, ldq, k, ldk, v, ldv, D, p, st) : launch_head_attn<128, 128>(q, ldq, k, ldk, v, ldv, D, p, st);
-  }
-#define TFB_ANY(T)                                                                                                                           \
-  launch_any<T, false>(AttnAnyArgs<T>{static_cast<const T*>(q), ldq, static_cast<const T*>(k), static_cast<const T*>(v), ldk, ldv, 0, nullptr, 0, 1, \
-                                      nullptr, static_cast<const T*>(gate), ldg, static_cast<T*>(o), ldo, B, S, Skv, Skv - S, H, G, D, V, 16, scale}, st)
-  return f32 ? TFB_ANY(float) : TFB_ANY(bf16);
-#undef TFB_ANY
 }
 
 // One product per head: x [M, ldx] (x_head entries between heads, K of them used), w: heads blocks [K, N] stacked on the rows, out [M, ldo]
@@ -1023,9 +657,9 @@ TFB_API int tfb_latent_decode(const void* q, long long ldq, const void* pool, lo
     if (splits > 1) launch_k(latent_combine_kernel, B * H, 128, 0, st, acc, ml, static_cast<bf16*>(o), ldo, H, W, splits);
     return int(cudaGetLastError());
   }
-#define TFB_ANY(T)                                                                                                                             \
-  launch_any<T, true>(AttnAnyArgs<T>{static_cast<const T*>(q), ldq, static_cast<const T*>(pool), nullptr, W, 0, nslots, block_table, max_pages, page, \
-                                     positions, nullptr, 0, static_cast<T*>(o), ldo, B, 1, 0, 0, H, 1, R, R, 16, scale}, st)
+#define TFB_ANY(T)                                                                                                                    \
+  launch_latent_any<T>(LatentAnyArgs<T>{static_cast<const T*>(q), ldq, static_cast<const T*>(pool), nslots, block_table, max_pages, page, positions, \
+                                        static_cast<T*>(o), ldo, H, R, W, 16, scale}, B, st)
   return f32 ? TFB_ANY(float) : TFB_ANY(bf16);
 #undef TFB_ANY
 }

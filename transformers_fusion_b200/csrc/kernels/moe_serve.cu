@@ -1,13 +1,14 @@
 // Mixture-of-experts feed-forward for serving: any sizes and pitches, bf16 or fp32 rows, no statistics and nothing kept for a
 // backward pass (the training form is moe_routing.cu).
 //
-//   moe_route          per token: the k largest of logits + bias (fp32, the lower index first among equals) and the softmax over them;
+//   moe_route          per token: the k largest of logits (+ bias) (fp32, the lower index first among equals) and the softmax over them,
+//                      or the k largest sigmoids among the experts of the best groups, weighted by them over their sum;
 //                      then the rows of the expert buffers: every expert's assignments are consecutive rows from a multiple
 //                      of 128 on, so that a 128-row tile of the grouped product belongs to one expert.  Few tokens (decode
 //                      steps): one block does all of it; many: selection with per-block counts, then the scan and row numbers.
 //   moe_gather         token rows to their assignments' rows
 //   moe_glu            silu(gate) * up of the assigned rows (a decode step's buffers are mostly padding)
-//   moe_weighted_sum   y[t] = base[t] + sum_k w[t, k] * rows[row_of[t, k]], summed in fp32
+//   moe_weighted_sum   y[t] = base[t] [* sigmoid(gate[t])] + sum_k w[t, k] * rows[row_of[t, k]], summed in fp32
 #include <limits.h>
 
 #include "tfb_elem.cuh"
@@ -19,7 +20,7 @@ TFB_BOUNDS_DEFINE(moe_serve)
 struct RouteArgs {
   const float* logits;        // [T, ld]
   long long ld;
-  const void* bias;           // [E], bf16 or fp32
+  const void* bias;           // [E], bf16 or fp32, or null
   int bias_f32, T, E, K;
   int* idx;                   // [T, K]
   float* w;                   // [T, K]
@@ -27,9 +28,13 @@ struct RouteArgs {
   int* expert_of_tile;        // [tiles]
   int* counts;                // [E]
   int tiles;
+  int sigmoid, groups, keep;  // scores are sigmoids, of the experts of `keep` of `groups` groups of E / groups neighbours
+  float scale;
 };
 
 __device__ __forceinline__ float biased_logit(const RouteArgs& p, const float* z, int e) {
+  if (p.sigmoid) return 1.f / (1.f + expf(-z[e]));
+  if (!p.bias) return z[e];
   return z[e] + (p.bias_f32 ? static_cast<const float*>(p.bias)[e] : to_f(static_cast<const __nv_bfloat16*>(p.bias)[e]));
 }
 // unsigned numbers in the order of the floats; 0 stands for "taken"
@@ -50,6 +55,36 @@ __device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int la
     uint32_t key[PER];
 #pragma unroll
     for (int i = 0; i < PER; ++i) key[i] = lane + i * 32 < p.E ? ordered(biased_logit(p, z, lane + i * 32)) : 0u;
+    if (p.sigmoid && p.keep < p.groups) {      // lane g holds the mark of group g; then the experts of the others are taken out
+      const int n = p.E / p.groups;
+      uint32_t mark = 0u;
+      for (int g = 0; g < p.groups; ++g) {
+        uint32_t b1 = 0u, b2 = 0u;
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+          const int e = lane + i * 32;
+          if (e < p.E && e / n == g) {
+            b2 = max(b2, min(b1, key[i]));
+            b1 = max(b1, key[i]);
+          }
+        }
+        const uint32_t t1 = __reduce_max_sync(0xffffffffu, b1);
+        const uint32_t owner = __ffs(__ballot_sync(0xffffffffu, b1 == t1)) - 1;
+        const uint32_t t2 = __reduce_max_sync(0xffffffffu, uint32_t(lane) == owner ? b2 : b1);
+        const float s = unordered(t1) + (t2 ? unordered(t2) : 0.f);
+        if (lane == g) mark = ordered(s);
+      }
+      uint32_t kept = 0u;
+      for (int k = 0; k < p.keep; ++k) {
+        const uint32_t best = __reduce_max_sync(0xffffffffu, mark);
+        const uint32_t g = __ffs(__ballot_sync(0xffffffffu, mark == best)) - 1;
+        kept |= 1u << g;
+        if (uint32_t(lane) == g) mark = 0u;
+      }
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if (lane + i * 32 < p.E && !((kept >> ((lane + i * 32) / n)) & 1u)) key[i] = 0u;
+    }
     float first = 0.f, sum = 0.f, mine = 0.f;
     int e_mine = 0;
     for (int k = 0; k < p.K; ++k) {
@@ -66,14 +101,14 @@ __device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int la
         if (chosen == lane + i * 32) key[i] = 0u;
       const float v = unordered(top);
       if (k == 0) first = v;
-      const float x = expf(v - first);
+      const float x = p.sigmoid ? v : expf(v - first);
       sum += x;
       if (lane == k) { mine = x; e_mine = chosen; }
     }
     if (lane < p.K) {
       const int i = t * p.K + lane;
       p.idx[i] = e_mine;
-      p.w[i] = mine / sum;
+      p.w[i] = p.sigmoid ? mine / (sum + 1e-20f) * p.scale : mine / sum;
       note(i, e_mine, atomicAdd(count + e_mine, 1));
     }
   } else {
@@ -97,7 +132,7 @@ __device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int la
       last = best;
       last_e = e_best;
       if (k == 0) first = best;
-      const float x = expf(best - first);
+      const float x = p.sigmoid ? best : expf(best - first);
       sum += x;
       if (lane == 0) {
         const int i = t * p.K + k;
@@ -107,7 +142,8 @@ __device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int la
       }
     }
     __syncwarp();
-    for (int k = lane; k < p.K; k += 32) p.w[(long long)t * p.K + k] /= sum;
+    const float f = p.sigmoid ? p.scale / (sum + 1e-20f) : 1.f / sum;
+    for (int k = lane; k < p.K; k += 32) p.w[(long long)t * p.K + k] *= f;
   }
 }
 
@@ -245,7 +281,8 @@ __global__ void __launch_bounds__(256) moe_glu_kernel(const T* __restrict__ in, 
 template <class T, int VEC>
 __global__ void __launch_bounds__(256) moe_weighted_sum_kernel(const T* __restrict__ yp, long long ldp, const int* __restrict__ row_of,
                                                                const float* __restrict__ w, const T* __restrict__ base, long long ldb,
-                                                               T* __restrict__ y, long long ldy, int Tn, int K, int H) {
+                                                               const float* __restrict__ gate, long long ldg, T* __restrict__ y, long long ldy,
+                                                               int Tn, int K, int H) {
   tfb::pdl_sync();
   const int per = H / VEC;
   const long long n = (long long)Tn * per;
@@ -265,8 +302,9 @@ __global__ void __launch_bounds__(256) moe_weighted_sum_kernel(const T* __restri
     if (base) {
       float v[VEC];
       load_n<VEC>(base + t * ldb + c, v);
+      const float f = gate ? 1.f / (1.f + expf(-gate[t * ldg])) : 1.f;
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) acc[e] += v[e];
+      for (int e = 0; e < VEC; ++e) acc[e] = fmaf(f, v[e], acc[e]);
     }
     store_n<VEC>(y + t * ldy + c, acc);
   }
@@ -282,17 +320,23 @@ static int blocks_for(long long items) {
 
 using bf16 = __nv_bfloat16;
 
-// logits [T, ld] fp32, bias [E] (bias_f32: fp32, otherwise bf16).  idx, row_of, rank (scratch): int [T, K]; w: fp32 [T, K]; counts
+// logits [T, ld] fp32, bias [E] (bias_f32: fp32, otherwise bf16) or null; sigmoid, groups, keep, scale: see RouteArgs.  idx, row_of, rank (scratch): int [T, K]; w: fp32 [T, K]; counts
 // (scratch): int [E]; expert_of_tile: int [tiles], tiles >= T K / 128 + min(E, T K).
 TFB_API int tfb_moe_route(const float* logits, const void* bias, int T, int E, int K, int* idx, float* w, int* row_of, int* expert_of_tile,
-                          int* counts, int* rank, int tiles, long long ld, int bias_f32, void* stream) {
+                          int* counts, int* rank, int tiles, long long ld, int bias_f32, int sigmoid, int groups, int keep, float scale,
+                          void* stream) {
   using namespace tfb;
-  if (T <= 0 || E <= 0 || K <= 0 || K > E || !bias) return TFB_ERR_ARG;
+  if (T <= 0 || E <= 0 || K <= 0 || K > E) return TFB_ERR_ARG;
+  if (sigmoid && (bias || groups <= 0 || E % groups || keep <= 0 || keep > groups || K > E / groups * keep)) return TFB_ERR_ARG;
+  if (!sigmoid && groups != 1) return TFB_ERR_ARG;
+  const bool grouped = sigmoid && keep < groups;
   const long long a = (long long)T * K;
   if (tiles < a / 128 + (E < a ? E : a)) return TFB_ERR_ARG;
   if (E > 8192 || a > INT_MAX / 2) return TFB_ERR_LIMIT;
-  RouteArgs p{logits, ld, bias, bias_f32, T, E, K, idx, w, rank, row_of, expert_of_tile, counts, tiles};
+  RouteArgs p{logits, ld, bias, bias_f32, T, E, K, idx, w, rank, row_of, expert_of_tile, counts, tiles, sigmoid, groups, keep, scale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (grouped && (groups > 32 || E > 1024 || K > 32)) return TFB_ERR_LIMIT;
+  if (grouped && E > 256) return launch_route<32>(p, st);
   if (K > 32 || E > 256) return launch_route<0>(p, st);
   return E <= 32 ? launch_route<1>(p, st) : E <= 64 ? launch_route<2>(p, st) : E <= 128 ? launch_route<4>(p, st) : launch_route<8>(p, st);
 }
@@ -330,14 +374,14 @@ TFB_API int tfb_moe_glu(const void* in, long long ldi, const int* row_of, void* 
   return int(cudaGetLastError());
 }
 
-TFB_API int tfb_moe_weighted_sum(const void* yp, long long ldp, const int* row_of, const float* w, const void* base, long long ldb, void* y,
-                                 long long ldy, int T, int K, int H, int f32, void* stream) {
+TFB_API int tfb_moe_weighted_sum(const void* yp, long long ldp, const int* row_of, const float* w, const void* base, long long ldb,
+                                 const float* gate, long long ldg, void* y, long long ldy, int T, int K, int H, int f32, void* stream) {
   using namespace tfb;
   if (T <= 0 || K <= 0 || H <= 0) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int vec = f32 ? 4 : 8;
   const bool v = H % vec == 0 && ldp % vec == 0 && ldy % vec == 0 && al16(yp) && al16(y) && (!base || (ldb % vec == 0 && al16(base)));
-#define TFB_ARGS(Ty) static_cast<const Ty*>(yp), ldp, row_of, w, static_cast<const Ty*>(base), ldb, static_cast<Ty*>(y), ldy, T, K, H
+#define TFB_ARGS(Ty) static_cast<const Ty*>(yp), ldp, row_of, w, static_cast<const Ty*>(base), ldb, gate, ldg, static_cast<Ty*>(y), ldy, T, K, H
   TFB_BY_TYPE(moe_weighted_sum_kernel, blocks_for((long long)T * (v ? H / vec : H)), v, TFB_ARGS);
 #undef TFB_ARGS
   return int(cudaGetLastError());

@@ -9,9 +9,9 @@ namespace tfb {
 TFB_BOUNDS_DEFINE(stack_ops)
 
 // ------------------------------------------------------------------------------------------------
-// x <- x + norm(y) [* scale_post];  a = norm(x), or x itself without w_pre
-// norm: LAYER false: v / rms(v) * (1 + w); LAYER true: (v - mean) / sqrt(mean squared deviation + eps) * w + b.
-// ids != null: x starts as scale * table[id] instead of being read.  rows != null: output row i is computed from row
+// x <- x + norm(y) [* scale_post] [+ y2], y itself without w_post;  a = norm(x), or x itself without w_pre
+// norm: NORM_CENTRED: v / rms(v) * (1 + w); NORM_PLAIN: v / rms(v) * w; NORM_LAYER: (v - mean) / sqrt(mean squared deviation + eps) * w + b.
+// ids != null: x starts as scale * table[id] (normed with w_post if there is no y) instead of being read.  rows != null: output row i is computed from row
 // rows[i] of x and y, and x is left alone (the last norm of a step, for the positions whose logits are wanted).
 // One block per row; the row lives in registers between the two statistics.
 // ------------------------------------------------------------------------------------------------
@@ -25,6 +25,8 @@ struct ResNormArgs {
   long long ldx;
   const void* y;
   long long ldy;
+  const void* y2;
+  long long ldy2;
   const void *w_post, *b_post, *scale_post, *w_pre, *b_pre;
   void* a;
   long long lda;
@@ -33,9 +35,12 @@ struct ResNormArgs {
   float eps;
 };
 
-// statistics of a row held in the block's registers: the mean to subtract (0 unless LAYER) and the factor
-template <bool LAYER, int VEC, int NV>
+enum { NORM_CENTRED = 0, NORM_LAYER = 1, NORM_PLAIN = 2 };
+
+// statistics of a row held in the block's registers: the mean to subtract (0 unless NORM_LAYER) and the factor
+template <int NORM, int VEC, int NV>
 __device__ __forceinline__ float2 row_stats(const float (&v)[NV][VEC], int H, float eps, float* red) {
+  constexpr bool LAYER = NORM == NORM_LAYER;
   const int nt = blockDim.x;
   float mean = 0.f;
   if constexpr (LAYER) {
@@ -61,22 +66,22 @@ __device__ __forceinline__ float2 row_stats(const float (&v)[NV][VEC], int H, fl
   return make_float2(mean, 1.f / sqrtf(block_add(ss, red) / H + eps));
 }
 
-template <class T, bool LAYER, int VEC>
+template <class T, int NORM, int VEC>
 __device__ __forceinline__ void apply_norm(float (&v)[VEC], float2 st, const void* w, const void* b, int col) {
   float wv[VEC];
   load_n<VEC>(static_cast<const T*>(w) + col, wv);
-  if constexpr (LAYER) {
+  if constexpr (NORM == NORM_LAYER) {
     float bv[VEC];
     load_n<VEC>(static_cast<const T*>(b) + col, bv);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) v[e] = (v[e] - st.x) * st.y * wv[e] + bv[e];
   } else {
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) v[e] = v[e] * st.y * (1.f + wv[e]);
+    for (int e = 0; e < VEC; ++e) v[e] = v[e] * st.y * (NORM == NORM_PLAIN ? wv[e] : 1.f + wv[e]);
   }
 }
 
-template <class T, bool LAYER, int VEC, int NV>
+template <class T, int NORM, int VEC, int NV>
 __global__ void res_norm_kernel(const ResNormArgs p) {
   tfb::pdl_sync();
   __shared__ float red[32];
@@ -109,20 +114,34 @@ __global__ void res_norm_kernel(const ResNormArgs p) {
       const int col = (c * nt + threadIdx.x) * VEC;
       if (col < p.H) load_n<VEC>(static_cast<const T*>(p.y) + r * p.ldy + col, yv[c]);
     }
-    const float2 st = row_stats<LAYER, VEC, NV>(yv, p.H, p.eps, red);
+    float2 st = make_float2(0.f, 1.f);
+    if (p.w_post) st = row_stats<NORM, VEC, NV>(yv, p.H, p.eps, red);
 #pragma unroll
     for (int c = 0; c < NV; ++c) {
       const int col = (c * nt + threadIdx.x) * VEC;
       if (col >= p.H) continue;
-      apply_norm<T, LAYER, VEC>(yv[c], st, p.w_post, p.b_post, col);
+      if (p.w_post) apply_norm<T, NORM, VEC>(yv[c], st, p.w_post, p.b_post, col);
       if (p.scale_post) {
         float s[VEC];
         load_n<VEC>(static_cast<const T*>(p.scale_post) + col, s);
 #pragma unroll
         for (int e = 0; e < VEC; ++e) yv[c][e] *= s[e];
       }
+      if (p.y2) {
+        float z[VEC];
+        load_n<VEC>(static_cast<const T*>(p.y2) + r * p.ldy2 + col, z);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) yv[c][e] += z[e];
+      }
 #pragma unroll
       for (int e = 0; e < VEC; ++e) v[c][e] += yv[c][e];
+    }
+  } else if (p.w_post) {                 // the embedding's own norm
+    const float2 st = row_stats<NORM, VEC, NV>(v, p.H, p.eps, red);
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+      const int col = (c * nt + threadIdx.x) * VEC;
+      if (col < p.H) apply_norm<T, NORM, VEC>(v[c], st, p.w_post, p.b_post, col);
     }
   }
   if (!p.rows && (p.y || p.ids)) {
@@ -134,27 +153,27 @@ __global__ void res_norm_kernel(const ResNormArgs p) {
   }
   if (!p.a) return;
   float2 st = make_float2(0.f, 1.f);
-  if (p.w_pre) st = row_stats<LAYER, VEC, NV>(v, p.H, p.eps, red);
+  if (p.w_pre) st = row_stats<NORM, VEC, NV>(v, p.H, p.eps, red);
 #pragma unroll
   for (int c = 0; c < NV; ++c) {
     const int col = (c * nt + threadIdx.x) * VEC;
     if (col >= p.H) continue;
-    if (p.w_pre) apply_norm<T, LAYER, VEC>(v[c], st, p.w_pre, p.b_pre, col);
+    if (p.w_pre) apply_norm<T, NORM, VEC>(v[c], st, p.w_pre, p.b_pre, col);
     store_n<VEC>(static_cast<T*>(p.a) + (long long)i * p.lda + col, v[c]);
   }
 }
 
-template <class T, bool LAYER, int VEC>
+template <class T, int NORM, int VEC>
 static int launch_res_norm(const ResNormArgs& p, int n, cudaStream_t st) {
   const int items = (p.H + VEC - 1) / VEC;
   int nt = (items + 31) / 32 * 32;
   const int cap = VEC == 1 ? 512 : 256;
   if (nt > cap) nt = cap;
   const int nv = (items + nt - 1) / nt;
-  if (nv <= 1) launch_k(res_norm_kernel<T, LAYER, VEC, 1>, n, nt, 0, st, p);
-  else if (nv <= 2) launch_k(res_norm_kernel<T, LAYER, VEC, 2>, n, nt, 0, st, p);
-  else if (nv <= 4) launch_k(res_norm_kernel<T, LAYER, VEC, 4>, n, nt, 0, st, p);
-  else if (nv <= 8) launch_k(res_norm_kernel<T, LAYER, VEC, 8>, n, nt, 0, st, p);
+  if (nv <= 1) launch_k(res_norm_kernel<T, NORM, VEC, 1>, n, nt, 0, st, p);
+  else if (nv <= 2) launch_k(res_norm_kernel<T, NORM, VEC, 2>, n, nt, 0, st, p);
+  else if (nv <= 4) launch_k(res_norm_kernel<T, NORM, VEC, 4>, n, nt, 0, st, p);
+  else if (nv <= 8) launch_k(res_norm_kernel<T, NORM, VEC, 8>, n, nt, 0, st, p);
   else return TFB_ERR_LIMIT;
   return int(cudaGetLastError());
 }
@@ -170,6 +189,12 @@ __device__ __forceinline__ float act_f32(float v, int act) {
   return v;
 }
 
+// 0.5 z (1 + tanh(u)) = z sigmoid(2 u), u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh_exact(float z) {
+  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return z / (1.f + expf(-2.f * u));
+}
+
 template <class T>
 __global__ void __launch_bounds__(256) act_rows_kernel(const T* __restrict__ in, long long ldi, T* __restrict__ out, long long ldo, int M, int N, int act) {
   tfb::pdl_sync();
@@ -179,10 +204,10 @@ __global__ void __launch_bounds__(256) act_rows_kernel(const T* __restrict__ in,
 }
 
 // ------------------------------------------------------------------------------------------------
-// [gate | up] -> silu(gate) * up
+// [gate | up] -> act(gate) * up; act: 0 silu, 1 the tanh form of gelu
 // ------------------------------------------------------------------------------------------------
-template <class T, int VEC>
-__global__ void __launch_bounds__(256) glu_silu_kernel(const T* __restrict__ in, long long ldi, T* __restrict__ out, long long ldo, int M, int F) {
+template <class T, int VEC, int ACT>
+__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, long long ldi, T* __restrict__ out, long long ldo, int M, int F) {
   tfb::pdl_sync();
   const int per = F / VEC;
   const long long n = (long long)M * per;
@@ -193,7 +218,7 @@ __global__ void __launch_bounds__(256) glu_silu_kernel(const T* __restrict__ in,
     load_n<VEC>(in + m * ldi + c, g);
     load_n<VEC>(in + m * ldi + F + c, u);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) g[e] = silu_exact(g[e]) * u[e];
+    for (int e = 0; e < VEC; ++e) g[e] = (ACT == 0 ? silu_exact(g[e]) : gelu_tanh_exact(g[e])) * u[e];
     store_n<VEC>(out + m * ldo + c, g);
   }
 }
@@ -255,6 +280,124 @@ __global__ void __launch_bounds__(256) rope_append_kernel(T* __restrict__ qkv, l
         load_n<VEC>(row + (long long)(nq + nk) * D + i, u);
         store_n<VEC>(vpool + slot * v_cols + i, u);
       }
+    }
+  }
+}
+
+// The same with an RMS norm of every q and k head (weights wq, wk) in front of the rotation.  L lanes share a head, each with eight
+// consecutive entries in registers (L a power of two, 8 L >= D; D, v_cols and half the rotated entries are multiples of eight); partners
+// of a rotation meet by shuffle.  Units of a row: nq + nk heads, then pieces of 8 L entries of v.
+template <class T, int L>
+__global__ void __launch_bounds__(256) norm_rope_append_kernel(T* __restrict__ qkv, long long ld, const T* __restrict__ wq, const T* __restrict__ wk,
+                                                               float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int max_pos,
+                                                               const int* __restrict__ positions, const long long* __restrict__ slots,
+                                                               T* __restrict__ kpool, T* __restrict__ vpool, long long nslots, int rows, int nq,
+                                                               int nk, int D, int dims, int v_cols) {
+  tfb::pdl_sync();
+  const int l = threadIdx.x % L, units = nq + nk + (v_cols + 8 * L - 1) / (8 * L);
+  const long long id = (blockIdx.x * 256ll + threadIdx.x) / L;
+  const bool on = id < (long long)rows * units;
+  const long long r = on ? id / units : 0;
+  const int u = on ? int(id % units) : 0;
+  long long slot = slots ? slots[r] : -1;
+  TFB_BOUNDS(slot < nslots, 51, slot, nslots);
+  if (slot >= nslots) slot = -1;
+  T* row = qkv + r * ld;
+  if (on && u >= nq + nk) {
+    const int c = ((u - nq - nk) * L + l) * 8;
+    if (slot >= 0 && c < v_cols) {
+      float x[8];
+      load_n<8>(row + (long long)(nq + nk) * D + c, x);
+      store_n<8>(vpool + slot * v_cols + c, x);
+    }
+  }
+  const bool head = on && u < nq + nk, mine = head && l * 8 < D;
+  float x[8], ss = 0.f;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) x[e] = 0.f;
+  if (mine) load_n<8>(row + u * D + l * 8, x);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (mine) {
+    float w[8];
+    const float f = 1.f / sqrtf(ss / D + eps);
+    load_n<8>((u < nq ? wq : wk) + l * 8, w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] = x[e] * f * w[e];
+  }
+  const int hv = dims / 16;                        // lanes with a first half of a pair
+  if (hv) {
+    const int other = l < hv ? l + hv : (l < 2 * hv ? l - hv : l), src = (threadIdx.x & 31) - l + other;
+    float y[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) y[e] = __shfl_sync(0xffffffffu, x[e], src);
+    if (mine && l < 2 * hv) {
+      int pos = positions[r];
+      TFB_BOUNDS(pos >= 0 && pos < max_pos, 61, pos, max_pos);
+      pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
+      const long long at = (long long)pos * (dims / 2) + (l < hv ? l : l - hv) * 8;
+      float c[8], s[8];
+      load_n<8>(cos_t + at, c);
+      load_n<8>(sin_t + at, s);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[e] = l < hv ? x[e] * c[e] - y[e] * s[e] : x[e] * c[e] + y[e] * s[e];
+    }
+  }
+  if (mine) {
+    store_n<8>(row + u * D + l * 8, x);
+    if (u >= nq && slot >= 0) store_n<8>(kpool + (slot * nk + (u - nq)) * D + l * 8, x);
+  }
+}
+
+// any sizes: one warp per head (or per 64 entries of v)
+template <class T>
+__global__ void __launch_bounds__(256) norm_rope_append_any_kernel(T* __restrict__ qkv, long long ld, const T* __restrict__ wq, const T* __restrict__ wk,
+                                                                   float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                                                   int max_pos, const int* __restrict__ positions, const long long* __restrict__ slots,
+                                                                   T* __restrict__ kpool, T* __restrict__ vpool, long long nslots, int rows, int nq,
+                                                                   int nk, int D, int dims, int v_cols) {
+  tfb::pdl_sync();
+  const int lane = threadIdx.x & 31, units = nq + nk + (v_cols + 63) / 64, half = dims / 2;
+  const long long id = (blockIdx.x * 256ll + threadIdx.x) / 32;
+  if (id >= (long long)rows * units) return;
+  const long long r = id / units;
+  const int u = int(id % units);
+  long long slot = slots ? slots[r] : -1;
+  TFB_BOUNDS(slot < nslots, 51, slot, nslots);
+  if (slot >= nslots) slot = -1;
+  T* row = qkv + r * ld;
+  if (u >= nq + nk) {
+    for (int c = (u - nq - nk) * 64 + lane; slot >= 0 && c < min(v_cols, (u - nq - nk + 1) * 64); c += 32)
+      vpool[slot * v_cols + c] = row[(long long)(nq + nk) * D + c];
+    return;
+  }
+  T* x = row + u * D;
+  const T* w = u < nq ? wq : wk;
+  T* kp = u >= nq && slot >= 0 ? kpool + (slot * nk + (u - nq)) * D : nullptr;
+  float ss = 0.f;
+  for (int d = lane; d < D; d += 32) ss = fmaf(to_f(x[d]), to_f(x[d]), ss);
+  const float f = 1.f / sqrtf(warp_add(ss) / D + eps);     // its shuffles also order the reads before the writes below
+  int pos = dims ? positions[r] : 0;
+  TFB_BOUNDS(dims == 0 || (pos >= 0 && pos < max_pos), 61, pos, max_pos);
+  pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
+  for (int d = lane; d < D; d += 32) {
+    if (d >= half && d < dims) continue;
+    const float a = to_f(x[d]) * f * to_f(w[d]);
+    if (d >= dims) {
+      x[d] = from_f<T>(a);
+      if (kp) kp[d] = from_f<T>(a);
+      continue;
+    }
+    const float b = to_f(x[d + half]) * f * to_f(w[d + half]);
+    const float c = cos_t[(long long)pos * half + d], s = sin_t[(long long)pos * half + d];
+    const T p = from_f<T>(a * c - b * s), q = from_f<T>(b * c + a * s);
+    x[d] = p;
+    x[d + half] = q;
+    if (kp) {
+      kp[d] = p;
+      kp[d + half] = q;
     }
   }
 }
@@ -369,22 +512,29 @@ static int grid_for(long long items) {
 
 using bf16 = __nv_bfloat16;
 
-// f32 = 1: activations, table and norm weights are fp32, otherwise bf16.  layer: the kind of norm.  See ResNormArgs.
+// f32 = 1: activations, table and norm weights are fp32, otherwise bf16.  norm: its kind (NORM_*).  See ResNormArgs.
 TFB_API int tfb_res_norm(const long long* ids, const void* table, long long ld_table, float scale, int vocab, float* x, long long ldx,
-                         const void* y, long long ldy, const void* w_post, const void* b_post, const void* scale_post, const void* w_pre,
-                         const void* b_pre, void* a, long long lda, const int* rows, int n, int H, float eps, int layer, int f32, void* stream) {
+                         const void* y, long long ldy, const void* y2, long long ldy2, const void* w_post, const void* b_post,
+                         const void* scale_post, const void* w_pre, const void* b_pre, void* a, long long lda, const int* rows, int n, int H,
+                         float eps, int norm, int f32, void* stream) {
   using namespace tfb;
-  if (n <= 0 || H <= 0 || (y && (!w_post || (layer && !b_post))) || (w_pre && (!a || (layer && !b_pre))) || (ids && !table)) return TFB_ERR_ARG;
-  ResNormArgs p{ids, table, ld_table, scale, vocab, x, ldx, y, ldy, w_post, b_post, scale_post, w_pre, b_pre, a, lda, rows, H, eps};
+  const bool layer = norm == NORM_LAYER;
+  if (n <= 0 || H <= 0 || (w_post && (!(y || ids) || (layer && !b_post))) || (w_pre && (!a || (layer && !b_pre))) || (ids && !table) || (y2 && !y) ||
+      norm < 0 || norm > NORM_PLAIN)
+    return TFB_ERR_ARG;
+  ResNormArgs p{ids, table, ld_table, scale, vocab, x, ldx, y, ldy, y2, ldy2, w_post, b_post, scale_post, w_pre, b_pre, a, lda, rows, H, eps};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int es = f32 ? 4 : 2;
   auto ok = [&](int vec) {
     for (const void* q : {w_post, b_post, scale_post, w_pre, b_pre})
       if (q && !aligned(q, vec * es)) return false;
     return H % vec == 0 && ldx % vec == 0 && aligned(x, 16) && (!y || (ldy % vec == 0 && aligned(y, vec * es))) &&
+           (!y2 || (ldy2 % vec == 0 && aligned(y2, vec * es))) &&
            (!a || (lda % vec == 0 && aligned(a, vec * es))) && (!ids || (ld_table % vec == 0 && aligned(table, vec * es)));
   };
-#define TFB_RN(T, VEC) (layer ? launch_res_norm<T, true, VEC>(p, n, st) : launch_res_norm<T, false, VEC>(p, n, st))
+#define TFB_RN(T, VEC)                                        \
+  (layer ? launch_res_norm<T, NORM_LAYER, VEC>(p, n, st)      \
+         : norm == NORM_PLAIN ? launch_res_norm<T, NORM_PLAIN, VEC>(p, n, st) : launch_res_norm<T, NORM_CENTRED, VEC>(p, n, st))
   if (f32) return ok(4) ? TFB_RN(float, 4) : TFB_RN(float, 1);
   if (ok(8)) return TFB_RN(bf16, 8);
   return ok(4) ? TFB_RN(bf16, 4) : TFB_RN(bf16, 1);
@@ -401,20 +551,48 @@ TFB_API int tfb_act_rows(const void* in, long long ldi, void* out, long long ldo
   return int(cudaGetLastError());
 }
 
-TFB_API int tfb_glu_silu(const void* in, long long ldi, void* out, long long ldo, int M, int F, int f32, void* stream) {
+// act: see glu_kernel
+TFB_API int tfb_glu(const void* in, long long ldi, void* out, long long ldo, int M, int F, int act, int f32, void* stream) {
   using namespace tfb;
-  if (M <= 0 || F <= 0) return TFB_ERR_ARG;
+  if (M <= 0 || F <= 0 || act < 0 || act > 1) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int vec = f32 ? 4 : 8;
   const bool v = F % vec == 0 && ldi % vec == 0 && ldo % vec == 0 && aligned(in, 16) && aligned(out, 16);
   const int grid = grid_for((long long)M * (v ? F / vec : F));
-  if (f32) {
-    if (v) launch_k(glu_silu_kernel<float, 4>, grid, 256, 0, st, static_cast<const float*>(in), ldi, static_cast<float*>(out), ldo, M, F);
-    else launch_k(glu_silu_kernel<float, 1>, grid, 256, 0, st, static_cast<const float*>(in), ldi, static_cast<float*>(out), ldo, M, F);
-  } else {
-    if (v) launch_k(glu_silu_kernel<bf16, 8>, grid, 256, 0, st, static_cast<const bf16*>(in), ldi, static_cast<bf16*>(out), ldo, M, F);
-    else launch_k(glu_silu_kernel<bf16, 1>, grid, 256, 0, st, static_cast<const bf16*>(in), ldi, static_cast<bf16*>(out), ldo, M, F);
-  }
+#define TFB_GLU1(T, VEC, ACT) launch_k(glu_kernel<T, VEC, ACT>, grid, 256, 0, st, static_cast<const T*>(in), ldi, static_cast<T*>(out), ldo, M, F)
+#define TFB_GLU(T, VEC) do { if (act) TFB_GLU1(T, VEC, 1); else TFB_GLU1(T, VEC, 0); } while (0)
+  if (f32) { if (v) TFB_GLU(float, 4); else TFB_GLU(float, 1); }
+  else { if (v) TFB_GLU(bf16, 8); else TFB_GLU(bf16, 1); }
+#undef TFB_GLU
+#undef TFB_GLU1
+  return int(cudaGetLastError());
+}
+
+// As tfb_rope_append behind an RMS norm (weights wq, wk of D entries) of every q and k head; dims may be 0.
+TFB_API int tfb_norm_rope_append(void* qkv, long long ld, const void* wq, const void* wk, float eps, const float* cos_t, const float* sin_t,
+                                 int max_pos, const int* positions, const long long* slots, void* kpool, void* vpool, long long nslots, int rows,
+                                 int nq, int nk, int D, int dims, int v_cols, int f32, void* stream) {
+  using namespace tfb;
+  if (rows <= 0 || nq <= 0 || nk <= 0 || D <= 0 || dims < 0 || (dims & 1) || dims > D || (dims && (!cos_t || !sin_t || max_pos <= 0)) || !wq || !wk)
+    return TFB_ERR_ARG;
+  if (nslots == 0) slots = nullptr;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool v = dims % 16 == 0 && D % 8 == 0 && D <= 256 && v_cols % 8 == 0 && ld % (f32 ? 4 : 8) == 0 && aligned(qkv, 16) && aligned(wq, 16) &&
+                 aligned(wk, 16) && (!slots || (aligned(kpool, 16) && aligned(vpool, 16)));
+  const int L = !v ? 32 : D <= 64 ? 8 : D <= 128 ? 16 : 32, piece = v ? 8 * L : 64;
+  const long long blocks = ((long long)rows * (nq + nk + (v_cols + piece - 1) / piece) * L + 255) / 256;
+  if (blocks > 0x7fffffffll) return TFB_ERR_LIMIT;
+#define TFB_NRA(KERN, T) launch_k(KERN, int(blocks), 256, 0, st, static_cast<T*>(qkv), ld, static_cast<const T*>(wq), static_cast<const T*>(wk), eps, \
+                                  cos_t, sin_t, max_pos, positions, slots, static_cast<T*>(kpool), static_cast<T*>(vpool), nslots, rows, nq, nk, D, \
+                                  dims, v_cols)
+#define TFB_NRL(T)                                                          \
+  if (!v) TFB_NRA(norm_rope_append_any_kernel<T>, T);                       \
+  else if (L == 8) TFB_NRA((norm_rope_append_kernel<T, 8>), T);             \
+  else if (L == 16) TFB_NRA((norm_rope_append_kernel<T, 16>), T);           \
+  else TFB_NRA((norm_rope_append_kernel<T, 32>), T);
+  if (f32) { TFB_NRL(float) } else { TFB_NRL(bf16) }
+#undef TFB_NRL
+#undef TFB_NRA
   return int(cudaGetLastError());
 }
 
@@ -422,8 +600,9 @@ TFB_API int tfb_rope_append(void* qkv, long long ld, const float* cos_t, const f
                             const long long* slots, void* kpool, void* vpool, long long nslots, int rows, int nq, int nk, int D, int dims,
                             int v_cols, int f32, void* stream) {
   using namespace tfb;
-  if (rows <= 0 || nq <= 0 || nk < 0 || dims <= 0 || (dims & 1) || dims > D) return TFB_ERR_ARG;
+  if (rows <= 0 || nq <= 0 || nk < 0 || dims < 0 || (dims & 1) || dims > D) return TFB_ERR_ARG;
   if (nk == 0) v_cols = 0;
+  if (dims == 0 && (nk == 0 || !slots || nslots == 0)) return 0;      // nothing to rotate, nothing to keep
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int vec = f32 ? 4 : 8;
   const bool v = (dims / 2) % vec == 0 && D % vec == 0 && v_cols % vec == 0 && ld % vec == 0 && aligned(qkv, 16) &&
