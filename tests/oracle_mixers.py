@@ -327,14 +327,10 @@ def sigmoid(z):
 def rotate_linear(x, pos0, dims, base, factor=1.0):
     """x [T, n, dim] at positions pos0, pos0 + 1, ...: entry i of the first ``dims`` with entry i + dims / 2, all frequencies divided
     by ``factor``."""
-    y = x.clone()
-    for t in range(x.shape[0]):
-        for i in range(dims // 2):
-            a = (pos0 + t) * float(base) ** (-2.0 * i / dims) / factor
-            u, v = x[t, :, i], x[t, :, i + dims // 2]
-            y[t, :, i] = u * math.cos(a) - v * math.sin(a)
-            y[t, :, i + dims // 2] = v * math.cos(a) + u * math.sin(a)
-    return y
+    f = torch.tensor([float(base) ** (-2.0 * i / dims) / factor for i in range(dims // 2)], dtype=DT)
+    a = (torch.arange(pos0, pos0 + x.shape[0], dtype=DT)[:, None] * f)[:, None]
+    u, v = x[..., :dims // 2], x[..., dims // 2:dims]
+    return torch.cat([u * a.cos() - v * a.sin(), v * a.cos() + u * a.sin(), x[..., dims:]], -1)
 
 
 def query_temperature(p, coef, every):
@@ -348,23 +344,21 @@ def soft_cap(s, cap):
 
 def seen(i, j, window=None, keep_first=0):
     """Whether position i looks at position j."""
-    return j <= i and (window is None or i - j < window or j < keep_first)
+    return (j <= i) & ((j < keep_first) | (True if window is None else i - j < window))
 
 
 def attend_options(q, k, v, pos0, scale, window=None, keep_first=0, cap=None, sink=False, temp=None):
     """One head.  q [T, dim] at positions pos0 ..., k [N, dim] and v [N, vdim] at 0 ...; ``cap``: soft cap of the scores; ``sink``: one
     more key of score 0 that has no value; ``temp``: (coef, every) of the queries' factor."""
-    out = []
-    for t in range(q.shape[0]):
-        i = pos0 + t
-        at = torch.tensor([j for j in range(k.shape[0]) if seen(i, j, window, keep_first)])
-        s = (k[at] @ (q[t] * (query_temperature(i, *temp) if temp else 1.0))) * scale
-        if cap:
-            s = soft_cap(s, cap)
-        m = max(float(s.max()), 0.0)
-        e = torch.exp(s - m)
-        out.append((e @ v[at]) / (e.sum() + (math.exp(-m) if sink else 0.0)))
-    return torch.stack(out)
+    at = range(pos0, pos0 + q.shape[0])
+    ok = seen(torch.tensor(at)[:, None], torch.arange(k.shape[0])[None], window, keep_first)
+    f = torch.tensor([query_temperature(p, *temp) if temp else 1.0 for p in at], dtype=DT)
+    s = (q * f[:, None]) @ k.T * scale
+    if cap:
+        s = soft_cap(s, cap)
+    m = torch.where(ok, s, -math.inf).max(-1, keepdim=True).values.clamp(min=0)
+    e = torch.where(ok, torch.exp(s - m), 0.0)
+    return (e @ v) / (e.sum(-1, keepdim=True) + (torch.exp(-m) if sink else 0.0))
 
 
 # ---------------------------------------------------------------------------------------------------- gated linear attention

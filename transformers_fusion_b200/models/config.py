@@ -525,7 +525,7 @@ class FigudraConfig:
         for i, e in enumerate(d["layers"]):
             m, f, src = e["mixer"], e.get("mlp"), e.get("weights_of")
             seen = set()
-            while src is not None and d["layers"][src].get("weights_of") is not None and src not in seen:
+            while src is not None and 0 <= src < len(d["layers"]) and d["layers"][src].get("weights_of") is not None and src not in seen:
                 seen.add(src)                  # the layer at the end of the chain has the tensors
                 src = d["layers"][src]["weights_of"]
             if e["type"] == "attention":
