@@ -432,7 +432,7 @@ def test_long_memory_of_the_state(device):
             if hi > lo:
                 r = K.gla_prep(c(x[lo:hi]).contiguous(), c(a2), c(bias), tau, None, 1, hi - lo, 1, D, V)
                 out.append(K.gla_scan(r, state, slot, None, 1, hi - lo, 1, D, V, lo > 0))
-        close(torch.cat(out)[-1], want, 1e-5)
+        close(torch.cat(out)[-1], want, 5e-5)                # 400 decays near one, each rounded to 2^-24
 
 
 @pytest.mark.parametrize("device", DEVICES)
