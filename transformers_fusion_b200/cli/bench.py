@@ -7,8 +7,8 @@ Kernels: gemm, gemm_nt_wgrad, gemm_fp8, attention_fwd, attention_bwd, rmsnorm, r
 cross_entropy, adamw, paged_decode, sampling, moe_ffn; those of stack models (``STACK_KERNELS``): diff_attention,
 diff_attention_window, attention_fwd_gqa128 (the plain form of the same layer), diff_decode, delta_prep, delta_scan,
 delta_scan_one, gated_norm, delta_prep_step, delta_step, res_norm, glu_silu, rope_append; those of latent attention and the serving
-mixture with the like kernels of the mixture-of-experts decoder (``LATENT_KERNELS``).  ``--kernel`` takes names and the groups all, stack, latent, with commas
-between them.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
+mixture with the like kernels of the mixture-of-experts decoder (``LATENT_KERNELS``); those of attention with options and gated linear
+attention (``GATED_KERNELS``).  ``--kernel`` takes names and the groups all, stack, latent, gated, with commas between them.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
 against their NCCL forms (cli/bench_comm.py)."""
 from __future__ import annotations
 
@@ -28,7 +28,9 @@ LATENT_KERNELS = ("head_attn", "attention_fwd_mha128", "latent_decode", "latent_
                   "head_linear_v", "output_norm", "layernorm", "linear_relu2", "linear_relu2_step", "route", "route_step", "router_topk", "expert_rows",
                   "moe_permute", "expert_gate_up", "expert_gate_up_step", "expert_down", "expert_down_step", "expert_glu", "expert_glu_step",
                   "weighted_sum", "moe_combine", "mixture", "mixture_step", "moe_ffn_step", "kv_append")
-FP32_FMA_PER_SM = 128          # fp32 FMA lanes of an SM (delta_scan is reported against them as well)
+GATED_KERNELS = ("head_attn_cap", "head_attn_window", "head_attn_gqa", "head_decode", "head_decode_cap", "head_decode_window", "gla_prep", "gla_scan",
+                 "gla_scan_one", "gla_step", "norm_rope_append", "parallel_norm", "glu_gelu", "grouped_route", "grouped_route_step", "weighted_sum_gated")
+FP32_FMA_PER_SM = 128          # fp32 FMA lanes of an SM (the scans are reported against them)
 
 
 def _build_stack(kernel, n, dev):
@@ -196,6 +198,70 @@ def _build_latent(kernel, n, dev):
     raise SystemExit(f"Error: unknown kernel '{kernel}'")
 
 
+def _build_gated(kernel, n, dev):
+    """The same for attention with options (16 heads over 4 kv heads of 128; cap 50, a window of 1024 keys and 16 kept ones), gated linear
+    attention (16 heads of 128 x 128) and the grouped mixture; like kernels: attention_fwd_gqa128, paged_decode, delta_*, rope_append,
+    res_norm, glu_silu, route."""
+    import torch
+
+    from ..ops import functional as F
+    from ..ops import moe as M
+    from ..ops import stack as K
+    bf = torch.bfloat16
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s, dtype=bf: torch.randn(*s, device=dev, generator=g).to(dtype)
+    H, G, D, Hd = 16, 4, 128, 2048
+    B = 1 if kernel == "gla_scan_one" else max(1, (1 << 14) // n)
+    T, sc = B * n, D ** -0.5
+    opt = K.HeadOptions(softcap=50.0, temp_coef=0.1, temp_every=8192) if kernel.endswith("_cap") else \
+        K.HeadOptions(window=1024, keep_first=16, sink=True) if kernel.endswith("_window") else K.PLAIN
+    if kernel.startswith("head_attn"):
+        p = rnd(T, (2 * H + 2 * G) * D)
+        q, k, v = p[:, :H * D], p[:, H * D:(H + G) * D], p[:, (H + G) * D:(H + 2 * G) * D]
+        gate = p[:, (H + 2 * G) * D:] if opt.softcap else None
+        keys = sum(min(i + 1, opt.window + opt.keep_first if opt.window else n) for i in range(n))
+        return (lambda: K.head_attn(q, k, v, B, n, n, H, G, D, D, sc, gate, opt)), 4.0 * B * H * keys * D, T * (p.shape[1] + H * D) * 2
+    if kernel.startswith("head_decode"):
+        B, pages = 64, 64 * (n // 16)
+        kp, vp, q, gate = rnd(pages * 16, G * D), rnd(pages * 16, G * D), rnd(B, H * D), rnd(B, H * D)
+        bt = torch.randperm(pages, device=dev, generator=g).int().view(B, -1).contiguous()
+        pos, keys = torch.full((B,), n - 1, dtype=torch.int32, device=dev), min(n, opt.window + opt.keep_first) if opt.window else n
+        return (lambda: K.head_decode(q, kp, vp, bt, pos, H, G, D, D, sc, gate if opt.softcap else None, opt)), 4.0 * B * H * keys * D, B * keys * G * 2 * D * 2
+    if kernel.startswith("gla_"):
+        if kernel == "gla_step":
+            B, n, T = 64, 1, 64
+        p, a2, bias, w = rnd(T, 4 * H * D + 16), rnd(H * D, 16), rnd(H * D), rnd(D)
+        st, sl = torch.zeros(B, H, D, D, device=dev), torch.arange(B, dtype=torch.int32, device=dev)
+        if kernel == "gla_step":
+            return (lambda: K.gla_step(p, a2, bias, 16.0, st, sl, w, 1e-5, B, H, D, D)), 0.0, B * H * D * D * 8
+        prep = lambda: K.gla_prep(p, a2, bias, 16.0, None, B, n, H, D, D)
+        if kernel == "gla_prep":
+            return prep, 0.0, T * H * (3 * D * (2 + 4) + D)
+        r = prep()
+        return (lambda: K.gla_scan(r, st, sl, None, B, n, H, D, D, False)), 6.0 * T * H * D * D, T * H * (4 * D * 4 + D + 16)
+    T = 64 if kernel.endswith("_step") else 1 << 14
+    if kernel == "norm_rope_append":
+        p, tab = rnd(T, (H + 2 * G) * D), F.rope_tables(64, T, device=dev)
+        pos, slots, w = torch.arange(T, device=dev, dtype=torch.int32), torch.arange(T, device=dev), rnd(D)
+        kp, vp = rnd(T, G * D), rnd(T, G * D)
+        return (lambda: K.rope_append(p, tab, pos, H, G, D, 64, G * D, slots, kp, vp, (w, w, 1e-5))), 0.0, T * D * ((H + G) * 4 + G * 2 + G * 4)
+    if kernel == "parallel_norm":
+        x, y, z, w = rnd(T, Hd, dtype=torch.float32), rnd(T, Hd), rnd(T, Hd), rnd(Hd)
+        return (lambda: K.res_norm(x, 1e-5, y=y, y2=z, w_pre=w, kind="plain")), 0.0, T * Hd * 14
+    if kernel == "glu_gelu":
+        gu = rnd(T, 2 * 5632)
+        return (lambda: K.glu(gu, "gelu_tanh")), 0.0, T * 5632 * 6
+    z = rnd(T, 63, dtype=torch.float32)
+    route = lambda: M.route(z[:, :62], None, 6, "sigmoid", 2, 1, 1.5)
+    if kernel.startswith("grouped_route"):
+        return route, 0.0, T * (62 * 4 + 6 * 12)
+    if kernel == "weighted_sum_gated":
+        h, r = rnd(T, Hd), route()
+        o = M.expert_rows(h, r)
+        return (lambda: M.weighted_sum(o, r, h, z[:, 62:])), 0.0, T * 8 * Hd * 2
+    raise SystemExit(f"Error: unknown kernel '{kernel}'")
+
+
 def _build(kernel, n, dev, heads=0, shape=None):
     """Returns (callable, flops, bytes) for one launch of ``kernel`` at problem size ``n``."""
     import torch
@@ -204,6 +270,8 @@ def _build(kernel, n, dev, heads=0, shape=None):
         return _build_stack(kernel, n, dev)
     if kernel in LATENT_KERNELS:
         return _build_latent(kernel, n, dev)
+    if kernel in GATED_KERNELS:
+        return _build_gated(kernel, n, dev)
 
     from ..ops import functional as F
     bf = torch.bfloat16
@@ -528,7 +596,7 @@ def main(argv=None):
         if not torch.cuda.is_available():
             print("Error: kernel benchmarks need a CUDA device", file=sys.stderr)
             return 1
-        groups = {"all": KERNELS, "stack": STACK_KERNELS, "latent": LATENT_KERNELS}
+        groups = {"all": KERNELS, "stack": STACK_KERNELS, "latent": LATENT_KERNELS, "gated": GATED_KERNELS}
         names = [n for k in a.kernel.split(",") for n in groups.get(k, (k,))]
         peaks = json.load(open(a.peaks)) if a.peaks else {}
         for name in names:
@@ -543,7 +611,7 @@ def main(argv=None):
                    "gbs": round(nbytes / best / 1e6, 1), "tflops": round(flops / best / 1e9, 2)}
             if peaks:
                 rec["frac_hbm_of_measured"] = round(rec["gbs"] / peaks["hbm_gbs"], 3)
-                if name.startswith("delta_scan"):      # fp32 arithmetic: against the FMA lanes at the largest clock
+                if name.startswith(("delta_scan", "gla_scan")):      # fp32 arithmetic: against the FMA lanes at the largest clock
                     sms = torch.cuda.get_device_properties(0).multi_processor_count
                     rec["frac_fp32_fma"] = round(rec["tflops"] / (2 * FP32_FMA_PER_SM * sms * peaks.get("sm_max_mhz", 1965.0) * 1e-6), 3)
                 elif flops:

@@ -45,6 +45,9 @@ __device__ __forceinline__ float rcp(float x) {
   return y;
 }
 
+// for the output gates; relative error about 3e-7
+__device__ __forceinline__ float sigmoid_gate(float x) { return rcp(1.f + ex2(-LOG2E * x)); }
+
 // tanh by its definition; absolute error about 2e-7
 __device__ __forceinline__ float tanh_any(float x) {
   const float t = fmaf(-2.f, rcp(1.f + ex2(2.f * LOG2E * fabsf(x))), 1.f);
@@ -393,7 +396,7 @@ head_attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
               float g[8];
               load_n<8>(p.gate + row * p.ldg + h * p.V + c * 8, g);
 #pragma unroll
-              for (int e = 0; e < 8; ++e) o[c * 8 + e] *= sigmoid_exact(g[e]);
+              for (int e = 0; e < 8; ++e) o[c * 8 + e] *= sigmoid_gate(g[e]);
             }
             uint4 u;
             u.x = pack_bf16(o[c * 8 + 0] * f, o[c * 8 + 1] * f);
@@ -700,7 +703,7 @@ __global__ void __launch_bounds__(128) head_combine_kernel(const float* __restri
     if (d >= V) continue;
     if (gate && gate_entry) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v[e] *= sigmoid_exact(__bfloat162float(gate[b * ldg + (long long)h * V + d + e]));
+      for (int e = 0; e < 4; ++e) v[e] *= sigmoid_gate(__bfloat162float(gate[b * ldg + (long long)h * V + d + e]));
     }
     store_n<4>(o + b * ldo + (long long)h * V + d, v);
   }

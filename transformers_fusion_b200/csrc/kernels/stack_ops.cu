@@ -284,70 +284,94 @@ __global__ void __launch_bounds__(256) rope_append_kernel(T* __restrict__ qkv, l
   }
 }
 
-// The same with an RMS norm of every q and k head (weights wq, wk) in front of the rotation.  L lanes share a head, each with eight
-// consecutive entries in registers (L a power of two, 8 L >= D; D, v_cols and half the rotated entries are multiples of eight); partners
-// of a rotation meet by shuffle.  Units of a row: nq + nk heads, then pieces of 8 L entries of v.
+// The same with an RMS norm of every q and k head (weights wq, wk) in front of the rotation.  L lanes share a head, each with two pieces
+// of four entries in registers: for rotated entries, four of the first half and their partners in the second (L a power of two,
+// 8 L >= D; D, v_cols and the rotated entries are multiples of eight).  Units of a row: nq + nk heads, then pieces of 8 L entries of v; a
+// group of L lanes takes NRA_UNITS of them, all loads ahead of the reductions.
+constexpr int NRA_UNITS = 2;
 template <class T, int L>
-__global__ void __launch_bounds__(256) norm_rope_append_kernel(T* __restrict__ qkv, long long ld, const T* __restrict__ wq, const T* __restrict__ wk,
-                                                               float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t, int max_pos,
-                                                               const int* __restrict__ positions, const long long* __restrict__ slots,
-                                                               T* __restrict__ kpool, T* __restrict__ vpool, long long nslots, int rows, int nq,
-                                                               int nk, int D, int dims, int v_cols) {
+__global__ void __launch_bounds__(256, 4) norm_rope_append_kernel(T* __restrict__ qkv, long long ld, const T* __restrict__ wq, const T* __restrict__ wk,
+                                                                  float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                                                  int max_pos, const int* __restrict__ positions, const long long* __restrict__ slots,
+                                                                  T* __restrict__ kpool, T* __restrict__ vpool, long long nslots, int rows, int nq,
+                                                                  int nk, int D, int dims, int v_cols) {
   tfb::pdl_sync();
-  const int l = threadIdx.x % L, units = nq + nk + (v_cols + 8 * L - 1) / (8 * L);
-  const long long id = (blockIdx.x * 256ll + threadIdx.x) / L;
-  const bool on = id < (long long)rows * units;
-  const long long r = on ? id / units : 0;
-  const int u = on ? int(id % units) : 0;
+  const int l = threadIdx.x % L, heads = nq + nk, units = heads + (v_cols + 8 * L - 1) / (8 * L), per = (units + NRA_UNITS - 1) / NRA_UNITS;
+  const int id = (blockIdx.x * 256 + threadIdx.x) / L, r = min(id / per, rows - 1), u0 = id - id / per * per;
+  const bool on = id < rows * per, turns = l * 8 < dims;
+  const int c0 = turns ? l * 4 : l * 8, c1 = turns ? dims / 2 + l * 4 : l * 8 + 4;     // this lane's entries of a head
+  T* row = qkv + r * ld;
+  float x[NRA_UNITS][2][4], w[NRA_UNITS][2][4], c[4], s[4];
+  int at[NRA_UNITS];                               // first entry of the unit in the row; negative: none for this lane
+#pragma unroll
+  for (int i = 0; i < NRA_UNITS; ++i) {
+    const int u = u0 + i * per;
+    at[i] = u < heads ? u * D : heads * D + (u - heads) * 8 * L;
+    if (!on || u >= units || (u < heads ? l * 8 >= D : at[i] + l * 8 >= heads * D + v_cols)) at[i] = -1;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[i][0][e] = x[i][1][e] = 0.f;
+    if (at[i] < 0) continue;
+    const int a = u < heads ? c0 : l * 8, b = u < heads ? c1 : l * 8 + 4;
+    load_n<4>(row + at[i] + a, x[i][0]);
+    load_n<4>(row + at[i] + b, x[i][1]);
+    if (u < heads) {
+      load_n<4>((u < nq ? wq : wk) + c0, w[i][0]);
+      load_n<4>((u < nq ? wq : wk) + c1, w[i][1]);
+    }
+  }
+  if (turns) {
+    int pos = positions[r];
+    TFB_BOUNDS(pos >= 0 && pos < max_pos, 61, pos, max_pos);
+    pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
+    load_n<4>(cos_t + (long long)pos * (dims / 2) + c0, c);
+    load_n<4>(sin_t + (long long)pos * (dims / 2) + c0, s);
+  }
   long long slot = slots ? slots[r] : -1;
   TFB_BOUNDS(slot < nslots, 51, slot, nslots);
   if (slot >= nslots) slot = -1;
-  T* row = qkv + r * ld;
-  if (on && u >= nq + nk) {
-    const int c = ((u - nq - nk) * L + l) * 8;
-    if (slot >= 0 && c < v_cols) {
-      float x[8];
-      load_n<8>(row + (long long)(nq + nk) * D + c, x);
-      store_n<8>(vpool + slot * v_cols + c, x);
+  float ss[NRA_UNITS];
+#pragma unroll
+  for (int i = 0; i < NRA_UNITS; ++i) {
+    ss[i] = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss[i] = fmaf(x[i][0][e], x[i][0][e], fmaf(x[i][1][e], x[i][1][e], ss[i]));
+  }
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1)
+#pragma unroll
+    for (int i = 0; i < NRA_UNITS; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+  const float inv = 1.f / D;
+#pragma unroll
+  for (int i = 0; i < NRA_UNITS; ++i) {
+    if (at[i] < 0) continue;
+    const int u = u0 + i * per;
+    if (u >= heads) {
+      if (slot >= 0) {
+        T* vp = vpool + slot * v_cols + (u - heads) * 8 * L + l * 8;
+        store_n<4>(vp, x[i][0]);
+        store_n<4>(vp + 4, x[i][1]);
+      }
+      continue;
     }
-  }
-  const bool head = on && u < nq + nk, mine = head && l * 8 < D;
-  float x[8], ss = 0.f;
+    const float f = rsqrtf(fmaf(ss[i], inv, eps));
+    float a[4], b[4];
 #pragma unroll
-  for (int e = 0; e < 8; ++e) x[e] = 0.f;
-  if (mine) load_n<8>(row + u * D + l * 8, x);
-#pragma unroll
-  for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
-#pragma unroll
-  for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  if (mine) {
-    float w[8];
-    const float f = 1.f / sqrtf(ss / D + eps);
-    load_n<8>((u < nq ? wq : wk) + l * 8, w);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) x[e] = x[e] * f * w[e];
-  }
-  const int hv = dims / 16;                        // lanes with a first half of a pair
-  if (hv) {
-    const int other = l < hv ? l + hv : (l < 2 * hv ? l - hv : l), src = (threadIdx.x & 31) - l + other;
-    float y[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) y[e] = __shfl_sync(0xffffffffu, x[e], src);
-    if (mine && l < 2 * hv) {
-      int pos = positions[r];
-      TFB_BOUNDS(pos >= 0 && pos < max_pos, 61, pos, max_pos);
-      pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
-      const long long at = (long long)pos * (dims / 2) + (l < hv ? l : l - hv) * 8;
-      float c[8], s[8];
-      load_n<8>(cos_t + at, c);
-      load_n<8>(sin_t + at, s);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] = l < hv ? x[e] * c[e] - y[e] * s[e] : x[e] * c[e] + y[e] * s[e];
+    for (int e = 0; e < 4; ++e) {
+      a[e] = x[i][0][e] * f * w[i][0][e];
+      b[e] = x[i][1][e] * f * w[i][1][e];
+      if (turns) {
+        const float p = a[e] * c[e] - b[e] * s[e];
+        b[e] = b[e] * c[e] + a[e] * s[e];
+        a[e] = p;
+      }
     }
-  }
-  if (mine) {
-    store_n<8>(row + u * D + l * 8, x);
-    if (u >= nq && slot >= 0) store_n<8>(kpool + (slot * nk + (u - nq)) * D + l * 8, x);
+    store_n<4>(row + at[i] + c0, a);
+    store_n<4>(row + at[i] + c1, b);
+    if (u >= nq && slot >= 0) {
+      T* kp = kpool + (slot * nk + (u - nq)) * D;
+      store_n<4>(kp + c0, a);
+      store_n<4>(kp + c1, b);
+    }
   }
 }
 
@@ -577,11 +601,12 @@ TFB_API int tfb_norm_rope_append(void* qkv, long long ld, const void* wq, const 
     return TFB_ERR_ARG;
   if (nslots == 0) slots = nullptr;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const bool v = dims % 16 == 0 && D % 8 == 0 && D <= 256 && v_cols % 8 == 0 && ld % (f32 ? 4 : 8) == 0 && aligned(qkv, 16) && aligned(wq, 16) &&
+  const bool v = dims % 8 == 0 && D % 8 == 0 && D <= 256 && v_cols % 8 == 0 && ld % (f32 ? 4 : 8) == 0 && aligned(qkv, 16) && aligned(wq, 16) &&
                  aligned(wk, 16) && (!slots || (aligned(kpool, 16) && aligned(vpool, 16)));
   const int L = !v ? 32 : D <= 64 ? 8 : D <= 128 ? 16 : 32, piece = v ? 8 * L : 64;
-  const long long blocks = ((long long)rows * (nq + nk + (v_cols + piece - 1) / piece) * L + 255) / 256;
-  if (blocks > 0x7fffffffll) return TFB_ERR_LIMIT;
+  const int units = nq + nk + (v_cols + piece - 1) / piece;
+  const long long blocks = ((long long)rows * (v ? (units + NRA_UNITS - 1) / NRA_UNITS : units) * L + 255) / 256;
+  if (blocks * 256 > 0x7fffffffll) return TFB_ERR_LIMIT;
 #define TFB_NRA(KERN, T) launch_k(KERN, int(blocks), 256, 0, st, static_cast<T*>(qkv), ld, static_cast<const T*>(wq), static_cast<const T*>(wk), eps, \
                                   cos_t, sin_t, max_pos, positions, slots, static_cast<T*>(kpool), static_cast<T*>(vpool), nslots, rows, nq, nk, D, \
                                   dims, v_cols)

@@ -649,6 +649,15 @@ def preset(name: str) -> TransformerConfig:
             (4096, 32, 32, 32000, MixtureSpec(7, 1, 14336, 14336), 43008)
         att = LatentAttentionSpec(heads, 128, 128, 512, 128 ** -0.5)
         return TekenexConfig(V, H, [StackLayer(att, 0 if i else ff, mix if i else None) for i in range(n)], 1e-5)
+    if name in ("figudra-7b", "figudra-8x7b"):
+        # beside mixture-7b and mixtral-8x7b: the same width, query and key / value rows and feed-forward work per token (one shared
+        # expert among it); one layer in three of each mixer, the first one's feed-forward dense
+        H, heads, kv, n, V, win, mix, ff = (2048, 16, 4, 24, 32000, 1024, MixtureSpec(62, 6, 704, 1408, True, "sigmoid", 2, 1, 1.5), 5632) \
+            if name == "figudra-7b" else (4096, 32, 8, 32, 32000, 4096, MixtureSpec(7, 1, 14336, 14336, True, "sigmoid"), 28672)
+        mixers = (HeadAttentionSpec(heads, kv, 128, 128, 128 ** -0.5, gate=True, softcap=50.0, temp_coef=0.1, temp_every=8192),
+                  HeadAttentionSpec(heads, kv, 128, 128, 128 ** -0.5, RotarySpec(64, 500000.0, linear=4.0), True, window=win, keep_first=16, sink=True),
+                  GatedLinearSpec(heads, 128, 128, 16.0))
+        return FigudraConfig(V, H, [StackLayer(mixers[i % 3], 0 if i else ff, mix if i else None) for i in range(n)], 1e-5)
     if name == "mixture-7b":
         return MoEConfig(vocab_size=32000, hidden_size=2048, num_layers=24, num_heads=16, num_kv_heads=4, ffn_hidden_size=704, rope_theta=500000.0,
                          max_seq_len=32768, activation="swiglu", num_experts=64, top_k=8)
