@@ -381,6 +381,8 @@ def test_gated_linear_prompts(device, H, D, V, rank, tau):
             out.copy_(rows[:, lo:hi].reshape(-1, p.shape[1]))
             return out
         n = torch.tensor(lens, dtype=torch.int32, device=device)
+        junk = torch.full((1 << 20,), float("nan"), device=device)   # what freed memory may hold
+        del junk
         whole = one(0, S, n, False)
         ends = state.clone()
         a = one(0, first, None, False)
@@ -388,6 +390,7 @@ def test_gated_linear_prompts(device, H, D, V, rank, tau):
         for i, L in enumerate(lens):
             want, _, last = gla_plain(rows[i, :L], a2, bias, tau, H, D, V)
             close(whole[i, :L], want, tol)
+            assert not whole[i, L:].any()                          # padding: zeros, whatever the memory held
             close(a[i], want[:first], tol)
             close(b[i, :L - first], want[first:], tol)
             for s in (ends, state):
@@ -530,6 +533,8 @@ def test_batches_of_unequal_requests(name, run):
     seqs = [toks(l + 20, V, 10 + i) for i, l in enumerate(lens)]
     want = [plain.run(s) for s in seqs]
     eng = engine(m, max_batch=5, num_pages=24)
+    junk = [torch.full((n,), float("nan"), device=run[0]) for n in (1 << 12, 1 << 16, 1 << 18, 1 << 20, 1 << 24)]
+    del junk                             # what freed memory may hold: padding must not bring it in
     for rep in range(2):                 # the second pass runs on pages and slots that the first one gave back
         reqs = [Request([]) for _ in seqs]
         outs = eng.feed([(r, s[:l], [l - 1] if i % 2 else list(range(l))) for i, (r, s, l) in enumerate(zip(reqs, seqs, lens))])

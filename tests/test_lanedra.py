@@ -228,6 +228,7 @@ def test_delta_rule(device, H, G, D, V, taps, dtype):
         o = o.cpu().double().view(B, S, -1)
         for b in range(B):
             ref = want[b][0][at[b]:at[b] + ln[b]]
+            assert not o[b, ln[b]:].any()                  # padding: zeros, whatever the memory held
             assert float((o[b, :ln[b]] - ref).abs().max()) < (1e-4 if dtype == torch.float32 else 0.01) * max(1.0, float(ref.abs().max()))
             at[b] += ln[b]
     for b, s in enumerate(slots):

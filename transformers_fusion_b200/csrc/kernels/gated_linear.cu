@@ -326,6 +326,8 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
     while (globaltimer_ns() - t0 < 200000ull) {}      // bounded wait for copies already issued
     return;
   }
+  if (writer)                            // padding: numbers, since a weight of zero does not silence what is not one
+    for (int s = len; s < p.S; ++s) orow[s * ostep] = 0.f;
   if (S0) {
 #pragma unroll
     for (int x = 0; x < CPT; ++x)

@@ -519,7 +519,7 @@ def delta_prep(proj, conv_w, conv_state, state_slots, A_log, dt_bias, lens, B, S
 
 def delta_scan(rows_: DeltaRows, state, state_slots, lens, B, S, G, H, D, V, has_past):
     """The recurrence over prepared rows; ``state`` [slots, H, D, V] fp32 is read (``has_past``) and updated.  Returns fp32
-    [B*S, H, V] (rows past a sequence's length are unspecified)."""
+    [B*S, H, V] (rows past a sequence's length are zero)."""
     r = rows_
     if not r.q.is_cuda:
         out = torch.zeros(B * S, H, V)
@@ -603,7 +603,7 @@ def gla_prep(proj, a2, bias, tau, lens, B, S, H, D, V) -> GlaRows:
 
 def gla_scan(rows_: GlaRows, state, state_slots, lens, B, S, H, D, V, has_past):
     """S <- diag(decay) S + k v^T, o = S^T q over prepared rows; ``state`` [slots, H, D, V] fp32 is read (``has_past``) and updated.
-    Returns fp32 [B*S, H, V] (rows past a sequence's length are unspecified)."""
+    Returns fp32 [B*S, H, V] (rows past a sequence's length are zero)."""
     r = rows_
     if not r.q.is_cuda:
         out = torch.zeros(B * S, H, V)
