@@ -911,11 +911,23 @@ TFB_API int tfb_head_attn(const void* q, long long ldq, const void* k, long long
 #undef TFB_ANY
 }
 
-// Blocks per sequence (and key split) of the tensor-core form of tfb_head_decode, which then needs acc and ml; 0: the other form.
-TFB_API int tfb_head_decode_blocks(int H, int G, int D, int V, int f32) {
-  if (f32 || G <= 0 || H % G || D % 8 || V % 8 || D <= 0 || V <= 0 || D > 128 || V > 128) return 0;
+// Key splits of the tensor-core form of tfb_head_decode for up to max_keys keys per query (it then needs acc and ml); 0: the other form.
+// The blocks of a step run in rounds of as many as fit on the device at once: the split with the fewest keys times rounds, and
+// something for every split's own start and merge.
+TFB_API int tfb_head_decode_plan(int B, int H, int G, int D, int V, int max_keys, int f32) {
+  if (f32 || B <= 0 || G <= 0 || H % G || D % 8 || V % 8 || D <= 0 || V <= 0 || D > 128 || V > 128) return 0;
   const int R = H / G;
-  return G * (R <= 8 ? 1 : (R + 15) / 16);
+  const long long items = (long long)B * G * (R <= 8 ? 1 : (R + 15) / 16), slots = (long long)tfb::sm_count() * (D <= 64 && V <= 64 ? 5 : 3);
+  int best = 1;
+  double cost = 1e30;
+  for (int s = 1; s <= 32 && (s == 1 || max_keys / s >= 128); ++s) {
+    const double c = double((items * s + slots - 1) / slots) * (double(max_keys) / s + 96);
+    if (c < cost) {
+      cost = c;
+      best = s;
+    }
+  }
+  return best;
 }
 
 // One query per sequence at positions[b] over the cached rows (k [nslots][G D], v [nslots][G V]); q [B, ldq], o [B, ldo].
@@ -927,7 +939,7 @@ TFB_API int tfb_head_decode(const void* q, long long ldq, const void* k, const v
   const HeadOpt opt{window, keep, cap, sink, temp_coef, temp_every};
   if (B <= 0 || B > 65535 || G <= 0 || H % G || D <= 0 || V <= 0 || page <= 0 || nslots < page || bad_opt(opt)) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (acc && tfb_head_decode_blocks(H, G, D, V, f32) > 0) {
+  if (acc && tfb_head_decode_plan(B, H, G, D, V, 1, f32) > 0) {
     if (!ml || splits < 1 || splits > 32 || ldq % 8 || ldo % 4 || !al16(q) || !al16(k) || !al16(v) || !al16(o)) return TFB_ERR_ARG;
     HeadDecodeArgs p{static_cast<const bf16*>(q), ldq, static_cast<const bf16*>(k), static_cast<const bf16*>(v), nslots, block_table, max_pages, page,
                      positions, H, G, D, V, splits, scale, opt, acc, ml, status};

@@ -40,7 +40,7 @@ _lib.register("tfb_skinny_linear_heads", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, 
 _lib.register("tfb_gemm_f32_heads", [c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_head_attn", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_f, c_i,
                                 c_f, c_i, c_i, c_i, c_p, c_p])
-_lib.register("tfb_head_decode_blocks", [c_i, c_i, c_i, c_i, c_i])
+_lib.register("tfb_head_decode_plan", [c_i, c_i, c_i, c_i, c_i, c_i, c_i])
 _lib.register("tfb_head_decode", [c_p, c_ll, c_p, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_ll, c_i, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
                                   c_i, c_i, c_f, c_i, c_f, c_i, c_i, c_p, c_p])
 _lib.register("tfb_gla_prep", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_f, c_p] + [c_p] * 5 + [c_i] * 7 + [c_p])
@@ -365,11 +365,11 @@ def head_decode(q, kpool, vpool, block_table, positions, H, G, D, V, scale, gate
     L, f32 = _lib.lib(), _f32(q)
     o = rows(B, H * V, q.dtype, q.device)
     acc = ml = None
-    n = L.tfb_head_decode_blocks(H, G, D, V, f32)        # blocks per sequence of the tensor-core form, 0: the other form
+    keys = block_table.shape[1] * PAGE
+    keys = min(keys, opt.window + opt.keep_first) if opt.window else keys
+    n = L.tfb_head_decode_plan(B, H, G, D, V, keys, f32)         # key splits of the tensor-core form, 0: the other form
     if n and q.stride(0) % 8 == 0:
-        keys = block_table.shape[1] * PAGE
-        keys = min(keys, opt.window + opt.keep_first) if opt.window else keys
-        splits = splits or max(1, min(32, (4 * 148) // (B * n), keys // 128))
+        splits = splits or n
         acc = torch.empty(B * H * splits * V, dtype=torch.float32, device=q.device)
         ml = torch.empty(B * H * splits * 2, dtype=torch.float32, device=q.device)
     check(L.tfb_head_decode(q.data_ptr(), q.stride(0), kpool.data_ptr(), vpool.data_ptr(), kpool.shape[0], block_table.data_ptr(),
