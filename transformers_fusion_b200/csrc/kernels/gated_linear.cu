@@ -32,37 +32,21 @@ struct GlaProj {
   int H, D, V;
 };
 
-// sigmoid(z)^(1 / tau)
-__device__ __forceinline__ float channel_decay(float z, float tau) {
-  const float ls = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
-  return expf(ls / tau);
-}
-
-// z of channel c (of all heads) for N tokens with rows a1[i]
-template <class T, int N>
-__device__ __forceinline__ void decay_logits(const GlaProj& p, const T* const (&a1)[N], long long c, bool vec, float (&z)[N]) {
-  const T* w = static_cast<const T*>(p.a2) + c * p.ld2;
-  const float b = to_f(static_cast<const T*>(p.bias)[c]);
-#pragma unroll
-  for (int i = 0; i < N; ++i) z[i] = b;
-  if (vec) {
-    for (int r = 0; r < p.rank; r += 8) {
-      float x[8], y[8];
-      load_n<8>(w + r, x);
-#pragma unroll
-      for (int i = 0; i < N; ++i) {
-        load_n<8>(a1[i] + r, y);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) z[i] = fmaf(x[e], y[e], z[i]);
-      }
-    }
-  } else {
-    for (int r = 0; r < p.rank; ++r) {
-      const float x = to_f(w[r]);
-#pragma unroll
-      for (int i = 0; i < N; ++i) z[i] = fmaf(x, to_f(a1[i][r]), z[i]);
-    }
-  }
+// sigmoid(z)^(1 / tau) = exp((min(z, 0) - ln(1 + x)) / tau), x = exp(-|z|).  ln(1 + x) = 2 atanh(u) with u = x / (2 + x) <= 1 / 3, by the
+// odd series up to u^13 (the next term is below 2^-25 of the sum); accurate relative to itself, so slow decays keep their digits.
+__device__ __forceinline__ float channel_decay(float z, float inv_tau) {
+  const float x = expf(-fabsf(z));
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(2.f + x));
+  const float u = x * r, y = u * u;
+  float p = 1.f / 13.f;
+  p = fmaf(p, y, 1.f / 11.f);
+  p = fmaf(p, y, 1.f / 9.f);
+  p = fmaf(p, y, 1.f / 7.f);
+  p = fmaf(p, y, 1.f / 5.f);
+  p = fmaf(p, y, 1.f / 3.f);
+  p = fmaf(p, y, 1.f);
+  return expf((fminf(z, 0.f) - 2.f * u * p) * inv_tau);
 }
 
 // ------------------------------------------------------------------------------------------------
@@ -73,59 +57,93 @@ struct GlaPrepArgs {
   const int* lens;                  // [B] tokens of each sequence in this call (null: S)
   float *q, *k, *v, *decay, *pair;  // [B, H, Sp, Dp] twice, [B, H, Sp, Vp], [B, H, Sp / 4, Dp], [B, H, Sp / 4, 16]
   int S, Sp, Dp, Vp;
-  int vec;                          // rows of a1 and a2 can be read eight entries at a time
+  int vec;                          // rows of a2 can be read eight entries at a time
 };
 
+constexpr int PREP_WARPS = 4;
+
 template <class T>
-__global__ void __launch_bounds__(128) gla_prep_kernel(const GlaPrepArgs p) {
+__global__ void __launch_bounds__(PREP_WARPS * 32) gla_prep_kernel(const GlaPrepArgs p) {
   tfb::pdl_sync();
+  extern __shared__ __align__(16) float s_a1[];       // [warp][4][rank rounded up to 8] rows of a1, zeros past the rank
   const GlaProj& g = p.g;
-  const int blk = blockIdx.x * 4 + (threadIdx.x >> 5), h = blockIdx.y, b = blockIdx.z, lane = threadIdx.x & 31;
-  const int len = p.lens ? p.lens[b] : p.S, s0 = blk * 4, n = min(4, len - s0);
+  const int blk = blockIdx.x * PREP_WARPS + (threadIdx.x >> 5), h = blockIdx.y, b = blockIdx.z, lane = threadIdx.x & 31;
+  const int len = p.lens ? p.lens[b] : p.S, s0 = blk * 4, n = min(4, len - s0), r8 = (g.rank + 7) / 8 * 8;
   if (n <= 0) return;
   const T* row[4];
-  const T* a1[4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {         // tokens past the end read the last one's rows and are made to change nothing
+  for (int i = 0; i < 4; ++i)           // tokens past the end read the last one's rows and are made to change nothing
     row[i] = static_cast<const T*>(g.proj) + ((long long)b * p.S + s0 + min(i, n - 1)) * g.ld;
-    a1[i] = row[i] + 2 * g.H * (g.D + g.V);
-  }
+  float* a1 = s_a1 + (threadIdx.x >> 5) * 4 * r8;
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    for (int r = lane; r < r8; r += 32) a1[i * r8 + r] = r < g.rank ? to_f(row[i][2 * g.H * (g.D + g.V) + r]) : 0.f;
+  __syncwarp();
   const long long hb = (long long)b * g.H + h;
   float* qo = p.q + (hb * p.Sp + s0) * p.Dp;
   float* ko = p.k + (hb * p.Sp + s0) * p.Dp;
-  const float scale = 1.f / sqrtf(float(g.D));
+  const float scale = 1.f / sqrtf(float(g.D)), inv_tau = 1.f / g.tau;
   float pr[16];
 #pragma unroll
   for (int i = 0; i < 16; ++i) pr[i] = 0.f;
-  for (int d = lane; d < p.Dp; d += 32) {
-    float q[4], k[4], a[4];
-    if (d < g.D) {
-      const long long c = (long long)h * g.D + d;
-      decay_logits<T, 4>(g, a1, c, p.vec, a);
+  for (int d0 = lane; d0 < p.Dp; d0 += 64) {          // two channels at a time: d0 and d0 + 32
+    float z[2][4];
+    float q[2][4], k[2][4];
+    const T* w[2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int d = d0 + 32 * x;
+      const bool on = d < g.D;
+      const long long c = (long long)h * g.D + (on ? d : 0);
+      w[x] = static_cast<const T*>(g.a2) + c * g.ld2;
+      const float bias = to_f(static_cast<const T*>(g.bias)[c]);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        q[i] = i < n ? to_f(row[i][c]) * scale : 0.f;
-        k[i] = i < n ? to_f(row[i][(long long)g.H * g.D + c]) : 0.f;
-        a[i] = i < n ? channel_decay(a[i], g.tau) : 1.f;
+        z[x][i] = bias;
+        q[x][i] = on && i < n ? to_f(row[i][c]) * scale : 0.f;
+        k[x][i] = on && i < n ? to_f(row[i][(long long)g.H * g.D + c]) : 0.f;
       }
-    } else {
-#pragma unroll
-      for (int i = 0; i < 4; ++i) q[i] = k[i] = 0.f, a[i] = 1.f;
     }
-    float G = 1.f, t[4];                // t[j] = R_ij k_j for the current i
+    for (int r = 0; r < r8; r += 8) {
+      float f[2][8];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      G *= a[i];
+      for (int x = 0; x < 2; ++x) {
+        if (p.vec) load_n<8>(w[x] + r, f[x]);
+        else {
 #pragma unroll
-      for (int j = 0; j < i; ++j) t[j] *= a[i];
-      t[i] = k[i];
+          for (int e = 0; e < 8; ++e) f[x][e] = r + e < g.rank ? to_f(w[x][r + e]) : 0.f;
+        }
+      }
 #pragma unroll
-      for (int j = 0; j <= i; ++j) pr[i * (i + 1) / 2 + j] = fmaf(q[i], t[j], pr[i * (i + 1) / 2 + j]);
-      qo[i * p.Dp + d] = G * q[i];
+      for (int i = 0; i < 4; ++i) {
+        float y[8];
+        load_n<8>(a1 + i * r8 + r, y);
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) z[x][i] = fmaf(f[x][e], y[e], z[x][i]);
+      }
     }
 #pragma unroll
-    for (int j = 0; j < 4; ++j) ko[j * p.Dp + d] = t[j];
-    p.decay[(hb * (p.Sp / 4) + blk) * p.Dp + d] = G;
+    for (int x = 0; x < 2; ++x) {
+      const int d = d0 + 32 * x;
+      if (d >= p.Dp) break;
+      float G = 1.f, t[4];              // t[j] = R_ij k_j for the current i
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float a = i < n && d < g.D ? channel_decay(z[x][i], inv_tau) : 1.f;
+        G *= a;
+#pragma unroll
+        for (int j = 0; j < i; ++j) t[j] *= a;
+        t[i] = k[x][i];
+#pragma unroll
+        for (int j = 0; j <= i; ++j) pr[i * (i + 1) / 2 + j] = fmaf(q[x][i], t[j], pr[i * (i + 1) / 2 + j]);
+        qo[i * p.Dp + d] = G * q[x][i];
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ko[j * p.Dp + d] = t[j];
+      p.decay[(hb * (p.Sp / 4) + blk) * p.Dp + d] = G;
+    }
   }
 #pragma unroll
   for (int i = 0; i < 16; ++i) pr[i] += __shfl_xor_sync(0xffffffffu, pr[i], 16);
@@ -388,7 +406,7 @@ struct GlaStepArgs {
 // 256 threads = 8 warps; warp w holds rows w, w + 8, ... (NR of them) of the state, lane l the columns 4 l .. 4 l + 3 of each 128-column
 // part.  D <= 8 NR, V <= 128 CV, V % 4 == 0.
 template <class T, int NR, int CV>
-__global__ void __launch_bounds__(256) gla_step_kernel(const GlaStepArgs p) {
+__global__ void __launch_bounds__(256, NR * CV <= 16 ? 2 : 1) gla_step_kernel(const GlaStepArgs p) {
   tfb::pdl_sync();
   constexpr int VM = 128 * CV;
   __shared__ float sk[8 * NR], sq[8 * NR], sa[8 * NR], sv[VM], so[8][VM], red[32];
@@ -407,18 +425,31 @@ __global__ void __launch_bounds__(256) gla_step_kernel(const GlaStepArgs p) {
       s[i][c] = (S0 && d < D && j < V) ? *reinterpret_cast<const float4*>(S0 + (long long)d * V + j) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
   const T* row = static_cast<const T*>(g.proj) + (long long)b * g.ld;
-  const T* const a1[1] = {row + 2 * g.H * (D + V)};
+  const T* a1 = row + 2 * g.H * (D + V);
   for (int d = tid; d < 8 * NR; d += 256) {
-    float q = 0.f, k = 0.f, z[1] = {0.f};
+    float q = 0.f, k = 0.f, a = 1.f;
     if (d < D) {
       const long long c = (long long)h * D + d;
-      decay_logits<T, 1>(g, a1, c, p.vec, z);
+      const T* w2 = static_cast<const T*>(g.a2) + c * g.ld2;
+      float z = to_f(static_cast<const T*>(g.bias)[c]);
+      if (p.vec) {
+        for (int r = 0; r < g.rank; r += 8) {
+          float x[8], y[8];
+          load_n<8>(w2 + r, x);
+          load_n<8>(a1 + r, y);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) z = fmaf(x[e], y[e], z);
+        }
+      } else {
+        for (int r = 0; r < g.rank; ++r) z = fmaf(to_f(w2[r]), to_f(a1[r]), z);
+      }
+      a = channel_decay(z, 1.f / g.tau);
       q = to_f(row[c]) / sqrtf(float(D));
       k = to_f(row[(long long)g.H * D + c]);
     }
     sq[d] = q;
     sk[d] = k;
-    sa[d] = d < D ? channel_decay(z[0], g.tau) : 1.f;
+    sa[d] = a;
   }
   const T* vrow = row + 2ll * g.H * D + (long long)h * V;
   for (int j = tid; j < VM; j += 256) sv[j] = j < V ? to_f(vrow[j]) : 0.f;
@@ -498,10 +529,12 @@ TFB_API int tfb_gla_prep(const void* proj, long long ld, const void* a2, long lo
   if (!Dp) return TFB_ERR_LIMIT;
   const GlaProj g{proj, ld, a2, ld2, bias, rank, tau, H, D, V};
   const GlaPrepArgs p{g, lens, q, k, v, decay, pair, S, (S + 3) / 4 * 4, Dp, (V + 3) / 4 * 4, vector_rows(g, f32)};
-  const dim3 grid((p.Sp / 4 + 3) / 4, H, B);
+  const dim3 grid((p.Sp / 4 + PREP_WARPS - 1) / PREP_WARPS, H, B);
+  const int smem = PREP_WARPS * 4 * ((rank + 7) / 8 * 8) * 4;
+  if (smem > 48 * 1024) return TFB_ERR_LIMIT;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) launch_k(gla_prep_kernel<float>, grid, 128, 0, st, p);
-  else launch_k(gla_prep_kernel<__nv_bfloat16>, grid, 128, 0, st, p);
+  if (f32) launch_k(gla_prep_kernel<float>, grid, PREP_WARPS * 32, smem, st, p);
+  else launch_k(gla_prep_kernel<__nv_bfloat16>, grid, PREP_WARPS * 32, smem, st, p);
   return int(cudaGetLastError());
 }
 

@@ -487,8 +487,8 @@ class FigudraConfig:
                     raise ValueError(f"layer {i}: {m.heads} heads do not divide over {m.kv_heads} kv heads")
                 if m.rot is not None and (m.rot.dims % 2 or not 0 < m.rot.dims <= m.dim):
                     raise ValueError(f"layer {i}: cannot rotate {m.rot.dims} of {m.dim} entries")
-            elif not 1 <= m.dim <= 512:
-                raise ValueError(f"layer {i}: key channels per head {m.dim} are not in 1 .. 512")
+            elif not 1 <= m.dim <= 512 or not 1 <= m.rank <= 768:
+                raise ValueError(f"layer {i}: key channels per head {m.dim} or rank {m.rank} are not in 1 .. 512, 1 .. 768")
             if x is not None:
                 if x.experts % x.groups or not 1 <= x.keep <= x.groups or not 1 <= x.top <= x.experts // x.groups * x.keep:
                     raise ValueError(f"layer {i}: cannot choose {x.top} of {x.experts} experts in {x.keep} of {x.groups} groups")
