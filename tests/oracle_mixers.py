@@ -468,3 +468,157 @@ class PlainFigudra:
         return plain_norm(x, w["final.norm"], eps) @ w["head"].T
 
     greedy = PlainLanedra.greedy
+
+
+# ---------------------------------------------------------------------------------------------------- chunked attention
+def seen_in_chunk(i, j, size):
+    """Whether position i looks at position j: earlier or the same, in the same chunk of ``size`` positions."""
+    return (j <= i) & (i // size == j // size)
+
+
+def attend_chunk(q, k, v, pos0, scale, size, sink=None, temp=1.0):
+    """One head.  q [T, dim] at positions pos0 ..., k [N, dim] and v [N, vdim] at 0 ...; ``sink``: a number whose exponential joins the
+    denominator; ``temp``: a factor of the scores."""
+    at = torch.arange(pos0, pos0 + q.shape[0])
+    ok = seen_in_chunk(at[:, None], torch.arange(k.shape[0])[None], size)
+    s = torch.where(ok, q @ k.T * scale * temp, -math.inf)
+    m = s.max(-1, keepdim=True).values
+    if sink is not None:
+        m = m.clamp(min=float(sink))
+    e = torch.exp(s - m)
+    return (e @ v) / (e.sum(-1, keepdim=True) + (torch.exp(sink - m) if sink is not None else 0.0))
+
+
+# ---------------------------------------------------------------------------------------------------- recurrences over a matrix state
+def forget_gate(z, lower):
+    """Between ``lower`` and one."""
+    return lower + (1 - lower) * sigmoid(z)
+
+
+def hgrn2_scan(q, f, v, state=None):
+    """One head: what is not kept is written, with no key of its own.  q, f [T, dim], v [T, vdim]."""
+    S = torch.zeros(q.shape[1], v.shape[1], dtype=q.dtype) if state is None else state.clone()
+    out = []
+    for t in range(q.shape[0]):
+        S = torch.diag(f[t]) @ S + torch.outer(1 - f[t], v[t])
+        out.append(S.T @ q[t])
+    return torch.stack(out), S
+
+
+def retention_scan(q, k, v, decay, state=None):
+    """One head with one decay.  q, k [T, dim] (rotated, k scaled), v [T, vdim]."""
+    S = torch.zeros(q.shape[1], v.shape[1], dtype=q.dtype) if state is None else state.clone()
+    out = []
+    for t in range(q.shape[0]):
+        S = decay * S + torch.outer(k[t], v[t])
+        out.append(S.T @ q[t])
+    return torch.stack(out), S
+
+
+# ---------------------------------------------------------------------------------------------------- grouped norm, streams
+def group_norm(x, w, groups, eps):
+    """RMS norm of every one of ``groups`` equal consecutive parts; one weight for the whole."""
+    return torch.cat([rms(p, eps) for p in x.chunk(groups, -1)], -1) * w
+
+
+def streams_in(xs, coef):
+    """What a sublayer reads of the streams xs (a list)."""
+    return sum(float(c) * x for c, x in zip(coef, xs))
+
+
+def streams_out(xs, y, mix, out):
+    """The streams behind a sublayer that returned y; mix [from, to]."""
+    return [sum(float(mix[s, t]) * xs[s] for s in range(len(xs))) + float(out[t]) * y for t in range(len(xs))]
+
+
+# ---------------------------------------------------------------------------------------------------- clamped experts
+def clamped_glu(h, gate, up, down, limit):
+    g = torch.clamp(h @ gate.T, max=limit)
+    u = torch.clamp(h @ up.T, -limit, limit)
+    return (g * sigmoid(1.702 * g) * (u + 1)) @ down.T
+
+
+def route_all(z, top):
+    """One token's router logits -> [(expert, weight)]: the softmax over all experts, of which the ``top`` largest keep their values."""
+    m = max(float(x) for x in z)
+    e = [math.exp(float(x) - m) for x in z]
+    order = sorted(range(len(e)), key=lambda i: (-e[i], i))[:top]
+    return [(i, e[i] / sum(e)) for i in order]
+
+
+def clamped_mixture(h, router, top, experts, limit, shared=None, shared_limit=None):
+    out = torch.zeros_like(h)
+    for t in range(h.shape[0]):
+        for i, w in route_all(router @ h[t], top):
+            out[t] += w * clamped_glu(h[t], *experts[i], limit)
+    return out if shared is None else out + clamped_glu(h, *shared, shared_limit)
+
+
+class PlainToderax:
+    """As PlainLanedra, for hyper-connected layers of HGRN2 or of chunked attention and retention side by side."""
+
+    def __init__(self, cfg, tensors):
+        self.cfg = cfg
+        self.w = {n: t.to(DT) for n, t in tensors.items()}
+
+    def start(self):
+        return {"pos": 0, "layers": [{} for _ in self.cfg["layers"]]}
+
+    def hgrn2(self, m, p, h, mine, pos, eps):
+        w, H, D, V, T = self.w, m["heads"], m["dim"], m["vdim"], h.shape[0]
+        q, v = silu(h @ w[p + "q"].T).view(T, H, D), (h @ w[p + "v"].T).view(T, H, V)
+        f = forget_gate(h @ w[p + "f"].T + w[p + "f.b"], w[p + "lower"]).view(T, H, D)
+        both = [hgrn2_scan(q[:, x], f[:, x], v[:, x], mine["S"][x] if "S" in mine else None) for x in range(H)]
+        mine["S"] = [s for _, s in both]
+        return plain_norm(torch.stack([o for o, _ in both], 1), w[p + "norm"], eps).reshape(T, H * V) @ w[p + "o"].T
+
+    def chunked(self, m, p, h, mine, pos, eps):
+        w, H, G, D, V, T = self.w, m["heads"], m["kv_heads"], m["dim"], m["vdim"], h.shape[0]
+        q, k, v = ((h @ w[p + n].T + w[p + n + ".b"]).view(T, c, -1) for n, c in (("q", H), ("k", G), ("v", G)))
+        q, k = rms(q, eps), rms(k, eps)
+        mine["k"] = torch.cat([mine["k"], k]) if "k" in mine else k
+        mine["v"] = torch.cat([mine["v"], v]) if "v" in mine else v
+        o = torch.stack([attend_chunk(q[:, x], mine["k"][:, x // (H // G)], mine["v"][:, x // (H // G)], pos, m["scale"], m["mask"]["size"],
+                                      w[p + "sink"][x], w[p + "temp"][x]) for x in range(H)], 1)
+        return o.reshape(T, H * V) @ w[p + "o"].T
+
+    def retention(self, m, p, h, mine, pos, eps):
+        w, H, D, V, T = self.w, m["heads"], m["dim"], m["vdim"], h.shape[0]
+        turn = lambda x: rotate_linear(x.view(T, H, D), pos, m["rot"]["dims"], m["rot"]["base"])
+        q, k, v = turn(h @ w[p + "q"].T), turn(h @ w[p + "k"].T) * D ** -0.5, (h @ w[p + "v"].T).view(T, H, V)
+        both = [retention_scan(q[:, x], k[:, x], v[:, x], m["decay"][x], mine["S"][x] if "S" in mine else None) for x in range(H)]
+        mine["S"] = [s for _, s in both]
+        o = rms(torch.stack([o for o, _ in both], 1), eps).reshape(T, H * V)
+        return (o * silu(h @ w[p + "g"].T)) @ w[p + "o"].T
+
+    def mixer(self, l, p, h, mine, pos, eps):
+        if l["type"] == "hgrn2":
+            return self.hgrn2(l["mixer"], p, h, mine, pos, eps)
+        a = self.chunked(l["mixer"]["left"], p + "left.", h, mine.setdefault("left", {}), pos, eps)
+        b = self.retention(l["mixer"]["right"], p + "right.", h, mine.setdefault("right", {}), pos, eps)
+        return (plain_norm(a, self.w[p + "left.out"], eps) + plain_norm(b, self.w[p + "right.out"], eps)) / 2
+
+    def ff(self, m, p, h):
+        three = lambda q: tuple(self.w[p + q + n] for n in (".gate", ".up", ".down"))
+        r, s = m["router"], m.get("shared")
+        return clamped_mixture(h, self.w[p + "router"], r["top"], [three(f"e{e}") for e in range(r["experts"])], m["expert"]["limit"],
+                               three("shared") if s else None, s["limit"] if s else None)
+
+    def run(self, tokens, st=None, residuals=None):
+        c, w = self.cfg, self.w
+        eps, groups = c["norm"]["eps"], c["norm"]["groups"]
+        st = st if st is not None else self.start()
+        xs = [w["embed"][torch.tensor(tokens)] * c["embedding"]["scale"]] * c["streams"]
+        for i, l in enumerate(c["layers"]):
+            p = f"l{i}."
+            for n, sub in ((1, lambda h: self.mixer(l, p + "mix.", h, st["layers"][i], st["pos"], eps)), (2, lambda h: self.ff(l["mlp"], p + "mlp.", h))):
+                if n == 2 and l["mlp"] is None:
+                    continue
+                y = sub(group_norm(streams_in(xs, w[f"{p}hc{n}.in"]), w[f"{p}norm{n}"], groups, eps))
+                xs = streams_out(xs, y, w[f"{p}hc{n}.mix"], w[f"{p}hc{n}.out"])
+            if residuals is not None:
+                residuals.append(sum(xs))
+        st["pos"] += len(tokens)
+        return group_norm(sum(xs), w["final.norm"], groups, eps) @ w["head"].T
+
+    greedy = PlainLanedra.greedy

@@ -30,7 +30,7 @@ NVCC_FLAGS = [
 ]
 # Translation units whose fp32 arithmetic has to be fp32 to the last bits (they serve the 32-bit mode of a model as well):
 # compiled without --use_fast_math.
-PRECISE = {"stack_ops", "delta_rule", "diff_attention", "head_attention", "latent_attention", "gated_linear", "moe_serve", "skinny_linear"}
+PRECISE = {"stack_ops", "streams", "delta_rule", "diff_attention", "head_attention", "latent_attention", "gated_linear", "moe_serve", "skinny_linear"}
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-fvisibility=hidden", "-pthread", "-Wall", "-Wno-unused-function"]
 
 

@@ -524,51 +524,6 @@ static int launch_scan(const DeltaScanArgs& p, int B, cudaStream_t st) {
 }
 
 // ------------------------------------------------------------------------------------------------
-// gated norm of the head outputs:  o / rms(o) * w * silu(gate)
-// ------------------------------------------------------------------------------------------------
-template <class T, int VEC>
-__global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ldg,
-                                                         const T* __restrict__ w, T* __restrict__ out, long long ldo, int rows, int H, int V,
-                                                         float eps) {
-  tfb::pdl_sync();
-  const int lane = threadIdx.x & 31;
-  const long long nwarps = (long long)gridDim.x * (blockDim.x >> 5), n = (long long)rows * H;
-  for (long long i = blockIdx.x * (long long)(blockDim.x >> 5) + (threadIdx.x >> 5); i < n; i += nwarps) {
-    const long long r = i / H;
-    const int h = int(i % H);
-    const float* src = o + i * V;
-    const T* gt = gate + r * ldg + h * V;
-    T* dst = out + r * ldo + h * V;
-    float x0[VEC], g0[VEC], x[VEC], g[VEC], wv[VEC];
-    float ss = 0.f;
-    for (int j = lane * VEC; j < V; j += 32 * VEC) {
-      load_n<VEC>(src + j, x);
-      if (j == lane * VEC) {
-        load_n<VEC>(gt + j, g0);
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) x0[e] = x[e];
-      }
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) ss = fmaf(x[e], x[e], ss);
-    }
-    const float rs = 1.f / sqrtf(warp_add(ss) / V + eps);
-    for (int j = lane * VEC; j < V; j += 32 * VEC) {
-      load_n<VEC>(w + j, wv);
-      if (j == lane * VEC) {
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) { x[e] = x0[e]; g[e] = g0[e]; }
-      } else {
-        load_n<VEC>(src + j, x);
-        load_n<VEC>(gt + j, g);
-      }
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) x[e] = x[e] * rs * wv[e] * silu_exact(g[e]);
-      store_n<VEC>(dst + j, x);
-    }
-  }
-}
-
-// ------------------------------------------------------------------------------------------------
 // one token per sequence
 // ------------------------------------------------------------------------------------------------
 struct DeltaStepArgs {
@@ -746,24 +701,6 @@ TFB_API int tfb_delta_scan(const float* q, const float* k, const float* v, const
     case 512: return launch_scan<16, 32>(p, B, st);
     default: return TFB_ERR_LIMIT;
   }
-}
-
-TFB_API int tfb_gated_norm(const float* o, const void* gate, long long ldg, const void* w, void* out, long long ldo, int rows, int H, int V,
-                           float eps, int f32, void* stream) {
-  using namespace tfb;
-  if (rows <= 0 || H <= 0 || V <= 0) return TFB_ERR_ARG;
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const long long blocks = ((long long)rows * H + 7) / 8;
-  const int grid = int(blocks < 148ll * 32 ? blocks : 148ll * 32);
-  auto al = [](const void* x, int n) { return (reinterpret_cast<uintptr_t>(x) & (n - 1)) == 0; };
-  const int es = f32 ? 4 : 2;
-  const bool v4 = V % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && al(o, 16) && al(gate, 4 * es) && al(w, 4 * es) && al(out, 4 * es);
-#define TFB_GN(T, VEC) launch_k(gated_norm_kernel<T, VEC>, grid, 256, 0, st, o, static_cast<const T*>(gate), ldg, static_cast<const T*>(w), \
-                                static_cast<T*>(out), ldo, rows, H, V, eps)
-  if (f32) { if (v4) TFB_GN(float, 4); else TFB_GN(float, 1); }
-  else { if (v4) TFB_GN(bf16, 4); else TFB_GN(bf16, 1); }
-#undef TFB_GN
-  return int(cudaGetLastError());
 }
 
 // One token for each of B sequences (prepared with Sp = 1), gated norm included.  Returns TFB_ERR_LIMIT for head sizes it

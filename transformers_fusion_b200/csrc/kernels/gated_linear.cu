@@ -1,10 +1,15 @@
-// Gated linear attention (a matrix state per head whose rows decay by key channel) for prompts and for decoding.
+// Linear attention with a matrix state per head whose rows decay, for prompts and for decoding.
 //
-//   a = sigmoid(z)^(1/tau);   S <- diag(a) S + k v^T;   o = S^T q            per head, S is [D, V] in fp32
+//   S <- diag(a) S + k v^T;   o = S^T q            per head, S is [D, V] in fp32
+//
+// Three sources of q, k and the decays a (entries of the key channels):
+//   GATED       a = sigmoid(z)^(1/tau), z out of a low-rank projection; q is scaled by D^(-1/2)
+//   FORGET      a = l + (1 - l) sigmoid(f + b) with a lower bound l per channel, k = 1 - a, q through silu
+//   RETENTION   a fixed number per head; q and k rotated by their position, k scaled by D^(-1/2)
 //
 // Kernels:
-//   gla_prep    one warp per (four tokens, head): the decays out of their low-rank projection, and what the scan needs of four
-//               tokens.  With G_i and R_ij the products of the decays up to token i and between tokens j and i (per channel),
+//   gla_prep    one warp per (four tokens, head): q, k and the decays, and what the scan needs of four tokens.  With G_i and R_ij the
+//               products of the decays up to token i and between tokens j and i (per channel),
 //                   q'_i = G_i q_i,   k'_j = R_3j k_j,   G_3,   P_ij = sum over the channels of q_i R_ij k_j   (j <= i)
 //               Every factor is a product of decays, at most one: nothing is divided, and a channel that forgets at once is
 //               no special case.
@@ -13,23 +18,30 @@
 //               registers as packed fp32 pairs).  The sums over D are needed for the output alone: no reduction is on the
 //               path from one state to the next.  The rows of the next tokens travel to shared memory (bulk copies) while the
 //               current ones are used; fp32 FMA throughout.
-//   gla_step    one token per sequence: one block per (sequence, head) computes the decays, streams the state through registers once
-//               (read, updated, written back), and applies the gated norm to the output.
+//   gla_step    one token per sequence: one block per (sequence, head) computes q, k and the decays, streams the state through registers
+//               once (read, updated, written back), and applies the norm (with weight and gate, where there are some) to the output.
 #include "tfb_elem.cuh"
 #include "tfb_host.h"
 
 namespace tfb {
 TFB_BOUNDS_DEFINE(gated_linear)
 
+enum GlaKind { GATED = 0, FORGET = 1, RETENTION = 2 };
+
 struct GlaProj {
-  const void* proj;       // [B*S, ld]: q (H D) | k (H D) | v (H V) | gate (H V) | a1 (rank)
+  const void* proj;       // [B*S, ld]: q (H D) | k, or the logits f (H D) | v (H V) | gate (H V), where there is one | a1 (rank), GATED
   long long ld;
-  const void* a2;         // [H D, ld2]
+  int H, D, V, gated;
+  const void* bias;       // [H D], GATED and FORGET
+  const void* a2;         // GATED: [H D, ld2]
   long long ld2;
-  const void* bias;       // [H D]
   int rank;
   float tau;
-  int H, D, V;
+  const void* lower;      // FORGET: [H D]
+  const float* decay;     // RETENTION: [H]
+  const float *cos_t, *sin_t;   // [max_pos, dims / 2]
+  const int* positions;   // [B*S]
+  int max_pos, dims;      // the first `dims` entries of a head are rotated, entry i with entry i + dims / 2
 };
 
 // sigmoid(z)^(1 / tau) = exp((min(z, 0) - ln(1 + x)) / tau), x = exp(-|z|).  ln(1 + x) = 2 atanh(u) with u = x / (2 + x) <= 1 / 3, by the
@@ -49,6 +61,41 @@ __device__ __forceinline__ float channel_decay(float z, float inv_tau) {
   return expf((fminf(z, 0.f) - 2.f * u * p) * inv_tau);
 }
 
+// entry d of head h, in a row with position pos, that starts at x: rotated
+template <class T>
+__device__ __forceinline__ float rotated(const GlaProj& g, const T* x, int d, int pos) {
+  const float u = to_f(x[d]);
+  if (d >= g.dims) return u;
+  const int half = g.dims >> 1, i = d < half ? d : d - half;
+  const float c = g.cos_t[(long long)pos * half + i], s = g.sin_t[(long long)pos * half + i];
+  return d < half ? u * c - to_f(x[d + half]) * s : u * c + to_f(x[d - half]) * s;
+}
+
+__device__ __forceinline__ int checked_position(const GlaProj& g, long long row) {
+  if (g.dims == 0) return 0;
+  int pos = g.positions[row];
+  TFB_BOUNDS(pos >= 0 && pos < g.max_pos, 61, pos, g.max_pos);
+  return pos < 0 ? 0 : (pos >= g.max_pos ? g.max_pos - 1 : pos);
+}
+
+// q, k and the decay of channel d < D of head h, for FORGET and RETENTION
+template <class T, int KIND>
+__device__ __forceinline__ void channel_of(const GlaProj& g, const T* row, int h, int d, int pos, float scale, float& q, float& k, float& a) {
+  const long long c = (long long)h * g.D + d, n = (long long)g.H * g.D;
+  if constexpr (KIND == FORGET) {
+    const float z = to_f(row[n + c]) + to_f(static_cast<const T*>(g.bias)[c]), l = to_f(static_cast<const T*>(g.lower)[c]);
+    const float e = expf(-fabsf(z)), big = 1.f / (1.f + e), small = e * big;      // sigmoid(|z|), sigmoid(-|z|)
+    q = silu_exact(to_f(row[c]));
+    k = (1.f - l) * (z < 0.f ? big : small);
+    a = fmaf(1.f - l, z < 0.f ? small : big, l);
+  } else {
+    const T* x = row + (long long)h * g.D;
+    q = rotated<T>(g, x, d, pos);
+    k = rotated<T>(g, x + n, d, pos) * scale;
+    a = g.decay[h];
+  }
+}
+
 // ------------------------------------------------------------------------------------------------
 // preparation
 // ------------------------------------------------------------------------------------------------
@@ -62,18 +109,21 @@ struct GlaPrepArgs {
 
 constexpr int PREP_WARPS = 4;
 
-template <class T>
+template <class T, int KIND>
 __global__ void __launch_bounds__(PREP_WARPS * 32) gla_prep_kernel(const GlaPrepArgs p) {
   tfb::pdl_sync();
   extern __shared__ __align__(16) float s_a1[];       // [warp][4][rank rounded up to 8] rows of a1, zeros past the rank
   const GlaProj& g = p.g;
   const int blk = blockIdx.x * PREP_WARPS + (threadIdx.x >> 5), h = blockIdx.y, b = blockIdx.z, lane = threadIdx.x & 31;
-  const int len = p.lens ? p.lens[b] : p.S, s0 = blk * 4, n = min(4, len - s0), r8 = (g.rank + 7) / 8 * 8;
+  const int len = p.lens ? p.lens[b] : p.S, s0 = blk * 4, n = min(4, len - s0), r8 = KIND == GATED ? (g.rank + 7) / 8 * 8 : 0;
   if (n <= 0) return;
+  int pos[4];
   const T* row[4];
 #pragma unroll
   for (int i = 0; i < 4; ++i)           // tokens past the end read the last one's rows and are made to change nothing
     row[i] = static_cast<const T*>(g.proj) + ((long long)b * p.S + s0 + min(i, n - 1)) * g.ld;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) pos[i] = KIND == RETENTION ? checked_position(g, (long long)b * p.S + s0 + min(i, n - 1)) : 0;
   float* a1 = s_a1 + (threadIdx.x >> 5) * 4 * r8;
 #pragma unroll
   for (int i = 0; i < 4; ++i)
@@ -82,46 +132,58 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) gla_prep_kernel(const GlaPrep
   const long long hb = (long long)b * g.H + h;
   float* qo = p.q + (hb * p.Sp + s0) * p.Dp;
   float* ko = p.k + (hb * p.Sp + s0) * p.Dp;
-  const float scale = 1.f / sqrtf(float(g.D)), inv_tau = 1.f / g.tau;
+  const float scale = 1.f / sqrtf(float(g.D)), inv_tau = KIND == GATED ? 1.f / g.tau : 0.f;
   float pr[16];
 #pragma unroll
   for (int i = 0; i < 16; ++i) pr[i] = 0.f;
   for (int d0 = lane; d0 < p.Dp; d0 += 64) {          // two channels at a time: d0 and d0 + 32
-    float z[2][4];
+    float z[2][4];                                    // logits of the decays (GATED), or the decays
     float q[2][4], k[2][4];
     const T* w[2];
-#pragma unroll
-    for (int x = 0; x < 2; ++x) {
-      const int d = d0 + 32 * x;
-      const bool on = d < g.D;
-      const long long c = (long long)h * g.D + (on ? d : 0);
-      w[x] = static_cast<const T*>(g.a2) + c * g.ld2;
-      const float bias = to_f(static_cast<const T*>(g.bias)[c]);
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        z[x][i] = bias;
-        q[x][i] = on && i < n ? to_f(row[i][c]) * scale : 0.f;
-        k[x][i] = on && i < n ? to_f(row[i][(long long)g.H * g.D + c]) : 0.f;
-      }
-    }
-    for (int r = 0; r < r8; r += 8) {
-      float f[2][8];
+    if constexpr (KIND != GATED) {
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
-        if (p.vec) load_n<8>(w[x] + r, f[x]);
-        else {
+        const int d = d0 + 32 * x;
 #pragma unroll
-          for (int e = 0; e < 8; ++e) f[x][e] = r + e < g.rank ? to_f(w[x][r + e]) : 0.f;
+        for (int i = 0; i < 4; ++i) {
+          channel_of<T, KIND>(g, row[i], h, d < g.D ? d : 0, pos[i], scale, q[x][i], k[x][i], z[x][i]);
+          if (d >= g.D || i >= n) q[x][i] = k[x][i] = 0.f;
         }
       }
+    } else {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        float y[8];
-        load_n<8>(a1 + i * r8 + r, y);
+      for (int x = 0; x < 2; ++x) {
+        const int d = d0 + 32 * x;
+        const bool on = d < g.D;
+        const long long c = (long long)h * g.D + (on ? d : 0);
+        w[x] = static_cast<const T*>(g.a2) + c * g.ld2;
+        const float bias = to_f(static_cast<const T*>(g.bias)[c]);
 #pragma unroll
-        for (int x = 0; x < 2; ++x)
+        for (int i = 0; i < 4; ++i) {
+          z[x][i] = bias;
+          q[x][i] = on && i < n ? to_f(row[i][c]) * scale : 0.f;
+          k[x][i] = on && i < n ? to_f(row[i][(long long)g.H * g.D + c]) : 0.f;
+        }
+      }
+      for (int r = 0; r < r8; r += 8) {
+        float f[2][8];
 #pragma unroll
-          for (int e = 0; e < 8; ++e) z[x][i] = fmaf(f[x][e], y[e], z[x][i]);
+        for (int x = 0; x < 2; ++x) {
+          if (p.vec) load_n<8>(w[x] + r, f[x]);
+          else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[x][e] = r + e < g.rank ? to_f(w[x][r + e]) : 0.f;
+          }
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          float y[8];
+          load_n<8>(a1 + i * r8 + r, y);
+#pragma unroll
+          for (int x = 0; x < 2; ++x)
+#pragma unroll
+            for (int e = 0; e < 8; ++e) z[x][i] = fmaf(f[x][e], y[e], z[x][i]);
+        }
       }
     }
 #pragma unroll
@@ -131,7 +193,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) gla_prep_kernel(const GlaPrep
       float G = 1.f, t[4];              // t[j] = R_ij k_j for the current i
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float a = i < n && d < g.D ? channel_decay(z[x][i], inv_tau) : 1.f;
+        const float a = i < n && d < g.D ? (KIND == GATED ? channel_decay(z[x][i], inv_tau) : z[x][i]) : 1.f;
         G *= a;
 #pragma unroll
         for (int j = 0; j < i; ++j) t[j] *= a;
@@ -397,7 +459,7 @@ struct GlaStepArgs {
   float* state;
   const int* state_slots;
   int nslots, vec;
-  const void* w;          // [V] weight of the norm
+  const void* w;          // [V] weight of the norm, or null
   void* out;
   long long ldo;
   float eps;
@@ -405,7 +467,7 @@ struct GlaStepArgs {
 
 // 256 threads = 8 warps; warp w holds rows w, w + 8, ... (NR of them) of the state, lane l the columns 4 l .. 4 l + 3 of each 128-column
 // part.  D <= 8 NR, V <= 128 CV, V % 4 == 0.
-template <class T, int NR, int CV>
+template <class T, int KIND, int NR, int CV>
 __global__ void __launch_bounds__(256, NR * CV <= 16 ? 2 : 1) gla_step_kernel(const GlaStepArgs p) {
   tfb::pdl_sync();
   constexpr int VM = 128 * CV;
@@ -426,9 +488,11 @@ __global__ void __launch_bounds__(256, NR * CV <= 16 ? 2 : 1) gla_step_kernel(co
     }
   const T* row = static_cast<const T*>(g.proj) + (long long)b * g.ld;
   const T* a1 = row + 2 * g.H * (D + V);
+  const int pos = KIND == RETENTION ? checked_position(g, b) : 0;
   for (int d = tid; d < 8 * NR; d += 256) {
     float q = 0.f, k = 0.f, a = 1.f;
-    if (d < D) {
+    if (KIND != GATED && d < D) channel_of<T, KIND>(g, row, h, d, pos, 1.f / sqrtf(float(D)), q, k, a);
+    if (KIND == GATED && d < D) {
       const long long c = (long long)h * D + d;
       const T* w2 = static_cast<const T*>(g.a2) + c * g.ld2;
       float z = to_f(static_cast<const T*>(g.bias)[c]);
@@ -483,15 +547,17 @@ __global__ void __launch_bounds__(256, NR * CV <= 16 ? 2 : 1) gla_step_kernel(co
   }
   const float rs = 1.f / sqrtf(block_add(ov * ov, red) / V + p.eps);
   if (tid < V) {
-    const float gt = to_f(vrow[(long long)g.H * V + tid]);
-    static_cast<T*>(p.out)[(long long)b * p.ldo + h * V + tid] = from_f<T>(ov * rs * to_f(static_cast<const T*>(p.w)[tid]) * silu_exact(gt));
+    float y = ov * rs;
+    if (p.w) y *= to_f(static_cast<const T*>(p.w)[tid]);
+    if (g.gated) y *= silu_exact(to_f(vrow[(long long)g.H * V + tid]));
+    static_cast<T*>(p.out)[(long long)b * p.ldo + h * V + tid] = from_f<T>(y);
   }
 }
 
-template <class T>
+template <class T, int KIND>
 static int launch_step(const GlaStepArgs& p, int B, cudaStream_t st) {
   const dim3 grid(p.g.H, B);
-#define TFB_STEP(NR, CV) launch_k(gla_step_kernel<T, NR, CV>, grid, 256, 0, st, p)
+#define TFB_STEP(NR, CV) launch_k(gla_step_kernel<T, KIND, NR, CV>, grid, 256, 0, st, p)
   if (p.g.V <= 128) {
     if (p.g.D <= 32) TFB_STEP(4, 1);
     else if (p.g.D <= 64) TFB_STEP(8, 1);
@@ -518,24 +584,89 @@ static int vector_rows(const GlaProj& g, int f32) {
   return g.rank % 8 == 0 && g.ld % m == 0 && g.ld2 % m == 0 && al(a1) && al(g.a2);
 }
 
+// Launches of a source of q, k and decays (g, kind) with elements fp32 or bf16
+static int run_prep(const GlaProj& g, int kind, const int* lens, float* q, float* k, float* v, float* decay, float* pair, int B, int S, int Dp, int f32,
+                    void* stream) {
+  if (B <= 0 || B > 65535 || S <= 0 || g.H <= 0 || g.H > 65535 || g.D <= 0 || g.V <= 0 || Dp != padded_dim(g.D)) return TFB_ERR_ARG;
+  if (!Dp) return TFB_ERR_LIMIT;
+  const GlaPrepArgs p{g, lens, q, k, v, decay, pair, S, (S + 3) / 4 * 4, Dp, (g.V + 3) / 4 * 4, kind == GATED && vector_rows(g, f32)};
+  const dim3 grid((p.Sp / 4 + PREP_WARPS - 1) / PREP_WARPS, g.H, B);
+  const int smem = kind == GATED ? PREP_WARPS * 4 * ((g.rank + 7) / 8 * 8) * 4 : 0;
+  if (smem > 48 * 1024) return TFB_ERR_LIMIT;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+#define TFB_PREP(KIND)                                                                             \
+  if (f32) launch_k(gla_prep_kernel<float, KIND>, grid, PREP_WARPS * 32, smem, st, p);             \
+  else launch_k(gla_prep_kernel<__nv_bfloat16, KIND>, grid, PREP_WARPS * 32, smem, st, p);         \
+  break
+  switch (kind) {
+    case GATED: TFB_PREP(GATED);
+    case FORGET: TFB_PREP(FORGET);
+    default: TFB_PREP(RETENTION);
+  }
+#undef TFB_PREP
+  return int(cudaGetLastError());
+}
+
+// TFB_ERR_LIMIT for head sizes that the kernel does not hold in registers (the caller then takes the preparation, the scan and the norm)
+static int run_step(const GlaProj& g, int kind, float* state, const int* state_slots, int nslots, const void* w, void* out, long long ldo, int B, float eps,
+                    int f32, void* stream) {
+  if (B <= 0 || B > 65535 || g.H <= 0 || g.D <= 0 || g.V <= 0 || !state_slots) return TFB_ERR_ARG;
+  if ((g.V & 3) || g.V > 256 || g.D > 256 || (g.V > 128 && g.D > 128)) return TFB_ERR_LIMIT;
+  const GlaStepArgs p{g, state, state_slots, nslots, kind == GATED && vector_rows(g, f32), w, out, ldo, eps};
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  switch (kind) {
+    case GATED: return f32 ? launch_step<float, GATED>(p, B, st) : launch_step<__nv_bfloat16, GATED>(p, B, st);
+    case FORGET: return f32 ? launch_step<float, FORGET>(p, B, st) : launch_step<__nv_bfloat16, FORGET>(p, B, st);
+    default: return f32 ? launch_step<float, RETENTION>(p, B, st) : launch_step<__nv_bfloat16, RETENTION>(p, B, st);
+  }
+}
+
+static GlaProj gated_source(const void* proj, long long ld, const void* a2, long long ld2, const void* bias, int rank, float tau, int H, int D, int V) {
+  GlaProj g{proj, ld, H, D, V, 1};
+  g.bias = bias, g.a2 = a2, g.ld2 = ld2, g.rank = rank, g.tau = tau;
+  return g;
+}
+static GlaProj forget_source(const void* proj, long long ld, const void* bias, const void* lower, int gated, int H, int D, int V) {
+  GlaProj g{proj, ld, H, D, V, gated};
+  g.bias = bias, g.lower = lower;
+  return g;
+}
+static GlaProj retention_source(const void* proj, long long ld, const float* decay, const float* cos_t, const float* sin_t, int max_pos, int dims,
+                                const int* positions, int gated, int H, int D, int V) {
+  GlaProj g{proj, ld, H, D, V, gated};
+  g.decay = decay, g.cos_t = cos_t, g.sin_t = sin_t, g.max_pos = max_pos, g.dims = dims, g.positions = positions;
+  return g;
+}
+static bool bad_retention(const GlaProj& g) {
+  return !g.decay || g.dims < 0 || (g.dims & 1) || g.dims > g.D || (g.dims && (!g.cos_t || !g.sin_t || !g.positions || g.max_pos <= 0));
+}
+
 }  // namespace tfb
 
-// proj, a2, bias: see GlaProj (fp32 or bf16); outputs: see GlaPrepArgs, Sp = S rounded up to 4, Dp as tfb_delta_padded_dim.
+// Preparation of the rows of B sequences for tfb_gla_scan; sources: see GlaProj; outputs: see GlaPrepArgs (Sp = S rounded up to 4, Dp: D
+// rounded up to a power of two from 32 to 512).
 TFB_API int tfb_gla_prep(const void* proj, long long ld, const void* a2, long long ld2, const void* bias, int rank, float tau, const int* lens,
                          float* q, float* k, float* v, float* decay, float* pair, int B, int S, int H, int D, int Dp, int V, int f32,
                          void* stream) {
   using namespace tfb;
-  if (B <= 0 || B > 65535 || S <= 0 || H <= 0 || H > 65535 || D <= 0 || V <= 0 || rank <= 0 || !(tau > 0.f) || Dp != padded_dim(D)) return TFB_ERR_ARG;
-  if (!Dp) return TFB_ERR_LIMIT;
-  const GlaProj g{proj, ld, a2, ld2, bias, rank, tau, H, D, V};
-  const GlaPrepArgs p{g, lens, q, k, v, decay, pair, S, (S + 3) / 4 * 4, Dp, (V + 3) / 4 * 4, vector_rows(g, f32)};
-  const dim3 grid((p.Sp / 4 + PREP_WARPS - 1) / PREP_WARPS, H, B);
-  const int smem = PREP_WARPS * 4 * ((rank + 7) / 8 * 8) * 4;
-  if (smem > 48 * 1024) return TFB_ERR_LIMIT;
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) launch_k(gla_prep_kernel<float>, grid, PREP_WARPS * 32, smem, st, p);
-  else launch_k(gla_prep_kernel<__nv_bfloat16>, grid, PREP_WARPS * 32, smem, st, p);
-  return int(cudaGetLastError());
+  if (rank <= 0 || !(tau > 0.f)) return TFB_ERR_ARG;
+  return run_prep(gated_source(proj, ld, a2, ld2, bias, rank, tau, H, D, V), GATED, lens, q, k, v, decay, pair, B, S, Dp, f32, stream);
+}
+
+TFB_API int tfb_forget_prep(const void* proj, long long ld, const void* bias, const void* lower, const int* lens, float* q, float* k, float* v,
+                            float* decay, float* pair, int B, int S, int H, int D, int Dp, int V, int f32, void* stream) {
+  using namespace tfb;
+  if (!bias || !lower) return TFB_ERR_ARG;
+  return run_prep(forget_source(proj, ld, bias, lower, 0, H, D, V), FORGET, lens, q, k, v, decay, pair, B, S, Dp, f32, stream);
+}
+
+TFB_API int tfb_retention_prep(const void* proj, long long ld, const float* head_decay, const float* cos_t, const float* sin_t, int max_pos, int dims,
+                               const int* positions, const int* lens, float* q, float* k, float* v, float* decay, float* pair, int B, int S, int H, int D,
+                               int Dp, int V, int f32, void* stream) {
+  using namespace tfb;
+  const GlaProj g = retention_source(proj, ld, head_decay, cos_t, sin_t, max_pos, dims, positions, 0, H, D, V);
+  if (bad_retention(g)) return TFB_ERR_ARG;
+  return run_prep(g, RETENTION, lens, q, k, v, decay, pair, B, S, Dp, f32, stream);
 }
 
 // The recurrence over prepared rows; o [B*S, H, V] fp32.
@@ -555,16 +686,27 @@ TFB_API int tfb_gla_scan(const float* q, const float* k, const float* v, const f
   }
 }
 
-// One token for each of B sequences that go on, gated norm included.  Returns TFB_ERR_LIMIT for head sizes it does not hold in
-// registers (the caller then takes the preparation, the scan and the norm kernel).
+// One token for each of B sequences that go on, with the norm of the heads' outputs: o / rms(o) [* w] [* silu(gate)].  TFB_ERR_LIMIT: see run_step.
 TFB_API int tfb_gla_step(const void* proj, long long ld, const void* a2, long long ld2, const void* bias, int rank, float tau, float* state,
                          const int* state_slots, int nslots, const void* w, void* out, long long ldo, int B, int H, int D, int V, float eps, int f32,
                          void* stream) {
   using namespace tfb;
-  if (B <= 0 || B > 65535 || H <= 0 || D <= 0 || V <= 0 || rank <= 0 || !(tau > 0.f) || !state_slots) return TFB_ERR_ARG;
-  if ((V & 3) || V > 256 || D > 256 || (V > 128 && D > 128)) return TFB_ERR_LIMIT;
-  const GlaProj g{proj, ld, a2, ld2, bias, rank, tau, H, D, V};
-  const GlaStepArgs p{g, state, state_slots, nslots, vector_rows(g, f32), w, out, ldo, eps};
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return f32 ? launch_step<float>(p, B, st) : launch_step<__nv_bfloat16>(p, B, st);
+  if (rank <= 0 || !(tau > 0.f)) return TFB_ERR_ARG;
+  return run_step(gated_source(proj, ld, a2, ld2, bias, rank, tau, H, D, V), GATED, state, state_slots, nslots, w, out, ldo, B, eps, f32, stream);
+}
+
+TFB_API int tfb_forget_step(const void* proj, long long ld, const void* bias, const void* lower, int gated, float* state, const int* state_slots, int nslots,
+                            const void* w, void* out, long long ldo, int B, int H, int D, int V, float eps, int f32, void* stream) {
+  using namespace tfb;
+  if (!bias || !lower) return TFB_ERR_ARG;
+  return run_step(forget_source(proj, ld, bias, lower, gated, H, D, V), FORGET, state, state_slots, nslots, w, out, ldo, B, eps, f32, stream);
+}
+
+TFB_API int tfb_retention_step(const void* proj, long long ld, const float* head_decay, const float* cos_t, const float* sin_t, int max_pos, int dims,
+                               const int* positions, int gated, float* state, const int* state_slots, int nslots, const void* w, void* out,
+                               long long ldo, int B, int H, int D, int V, float eps, int f32, void* stream) {
+  using namespace tfb;
+  const GlaProj g = retention_source(proj, ld, head_decay, cos_t, sin_t, max_pos, dims, positions, gated, H, D, V);
+  if (bad_retention(g)) return TFB_ERR_ARG;
+  return run_step(g, RETENTION, state, state_slots, nslots, w, out, ldo, B, eps, f32, stream);
 }

@@ -1,8 +1,9 @@
 // Causal softmax attention with grouped key / value heads, keys and values of different sizes and a set of options:
 //
 //   window, keep_first  a query at position i sees the keys j with i - j < window or j < keep_first (window 0: all j <= i)
+//   chunk               it sees the keys of its own chunk of positions (multiples of `chunk` on), and those first ones
 //   softcap             scores become cap tanh(score / cap)
-//   sink                the denominator counts one more key of score 0 without a value
+//   sink                the denominator counts one more key without a value, of score 0 or of a score per head
 //   temp                the query at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)
 //   gate                heads (one logit each) or their entries (one logit each) are multiplied by its sigmoid
 //
@@ -23,12 +24,22 @@ TFB_BOUNDS_DEFINE(head_attention)
 constexpr float LOG2E = 1.4426950408889634f;
 
 struct HeadOpt {
-  int window, keep;
+  int window, chunk, keep;
   float cap;
-  int sink;
+  int sink;               // 1: score 0; 2: sinks[h]
+  const void* sinks;      // [H], in the type of the queries
   float temp_coef;
   int temp_every;
+
+  // the first key that the query behind key i sees, kept ones aside (i, like the keys, counted from a multiple of `chunk`)
+  __host__ __device__ __forceinline__ int first_key(int i) const {
+    return window > 0 ? (i >= window ? i - window + 1 : 0) : chunk > 0 ? i - i % chunk : 0;
+  }
+  __host__ __device__ __forceinline__ bool bounded() const { return window > 0 || chunk > 0; }
 };
+
+template <class T>
+__device__ __forceinline__ float sink_score(const HeadOpt& o, int h) { return o.sink == 2 ? to_f(static_cast<const T*>(o.sinks)[h]) : 0.f; }
 
 __device__ __forceinline__ float query_temp(const HeadOpt& o, int pos) {
   return o.temp_coef == 0.f ? 1.f : fmaf(o.temp_coef, logf(float((pos + 1) / o.temp_every + 1)), 1.f);
@@ -203,8 +214,8 @@ head_attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
   const int b = rem / p.H, h = rem % p.H, hk = h / (p.H / p.G);
   // key blocks: those of the kept first keys, then from the window of the first query on
   int lo_blk = 0, n_first = 0;
-  if (MODE > 0 && p.opt.window > 0) {
-    lo_blk = max(0, pair * 2 * HA_BM + p.q_off - p.opt.window + 1) / HA_BN;
+  if (MODE > 0 && p.opt.bounded()) {
+    lo_blk = p.opt.first_key(pair * 2 * HA_BM + p.q_off) / HA_BN;
     n_first = min((p.opt.keep + HA_BN - 1) / HA_BN, lo_blk);
   }
   auto block_of = [&](int j) { return j < n_first ? j : lo_blk + j - n_first; };
@@ -324,8 +335,9 @@ head_attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
     const float kc = MODE == 2 ? p.opt.cap * LOG2E : 0.f;
     const float sl2 = MODE == 2 ? p.scale * temp / p.opt.cap : p.scale * temp * LOG2E;
     const int hi_g = min(q_idx + p.q_off, p.Skv - 1);
-    const int window = MODE > 0 ? p.opt.window : 0, keep_g = window ? p.opt.keep : 0;
-    const int lo_g = window ? q_idx + p.q_off - window + 1 : -(1 << 30);
+    const bool bounded = MODE > 0 && p.opt.bounded();
+    const int keep_g = bounded ? p.opt.keep : 0, lo_g = bounded ? p.opt.first_key(q_idx + p.q_off) : 0;
+    const int lo_last = bounded ? p.opt.first_key(q0 + HA_BM - 1 + p.q_off) : 0;      // of the tile's last row
     float m = -INFINITY, l = 0.f, alpha_prev = 1.f, mb_prev = 0.f;
     float o[DV];
 #pragma unroll
@@ -339,7 +351,7 @@ head_attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
       tc_fence_after();
       const int k0 = block_of(j) * HA_BN, hi = hi_g - k0, lo = lo_g - k0, keep = keep_g - k0;
       const bool need_mask = k0 + HA_BN - 1 > q0 + p.q_off || k0 + HA_BN > p.Skv ||
-                             (window && q0 + HA_BM + p.q_off - window > k0 && k0 + HA_BN > keep_g);
+                             (bounded && lo_last > k0 && k0 + HA_BN > keep_g);
       // a row may see no key of a block (a query past the end of its sequence, whose row is not stored, or a block before the window
       // of a later query)
       const float2 mxb = need_mask ? tile_max<true, MODE == 2>(tS, m, lo, hi, keep) : tile_max<false, MODE == 2>(tS, m, lo, hi, keep);
@@ -385,8 +397,11 @@ head_attn_fwd_kernel(const __grid_constant__ CUtensorMap tq, const __grid_consta
       }
       if (q_idx < p.S) {
         const long long row = (long long)b * p.S + q_idx;
-        if (MODE > 0 && p.opt.sink) l += ex2(-mb_prev);
         float f = l > 0.f ? 1.f / l : 0.f;
+        if (MODE > 0 && p.opt.sink) {
+          const float sk = sink_score<__nv_bfloat16>(p.opt, h) * LOG2E, M = fmaxf(mb_prev, sk), fm = ex2(mb_prev - M);
+          f = fm / fmaf(l, fm, ex2(sk - M));
+        }
         if (p.gate && !(MODE > 0 && p.gate_entry)) f *= sigmoid_exact(__bfloat162float(p.gate[row * p.ldg + h]));
         __nv_bfloat16* op = p.O + row * p.ldo + h * p.V;
 #pragma unroll
@@ -502,7 +517,7 @@ __global__ void __launch_bounds__(HD_THREADS) head_decode_kernel(const HeadDecod
   for (int k = 0; k < KS; ++k) ldsm(s0 + ((lane & 7) + ((lane >> 3) & 1) * 8) * L::KP + k * 32 + (lane >> 4) * 16, qa[k]);
 
   // the keys that the query sees, in order: the kept first ones, then the window
-  const int pos = p.positions[b], lo = p.opt.window ? max(0, pos + 1 - p.opt.window) : 0, first = min(p.opt.window ? p.opt.keep : 0, lo);
+  const int pos = p.positions[b], lo = p.opt.first_key(pos), first = min(p.opt.bounded() ? p.opt.keep : 0, lo);
   const int total = first + pos + 1 - lo;
   const int per = ((total + p.splits - 1) / p.splits + HD_CHUNK - 1) / HD_CHUNK * HD_CHUNK;
   const int t_begin = sp * per, t_end = min(total, t_begin + per);
@@ -676,7 +691,7 @@ __global__ void __launch_bounds__(HD_THREADS) head_decode_kernel(const HeadDecod
 // one warp per (sequence, head): merge the splits (at most 32), sink, gate
 __global__ void __launch_bounds__(128) head_combine_kernel(const float* __restrict__ acc, const float* __restrict__ ml, const __nv_bfloat16* __restrict__ gate,
                                                            long long ldg, int gate_entry, __nv_bfloat16* __restrict__ o, long long ldo, int n, int H,
-                                                           int V, int splits, int sink) {
+                                                           int V, int splits, const HeadOpt opt) {
   tfb::pdl_sync();
   const int id = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (id >= n) return;
@@ -685,9 +700,13 @@ __global__ void __launch_bounds__(128) head_combine_kernel(const float* __restri
   const float m = lane < splits ? ml[(base + lane) * 2] : -INFINITY;
   const float M = warp_max(m);
   float f = m == -INFINITY ? 0.f : ex2(m - M);
-  float l = warp_add(lane < splits ? ml[(base + lane) * 2 + 1] * f : 0.f);
-  if (sink) l += ex2(-M);
-  f /= l;
+  float l = warp_add(lane < splits ? ml[(base + lane) * 2 + 1] * f : 0.f), fm = 1.f;
+  if (opt.sink) {
+    const float sk = sink_score<__nv_bfloat16>(opt, h) * LOG2E, M2 = fmaxf(M, sk);
+    fm = ex2(M - M2);
+    l = fmaf(l, fm, ex2(sk - M2));
+  }
+  f *= fm / l;
   if (gate && !gate_entry) f *= sigmoid_exact(__bfloat162float(gate[b * ldg + h]));
   for (int d = lane * 4; d < (V + 127) / 128 * 128; d += 128) {
     float v[4] = {0.f, 0.f, 0.f, 0.f};
@@ -784,7 +803,7 @@ __global__ void __launch_bounds__(128) head_any_kernel(const HeadAnyArgs<T> p) {
     f_row[i] = p.scale * query_temp(p.opt, PAGED ? hi_first : p.pos0 + i0 + warp + 4 * i);
   }
   // keys that some row sees, in order: the kept first ones, then from the first row's window on
-  const int keep = p.opt.window ? p.opt.keep : 0, lo = p.opt.window ? max(0, hi_first - p.opt.window + 1) : 0, first = min(keep, lo);
+  const int keep = p.opt.bounded() ? p.opt.keep : 0, lo = p.opt.first_key(hi_first), first = min(keep, lo);
   const int total = first + hi_max + 1 - lo;
   for (int t0 = 0; t0 < total; t0 += AN_K) {
     const int nk = min(AN_K, total - t0);
@@ -814,7 +833,7 @@ __global__ void __launch_bounds__(128) head_any_kernel(const HeadAnyArgs<T> p) {
       s *= f_row[i];
       if (p.opt.cap > 0.f) s = p.opt.cap * tanhf(s / p.opt.cap);
       const int hi = PAGED ? hi_first : i0 + r + p.q_off;
-      if (!(r < n && lane < nk && at <= hi && (p.opt.window == 0 || hi - at < p.opt.window || at < keep))) s = -INFINITY;
+      if (!(r < n && lane < nk && at <= hi && (at >= p.opt.first_key(hi) || at < keep))) s = -INFINITY;
       const float mx = fmaxf(m_run[i], warp_max(s));
       const float mb = mx == -INFINITY ? 0.f : mx;
       const float a = m_run[i] == -INFINITY ? 0.f : expf(m_run[i] - mb);
@@ -835,13 +854,21 @@ __global__ void __launch_bounds__(128) head_any_kernel(const HeadAnyArgs<T> p) {
   }
   __syncthreads();
 #pragma unroll
-  for (int i = 0; i < 4; ++i)
-    if (lane == 0 && warp + 4 * i < QR) sA[warp + 4 * i] = l_run[i] + (p.opt.sink ? expf(-m_run[i]) : 0.f);
+  for (int i = 0; i < 4; ++i) {
+    const int r = warp + 4 * i;
+    if (lane != 0 || r >= QR) continue;
+    float f = 1.f / l_run[i];
+    if (p.opt.sink && r < n) {
+      const float sk = sink_score<T>(p.opt, head_of(r)), M = fmaxf(m_run[i], sk), fm = expf(m_run[i] - M);
+      f = fm / fmaf(l_run[i], fm, expf(sk - M));
+    }
+    sA[r] = f;
+  }
   __syncthreads();
   for (int r = warp; r < n; r += 4) {
     const long long row = row_of(r);
     const int h = head_of(r);
-    float f = 1.f / sA[r];
+    float f = sA[r];
     if (p.gate && !p.gate_entry) f *= sigmoid_exact(to_f(p.gate[row * p.ldg + h]));
     for (int d = lane; d < V; d += 32) {
       float v = sO[r * V + d] * f;
@@ -869,20 +896,25 @@ static int launch_any(HeadAnyArgs<T> p, int B, cudaStream_t st) {
 }
 
 static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
-static bool bad_opt(const HeadOpt& o) { return o.window < 0 || o.keep < 0 || !(o.cap >= 0.f) || o.temp_every < 1; }
+static bool bad_opt(const HeadOpt& o) {
+  return o.window < 0 || o.chunk < 0 || (o.window && o.chunk) || o.keep < 0 || !(o.cap >= 0.f) || o.temp_every < 1 || o.sink < 0 || o.sink > 2 ||
+         (o.sink == 2 && !o.sinks);
+}
 
 }  // namespace tfb
 
 using bf16 = __nv_bfloat16;
 
 // q [B*S, ldq]: H heads of D entries; k, v [B*Skv, ldk / ldv]: G heads of D / V entries; gate [B*S, ldg]: one logit per head, or per entry
-// of the heads (gate_entry), or null.  The queries are the last S of the Skv keys; query i stands at position pos0 + i.  With a window,
-// keys between the kept first ones and the first query's window may be left out of k and v.  o [B*S, ldo]: H heads of V entries.
+// of the heads (gate_entry), or null.  The queries are the last S of the Skv keys; query i stands at position pos0 + i.  With a window or
+// chunks, keys between the kept first ones and the first query's window, or the start of its chunk, may be left out of k and v (with chunks
+// and no kept ones, the first key then stands at a multiple of the chunk).  sink, sinks: see HeadOpt.  o [B*S, ldo]: H heads of V entries.
 TFB_API int tfb_head_attn(const void* q, long long ldq, const void* k, long long ldk, const void* v, long long ldv, void* o, long long ldo,
                           const void* gate, long long ldg, int gate_entry, int B, int S, int Skv, int H, int G, int D, int V, float scale, int window,
-                          int keep, float cap, int sink, float temp_coef, int temp_every, int pos0, int f32, int* status, void* stream) {
+                          int chunk, int keep, float cap, int sink, const void* sinks, float temp_coef, int temp_every, int pos0, int f32, int* status,
+                          void* stream) {
   using namespace tfb;
-  const HeadOpt opt{window, keep, cap, sink, temp_coef, temp_every};
+  const HeadOpt opt{window, chunk, keep, cap, sink, sinks, temp_coef, temp_every};
   if (B <= 0 || B > 65535 || S <= 0 || Skv < S || G <= 0 || H % G || H > 65535 || D <= 0 || V <= 0 || pos0 < 0 || bad_opt(opt)) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   // the running maximum is taken of the scores before the factors: those have to be positive
@@ -891,7 +923,7 @@ TFB_API int tfb_head_attn(const void* q, long long ldq, const void* k, long long
   if (tc) {
     HeadAttnParams p{B, S, H, G, Skv, Skv - S, D, V, scale, opt, pos0, static_cast<const bf16*>(gate), ldg, gate ? gate_entry : 0,
                      static_cast<bf16*>(o), ldo, status};
-    const int mode = cap > 0.f ? 2 : (window || sink || temp_coef != 0.f || p.gate_entry) ? 1 : 0;
+    const int mode = cap > 0.f ? 2 : (opt.bounded() || sink || temp_coef != 0.f || p.gate_entry) ? 1 : 0;
 #define TFB_HA(DK, DV)                                                                                                            \
   return mode == 0 ? launch_head_attn<DK, DV, 0>(q, ldq, k, ldk, v, ldv, p, st)                                                   \
                    : mode == 1 ? launch_head_attn<DK, DV, 1>(q, ldq, k, ldk, v, ldv, p, st) : launch_head_attn<DK, DV, 2>(q, ldq, k, ldk, v, ldv, p, st)
@@ -933,10 +965,10 @@ TFB_API int tfb_head_decode_plan(int B, int H, int G, int D, int V, int max_keys
 // One query per sequence at positions[b] over the cached rows (k [nslots][G D], v [nslots][G V]); q [B, ldq], o [B, ldo].
 TFB_API int tfb_head_decode(const void* q, long long ldq, const void* k, const void* v, long long nslots, const int* block_table, int max_pages,
                             int page, const int* positions, void* o, long long ldo, const void* gate, long long ldg, int gate_entry, float* acc,
-                            float* ml, int splits, int B, int H, int G, int D, int V, float scale, int window, int keep, float cap, int sink,
-                            float temp_coef, int temp_every, int f32, int* status, void* stream) {
+                            float* ml, int splits, int B, int H, int G, int D, int V, float scale, int window, int chunk, int keep, float cap, int sink,
+                            const void* sinks, float temp_coef, int temp_every, int f32, int* status, void* stream) {
   using namespace tfb;
-  const HeadOpt opt{window, keep, cap, sink, temp_coef, temp_every};
+  const HeadOpt opt{window, chunk, keep, cap, sink, sinks, temp_coef, temp_every};
   if (B <= 0 || B > 65535 || G <= 0 || H % G || D <= 0 || V <= 0 || page <= 0 || nslots < page || bad_opt(opt)) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (acc && tfb_head_decode_plan(B, H, G, D, V, 1, f32) > 0) {
@@ -947,7 +979,7 @@ TFB_API int tfb_head_decode(const void* q, long long ldq, const void* k, const v
                            : (V <= 64 ? launch_head_decode<128, 64>(p, B, st) : launch_head_decode<128, 128>(p, B, st));
     if (rc) return rc;
     launch_k(head_combine_kernel, (B * H + 3) / 4, 128, 0, st, acc, ml, static_cast<const bf16*>(gate), ldg, gate_entry, static_cast<bf16*>(o), ldo,
-             B * H, H, V, splits, sink);
+             B * H, H, V, splits, opt);
     return int(cudaGetLastError());
   }
 #define TFB_ANY(T)                                                                                                                              \

@@ -2,12 +2,13 @@
 // backward pass (the training form is moe_routing.cu).
 //
 //   moe_route          per token: the k largest of logits (+ bias) (fp32, the lower index first among equals) and the softmax over them,
-//                      or the k largest sigmoids among the experts of the best groups, weighted by them over their sum;
+//                      or the k largest sigmoids among the experts of the best groups, weighted by them over their sum, or the k
+//                      largest entries of the softmax over all experts, weighted by themselves;
 //                      then the rows of the expert buffers: every expert's assignments are consecutive rows from a multiple
 //                      of 128 on, so that a 128-row tile of the grouped product belongs to one expert.  Few tokens (decode
 //                      steps): one block does all of it; many: selection with per-block counts, then the scan and row numbers.
 //   moe_gather         token rows to their assignments' rows
-//   moe_glu            silu(gate) * up of the assigned rows (a decode step's buffers are mostly padding)
+//   moe_glu            act(gate) * up of the assigned rows (a decode step's buffers are mostly padding)
 //   moe_weighted_sum   y[t] = base[t] [* sigmoid(gate[t])] + sum_k w[t, k] * rows[row_of[t, k]], summed in fp32
 #include <limits.h>
 
@@ -29,6 +30,7 @@ struct RouteArgs {
   int* counts;                // [E]
   int tiles;
   int sigmoid, groups, keep;  // scores are sigmoids, of the experts of `keep` of `groups` groups of E / groups neighbours
+  int all;                    // the softmax is over all experts, not over the chosen ones
   float scale;
 };
 
@@ -85,8 +87,18 @@ __device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int la
       for (int i = 0; i < PER; ++i)
         if (lane + i * 32 < p.E && !((kept >> ((lane + i * 32) / n)) & 1u)) key[i] = 0u;
     }
-    float first = 0.f, sum = 0.f, mine = 0.f;
+    float first = 0.f, sum = 0.f, mine = 0.f, total = 0.f;
     int e_mine = 0;
+    if (p.all) {
+      uint32_t top = 0u;
+#pragma unroll
+      for (int i = 0; i < PER; ++i) top = max(top, key[i]);
+      first = unordered(__reduce_max_sync(0xffffffffu, top));
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if (key[i]) total += expf(unordered(key[i]) - first);
+      total = warp_add(total);
+    }
     for (int k = 0; k < p.K; ++k) {
       uint32_t best = key[0];
       int e = lane;
@@ -108,12 +120,19 @@ __device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int la
     if (lane < p.K) {
       const int i = t * p.K + lane;
       p.idx[i] = e_mine;
-      p.w[i] = p.sigmoid ? mine / (sum + 1e-20f) * p.scale : mine / sum;
+      p.w[i] = p.sigmoid ? mine / (sum + 1e-20f) * p.scale : mine / (p.all ? total : sum);
       note(i, e_mine, atomicAdd(count + e_mine, 1));
     }
   } else {
-    float last = INFINITY, first = 0.f, sum = 0.f;
+    float last = INFINITY, first = 0.f, sum = 0.f, total = 0.f;
     int last_e = -1;
+    if (p.all) {
+      float top = -INFINITY;
+      for (int e = lane; e < p.E; e += 32) top = fmaxf(top, biased_logit(p, z, e));
+      top = warp_max(top);
+      for (int e = lane; e < p.E; e += 32) total += expf(biased_logit(p, z, e) - top);
+      total = warp_add(total);
+    }
     for (int k = 0; k < p.K; ++k) {
       float best = -INFINITY;
       int e_best = INT_MAX;
@@ -142,7 +161,7 @@ __device__ __forceinline__ void choose_experts(const RouteArgs& p, int t, int la
       }
     }
     __syncwarp();
-    const float f = p.sigmoid ? p.scale / (sum + 1e-20f) : 1.f / sum;
+    const float f = p.sigmoid ? p.scale / (sum + 1e-20f) : 1.f / (p.all ? total : sum);
     for (int k = lane; k < p.K; k += 32) p.w[(long long)t * p.K + k] *= f;
   }
 }
@@ -260,9 +279,9 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ x
   }
 }
 
-template <class T, int VEC>
+template <class T, int VEC, int ACT>
 __global__ void __launch_bounds__(256) moe_glu_kernel(const T* __restrict__ in, long long ldi, const int* __restrict__ row_of, T* __restrict__ out,
-                                                      long long ldo, long long assignments, int F) {
+                                                      long long ldo, long long assignments, int F, float limit) {
   tfb::pdl_sync();
   const int per = F / VEC;
   const long long n = assignments * per;
@@ -273,7 +292,7 @@ __global__ void __launch_bounds__(256) moe_glu_kernel(const T* __restrict__ in, 
     load_n<VEC>(in + row * ldi + c, g);
     load_n<VEC>(in + row * ldi + F + c, u);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) g[e] = silu_exact(g[e]) * u[e];
+    for (int e = 0; e < VEC; ++e) g[e] = glu_value<ACT>(g[e], u[e], limit);
     store_n<VEC>(out + row * ldo + c, g);
   }
 }
@@ -320,20 +339,22 @@ static int blocks_for(long long items) {
 
 using bf16 = __nv_bfloat16;
 
-// logits [T, ld] fp32, bias [E] (bias_f32: fp32, otherwise bf16) or null; sigmoid, groups, keep, scale: see RouteArgs.  idx, row_of, rank (scratch): int [T, K]; w: fp32 [T, K]; counts
+// logits [T, ld] fp32, bias [E] (bias_f32: fp32, otherwise bf16) or null; groups, keep, scale: see RouteArgs;
+// score: 0 softmax over the chosen, 1 sigmoid, 2 softmax over all.  idx, row_of, rank (scratch): int [T, K]; w: fp32 [T, K]; counts
 // (scratch): int [E]; expert_of_tile: int [tiles], tiles >= T K / 128 + min(E, T K).
 TFB_API int tfb_moe_route(const float* logits, const void* bias, int T, int E, int K, int* idx, float* w, int* row_of, int* expert_of_tile,
-                          int* counts, int* rank, int tiles, long long ld, int bias_f32, int sigmoid, int groups, int keep, float scale,
+                          int* counts, int* rank, int tiles, long long ld, int bias_f32, int score, int groups, int keep, float scale,
                           void* stream) {
   using namespace tfb;
-  if (T <= 0 || E <= 0 || K <= 0 || K > E) return TFB_ERR_ARG;
+  if (T <= 0 || E <= 0 || K <= 0 || K > E || score < 0 || score > 2) return TFB_ERR_ARG;
+  const int sigmoid = score == 1;
   if (sigmoid && (bias || groups <= 0 || E % groups || keep <= 0 || keep > groups || K > E / groups * keep)) return TFB_ERR_ARG;
   if (!sigmoid && groups != 1) return TFB_ERR_ARG;
   const bool grouped = sigmoid && keep < groups;
   const long long a = (long long)T * K;
   if (tiles < a / 128 + (E < a ? E : a)) return TFB_ERR_ARG;
   if (E > 8192 || a > INT_MAX / 2) return TFB_ERR_LIMIT;
-  RouteArgs p{logits, ld, bias, bias_f32, T, E, K, idx, w, rank, row_of, expert_of_tile, counts, tiles, sigmoid, groups, keep, scale};
+  RouteArgs p{logits, ld, bias, bias_f32, T, E, K, idx, w, rank, row_of, expert_of_tile, counts, tiles, sigmoid, groups, keep, score == 2, scale};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (grouped && (groups > 32 || E > 1024 || K > 32)) return TFB_ERR_LIMIT;
   if (grouped && E > 256) return launch_route<32>(p, st);
@@ -360,17 +381,28 @@ TFB_API int tfb_moe_gather(const void* x, long long ldx, const int* row_of, void
   return int(cudaGetLastError());
 }
 
-// rows [gate | up] of 2 F entries -> silu(gate) * up, for the `assignments` rows that row_of names
-TFB_API int tfb_moe_glu(const void* in, long long ldi, const int* row_of, void* out, long long ldo, int assignments, int F, int f32, void* stream) {
+// rows [gate | up] of 2 F entries -> act(gate) * up, for the `assignments` rows that row_of names; act, limit: see glu_value
+TFB_API int tfb_moe_glu(const void* in, long long ldi, const int* row_of, void* out, long long ldo, int assignments, int F, int act, float limit, int f32,
+                        void* stream) {
   using namespace tfb;
-  if (assignments <= 0 || F <= 0) return TFB_ERR_ARG;
+  if (assignments <= 0 || F <= 0 || act < 0 || act > GLU_CLAMPED) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int vec = f32 ? 4 : 8;
   const bool v = F % vec == 0 && ldi % vec == 0 && ldo % vec == 0 && al16(in) && al16(out);
   const long long a = assignments;
-#define TFB_ARGS(T) static_cast<const T*>(in), ldi, row_of, static_cast<T*>(out), ldo, a, F
-  TFB_BY_TYPE(moe_glu_kernel, blocks_for(a * (v ? F / vec : F)), v, TFB_ARGS);
-#undef TFB_ARGS
+  const int grid = blocks_for(a * (v ? F / vec : F));
+#define TFB_GLU1(T, VEC, ACT) \
+  launch_k(moe_glu_kernel<T, VEC, ACT>, grid, 256, 0, st, static_cast<const T*>(in), ldi, row_of, static_cast<T*>(out), ldo, a, F, limit)
+#define TFB_GLU(T, VEC)                                    \
+  do {                                                     \
+    if (act == GLU_CLAMPED) TFB_GLU1(T, VEC, GLU_CLAMPED); \
+    else if (act == GLU_GELU) TFB_GLU1(T, VEC, GLU_GELU);  \
+    else TFB_GLU1(T, VEC, GLU_SILU);                       \
+  } while (0)
+  if (f32) { if (v) TFB_GLU(float, 4); else TFB_GLU(float, 1); }
+  else { if (v) TFB_GLU(bf16, 8); else TFB_GLU(bf16, 1); }
+#undef TFB_GLU
+#undef TFB_GLU1
   return int(cudaGetLastError());
 }
 

@@ -1,4 +1,4 @@
-// Products of few rows (decode steps): out[M, N] = act(x[M, K] . W[N, K]^T) for M <= 64 in bf16 with fp32 accumulation, one launch
+// Products of few rows (decode steps): out[M, N] = act(x[M, K] . W[N, K]^T [+ bias]) for M <= 64 in bf16 with fp32 accumulation, one launch
 // and no workspace.  A 128-row tcgen05 tile would be mostly padding and its split-K form needs a second kernel; here a block
 // takes 16 columns, its eight warps share the reduction dimension, and the weights go from global memory to the operand registers of
 // mma.sync without a stop: both operands may be read in the same permuted order of k, so a lane takes 16 consecutive entries of a
@@ -21,6 +21,7 @@ struct SkinnyArgs {
   int x_head, out_head;             // entries between the heads of x and of out; W advances by N rows
   const __nv_bfloat16* gate;        // [M, ldg] or null: head h is multiplied by sigmoid(gate[:, h])
   long long ldg;
+  const __nv_bfloat16* bias;        // [N] or null
 };
 
 struct Row16 { uint32_t u[8]; };      // 16 consecutive entries of a row
@@ -77,6 +78,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32) skinny_linear_kernel(const Skin
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < SK_WARPS; ++w) v += red[w][m][n];
+    if (p.bias) v += __bfloat162float(p.bias[n0 + n]);
     if (p.act == 4) {
       v = fmaxf(v, 0.f);
       v *= v;
@@ -118,10 +120,10 @@ TFB_API int tfb_skinny_fits(int M, int N, int K) {
 
 // act: 0 none, 4 relu squared.  rows: rows of a block (16, 32 or 64; 0: the kernel's choice).  Row pitches are multiples of 8 entries, x and w aligned to 16 bytes.
 TFB_API int tfb_skinny_linear(const void* x, long long ldx, const void* w, long long ldw, void* out, long long ldo, int M, int N, int K, int act,
-                              int out_f32, int rows, void* stream) {
+                              int out_f32, int rows, const void* bias, void* stream) {
   if (M > 64 || (act != 0 && act != 4)) return TFB_ERR_ARG;
   return launch_skinny(tfb::SkinnyArgs{static_cast<const bf16*>(x), static_cast<const bf16*>(w), ldx, ldw, out, ldo, M, N, K, act, out_f32, 0, 0,
-                                       nullptr, 0}, 1, rows, stream);
+                                       nullptr, 0, static_cast<const bf16*>(bias)}, 1, rows, stream);
 }
 
 // One product per head: x [M, ldx] (x_head entries between heads), w: heads blocks [N, K] stacked on the rows, out [M, ldo] (N entries per
@@ -129,5 +131,5 @@ TFB_API int tfb_skinny_linear(const void* x, long long ldx, const void* w, long 
 TFB_API int tfb_skinny_linear_heads(const void* x, long long ldx, int x_head, const void* w, long long ldw, void* out, long long ldo, const void* gate,
                                     long long ldg, int M, int heads, int N, int K, int rows, void* stream) {
   return launch_skinny(tfb::SkinnyArgs{static_cast<const bf16*>(x), static_cast<const bf16*>(w), ldx, ldw, out, ldo, M, N, K, 0, 0, x_head, N,
-                                       static_cast<const bf16*>(gate), ldg}, heads, rows, stream);
+                                       static_cast<const bf16*>(gate), ldg, nullptr}, heads, rows, stream);
 }

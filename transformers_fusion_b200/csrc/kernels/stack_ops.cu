@@ -1,6 +1,7 @@
 // Row operators of decoders with a 32-bit residual stream: scaled embedding, norm of a sublayer's output + residual + norm of (or
-// rounding for) the next sublayer's input in one pass, activations, partial rotary embedding fused with the append to the paged
-// cache, gather of cached rows, and a true fp32 matrix product (dense, one block per head, or rows grouped by expert).  Every kernel exists for bf16 and for fp32
+// rounding for) the next sublayer's input in one pass, activations, norm of the recurrent mixers' head outputs, partial rotary embedding
+// (with a norm of the heads in front) fused with the append to the paged cache, gather of cached rows, and a true fp32 matrix product
+// (dense, one block per head, or rows grouped by expert).  Every kernel exists for bf16 and for fp32
 // activations; the statistics, the residual and the rotation are fp32 in both.
 #include "tfb_elem.cuh"
 #include "tfb_host.h"
@@ -189,12 +190,6 @@ __device__ __forceinline__ float act_f32(float v, int act) {
   return v;
 }
 
-// 0.5 z (1 + tanh(u)) = z sigmoid(2 u), u = sqrt(2 / pi) (z + 0.044715 z^3)
-__device__ __forceinline__ float gelu_tanh_exact(float z) {
-  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
-  return z / (1.f + expf(-2.f * u));
-}
-
 template <class T>
 __global__ void __launch_bounds__(256) act_rows_kernel(const T* __restrict__ in, long long ldi, T* __restrict__ out, long long ldo, int M, int N, int act) {
   tfb::pdl_sync();
@@ -204,10 +199,11 @@ __global__ void __launch_bounds__(256) act_rows_kernel(const T* __restrict__ in,
 }
 
 // ------------------------------------------------------------------------------------------------
-// [gate | up] -> act(gate) * up; act: 0 silu, 1 the tanh form of gelu
+// [gate | up] -> act(gate) * up; act: see glu_value (tfb_elem.cuh)
 // ------------------------------------------------------------------------------------------------
 template <class T, int VEC, int ACT>
-__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, long long ldi, T* __restrict__ out, long long ldo, int M, int F) {
+__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, long long ldi, T* __restrict__ out, long long ldo, int M, int F,
+                                                  float limit) {
   tfb::pdl_sync();
   const int per = F / VEC;
   const long long n = (long long)M * per;
@@ -218,8 +214,53 @@ __global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ in, long
     load_n<VEC>(in + m * ldi + c, g);
     load_n<VEC>(in + m * ldi + F + c, u);
 #pragma unroll
-    for (int e = 0; e < VEC; ++e) g[e] = (ACT == 0 ? silu_exact(g[e]) : gelu_tanh_exact(g[e])) * u[e];
+    for (int e = 0; e < VEC; ++e) g[e] = glu_value<ACT>(g[e], u[e], limit);
     store_n<VEC>(out + m * ldo + c, g);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------
+// norm of the head outputs of a recurrent mixer:  o / rms(o) [* w] [* silu(gate)]
+// ------------------------------------------------------------------------------------------------
+template <class T, int VEC>
+__global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long ldg,
+                                                         const T* __restrict__ w, T* __restrict__ out, long long ldo, int rows, int H, int V,
+                                                         float eps) {
+  tfb::pdl_sync();
+  const int lane = threadIdx.x & 31;
+  const long long nwarps = (long long)gridDim.x * (blockDim.x >> 5), n = (long long)rows * H;
+  for (long long i = blockIdx.x * (long long)(blockDim.x >> 5) + (threadIdx.x >> 5); i < n; i += nwarps) {
+    const long long r = i / H;
+    const int h = int(i % H);
+    const float* src = o + i * V;
+    const T* gt = gate ? gate + r * ldg + h * V : nullptr;
+    T* dst = out + r * ldo + h * V;
+    float x0[VEC], g0[VEC], x[VEC], g[VEC], wv[VEC];
+    float ss = 0.f;
+    for (int j = lane * VEC; j < V; j += 32 * VEC) {
+      load_n<VEC>(src + j, x);
+      if (j == lane * VEC) {
+        if (gt) load_n<VEC>(gt + j, g0);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) x0[e] = x[e];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss = fmaf(x[e], x[e], ss);
+    }
+    const float rs = 1.f / sqrtf(warp_add(ss) / V + eps);
+    for (int j = lane * VEC; j < V; j += 32 * VEC) {
+      if (w) load_n<VEC>(w + j, wv);
+      if (j == lane * VEC) {
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) { x[e] = x0[e]; g[e] = g0[e]; }
+      } else {
+        load_n<VEC>(src + j, x);
+        if (gt) load_n<VEC>(gt + j, g);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x[e] *= rs * (w ? wv[e] : 1.f) * (gt ? silu_exact(g[e]) : 1.f);
+      store_n<VEC>(dst + j, x);
+    }
   }
 }
 
@@ -284,14 +325,15 @@ __global__ void __launch_bounds__(256) rope_append_kernel(T* __restrict__ qkv, l
   }
 }
 
-// The same with an RMS norm of every q and k head (weights wq, wk) in front of the rotation.  L lanes share a head, each with two pieces
+// The same with an RMS norm of every q and k head (weights wq, wk; null: none) in front of the rotation and, behind it, a factor per query
+// head (qf, or null).  L lanes share a head, each with two pieces
 // of four entries in registers: for rotated entries, four of the first half and their partners in the second (L a power of two,
 // 8 L >= D; D, v_cols and the rotated entries are multiples of eight).  Units of a row: nq + nk heads, then pieces of 8 L entries of v; a
 // group of L lanes takes NRA_UNITS of them, all loads ahead of the reductions.
 constexpr int NRA_UNITS = 2;
 template <class T, int L>
 __global__ void __launch_bounds__(256, 4) norm_rope_append_kernel(T* __restrict__ qkv, long long ld, const T* __restrict__ wq, const T* __restrict__ wk,
-                                                                  float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                                                  const T* __restrict__ qf, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                                                                   int max_pos, const int* __restrict__ positions, const long long* __restrict__ slots,
                                                                   T* __restrict__ kpool, T* __restrict__ vpool, long long nslots, int rows, int nq,
                                                                   int nk, int D, int dims, int v_cols) {
@@ -314,7 +356,7 @@ __global__ void __launch_bounds__(256, 4) norm_rope_append_kernel(T* __restrict_
     const int a = u < heads ? c0 : l * 8, b = u < heads ? c1 : l * 8 + 4;
     load_n<4>(row + at[i] + a, x[i][0]);
     load_n<4>(row + at[i] + b, x[i][1]);
-    if (u < heads) {
+    if (u < heads && wq) {
       load_n<4>((u < nq ? wq : wk) + c0, w[i][0]);
       load_n<4>((u < nq ? wq : wk) + c1, w[i][1]);
     }
@@ -353,12 +395,12 @@ __global__ void __launch_bounds__(256, 4) norm_rope_append_kernel(T* __restrict_
       }
       continue;
     }
-    const float f = rsqrtf(fmaf(ss[i], inv, eps));
+    const float f = rsqrtf(fmaf(ss[i], inv, eps)) * (qf && u < nq ? to_f(qf[u]) : 1.f);
     float a[4], b[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      a[e] = x[i][0][e] * f * w[i][0][e];
-      b[e] = x[i][1][e] * f * w[i][1][e];
+      a[e] = x[i][0][e] * f * (wq ? w[i][0][e] : 1.f);
+      b[e] = x[i][1][e] * f * (wq ? w[i][1][e] : 1.f);
       if (turns) {
         const float p = a[e] * c[e] - b[e] * s[e];
         b[e] = b[e] * c[e] + a[e] * s[e];
@@ -378,7 +420,7 @@ __global__ void __launch_bounds__(256, 4) norm_rope_append_kernel(T* __restrict_
 // any sizes: one warp per head (or per 64 entries of v)
 template <class T>
 __global__ void __launch_bounds__(256) norm_rope_append_any_kernel(T* __restrict__ qkv, long long ld, const T* __restrict__ wq, const T* __restrict__ wk,
-                                                                   float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
+                                                                   const T* __restrict__ qf, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                                                                    int max_pos, const int* __restrict__ positions, const long long* __restrict__ slots,
                                                                    T* __restrict__ kpool, T* __restrict__ vpool, long long nslots, int rows, int nq,
                                                                    int nk, int D, int dims, int v_cols) {
@@ -402,19 +444,19 @@ __global__ void __launch_bounds__(256) norm_rope_append_any_kernel(T* __restrict
   T* kp = u >= nq && slot >= 0 ? kpool + (slot * nk + (u - nq)) * D : nullptr;
   float ss = 0.f;
   for (int d = lane; d < D; d += 32) ss = fmaf(to_f(x[d]), to_f(x[d]), ss);
-  const float f = 1.f / sqrtf(warp_add(ss) / D + eps);     // its shuffles also order the reads before the writes below
+  const float f = 1.f / sqrtf(warp_add(ss) / D + eps) * (qf && u < nq ? to_f(qf[u]) : 1.f);     // its shuffles also order the reads before the writes below
   int pos = dims ? positions[r] : 0;
   TFB_BOUNDS(dims == 0 || (pos >= 0 && pos < max_pos), 61, pos, max_pos);
   pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
   for (int d = lane; d < D; d += 32) {
     if (d >= half && d < dims) continue;
-    const float a = to_f(x[d]) * f * to_f(w[d]);
+    const float a = to_f(x[d]) * f * (w ? to_f(w[d]) : 1.f);
     if (d >= dims) {
       x[d] = from_f<T>(a);
       if (kp) kp[d] = from_f<T>(a);
       continue;
     }
-    const float b = to_f(x[d + half]) * f * to_f(w[d + half]);
+    const float b = to_f(x[d + half]) * f * (w ? to_f(w[d + half]) : 1.f);
     const float c = cos_t[(long long)pos * half + d], s = sin_t[(long long)pos * half + d];
     const T p = from_f<T>(a * c - b * s), q = from_f<T>(b * c + a * s);
     x[d] = p;
@@ -461,6 +503,7 @@ struct GemmF32 {
   long long ldg;
   const int* expert_of_tile;
   int experts;
+  const float* bias;          // [N], added ahead of the activation, or null
 };
 
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32 p) {
@@ -515,7 +558,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32 p) {
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < p.N) C[(long long)m * p.ldc + n] = act_f32(acc[i][j], p.act) * f;
+      if (n < p.N) C[(long long)m * p.ldc + n] = act_f32(acc[i][j] + (p.bias ? p.bias[n] : 0.f), p.act) * f;
     }
   }
 }
@@ -575,16 +618,21 @@ TFB_API int tfb_act_rows(const void* in, long long ldi, void* out, long long ldo
   return int(cudaGetLastError());
 }
 
-// act: see glu_kernel
-TFB_API int tfb_glu(const void* in, long long ldi, void* out, long long ldo, int M, int F, int act, int f32, void* stream) {
+// act, limit: see glu_value
+TFB_API int tfb_glu(const void* in, long long ldi, void* out, long long ldo, int M, int F, int act, float limit, int f32, void* stream) {
   using namespace tfb;
-  if (M <= 0 || F <= 0 || act < 0 || act > 1) return TFB_ERR_ARG;
+  if (M <= 0 || F <= 0 || act < 0 || act > GLU_CLAMPED) return TFB_ERR_ARG;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int vec = f32 ? 4 : 8;
   const bool v = F % vec == 0 && ldi % vec == 0 && ldo % vec == 0 && aligned(in, 16) && aligned(out, 16);
   const int grid = grid_for((long long)M * (v ? F / vec : F));
-#define TFB_GLU1(T, VEC, ACT) launch_k(glu_kernel<T, VEC, ACT>, grid, 256, 0, st, static_cast<const T*>(in), ldi, static_cast<T*>(out), ldo, M, F)
-#define TFB_GLU(T, VEC) do { if (act) TFB_GLU1(T, VEC, 1); else TFB_GLU1(T, VEC, 0); } while (0)
+#define TFB_GLU1(T, VEC, ACT) launch_k(glu_kernel<T, VEC, ACT>, grid, 256, 0, st, static_cast<const T*>(in), ldi, static_cast<T*>(out), ldo, M, F, limit)
+#define TFB_GLU(T, VEC)                                   \
+  do {                                                    \
+    if (act == GLU_CLAMPED) TFB_GLU1(T, VEC, GLU_CLAMPED); \
+    else if (act == GLU_GELU) TFB_GLU1(T, VEC, GLU_GELU); \
+    else TFB_GLU1(T, VEC, GLU_SILU);                      \
+  } while (0)
   if (f32) { if (v) TFB_GLU(float, 4); else TFB_GLU(float, 1); }
   else { if (v) TFB_GLU(bf16, 8); else TFB_GLU(bf16, 1); }
 #undef TFB_GLU
@@ -592,12 +640,32 @@ TFB_API int tfb_glu(const void* in, long long ldi, void* out, long long ldo, int
   return int(cudaGetLastError());
 }
 
-// As tfb_rope_append behind an RMS norm (weights wq, wk of D entries) of every q and k head; dims may be 0.
-TFB_API int tfb_norm_rope_append(void* qkv, long long ld, const void* wq, const void* wk, float eps, const float* cos_t, const float* sin_t,
+// o [rows, H, V] fp32; gate [rows, ldg] and w [V] may be null
+TFB_API int tfb_gated_norm(const float* o, const void* gate, long long ldg, const void* w, void* out, long long ldo, int rows, int H, int V,
+                           float eps, int f32, void* stream) {
+  using namespace tfb;
+  if (rows <= 0 || H <= 0 || V <= 0) return TFB_ERR_ARG;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const long long blocks = ((long long)rows * H + 7) / 8;
+  const int grid = int(blocks < 148ll * 32 ? blocks : 148ll * 32);
+  auto al = [](const void* x, int n) { return (reinterpret_cast<uintptr_t>(x) & (n - 1)) == 0; };
+  const int es = f32 ? 4 : 2;
+  const bool v4 = V % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && al(o, 16) && (!gate || al(gate, 4 * es)) && (!w || al(w, 4 * es)) && al(out, 4 * es);
+#define TFB_GN(T, VEC) launch_k(gated_norm_kernel<T, VEC>, grid, 256, 0, st, o, static_cast<const T*>(gate), ldg, static_cast<const T*>(w), \
+                                static_cast<T*>(out), ldo, rows, H, V, eps)
+  if (f32) { if (v4) TFB_GN(float, 4); else TFB_GN(float, 1); }
+  else { if (v4) TFB_GN(bf16, 4); else TFB_GN(bf16, 1); }
+#undef TFB_GN
+  return int(cudaGetLastError());
+}
+
+// As tfb_rope_append behind an RMS norm (weights wq, wk of D entries, or none) of every q and k head; qf: a factor per query head, or
+// null; dims may be 0.
+TFB_API int tfb_norm_rope_append(void* qkv, long long ld, const void* wq, const void* wk, const void* qf, float eps, const float* cos_t, const float* sin_t,
                                  int max_pos, const int* positions, const long long* slots, void* kpool, void* vpool, long long nslots, int rows,
                                  int nq, int nk, int D, int dims, int v_cols, int f32, void* stream) {
   using namespace tfb;
-  if (rows <= 0 || nq <= 0 || nk <= 0 || D <= 0 || dims < 0 || (dims & 1) || dims > D || (dims && (!cos_t || !sin_t || max_pos <= 0)) || !wq || !wk)
+  if (rows <= 0 || nq <= 0 || nk <= 0 || D <= 0 || dims < 0 || (dims & 1) || dims > D || (dims && (!cos_t || !sin_t || max_pos <= 0)) || !wq != !wk)
     return TFB_ERR_ARG;
   if (nslots == 0) slots = nullptr;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
@@ -607,7 +675,7 @@ TFB_API int tfb_norm_rope_append(void* qkv, long long ld, const void* wq, const 
   const int units = nq + nk + (v_cols + piece - 1) / piece;
   const long long blocks = ((long long)rows * (v ? (units + NRA_UNITS - 1) / NRA_UNITS : units) * L + 255) / 256;
   if (blocks * 256 > 0x7fffffffll) return TFB_ERR_LIMIT;
-#define TFB_NRA(KERN, T) launch_k(KERN, int(blocks), 256, 0, st, static_cast<T*>(qkv), ld, static_cast<const T*>(wq), static_cast<const T*>(wk), eps, \
+#define TFB_NRA(KERN, T) launch_k(KERN, int(blocks), 256, 0, st, static_cast<T*>(qkv), ld, static_cast<const T*>(wq), static_cast<const T*>(wk), static_cast<const T*>(qf), eps, \
                                   cos_t, sin_t, max_pos, positions, slots, static_cast<T*>(kpool), static_cast<T*>(vpool), nslots, rows, nq, nk, D, \
                                   dims, v_cols)
 #define TFB_NRL(T)                                                          \
@@ -659,16 +727,16 @@ TFB_API int tfb_gather_rows(const void* pool, long long nslots, const int* pages
 }
 
 TFB_API int tfb_gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N, int K, int act,
-                         void* stream) {
+                         const float* bias, void* stream) {
   using namespace tfb;
-  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, 0, act, 0, 0, 0, nullptr, 0, nullptr, 0}, 1, stream);
+  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, 0, act, 0, 0, 0, nullptr, 0, nullptr, 0, bias}, 1, stream);
 }
 
 // One product per head: C[:, h * c_head ...] = A[:, h * a_head ...] . B_h^T (B_h: N rows of B, or K rows with b_kn) * sigmoid(gate[:, h]).
 TFB_API int tfb_gemm_f32_heads(const float* A, long long lda, int a_head, const float* B, long long ldb, int b_kn, float* C, long long ldc, int c_head,
                                const float* gate, long long ldg, int M, int heads, int N, int K, void* stream) {
   using namespace tfb;
-  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, b_kn, 0, a_head, (long long)(b_kn ? K : N) * ldb, c_head, gate, ldg, nullptr, 0},
+  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, b_kn, 0, a_head, (long long)(b_kn ? K : N) * ldb, c_head, gate, ldg, nullptr, 0, nullptr},
                          heads, stream);
 }
 
@@ -677,5 +745,5 @@ TFB_API int tfb_moe_gemm_f32(const float* A, long long lda, const float* B, long
                              const int* expert_of_tile, int experts, int M, int N, int K, void* stream) {
   using namespace tfb;
   if (!expert_of_tile || experts <= 0) return TFB_ERR_ARG;
-  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, 0, 0, 0, stride, 0, nullptr, 0, expert_of_tile, experts}, 1, stream);
+  return launch_gemm_f32(GemmF32{A, B, C, lda, ldb, ldc, M, N, K, 0, 0, 0, stride, 0, nullptr, 0, expert_of_tile, experts, nullptr}, 1, stream);
 }

@@ -106,6 +106,22 @@ __device__ __forceinline__ float block_add(float v, float* red) {
 
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.f + expf(-x)); }
 __device__ __forceinline__ float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
+// 0.5 z (1 + tanh(u)) = z sigmoid(2 u), u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh_exact(float z) {
+  const float u = 0.7978845608028654f * fmaf(0.044715f * z * z, z, z);
+  return z / (1.f + expf(-2.f * u));
+}
+
+// gated feed-forwards: silu(g) u, gelu(g) u (tanh form), or, with g = min(g, limit) and u clamped to +-limit, g sigmoid(1.702 g) (u + 1)
+enum { GLU_SILU = 0, GLU_GELU = 1, GLU_CLAMPED = 2 };
+template <int ACT>
+__device__ __forceinline__ float glu_value(float g, float u, float limit) {
+  if constexpr (ACT == GLU_CLAMPED) {
+    g = fminf(g, limit);
+    return g / (1.f + expf(-1.702f * g)) * (fminf(fmaxf(u, -limit), limit) + 1.f);
+  }
+  return (ACT == GLU_GELU ? gelu_tanh_exact(g) : silu_exact(g)) * u;
+}
 
 // pairs of fp32 in one register pair: one instruction, two IEEE operations
 typedef unsigned long long u64;

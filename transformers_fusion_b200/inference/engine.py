@@ -393,11 +393,11 @@ class InferenceEngine:
                           torch.tensor([max(p, 0) for p in reqs[0].pages], dtype=torch.int32, device=dev) if pos0 else None)
         return self.model.run(batch, self.cache, self.max_len, rows, self._stack_lin)
 
-    def _stack_lin(self, x, li, name, w, act=None):
+    def _stack_lin(self, x, li, name, w, act=None, bias=None):
         pw = self.packed.get(f"layers.{li}.{name}")
         if pw is None:
-            return self.model.linear(x, w.data, act=act)
-        y = self._wq.gemm_wq(x.contiguous(), pw, None)
+            return self.model.linear(x, w.data, act=act, bias=bias)
+        y = self._wq.gemm_wq(x.contiguous(), pw, bias)
         return y if act is None else self.model.activation(y, act)
 
     def _layers_prefill_batch(self, reqs: List[Request]):

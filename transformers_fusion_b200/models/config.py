@@ -166,6 +166,11 @@ class RotarySpec:
     linear: float = 1.0
 
 
+def first_key(pos: int, window: int = 0, chunk: int = 0) -> int:
+    """The first position that a query at ``pos`` looks at: of its window, or of its chunk of positions, or 0."""
+    return max(0, pos - window + 1) if window else pos // chunk * chunk if chunk else 0
+
+
 @dataclass(frozen=True)
 class DiffAttentionSpec:
     """Differential attention: per head two query / key maps of ``dim`` entries over one set of values of ``vdim`` entries.
@@ -225,7 +230,9 @@ class HeadAttentionSpec:
     no positions); ``qk_norm``: RMS norm of every query and key head in front of it; ``gate``: one output gate per entry of the
     heads; ``window`` > 0: a position sees that many keys up to itself, and the first ``keep_first`` of the sequence; ``softcap``
     > 0: scores are cap tanh(score / cap); ``sink``: the denominator counts one more key of score 0; queries at position p are
-    multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)."""
+    multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1).  ``chunk`` > 0 (instead of a window): a position sees its own chunk of
+    so many positions; ``bias``: on the projections of q, k and v; ``qk_weight``: the norms have a learnt weight; ``head_temp``: a learnt
+    factor of the scores per head (with ``qk_norm``); ``head_sink``: a learnt score of the sink per head."""
     heads: int
     kv_heads: int
     dim: int
@@ -240,8 +247,18 @@ class HeadAttentionSpec:
     sink: bool = False
     temp_coef: float = 0.0
     temp_every: int = 1
+    chunk: int = 0
+    bias: bool = False
+    qk_weight: bool = True
+    head_temp: bool = False
+    head_sink: bool = False
 
     kind = "head_attention"
+
+    def params(self, hidden: int) -> int:
+        q, kv, o = self.heads * self.dim, self.kv_heads * (self.dim + self.vdim), self.heads * self.vdim
+        return hidden * (q + kv + o * (2 if self.gate else 1)) + (q + kv if self.bias else 0) + \
+            (2 * self.dim if self.qk_norm and self.qk_weight else 0) + self.heads * (int(self.head_temp) + int(self.head_sink))
 
 
 @dataclass(frozen=True)
@@ -258,11 +275,59 @@ class GatedLinearSpec:
 
 
 @dataclass(frozen=True)
+class ForgetLinearSpec:
+    """Linear attention whose forget gate also decides what is written (HGRN2): per head a [dim, vdim] state whose rows keep a share of
+    themselves, at least a lower bound per channel, and take the rest from the values."""
+    heads: int
+    dim: int
+    vdim: int
+
+    kind = "hgrn2"
+
+    def params(self, hidden: int) -> int:
+        return hidden * self.heads * 2 * (self.dim + self.vdim) + 2 * self.heads * self.dim + self.vdim
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """Retention: linear attention with one fixed decay per head, rotated queries and keys, and a gate per entry of the heads."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+    rot: RotarySpec = None
+
+    kind = "retention"
+
+    def params(self, hidden: int) -> int:
+        return hidden * self.heads * (2 * self.dim + 3 * self.vdim)
+
+
+@dataclass(frozen=True)
+class PairSpec:
+    """Two mixers side by side on the same input; the result is half the sum of their outputs, each normed."""
+    left: object
+    right: object
+
+    kind = "pair"
+
+    def params(self, hidden: int) -> int:
+        return self.left.params(hidden) + self.right.params(hidden) + 2 * hidden
+
+
+def mixers_of(m):
+    """The mixers that a layer's mixer consists of."""
+    return (m.left, m.right) if m.kind == "pair" else (m,)
+
+
+@dataclass(frozen=True)
 class MixtureSpec:
     """Mixture of gated feed-forward experts: ``top`` of ``experts`` per token; ``shared_ff`` > 0: one more expert of that size that
     every token runs (``shared_gate``: times the sigmoid of a logit per token).  ``score`` "softmax": the largest logits (plus a
     bias), weighted by the softmax over the chosen ones.  "sigmoid": the largest sigmoids (no bias) among the experts of the ``keep``
-    best of ``groups`` equal groups (by the sum of a group's two largest), weighted by them over their sum, times ``scale``."""
+    best of ``groups`` equal groups (by the sum of a group's two largest), weighted by them over their sum, times ``scale``.
+    "softmax_all": the largest of the softmax over all experts (no bias), weighted by themselves.  ``act``: the gated unit (``stack.glu``),
+    with its ``limit`` and that of the shared expert."""
     experts: int
     top: int
     ff: int
@@ -272,6 +337,9 @@ class MixtureSpec:
     groups: int = 1
     keep: int = 1
     scale: float = 1.0
+    act: str = "silu"
+    limit: float = 0.0
+    shared_limit: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -611,6 +679,119 @@ class FigudraConfig:
         return self._count(True)
 
 
+@dataclass
+class ToderaxConfig:
+    """Toderax: HGRN2, or chunked softmax attention (no positions, normed queries and keys, learnt sinks and temperatures) and retention side
+    by side, in any order, each with a mixture of clamped experts or none, norms in groups, and a residual of several hyper-connected
+    streams; a scaled embedding and a separate head.  ``from_dict`` reads the model folder's config.json; ``max_seq_len`` as in
+    ``LanedraConfig``."""
+    vocab_size: int
+    hidden_size: int
+    layers: list
+    norm_eps: float
+    norm_groups: int = 1
+    streams: int = 1
+    embedding_scale: float = 1.0
+    max_seq_len: int = 32768
+
+    architecture = "Toderax"
+    tie_embeddings = False
+
+    def __post_init__(self):
+        if self.norm_groups < 1 or self.hidden_size % self.norm_groups:
+            raise ValueError(f"a width of {self.hidden_size} does not divide into {self.norm_groups} groups")
+        if not 1 <= self.streams <= 16:
+            raise ValueError(f"{self.streams} streams are not in 1 .. 16")
+        for i, l in enumerate(self.layers):
+            x = l.mixture
+            for m in mixers_of(l.mixer):
+                if m.kind == "head_attention":
+                    if m.heads % m.kv_heads:
+                        raise ValueError(f"layer {i}: {m.heads} heads do not divide over {m.kv_heads} kv heads")
+                    if m.chunk < 1:
+                        raise ValueError(f"layer {i}: a chunk of {m.chunk} positions")
+                elif not 1 <= m.dim <= 512:
+                    raise ValueError(f"layer {i}: key channels per head {m.dim} are not in 1 .. 512")
+                if m.kind == "retention":
+                    if len(m.decay) != m.heads:
+                        raise ValueError(f"layer {i}: {len(m.decay)} decays for {m.heads} heads")
+                    if m.rot.dims % 2 or not 0 <= m.rot.dims <= m.dim:
+                        raise ValueError(f"layer {i}: cannot rotate {m.rot.dims} of {m.dim} entries")
+            if x is not None and not 1 <= x.top <= x.experts:
+                raise ValueError(f"layer {i}: cannot choose {x.top} of {x.experts} experts")
+
+    @property
+    def num_layers(self) -> int:
+        return len(self.layers)
+
+    @property
+    def window(self) -> int:
+        """Positions that any attention layer may still look at, the current one included; 0: there is no such layer."""
+        return max((m.chunk for l in self.layers for m in mixers_of(l.mixer) if m.kind == "head_attention"), default=0)
+
+    @classmethod
+    def from_dict(cls, d: dict, **extra) -> "ToderaxConfig":
+        layers = []
+        for i, e in enumerate(d["layers"]):
+            m, f = e["mixer"], e.get("mlp")
+            if e["type"] == "hgrn2":
+                mix = ForgetLinearSpec(m["heads"], m["dim"], m["vdim"])
+            elif e["type"] == "parallel":
+                a, b = m["left"], m["right"]
+                r = b["rot"]
+                mix = PairSpec(HeadAttentionSpec(a["heads"], a["kv_heads"], a["dim"], a["vdim"], float(a["scale"]), qk_norm=True, chunk=a["mask"]["size"],
+                                                 bias=True, qk_weight=False, head_temp=True, head_sink=True),
+                               RetentionSpec(b["heads"], b["dim"], b["vdim"], tuple(float(x) for x in b["decay"]),
+                                             RotarySpec(int(r["dims"]), float(r["base"]))))
+            else:
+                raise ValueError(f"layer {i}: unknown mixer '{e['type']}'")
+            if f is not None and f.get("kind", "moe") != "moe":
+                raise ValueError(f"layer {i}: unknown feed-forward '{f['kind']}'")
+            mixture = None
+            if f is not None:
+                r, x, sh = f["router"], f["expert"], f.get("shared")
+                mixture = MixtureSpec(r["experts"], r["top"], x["ff"], sh["ff"] if sh else 0, score="softmax_all", act="clamped", limit=float(x["limit"]),
+                                      shared_limit=float(sh["limit"]) if sh else 0.0)
+            layers.append(StackLayer(mix, 0, mixture))
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], layers=layers, norm_eps=float(d["norm"]["eps"]), norm_groups=int(d["norm"]["groups"]),
+                   streams=int(d["streams"]), embedding_scale=float(d["embedding"]["scale"]), **extra)
+
+    def to_dict(self) -> dict:
+        """The config.json form."""
+        out = []
+        for l in self.layers:
+            m, x, f = l.mixer, l.mixture, None
+            if m.kind == "pair":
+                a, b = m.left, m.right
+                mix = {"left": {"heads": a.heads, "kv_heads": a.kv_heads, "dim": a.dim, "vdim": a.vdim, "scale": a.scale, "mask": {"size": a.chunk}},
+                       "right": {"heads": b.heads, "dim": b.dim, "vdim": b.vdim, "decay": list(b.decay), "rot": {"dims": b.rot.dims, "base": b.rot.base}}}
+            else:
+                mix = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim}
+            if x is not None:
+                f = {"kind": "moe", "expert": {"ff": x.ff, "limit": x.limit}, "router": {"experts": x.experts, "top": x.top}}
+                if x.shared_ff:
+                    f["shared"] = {"ff": x.shared_ff, "limit": x.shared_limit}
+            out.append({"type": "parallel" if m.kind == "pair" else m.kind, "mixer": mix, "mlp": f})
+        return {"architecture": self.architecture, "embedding": {"scale": self.embedding_scale}, "layers": out,
+                "norm": {"eps": self.norm_eps, "groups": self.norm_groups}, "streams": self.streams, "vocab": self.vocab_size, "width": self.hidden_size}
+
+    def _count(self, active: bool) -> int:
+        H, s, n = self.hidden_size, self.streams, 2 * self.vocab_size * self.hidden_size + self.hidden_size
+        for l in self.layers:
+            x, around = l.mixture, H + 2 * s + s * s
+            n += l.mixer.params(H) + around
+            if x is not None:
+                n += 3 * H * (x.ff * (x.top if active else x.experts) + x.shared_ff) + H * x.experts + around
+        return n
+
+    def num_params(self) -> int:
+        return self._count(False)
+
+    def active_params(self) -> int:
+        """Parameters that take part in one token's pass."""
+        return self._count(True)
+
+
 # Named shapes used by the benchmarks and tests (BASELINE configs).
 def preset(name: str) -> TransformerConfig:
     name = name.lower()
@@ -658,6 +839,16 @@ def preset(name: str) -> TransformerConfig:
                   HeadAttentionSpec(heads, kv, 128, 128, 128 ** -0.5, RotarySpec(64, 500000.0, linear=4.0), True, window=win, keep_first=16, sink=True),
                   GatedLinearSpec(heads, 128, 128, 16.0))
         return FigudraConfig(V, H, [StackLayer(mixers[i % 3], 0 if i else ff, mix if i else None) for i in range(n)], 1e-5)
+    if name in ("toderax-7b", "toderax-8x7b"):
+        # beside figudra-7b and figudra-8x7b: the same width, heads, feed-forward work per token and one shared expert; two layers in three
+        # with attention and retention side by side (each with half of the heads), one with HGRN2; two streams
+        H, heads, kv, n, V, chunk, mix = (2048, 16, 4, 24, 32000, 2048, MixtureSpec(62, 6, 704, 1408, False, "softmax_all", act="clamped", limit=7.0, shared_limit=7.0)) \
+            if name == "toderax-7b" else (4096, 32, 8, 32, 32000, 8192, MixtureSpec(7, 1, 14336, 14336, False, "softmax_all", act="clamped", limit=7.0, shared_limit=7.0))
+        h = heads // 2
+        pair = PairSpec(HeadAttentionSpec(h, kv // 2, 128, 128, 128 ** 0.5, qk_norm=True, chunk=chunk, bias=True, qk_weight=False, head_temp=True, head_sink=True),
+                        RetentionSpec(h, 128, 128, tuple(1 - 2.0 ** (-5 - 5.0 * i / h) for i in range(h)), RotarySpec(128, 10000.0)))
+        mixers = (pair, pair, ForgetLinearSpec(heads, 128, 128))
+        return ToderaxConfig(V, H, [StackLayer(mixers[i % 3], 0, mix) for i in range(n)], 1e-5, 4, 2)
     if name == "mixture-7b":
         return MoEConfig(vocab_size=32000, hidden_size=2048, num_layers=24, num_heads=16, num_kv_heads=4, ffn_hidden_size=704, rope_theta=500000.0,
                          max_seq_len=32768, activation="swiglu", num_experts=64, top_k=8)

@@ -17,6 +17,7 @@ ARCHITECTURES: Dict[str, Tuple[str, str]] = {
     "Lanedra": ("lanedra", "LanedraModel"),
     "Tekenex": ("tekenex", "TekenexModel"),
     "Figudra": ("figudra", "FigudraModel"),
+    "Toderax": ("toderax", "ToderaxModel"),
 }
 
 

@@ -1,7 +1,7 @@
 """Decoders built from a list of layers with different sequence mixers: the mixers and the feed-forwards as parameter modules
 with one forward pass each over a batch description (``StepBatch``), and the model that runs them over a 32-bit residual
-stream.  Where the norms stand is the layer class's business: before and after every sublayer (``SandwichLayer``) or on its output
-only (``OutputNormLayer``).
+stream, or over several (``StreamResidual``).  Where the norms stand is the layer class's business: before and after every sublayer
+(``SandwichLayer``), on its output only (``OutputNormLayer``), before it (``StreamLayer``).
 
 The engine drives the same passes for prompts, for portions of prompts and for decoding; what is remembered between steps
 lives in ``inference.mixer_cache``.  A pass of one layer is, for a prompt or a decode step alike:
@@ -14,11 +14,14 @@ lives in ``inference.mixer_cache``.  A pass of one layer is, for a prompt or a d
                           head by head with the gates, GEMM
   delta       GEMM [q | k | v | gate | b | a], convolution + unit lengths + gates, recurrence (+ gated norm), GEMM
   gla         GEMM [q | k | v | gate | a1], decays + products of four tokens, recurrence, gated norm (decoding: one kernel), GEMM
+  hgrn2       GEMM [q | f | v], forget gates + products of four tokens, recurrence, norm (decoding: one kernel), GEMM
+  pair        GEMM [left | right], then on its columns the steps of head_attention and of
+                retention  rotation + products of four tokens, recurrence, gated norm (decoding: one kernel), GEMM
   MLP         GEMM [gate | up], act(gate) * up, GEMM;  or GEMM with the squared relu in its epilogue, GEMM
   mixture     router GEMM (fp32 logits), top-k + expert segments, rows by expert, grouped GEMM, silu(gate) * up, grouped GEMM,
               weighted sum + (gated) shared expert
-  between     norm and scale of the sublayer's output (or the sum of two), residual add and norm of (or rounding for) the next
-              sublayer, one kernel
+  between     norm and scale of the sublayer's output (or the sum of two), residual add (or the mixing of the streams) and norm of (or
+              rounding for) the next sublayer, one kernel
 
 bf16 parameters: bf16 activations and tensor-core products; fp32 parameters: everything in true fp32."""
 from __future__ import annotations
@@ -111,7 +114,7 @@ class DiffAttention(Sublayer):
             self.finalize()
         qkv = lin(h, self.source, "qkv", self.qkv)
         pool = self.index if self.nk else s.kv_from
-        K.rope_append(qkv, rope, b.positions, self.nq, self.nk, s.dim, s.rot.dims, self.v_cols, b.slots if self.nk else None,
+        K.rope_append(qkv, rope(s.rot), b.positions, self.nq, self.nk, s.dim, s.rot.dims, self.v_cols, b.slots if self.nk else None,
                       cache.k[pool] if self.nk else None, cache.v[pool] if self.nk else None)
         q = qkv[:, :self.nq * s.dim]
         args = (s.heads, s.kv_heads, s.dim, s.vdim, s.window, s.scale, self._lambda, 1.0 - s.diff, self.eps)
@@ -132,37 +135,50 @@ class DiffAttention(Sublayer):
 
 
 class HeadAttention(Sublayer):
-    """Softmax attention with the options of its spec (see ``HeadAttentionSpec``)."""
+    """Softmax attention with the options of its spec (see ``HeadAttentionSpec``).  ``proj``, ``proj_bias``: rows of another module's
+    projection and bias that are this one's (``mix`` then gets its columns of the product)."""
     linear_names = ("proj", "o")
 
-    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype, proj=None, proj_bias=None):
         super().__init__(index)
         self.spec, self.eps = spec, eps
         kw = dict(device=device, dtype=dtype)
         self.nq, self.nk, self.nv, self.no = spec.heads * spec.dim, spec.kv_heads * spec.dim, spec.kv_heads * spec.vdim, spec.heads * spec.vdim
-        self.proj = _param(self.nq + self.nk + self.nv + (self.no if spec.gate else 0), hidden, **kw)
+        n = self.columns(spec)
+        self.proj = _param(n, hidden, **kw) if proj is None else proj
+        self.proj_bias = proj_bias if proj is not None else _param(n, **kw) if spec.bias else None
         self.o = _param(hidden, self.no, **kw)
-        if spec.qk_norm:
+        if spec.qk_norm and spec.qk_weight:
             self.q_norm, self.k_norm = _param(spec.dim, **kw), _param(spec.dim, **kw)
-        self.options = K.HeadOptions(spec.window, spec.keep_first, spec.softcap, spec.sink, spec.temp_coef, spec.temp_every)
+        self.temp = _param(spec.heads, **kw) if spec.head_temp else None
+        self.sink = _param(spec.heads, **kw) if spec.head_sink else None
+        self.options = K.HeadOptions(spec.window, spec.keep_first, spec.softcap, spec.sink, spec.temp_coef, spec.temp_every, spec.chunk)
+
+    @staticmethod
+    def columns(spec) -> int:
+        return spec.heads * spec.dim + spec.kv_heads * (spec.dim + spec.vdim) + (spec.heads * spec.vdim if spec.gate else 0)
 
     def tensors(self):
         a, b, c = self.nq, self.nq + self.nk, self.nq + self.nk + self.nv
-        yield "q", self.proj.data[:a]
-        yield "k", self.proj.data[a:b]
-        yield "v", self.proj.data[b:c]
+        for n, lo, hi in (("q", 0, a), ("k", a, b), ("v", b, c)):
+            yield n, self.proj.data[lo:hi]
+            if self.spec.bias:
+                yield n + ".b", self.proj_bias.data[lo:hi]
         if self.spec.gate:
             yield "g", self.proj.data[c:]
-        if self.spec.qk_norm:
+        if self.spec.qk_norm and self.spec.qk_weight:
             yield "q.norm", self.q_norm.data
             yield "k.norm", self.k_norm.data
+        for n in ("temp", "sink"):
+            if getattr(self, n) is not None:
+                yield n, getattr(self, n).data
         yield "o", self.o.data
 
     def _past(self, cache, b):
-        """Keys and values that the portion from b.pos0 on looks at: the kept first tokens and the window of its first query, or
+        """Keys and values that the portion from b.pos0 on looks at: the kept first tokens and the window (or chunk) of its first query, or
         the whole sequence, this portion's included."""
         s, n = self.spec, b.pos0 + b.S
-        lo = max(0, b.pos0 - s.window + 1) if s.window else 0
+        lo = 0 if s.chunk and s.keep_first else self.options.first_key(b.pos0)
         kept = min(s.keep_first, lo)
         out = []
         for pool in (cache.k[self.index], cache.v[self.index]):
@@ -170,20 +186,23 @@ class HeadAttention(Sublayer):
             out.append(torch.cat([K.gather_rows(pool, b.pages, 0, kept), t]) if kept else t)
         return out[0], out[1], kept + n - lo
 
-    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+    def mix(self, p, b: StepBatch, cache, rope):
+        """The heads' outputs, of the projected rows p."""
         s, i = self.spec, self.index
-        p = lin(h, self.source, "proj", self.proj)
-        K.rope_append(p, rope, b.positions, s.heads, s.kv_heads, s.dim, s.rot.dims if s.rot else 0, self.nv, b.slots, cache.k[i], cache.v[i],
-                      (self.q_norm.data, self.k_norm.data, self.eps) if s.qk_norm else None)
+        norms = ((self.q_norm.data, self.k_norm.data) if s.qk_weight else (None, None)) + (self.eps,) if s.qk_norm else None
+        K.rope_append(p, rope(s.rot), b.positions, s.heads, s.kv_heads, s.dim, s.rot.dims if s.rot else 0, self.nv, b.slots, cache.k[i], cache.v[i],
+                      norms, self.temp.data if self.temp is not None else None)
         c = self.nq + self.nk
-        q, gate = p[:, :self.nq], p[:, c + self.nv:] if s.gate else None
-        sizes = (s.heads, s.kv_heads, s.dim, s.vdim, s.scale, gate, self.options)
+        q, gate = p[:, :self.nq], p[:, c + self.nv:c + self.nv + self.no] if s.gate else None
+        sizes, sinks = (s.heads, s.kv_heads, s.dim, s.vdim, s.scale, gate, self.options), self.sink.data if self.sink is not None else None
         if b.decode:
-            o = K.head_decode(q, cache.k[i], cache.v[i], b.block_table, b.positions, *sizes)
-        else:
-            k, v, n = self._past(cache, b) if b.pos0 else (p[:, self.nq:c], p[:, c:c + self.nv], b.S)
-            o = K.head_attn(q, k, v, b.B, b.S, n, *sizes, b.pos0)
-        return lin(o, self.source, "o", self.o)
+            return K.head_decode(q, cache.k[i], cache.v[i], b.block_table, b.positions, *sizes, sinks=sinks)
+        k, v, n = self._past(cache, b) if b.pos0 else (p[:, self.nq:c], p[:, c:c + self.nv], b.S)
+        return K.head_attn(q, k, v, b.B, b.S, n, *sizes, b.pos0, sinks)
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        bias = {"bias": self.proj_bias.data} if self.proj_bias is not None else {}
+        return lin(self.mix(lin(h, self.source, "proj", self.proj, **bias), b, cache, rope), self.source, "o", self.o)
 
 
 class GatedDelta(Sublayer):
@@ -262,6 +281,121 @@ class GatedLinear(Sublayer):
         return lin(o, self.source, "o", self.o)
 
 
+class ForgetLinear(Sublayer):
+    """Linear attention whose forget gate also decides what is written (HGRN2), with a norm of the heads behind."""
+    linear_names = ("proj", "o")
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+        super().__init__(index)
+        self.spec, self.eps = spec, eps
+        kw = dict(device=device, dtype=dtype)
+        self.hd, self.hv = spec.heads * spec.dim, spec.heads * spec.vdim
+        self.proj = _param(2 * self.hd + self.hv, hidden, **kw)
+        self.f_b, self.lower, self.norm = _param(self.hd, **kw), _param(self.hd, **kw), _param(spec.vdim, **kw)
+        self.o = _param(hidden, self.hv, **kw)
+
+    def tensors(self):
+        yield "q", self.proj.data[:self.hd]
+        yield "f", self.proj.data[self.hd:2 * self.hd]
+        yield "f.b", self.f_b.data
+        yield "lower", self.lower.data
+        yield "v", self.proj.data[2 * self.hd:]
+        yield "norm", self.norm.data
+        yield "o", self.o.data
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        s, state = self.spec, cache.state[self.index]
+        p = lin(h, self.source, "proj", self.proj)
+        gates, sizes = (self.f_b.data, self.lower.data), (s.heads, s.dim, s.vdim)
+        if b.decode:
+            o = K.forget_step(p, *gates, state, b.state_slots, self.norm.data, self.eps, b.B, *sizes)
+        else:
+            r = K.forget_prep(p, *gates, b.lens, b.B, b.S, *sizes)
+            o = K.gated_norm(K.gla_scan(r, state, b.state_slots, b.lens, b.B, b.S, *sizes, b.pos0 > 0), None, self.norm.data, self.eps, p.dtype)
+        return lin(o, self.source, "o", self.o)
+
+
+class Retention(Sublayer):
+    """Retention: a fixed decay per head, rotated queries and keys, a norm of the heads without a weight, a gate.  ``proj``: as in
+    ``HeadAttention``."""
+    linear_names = ("proj", "o")
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype, proj=None, proj_bias=None):
+        super().__init__(index)
+        self.spec, self.eps = spec, eps
+        self.hd, self.hv = spec.heads * spec.dim, spec.heads * spec.vdim
+        self.proj = _param(self.columns(spec), hidden, device=device, dtype=dtype) if proj is None else proj
+        self.o = _param(hidden, self.hv, device=device, dtype=dtype)
+        self.decay = torch.tensor(spec.decay, dtype=torch.float32, device=device)
+
+    @staticmethod
+    def columns(spec) -> int:
+        return 2 * spec.heads * (spec.dim + spec.vdim)
+
+    def tensors(self):
+        at = 0
+        for n, width in (("q", self.hd), ("k", self.hd), ("v", self.hv), ("g", self.hv)):
+            yield n, self.proj.data[at:at + width]
+            at += width
+        yield "o", self.o.data
+
+    def mix(self, p, b: StepBatch, cache, rope):
+        s, state = self.spec, cache.state[self.index]
+        turn, sizes = (self.decay, rope(s.rot), s.rot.dims if s.rot else 0, b.positions), (s.heads, s.dim, s.vdim)
+        if b.decode:
+            return K.retention_step(p, *turn, state, b.state_slots, None, self.eps, b.B, *sizes)
+        r = K.retention_prep(p, *turn, b.lens, b.B, b.S, *sizes)
+        o = K.gla_scan(r, state, b.state_slots, b.lens, b.B, b.S, *sizes, b.pos0 > 0)
+        return K.gated_norm(o, p[:, 2 * self.hd + self.hv:2 * (self.hd + self.hv)], None, self.eps)
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        return lin(self.mix(lin(h, self.source, "proj", self.proj), b, cache, rope), self.source, "o", self.o)
+
+
+class MixerPair(Sublayer):
+    """Two mixers on the same input, with one product for the projections of both; returns their two outputs (the layer norms and adds
+    them, with the weights ``left_out`` and ``right_out``)."""
+    linear_names = ("proj", "left_o", "right_o")
+
+    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+        super().__init__(index)
+        self.spec = spec
+        kw = dict(device=device, dtype=dtype)
+        kinds = [MIXERS[m.kind] for m in (spec.left, spec.right)]
+        self.cut = kinds[0].columns(spec.left)
+        n = self.cut + kinds[1].columns(spec.right)
+        self.proj = _param(n, hidden, **kw)
+        self.proj_bias = _param(n, **kw) if any(getattr(m, "bias", False) for m in (spec.left, spec.right)) else None     # zeros where one has none
+        part = lambda t, s: None if t is None else t.data[s]
+        self.left, self.right = (c(m, hidden, eps, index, device, dtype, self.proj.data[s], part(self.proj_bias, s))
+                                 for c, m, s in zip(kinds, (spec.left, spec.right), (slice(None, self.cut), slice(self.cut, None))))
+        self.left_out, self.right_out = _param(hidden, **kw), _param(hidden, **kw)
+
+    left_o = property(lambda self: self.left.o)
+    right_o = property(lambda self: self.right.o)
+
+    def finalize(self):
+        self.left.finalize()
+        self.right.finalize()
+
+    def at(self, index: int):
+        m = super().at(index)
+        m._modules = dict(self._modules, left=self.left.at(index), right=self.right.at(index))
+        return m
+
+    def tensors(self):
+        for side in ("left", "right"):
+            for n, t in getattr(self, side).tensors():
+                yield f"{side}.{n}", t
+        yield "left.out", self.left_out.data
+        yield "right.out", self.right_out.data
+
+    def forward(self, h, b: StepBatch, cache, rope, lin, kv):
+        p = lin(h, self.source, "proj", self.proj, **({"bias": self.proj_bias.data} if self.proj_bias is not None else {}))
+        left = lin(self.left.mix(p[:, :self.cut], b, cache, rope), self.source, "left_o", self.left_o)
+        return left, lin(self.right.mix(p[:, self.cut:], b, cache, rope), self.source, "right_o", self.right_o)
+
+
 class LatentAttention(Sublayer):
     """Attention without positions over one cached latent per token, with an output gate per head."""
     linear_names = ("proj", "o")
@@ -308,11 +442,13 @@ class LatentAttention(Sublayer):
 
 class GatedMLP(Sublayer):
     linear_names = ("gate_up", "down")
-    act = "silu"
+    act, limit = "silu", 0.0
 
-    def __init__(self, hidden: int, ff: int, index: int, device, dtype):
+    def __init__(self, hidden: int, ff: int, index: int, device, dtype, act=None, limit: float = 0.0):
         super().__init__(index)
         self.ff = ff
+        if act:
+            self.act, self.limit = act, limit
         self.gate_up = _param(2 * ff, hidden, device=device, dtype=dtype)
         self.down = _param(hidden, ff, device=device, dtype=dtype)
 
@@ -322,7 +458,7 @@ class GatedMLP(Sublayer):
         yield "down", self.down.data
 
     def forward(self, h, lin):
-        return lin(K.glu(lin(h, self.source, "gate_up", self.gate_up), self.act), self.source, "down", self.down)
+        return lin(K.glu(lin(h, self.source, "gate_up", self.gate_up), self.act, self.limit), self.source, "down", self.down)
 
 
 class GeluMLP(GatedMLP):
@@ -356,7 +492,7 @@ class MixtureMLP(Sublayer):
         self.router = _param(spec.experts + int(spec.shared_gate), hidden, **kw)
         self.router_bias = _param(spec.experts, **kw) if spec.score == "softmax" else None
         self.gate_up, self.down = _param(spec.experts, 2 * spec.ff, hidden, **kw), _param(spec.experts, hidden, spec.ff, **kw)
-        self.shared = GatedMLP(hidden, spec.shared_ff, index, device, dtype) if spec.shared_ff else None
+        self.shared = GatedMLP(hidden, spec.shared_ff, index, device, dtype, spec.act, spec.shared_limit) if spec.shared_ff else None
 
     def tensors(self):
         F = self.spec.ff
@@ -378,11 +514,12 @@ class MixtureMLP(Sublayer):
         z = K.linear(h, self.router.data, out_dtype=torch.float32)
         r = X.route(z[:, :E], self.router_bias.data if self.router_bias is not None else None, s.top, s.score, s.groups, s.keep, s.scale)
         g = X.expert_linear(X.expert_rows(h, r), self.gate_up.data, r)
-        y = X.expert_linear(X.expert_glu(g, r), self.down.data, r)
+        y = X.expert_linear(X.expert_glu(g, r, s.act, s.limit), self.down.data, r)
         return X.weighted_sum(y, r, self.shared(h, lin) if self.shared is not None else None, z[:, E:] if s.shared_gate else None)
 
 
-MIXERS = {"attention": DiffAttention, "delta": GatedDelta, "latent_attention": LatentAttention, "head_attention": HeadAttention, "gla": GatedLinear}
+MIXERS = {"attention": DiffAttention, "delta": GatedDelta, "latent_attention": LatentAttention, "head_attention": HeadAttention, "gla": GatedLinear,
+          "hgrn2": ForgetLinear, "retention": Retention, "pair": MixerPair}
 
 
 class ResidualLayer(nn.Module):
@@ -391,9 +528,10 @@ class ResidualLayer(nn.Module):
     norm_kind = "rms"
     dense_mlp = GatedMLP
 
-    def __init__(self, spec, hidden: int, eps: float, index: int, device, dtype):
+    def __init__(self, spec, cfg, index: int, device, dtype):
         super().__init__()
-        self.mixer = MIXERS[spec.mixer.kind](spec.mixer, hidden, eps, index, device, dtype)
+        hidden = cfg.hidden_size
+        self.mixer = MIXERS[spec.mixer.kind](spec.mixer, hidden, cfg.norm_eps, index, device, dtype)
         self.mlp = None
         if spec.mixture is not None:
             self.mlp = MixtureMLP(hidden, spec.mixture, index, device, dtype)
@@ -477,8 +615,40 @@ class ParallelLayer(ResidualLayer):
         yield (self.mixer,) if self.mlp is None else (self.mixer, self.mlp), {"w_pre": self.vector("norm1")}, {}
 
 
-def _plain_linear(x, index, name, w, act=None):
-    return K.linear(x, w.data, act=act)
+class StreamLayer(ResidualLayer):
+    """A norm in groups (norm1, norm2) in front of the mixer and the feed-forward, each between a reading (hc<q>.in) and a mixing (hc<q>.mix,
+    hc<q>.out) of the residual's streams."""
+    norm_kind = "plain"
+    final_names = ("final.norm",)
+
+    def __init__(self, spec, cfg, index: int, device, dtype):
+        super().__init__(spec, cfg, index, device, dtype)
+        self.hc = nn.ModuleList()
+        for _ in range(1 if self.mlp is None else 2):
+            m = nn.Module()
+            m.read, m.write = (_param(cfg.streams, device=device, dtype=dtype) for _ in range(2))
+            m.mix = _param(cfg.streams, cfg.streams, device=device, dtype=dtype, pitched=False)
+            self.hc.append(m)
+
+    def vector_names(self):
+        return ("norm1",) + (("norm2",) if self.mlp is not None else ())
+
+    def tensors(self):
+        yield from super().tensors()
+        for q, m in enumerate(self.hc, 1):
+            for n, t in (("in", m.read), ("out", m.write), ("mix", m.mix)):
+                yield f"hc{q}.{n}", t.data
+
+    def parts(self):
+        for q, (m, hc) in enumerate(zip((self.mixer, self.mlp), self.hc), 1):
+            post = {"mix": hc.mix.data, "out": hc.write.data}
+            if isinstance(m, MixerPair):
+                post.update(w_post=m.left_out.data, w_post2=m.right_out.data, share=0.5)
+            yield (m,), {"w_pre": self.vector(f"norm{q}"), "w_in": hc.read.data}, post
+
+
+def _plain_linear(x, index, name, w, act=None, bias=None):
+    return K.linear(x, w.data, act=act, bias=bias)
 
 
 class StackModel(nn.Module):
@@ -496,7 +666,7 @@ class StackModel(nn.Module):
         device = torch.device(device if device is not None else "cpu")
         kw = dict(device=device, dtype=dtype)
         self.tok_embeddings = _param(cfg.vocab_size, cfg.hidden_size, **kw)
-        own = {i: self.layer_cls(l, cfg.hidden_size, cfg.norm_eps, i, device, dtype) for i, l in enumerate(cfg.layers) if l.weights_of is None}
+        own = {i: self.layer_cls(l, cfg, i, device, dtype) for i, l in enumerate(cfg.layers) if l.weights_of is None}
         self.layers = nn.ModuleList([own[i] if i in own else own[l.weights_of].at(i) for i, l in enumerate(cfg.layers)])
         self.embed_norm = _param(cfg.hidden_size, **kw) if self.embed_norm_name else None
         self.norm = _param(cfg.hidden_size, **kw)
@@ -508,8 +678,8 @@ class StackModel(nn.Module):
 
     def init_weights(self, seed: int = 0):
         """Random weights that keep activations of order one: N(0, 1 / fan-in) matrices, small deviations for the norms, decays
-        between about 0.5 and 1."""
-        about_one = lambda n: n.endswith(("mix.norm", "dkv.norm")) or \
+        between about 0.5 and 1, streams that go on with a part of one another."""
+        about_one = lambda n: n.endswith(("mix.norm", "dkv.norm", ".temp", "left.out", "right.out")) or \
             (self.layer_cls.norm_kind != "rms" and n.rsplit(".", 1)[-1] in ("norm", "norm1", "norm2", "ls1", "ls2"))
         g = torch.Generator(device="cpu").manual_seed(seed)
         with torch.no_grad():
@@ -520,6 +690,10 @@ class StackModel(nn.Module):
                     r = r * 0.5 - 1.5
                 elif leaf == "conv":
                     r = r * t.shape[1] ** -0.5
+                elif ".hc" in name:
+                    r = (torch.eye(t.shape[0]) * 0.8 if leaf == "mix" else 1 / t.shape[0] if leaf == "in" else 1) + 0.2 * r
+                elif leaf == "lower":
+                    r = torch.sigmoid(r)
                 elif t.dim() == 2:
                     r = r * (1.0 if name == self.embed_name else t.shape[1] ** -0.5)
                 elif about_one(name):
@@ -579,32 +753,41 @@ class StackModel(nn.Module):
         from ..inference.mixer_cache import MixerCache
         return MixerCache(self.cfg, num_pages, num_slots, self.dtype, self.device)
 
+    def new_residual(self, n: int):
+        return torch.empty((n, self.cfg.hidden_size), dtype=torch.float32, device=self.device)
+
+    def between(self, x, **kw):
+        """What stands between two groups of sublayers (see ``parts`` of the layer classes)."""
+        return K.res_norm(x, self.cfg.norm_eps, kind=self.layer_cls.norm_kind, **kw)
+
+    def first(self, x, b, pre):
+        return self.between(x, ids=b.tokens, table=self.tok_embeddings.data, scale=self.cfg.embedding_scale,
+                            w_post=self.embed_norm.data if self.embed_norm is not None else None, **pre)
+
+    def last_norm(self):
+        return {"w_pre": self.norm.data, "b_pre": self.norm_bias.data if self.norm_bias is not None else None}
+
     def run(self, b: StepBatch, cache, max_pos: int, row_index=None, lin=_plain_linear, residuals=None):
         """One step over all layers.  Returns the final-normed rows (of ``row_index``, int32; all rows without it).
         ``residuals``: a list that receives a copy of the residual stream after every layer."""
-        cfg = self.cfg
-        eps, n, kind = cfg.norm_eps, b.tokens.shape[0], self.layer_cls.norm_kind
-        x = torch.empty((n, cfg.hidden_size), dtype=torch.float32, device=self.device)
+        x = self.new_residual(b.tokens.shape[0])
+        rope = lambda spec: self.rope(spec, max_pos) if spec is not None else None
         parts = [(i, l) + p for i, l in enumerate(self.layers) for p in l.parts()]
-        pre = [p[3] for p in parts] + [{"w_pre": self.norm.data, "b_pre": self.norm_bias.data if self.norm_bias is not None else None}]
-        h = K.res_norm(x, eps, ids=b.tokens, table=self.tok_embeddings.data, scale=cfg.embedding_scale, kind=kind,
-                       w_post=self.embed_norm.data if self.embed_norm is not None else None, **pre[0])
+        pre = [p[3] for p in parts] + [self.last_norm()]
+        h = self.first(x, b, pre[0])
         kv = {}
         for k, (i, l, group, _, post) in enumerate(parts):
-            ys = []
+            ys = ()
             for m in group:
-                if m is l.mixer:
-                    rot = getattr(m.spec, "rot", None)
-                    ys.append(m(h, b, cache, self.rope(rot, max_pos) if rot is not None else None, lin, kv))
-                else:
-                    ys.append(m(h, lin))
+                y = m(h, b, cache, rope, lin, kv) if m is l.mixer else m(h, lin)
+                ys += y if isinstance(y, tuple) else (y,)
             post = dict(post, y=ys[0], y2=ys[1] if len(ys) > 1 else None)
             last = k + 1 == len(parts)
             if residuals is not None and (last or parts[k + 1][0] != i):
                 z = x.clone()
-                K.res_norm(z, eps, kind=kind, **post)
-                residuals.append(z)
-            h = K.res_norm(x, eps, kind=kind, row_index=row_index if last else None, **post, **pre[k + 1])
+                self.between(z, **post)
+                residuals.append(z if z.dim() == 2 else z.sum(1))
+            h = self.between(x, row_index=row_index if last else None, **post, **pre[k + 1])
         return h
 
     def head(self, h):
@@ -623,3 +806,19 @@ class StackModel(nn.Module):
     @torch.no_grad()
     def forward(self, ids):
         return self.head(self.hidden_states(ids)).view(*ids.shape, -1)
+
+
+class StreamResidual:
+    """For a ``StackModel`` whose residual is ``cfg.streams`` hyper-connected streams (with ``StreamLayer``), normed in groups."""
+
+    def new_residual(self, n: int):
+        return torch.empty((n, self.cfg.streams, self.cfg.hidden_size), dtype=torch.float32, device=self.device)
+
+    def between(self, x, **kw):
+        return K.stream_norm(x, self.cfg.norm_eps, groups=self.cfg.norm_groups, **kw)
+
+    def first(self, x, b, pre):
+        return self.between(x, ids=b.tokens, table=self.tok_embeddings.data, scale=self.cfg.embedding_scale, **pre)
+
+    def last_norm(self):
+        return {"w_pre": self.norm.data}         # of the sum of the streams

@@ -71,7 +71,7 @@ def bounds_report(reset: bool = True) -> dict:
     if not bounds_check_build():
         return out
     for unit in ("elementwise", "loss_optim", "moe_routing", "gemm_bf16", "fsdp_fused", "loss_vocab_parallel", "ep_fused",
-                 "paged_attention", "stack_ops", "delta_rule", "diff_attention", "head_attention", "latent_attention", "gated_linear", "moe_serve"):
+                 "paged_attention", "stack_ops", "streams", "delta_rule", "diff_attention", "head_attention", "latent_attention", "gated_linear", "moe_serve"):
         fn = getattr(lib(), f"tfb_bounds_report_{unit}", None)
         if fn is None:
             continue

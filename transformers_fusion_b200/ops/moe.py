@@ -17,7 +17,7 @@ from dataclasses import dataclass
 
 import torch
 
-from . import _lib, functional as F
+from . import _lib, functional as F, stack as K
 from ._lib import c_f, c_i, c_ll, c_p, check, ptr, stream
 
 _lib.register("tfb_router_topk", [c_p, c_i, c_i, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_p])
@@ -33,7 +33,7 @@ _lib.register("tfb_moe_permute_bwd", [c_p, c_p, c_p, c_i, c_i, c_i, c_p])
 
 _lib.register("tfb_moe_route", [c_p, c_p, c_i, c_i, c_i, c_p, c_p, c_p, c_p, c_p, c_p, c_i, c_ll, c_i, c_i, c_i, c_i, c_f, c_p])
 _lib.register("tfb_moe_gather", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
-_lib.register("tfb_moe_glu", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_p])
+_lib.register("tfb_moe_glu", [c_p, c_ll, c_p, c_p, c_ll, c_i, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_moe_gemm_f32", [c_p, c_ll, c_p, c_ll, c_ll, c_p, c_ll, c_p, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_moe_weighted_sum", [c_p, c_ll, c_p, c_p, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 
@@ -324,10 +324,14 @@ class Routing:
     max_rows: int
 
 
+SCORE = {"softmax": 0, "sigmoid": 1, "softmax_all": 2}
+
+
 def route(logits, bias, k, score="softmax", groups=1, keep=1, scale=1.0) -> Routing:
     """The k largest of the fp32 logits [T, E] (+ bias) (the lower index first among equals), weighted by the softmax over them.
     ``score`` "sigmoid": the k largest sigmoids among the experts of the ``keep`` best of ``groups`` equal groups of neighbours (by the
-    sum of a group's two largest), weighted by them over their sum, times ``scale``."""
+    sum of a group's two largest), weighted by them over their sum, times ``scale``.  "softmax_all": the k largest entries of the softmax over
+    all experts, weighted by themselves."""
     T, E = logits.shape
     assert logits.dtype == torch.float32
     tiles = T * k // 128 + min(E, T * k)       # enough for any distribution of the assignments
@@ -344,7 +348,7 @@ def route(logits, bias, k, score="softmax", groups=1, keep=1, scale=1.0) -> Rout
             w = w / (w.sum(-1, keepdim=True) + 1e-20) * scale
         else:
             idx = torch.argsort(z, dim=-1, descending=True, stable=True)[:, :k]
-            w = torch.softmax(z.gather(1, idx), -1)
+            w = torch.softmax(z.gather(1, idx), -1) if score == "softmax" else torch.softmax(z, -1).gather(1, idx)
         row_of, of_tile, off = torch.empty(T * k, dtype=torch.int32), [], 0
         flat = idx.reshape(-1)
         for e in range(E):
@@ -360,7 +364,7 @@ def route(logits, bias, k, score="softmax", groups=1, keep=1, scale=1.0) -> Rout
     rank, counts = i32(T, k), i32(E)
     check(_lib.lib().tfb_moe_route(logits.data_ptr(), ptr(bias), T, E, k, r.idx.data_ptr(), r.w.data_ptr(), r.row_of.data_ptr(),
                                    r.expert_of_tile.data_ptr(), counts.data_ptr(), rank.data_ptr(), tiles,
-                                   logits.stride(0), int(bias is not None and bias.dtype == torch.float32), int(score == "sigmoid"), groups, keep,
+                                   logits.stride(0), int(bias is not None and bias.dtype == torch.float32), SCORE[score], groups, keep,
                                    float(scale), stream()), "moe_route", 1 if T <= 256 else 2)
     return r
 
@@ -406,15 +410,14 @@ def expert_linear(xp, w, r: Routing):
     return out
 
 
-def expert_glu(gu, r: Routing):
-    """silu(gate) * up of the assigned rows of [gate | up]."""
+def expert_glu(gu, r: Routing, act="silu", limit=0.0):
+    """act(gate) * up of the assigned rows of [gate | up]; ``act``, ``limit``: as in ``stack.glu``."""
     Fh = gu.shape[1] // 2
     if not gu.is_cuda:
-        g = gu[:, :Fh].float()
-        return (g * torch.sigmoid(g) * gu[:, Fh:].float()).to(gu.dtype)
+        return K.glu_ref(gu, act, limit)
     out = _out_rows(gu.shape[0], Fh, gu)
-    check(_lib.lib().tfb_moe_glu(gu.data_ptr(), gu.stride(0), r.row_of.data_ptr(), out.data_ptr(), out.stride(0), r.row_of.numel(), Fh, _is32(gu),
-                                 stream()), "moe_glu")
+    check(_lib.lib().tfb_moe_glu(gu.data_ptr(), gu.stride(0), r.row_of.data_ptr(), out.data_ptr(), out.stride(0), r.row_of.numel(), Fh, K.GLU[act], float(limit),
+                                 _is32(gu), stream()), "moe_glu")
     return out
 
 

@@ -1,8 +1,8 @@
 """Raw operators of decoders that are a stack of different sequence mixers over a 32-bit residual stream: norms around
-every sublayer, partial rotary embedding, differential attention, softmax attention with options, latent attention, gated delta rule, gated linear
-attention, true fp32 products.
+every sublayer, streams of residuals, partial rotary embedding, differential attention, softmax attention with options, latent attention, gated
+delta rule, linear attention with decays (gated, forget-gated, retention), true fp32 products.
 
-As in ``functional``: CUDA tensors go to the sm_100a kernels (``csrc/kernels/stack_ops.cu``, ``diff_attention.cu``, ``head_attention.cu``,
+As in ``functional``: CUDA tensors go to the sm_100a kernels (``csrc/kernels/stack_ops.cu``, ``streams.cu``, ``diff_attention.cu``, ``head_attention.cu``,
 ``latent_attention.cu``, ``delta_rule.cu``, ``gated_linear.cu``), CPU tensors run the plain PyTorch statement of the same math.  Activations are bf16 or fp32 (the dtype of
 the tensors decides); the residual, norms, rotation, attention scores and weights, and the recurrence are fp32 in both."""
 from __future__ import annotations
@@ -19,33 +19,40 @@ from ._lib import c_f, c_i, c_ll, c_p, check, ptr, stream
 
 UNITS = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "diff_attention", "delta_rule")    # translation units these operators need
 UNITS_LATENT = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "head_attention", "latent_attention", "moe_serve")
-UNITS_GATED = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "head_attention", "gated_linear", "delta_rule", "moe_serve")
+UNITS_GATED = ("tfb_host", "gemm_bf16", "skinny_linear", "stack_ops", "head_attention", "gated_linear", "moe_serve")
+UNITS_STREAMS = UNITS_GATED + ("streams",)
 PAGE = 16
 ACT = {None: 0, "relu2": 4}      # codes of the product epilogues (gemm_bf16.cu: apply_act)
-GLU = {"silu": 0, "gelu_tanh": 1}
+GLU = {"silu": 0, "gelu_tanh": 1, "clamped": 2}      # tfb_elem.cuh: glu_value
 NORM = {"rms": 0, "layer": 1, "plain": 2}
 
 _lib.register("tfb_res_norm", [c_p, c_p, c_ll, c_f, c_i, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_p, c_p, c_p, c_p, c_p, c_ll, c_p, c_i, c_i, c_f, c_i, c_i, c_p])
-_lib.register("tfb_glu", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_stream_norm", [c_p, c_p, c_ll, c_f, c_i, c_p, c_i, c_p, c_ll, c_p, c_ll, c_p, c_p, c_f, c_p, c_p, c_p, c_p, c_i, c_p, c_ll, c_p, c_i, c_i,
+                                  c_f, c_i, c_p])
+_lib.register("tfb_glu", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_rope_append", [c_p, c_ll, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
-_lib.register("tfb_norm_rope_append", [c_p, c_ll, c_p, c_p, c_f, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_norm_rope_append", [c_p, c_ll, c_p, c_p, c_p, c_f, c_p, c_p, c_i, c_p, c_p, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_gather_rows", [c_p, c_ll, c_p, c_i, c_i, c_i, c_p, c_i, c_i, c_p])
-_lib.register("tfb_gemm_f32", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_gemm_f32", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p, c_p])
 _lib.register("tfb_skinny_fits", [c_i, c_i, c_i])
-_lib.register("tfb_skinny_linear", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_p])
+_lib.register("tfb_skinny_linear", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_p, c_p])
 _lib.register("tfb_act_rows", [c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_latent_append", [c_p, c_ll, c_p, c_f, c_p, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_head_linear", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_skinny_linear_heads", [c_p, c_ll, c_i, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_p])
 _lib.register("tfb_gemm_f32_heads", [c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_p, c_ll, c_i, c_i, c_i, c_i, c_p])
-_lib.register("tfb_head_attn", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_f, c_i,
-                                c_f, c_i, c_i, c_i, c_p, c_p])
+_lib.register("tfb_head_attn", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_i, c_i, c_f, c_i,
+                                c_p, c_f, c_i, c_i, c_i, c_p, c_p])
 _lib.register("tfb_head_decode_plan", [c_i, c_i, c_i, c_i, c_i, c_i, c_i])
 _lib.register("tfb_head_decode", [c_p, c_ll, c_p, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_ll, c_i, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
-                                  c_i, c_i, c_f, c_i, c_f, c_i, c_i, c_p, c_p])
+                                  c_i, c_i, c_i, c_f, c_i, c_p, c_f, c_i, c_i, c_p, c_p])
 _lib.register("tfb_gla_prep", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_f, c_p] + [c_p] * 5 + [c_i] * 7 + [c_p])
 _lib.register("tfb_gla_scan", [c_p] * 7 + [c_i, c_p] + [c_i] * 6 + [c_p, c_p, c_p])
 _lib.register("tfb_gla_step", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_f, c_p, c_p, c_i, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
+_lib.register("tfb_forget_prep", [c_p, c_ll, c_p, c_p, c_p] + [c_p] * 5 + [c_i] * 7 + [c_p])
+_lib.register("tfb_forget_step", [c_p, c_ll, c_p, c_p, c_i, c_p, c_p, c_i, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
+_lib.register("tfb_retention_prep", [c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_p, c_p] + [c_p] * 5 + [c_i] * 7 + [c_p])
+_lib.register("tfb_retention_step", [c_p, c_ll, c_p, c_p, c_p, c_i, c_i, c_p, c_i, c_p, c_p, c_i, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_latent_decode_plan", [c_i, c_i, c_i, c_i, c_i])
 _lib.register("tfb_latent_decode", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_f, c_i, c_p, c_p])
 _lib.register("tfb_diff_attn_fwd", [c_p, c_ll, c_p, c_ll, c_p, c_ll, c_p, c_ll, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_i, c_f, c_f, c_f, c_f, c_i,
@@ -76,29 +83,31 @@ def padded_weight(n: int, width: int, dtype, device, lead=()) -> torch.Tensor:
 
 
 # ---------------------------------------------------------------------------------------------------- products
-def linear(x, w, out_dtype=None, act=None):
-    """act(x [M, K] @ w [N, K]^T).  bf16 operands: tensor-core product with fp32 accumulation (``out_dtype`` fp32 keeps the
+def linear(x, w, out_dtype=None, act=None, bias=None):
+    """act(x [M, K] @ w [N, K]^T + bias [N]).  bf16 operands: tensor-core product with fp32 accumulation (``out_dtype`` fp32 keeps the
     accumulator's precision), in a form of its own for few rows; fp32 operands: FFMA in true fp32.  ``act``: None or "relu2"."""
     out_dtype = out_dtype or x.dtype
     if not x.is_cuda:
-        return activation(x.float() @ w.float().t(), act).to(out_dtype)
+        y = x.float() @ w.float().t()
+        return activation(y if bias is None else y + bias.float(), act).to(out_dtype)
     M, K = x.shape
     N = w.shape[0]
     out = rows(M, N, out_dtype, x.device)
+    assert bias is None or (bias.dtype == x.dtype and bias.shape == (N,) and bias.is_contiguous())
     if x.dtype == torch.float32:
         assert w.dtype == torch.float32 and w.shape[1] == K and x.stride(1) == 1 and w.stride(1) == 1
         check(_lib.lib().tfb_gemm_f32(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, ACT[act],
-                                      stream()), "gemm_f32")
+                                      ptr(bias), stream()), "gemm_f32")
         return out
     if x.dtype == w.dtype == torch.bfloat16 and x.stride(1) == w.stride(1) == 1 and (x.stride(0) | w.stride(0)) % 8 == 0 and \
             (x.data_ptr() | w.data_ptr()) % 16 == 0 and _lib.lib().tfb_skinny_fits(M, N, K):
         check(_lib.lib().tfb_skinny_linear(x.data_ptr(), x.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), M, N, K, ACT[act],
-                                           int(out_dtype == torch.float32), 0, stream()), "skinny_linear")
+                                           int(out_dtype == torch.float32), 0, ptr(bias), stream()), "skinny_linear")
         return out
     if act is None:
-        return F.gemm(x, w, out=out)
+        return F.gemm(x, w, out=out, bias=bias)
     assert x.dtype == w.dtype == torch.bfloat16 and x.stride(1) == w.stride(1) == 1 and out_dtype == torch.bfloat16
-    check(_lib.lib().tfb_gemm_bf16(x.data_ptr(), x.stride(0), 0, w.data_ptr(), w.stride(0), 0, out.data_ptr(), out.stride(0), M, N, K, None, None, 0,
+    check(_lib.lib().tfb_gemm_bf16(x.data_ptr(), x.stride(0), 0, w.data_ptr(), w.stride(0), 0, out.data_ptr(), out.stride(0), M, N, K, ptr(bias), None, 0,
                                    1.0, ACT[act], 0, 0, _lib.status_word(x.device).data_ptr(), stream()), "gemm_bf16")
     return out
 
@@ -169,36 +178,90 @@ def res_norm(x, eps, *, y=None, y2=None, w_post=None, b_post=None, scale_post=No
     return a
 
 
+def group_rms(x, w, groups, eps):
+    """RMS norm of every one of ``groups`` equal consecutive parts of a row; the weight is the factor itself."""
+    xf = x.float().unflatten(-1, (groups, -1))
+    return (xf / torch.sqrt(xf.pow(2).mean(-1, keepdim=True) + eps)).flatten(-2) * w.float()
+
+
+def stream_norm(x, eps, *, y=None, y2=None, w_post=None, w_post2=None, share=1.0, mix=None, out=None, w_in=None, w_pre=None, groups=1, ids=None,
+                table=None, scale=1.0, row_index=None):
+    """What stands between two sublayers over a residual of several streams, fp32 ``x`` [n, S, H], in place:
+    x_t <- sum_s mix[s, t] x_s + out[t] y', with y' = share * (y + y2), each an RMS norm of itself first where it has a weight (``w_post``,
+    ``w_post2``).  Returns group_rms(sum_s w_in[s] x_s; w_pre) in the weight's dtype (``w_in`` None: the plain sum), None without
+    ``w_pre``.  ``ids``: all streams start as scale * table[ids].  ``row_index`` (int32): only those rows are computed and returned, and x
+    keeps its values."""
+    n, S, H = x.shape
+    if not x.is_cuda:
+        v = (table[ids.long()].float() * scale)[:, None].expand(-1, S, -1) if ids is not None else x
+        if y is not None:
+            z = (plain_rms(y, w_post, eps) if w_post is not None else y.float())
+            if y2 is not None:
+                z = z + (plain_rms(y2, w_post2, eps) if w_post2 is not None else y2.float())
+            v = torch.einsum("nsh,st->nth", v, mix.float()) + out.float()[:, None] * (z * share)[:, None]
+        if row_index is None:
+            x.copy_(v)
+        else:
+            v = v[row_index.long()]
+        if w_pre is None:
+            return None
+        u = v.sum(1) if w_in is None else torch.einsum("nsh,s->nh", v, w_in.float())
+        return group_rms(u, w_pre, groups, eps).to(w_pre.dtype)
+    n = n if row_index is None else row_index.shape[0]
+    dt = next(t for t in (w_pre, table, y) if t is not None).dtype
+    assert x.is_contiguous() and x.dtype == torch.float32 and dt in (torch.float32, torch.bfloat16)
+    for t in (y, y2, w_post, w_post2, mix, out, w_in, w_pre, table):
+        assert t is None or (t.dtype == dt and t.stride(-1) == 1)
+    a = rows(n, H, dt, x.device) if w_pre is not None else None
+    ld = lambda t: t.stride(0) if t is not None else 0
+    check(_lib.lib().tfb_stream_norm(ptr(ids), ptr(table), ld(table), float(scale), table.shape[0] if table is not None else 0, x.data_ptr(), S, ptr(y),
+                                     ld(y), ptr(y2), ld(y2), ptr(w_post), ptr(w_post2), float(share), ptr(mix), ptr(out), ptr(w_in), ptr(w_pre), groups,
+                                     ptr(a), ld(a), ptr(row_index), n, H, float(eps), int(dt == torch.float32), stream()), "stream_norm")
+    return a
+
+
 def glu_silu(gu):
     return glu(gu, "silu")
 
 
-def glu(gu, act):
-    """[gate | up] -> act(gate) * up; ``act``: "silu" or "gelu_tanh"."""
+def glu_ref(gu, act, limit=0.0):
+    Fh = gu.shape[1] // 2
+    g, u = gu[:, :Fh].float(), gu[:, Fh:].float()
+    if act == "clamped":
+        g = g.clamp(max=limit)
+        return (g * torch.sigmoid(1.702 * g) * (u.clamp(-limit, limit) + 1)).to(gu.dtype)
+    return ((g * torch.sigmoid(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")) * u).to(gu.dtype)
+
+
+def glu(gu, act, limit=0.0):
+    """[gate | up] -> act(gate) * up; ``act``: "silu", "gelu_tanh" or "clamped": with g = min(gate, limit) and u = up clamped to
+    +-limit, g sigmoid(1.702 g) (u + 1)."""
     M, F2 = gu.shape
     Fh = F2 // 2
     if not gu.is_cuda:
-        g = gu[:, :Fh].float()
-        g = g * torch.sigmoid(g) if act == "silu" else torch.nn.functional.gelu(g, approximate="tanh")
-        return (g * gu[:, Fh:].float()).to(gu.dtype)
+        return glu_ref(gu, act, limit)
     out = rows(M, Fh, gu.dtype, gu.device)
-    check(_lib.lib().tfb_glu(gu.data_ptr(), gu.stride(0), out.data_ptr(), out.stride(0), M, Fh, GLU[act], _f32(gu), stream()), "glu")
+    check(_lib.lib().tfb_glu(gu.data_ptr(), gu.stride(0), out.data_ptr(), out.stride(0), M, Fh, GLU[act], float(limit), _f32(gu), stream()), "glu")
     return out
 
 
 # ---------------------------------------------------------------------------------------------------- rotation + cache
-def rope_append(qkv, tables, positions, nq, nk, D, dims, v_cols, slots=None, kpool=None, vpool=None, norms=None):
+def rope_append(qkv, tables, positions, nq, nk, D, dims, v_cols, slots=None, kpool=None, vpool=None, norms=None,
+                q_factor=None):
     """Rotate the first ``dims`` entries of the nq query and nk key heads of every row of ``qkv`` ([q | k | v | ...]) in place and
     write k and v to flat slots of the pools ([slots, nk * D], [slots, v_cols]; negative slots are not cached).  ``norms``
-    (weights of the queries, of the keys, eps): every head is divided by its root mean square and weighted first.  ``dims`` 0:
-    no rotation (``tables`` None)."""
+    (weights of the queries, of the keys, eps; no weights: None, None, eps): every head is divided by its root mean square and weighted
+    first; ``q_factor`` [nq] (with ``norms`` only) multiplies the normed query heads.  ``dims`` 0: no rotation (``tables`` None)."""
+    assert q_factor is None or norms
     cos, sin = tables or (None, None)
     T = qkv.shape[0]
     if not qkv.is_cuda:
         half = dims // 2
         x = qkv[:, :(nq + nk) * D].reshape(T, nq + nk, D).float()
         if norms:
-            x = torch.cat([plain_rms(x[:, :nq], norms[0], norms[2]), plain_rms(x[:, nq:], norms[1], norms[2])], 1)
+            one = torch.ones(D)
+            q, k = (plain_rms(t, one if w is None else w, norms[2]) for t, w in ((x[:, :nq], norms[0]), (x[:, nq:], norms[1])))
+            x = torch.cat([q if q_factor is None else q * q_factor.float()[:, None], k], 1)
         if dims:
             c, s = cos[positions.long()][:, None], sin[positions.long()][:, None]
             u, v = x[..., :half], x[..., half:dims]
@@ -211,7 +274,7 @@ def rope_append(qkv, tables, positions, nq, nk, D, dims, v_cols, slots=None, kpo
             vpool[slots[keep]] = qkv[keep, (nq + nk) * D:(nq + nk) * D + v_cols]
         return qkv
     if norms:
-        check(_lib.lib().tfb_norm_rope_append(qkv.data_ptr(), qkv.stride(0), norms[0].data_ptr(), norms[1].data_ptr(), float(norms[2]), ptr(cos),
+        check(_lib.lib().tfb_norm_rope_append(qkv.data_ptr(), qkv.stride(0), ptr(norms[0]), ptr(norms[1]), ptr(q_factor), float(norms[2]), ptr(cos),
                                               ptr(sin), cos.shape[0] if dims else 0, positions.data_ptr(), ptr(slots), ptr(kpool), ptr(vpool),
                                               kpool.shape[0] if kpool is not None else 0, T, nq, nk, D, dims, v_cols, _f32(qkv), stream()),
               "norm_rope_append")
@@ -298,19 +361,29 @@ def diff_decode(q, kpool, vpool, block_table, positions, H, G, D, V, window, sca
 class HeadOptions(NamedTuple):
     """``window`` > 0: a query sees that many keys up to its own, and the first ``keep_first`` of the sequence; ``softcap`` > 0: scores
     become cap tanh(score / cap); ``sink``: one more key of score 0 in the denominator; the query at position p is multiplied by
-    1 + temp_coef ln(floor((p + 1) / temp_every) + 1)."""
+    1 + temp_coef ln(floor((p + 1) / temp_every) + 1); ``chunk`` > 0 (no window then): it sees the keys of its own chunk of so many
+    positions, counted from 0, and those first ones."""
     window: int = 0
     keep_first: int = 0
     softcap: float = 0.0
     sink: bool = False
     temp_coef: float = 0.0
     temp_every: int = 1
+    chunk: int = 0
+
+    def first_key(self, i: int) -> int:
+        """The first key that the query at position i sees, kept ones aside."""
+        return max(0, i - self.window + 1) if self.window else i // self.chunk * self.chunk if self.chunk else 0
+
+    def args(self, sinks):
+        """Of the entry points: window, chunk, keep, cap, sink, sinks, temp."""
+        return self.window, self.chunk, self.keep_first, self.softcap, 2 if sinks is not None else int(self.sink), ptr(sinks), self.temp_coef, self.temp_every
 
 
 PLAIN = HeadOptions()
 
 
-def _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None, opt=PLAIN, pos0=0):
+def _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None, opt=PLAIN, pos0=0, sinks=None):
     R = H // G
     Q = q.reshape(B, S, H, D).transpose(1, 2).float()
     K = k.reshape(B, Skv, G, D).transpose(1, 2).float().repeat_interleave(R, 1)
@@ -319,13 +392,15 @@ def _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None, opt=PLAIN, 
     hide = j > i
     if opt.window:
         hide = hide | ((i - j >= opt.window) & (j >= opt.keep_first))
+    if opt.chunk:
+        hide = hide | ((i // opt.chunk != j // opt.chunk) & (j >= opt.keep_first))
     temp = 1 + opt.temp_coef * torch.log(((torch.arange(S) + pos0 + 1) // opt.temp_every + 1).float())
     s = Q * temp[:, None] @ K.transpose(-1, -2) * scale
     if opt.softcap:
         s = opt.softcap * torch.tanh(s / opt.softcap)
     s = s.masked_fill(hide, -math.inf)
-    if opt.sink:
-        s = torch.cat([s, torch.zeros(B, H, S, 1)], -1)
+    if opt.sink or sinks is not None:
+        s = torch.cat([s, torch.zeros(B, H, S, 1) if sinks is None else sinks.float()[:, None, None].expand(B, H, S, 1)], -1)
         W = torch.cat([W, torch.zeros(B, H, 1, V)], 2)
     o = (torch.softmax(s, -1) @ W).transpose(1, 2)                                 # [B, S, H, V]
     if gate is not None:
@@ -333,40 +408,44 @@ def _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None, opt=PLAIN, 
     return o.reshape(B * S, H * V).to(q.dtype)
 
 
-def head_attn(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None, opt=PLAIN, pos0=0):
+def head_attn(q, k, v, B, S, Skv, H, G, D, V, scale, gate=None, opt=PLAIN, pos0=0, sinks=None):
     """Causal softmax attention of B prompts whose keys and values may have different sizes.  q [B*S, H D], k [B*Skv, G D],
     v [B*Skv, G V]; the queries are the last S of the Skv keys and stand at positions pos0 ... (with a window, keys between the
-    kept ones and the window of the first query may be left out); ``gate`` [B*S, H] or [B*S, H V]: heads, or their entries, are
-    multiplied by its sigmoid.  Returns [B*S, H V]."""
+    kept ones and the window of the first query may be left out; with chunks and no kept ones those of earlier chunks);
+    ``gate`` [B*S, H] or [B*S, H V]: heads, or their entries, are multiplied by its sigmoid; ``sinks`` [H]: the score of one more key per
+    head in the denominator.  Returns [B*S, H V]."""
     if not q.is_cuda:
-        return _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate, opt, pos0)
+        return _head_attn_ref(q, k, v, B, S, Skv, H, G, D, V, scale, gate, opt, pos0, sinks)
+    assert sinks is None or sinks.dtype == q.dtype
     o = rows(B * S, H * V, q.dtype, q.device)
     check(_lib.lib().tfb_head_attn(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), o.data_ptr(), o.stride(0),
                                    ptr(gate), gate.stride(0) if gate is not None else 0, int(gate is not None and gate.shape[1] != H), B, S, Skv, H,
-                                   G, D, V, float(scale), opt.window, opt.keep_first, opt.softcap, int(opt.sink), opt.temp_coef, opt.temp_every, pos0,
+                                   G, D, V, float(scale), *opt.args(sinks), pos0,
                                    _f32(q), _lib.status_word(q.device).data_ptr(), stream()), "head_attn")
     return o
 
 
-def head_decode(q, kpool, vpool, block_table, positions, H, G, D, V, scale, gate=None, opt=PLAIN, splits: Optional[int] = None):
+def head_decode(q, kpool, vpool, block_table, positions, H, G, D, V, scale, gate=None, opt=PLAIN, splits: Optional[int] = None,
+                sinks=None):
     """One query per sequence (q [B, H D] at ``positions``) over its cached rows (pools [slots, G D] and [slots, G V]); ``gate`` [B, H]
-    or [B, H V]."""
+    or [B, H V]; ``sinks`` [H]."""
     B = q.shape[0]
     if not q.is_cuda:
         out = torch.zeros((B, H * V), dtype=q.dtype)
         for b in range(B):
             n = int(positions[b]) + 1
-            lo = max(0, n - opt.window) if opt.window else 0
+            lo = opt.first_key(n - 1)
             p = torch.cat([torch.arange(min(opt.keep_first, lo)), torch.arange(lo, n)])
             s = block_table[b, (p // PAGE).long()].long() * PAGE + p % PAGE
-            out[b] = _head_attn_ref(q[b:b + 1], kpool[s], vpool[s], 1, 1, len(p), H, G, D, V, scale, gate[b:b + 1] if gate is not None else None, opt,
-                                    n - 1)[0]
+            out[b] = _head_attn_ref(q[b:b + 1], kpool[s], vpool[s], 1, 1, len(p), H, G, D, V, scale, gate[b:b + 1] if gate is not None else None,
+                                    opt._replace(window=0, chunk=0), n - 1, sinks)[0]
         return out
+    assert sinks is None or sinks.dtype == q.dtype
     L, f32 = _lib.lib(), _f32(q)
     o = rows(B, H * V, q.dtype, q.device)
     acc = ml = None
     keys = block_table.shape[1] * PAGE
-    keys = min(keys, opt.window + opt.keep_first) if opt.window else keys
+    keys = min(keys, (opt.window or opt.chunk) + opt.keep_first) if opt.window or opt.chunk else keys
     n = L.tfb_head_decode_plan(B, H, G, D, V, keys, f32)         # key splits of the tensor-core form, 0: the other form
     if n and q.stride(0) % 8 == 0:
         splits = splits or n
@@ -375,7 +454,7 @@ def head_decode(q, kpool, vpool, block_table, positions, H, G, D, V, scale, gate
     check(L.tfb_head_decode(q.data_ptr(), q.stride(0), kpool.data_ptr(), vpool.data_ptr(), kpool.shape[0], block_table.data_ptr(),
                             block_table.shape[1], PAGE, positions.data_ptr(), o.data_ptr(), o.stride(0), ptr(gate),
                             gate.stride(0) if gate is not None else 0, int(gate is not None and gate.shape[1] != H), ptr(acc), ptr(ml), splits or 1, B,
-                            H, G, D, V, float(scale), opt.window, opt.keep_first, opt.softcap, int(opt.sink), opt.temp_coef, opt.temp_every, f32,
+                            H, G, D, V, float(scale), *opt.args(sinks), f32,
                             _lib.status_word(q.device).data_ptr(), stream()), "head_decode", 2 if acc is not None else 1)
     return o
 
@@ -544,16 +623,22 @@ def delta_scan(rows_: DeltaRows, state, state_slots, lens, B, S, G, H, D, V, has
     return o
 
 
-def gated_norm(o, gate, w, eps):
-    """o [T, H, V] fp32 -> o / rms(o) * w * silu(gate), [T, H V] in the dtype of ``gate`` [T, H V]."""
+def gated_norm(o, gate, w, eps, dtype=None):
+    """o [T, H, V] fp32 -> o / rms(o) [* w [V]] [* silu(gate [T, H V])], [T, H V] in ``dtype`` (that of the gate, if there is one)."""
     T, H, V = o.shape
+    dtype = gate.dtype if gate is not None else dtype
     if not o.is_cuda:
-        g = gate.reshape(T, H, V).float()
-        y = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w.float() * (g * torch.sigmoid(g))
-        return y.reshape(T, H * V).to(gate.dtype)
-    out = rows(T, H * V, gate.dtype, o.device)
-    check(_lib.lib().tfb_gated_norm(o.data_ptr(), gate.data_ptr(), gate.stride(0), w.data_ptr(), out.data_ptr(), out.stride(0), T, H, V, float(eps),
-                                    _f32(gate), stream()), "gated_norm")
+        y = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps)
+        if w is not None:
+            y = y * w.float()
+        if gate is not None:
+            g = gate.reshape(T, H, V).float()
+            y = y * (g * torch.sigmoid(g))
+        return y.reshape(T, H * V).to(dtype)
+    out = rows(T, H * V, dtype, o.device)
+    assert w is None or w.dtype == dtype
+    check(_lib.lib().tfb_gated_norm(o.data_ptr(), ptr(gate), gate.stride(0) if gate is not None else 0, ptr(w), out.data_ptr(), out.stride(0), T, H, V,
+                                    float(eps), _f32(out), stream()), "gated_norm")
     return out
 
 
@@ -569,7 +654,7 @@ def delta_step(rows_: DeltaRows, state, state_slots, gate, w, eps, B, G, H, D, V
     return out
 
 
-# ---------------------------------------------------------------------------------------------------- gated linear attention
+# ---------------------------------------------------------------------------------------------------- linear attention with decays
 @dataclass
 class GlaRows:
     """Prepared rows of B sequences.  On CUDA the scan's own layouts (see csrc/kernels/gated_linear.cu): per four tokens queries times
@@ -582,6 +667,16 @@ class GlaRows:
     pair: Optional[torch.Tensor] = None
 
 
+def _gla_rows(B, S, H, D, V, device):
+    Dp, Vp, n4 = next((d for d in (32, 64, 128, 256, 512) if D <= d), 0), (V + 3) // 4 * 4, (S + 3) // 4
+    e = lambda *shape: torch.empty(shape, dtype=torch.float32, device=device)
+    return GlaRows(e(B, H, 4 * n4, Dp), e(B, H, 4 * n4, Dp), e(B, H, 4 * n4, Vp), e(B, H, n4, Dp), e(B, H, n4, 16)), Dp
+
+
+def _ptrs(r: GlaRows):
+    return r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.decay.data_ptr(), r.pair.data_ptr()
+
+
 def gla_prep(proj, a2, bias, tau, lens, B, S, H, D, V) -> GlaRows:
     """proj [B*S, 2 H D + 2 H V + rank] = q | k | v | gate | a1, a2 [H D, rank], bias [H D]: scaled queries, decays
     sigmoid(a2 a1 + bias)^(1/tau) and rows for ``gla_scan``, all fp32."""
@@ -591,13 +686,43 @@ def gla_prep(proj, a2, bias, tau, lens, B, S, H, D, V) -> GlaRows:
         z = x[:, 2 * n + 2 * H * V:] @ a2.float().t() + bias.float()
         return GlaRows(x[:, :n].reshape(T, H, D) * D ** -0.5, x[:, n:2 * n].reshape(T, H, D), x[:, 2 * n:2 * n + H * V].reshape(T, H, V),
                        torch.exp(torch.nn.functional.logsigmoid(z) / tau).reshape(T, H, D))
-    L = _lib.lib()
-    Dp, Vp, n4 = L.tfb_delta_padded_dim(D), (V + 3) // 4 * 4, (S + 3) // 4
-    e = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
-    r = GlaRows(e(B, H, 4 * n4, Dp), e(B, H, 4 * n4, Dp), e(B, H, 4 * n4, Vp), e(B, H, n4, Dp), e(B, H, n4, 16))
-    check(L.tfb_gla_prep(proj.data_ptr(), proj.stride(0), a2.data_ptr(), a2.stride(0), bias.data_ptr(), a2.shape[1], float(tau), ptr(lens),
-                         r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.decay.data_ptr(), r.pair.data_ptr(), B, S, H, D, Dp, V, _f32(proj),
-                         stream()), "gla_prep")
+    r, Dp = _gla_rows(B, S, H, D, V, proj.device)
+    check(_lib.lib().tfb_gla_prep(proj.data_ptr(), proj.stride(0), a2.data_ptr(), a2.stride(0), bias.data_ptr(), a2.shape[1], float(tau), ptr(lens),
+                                  *_ptrs(r), B, S, H, D, Dp, V, _f32(proj), stream()), "gla_prep")
+    return r
+
+
+def forget_prep(proj, bias, lower, lens, B, S, H, D, V) -> GlaRows:
+    """proj [B*S, 2 H D + H V ...] = q | f | v ..., bias, lower [H D]: queries silu(q), decays a = lower + (1 - lower) sigmoid(f + bias), keys
+    1 - a; rows for ``gla_scan``, all fp32."""
+    if not proj.is_cuda:
+        T, n = proj.shape[0], H * D
+        x, l = proj.float(), lower.float()
+        z = x[:, n:2 * n] + bias.float()
+        return GlaRows((x[:, :n] * torch.sigmoid(x[:, :n])).reshape(T, H, D), ((1 - l) * torch.sigmoid(-z)).reshape(T, H, D),
+                       x[:, 2 * n:2 * n + H * V].reshape(T, H, V), (l + (1 - l) * torch.sigmoid(z)).reshape(T, H, D))
+    r, Dp = _gla_rows(B, S, H, D, V, proj.device)
+    check(_lib.lib().tfb_forget_prep(proj.data_ptr(), proj.stride(0), bias.data_ptr(), lower.data_ptr(), ptr(lens), *_ptrs(r), B, S, H, D, Dp, V,
+                                     _f32(proj), stream()), "forget_prep")
+    return r
+
+
+def retention_prep(proj, decay, tables, dims, positions, lens, B, S, H, D, V) -> GlaRows:
+    """proj [B*S, 2 H D + H V ...] = q | k | v ..., decay [H] fp32: q and k rotated by their positions (first ``dims`` entries, 0: no
+    rotation), k scaled by D^(-1/2); rows for ``gla_scan``, all fp32."""
+    cos, sin = tables or (None, None)
+    if not proj.is_cuda:
+        T, n, half = proj.shape[0], H * D, dims // 2
+        x = proj.float()
+        qk = x[:, :2 * n].reshape(T, 2 * H, D)
+        if dims:
+            c, s = cos[positions.long()][:, None], sin[positions.long()][:, None]
+            u, v = qk[..., :half], qk[..., half:dims]
+            qk = torch.cat([u * c - v * s, v * c + u * s, qk[..., dims:]], -1)
+        return GlaRows(qk[:, :H], qk[:, H:] * D ** -0.5, x[:, 2 * n:2 * n + H * V].reshape(T, H, V), decay[:, None].expand(T, H, D))
+    r, Dp = _gla_rows(B, S, H, D, V, proj.device)
+    check(_lib.lib().tfb_retention_prep(proj.data_ptr(), proj.stride(0), decay.data_ptr(), ptr(cos), ptr(sin), cos.shape[0] if dims else 0, dims,
+                                        positions.data_ptr(), ptr(lens), *_ptrs(r), B, S, H, D, Dp, V, _f32(proj), stream()), "retention_prep")
     return r
 
 
@@ -624,13 +749,42 @@ def gla_scan(rows_: GlaRows, state, state_slots, lens, B, S, H, D, V, has_past):
     return o
 
 
+def _gate(proj, H, D, V):
+    return proj[:, 2 * H * D + H * V:2 * H * D + 2 * H * V]
+
+
 def gla_step(proj, a2, bias, tau, state, state_slots, w, eps, B, H, D, V):
     """One token per sequence: decays, recurrence and the gated norm of its output; [B, H V]."""
-    gate = proj[:, 2 * H * D + H * V:2 * H * D + 2 * H * V]
+    gate = _gate(proj, H, D, V)
     if not proj.is_cuda or not _step_fits(D, V):
         return gated_norm(gla_scan(gla_prep(proj, a2, bias, tau, None, B, 1, H, D, V), state, state_slots, None, B, 1, H, D, V, True), gate, w, eps)
     out = rows(B, H * V, proj.dtype, proj.device)
     check(_lib.lib().tfb_gla_step(proj.data_ptr(), proj.stride(0), a2.data_ptr(), a2.stride(0), bias.data_ptr(), a2.shape[1], float(tau),
                                   state.data_ptr(), state_slots.data_ptr(), state.shape[0], w.data_ptr(), out.data_ptr(), out.stride(0), B, H, D, V,
                                   float(eps), _f32(proj), stream()), "gla_step")
+    return out
+
+
+def forget_step(proj, bias, lower, state, state_slots, w, eps, B, H, D, V, gated=False):
+    """One token per sequence, as ``gla_step``; [B, H V].  ``gated``: v is followed by the gate."""
+    if not proj.is_cuda or not _step_fits(D, V):
+        o = gla_scan(forget_prep(proj, bias, lower, None, B, 1, H, D, V), state, state_slots, None, B, 1, H, D, V, True)
+        return gated_norm(o, _gate(proj, H, D, V) if gated else None, w, eps, proj.dtype)
+    out = rows(B, H * V, proj.dtype, proj.device)
+    check(_lib.lib().tfb_forget_step(proj.data_ptr(), proj.stride(0), bias.data_ptr(), lower.data_ptr(), int(gated), state.data_ptr(),
+                                     state_slots.data_ptr(), state.shape[0], ptr(w), out.data_ptr(), out.stride(0), B, H, D, V, float(eps), _f32(proj),
+                                     stream()), "forget_step")
+    return out
+
+
+def retention_step(proj, decay, tables, dims, positions, state, state_slots, w, eps, B, H, D, V, gated=True):
+    """One token per sequence, as ``gla_step``; [B, H V]."""
+    cos, sin = tables or (None, None)
+    if not proj.is_cuda or not _step_fits(D, V):
+        o = gla_scan(retention_prep(proj, decay, tables, dims, positions, None, B, 1, H, D, V), state, state_slots, None, B, 1, H, D, V, True)
+        return gated_norm(o, _gate(proj, H, D, V) if gated else None, w, eps, proj.dtype)
+    out = rows(B, H * V, proj.dtype, proj.device)
+    check(_lib.lib().tfb_retention_step(proj.data_ptr(), proj.stride(0), decay.data_ptr(), ptr(cos), ptr(sin), cos.shape[0] if dims else 0, dims,
+                                        positions.data_ptr(), int(gated), state.data_ptr(), state_slots.data_ptr(), state.shape[0], ptr(w),
+                                        out.data_ptr(), out.stride(0), B, H, D, V, float(eps), _f32(proj), stream()), "retention_step")
     return out
