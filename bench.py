@@ -229,13 +229,14 @@ def torch_library_arm(cfg, world, rank, dev, local_batch, seq, steps, warmup, di
 SERVING = {   # --config -> [(preset, layers), ...] (the first one's decode rate is the metric)
     "lanedra-serving": [("lanedra-1.5b", 24), ("dense-1.5b", 24), ("lanedra-8b", 8), ("llama-3-8b", 8)],
     "tekenex-serving": [("tekenex-7b", 24), ("mixture-7b", 24), ("tekenex-8x7b", 8), ("mixtral-8x7b", 8)],
+    "toderax-serving": [("toderax-7b", 24), ("figudra-7b", 24), ("toderax-8x7b", 8), ("figudra-8x7b", 8)],
     "figudra-serving": [("figudra-7b", 24), ("mixture-7b", 24), ("figudra-8x7b", 8), ("mixtral-8x7b", 8)],
 }
 
 
 def serving_config(args):
     """Prefill and decode throughput of a stack model beside the closest model of the framework at equal layer sizes (Lanedra: the dense
-    decoder; Tekenex, Figudra: the mixture-of-experts decoder), on one GPU, random-init bf16 weights and seeded token ids, through the
+    decoder; Tekenex, Figudra: the mixture-of-experts decoder; Toderax: Figudra), on one GPU, random-init bf16 weights and seeded token ids, through the
     serving engine's own passes (paged cache, state slots, decode CUDA graphs).  Two sizes: 2048 wide (24 layers) and 4096 wide
     (8 layers of the 32-layer shape).  Device-timed (CUDA events around K steps, W untimed ones first); each step reads the weights
     (larger than L2).  One JSON line; ``rows`` has every measurement."""
@@ -345,7 +346,7 @@ def main(argv=None):
                          "1/2/4/8 GPUs).  llama3-8b-fsdp-tp2: Llama-3-8B shape, ZeRO-3 over dp x tensor parallel 2, seq 4096, "
                          "one sequence per GPU (2, 4 or 8 GPUs).  gpt2-small-cpu: GPT-2-small-shaped greedy generation on the CPU "
                          "(32 prompt + 64 new tokens), the configuration the reference's own build can run as well.  lanedra-serving, "
-                         "tekenex-serving, figudra-serving: prefill and decode throughput of the stack model beside the dense / mixture-of-experts decoder of "
+                         "tekenex-serving, figudra-serving, toderax-serving: prefill and decode throughput of the stack model beside its closest relative of "
                          "equal sizes (1 GPU)")
     ap.add_argument("--capacity-factor", type=float, default=2.0,
                     help="mixtral-8x7b-ep: expert buffer rows per rank as a multiple of the balanced load")

@@ -8,7 +8,8 @@ cross_entropy, adamw, paged_decode, sampling, moe_ffn; those of stack models (``
 diff_attention_window, attention_fwd_gqa128 (the plain form of the same layer), diff_decode, delta_prep, delta_scan,
 delta_scan_one, gated_norm, delta_prep_step, delta_step, res_norm, glu_silu, rope_append; those of latent attention and the serving
 mixture with the like kernels of the mixture-of-experts decoder (``LATENT_KERNELS``); those of attention with options and gated linear
-attention (``GATED_KERNELS``).  ``--kernel`` takes names and the groups all, stack, latent, gated, with commas between them.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
+attention (``GATED_KERNELS``); those of chunked attention, HGRN2, retention and streams of residuals (``STREAM_KERNELS``).  ``--kernel`` takes names and the
+groups all, stack, latent, gated, streams, with commas between them.  ``--comm`` (multi-GPU) times the fused compute+collective kernels
 against their NCCL forms (cli/bench_comm.py)."""
 from __future__ import annotations
 
@@ -30,6 +31,8 @@ LATENT_KERNELS = ("head_attn", "attention_fwd_mha128", "latent_decode", "latent_
                   "weighted_sum", "moe_combine", "mixture", "mixture_step", "moe_ffn_step", "kv_append")
 GATED_KERNELS = ("head_attn_cap", "head_attn_window", "head_attn_gqa", "head_decode", "head_decode_cap", "head_decode_window", "gla_prep", "gla_scan",
                  "gla_scan_one", "gla_step", "norm_rope_append", "parallel_norm", "glu_gelu", "grouped_route", "grouped_route_step", "weighted_sum_gated")
+STREAM_KERNELS = ("head_attn_chunk", "head_decode_chunk", "unit_norm_append", "forget_prep", "forget_scan", "forget_step", "retention_prep", "retention_scan",
+                  "retention_step", "head_norm", "stream_norm", "stream_norm_pair", "glu_clamped", "route_all", "route_all_step", "expert_glu_clamped")
 FP32_FMA_PER_SM = 128          # fp32 FMA lanes of an SM (the scans are reported against them)
 
 
@@ -262,6 +265,75 @@ def _build_gated(kernel, n, dev):
     raise SystemExit(f"Error: unknown kernel '{kernel}'")
 
 
+def _build_streams(kernel, n, dev):
+    """The same for the layers of a model with attention in chunks of 1024 keys and retention side by side (8 heads each, 2 kv heads, 128
+    entries), HGRN2 (16 heads of 128 x 128) and two streams of residuals; like kernels: those of ``GATED_KERNELS``."""
+    import torch
+
+    from ..ops import functional as F
+    from ..ops import moe as M
+    from ..ops import stack as K
+    bf = torch.bfloat16
+    g = torch.Generator(device=dev).manual_seed(0)
+    rnd = lambda *s, dtype=bf: torch.randn(*s, device=dev, generator=g).to(dtype)
+    H, G, D, Hd = 8, 2, 128, 2048
+    B = max(1, (1 << 14) // n)
+    T, sc, opt = B * n, D ** -0.5, K.HeadOptions(chunk=1024)
+    if kernel == "head_attn_chunk":
+        p, sinks = rnd(T, (H + 2 * G) * D), rnd(H)
+        q, k, v = p[:, :H * D], p[:, H * D:(H + G) * D], p[:, (H + G) * D:]
+        keys = sum(i % opt.chunk + 1 for i in range(n))
+        return (lambda: K.head_attn(q, k, v, B, n, n, H, G, D, D, sc, None, opt, 0, sinks)), 4.0 * B * H * keys * D, T * (p.shape[1] + H * D) * 2
+    if kernel == "head_decode_chunk":
+        B, pages = 64, 64 * (n // 16)
+        kp, vp, q, sinks = rnd(pages * 16, G * D), rnd(pages * 16, G * D), rnd(B, H * D), rnd(H)
+        bt = torch.randperm(pages, device=dev, generator=g).int().view(B, -1).contiguous()
+        pos, keys = torch.full((B,), n - 1, dtype=torch.int32, device=dev), (n - 1) % opt.chunk + 1
+        return (lambda: K.head_decode(q, kp, vp, bt, pos, H, G, D, D, sc, None, opt, sinks=sinks)), 4.0 * B * H * keys * D, B * keys * G * 2 * D * 2
+    if kernel.startswith(("forget_", "retention_")):
+        forget = kernel.startswith("forget_")
+        H = 16 if forget else 8
+        step = kernel.endswith("_step")
+        if step:
+            B, n, T = 64, 1, 64
+        p, bias, lower, w = rnd(T, (3 if forget else 4) * H * D), rnd(H * D), torch.rand(H * D, device=dev, generator=g).to(bf), rnd(D)
+        decay, tab = torch.rand(H, device=dev, generator=g) * 0.1 + 0.9, F.rope_tables(D, max(n, 2048), device=dev)
+        st, sl, pos = torch.zeros(B, H, D, D, device=dev), torch.arange(B, dtype=torch.int32, device=dev), torch.arange(n, dtype=torch.int32, device=dev).repeat(B)
+        if step:
+            fn = (lambda: K.forget_step(p, bias, lower, st, sl, w, 1e-5, B, H, D, D)) if forget else \
+                (lambda: K.retention_step(p, decay, tab, D, pos, st, sl, None, 1e-5, B, H, D, D))
+            return fn, 0.0, B * H * D * D * 8
+        prep = (lambda: K.forget_prep(p, bias, lower, None, B, n, H, D, D)) if forget else (lambda: K.retention_prep(p, decay, tab, D, pos, None, B, n, H, D, D))
+        if kernel.endswith("_prep"):
+            return prep, 0.0, T * H * (3 * D * (2 + 4) + D)
+        r = prep()
+        return (lambda: K.gla_scan(r, st, sl, None, B, n, H, D, D, False)), 6.0 * T * H * D * D, T * H * (4 * D * 4 + D + 16)
+    T = 64 if kernel.endswith("_step") else 1 << 14
+    if kernel == "unit_norm_append":
+        p, pos, slots, temp = rnd(T, (H + 2 * G) * D), torch.arange(T, device=dev, dtype=torch.int32), torch.arange(T, device=dev), rnd(H)
+        kp, vp = rnd(T, G * D), rnd(T, G * D)
+        return (lambda: K.rope_append(p, None, pos, H, G, D, 0, G * D, slots, kp, vp, (None, None, 1e-5), temp)), 0.0, T * D * ((H + G) * 4 + G * 2 + G * 4)
+    if kernel == "head_norm":
+        o, w = rnd(T, 16, D, dtype=torch.float32), rnd(D)
+        return (lambda: K.gated_norm(o, None, w, 1e-5, bf)), 0.0, T * 16 * D * 6
+    if kernel.startswith("stream_norm"):
+        S = 2
+        x, y, z, w, c, m = rnd(T, S, Hd, dtype=torch.float32), rnd(T, Hd), rnd(T, Hd), rnd(Hd), rnd(S), torch.eye(S, device=dev).to(bf)
+        kw = dict(y2=z, w_post=w, w_post2=w, share=0.5) if kernel.endswith("_pair") else {}
+        return (lambda: K.stream_norm(x, 1e-5, y=y, mix=m, out=c, w_in=c, w_pre=w, groups=4, **kw)), 0.0, T * Hd * (S * 8 + (6 if kw else 4))
+    if kernel == "glu_clamped":
+        gu = rnd(T, 2 * 5632)
+        return (lambda: K.glu(gu, "clamped", 7.0)), 0.0, T * 5632 * 6
+    z = rnd(T, 62, dtype=torch.float32)
+    r = M.route(z, None, 6, "softmax_all")
+    if kernel.startswith("route_all"):
+        return (lambda: M.route(z, None, 6, "softmax_all")), 0.0, T * (62 * 4 + 6 * 12)
+    if kernel == "expert_glu_clamped":
+        gu = rnd(r.max_rows, 2 * 704)
+        return (lambda: M.expert_glu(gu, r, "clamped", 7.0)), 0.0, T * 6 * 704 * 6
+    raise SystemExit(f"Error: unknown kernel '{kernel}'")
+
+
 def _build(kernel, n, dev, heads=0, shape=None):
     """Returns (callable, flops, bytes) for one launch of ``kernel`` at problem size ``n``."""
     import torch
@@ -272,6 +344,8 @@ def _build(kernel, n, dev, heads=0, shape=None):
         return _build_latent(kernel, n, dev)
     if kernel in GATED_KERNELS:
         return _build_gated(kernel, n, dev)
+    if kernel in STREAM_KERNELS:
+        return _build_streams(kernel, n, dev)
 
     from ..ops import functional as F
     bf = torch.bfloat16
@@ -596,7 +670,7 @@ def main(argv=None):
         if not torch.cuda.is_available():
             print("Error: kernel benchmarks need a CUDA device", file=sys.stderr)
             return 1
-        groups = {"all": KERNELS, "stack": STACK_KERNELS, "latent": LATENT_KERNELS, "gated": GATED_KERNELS}
+        groups = {"all": KERNELS, "stack": STACK_KERNELS, "latent": LATENT_KERNELS, "gated": GATED_KERNELS, "streams": STREAM_KERNELS}
         names = [n for k in a.kernel.split(",") for n in groups.get(k, (k,))]
         peaks = json.load(open(a.peaks)) if a.peaks else {}
         for name in names:
@@ -611,7 +685,7 @@ def main(argv=None):
                    "gbs": round(nbytes / best / 1e6, 1), "tflops": round(flops / best / 1e9, 2)}
             if peaks:
                 rec["frac_hbm_of_measured"] = round(rec["gbs"] / peaks["hbm_gbs"], 3)
-                if name.startswith(("delta_scan", "gla_scan")):      # fp32 arithmetic: against the FMA lanes at the largest clock
+                if name.startswith(("delta_scan", "gla_scan", "forget_scan", "retention_scan")):      # fp32 arithmetic: against the FMA lanes at the largest clock
                     sms = torch.cuda.get_device_properties(0).multi_processor_count
                     rec["frac_fp32_fma"] = round(rec["tflops"] / (2 * FP32_FMA_PER_SM * sms * peaks.get("sm_max_mhz", 1965.0) * 1e-6), 3)
                 elif flops:

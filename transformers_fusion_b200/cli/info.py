@@ -7,6 +7,7 @@ import sys
 def _folder_info(path):
     """Model folder: architecture, sizes, layer list, tensors."""
     from ..models import registry
+    from ..models.config import mixers_of
     from ..quant.importers import _sources
     try:
         _, c = registry.read_config(path)
@@ -18,13 +19,14 @@ def _folder_info(path):
     print(f"Architecture: {c.architecture}")
     print(f"Config: vocab={c.vocab_size} hidden={c.hidden_size} layers={c.num_layers}")
     for i, l in enumerate(c.layers):
-        m, x = l.mixer, l.mixture
-        sizes = "".join(f" {n}={getattr(m, n)}" for n in ("heads", "kv_heads", "dim", "vdim", "kv_rank", "rank") if hasattr(m, n))
-        extra = "".join(f" {n}={getattr(m, n)}" for n in ("window", "keep_first", "softcap") if getattr(m, n, 0))
-        extra += f" kv_from={m.kv_from}" if getattr(m, "kv_from", None) is not None else ""
-        extra += f" weights_of={l.weights_of}" if l.weights_of is not None else ""
+        x, mix = l.mixture, []
+        for m in mixers_of(l.mixer):
+            t = m.kind + "".join(f" {n}={getattr(m, n)}" for n in ("heads", "kv_heads", "dim", "vdim", "kv_rank", "rank") if hasattr(m, n))
+            t += "".join(f" {n}={getattr(m, n)}" for n in ("window", "chunk", "keep_first", "softcap") if getattr(m, n, 0))
+            mix.append(t + (f" kv_from={m.kv_from}" if getattr(m, "kv_from", None) is not None else ""))
+        extra = f" weights_of={l.weights_of}" if l.weights_of is not None else ""
         ffn = f"ffn={l.ffn_hidden_size or 'none'}" if x is None else f"experts={x.experts} top={x.top} ffn={x.ff}" + (f" shared={x.shared_ff}" if x.shared_ff else "") + (f" groups={x.keep}/{x.groups}" if x.groups > 1 else "")
-        print(f"  layer {i}: {m.kind}{sizes}{extra} {ffn}")
+        print(f"  layer {i}: {' + '.join(mix)}{extra} {ffn}")
     total = 0
     for s in srcs:
         for n in s.names:

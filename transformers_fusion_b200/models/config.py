@@ -842,10 +842,10 @@ def preset(name: str) -> TransformerConfig:
     if name in ("toderax-7b", "toderax-8x7b"):
         # beside figudra-7b and figudra-8x7b: the same width, heads, feed-forward work per token and one shared expert; two layers in three
         # with attention and retention side by side (each with half of the heads), one with HGRN2; two streams
-        H, heads, kv, n, V, chunk, mix = (2048, 16, 4, 24, 32000, 2048, MixtureSpec(62, 6, 704, 1408, False, "softmax_all", act="clamped", limit=7.0, shared_limit=7.0)) \
-            if name == "toderax-7b" else (4096, 32, 8, 32, 32000, 8192, MixtureSpec(7, 1, 14336, 14336, False, "softmax_all", act="clamped", limit=7.0, shared_limit=7.0))
+        H, heads, kv, n, V, experts = (2048, 16, 4, 24, 32000, (62, 6, 704, 1408)) if name == "toderax-7b" else (4096, 32, 8, 32, 32000, (7, 1, 14336, 14336))
+        mix = MixtureSpec(*experts, score="softmax_all", act="clamped", limit=7.0, shared_limit=7.0)
         h = heads // 2
-        pair = PairSpec(HeadAttentionSpec(h, kv // 2, 128, 128, 128 ** 0.5, qk_norm=True, chunk=chunk, bias=True, qk_weight=False, head_temp=True, head_sink=True),
+        pair = PairSpec(HeadAttentionSpec(h, kv // 2, 128, 128, 128 ** -0.5, qk_norm=True, chunk=8192, bias=True, qk_weight=False, head_temp=True, head_sink=True),
                         RetentionSpec(h, 128, 128, tuple(1 - 2.0 ** (-5 - 5.0 * i / h) for i in range(h)), RotarySpec(128, 10000.0)))
         mixers = (pair, pair, ForgetLinearSpec(heads, 128, 128))
         return ToderaxConfig(V, H, [StackLayer(mixers[i % 3], 0, mix) for i in range(n)], 1e-5, 4, 2)
