@@ -382,7 +382,7 @@ class Retain:
     gated = True
 
     def __init__(self, H, D, V, dt, device, base=300.0):
-        self.dims, self.base, self.device = D // 4 * 2, base, device
+        self.dims, self.base, self.device = D if D in (64, 128) else D // 4 * 2, base, device
         self.decay = torch.linspace(0.4, 1.0, H) if H > 1 else torch.tensor([0.96875])
         self.args = (self.decay.to(device), F.rope_tables(self.dims, 2000, base, device=device) if self.dims else None, self.dims)
         self.sizes, self.width = (H, D, V), 2 * H * (D + V)
@@ -437,6 +437,46 @@ def test_recurrent_prompts(device, kind, H, D, V):
             for s in (ends, state):
                 close(s[slots[i]], last, tol)
         assert torch.equal(state[[1, 2]].cpu(), torch.full((2, H, D, V), 9.0))
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("kind", [Forget, Retain])
+@pytest.mark.parametrize("H,D,V", LINEAR_SIZES)
+def test_sequences_in_segments(device, kind, H, D, V):
+    """Segments of a sequence side by side: as many as fit or more, sequences that end in the first, in the middle and at the end of one,
+    fresh ones and ones that go on, in slots and without."""
+    B, S, lens = 4, 100, [100, 5, 48, 81]
+    for dt, tol in types(device, 2e-5, 2e-5):
+        m = kind(H, D, V, dt, device)
+        p = rows_of(B, S, m.width, D, dt, device)
+        rows = p.reshape(B, S, -1)
+        slots, n = torch.tensor([3, 0, 4, -1], dtype=torch.int32, device=device), torch.tensor(lens, dtype=torch.int32, device=device)
+        begin = torch.randn(5, H, D, V, generator=torch.Generator().manual_seed(5)).to(device)
+        for past in (False, True):
+            want = [m.plain(rows[i, :L], 0, begin[slots[i]].cpu().double() if past and slots[i] >= 0 else None) for i, L in enumerate(lens)]
+            for segments in (1, 2, 3, 7, 30):
+                state = begin.clone()
+                got = K.gla_scan(m.prep(p, n, B, S, 0), state, slots, n, B, S, H, D, V, past, segments).view(B, S, H, V)
+                for i, L in enumerate(lens):
+                    close(got[i, :L], want[i][0], tol)
+                    assert not got[i, L:].any()
+                    if slots[i] >= 0:
+                        close(state[slots[i]], want[i][1], tol)
+                assert torch.equal(state[[1, 2]], begin[[1, 2]])
+
+
+@pytest.mark.parametrize("device", DEVICES)
+def test_long_sequence_in_segments(device):
+    """Of the kernel's own choice, against the sequence in one piece."""
+    H, D, V, S = 2, 32, 16, 1500
+    for kind in (Forget, Retain):
+        m = kind(H, D, V, torch.float32, device)
+        p = rows_of(1, S, m.width, 1, torch.float32, device)
+        state, slot = torch.zeros(1, H, D, V, device=device), torch.zeros(1, dtype=torch.int32, device=device)
+        want, last = m.plain(p)
+        for segments in (None, 1):
+            close(K.gla_scan(m.prep(p, None, 1, S, 0), state, slot, None, 1, S, H, D, V, False, segments), want, 2e-5)
+            close(state[0], last, 2e-5)
 
 
 @pytest.mark.parametrize("device", DEVICES)

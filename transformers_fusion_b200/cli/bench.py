@@ -32,7 +32,7 @@ LATENT_KERNELS = ("head_attn", "attention_fwd_mha128", "latent_decode", "latent_
 GATED_KERNELS = ("head_attn_cap", "head_attn_window", "head_attn_gqa", "head_decode", "head_decode_cap", "head_decode_window", "gla_prep", "gla_scan",
                  "gla_scan_one", "gla_step", "norm_rope_append", "parallel_norm", "glu_gelu", "grouped_route", "grouped_route_step", "weighted_sum_gated")
 STREAM_KERNELS = ("head_attn_chunk", "head_decode_chunk", "unit_norm_append", "forget_prep", "forget_scan", "forget_step", "retention_prep", "retention_scan",
-                  "retention_step", "head_norm", "stream_norm", "stream_norm_pair", "glu_clamped", "route_all", "route_all_step", "expert_glu_clamped")
+                  "forget_scan_one", "retention_scan_one", "retention_step", "head_norm", "stream_norm", "stream_norm_pair", "glu_clamped", "route_all", "route_all_step", "expert_glu_clamped")
 FP32_FMA_PER_SM = 128          # fp32 FMA lanes of an SM (the scans are reported against them)
 
 
@@ -277,7 +277,7 @@ def _build_streams(kernel, n, dev):
     g = torch.Generator(device=dev).manual_seed(0)
     rnd = lambda *s, dtype=bf: torch.randn(*s, device=dev, generator=g).to(dtype)
     H, G, D, Hd = 8, 2, 128, 2048
-    B = max(1, (1 << 14) // n)
+    B = 1 if kernel.endswith("_one") else max(1, (1 << 14) // n)
     T, sc, opt = B * n, D ** -0.5, K.HeadOptions(chunk=1024)
     if kernel == "head_attn_chunk":
         p, sinks = rnd(T, (H + 2 * G) * D), rnd(H)

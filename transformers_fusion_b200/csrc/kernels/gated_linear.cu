@@ -17,7 +17,9 @@
 //               tokens.  The columns of S are independent, so a group of TPC threads owns CPT columns (D / TPC entries of each, in
 //               registers as packed fp32 pairs).  The sums over D are needed for the output alone: no reduction is on the
 //               path from one state to the next.  The rows of the next tokens travel to shared memory (bulk copies) while the
-//               current ones are used; fp32 FMA throughout.
+//               current ones are used; fp32 FMA throughout.  Few sequences leave most of the device idle, so theirs are cut into
+//               segments: a first pass over all but the last computes what each adds to the state and the product of its decays, the
+//               second, with the start of a segment put together from those before it, everything else.
 //   gla_step    one token per sequence: one block per (sequence, head) computes q, k and the decays, streams the state through registers
 //               once (read, updated, written back), and applies the norm (with weight and gate, where there are some) to the output.
 #include "tfb_elem.cuh"
@@ -136,11 +138,27 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) gla_prep_kernel(const GlaPrep
   float pr[16];
 #pragma unroll
   for (int i = 0; i < 16; ++i) pr[i] = 0.f;
-  for (int d0 = lane; d0 < p.Dp; d0 += 64) {          // two channels at a time: d0 and d0 + 32
+  // two channels at a time: d0 and d0 + 32, or, where all entries turn, a pair that turns together
+  const bool turns = KIND == RETENTION && g.dims == g.D && p.Dp == g.D;
+  const int apart = turns ? g.D / 2 : 32, d_end = turns ? g.D / 2 : p.Dp, d_step = turns ? 32 : 64;
+  for (int d0 = lane; d0 < d_end; d0 += d_step) {
     float z[2][4];                                    // logits of the decays (GATED), or the decays
     float q[2][4], k[2][4];
     const T* w[2];
-    if constexpr (KIND != GATED) {
+    if (turns) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const T* x = row[i] + (long long)h * g.D + d0;
+        const long long at = (long long)pos[i] * apart + d0, kk = (long long)g.H * g.D;
+        const float c = g.cos_t[at], s = g.sin_t[at], q0 = to_f(x[0]), q1 = to_f(x[apart]), k0 = to_f(x[kk]) * scale, k1 = to_f(x[kk + apart]) * scale;
+        const float f = i < n ? 1.f : 0.f;
+        q[0][i] = f * (q0 * c - q1 * s);
+        q[1][i] = f * (q1 * c + q0 * s);
+        k[0][i] = f * (k0 * c - k1 * s);
+        k[1][i] = f * (k1 * c + k0 * s);
+        z[0][i] = z[1][i] = g.decay[h];
+      }
+    } else if constexpr (KIND != GATED) {
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         const int d = d0 + 32 * x;
@@ -188,7 +206,7 @@ __global__ void __launch_bounds__(PREP_WARPS * 32) gla_prep_kernel(const GlaPrep
     }
 #pragma unroll
     for (int x = 0; x < 2; ++x) {
-      const int d = d0 + 32 * x;
+      const int d = d0 + apart * x;
       if (d >= p.Dp) break;
       float G = 1.f, t[4];              // t[j] = R_ij k_j for the current i
 #pragma unroll
@@ -237,23 +255,29 @@ struct GlaScanArgs {
   const int* lens;        // [B] or null
   int S, Sp, H, D, V, Vp, has_past, nslots;
   int* status;
+  int seg, nseg;          // tokens of a segment (a multiple of GS_CHUNK), segments of a sequence
+  float* part;            // nseg > 1: [B, nseg, H, D, V]: the state behind segment i, of itself alone but for segment 0; last: the first state
+  float* prod;            // nseg > 1: [B, nseg - 1, H, Dp]: products of the decays of segment i
 };
 
 constexpr int GS_CHUNK = 16;   // tokens per shared-memory stage
 
 // EPT: entries of one column per thread (a multiple of 4); TPC: threads per column group; CPT: columns per group (powers of two, CPT <=
 // TPC); Dp = EPT TPC.  A shuffle reduction of the CPT columns' four sums each leaves one column with each TPC / CPT threads.
-template <int EPT, int TPC, int CPT>
+// FIRST: the first pass over segments (states and decays only).
+template <int EPT, int TPC, int CPT, bool FIRST>
 __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
   tfb::pdl_sync();
   extern __shared__ __align__(128) float sm[];
   constexpr int Dp = EPT * TPC, CPW = 32 / TPC * CPT, W = TPC / CPT;
   static_assert(CPT <= TPC && EPT % 4 == 0, "tile shape");
   const int tid = threadIdx.x, lane = tid & 31, cols = (blockDim.x >> 5) * CPW;
-  const int h = blockIdx.y, b = blockIdx.z, col0 = blockIdx.x * cols;
+  const int nz = FIRST ? p.nseg - 1 : p.nseg, h = blockIdx.y, b = blockIdx.z / nz, si = blockIdx.z % nz, col0 = blockIdx.x * cols;
   const int t = lane % TPC, cl = (tid >> 5) * CPW + lane / TPC * CPT;      // first column of the group, within the block
   const int my_cl = cl + t / W, my_col = col0 + my_cl;                      // the column this thread ends up with
-  const int len = p.lens ? p.lens[b] : p.S;
+  // this segment: rows first .. first + len - 1 of the sequence, and padding up to `end`
+  const int total = p.lens ? p.lens[b] : p.S, first = si * p.seg, len = max(0, min(total - first, p.seg)), end = min(p.S, first + p.seg);
+  if (FIRST && len < p.seg) return;      // nothing comes behind it
   constexpr int KQ = GS_CHUNK * Dp, DEC = GS_CHUNK / 4 * Dp, PR = GS_CHUNK * 4;
   const int stage_f = 2 * KQ + DEC + PR + GS_CHUNK * cols;
   const uint32_t bar = smem_u32(sm + 2 * stage_f);
@@ -269,23 +293,23 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
   fence_proxy_async_smem();
   __syncthreads();
   const long long hb = (long long)b * p.H + h;
-  const float* qb = p.q + hb * p.Sp * Dp;
-  const float* kb = p.k + hb * p.Sp * Dp;
-  const float* db = p.decay + hb * (p.Sp / 4) * Dp;
-  const float* pb = p.pair + hb * (p.Sp / 4) * 16;
-  const float* vb = p.v + hb * p.Sp * p.Vp + col0;
+  const float* qb = p.q + (hb * p.Sp + first) * Dp;
+  const float* kb = p.k + (hb * p.Sp + first) * Dp;
+  const float* db = p.decay + (hb * (p.Sp / 4) + first / 4) * Dp;
+  const float* pb = p.pair + (hb * (p.Sp / 4) + first / 4) * 16;
+  const float* vb = p.v + (hb * p.Sp + first) * p.Vp + col0;
   const int nrow = (len + 3) / 4 * 4, nc = min(cols, p.Vp - col0);
   auto issue = [&](int c) {              // warp 0: the rows of chunk c (whole groups of four)
     const int s0 = c * GS_CHUNK, n = min(GS_CHUNK, nrow - s0);
     if (n <= 0 || tid >= 32) return;
     float* base = sm + (c & 1) * stage_f;
     const uint32_t br = bar + (c & 1) * 8;
-    if (lane == 0) mbar_expect_tx(br, uint32_t(n) * (2 * Dp + Dp / 4 + 4 + nc) * 4);
+    if (lane == 0) mbar_expect_tx(br, uint32_t(n) * ((FIRST ? Dp : 2 * Dp + 4) + Dp / 4 + nc) * 4);
     __syncwarp();
-    if (lane == 0) bulk_load(smem_u32(base), qb + (long long)s0 * Dp, n * Dp * 4, br);
+    if (lane == 0 && !FIRST) bulk_load(smem_u32(base), qb + (long long)s0 * Dp, n * Dp * 4, br);
     if (lane == 1) bulk_load(smem_u32(base + KQ), kb + (long long)s0 * Dp, n * Dp * 4, br);
     if (lane == 2) bulk_load(smem_u32(base + 2 * KQ), db + (long long)(s0 / 4) * Dp, n * Dp, br);
-    if (lane == 3) bulk_load(smem_u32(base + 2 * KQ + DEC), pb + (long long)s0 * 4, n * 16, br);
+    if (lane == 3 && !FIRST) bulk_load(smem_u32(base + 2 * KQ + DEC), pb + (long long)s0 * 4, n * 16, br);
     if (lane >= 16 && lane - 16 < n)
       bulk_load(smem_u32(base + 2 * KQ + DEC + PR + (lane - 16) * cols), vb + (long long)(s0 + lane - 16) * p.Vp, nc * 4, br);
   };
@@ -296,6 +320,10 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
   TFB_BOUNDS(slot < p.nslots, 72, slot, p.nslots);
   if (slot >= p.nslots) slot = -1;
   float* S0 = slot >= 0 ? p.state + ((long long)slot * p.H + h) * p.D * p.V : nullptr;
+  const long long DV = (long long)p.D * p.V;
+  auto part_of = [&](int i) { return p.part + (((long long)b * p.nseg + i) * p.H + h) * DV; };
+  const float* start = nullptr;
+  if (p.has_past && si == 0 && S0) start = FIRST || total < p.seg || p.nseg == 1 ? S0 : part_of(p.nseg - 1);
   // entry d of a column sits with thread (d / 4) % TPC, register (d / 4) / TPC * 4 + d % 4
   u64 st[CPT][EPT / 2];
 #pragma unroll
@@ -306,15 +334,24 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int d = (i * TPC + t) * 4 + e, col = col0 + cl + x;
-        f[e] = (S0 && p.has_past && col < p.V && d < p.D) ? S0[(long long)d * p.V + col] : 0.f;
+        const bool on = col < p.V && d < p.D;
+        const long long at = (long long)d * p.V + col;
+        f[e] = start && on ? start[at] : 0.f;
+        if (FIRST && start && on) part_of(p.nseg - 1)[at] = f[e];        // the second pass may find it overwritten
+        if (!FIRST && on && len > 0)
+          for (int j = 0; j < si; ++j)
+            f[e] = fmaf(j ? p.prod[(((long long)b * (p.nseg - 1) + j) * p.H + h) * Dp + d] : 0.f, f[e], part_of(j)[at]);
       }
       st[x][2 * i] = pack2(f[0], f[1]);
       st[x][2 * i + 1] = pack2(f[2], f[3]);
     }
+  u64 all[FIRST ? EPT / 2 : 1];          // products of the decays
+#pragma unroll
+  for (int i = 0; i < (FIRST ? EPT / 2 : 1); ++i) all[i] = pack2(1.f, 1.f);
 
   const int nchunk = (len + GS_CHUNK - 1) / GS_CHUNK;
   const long long ostep = (long long)p.H * p.V;
-  float* orow = p.o + ((long long)b * p.S * p.H + h) * p.V + my_col;
+  float* orow = p.o + (((long long)b * p.S + first) * p.H + h) * p.V + my_col;
   const bool writer = t % W == 0 && my_col < p.V;
   for (int c = 0; c < nchunk; ++c) {
     if (!mbar_wait_warp(bar + (c & 1) * 8, (c >> 1) & 1, abort_flag, p.status, ST_TIMEOUT_FULL)) break;
@@ -342,14 +379,20 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
         const ulonglong2 g = sg[e * TPC];
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-          q[i] = sq[i * (Dp / 4) + e * TPC];
+          if (!FIRST) q[i] = sq[i * (Dp / 4) + e * TPC];
           k[i] = sk[i * (Dp / 4) + e * TPC];
+        }
+        if constexpr (FIRST) {
+          all[2 * e] = mul2(all[2 * e], g.x);
+          all[2 * e + 1] = mul2(all[2 * e + 1], g.y);
         }
 #pragma unroll
         for (int x = 0; x < CPT; ++x) {
           const u64 s0 = st[x][2 * e], s1 = st[x][2 * e + 1];
+          if constexpr (!FIRST) {
 #pragma unroll
-          for (int i = 0; i < 4; ++i) acc[x][i] = fma2(s1, q[i].y, fma2(s0, q[i].x, acc[x][i]));
+            for (int i = 0; i < 4; ++i) acc[x][i] = fma2(s1, q[i].y, fma2(s0, q[i].x, acc[x][i]));
+          }
           u64 u0 = mul2(s0, g.x), u1 = mul2(s1, g.y);
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
@@ -360,6 +403,7 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
           st[x][2 * e + 1] = u1;
         }
       }
+      if constexpr (FIRST) continue;
       float val[CPT][4];
 #pragma unroll
       for (int x = 0; x < CPT; ++x)
@@ -406,9 +450,10 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
     while (globaltimer_ns() - t0 < 200000ull) {}      // bounded wait for copies already issued
     return;
   }
-  if (writer)                            // padding: numbers, since a weight of zero does not silence what is not one
-    for (int s = len; s < p.S; ++s) orow[s * ostep] = 0.f;
-  if (S0) {
+  if (!FIRST && writer)                  // padding: numbers, since a weight of zero does not silence what is not one
+    for (int s = len; s < end - first; ++s) orow[s * ostep] = 0.f;
+  float* out = FIRST ? part_of(si) : (total > first || si == 0) && total <= first + p.seg ? S0 : nullptr;
+  if (out) {
 #pragma unroll
     for (int x = 0; x < CPT; ++x)
 #pragma unroll
@@ -418,9 +463,19 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
           const int d = (i * TPC + t) * 4 + e, col = col0 + cl + x;
-          if (d < p.D && col < p.V) S0[(long long)d * p.V + col] = f[e];
+          if (d < p.D && col < p.V) out[(long long)d * p.V + col] = f[e];
         }
       }
+  }
+  if constexpr (FIRST) {
+    if (blockIdx.x == 0 && tid < TPC) {
+      float* g = p.prod + (((long long)b * (p.nseg - 1) + si) * p.H + h) * Dp;
+#pragma unroll
+      for (int i = 0; i < EPT / 4; ++i) {
+        const float2 a = unpack2(all[2 * i]), c = unpack2(all[2 * i + 1]);
+        *reinterpret_cast<float4*>(g + (i * TPC + t) * 4) = make_float4(a.x, a.y, c.x, c.y);
+      }
+    }
   }
 }
 
@@ -429,24 +484,30 @@ static int launch_scan_tile(const GlaScanArgs& p, int B, cudaStream_t st) {
   constexpr int CPW = 32 / TPC * CPT;
   auto bytes = [](int w) { return (2 * (2 * GS_CHUNK * EPT * TPC + GS_CHUNK / 4 * EPT * TPC + GS_CHUNK * 4 + GS_CHUNK * w * CPW) + 8) * int(sizeof(float)); };
   // warps per block: rows of v are copied in 16-byte pieces, so at least four columns; blocks for most of the SMs
-  const long long warps = (long long)((p.V + CPW - 1) / CPW) * p.H * B;
+  const long long warps = (long long)((p.V + CPW - 1) / CPW) * p.H * B * p.nseg;
   int nw = 4;
   while (nw > 1 && nw / 2 * CPW >= 4 && (nw * CPW > p.Vp || (warps + nw - 1) / nw < 4 * sm_count() / 5)) nw >>= 1;
   if ((nw * CPW) % 4) return TFB_ERR_ARG;
-  static DeviceOnce once;
-  auto kern = gla_scan_kernel<EPT, TPC, CPT>;
+  static DeviceOnce once, once_first;
+  auto kern = gla_scan_kernel<EPT, TPC, CPT, false>, kern_first = gla_scan_kernel<EPT, TPC, CPT, true>;
   if (int e = ensure_dyn_smem(once, kern, bytes(4))) return e;
+  if (int e = ensure_dyn_smem(once_first, kern_first, bytes(4))) return e;
   const int cols = nw * CPW;
-  launch_k(kern, dim3((p.V + cols - 1) / cols, p.H, B), nw * 32, bytes(nw), st, p);
+  if (p.nseg > 1) launch_k(kern_first, dim3((p.V + cols - 1) / cols, p.H, B * (p.nseg - 1)), nw * 32, bytes(nw), st, p);
+  launch_k(kern, dim3((p.V + cols - 1) / cols, p.H, B * p.nseg), nw * 32, bytes(nw), st, p);
   return int(cudaGetLastError());
+}
+
+// Warps of the form with four columns per group, the one that reads q' and k' from shared memory least often
+static long long scan_warps(int B, int H, int Dp, int V) {
+  const int TPC = Dp <= 128 ? 8 : Dp / 16, CPW = 32 / TPC * 4;
+  return (long long)((V + CPW - 1) / CPW) * H * B;
 }
 
 template <int EPT, int TPC>
 static int launch_scan(const GlaScanArgs& p, int B, cudaStream_t st) {
-  // Four columns per group read q' and k' from shared memory a quarter as often; for few sequences two columns per group of twice as
-  // many threads give each scheduler something to do.
-  constexpr int CPW = 32 / TPC * 4;
-  if ((long long)((p.V + CPW - 1) / CPW) * p.H * B >= 3ll * sm_count()) return launch_scan_tile<EPT, TPC, 4>(p, B, st);
+  // For few columns, two per group of twice as many threads give each scheduler something to do.
+  if (scan_warps(B, p.H, EPT * TPC, p.V) * p.nseg >= 3ll * sm_count()) return launch_scan_tile<EPT, TPC, 4>(p, B, st);
   if constexpr (EPT >= 8 && TPC <= 16) return launch_scan_tile<EPT / 2, TPC * 2, 2>(p, B, st);
   else return launch_scan_tile<EPT, TPC, 2>(p, B, st);
 }
@@ -669,12 +730,29 @@ TFB_API int tfb_retention_prep(const void* proj, long long ld, const float* head
   return run_prep(g, RETENTION, lens, q, k, v, decay, pair, B, S, Dp, f32, stream);
 }
 
-// The recurrence over prepared rows; o [B*S, H, V] fp32.
-TFB_API int tfb_gla_scan(const float* q, const float* k, const float* v, const float* decay, const float* pair, float* o, float* state, int nslots,
-                         const int* state_slots, int B, int S, int H, int D, int V, int has_past, const int* lens, int* status, void* stream) {
+// Segments into which tfb_gla_scan cuts sequences of S tokens: as many as give the device enough warps, if the sequences alone give it less
+// than half of them (the first pass costs about half of the second), of at least 256 tokens.
+TFB_API int tfb_gla_scan_segments(int B, int S, int H, int D, int V) {
   using namespace tfb;
-  if (B <= 0 || B > 65535 || S <= 0 || H <= 0 || H > 65535 || D <= 0 || V <= 0) return TFB_ERR_ARG;
-  const GlaScanArgs p{q, k, v, decay, pair, o, state, state_slots, lens, S, (S + 3) / 4 * 4, H, D, V, (V + 3) / 4 * 4, has_past, nslots, status};
+  if (B <= 0 || S <= 0 || H <= 0 || D <= 0 || V <= 0 || !padded_dim(D)) return 1;
+  const long long warps = scan_warps(B, H, padded_dim(D), V), want = 7ll * sm_count();
+  int n = 1;
+  if (warps * 5 <= want * 2)
+    while (n < 32 && warps * n < want && S / (2 * n) >= 256) n *= 2;
+  return n;
+}
+
+// The recurrence over prepared rows; o [B*S, H, V] fp32.  segments > 1: every sequence is cut into (at most) so many, with work (fp32) of
+// B segments H (D V + Dp) entries.
+TFB_API int tfb_gla_scan(const float* q, const float* k, const float* v, const float* decay, const float* pair, float* o, float* state, int nslots,
+                         const int* state_slots, int B, int S, int H, int D, int V, int has_past, const int* lens, int segments, float* work, int* status,
+                         void* stream) {
+  using namespace tfb;
+  if (B <= 0 || B > 65535 || S <= 0 || H <= 0 || H > 65535 || D <= 0 || V <= 0 || segments < 1 || (segments > 1 && !work)) return TFB_ERR_ARG;
+  const int seg = ((S + segments - 1) / segments + GS_CHUNK - 1) / GS_CHUNK * GS_CHUNK, nseg = (S + seg - 1) / seg;
+  if ((long long)B * nseg > 65535) return TFB_ERR_LIMIT;
+  const GlaScanArgs p{q, k, v, decay, pair, o, state, state_slots, lens, S, (S + 3) / 4 * 4, H, D, V, (V + 3) / 4 * 4, has_past, nslots, status, seg, nseg,
+                      work ? work + (long long)B * (nseg - 1) * H * padded_dim(D) : nullptr, work};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   switch (padded_dim(D)) {
     case 32: return launch_scan<4, 8>(p, B, st);

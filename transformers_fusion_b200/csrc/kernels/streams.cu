@@ -79,6 +79,31 @@ __global__ void stream_norm_kernel(const StreamArgs p) {
     id = id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id);
     trow = static_cast<const T*>(p.table) + id * p.ld_table;
   }
+  // the streams are on their way while the statistics of y are taken, where the registers hold them
+  constexpr bool EARLY = ST > 0 && ST * NV * VEC <= 32;
+  float early[EARLY ? NV : 1][SM][VEC];
+  auto load_streams = [&](int col, float (&v)[SM][VEC]) {
+    if (trow) {
+      load_n<VEC>(trow + col, v[0]);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[0][e] *= p.scale;
+#pragma unroll
+      for (int s = 1; s < SM; ++s)
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[s][e] = v[0][e];
+    } else {
+#pragma unroll
+      for (int s = 0; s < SM; ++s)
+        if (s < S) load_n<VEC>(p.x + (r * S + s) * H + col, v[s]);
+    }
+  };
+  if constexpr (EARLY) {
+#pragma unroll
+    for (int c = 0; c < NV; ++c) {
+      const int col = (c * nt + threadIdx.x) * VEC;
+      if (col < H) load_streams(col, early[c]);
+    }
+  }
   float y[NV][VEC];
   if (p.y) {
     float y2[NV][VEC];
@@ -121,21 +146,10 @@ __global__ void stream_norm_kernel(const StreamArgs p) {
   for (int c = 0; c < NV; ++c) {
     const int col = (c * nt + threadIdx.x) * VEC;
     if (col >= H) continue;
-    float v[SM][VEC];
+    float late[SM][VEC];
     float* xr = p.x + r * S * H + col;
-    if (trow) {
-      load_n<VEC>(trow + col, v[0]);
-#pragma unroll
-      for (int e = 0; e < VEC; ++e) v[0][e] *= p.scale;
-#pragma unroll
-      for (int s = 1; s < SM; ++s)
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) v[s][e] = v[0][e];
-    } else {
-#pragma unroll
-      for (int s = 0; s < SM; ++s)
-        if (s < S) load_n<VEC>(xr + (long long)s * H, v[s]);
-    }
+    if constexpr (!EARLY) load_streams(col, late);
+    float (&v)[SM][VEC] = EARLY ? early[EARLY ? c : 0] : late;
 #pragma unroll
     for (int e = 0; e < VEC; ++e) u[c][e] = 0.f;
 #pragma unroll

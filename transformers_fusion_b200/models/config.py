@@ -753,8 +753,8 @@ class ToderaxConfig:
                 mixture = MixtureSpec(r["experts"], r["top"], x["ff"], sh["ff"] if sh else 0, score="softmax_all", act="clamped", limit=float(x["limit"]),
                                       shared_limit=float(sh["limit"]) if sh else 0.0)
             layers.append(StackLayer(mix, 0, mixture))
-        return cls(vocab_size=d["vocab"], hidden_size=d["width"], layers=layers, norm_eps=float(d["norm"]["eps"]), norm_groups=int(d["norm"]["groups"]),
-                   streams=int(d["streams"]), embedding_scale=float(d["embedding"]["scale"]), **extra)
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], layers=layers, norm_eps=float(d["norm"]["eps"]), norm_groups=int(d["norm"].get("groups", 1)),
+                   streams=int(d.get("streams", 1)), embedding_scale=float(d["embedding"]["scale"]), **extra)
 
     def to_dict(self) -> dict:
         """The config.json form."""

@@ -47,7 +47,8 @@ _lib.register("tfb_head_decode_plan", [c_i, c_i, c_i, c_i, c_i, c_i, c_i])
 _lib.register("tfb_head_decode", [c_p, c_ll, c_p, c_p, c_ll, c_p, c_i, c_i, c_p, c_p, c_ll, c_p, c_ll, c_i, c_p, c_p, c_i, c_i, c_i, c_i, c_i, c_i, c_f,
                                   c_i, c_i, c_i, c_f, c_i, c_p, c_f, c_i, c_i, c_p, c_p])
 _lib.register("tfb_gla_prep", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_f, c_p] + [c_p] * 5 + [c_i] * 7 + [c_p])
-_lib.register("tfb_gla_scan", [c_p] * 7 + [c_i, c_p] + [c_i] * 6 + [c_p, c_p, c_p])
+_lib.register("tfb_gla_scan_segments", [c_i] * 5)
+_lib.register("tfb_gla_scan", [c_p] * 7 + [c_i, c_p] + [c_i] * 6 + [c_p, c_i, c_p, c_p, c_p])
 _lib.register("tfb_gla_step", [c_p, c_ll, c_p, c_ll, c_p, c_i, c_f, c_p, c_p, c_i, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
 _lib.register("tfb_forget_prep", [c_p, c_ll, c_p, c_p, c_p] + [c_p] * 5 + [c_i] * 7 + [c_p])
 _lib.register("tfb_forget_step", [c_p, c_ll, c_p, c_p, c_i, c_p, c_p, c_i, c_p, c_p, c_ll, c_i, c_i, c_i, c_i, c_f, c_i, c_p])
@@ -726,9 +727,10 @@ def retention_prep(proj, decay, tables, dims, positions, lens, B, S, H, D, V) ->
     return r
 
 
-def gla_scan(rows_: GlaRows, state, state_slots, lens, B, S, H, D, V, has_past):
+def gla_scan(rows_: GlaRows, state, state_slots, lens, B, S, H, D, V, has_past, segments: Optional[int] = None):
     """S <- diag(decay) S + k v^T, o = S^T q over prepared rows; ``state`` [slots, H, D, V] fp32 is read (``has_past``) and updated.
-    Returns fp32 [B*S, H, V] (rows past a sequence's length are zero)."""
+    Returns fp32 [B*S, H, V] (rows past a sequence's length are zero).  ``segments``: parts of a sequence that run side by side (None: the
+    kernel's choice)."""
     r = rows_
     if not r.q.is_cuda:
         out = torch.zeros(B * S, H, V)
@@ -743,9 +745,11 @@ def gla_scan(rows_: GlaRows, state, state_slots, lens, B, S, H, D, V, has_past):
                 state[sl] = st
         return out
     o = torch.empty((B * S, H, V), dtype=torch.float32, device=r.q.device)
-    check(_lib.lib().tfb_gla_scan(r.q.data_ptr(), r.k.data_ptr(), r.v.data_ptr(), r.decay.data_ptr(), r.pair.data_ptr(), o.data_ptr(),
-                                  state.data_ptr(), state.shape[0], state_slots.data_ptr(), B, S, H, D, V, int(has_past), ptr(lens),
-                                  _lib.status_word(o.device).data_ptr(), stream()), "gla_scan")
+    L = _lib.lib()
+    n = segments or L.tfb_gla_scan_segments(B, S, H, D, V)
+    work = torch.empty(B * n * H * (D * V + r.q.shape[-1]), dtype=torch.float32, device=o.device) if n > 1 else None
+    check(L.tfb_gla_scan(*_ptrs(r), o.data_ptr(), state.data_ptr(), state.shape[0], state_slots.data_ptr(), B, S, H, D, V, int(has_past), ptr(lens), n,
+                         ptr(work), _lib.status_word(o.device).data_ptr(), stream()), "gla_scan", 1 + int(n > 1))
     return o
 
 
