@@ -264,15 +264,38 @@ constexpr int GS_CHUNK = 16;   // tokens per shared-memory stage
 
 // EPT: entries of one column per thread (a multiple of 4); TPC: threads per column group; CPT: columns per group (powers of two, CPT <=
 // TPC); Dp = EPT TPC.  A shuffle reduction of the CPT columns' four sums each leaves one column with each TPC / CPT threads.
-// FIRST: the first pass over segments (states and decays only).
-template <int EPT, int TPC, int CPT, bool FIRST>
-__global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
+enum { WHOLE = 0, SEG_FIRST = 1, SEG_SECOND = 2 };     // sequences in one piece; the first pass over segments (states and decays only); the second
+
+// CPT neighbouring entries of a row, `n` of them in range (vec: a multiple of CPT, and aligned)
+template <int CPT>
+__device__ __forceinline__ void load_columns(const float* row, int n, bool vec, float (&f)[CPT]) {
+  if constexpr (CPT == 4) {
+    if (vec) {
+      const float4 u = n > 0 ? *reinterpret_cast<const float4*>(row) : make_float4(0.f, 0.f, 0.f, 0.f);
+      f[0] = u.x, f[1] = u.y, f[2] = u.z, f[3] = u.w;
+      return;
+    }
+  } else if constexpr (CPT == 2) {
+    if (vec) {
+      const float2 u = n > 0 ? *reinterpret_cast<const float2*>(row) : make_float2(0.f, 0.f);
+      f[0] = u.x, f[1] = u.y;
+      return;
+    }
+  }
+#pragma unroll
+  for (int x = 0; x < CPT; ++x) f[x] = x < n ? row[x] : 0.f;
+}
+
+template <int EPT, int TPC, int CPT, int PASS>
+__global__ void __launch_bounds__(128, 2) gla_scan_kernel(const GlaScanArgs p) {
+  constexpr bool FIRST = PASS == SEG_FIRST;
   tfb::pdl_sync();
   extern __shared__ __align__(128) float sm[];
   constexpr int Dp = EPT * TPC, CPW = 32 / TPC * CPT, W = TPC / CPT;
   static_assert(CPT <= TPC && EPT % 4 == 0, "tile shape");
   const int tid = threadIdx.x, lane = tid & 31, cols = (blockDim.x >> 5) * CPW;
-  const int nz = FIRST ? p.nseg - 1 : p.nseg, h = blockIdx.y, b = blockIdx.z / nz, si = blockIdx.z % nz, col0 = blockIdx.x * cols;
+  const int nz = PASS == WHOLE ? 1 : FIRST ? p.nseg - 1 : p.nseg, si = PASS == WHOLE ? 0 : blockIdx.z % nz;
+  const int h = blockIdx.y, b = PASS == WHOLE ? blockIdx.z : blockIdx.z / nz, col0 = blockIdx.x * cols;
   const int t = lane % TPC, cl = (tid >> 5) * CPW + lane / TPC * CPT;      // first column of the group, within the block
   const int my_cl = cl + t / W, my_col = col0 + my_cl;                      // the column this thread ends up with
   // this segment: rows first .. first + len - 1 of the sequence, and padding up to `end`
@@ -323,28 +346,55 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
   const long long DV = (long long)p.D * p.V;
   auto part_of = [&](int i) { return p.part + (((long long)b * p.nseg + i) * p.H + h) * DV; };
   const float* start = nullptr;
-  if (p.has_past && si == 0 && S0) start = FIRST || total < p.seg || p.nseg == 1 ? S0 : part_of(p.nseg - 1);
+  if (p.has_past && si == 0 && S0) start = PASS != SEG_SECOND || total < p.seg ? S0 : part_of(p.nseg - 1);
+  const int nv = p.V - (col0 + cl);        // columns of this group that there are
+  const bool vec = p.V % CPT == 0;
   // entry d of a column sits with thread (d / 4) % TPC, register (d / 4) / TPC * 4 + d % 4
   u64 st[CPT][EPT / 2];
+  if constexpr (PASS == WHOLE) {
 #pragma unroll
-  for (int x = 0; x < CPT; ++x)
+    for (int x = 0; x < CPT; ++x)
 #pragma unroll
-    for (int i = 0; i < EPT / 4; ++i) {
-      float f[4];
+      for (int i = 0; i < EPT / 4; ++i) {
+        float f[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int d = (i * TPC + t) * 4 + e, col = col0 + cl + x;
-        const bool on = col < p.V && d < p.D;
-        const long long at = (long long)d * p.V + col;
-        f[e] = start && on ? start[at] : 0.f;
-        if (FIRST && start && on) part_of(p.nseg - 1)[at] = f[e];        // the second pass may find it overwritten
-        if (!FIRST && on && len > 0)
-          for (int j = 0; j < si; ++j)
-            f[e] = fmaf(j ? p.prod[(((long long)b * (p.nseg - 1) + j) * p.H + h) * Dp + d] : 0.f, f[e], part_of(j)[at]);
+        for (int e = 0; e < 4; ++e) {
+          const int d = (i * TPC + t) * 4 + e, col = col0 + cl + x;
+          f[e] = (start && col < p.V && d < p.D) ? start[(long long)d * p.V + col] : 0.f;
+        }
+        st[x][2 * i] = pack2(f[0], f[1]);
+        st[x][2 * i + 1] = pack2(f[2], f[3]);
       }
-      st[x][2 * i] = pack2(f[0], f[1]);
-      st[x][2 * i + 1] = pack2(f[2], f[3]);
+  } else {
+#pragma unroll
+    for (int i = 0; i < EPT / 2; ++i) {
+      float f[2][CPT];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int d = (i / 2 * TPC + t) * 4 + i % 2 * 2 + e, n = d < p.D ? nv : 0;
+        const long long at = (long long)d * p.V + col0 + cl;
+#pragma unroll
+        for (int x = 0; x < CPT; ++x) f[e][x] = 0.f;
+        if (start) load_columns<CPT>(start + at, n, vec, f[e]);
+        if (FIRST && start) {                // the second pass may find it overwritten
+#pragma unroll
+          for (int x = 0; x < CPT; ++x)
+            if (x < n) part_of(p.nseg - 1)[at + x] = f[e][x];
+        }
+        if (PASS == SEG_SECOND && len > 0 && n > 0) {
+          for (int j = 0; j < si; ++j) {
+            const float g = j ? p.prod[(((long long)b * (p.nseg - 1) + j) * p.H + h) * Dp + d] : 0.f;
+            float u[CPT];
+            load_columns<CPT>(part_of(j) + at, n, vec, u);
+#pragma unroll
+            for (int x = 0; x < CPT; ++x) f[e][x] = fmaf(g, f[e][x], u[x]);
+          }
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < CPT; ++x) st[x][i] = pack2(f[0][x], f[1][x]);
     }
+  }
   u64 all[FIRST ? EPT / 2 : 1];          // products of the decays
 #pragma unroll
   for (int i = 0; i < (FIRST ? EPT / 2 : 1); ++i) all[i] = pack2(1.f, 1.f);
@@ -403,42 +453,43 @@ __global__ void __launch_bounds__(128) gla_scan_kernel(const GlaScanArgs p) {
           st[x][2 * e + 1] = u1;
         }
       }
-      if constexpr (FIRST) continue;
-      float val[CPT][4];
+      if constexpr (!FIRST) {
+        float val[CPT][4];
 #pragma unroll
-      for (int x = 0; x < CPT; ++x)
+        for (int x = 0; x < CPT; ++x)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const float2 f = unpack2(acc[x][i]);
-          val[x][i] = f.x + f.y;
+          for (int i = 0; i < 4; ++i) {
+            const float2 f = unpack2(acc[x][i]);
+            val[x][i] = f.x + f.y;
+          }
+#pragma unroll
+        for (int o = TPC >> 1, m = CPT; o > 0; o >>= 1) {
+          if (m > 1) {                     // halve the columns: keep those of this thread's half, send the others
+            const bool up = t & o;
+#pragma unroll
+            for (int y = 0; y < m / 2; ++y)
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                const float send = up ? val[y][i] : val[y + m / 2][i], keep = up ? val[y + m / 2][i] : val[y][i];
+                val[y][i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+              }
+            m >>= 1;
+          } else {
+#pragma unroll
+            for (int i = 0; i < 4; ++i) val[0][i] += __shfl_xor_sync(0xffffffffu, val[0][i], o);
+          }
         }
-#pragma unroll
-      for (int o = TPC >> 1, m = CPT; o > 0; o >>= 1) {
-        if (m > 1) {                     // halve the columns: keep those of this thread's half, send the others
-          const bool up = t & o;
-#pragma unroll
-          for (int y = 0; y < m / 2; ++y)
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-              const float send = up ? val[y][i] : val[y + m / 2][i], keep = up ? val[y + m / 2][i] : val[y][i];
-              val[y][i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-            }
-          m >>= 1;
-        } else {
-#pragma unroll
-          for (int i = 0; i < 4; ++i) val[0][i] += __shfl_xor_sync(0xffffffffu, val[0][i], o);
+        if (writer) {
+          const float4* pp = reinterpret_cast<const float4*>(sp + r * 4);
+          const float4 p0 = pp[0], p1 = pp[1], p2 = pp[2];                   // (0,0) (1,0) (1,1) (2,0) | (2,1) (2,2) (3,0) (3,1) | (3,2) (3,3)
+          const float* vr = sv + r * cols + my_cl;
+          const float v0 = vr[0], v1 = vr[cols], v2 = vr[2 * cols], v3 = vr[3 * cols];
+          float* op = orow + (long long)(c * GS_CHUNK + r) * ostep;
+          op[0] = fmaf(p0.x, v0, val[0][0]);
+          if (r + 1 < n) op[ostep] = fmaf(p0.z, v1, fmaf(p0.y, v0, val[0][1]));
+          if (r + 2 < n) op[2 * ostep] = fmaf(p1.y, v2, fmaf(p1.x, v1, fmaf(p0.w, v0, val[0][2])));
+          if (r + 3 < n) op[3 * ostep] = fmaf(p2.y, v3, fmaf(p2.x, v2, fmaf(p1.w, v1, fmaf(p1.z, v0, val[0][3]))));
         }
-      }
-      if (writer) {
-        const float4* pp = reinterpret_cast<const float4*>(sp + r * 4);
-        const float4 p0 = pp[0], p1 = pp[1], p2 = pp[2];                   // (0,0) (1,0) (1,1) (2,0) | (2,1) (2,2) (3,0) (3,1) | (3,2) (3,3)
-        const float* vr = sv + r * cols + my_cl;
-        const float v0 = vr[0], v1 = vr[cols], v2 = vr[2 * cols], v3 = vr[3 * cols];
-        float* op = orow + (long long)(c * GS_CHUNK + r) * ostep;
-        op[0] = fmaf(p0.x, v0, val[0][0]);
-        if (r + 1 < n) op[ostep] = fmaf(p0.z, v1, fmaf(p0.y, v0, val[0][1]));
-        if (r + 2 < n) op[2 * ostep] = fmaf(p1.y, v2, fmaf(p1.x, v1, fmaf(p0.w, v0, val[0][2])));
-        if (r + 3 < n) op[3 * ostep] = fmaf(p2.y, v3, fmaf(p2.x, v2, fmaf(p1.w, v1, fmaf(p1.z, v0, val[0][3]))));
       }
     }
     __syncthreads();
@@ -488,13 +539,20 @@ static int launch_scan_tile(const GlaScanArgs& p, int B, cudaStream_t st) {
   int nw = 4;
   while (nw > 1 && nw / 2 * CPW >= 4 && (nw * CPW > p.Vp || (warps + nw - 1) / nw < 4 * sm_count() / 5)) nw >>= 1;
   if ((nw * CPW) % 4) return TFB_ERR_ARG;
-  static DeviceOnce once, once_first;
-  auto kern = gla_scan_kernel<EPT, TPC, CPT, false>, kern_first = gla_scan_kernel<EPT, TPC, CPT, true>;
-  if (int e = ensure_dyn_smem(once, kern, bytes(4))) return e;
-  if (int e = ensure_dyn_smem(once_first, kern_first, bytes(4))) return e;
+  static DeviceOnce once, once_first, once_second;
   const int cols = nw * CPW;
-  if (p.nseg > 1) launch_k(kern_first, dim3((p.V + cols - 1) / cols, p.H, B * (p.nseg - 1)), nw * 32, bytes(nw), st, p);
-  launch_k(kern, dim3((p.V + cols - 1) / cols, p.H, B * p.nseg), nw * 32, bytes(nw), st, p);
+  const unsigned gx = (p.V + cols - 1) / cols;
+  if (p.nseg == 1) {
+    auto kern = gla_scan_kernel<EPT, TPC, CPT, WHOLE>;
+    if (int e = ensure_dyn_smem(once, kern, bytes(4))) return e;
+    launch_k(kern, dim3(gx, p.H, B), nw * 32, bytes(nw), st, p);
+    return int(cudaGetLastError());
+  }
+  auto first = gla_scan_kernel<EPT, TPC, CPT, SEG_FIRST>, second = gla_scan_kernel<EPT, TPC, CPT, SEG_SECOND>;
+  if (int e = ensure_dyn_smem(once_first, first, bytes(4))) return e;
+  if (int e = ensure_dyn_smem(once_second, second, bytes(4))) return e;
+  launch_k(first, dim3(gx, p.H, B * (p.nseg - 1)), nw * 32, bytes(nw), st, p);
+  launch_k(second, dim3(gx, p.H, B * p.nseg), nw * 32, bytes(nw), st, p);
   return int(cudaGetLastError());
 }
 
@@ -735,7 +793,7 @@ TFB_API int tfb_retention_prep(const void* proj, long long ld, const float* head
 TFB_API int tfb_gla_scan_segments(int B, int S, int H, int D, int V) {
   using namespace tfb;
   if (B <= 0 || S <= 0 || H <= 0 || D <= 0 || V <= 0 || !padded_dim(D)) return 1;
-  const long long warps = scan_warps(B, H, padded_dim(D), V), want = 7ll * sm_count();
+  const long long warps = scan_warps(B, H, padded_dim(D), V), want = 6ll * sm_count();
   int n = 1;
   if (warps * 5 <= want * 2)
     while (n < 32 && warps * n < want && S / (2 * n) >= 256) n *= 2;

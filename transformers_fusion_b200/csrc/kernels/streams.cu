@@ -241,17 +241,15 @@ static int launch_streams(const StreamArgs& p, int n, cudaStream_t st) {
   return int(cudaGetLastError());
 }
 
-template <class T>
-static int launch_by_streams(const StreamArgs& p, int n, bool vec, cudaStream_t st) {
-  if (vec) {
-    switch (p.S) {
-      case 1: return launch_streams<T, 1, 4>(p, n, st);
-      case 2: return launch_streams<T, 2, 4>(p, n, st);
-      case 3: return launch_streams<T, 3, 4>(p, n, st);
-      case 4: return launch_streams<T, 4, 4>(p, n, st);
-    }
+template <class T, int VEC>
+static int launch_by_streams(const StreamArgs& p, int n, cudaStream_t st) {
+  switch (p.S) {
+    case 1: return launch_streams<T, 1, VEC>(p, n, st);
+    case 2: return launch_streams<T, 2, VEC>(p, n, st);
+    case 3: return launch_streams<T, 3, VEC>(p, n, st);
+    case 4: return launch_streams<T, 4, VEC>(p, n, st);
+    default: return launch_streams<T, 0, 1>(p, n, st);
   }
-  return launch_streams<T, 0, 1>(p, n, st);
 }
 
 }  // namespace tfb
@@ -267,10 +265,15 @@ TFB_API int tfb_stream_norm(const long long* ids, const void* table, long long l
     return TFB_ERR_ARG;
   if (S > MAX_STREAMS) return TFB_ERR_LIMIT;
   const StreamArgs p{ids, table, ld_table, scale, vocab, x, S, H, y, y2, ldy, ldy2, w_post, w_post2, share, mix, out, in, w, groups, a, lda, rows, eps};
-  const int bytes = f32 ? 16 : 8;
+  const int es = f32 ? 4 : 2;
   auto al = [](const void* q, int b) { return (reinterpret_cast<uintptr_t>(q) & (b - 1)) == 0; };
-  bool vec = H % 4 == 0 && H / groups % 4 == 0 && al(x, 16) && ldy % 4 == 0 && ldy2 % 4 == 0 && lda % 4 == 0 && ld_table % 4 == 0;
-  for (const void* q : {y, y2, w_post, w_post2, w, table, static_cast<const void*>(a)}) vec = vec && al(q, bytes);
+  auto ok = [&](int vec) {
+    bool v = H % vec == 0 && H / groups % vec == 0 && al(x, 16) && ldy % vec == 0 && ldy2 % vec == 0 && lda % vec == 0 && ld_table % vec == 0;
+    for (const void* q : {y, y2, w_post, w_post2, w, table, static_cast<const void*>(a)}) v = v && al(q, vec * es);
+    return v;
+  };
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  return f32 ? launch_by_streams<float>(p, n, vec, st) : launch_by_streams<__nv_bfloat16>(p, n, vec, st);
+  if (f32) return ok(4) ? launch_by_streams<float, 4>(p, n, st) : launch_streams<float, 0, 1>(p, n, st);
+  if (ok(8) && H > 512) return launch_by_streams<__nv_bfloat16, 8>(p, n, st);
+  return ok(4) ? launch_by_streams<__nv_bfloat16, 4>(p, n, st) : launch_streams<__nv_bfloat16, 0, 1>(p, n, st);
 }
